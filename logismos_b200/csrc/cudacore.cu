@@ -177,6 +177,15 @@ uint32_t lg_error_kind_from_raw(uint32_t code) {
 
 #include <atomic>
 #include <cstdlib>
+#include <string>
+
+// message of the last failure of the calling thread, shared by the executors and the loaders
+namespace lgm {
+static thread_local std::string g_last_error;
+void set_error(const std::string& s) { g_last_error = s; }
+}  // namespace lgm
+extern "C" const char* lg_last_error(void) { return lgm::g_last_error.c_str(); }
+
 namespace lg {
 static std::atomic<int> g_deterministic{-1};
 bool deterministic() {

@@ -29,6 +29,7 @@
 #include "logismos_kernels.h"
 #include "logismos_model.h"
 #include "model_util.h"
+#include "step_batch.h"
 
 namespace {
 
@@ -41,7 +42,7 @@ struct HLayer {
 };
 
 constexpr int kChunkTokens = 512;
-constexpr int kBlock = 16;
+constexpr int kBlock = kKvBlock;
 constexpr int kGdnDim = 128;
 
 struct Hybrid {
@@ -62,22 +63,15 @@ struct Hybrid {
   Buf gdn_scratch;  // per (chunk, head) intermediates of the chunk-parallel recurrence (two-launch form)
   Buf gdn_pairs;    // arrival counters of the fused decode kernel's CTA pairs, all zero between launches
   Buf ids, pos, slots, cu_all, cu_prefill, last_idx, dec_ctx, dec_tables, dec_chunks, dec_scratch, attn_ws, state_slots, fresh, pre_kv;
-  uint8_t* pinned = nullptr;
-  size_t pinned_bytes = 0;
+  StepBatch batch;  // the last step (kept for replay and diagnostics)
   cudaStream_t stream = nullptr;
   std::mutex mu;
   int T = 0, n_dec = 0, n_pre = 0, n_seqs = 0, max_pre_len = 0, total_chunks = 0, chunk_tokens = kChunkTokens, launches = 0, logits_f32 = 0;
-  std::vector<int> order;
   size_t max_chunks = 0;
   // the fused int4 linears rely on `accws` being all zero between calls, which their finishing kernels
   // restore; a step that failed part-way may have left partial sums there, so the next one clears it
   bool acc_dirty = false;
   size_t accws_bytes = 0;
-  // prefill chunks that continue cached sequences: runs of prefill sequences whose keys fit the gather
-  // workspace together (one gather + attention launch pair per run)
-  struct PrefixRun { int s0, s1, total_kv, max_q, max_kv; };
-  std::vector<PrefixRun> prefix_runs;
-  bool pre_has_prefix = false;
   size_t prefix_cap_tokens = 0;
 };
 
@@ -145,11 +139,11 @@ uint32_t run_device(Hybrid* m, cudaStream_t s) {
                                                            c.n_heads, c.n_kv_heads, D, s), "paged_attention_decode");
         m->launches += 2;
       }
-      if (m->n_pre > 0 && m->pre_has_prefix) {
+      if (m->n_pre > 0 && m->batch.has_prefix) {
         // some chunk continues a cached sequence: keys and values come from the cache (the chunk's own rows
         // were stored above), gathered per run of sequences into attn_ws
         const int32_t* tabs = (const int32_t*)m->dec_tables.p + (size_t)m->n_dec * c.max_blocks_per_seq;
-        for (const Hybrid::PrefixRun& r : m->prefix_runs) {
+        for (const PrefixRun& r : m->batch.runs) {
           LG_TRY(logismos_launch_paged_prefix_attention_tc_bf16(
                      p16 + (size_t)m->n_dec * AN, AN, (const int32_t*)m->cu_prefill.p + r.s0, (const int32_t*)m->pre_kv.p + r.s0,
                      L.kpool.p, L.vpool.p, tabs + (size_t)r.s0 * c.max_blocks_per_seq, c.max_blocks_per_seq, c.n_pool_blocks,
@@ -255,7 +249,7 @@ uint32_t read_rows_bf16(Hybrid* m, const Buf& src, int n_seqs, size_t width, flo
   for (int k = 0; k < n_seqs; ++k)
     for (size_t j = 0; j < width; ++j) {
       const uint32_t u = (uint32_t)tmp[(size_t)k * width + j] << 16;
-      std::memcpy(&host_out[(size_t)m->order[k] * width + j], &u, 4);
+      std::memcpy(&host_out[(size_t)m->batch.order[k] * width + j], &u, 4);
     }
   return LG_EMB_OK;
 }
@@ -359,8 +353,11 @@ uint32_t lg_hybrid_create(int32_t device, const lg_hybrid_config_t* cfg, const l
   m->accws_bytes = (size_t)kFusedDequantMaxRows * acc_n * 4;
   ok = ok && cudaMemset(m->accws.p, 0, m->accws_bytes) == cudaSuccess;
   ok = ok && cudaMemset(m->gdn_pairs.p, 0, S * GH * 4) == cudaSuccess;
-  m->pinned_bytes = T * 16 + (S + 1) * 4 * 4 + S * MB * 4 + S * 4 + S * 4 + S * 4 + S + 64;
-  ok = ok && cudaMallocHost((void**)&m->pinned, m->pinned_bytes) == cudaSuccess;
+  StepLimits lim;
+  lim.max_pos = c.max_pos; lim.max_blocks_per_seq = c.max_blocks_per_seq; lim.n_pool_blocks = c.n_pool_blocks;
+  lim.max_step_tokens = c.max_step_tokens; lim.max_step_seqs = c.max_step_seqs; lim.n_state_slots = c.n_state_slots;
+  lim.prefix_cap_tokens = m->prefix_cap_tokens;
+  ok = ok && m->batch.alloc(lim);
   ok = ok && cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking) == cudaSuccess;
   if (!ok) {
     set_error(std::string("lg_hybrid_create: missing weights, or allocation or upload failed: ") + cudaGetErrorString(cudaGetLastError()));
@@ -386,7 +383,7 @@ void lg_hybrid_destroy(void* model) {
                  &L.wdown.scales, &L.w_in.dense, &L.w_out.dense, &L.wgu.dense, &L.wdown.dense};
     for (Buf* b : lb) b->release();
   }
-  if (m->pinned) cudaFreeHost(m->pinned);
+  m->batch.release();
   if (m->stream) cudaStreamDestroy(m->stream);
   delete m;
 }
@@ -396,119 +393,42 @@ uint32_t lg_hybrid_step(void* model, const uint32_t* host_ids, const int32_t* ca
   Hybrid* m = static_cast<Hybrid*>(model);
   if (!m) { set_error("lg_hybrid_step: null model"); return LG_EMB_COMPUTE; }
   const lg_hybrid_config_t& c = m->cfg;
-  if (n_seqs <= 0 || n_seqs > c.max_step_seqs || !host_ids || !cached || !newl || !tables || !state_slots || !next_tokens) {
-    set_error("lg_hybrid_step: bad arguments or too many sequences for the workspace");
-    return LG_EMB_COMPUTE;
-  }
+  if (!next_tokens) { set_error("lg_hybrid_step: null argument"); return LG_EMB_COMPUTE; }
   std::lock_guard<std::mutex> lock(m->mu);
   if (cudaSetDevice(m->device) != cudaSuccess) { set_error("cudaSetDevice failed"); return LG_EMB_COMPUTE; }
   const int MB = c.max_blocks_per_seq;
-  std::vector<int> order;
-  std::vector<int64_t> src_off(n_seqs);
-  std::vector<uint8_t> slot_used((size_t)c.n_state_slots, 0);
-  int64_t off = 0, total = 0;
-  for (int i = 0; i < n_seqs; ++i) {
-    if (newl[i] <= 0 || cached[i] < 0) { set_error("lg_hybrid_step: every sequence needs >= 1 new token"); return LG_EMB_COMPUTE; }
-    if ((int64_t)cached[i] + newl[i] > c.max_pos || (int64_t)cached[i] + newl[i] > (int64_t)MB * kBlock) {
-      set_error("lg_hybrid_step: sequence exceeds max_pos or its block table");
-      return LG_EMB_INPUT_TOO_LONG;
-    }
-    if (state_slots[i] < 0 || state_slots[i] >= c.n_state_slots || slot_used[state_slots[i]]) {
-      set_error("lg_hybrid_step: state slot out of range or used twice in one step");
-      return LG_EMB_COMPUTE;
-    }
-    slot_used[state_slots[i]] = 1;
-    src_off[i] = off;
-    off += newl[i];
-    total += newl[i];
-  }
-  if (total > c.max_step_tokens) { set_error("lg_hybrid_step: step exceeds max_step_tokens"); return LG_EMB_COMPUTE; }
-  for (int i = 0; i < n_seqs; ++i) if (newl[i] == 1) order.push_back(i);
-  const int n_dec = (int)order.size();
-  for (int i = 0; i < n_seqs; ++i) if (newl[i] > 1) order.push_back(i);
-  const int n_pre = n_seqs - n_dec;
-  uint8_t* pp = m->pinned;
-  uint32_t* h_ids = (uint32_t*)pp; pp += (size_t)total * 4;
-  int32_t* h_pos = (int32_t*)pp; pp += (size_t)total * 4;
-  int64_t* h_slots = (int64_t*)pp; pp += (size_t)total * 8;
-  int32_t* h_cu = (int32_t*)pp; pp += (size_t)(n_seqs + 1) * 4;
-  int32_t* h_cu_pre = (int32_t*)pp; pp += (size_t)(n_seqs + 1) * 4;
-  int32_t* h_last = (int32_t*)pp; pp += (size_t)(n_seqs + 1) * 4;
-  int32_t* h_chunks = (int32_t*)pp; pp += (size_t)(n_seqs + 1) * 4;
-  int32_t* h_tables = (int32_t*)pp; pp += (size_t)n_seqs * MB * 4;
-  int32_t* h_ctx = (int32_t*)pp; pp += (size_t)n_seqs * 4;
-  int32_t* h_state = (int32_t*)pp; pp += (size_t)n_seqs * 4;
-  int32_t* h_prekv = (int32_t*)pp; pp += (size_t)n_seqs * 4;
-  uint8_t* h_fresh = pp;
-  std::vector<int32_t> o_cached(n_seqs), o_new(n_seqs), o_seqids((size_t)total);
-  int64_t t = 0;
-  for (int s = 0; s < n_seqs; ++s) {
-    const int i = order[s];
-    o_cached[s] = cached[i];
-    o_new[s] = newl[i];
-    h_state[s] = state_slots[i];
-    h_fresh[s] = cached[i] == 0 ? 1 : 0;
-    std::memcpy(h_tables + (size_t)s * MB, tables + (size_t)i * MB, (size_t)MB * 4);
-    std::memcpy(h_ids + t, host_ids + src_off[i], (size_t)newl[i] * 4);
-    t += newl[i];
-  }
-  const int64_t built = logismos_build_packing(o_cached.data(), o_new.data(), n_seqs, h_tables, MB, kBlock, c.n_pool_blocks, h_cu,
-                                               h_pos, h_slots, o_seqids.data());
-  if (built != total) { set_error("lg_hybrid_step: a block table entry is missing or outside the pool"); return LG_EMB_COMPUTE; }
-  int max_pre = 0;
-  bool has_prefix = false;
-  h_cu_pre[0] = 0;
-  for (int s = 0; s < n_seqs; ++s) {
-    h_last[s] = h_cu[s + 1] - 1;
-    if (s < n_dec) h_ctx[s] = o_cached[s] + 1;
-    else {
-      h_cu_pre[s - n_dec + 1] = h_cu[s + 1] - n_dec;
-      h_prekv[s - n_dec] = o_cached[s] + o_new[s];
-      if (o_cached[s] > 0) has_prefix = true;
-      if (o_new[s] > max_pre) max_pre = o_new[s];
-    }
-  }
-  std::vector<Hybrid::PrefixRun> runs;
-  if (has_prefix) {
-    Hybrid::PrefixRun r{0, 0, 0, 0, 0};
-    for (int k = 0; k < n_pre; ++k) {
-      const int kv = h_prekv[k], q = o_new[n_dec + k];
-      if (r.s1 > r.s0 && (size_t)r.total_kv + kv > m->prefix_cap_tokens) { runs.push_back(r); r = Hybrid::PrefixRun{k, k, 0, 0, 0}; }
-      r.s1 = k + 1; r.total_kv += kv;
-      if (q > r.max_q) r.max_q = q;
-      if (kv > r.max_kv) r.max_kv = kv;
-    }
-    runs.push_back(r);
-  }
-  m->chunk_tokens = n_dec > 0 ? logismos_pick_decode_chunk(h_ctx, n_dec, m->cfg.n_kv_heads, m->cfg.attn_head_dim) : kChunkTokens;
-  const int total_chunks = n_dec > 0 ? logismos_build_decode_chunks(h_ctx, n_dec, m->chunk_tokens, h_chunks) : 0;
+  StepBatch& B = m->batch;
+  m->T = 0;  // nothing to replay until this step is on the device
+  if (uint32_t rc = B.build("lg_hybrid_step", host_ids, cached, newl, n_seqs, tables, state_slots, false)) return rc;
+  const int n_dec = B.n_dec, n_pre = B.n_pre;
+  const bool has_prefix = B.has_prefix;
+  const size_t total = (size_t)B.T;
+  m->chunk_tokens = n_dec > 0 ? logismos_pick_decode_chunk(B.ctx, n_dec, m->cfg.n_kv_heads, m->cfg.attn_head_dim) : kChunkTokens;
+  const int total_chunks = n_dec > 0 ? logismos_build_decode_chunks(B.ctx, n_dec, m->chunk_tokens, B.chunks) : 0;
   if (total_chunks < 0 || (size_t)total_chunks > m->max_chunks) { set_error("lg_hybrid_step: decode chunk count exceeds the scratch"); return LG_EMB_COMPUTE; }
-  m->T = (int)total; m->n_dec = n_dec; m->n_pre = n_pre; m->n_seqs = n_seqs; m->max_pre_len = max_pre; m->total_chunks = total_chunks;
-  m->order = order;
-  m->pre_has_prefix = has_prefix;
-  m->prefix_runs = runs;
+  m->T = B.T; m->n_dec = n_dec; m->n_pre = n_pre; m->n_seqs = n_seqs; m->max_pre_len = B.max_pre_len; m->total_chunks = total_chunks;
   cudaStream_t s = m->stream;
   LG_TRY(cudaMemsetAsync(m->status.p, 0, 4, s), "clear status");  // the status word describes this step only
-  LG_TRY(cudaMemcpyAsync(m->ids.p, h_ids, (size_t)total * 4, cudaMemcpyHostToDevice, s), "H2D ids");
-  LG_TRY(cudaMemcpyAsync(m->pos.p, h_pos, (size_t)total * 4, cudaMemcpyHostToDevice, s), "H2D positions");
-  LG_TRY(cudaMemcpyAsync(m->slots.p, h_slots, (size_t)total * 8, cudaMemcpyHostToDevice, s), "H2D slots");
-  LG_TRY(cudaMemcpyAsync(m->cu_all.p, h_cu, (size_t)(n_seqs + 1) * 4, cudaMemcpyHostToDevice, s), "H2D cu_seqlens");
-  LG_TRY(cudaMemcpyAsync(m->cu_prefill.p, h_cu_pre, (size_t)(n_pre + 1) * 4, cudaMemcpyHostToDevice, s), "H2D prefill cu_seqlens");
-  LG_TRY(cudaMemcpyAsync(m->last_idx.p, h_last, (size_t)n_seqs * 4, cudaMemcpyHostToDevice, s), "H2D last rows");
-  LG_TRY(cudaMemcpyAsync(m->state_slots.p, h_state, (size_t)n_seqs * 4, cudaMemcpyHostToDevice, s), "H2D state slots");
-  LG_TRY(cudaMemcpyAsync(m->fresh.p, h_fresh, (size_t)n_seqs, cudaMemcpyHostToDevice, s), "H2D fresh flags");
+  LG_TRY(cudaMemcpyAsync(m->ids.p, B.ids, (size_t)total * 4, cudaMemcpyHostToDevice, s), "H2D ids");
+  LG_TRY(cudaMemcpyAsync(m->pos.p, B.pos, (size_t)total * 4, cudaMemcpyHostToDevice, s), "H2D positions");
+  LG_TRY(cudaMemcpyAsync(m->slots.p, B.slots, (size_t)total * 8, cudaMemcpyHostToDevice, s), "H2D slots");
+  LG_TRY(cudaMemcpyAsync(m->cu_all.p, B.cu, (size_t)(n_seqs + 1) * 4, cudaMemcpyHostToDevice, s), "H2D cu_seqlens");
+  LG_TRY(cudaMemcpyAsync(m->cu_prefill.p, B.cu_pre, (size_t)(n_pre + 1) * 4, cudaMemcpyHostToDevice, s), "H2D prefill cu_seqlens");
+  LG_TRY(cudaMemcpyAsync(m->last_idx.p, B.last, (size_t)n_seqs * 4, cudaMemcpyHostToDevice, s), "H2D last rows");
+  LG_TRY(cudaMemcpyAsync(m->state_slots.p, B.state, (size_t)n_seqs * 4, cudaMemcpyHostToDevice, s), "H2D state slots");
+  LG_TRY(cudaMemcpyAsync(m->fresh.p, B.fresh, (size_t)n_seqs, cudaMemcpyHostToDevice, s), "H2D fresh flags");
   if (n_dec > 0) {
-    LG_TRY(cudaMemcpyAsync(m->dec_ctx.p, h_ctx, (size_t)n_dec * 4, cudaMemcpyHostToDevice, s), "H2D context lens");
-    LG_TRY(cudaMemcpyAsync(m->dec_chunks.p, h_chunks, (size_t)(n_dec + 1) * 4, cudaMemcpyHostToDevice, s), "H2D chunk offsets");
+    LG_TRY(cudaMemcpyAsync(m->dec_ctx.p, B.ctx, (size_t)n_dec * 4, cudaMemcpyHostToDevice, s), "H2D context lens");
+    LG_TRY(cudaMemcpyAsync(m->dec_chunks.p, B.chunks, (size_t)(n_dec + 1) * 4, cudaMemcpyHostToDevice, s), "H2D chunk offsets");
   }
   if (n_dec > 0 || has_prefix)  // block tables in packed order: decode rows first, prefill rows after them
-    LG_TRY(cudaMemcpyAsync(m->dec_tables.p, h_tables, (size_t)(has_prefix ? n_seqs : n_dec) * MB * 4, cudaMemcpyHostToDevice, s), "H2D block tables");
-  if (has_prefix) LG_TRY(cudaMemcpyAsync(m->pre_kv.p, h_prekv, (size_t)n_pre * 4, cudaMemcpyHostToDevice, s), "H2D prefill key counts");
+    LG_TRY(cudaMemcpyAsync(m->dec_tables.p, B.tables, (size_t)(has_prefix ? n_seqs : n_dec) * MB * 4, cudaMemcpyHostToDevice, s), "H2D block tables");
+  if (has_prefix) LG_TRY(cudaMemcpyAsync(m->pre_kv.p, B.pre_kv, (size_t)n_pre * 4, cudaMemcpyHostToDevice, s), "H2D prefill key counts");
   if (uint32_t rc = run_device(m, s)) { m->acc_dirty = true; return rc; }
   std::vector<uint32_t> toks(n_seqs);
   LG_TRY(cudaMemcpyAsync(toks.data(), m->tokens.p, (size_t)n_seqs * 4, cudaMemcpyDeviceToHost, s), "D2H tokens");
   LG_TRY(cudaStreamSynchronize(s), "stream synchronize");
-  for (int k = 0; k < n_seqs; ++k) next_tokens[order[k]] = toks[k];
+  for (int k = 0; k < n_seqs; ++k) next_tokens[B.order[k]] = toks[k];
   if (const int dev_status = lg_hybrid_device_status(m)) {
     m->acc_dirty = true;
     char buf[160];
@@ -563,7 +483,7 @@ uint32_t lg_hybrid_last_logits(void* model, int32_t n_seqs, float* host_out) {
   std::vector<float> tmp((size_t)n_seqs * V);
   LG_TRY(cudaDeviceSynchronize(), "device synchronize");
   LG_TRY(cudaMemcpy(tmp.data(), m->logits.p, tmp.size() * 4, cudaMemcpyDeviceToHost), "D2H logits");
-  for (int k = 0; k < n_seqs; ++k) std::memcpy(host_out + (size_t)m->order[k] * V, tmp.data() + (size_t)k * V, V * 4);
+  for (int k = 0; k < n_seqs; ++k) std::memcpy(host_out + (size_t)m->batch.order[k] * V, tmp.data() + (size_t)k * V, V * 4);
   return LG_EMB_OK;
 }
 

@@ -19,19 +19,11 @@
 #include "logismos_kernels.h"
 #include "logismos_model.h"
 
-namespace {
-
-thread_local std::string g_last_error;
-
-void set_error(const std::string& s) { g_last_error = s; }
-}  // namespace
-
-// shared with the other executors of the library
-namespace lgm {
-void set_error(const std::string& s) { g_last_error = s; }
-}  // namespace lgm
+namespace lgm { void set_error(const std::string& s); }
 
 namespace {
+
+using lgm::set_error;
 
 inline uint16_t f32_to_bf16(float f) {
   uint32_t u;
@@ -146,7 +138,6 @@ uint32_t forward_device(Stella* m, const void* ids, const void* cu, const void* 
 
 extern "C" {
 
-const char* lg_last_error(void) { return g_last_error.c_str(); }
 
 uint32_t lg_stella_create(int32_t device, const lg_stella_config_t* cfg, const lg_stella_weights_t* w, void** model) {
   if (!cfg || !w || !model) { set_error("null argument"); return LG_EMB_COMPUTE; }

@@ -1,5 +1,5 @@
 """Continuous-batching decoder step (int4 group-32 weights, paged KV cache) over the C ABI
-(``lg_decoder_*``), plus the small host-side block allocator a caller needs to drive it.
+(``lg_decoder_*``).
 
 The reference has no decoder executor and no scheduler (crates/decoders, crates/sched are empty
 scaffolds); the semantics are "a packed step equals running every sequence alone".
@@ -7,11 +7,12 @@ scaffolds); the semantics are "a packed step equals running every sequence alone
 from __future__ import annotations
 
 import ctypes as C
-from typing import Dict, List, Sequence
+from typing import Sequence
 
 import numpy as np
 
 from ._lib import lib
+from .cache import BlockAllocator  # noqa: F401  (callers drive the executor with it)
 from .embed import ComputeError, InputTooLong
 
 _fp = C.POINTER(C.c_float)
@@ -47,32 +48,6 @@ def _q(pair):
     codes, scales = pair
     assert codes.dtype == np.uint8 and codes.flags["C_CONTIGUOUS"] and scales.flags["C_CONTIGUOUS"] and scales.itemsize == 2
     return _Q(codes.ctypes.data_as(_u8), scales.ctypes.data_as(_u16))
-
-
-class BlockAllocator:
-    """Hands out KV blocks of 16 tokens from a fixed pool; one table row per sequence."""
-
-    def __init__(self, n_pool_blocks: int, max_blocks_per_seq: int, seed: int = 0):
-        rng = np.random.default_rng(seed)
-        self.free: List[int] = rng.permutation(n_pool_blocks).tolist()
-        self.max_blocks = max_blocks_per_seq
-        self.tables: Dict[int, List[int]] = {}
-
-    def ensure(self, seq_id: int, n_tokens: int) -> np.ndarray:
-        t = self.tables.setdefault(seq_id, [])
-        need = -(-n_tokens // 16)
-        if need > self.max_blocks:
-            raise ValueError("sequence exceeds max_blocks_per_seq")
-        while len(t) < need:
-            if not self.free:
-                raise MemoryError("KV pool exhausted")
-            t.append(self.free.pop())
-        row = np.full(self.max_blocks, -1, np.int32)
-        row[: len(t)] = t
-        return row
-
-    def release(self, seq_id: int):
-        self.free.extend(self.tables.pop(seq_id, []))
 
 
 class DecoderModel:

@@ -1,6 +1,5 @@
 """Hybrid decoder step (gated-delta-rule linear-attention layers interleaved with gated
-full-attention layers, int4 group-32 weights) over the C ABI (``lg_hybrid_*``), with the host-side
-slot allocator for the recurrent states.
+full-attention layers, int4 group-32 weights) over the C ABI (``lg_hybrid_*``).
 
 The reference has no decoder model (crates/decoders is an empty scaffold); the recurrence is
 crates/kernels/src/gated_delta_rule/cpu.rs:92-182 and the contract is "a packed step equals running
@@ -9,11 +8,12 @@ every sequence alone".
 from __future__ import annotations
 
 import ctypes as C
-from typing import Dict, List, Sequence
+from typing import Sequence
 
 import numpy as np
 
 from ._lib import lib
+from .cache import SlotAllocator  # noqa: F401  (callers drive the executor with it)
 from .decoder import _Q, _f, _fp, _q
 from .embed import ComputeError, InputTooLong
 
@@ -40,26 +40,6 @@ class _Weights(C.Structure):
 
 def is_full_attention(layer: int, interval: int) -> bool:
     return (layer + 1) % interval == 0
-
-
-class SlotAllocator:
-    """Recurrent-state slots: one per live sequence."""
-
-    def __init__(self, n_slots: int):
-        self.free: List[int] = list(range(n_slots - 1, -1, -1))
-        self.slots: Dict[int, int] = {}
-
-    def get(self, seq_id: int) -> int:
-        if seq_id not in self.slots:
-            if not self.free:
-                raise MemoryError("state slots exhausted")
-            self.slots[seq_id] = self.free.pop()
-        return self.slots[seq_id]
-
-    def release(self, seq_id: int):
-        s = self.slots.pop(seq_id, None)
-        if s is not None:
-            self.free.append(s)
 
 
 class HybridModel:

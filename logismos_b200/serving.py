@@ -19,7 +19,7 @@ from typing import Deque, Dict, List, Optional
 
 import numpy as np
 
-BLOCK = 16
+from .cache import BlockAllocator, SlotAllocator, blocks_for
 
 
 @dataclass
@@ -70,19 +70,29 @@ class Scheduler:
         self.prefill_budget = prefill_token_budget or max_step_tokens
         self.chunked = chunked_prefill
         self.prefilling: Dict[int, Request] = {}   # admitted, prompt not yet fully fed (insertion order = age)
-        self.free_blocks: List[int] = list(range(n_pool_blocks - 1, -1, -1))
-        self.free_slots: List[int] = list(range(n_state_slots - 1, -1, -1))
+        self.blocks = BlockAllocator(n_pool_blocks, max_blocks_per_seq, seed=None)
+        self.slots = SlotAllocator(n_state_slots)
         self.waiting: Deque[Request] = deque()
         self.running: Dict[int, Request] = {}
-        self.tables: Dict[int, np.ndarray] = {}
-        self.slot_of: Dict[int, int] = {}
         self.cached: Dict[int, int] = {}
         self.done: List[Request] = []
         self.generated = 0
         self.prefilled = 0
 
+    @property
+    def free_blocks(self) -> List[int]:
+        return self.blocks.free
+
+    @property
+    def free_slots(self) -> List[int]:
+        return self.slots.free
+
+    @property
+    def tables(self) -> Dict[int, np.ndarray]:
+        return {rid: self.blocks.row(rid) for rid in self.blocks.tables}
+
     def add(self, req: Request):
-        need = -(-(len(req.prompt) + req.max_new) // BLOCK)
+        need = blocks_for(len(req.prompt) + req.max_new)
         if need > self.max_blocks or len(req.prompt) < 1 or req.max_new < 1 or (not self.chunked and len(req.prompt) > self.max_step_tokens):
             raise ValueError(f"request {req.rid} cannot be served: {len(req.prompt)} + {req.max_new} tokens")
         self.waiting.append(req)
@@ -121,7 +131,7 @@ class Scheduler:
         while self.waiting and self.waiting[0].arrival <= now and len(rids) < self.max_step_seqs:
             req = self.waiting[0]
             p = len(req.prompt)
-            need = -(-(p + req.max_new) // BLOCK)
+            need = blocks_for(p + req.max_new)
             if not self.free_slots or need > len(self.free_blocks):
                 break
             if self.chunked:
@@ -133,9 +143,9 @@ class Scheduler:
                 if tokens + p > self.max_step_tokens or (pre_tokens > 0 and pre_tokens + p > self.prefill_budget):
                     break
             self.waiting.popleft()
-            row = np.full(self.max_blocks, -1, np.int32)
-            row[:need] = [self.free_blocks.pop() for _ in range(need)]
-            self.tables[req.rid], self.slot_of[req.rid], self.cached[req.rid] = row, self.free_slots.pop(), 0
+            self.blocks.ensure(req.rid, p + req.max_new)
+            self.slots.get(req.rid)
+            self.cached[req.rid] = 0
             self.running[req.rid] = req
             if n < p:
                 self.prefilling[req.rid] = req
@@ -144,7 +154,7 @@ class Scheduler:
         if not rids:
             return None
         return StepPlan(np.concatenate(ids).astype(np.uint32), np.asarray(cached, np.int32), np.asarray(new, np.int32),
-                        np.stack([self.tables[r] for r in rids]), np.asarray([self.slot_of[r] for r in rids], np.int32), rids,
+                        np.stack([self.blocks.row(r) for r in rids]), np.asarray([self.slots.get(r) for r in rids], np.int32), rids,
                         n_decode, pre_tokens, np.asarray(emits, bool))
 
     def commit(self, plan: StepPlan, next_tokens, now: float):
@@ -162,9 +172,8 @@ class Scheduler:
                 req.first_token_at = now
             if len(req.output) >= req.max_new:
                 req.finished_at = now
-                row = self.tables.pop(rid)
-                self.free_blocks.extend(int(b) for b in row[row >= 0][::-1])
-                self.free_slots.append(self.slot_of.pop(rid))
+                self.blocks.release(rid)
+                self.slots.release(rid)
                 del self.cached[rid], self.running[rid]
                 self.done.append(req)
         self.prefilled += plan.n_prefill_tokens
