@@ -107,6 +107,34 @@ uint32_t logismos_launch_linear_t_bf16(const void* a_bf16, const void* w_bf16,
                                        const void* bias_f32, void* out, int32_t m, int32_t n,
                                        int32_t k, int32_t lda, int32_t ldc, int32_t epilogue,
                                        void* status_i32, void* stream);
+/* The same launch with the epilogues that take constants (the three epilogues above ignore them):
+ *   LG_EPI_F32        out f32 [m, n]       = acc + bias, then p0 tanh(. / p0) when p0 > 0 (soft cap);
+ *                     any n, ldc >= n
+ *   LG_EPI_GLU_CLAMP  out bf16 [m, n / 2]  = g sigmoid(alpha g) (u + shift) with g = min(gate, limit), u =
+ *                     clamp(up, -limit, limit), alpha = p0, limit = p1, shift = p2; rows (and bias)
+ *                     interleaved as for LG_EPI_SWIGLU, n % 64 == 0 */
+enum { LG_EPI_F32 = 3, LG_EPI_GLU_CLAMP = 4 };
+uint32_t logismos_launch_linear_t_act_bf16(const void* a_bf16, const void* w_bf16, const void* bias_f32,
+                                           void* out, int32_t m, int32_t n, int32_t k, int32_t lda,
+                                           int32_t ldc, int32_t epilogue, float p0, float p1, float p2,
+                                           void* status_i32, void* stream);
+/* The same contract for few rows (decode steps): the weights are streamed once and shared by up to 64
+ * rows, the reduction order is fixed. W must be static (it is requested before the preceding kernel has
+ * finished: LG_EPI_STATIC_W is implied). batch independent products are done in one launch, entry b at
+ * a + b * a_stride, w + b * w_stride, out + b * out_stride (elements). All five epilogues; k % 32 == 0,
+ * lda % 8 == 0, strides of a and w multiples of 8; a and w 16-byte aligned. */
+uint32_t logismos_launch_linear_small_bf16(const void* a_bf16, const void* w_bf16, const void* bias_f32,
+                                           void* out, int32_t m, int32_t n, int32_t k, int32_t lda,
+                                           int32_t ldc, int32_t batch, int64_t a_stride, int64_t w_stride,
+                                           int64_t out_stride, int32_t epilogue, float p0, float p1,
+                                           float p2, void* stream);
+/* The batched contract with fp32 activations and outputs, true fp32 products and sums over the bf16
+ * weights (which fp32 represents exactly). Epilogues LG_EPI_F32, LG_EPI_RESID_F32, LG_EPI_GLU_CLAMP (fp32
+ * out); k % 16 == 0, lda % 4 == 0, strides of a and w multiples of 4. */
+uint32_t logismos_launch_linear_f32(const void* a_f32, const void* w_bf16, const void* bias_f32, void* out_f32,
+                                    int32_t m, int32_t n, int32_t k, int32_t lda, int32_t ldc, int32_t batch,
+                                    int64_t a_stride, int64_t w_stride, int64_t out_stride, int32_t epilogue,
+                                    float p0, float p1, float p2, void* stream);
 /* The same contract one thread per output, as the on-device correctness anchor (the role
  * matmul_naive.hip plays in the reference). LG_EPI_SWIGLU is not supported here. */
 uint32_t logismos_launch_linear_t_naive_bf16(const void* a_bf16, const void* w_bf16,
@@ -207,6 +235,19 @@ uint32_t logismos_launch_paged_prefix_attention_turbo3_bf16(
     int32_t n_pool_blocks, void* out_bf16, void* scratch, int32_t n_q_tokens, int32_t total_kv_tokens,
     int32_t n_seqs, int32_t max_q_len, int32_t max_kv_len, int32_t n_heads, int32_t n_kv_heads,
     int32_t head_dim, void* status, void* stream);
+
+/* Causal attention of query rows over keys and values given contiguously: q bf16 [n_q_tokens, q_row_stride]
+ * (head h at column h * head_dim), k bf16 [n_kv_rows, n_kv_heads * head_dim], v_t bf16 [n_kv_heads *
+ * head_dim, n_kv_rows] (transposed). Sequence s has the queries cu_seqlens_q[s] .. cu_seqlens_q[s+1] and the
+ * kv_lens[s] keys at rows / columns kv_start[s] .. (kv_start a multiple of 8; what lies between sequences
+ * must be finite); query i sees its first kv_lens[s] - new + i + 1 keys. Scores are scaled by `scale` (> 0).
+ * out bf16, rows out_row_stride apart. head_dim 64, 128 or 256; n_kv_rows % 8 == 0. One launch of the
+ * tcgen05 kernel above. status as there. */
+uint32_t logismos_launch_varlen_attention_kv_tc_bf16(
+    const void* q_bf16, int32_t q_row_stride, const void* cu_seqlens_q_i32, const void* kv_lens_i32,
+    const void* kv_start_i32, const void* k_bf16, const void* v_t_bf16, int32_t n_kv_rows, void* out_bf16,
+    int32_t out_row_stride, int32_t n_q_tokens, int32_t n_seqs, int32_t max_q_len, int32_t n_heads,
+    int32_t n_kv_heads, int32_t head_dim, float scale, void* status_i32, void* stream);
 
 /* mean_pool_masked -> l2_normalize -> linear_t(head) -> l2_normalize (cpu_f32 mod.rs:553-591 as
  * composed by StellaModel::encode_raw, crates/embed/src/stella.rs:231-246), mask all ones.
@@ -475,6 +516,79 @@ uint32_t logismos_launch_add_f32(void* x_f32, const void* d_f32, int64_t n, void
  * never selected. logits bf16 or f32 [rows, n]; out u32 [rows]. */
 uint32_t logismos_launch_greedy_argmax(const void* logits, int32_t logits_f32, void* out_u32,
                                        int32_t rows, int32_t n, void* stream);
+
+/* ====================================================================================
+ * Mechanisms of parallel-block decoders with latent attention (no reference counterpart: the reference has
+ * no decoder model). Rows of fp32 data are `ld` columns wide, a multiple of 4; columns n .. ld are
+ * padding and must hold zeros in weights, gains and filters.
+ * ==================================================================================== */
+
+/* Depth average and RMS norm: x = sum_{j < n_hist} coef[j] X_j, X_j f32 rows at hist + j * hist_stride
+ * (elements), h = x / sqrt(mean over n of x^2 + eps) * gain. Row r reads source row row_idx[r] (NULL: r;
+ * an index outside [0, n_src_rows) raises status to 1). Any of x (f32 [rows, ld]), inv_rms (f32 [rows]) and
+ * norm_out ([rows, ld], bf16 or with out_f32 f32; needs gain) may be NULL. ld <= 16384. */
+uint32_t logismos_launch_depth_mix_f32(const void* hist_f32, int64_t hist_stride, int32_t n_hist,
+                                       const void* coef_f32, const void* row_idx_i32, int32_t n_src_rows,
+                                       void* x_f32, void* inv_rms_f32, const void* gain_f32, void* norm_out,
+                                       int32_t out_f32, int32_t rows, int32_t n, int32_t ld, float eps,
+                                       void* status_i32, void* stream);
+/* Input convolution over a ragged batch: h = x * inv_rms * gain per row, o1 = h + sum_j w1[j] *
+ * h_(t - taps + 1 + j) and the same for o2 with w2 (o2 may be NULL; w1 / w2 NULL: no filter), causal inside
+ * each sequence. w f32 [taps, ld], taps 1..8. Row t belongs to sequence seq_ids[t], whose rows are
+ * cu_seqlens[s] .. cu_seqlens[s+1]. state f32 [n_slots, 2, taps - 1, ld]: the last taps - 1 rows h of a
+ * sequence in slot state_slots[s]; read from copy phase[s] (zeros when fresh[s]), the new state goes to copy
+ * 1 - phase[s]. o1, o2 bf16 or with out_f32 f32, [rows, ld]. */
+uint32_t logismos_launch_norm_conv(const void* x_f32, const void* inv_rms_f32, const void* gain_f32,
+                                   const void* w1_f32, const void* w2_f32, void* o1, void* o2, int32_t out_f32,
+                                   void* state_f32, const void* state_slots_i32, const void* fresh_u8,
+                                   const void* phase_u8, const void* seq_ids_i32, const void* cu_seqlens_i32,
+                                   int32_t rows, int32_t ld, int32_t taps, void* stream);
+/* Both of the above in one launch for a step whose sequences bring one token each (row = sequence). */
+uint32_t logismos_launch_depth_mix_conv_decode(const void* hist_f32, int64_t hist_stride, int32_t n_hist,
+                                               const void* coef_f32, void* x_f32, const void* gain_f32,
+                                               const void* w1_f32, const void* w2_f32, void* o1, void* o2,
+                                               int32_t out_f32, void* state_f32, const void* state_slots_i32,
+                                               const void* fresh_u8, const void* phase_u8, int32_t rows,
+                                               int32_t n, int32_t ld, float eps, int32_t taps, void* stream);
+
+/* Latent attention. A token's cache row is its normed key/value latent, c_width values: pool bf16 or f32
+ * [n_pool_blocks, 16, c_width].
+ * norm_store: raw f32 [rows, ld] holds the query latent in columns 0 .. q_width and the key/value latent in
+ * q_width .. q_width + c_width; both are RMS-normed (means over the first q_n and c_n columns) with their
+ * gains; the first goes to q_latent [rows, q_width], the second to the pool at slot_mapping[row] (a slot
+ * outside the pool is skipped and raises status to 1). is_f32 selects the type of both. */
+uint32_t logismos_launch_latent_norm_store(const void* raw_f32, int32_t ld, const void* gain_q_f32,
+                                           const void* gain_c_f32, void* q_latent, void* pool,
+                                           const void* slot_mapping_i64, int32_t rows, int32_t q_width,
+                                           int32_t q_n, int32_t c_width, int32_t c_n, float eps,
+                                           int64_t n_pool_slots, int32_t is_f32, void* status_i32, void* stream);
+/* The cached rows of whole sequences made contiguous: out bf16 [logismos_latent_gather_rows(total, n_seqs),
+ * width], sequence s at kv_start[s] (written, a multiple of 8), gaps zeroed. */
+int32_t logismos_latent_gather_rows(int32_t total_kv_tokens, int32_t n_seqs);
+uint32_t logismos_launch_latent_gather_bf16(const void* pool, const void* block_tables_i32, int32_t max_blocks,
+                                            int32_t n_pool_blocks, const void* kv_lens_i32, void* out,
+                                            void* kv_start_i32, int32_t total_kv_tokens, int32_t n_seqs,
+                                            int32_t max_kv_len, int32_t width, void* status_i32, void* stream);
+/* Decode in the latent space, one query row per sequence: out[r, h] = sum_j softmax_j(scale q[r, h] . c_j)
+ * c_j over the first context_lens[r] cached rows. q, out bf16 [rows, heads, rank]; rank % 64 == 0, rank <=
+ * 1024. chunk_offsets as for the paged decode kernel, with chunk_tokens % 64 == 0
+ * (logismos_pick_latent_chunk, whose choice leaves at most logismos_latent_max_chunks(rows) chunks). scratch:
+ * logismos_latent_decode_scratch_bytes(total_chunks, heads, rank). A second launch merges split contexts. */
+int32_t logismos_pick_latent_chunk(const int32_t* host_context_lens, int32_t n_seqs, int32_t heads);
+int32_t logismos_latent_max_chunks(int32_t max_rows);
+size_t logismos_latent_decode_scratch_bytes(int32_t total_chunks, int32_t heads, int32_t rank);
+uint32_t logismos_launch_latent_decode_bf16(const void* q_bf16, const void* pool_bf16, const void* block_tables_i32,
+                                            const void* context_lens_i32, const void* chunk_offsets_i32,
+                                            void* out_bf16, void* scratch, int32_t rows, int32_t total_chunks,
+                                            int32_t chunk_tokens, int32_t max_blocks, int32_t n_pool_blocks,
+                                            int32_t heads, int32_t rank, float scale, void* status_i32,
+                                            void* stream);
+/* The fp32 form for any rows of a step: row t of sequence seq_ids[t] sees keys 0 .. positions[t]. */
+uint32_t logismos_launch_latent_attention_f32(const void* q_f32, const void* pool_f32, const void* block_tables_i32,
+                                              const void* seq_ids_i32, const void* positions_i32, void* out_f32,
+                                              int32_t rows, int32_t max_blocks, int32_t n_pool_blocks,
+                                              int32_t heads, int32_t rank, float scale, void* status_i32,
+                                              void* stream);
 
 /* ====================================================================================
  * Sampling chain on the device: the logit processors and the multinomial sampler of

@@ -254,6 +254,72 @@ int32_t lg_hybrid_launches_last_step(const void* model);
 int32_t lg_hybrid_device_status(void* model);
 
 /* ====================================================================================
+ * Latent-attention decoder step: a stack of parallel blocks over a paged cache of latents. No reference
+ * counterpart; the contract is that of lg_decoder_step. Weights are bf16, dense.
+ *   h = rms_norm(x) * (norm_offset + w);  h1 = h + conv1(h), h2 = h + conv2(h)  (causal, depthwise, conv_taps)
+ *   X_(i+1) = x + attention(h1) + ff(h2);  x = sum_{j <= i+1} dwa_i[j] X_j  (X_0 = embedding)
+ *   attention: q = W_uq (rms_norm(W_dq h1) * g_q); c = rms_norm(W_dkv h1) * g_c (the cached latent);
+ *     per head k = W_uk c, v = W_uv c, scores (q . k) * scale, causal softmax; W_o over the heads
+ *   ff: g = min(W_gate h2 + b, limit), u = clamp(W_up h2 + b, +-limit); W_down (g sigmoid(alpha g) (u + shift)) + b
+ *   logits = cap tanh(head (rms_norm(x) * (norm_offset + w)) / cap)
+ * Sizes may differ from layer to layer. is_f32 != 0 computes everything in fp32 (activations, cache, products,
+ * sums; the bf16 weights are exact in fp32); otherwise activations and the cache are bf16 and the residual
+ * stream, norms, scores, softmax and convolution state fp32.
+ * ==================================================================================== */
+typedef struct lg_latent_layer_config {
+  int32_t heads, dim, vdim;     /* query/key and value dimensions per head, <= 256 */
+  int32_t q_rank, kv_rank;      /* latent sizes; kv_rank <= 1024 */
+  int32_t ff;                   /* 0: no feed-forward */
+  float scale, glu_limit;
+} lg_latent_layer_config_t;
+typedef struct lg_latent_config {
+  int32_t vocab, width, n_layers, conv_taps;
+  float rms_eps, norm_offset, glu_alpha, glu_shift;
+  float logit_softcap;          /* 0: none */
+  int32_t is_f32;
+  int32_t n_pool_blocks;        /* cache blocks of 16 tokens per layer */
+  int32_t max_blocks_per_seq, max_step_tokens, max_step_seqs;
+  int32_t n_state_slots;        /* convolution-state slots */
+  int32_t max_out_rows;         /* rows of logits per step (>= max_step_seqs for generation) */
+  const lg_latent_layer_config_t* layers;
+} lg_latent_config_t;
+/* bf16 values on the host, [out, in]; the feed-forward entries are NULL when ff == 0 */
+typedef struct lg_latent_layer_weights {
+  const void *norm1, *dq, *dq_norm, *uq, *dkv, *dkv_norm, *uk, *uv, *o;
+  const void *gate, *gate_b, *up, *up_b, *down, *down_b;
+  const void *conv1, *conv2;    /* [width, taps] */
+  const void *dwa;              /* [layer index + 2] */
+} lg_latent_layer_weights_t;
+typedef struct lg_latent_weights {
+  const void *embed, *final_norm, *head;
+  const lg_latent_layer_weights_t* layers;
+} lg_latent_weights_t;
+
+uint32_t lg_latent_create(int32_t device, const lg_latent_config_t* cfg, const lg_latent_weights_t* w, void** model);
+/* The same from a bf16 safetensors file with exactly these tensors: embed, final.norm, head and per layer i
+ * l<i>.norm1, l<i>.canon1, l<i>.dwa, l<i>.mix.{dq,dq.norm,uq,dkv,dkv.norm,uk,uv,o} and with a feed-forward
+ * l<i>.canon2, l<i>.mlp.{gate,up,down} and their .b. */
+uint32_t lg_latent_load(int32_t device, const char* path, const lg_latent_config_t* cfg, void** model);
+void lg_latent_destroy(void* model);
+/* As lg_hybrid_step (cached_lens[i] == 0 starts a sequence, otherwise its slot and blocks must hold what its
+ * previous step left). host_out_rows i32 [n_out]: the tokens of the step (indices into host_ids) whose logits
+ * are computed; NULL: the last token of every sequence (n_out is then n_seqs). host_next_tokens u32 [n_out]
+ * receives the greedy tokens. n_out may be 0. */
+uint32_t lg_latent_step(void* model, const uint32_t* host_ids, const int32_t* host_cached_lens,
+                        const int32_t* host_new_lens, int32_t n_seqs, const int32_t* host_block_tables,
+                        const int32_t* host_state_slots, const int32_t* host_out_rows, int32_t n_out,
+                        uint32_t* host_next_tokens);
+uint32_t lg_latent_replay_device(void* model, void* stream);
+/* fp32 logits of the last step [n_out, vocab], in the order asked for: copied to the host, or the device
+ * buffer itself (valid until the next step; for the sampling chain). */
+uint32_t lg_latent_last_logits(void* model, int32_t n_out, float* host_out);
+void* lg_latent_logits_device(void* model);
+/* X_j of the last step, fp32 [tokens, width], rows in the order of host_ids (diagnostics). */
+uint32_t lg_latent_snapshot(void* model, int32_t j, int32_t n_tokens, float* host_out);
+int32_t lg_latent_launches_last_step(const void* model);
+int32_t lg_latent_device_status(void* model);
+
+/* ====================================================================================
  * Tensor-parallel exchange over NVLink peer memory (ranks = processes on different GPUs of one node).
  * No reference counterpart (the reference is single-device, README.md:19-21). One kernel per rank
  * writes the local partial sum into every peer's receive buffer with plain peer stores, raises a

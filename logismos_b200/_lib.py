@@ -31,7 +31,7 @@ class _LStella(C.Structure):
     pass
 
 
-def _declare(l):
+def _declare(l, partial=False):
     sig = {
         # runtime shim
         "lg_device_count": [C.POINTER(i32)],
@@ -133,70 +133,78 @@ def _declare(l):
         "lg_hybrid_replay_device": [vp, vp],
         "lg_hybrid_last_hidden": [vp, i32, vp],
         "lg_hybrid_last_logits": [vp, i32, vp],
+        # latent-attention decoder
+        "logismos_launch_linear_t_act_bf16": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp, vp],
+        "logismos_launch_linear_small_bf16": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i64, i64, i64, i32, f32, f32, f32, vp],
+        "logismos_launch_linear_f32": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i64, i64, i64, i32, f32, f32, f32, vp],
+        "logismos_launch_varlen_attention_kv_tc_bf16": [vp, i32, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp],
+        "logismos_launch_depth_mix_f32": [vp, i64, i32, vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, vp],
+        "logismos_launch_norm_conv": [vp, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, vp],
+        "logismos_launch_depth_mix_conv_decode": [vp, i64, i32, vp, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp],
+        "logismos_launch_latent_norm_store": [vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i64, i32, vp, vp],
+        "logismos_launch_latent_gather_bf16": [vp, vp, i32, i32, vp, vp, vp, i32, i32, i32, i32, vp, vp],
+        "logismos_launch_latent_decode_bf16": [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp],
+        "logismos_launch_latent_attention_f32": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, vp],
+        "lg_latent_create": [i32, vp, vp, C.POINTER(vp)],
+        "lg_latent_load": [i32, C.c_char_p, vp, C.POINTER(vp)],
+        "lg_latent_step": [vp, vp, vp, vp, i32, vp, vp, vp, i32, vp],
+        "lg_latent_replay_device": [vp, vp],
+        "lg_latent_last_logits": [vp, i32, vp],
+        "lg_latent_snapshot": [vp, i32, i32, vp],
     }
-    for name, args in sig.items():
-        fn = getattr(l, name)
+    # everything that does not return a status
+    other = {
+        "lg_error_kind_name": ([u32], C.c_char_p),
+        "lg_error_string": ([u32], C.c_char_p),
+        "lg_last_error": ([], C.c_char_p),
+        "logismos_paged_decode_scratch_bytes": ([i32, i32, i32], sz),
+        "logismos_varlen_attention_tc_scratch_bytes": ([i32, i32, i32, i32], sz),
+        "logismos_paged_prefix_attention_scratch_bytes": ([i32, i32, i32, i32], sz),
+        "logismos_turbo3_row_bytes": ([i32], sz),
+        "logismos_build_packing": ([vp, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp], i64),
+        "logismos_build_decode_chunks": ([vp, i32, i32, vp], i32),
+        "logismos_pick_decode_chunk": ([vp, i32, i32, i32], i32),
+        "lg_tp_comm_region_bytes": ([i32, u64], sz),
+        "lg_tp_comm_destroy": ([vp, i32], None),
+        "logismos_set_deterministic": ([i32], None),
+        "logismos_get_deterministic": ([], i32),
+        "logismos_skinny_int4_route": ([i32, i32, i32], i32),
+        "logismos_gdn_chunked_scratch_bytes": ([i32, i32, i32], sz),
+        "logismos_set_dependent_launch": ([i32], None),
+        "logismos_get_dependent_launch": ([], i32),
+        "lg_safetensors_close": ([vp], None),
+        "lg_safetensors_len": ([vp], i32),
+        "lg_safetensors_name": ([vp, i32], C.c_char_p),
+        "lg_safetensors_data_region_start": ([vp], u64),
+        "lg_stella_destroy": ([vp], None),
+        "lg_decoder_destroy": ([vp], None),
+        "lg_hybrid_destroy": ([vp], None),
+        "lg_stella_supported_dims": ([vp, C.POINTER(i32), i32], i32),
+        "lg_decoder_launches_last_step": ([vp], i32),
+        "lg_decoder_device_status": ([vp], i32),
+        "lg_hybrid_launches_last_step": ([vp], i32),
+        "lg_hybrid_device_status": ([vp], i32),
+        "lg_stella_default_dim": ([vp], i32),
+        "lg_stella_max_tokens": ([vp], i32),
+        "lg_stella_launches_per_forward": ([vp], i32),
+        "lg_stella_device_status": ([vp], i32),
+        "lg_latent_launches_last_step": ([vp], i32),
+        "lg_latent_device_status": ([vp], i32),
+        "lg_latent_destroy": ([vp], None),
+        "lg_latent_logits_device": ([vp], vp),
+        "logismos_latent_gather_rows": ([i32, i32], i32),
+        "logismos_pick_latent_chunk": ([vp, i32, i32], i32),
+        "logismos_latent_max_chunks": ([i32], i32),
+        "logismos_latent_decode_scratch_bytes": ([i32, i32, i32], sz),
+    }
+    for name, (args, res) in {**{n: (a, u32) for n, a in sig.items()}, **other}.items():
+        fn = getattr(l, name, None)
+        if fn is None:
+            if partial:
+                continue  # a build of one model family: the other families' entry points are not in it
+            raise AttributeError(f"{_SO} lacks {name}: rebuild it with `python -m logismos_b200.build`")
         fn.argtypes = args
-        fn.restype = u32
-    l.lg_error_kind_name.argtypes = [u32]
-    l.lg_error_kind_name.restype = C.c_char_p
-    l.lg_error_string.argtypes = [u32]
-    l.lg_error_string.restype = C.c_char_p
-    l.lg_last_error.argtypes = []
-    l.lg_last_error.restype = C.c_char_p
-    l.logismos_paged_decode_scratch_bytes.argtypes = [i32, i32, i32]
-    l.logismos_paged_decode_scratch_bytes.restype = sz
-    l.logismos_varlen_attention_tc_scratch_bytes.argtypes = [i32, i32, i32, i32]
-    l.logismos_varlen_attention_tc_scratch_bytes.restype = sz
-    l.logismos_paged_prefix_attention_scratch_bytes.argtypes = [i32, i32, i32, i32]
-    l.logismos_paged_prefix_attention_scratch_bytes.restype = sz
-    l.logismos_turbo3_row_bytes.argtypes = [i32]
-    l.logismos_turbo3_row_bytes.restype = sz
-    l.logismos_build_packing.argtypes = [vp, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp]
-    l.logismos_build_packing.restype = i64
-    l.logismos_build_decode_chunks.argtypes = [vp, i32, i32, vp]
-    l.logismos_build_decode_chunks.restype = i32
-    l.logismos_pick_decode_chunk.argtypes = [vp, i32, i32, i32]
-    l.logismos_pick_decode_chunk.restype = i32
-    l.lg_tp_comm_region_bytes.argtypes = [i32, u64]
-    l.lg_tp_comm_region_bytes.restype = sz
-    l.lg_tp_comm_destroy.argtypes = [vp, i32]
-    l.lg_tp_comm_destroy.restype = None
-    l.logismos_set_deterministic.argtypes = [i32]
-    l.logismos_set_deterministic.restype = None
-    l.logismos_get_deterministic.argtypes = []
-    l.logismos_get_deterministic.restype = i32
-    l.logismos_skinny_int4_route.restype = i32
-    l.logismos_gdn_chunked_scratch_bytes.argtypes = [i32, i32, i32]
-    l.logismos_gdn_chunked_scratch_bytes.restype = sz
-    l.logismos_set_dependent_launch.argtypes = [i32]
-    l.logismos_set_dependent_launch.restype = None
-    l.logismos_get_dependent_launch.argtypes = []
-    l.logismos_get_dependent_launch.restype = i32
-    l.lg_safetensors_close.argtypes = [vp]
-    l.lg_safetensors_close.restype = None
-    l.lg_safetensors_len.argtypes = [vp]
-    l.lg_safetensors_len.restype = i32
-    l.lg_safetensors_name.argtypes = [vp, i32]
-    l.lg_safetensors_name.restype = C.c_char_p
-    l.lg_safetensors_data_region_start.argtypes = [vp]
-    l.lg_safetensors_data_region_start.restype = u64
-    l.lg_stella_destroy.argtypes = [vp]
-    l.lg_stella_destroy.restype = None
-    l.lg_decoder_destroy.argtypes = [vp]
-    l.lg_decoder_destroy.restype = None
-    l.lg_hybrid_destroy.argtypes = [vp]
-    l.lg_hybrid_destroy.restype = None
-    for name in ("lg_decoder_launches_last_step", "lg_decoder_device_status", "lg_hybrid_launches_last_step",
-                 "lg_hybrid_device_status"):
-        getattr(l, name).argtypes = [vp]
-        getattr(l, name).restype = i32
-    for name in ("lg_stella_default_dim", "lg_stella_max_tokens", "lg_stella_launches_per_forward",
-                 "lg_stella_device_status"):
-        getattr(l, name).argtypes = [vp]
-        getattr(l, name).restype = i32
-    l.lg_stella_supported_dims.argtypes = [vp, C.POINTER(i32), i32]
-    l.lg_stella_supported_dims.restype = i32
+        fn.restype = res
     return l
 
 
@@ -204,15 +212,22 @@ class _Lazy:
     """Loads the shared library on first use; a missing library is an error, never a fallback."""
 
     def __init__(self):
-        self._l = None
+        self._l, self._path = None, _SO
+
+    def use(self, path: str):
+        """Load this file instead of the whole library: a build of one model family (build.ensure)."""
+        if self._l is not None and path != self._path:
+            raise LogismosError("load", 0, "", f"{self._path} is loaded already")
+        self._path = path
 
     def _load(self):
         if self._l is None:
+            _SO = self._path
             if not os.path.exists(_SO):
                 raise NoGpuBuild("load", 0, "NoGpuBuild",
                                  f"{_SO} is missing: build it with `python -m logismos_b200.build` "
                                  "(there is no CPU fallback)")
-            self._l = _declare(C.CDLL(_SO))
+            self._l = _declare(C.CDLL(_SO), partial=_SO != library_path())
         return self._l
 
     def __getattr__(self, name):

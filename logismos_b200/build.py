@@ -11,6 +11,7 @@ Run as a module:  python -m logismos_b200.build [--force] [--verbose]
 from __future__ import annotations
 
 import concurrent.futures as cf
+import fcntl
 import os
 import shutil
 import subprocess
@@ -24,8 +25,15 @@ SO = os.path.join(HERE, "liblogismos_kernels.so")
 AR = os.path.join(HERE, "liblogismos_kernels.a")
 
 CU_SOURCES = ["cudacore.cu", "legacy_fp16.cu", "elementwise.cu", "gemv_int4.cu", "dequant_int4.cu", "gemm_tcgen05.cu", "qgemm_tcgen05.cu",
-              "attention.cu", "attention_tcgen05.cu", "gdn.cu", "gdn_chunk.cu", "sampling.cu", "kvquant.cu", "stella_model.cu", "decoder_model.cu", "hybrid_model.cu", "tp_comm.cu"]
+              "attention.cu", "attention_tcgen05.cu", "gdn.cu", "gdn_chunk.cu", "sampling.cu", "kvquant.cu", "stella_model.cu", "decoder_model.cu", "hybrid_model.cu", "tp_comm.cu",
+              "linear_small.cu", "depth_conv.cu", "latent_attention.cu", "latent_model.cu"]
 CPP_SOURCES = ["sched.cpp", "loader.cpp", "checkpoints.cpp"]
+
+# what one model family needs: the sources of a library that serves it alone
+GROUPS = {
+    "latent": ["cudacore.cu", "elementwise.cu", "gemm_tcgen05.cu", "attention_tcgen05.cu", "linear_small.cu", "depth_conv.cu",
+               "latent_attention.cu", "latent_model.cu", "sampling.cu", "sched.cpp", "loader.cpp"],
+}
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-std=c++17", "-lineinfo",
               "-Xcompiler", "-fPIC", "-I" + os.path.join(ROOT, "include"), "-I" + CSRC]
@@ -38,13 +46,18 @@ def _nvcc() -> str:
     return n
 
 
-def _sources():
-    out = []
-    for s in CU_SOURCES + CPP_SOURCES:
-        p = os.path.join(CSRC, s)
-        if os.path.exists(p):
-            out.append(p)
-    return out
+def _sources(group=None):
+    names = GROUPS[group] if group else CU_SOURCES + CPP_SOURCES
+    return [os.path.join(CSRC, s) for s in names]
+
+
+def _headers():
+    out = [os.path.join(ROOT, "include", h) for h in os.listdir(os.path.join(ROOT, "include"))]
+    return out + [os.path.join(CSRC, h) for h in os.listdir(CSRC) if h.endswith((".cuh", ".h"))]
+
+
+def group_library(group) -> str:
+    return os.path.join(HERE, f"liblogismos_{group}.so") if group else SO
 
 
 def _stale(target: str, deps) -> bool:
@@ -54,16 +67,18 @@ def _stale(target: str, deps) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
+def build(force: bool = False, verbose: bool = False, group=None) -> str:
+    """Compiles what is out of date and links the whole library, or with ``group`` the library of one model
+    family. Object files are shared between the two. Returns the library's path."""
     if os.environ.get("LOGISMOS_SKIP_CUDA_BUILD"):
         raise RuntimeError("LOGISMOS_SKIP_CUDA_BUILD is set: no GPU kernels are built")
     nvcc = _nvcc()
     os.makedirs(OBJ, exist_ok=True)
-    headers = [os.path.join(ROOT, "include", h) for h in os.listdir(os.path.join(ROOT, "include"))]
-    headers += [os.path.join(CSRC, h) for h in os.listdir(CSRC) if h.endswith((".cuh", ".h"))]
+    headers = _headers()
+    target = group_library(group)
     jobs = []
     objs = []
-    for src in _sources():
+    for src in _sources(group):
         obj = os.path.join(OBJ, os.path.basename(src) + ".o")
         objs.append(obj)
         if force or _stale(obj, [src] + headers):
@@ -81,12 +96,32 @@ def build(force: bool = False, verbose: bool = False) -> str:
                     sys.stderr.write(" ".join(cmd) + "\n" + r.stdout + r.stderr)
                 if r.returncode:
                     raise RuntimeError("nvcc failed for " + cmd[-3])
-    if force or jobs or _stale(SO, objs):
-        subprocess.check_call([nvcc, "-shared", "-o", SO] + objs + ["-gencode", "arch=compute_100a,code=sm_100a"])
-        if os.path.exists(AR):
-            os.remove(AR)
-        subprocess.check_call(["ar", "rcs", AR] + objs)
-    return SO
+    if force or jobs or _stale(target, objs):
+        part = f"{target}.{os.getpid()}"  # a process that has the old file mapped keeps it
+        subprocess.check_call([nvcc, "-shared", "-o", part] + objs + ["-gencode", "arch=compute_100a,code=sm_100a"])
+        os.replace(part, target)
+        if not group:
+            if os.path.exists(AR):
+                os.remove(AR)
+            subprocess.check_call(["ar", "rcs", AR] + objs)
+    return target
+
+
+def ensure(group=None) -> str:
+    """Makes a library for one model family (None: all) available and selects it: the whole library when it is
+    there and up to date, else the family's own, compiled at the first call. For command-line tools that must run from a
+    fresh checkout."""
+    from ._lib import lib
+    if not _stale(SO, _sources() + _headers()):
+        return SO
+    os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(OBJ, ".lock"), "w") as lock:  # one build at a time in a checkout
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        path = group_library(group)
+        if _stale(path, _sources(group) + _headers()):
+            build(group=group)
+    lib.use(path)
+    return path
 
 
 if __name__ == "__main__":

@@ -36,14 +36,14 @@ constexpr int kTileBytes = 128 * 128;        // one [128 rows x 64 bf16] tile
 constexpr int kBars = 8;                     // q_full, k_full, k_empty, v_full, v_empty, s_full, p_full, o_done
 constexpr uint32_t kColS = 0, kColO = 128;   // P replaces S in place; O takes HD columns after it
 
-// HD = head_dim, 128 or 256. Q and K: HD / 64 tiles of [128 rows x 64]; V^T: two tiles of [HD rows x 64 keys].
+// HD = head_dim, 64, 128 or 256. Q and K: HD / 64 tiles of [128 rows x 64]; V^T: two tiles of [HD rows x 64 keys].
 template <int HD> struct Attn {
   static constexpr int kQBytes = (HD / 64) * kTileBytes;
   static constexpr int kKBytes = (HD / 64) * kTileBytes;
   static constexpr int kVTile = HD * 128;
   static constexpr int kVBytes = 2 * kVTile;
   static constexpr size_t kSmem = 1024 + kQBytes + kKBytes + kVBytes + 8 * kBars + 16;  // 97 KB (two CTAs per SM) or 193 KB
-  static constexpr uint32_t kTmemCols = HD == 128 ? 256 : 512;
+  static constexpr uint32_t kTmemCols = HD <= 128 ? 256 : 512;
 };
 
 LG_DEVINL float fast_exp2(float x) {
@@ -349,10 +349,10 @@ gather_paged_kv_turbo3_kernel(const uint8_t* __restrict__ kpool, const uint8_t* 
 }
 
 template <bool CAUSAL, int HD>
-__global__ void __launch_bounds__(192, HD == 128 ? 2 : 1)
+__global__ void __launch_bounds__(192, HD <= 128 ? 2 : 1)
 attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_vt, const int* __restrict__ cu, const int* __restrict__ pstart,
-                    const int* __restrict__ kv_lens, __nv_bfloat16* __restrict__ out, int n_heads, int n_kv, int k_off,
+                    const int* __restrict__ kv_lens, __nv_bfloat16* __restrict__ out, int out_stride, int n_heads, int n_kv, int k_off,
                     float sl2, int* __restrict__ status) {
   lg::pdl_prologue();
   using C = Attn<HD>;
@@ -547,7 +547,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       tc_fence_after();
       const float inv = 1.0f / l;
       const bool store = q0 + row < len;
-      __nv_bfloat16* dst = out + (size_t)(t0 + q0 + row) * (size_t)(n_heads * HD) + h * HD;
+      __nv_bfloat16* dst = out + (size_t)(t0 + q0 + row) * (size_t)out_stride + h * HD;
 #pragma unroll
       for (int c = 0; c < HD / 32; ++c) {
         uint32_t r[32];
@@ -639,7 +639,7 @@ static uint32_t launch_attn_tc(const void* qkv, const void* cu_seqlens, void* ou
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (uint32_t)e;
     lg::launch(kern, grid, dim3(192), smem, s, map_qk, map_qk, map_vt, (const int*)cu_seqlens, pstart, (const int*)nullptr, (__nv_bfloat16*)out,
-                                 n_heads, n_kv_heads, k_off, sl2, (int*)status);
+                                 n_heads * D, n_heads, n_kv_heads, k_off, sl2, (int*)status);
     return lg::launch_status();
   };
   if (D == 128) return causal ? launch(attn_tcgen05_kernel<true, 128>, Attn<128>::kSmem) : launch(attn_tcgen05_kernel<false, 128>, Attn<128>::kSmem);
@@ -722,7 +722,7 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (uint32_t)e;
     lg::launch(kern, grid, dim3(192), smem, s, map_q, map_k, map_vt, (const int*)cu_seqlens_q, pstart, (const int*)kv_lens, (__nv_bfloat16*)out,
-                                 n_heads, n_kv_heads, 0, sl2, (int*)status);
+                                 n_heads * D, n_heads, n_kv_heads, 0, sl2, (int*)status);
     return lg::launch_status();
   };
   if (D == 128) return launch(attn_tcgen05_kernel<true, 128>, Attn<128>::kSmem);
@@ -750,6 +750,38 @@ uint32_t logismos_launch_paged_prefix_attention_turbo3_bf16(const void* q, int32
   return launch_prefix_attn(q, q_row_stride, cu_seqlens_q, kv_lens, k_pool_t3, v_pool_t3, block_tables, max_blocks, n_pool_blocks, out,
                             scratch, n_q_tokens, total_kv_tokens, n_seqs, max_q_len, max_kv_len, n_heads, n_kv_heads, head_dim, true, status,
                             stream);
+}
+
+uint32_t logismos_launch_varlen_attention_kv_tc_bf16(const void* q, int32_t q_row_stride, const void* cu_seqlens_q, const void* kv_lens,
+                                                     const void* kv_start, const void* k, const void* v_t, int32_t n_kv_rows, void* out,
+                                                     int32_t out_row_stride, int32_t n_q_tokens, int32_t n_seqs, int32_t max_q_len,
+                                                     int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, float scale, void* status,
+                                                     void* stream) {
+  lg::LaunchScope launch_scope_;
+  const int D = head_dim;
+  if (n_q_tokens < 0 || n_seqs < 0 || max_q_len < 0 || n_kv_rows <= 0 || (n_kv_rows % 8) || n_heads <= 0 || n_kv_heads <= 0 ||
+      (n_heads % n_kv_heads) || (D != 64 && D != 128 && D != 256) || (q_row_stride % 8) || n_heads * D > q_row_stride ||
+      (out_row_stride % 8) || n_heads * D > out_row_stride || !(scale > 0.0f) || !q || !k || !v_t || !out || !cu_seqlens_q || !kv_lens ||
+      !kv_start || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v_t | (uintptr_t)out) & 15))
+    return lg::kInvalidValue;
+  if (n_seqs == 0 || max_q_len == 0 || n_q_tokens == 0) return 0;
+  const int row_w = n_kv_heads * D;
+  CUtensorMap map_q, map_k, map_vt;
+  if (!make_map(&map_q, q, (uint64_t)n_q_tokens, (uint64_t)n_heads * D, (uint64_t)q_row_stride, 128) ||
+      !make_map(&map_k, k, (uint64_t)n_kv_rows, (uint64_t)row_w, (uint64_t)row_w, 128) ||
+      !make_map(&map_vt, v_t, (uint64_t)row_w, (uint64_t)n_kv_rows, (uint64_t)n_kv_rows, (uint32_t)D))
+    return lg::kInvalidValue;
+  dim3 grid((max_q_len + 127) / 128, n_heads, n_seqs);
+  auto launch = [&](auto kern, size_t smem) -> uint32_t {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+    lg::launch(kern, grid, dim3(192), smem, (cudaStream_t)stream, map_q, map_k, map_vt, (const int*)cu_seqlens_q, (const int*)kv_start, (const int*)kv_lens,
+               (__nv_bfloat16*)out, out_row_stride, n_heads, n_kv_heads, 0, scale * 1.4426950408889634f, (int*)status);
+    return lg::launch_status();
+  };
+  if (D == 64) return launch(attn_tcgen05_kernel<true, 64>, Attn<64>::kSmem);
+  if (D == 128) return launch(attn_tcgen05_kernel<true, 128>, Attn<128>::kSmem);
+  return launch(attn_tcgen05_kernel<true, 256>, Attn<256>::kSmem);
 }
 
 }  // extern "C"

@@ -111,6 +111,13 @@ LG_DEVINL float block_max(float v, float* red) {
   return t;
 }
 
+// clamped gated unit: g' = min(g, limit), u' = clamp(u, -limit, limit); g' sigmoid(alpha g') (u' + shift)
+LG_DEVINL float glu_clamp(float g, float u, float alpha, float limit, float shift) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + __expf(-alpha * g)) * (u + shift);
+}
+
 LG_DEVINL uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
 LG_DEVINL uint32_t pack_bf16x2(float lo, float hi) {

@@ -45,12 +45,15 @@ struct Cfg {
 
 LG_DEVINL float silu_f(float x) { return x / (1.0f + __expf(-x)); }
 
+// constants of the parametrised epilogues (see LG_EPI_F32 and LG_EPI_GLU_CLAMP)
+struct EpiParams { float p0, p1, p2; };
+
 template <int BN, int EPI>
 __global__ void __launch_bounds__(kThreads, 1)
 linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                         const __grid_constant__ CUtensorMap map_out, const float* __restrict__ bias,
                         void* __restrict__ out, int M, int N, int K, int ldc, int splits, int w_static,
-                        int* __restrict__ status) {
+                        EpiParams ep, int* __restrict__ status) {
   using C = Cfg<BN>;
   lg::pdl_trigger();
   extern __shared__ uint8_t smem_raw[];
@@ -237,7 +240,34 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
               }
           }
         }
-      } else {  // LG_EPI_SWIGLU
+      } else if (EPI == LG_EPI_F32) {
+        const bool vec = (ldc & 3) == 0;
+        for (int c = 0; c < BN; c += 32) {
+          uint32_t r[32];
+          tc_ld32(t_row + c, r);
+          tc_wait_ld();
+          const int ncol = n_blk * BN + c;
+          if (row < M) {
+            float* dst = reinterpret_cast<float*>(out) + (size_t)row * ldc + ncol;
+#pragma unroll
+            for (int j = 0; j < 32; j += 4) {
+              float v[4];
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                v[i] = __uint_as_float(r[j + i]);
+                if (bias && ncol + j + i < N) v[i] += bias[ncol + j + i];
+                if (ep.p0 > 0.0f) v[i] = ep.p0 * tanhf(v[i] / ep.p0);
+              }
+              if (vec && ncol + j + 4 <= N) {
+                *reinterpret_cast<float4*>(dst + j) = make_float4(v[0], v[1], v[2], v[3]);
+              } else {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) if (ncol + j + i < N) dst[j + i] = v[i];
+              }
+            }
+          }
+        }
+      } else {  // LG_EPI_SWIGLU, LG_EPI_GLU_CLAMP
         // W rows interleave 32 gate rows with the 32 matching up rows
         for (int c = 0; c < BN; c += 64) {
           uint32_t g[32], u[32];
@@ -257,7 +287,8 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                 float g0 = __uint_as_float(g[e]), g1 = __uint_as_float(g[e + 1]);
                 float u0 = __uint_as_float(u[e]), u1 = __uint_as_float(u[e + 1]);
                 if (bias) { g0 += bias[ncol + e]; g1 += bias[ncol + e + 1]; u0 += bias[ncol + 32 + e]; u1 += bias[ncol + 32 + e + 1]; }
-                w[i] = pack_bf16x2(silu_f(g0) * u0, silu_f(g1) * u1);
+                if (EPI == LG_EPI_GLU_CLAMP) w[i] = pack_bf16x2(lg::glu_clamp(g0, u0, ep.p0, ep.p1, ep.p2), lg::glu_clamp(g1, u1, ep.p0, ep.p1, ep.p2));
+                else w[i] = pack_bf16x2(silu_f(g0) * u0, silu_f(g1) * u1);
               }
               *reinterpret_cast<uint4*>(dst + j * 8) = make_uint4(w[0], w[1], w[2], w[3]);
             }
@@ -309,7 +340,7 @@ __global__ void linear_t_naive_kernel(const __nv_bfloat16* __restrict__ a, const
 
 template <int BN, int EPI>
 uint32_t launch_cfg(const void* a, const void* w, const float* bias, void* out, int m, int n, int k, int lda,
-                    int ldc, int w_static, int* status, cudaStream_t stream) {
+                    int ldc, int w_static, EpiParams ep, int* status, cudaStream_t stream) {
   CUtensorMap ma, mw, mo;
   if (!make_map(&ma, a, (uint64_t)m, (uint64_t)k, (uint64_t)lda, BM)) return lg::kInvalidValue;
   if (!make_map(&mw, w, (uint64_t)n, (uint64_t)k, (uint64_t)k, BN)) return lg::kInvalidValue;
@@ -336,13 +367,13 @@ uint32_t launch_cfg(const void* a, const void* w, const float* bias, void* out, 
   }
   const int items = tiles * splits;
   const int grid = items < sm_count() ? items : sm_count();
-  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, mo, bias, out, m, n, k, ldc, splits, w_static, status);
+  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, mo, bias, out, m, n, k, ldc, splits, w_static, ep, status);
   return lg::launch_status();
 }
 
 template <int EPI>
 uint32_t launch_epi(const void* a, const void* w, const float* bias, void* out, int m, int n, int k, int lda,
-                    int ldc, int w_static, int* status, cudaStream_t stream) {
+                    int ldc, int w_static, EpiParams ep, int* status, cudaStream_t stream) {
   // tile width by wave quantisation: time ~ waves(BN) * BN; ties go to the wider tile
   const int sms = sm_count();
   const int mt = (m + BM - 1) / BM;
@@ -356,35 +387,48 @@ uint32_t launch_epi(const void* a, const void* w, const float* bias, void* out, 
     const long cost = waves * bn;
     if (best_cost < 0 || cost < best_cost) { best_cost = cost; best_bn = bn; }
   }
-  if (best_bn == 256) return launch_cfg<256, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, status, stream);
-  if (best_bn == 192) return launch_cfg<192, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, status, stream);
-  return launch_cfg<128, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, status, stream);
+  if (best_bn == 256) return launch_cfg<256, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream);
+  if (best_bn == 192) return launch_cfg<192, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream);
+  return launch_cfg<128, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream);
 }
 
 }  // namespace
 
 extern "C" {
 
-uint32_t logismos_launch_linear_t_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m,
-                                       int32_t n, int32_t k, int32_t lda, int32_t ldc, int32_t epilogue,
-                                       void* status_i32, void* stream) {
+uint32_t logismos_launch_linear_t_act_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m,
+                                           int32_t n, int32_t k, int32_t lda, int32_t ldc, int32_t epilogue, float p0,
+                                           float p1, float p2, void* status_i32, void* stream) {
   lg::LaunchScope launch_scope_;
   const int w_static = (epilogue & LG_EPI_STATIC_W) ? 1 : 0;
   epilogue &= ~LG_EPI_STATIC_W;
-  if (m <= 0 || n <= 0 || k <= 0 || (k % BK) || (n % 16) || (lda % 8) || lda < k) return lg::kInvalidValue;
+  if (m <= 0 || n <= 0 || k <= 0 || (k % BK) || (epilogue != LG_EPI_F32 && (n % 16)) || (lda % 8) || lda < k) return lg::kInvalidValue;
   if (((uintptr_t)a & 15) || ((uintptr_t)w & 15) || ((uintptr_t)out & 15)) return lg::kInvalidValue;
-  if (epilogue == LG_EPI_SWIGLU && (n % 64)) return lg::kInvalidValue;
-  const int out_cols = epilogue == LG_EPI_SWIGLU ? n / 2 : n;
-  if (ldc < out_cols || (ldc % (epilogue == LG_EPI_RESID_F32 ? 4 : 8))) return lg::kInvalidValue;
+  const bool glu = epilogue == LG_EPI_SWIGLU || epilogue == LG_EPI_GLU_CLAMP;
+  if (glu && (n % 64)) return lg::kInvalidValue;
+  const int out_cols = glu ? n / 2 : n;
+  const int align = epilogue == LG_EPI_F32 ? 1 : epilogue == LG_EPI_RESID_F32 ? 4 : 8;
+  if (ldc < out_cols || (ldc % align)) return lg::kInvalidValue;
   cudaStream_t s = (cudaStream_t)stream;
   const float* b = (const float*)bias;
   int* st = (int*)status_i32;
+  const EpiParams ep{p0, p1, p2};
   switch (epilogue) {
-    case LG_EPI_BF16: return launch_epi<LG_EPI_BF16>(a, w, b, out, m, n, k, lda, ldc, w_static, st, s);
-    case LG_EPI_RESID_F32: return launch_epi<LG_EPI_RESID_F32>(a, w, b, out, m, n, k, lda, ldc, w_static, st, s);
-    case LG_EPI_SWIGLU: return launch_epi<LG_EPI_SWIGLU>(a, w, b, out, m, n, k, lda, ldc, w_static, st, s);
+    case LG_EPI_BF16: return launch_epi<LG_EPI_BF16>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
+    case LG_EPI_RESID_F32: return launch_epi<LG_EPI_RESID_F32>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
+    case LG_EPI_SWIGLU: return launch_epi<LG_EPI_SWIGLU>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
+    case LG_EPI_F32: return launch_epi<LG_EPI_F32>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
+    case LG_EPI_GLU_CLAMP: return launch_epi<LG_EPI_GLU_CLAMP>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
     default: return lg::kInvalidValue;
   }
+}
+
+uint32_t logismos_launch_linear_t_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m,
+                                       int32_t n, int32_t k, int32_t lda, int32_t ldc, int32_t epilogue,
+                                       void* status_i32, void* stream) {
+  const int e = epilogue & ~LG_EPI_STATIC_W;
+  if (e != LG_EPI_BF16 && e != LG_EPI_RESID_F32 && e != LG_EPI_SWIGLU) return lg::kInvalidValue;
+  return logismos_launch_linear_t_act_bf16(a, w, bias, out, m, n, k, lda, ldc, epilogue, 0.0f, 0.0f, 0.0f, status_i32, stream);
 }
 
 uint32_t logismos_launch_linear_t_naive_bf16(const void* a, const void* w, const void* bias, void* out,

@@ -1,0 +1,286 @@
+// C = A W^T for few rows and bf16 weights (decode steps): the weights are streamed once, straight from
+// global memory into mma.sync fragments. Also the batched form (one small matrix per head) and the
+// fp32-activation form of the same contract.
+//
+// linear_small_kernel: CTA = 16 * MT weight rows x up to 8 * NT activation rows, its warps split k in
+// steps of 32. A lane reads 16 consecutive bytes (8 values along k) of weight rows g and g + 8 and of
+// activation row g (g = lane / 4): the k order inside a 32-wide step is permuted the same way on both
+// sides, so each 16-byte read feeds two m16n8k16 instructions without any shuffle. The partial sums of
+// the warps meet in shared memory in a fixed order, so results do not depend on timing.
+#include "common.cuh"
+#include "logismos_kernels.h"
+
+namespace {
+
+using namespace lg;
+
+struct SmallArgs {
+  const __nv_bfloat16* a;
+  const __nv_bfloat16* w;
+  const float* bias;
+  void* out;
+  int m, n, k, lda, ldc, epi;
+  int64_t a_stride, w_stride, out_stride;  // per batch entry (elements)
+  float p0, p1, p2;
+};
+
+LG_DEVINL uint4 ldg16(const void* p) { return __ldg(reinterpret_cast<const uint4*>(p)); }
+
+template <int MT, int NT>
+__global__ void __launch_bounds__(512)
+linear_small_kernel(SmallArgs p) {
+  lg::pdl_trigger();
+  constexpr int kUnroll = MT * NT >= 8 ? 2 : 4;
+  extern __shared__ float red[];  // [warps][16 * MT][8 * NT]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int g = lane >> 2, t = lane & 3;
+  const bool glu = p.epi == LG_EPI_SWIGLU || p.epi == LG_EPI_GLU_CLAMP;
+  // first weight row of each m16 tile: gated epilogues take 16 gate rows and the 16 matching up rows
+  // (rows interleave in blocks of 32), the others consecutive rows
+  int row0[MT];
+  if (glu) {
+    const int u = blockIdx.x;  // MT == 2
+    row0[0] = (u >> 1) * 64 + (u & 1) * 16;
+    if (MT == 2) row0[MT - 1] = row0[0] + 32;
+  } else {
+#pragma unroll
+    for (int i = 0; i < MT; ++i) row0[i] = (blockIdx.x * MT + i) * 16;
+  }
+  const int m0 = blockIdx.y * 8 * NT;
+  const __nv_bfloat16* wb = p.w + (size_t)blockIdx.z * p.w_stride;
+  const __nv_bfloat16* ab = p.a + (size_t)blockIdx.z * p.a_stride;
+  const __nv_bfloat16* wr[MT][2];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) wr[i][h] = wb + (size_t)min(row0[i] + g + 8 * h, p.n - 1) * p.k + 8 * t;
+  const int steps = p.k >> 5;
+  float acc[MT][NT][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.0f;
+  uint4 wv[kUnroll][MT][2];
+  auto load_w = [&](int s0) {
+#pragma unroll
+    for (int u = 0; u < kUnroll; ++u) {
+      const int s = s0 + u * n_warps;
+#pragma unroll
+      for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) wv[u][i][h] = s < steps ? ldg16(wr[i][h] + (size_t)s * 32) : make_uint4(0u, 0u, 0u, 0u);
+    }
+  };
+  load_w(warp);      // the weights are static: requested before the dependency wait
+  lg::pdl_wait();
+  for (int s0 = warp; s0 < steps; s0 += kUnroll * n_warps) {
+#pragma unroll
+    for (int u = 0; u < kUnroll; ++u) {
+      const int s = s0 + u * n_warps;
+      if (s < steps) {
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          const int r = m0 + 8 * j + g;
+          uint4 x = make_uint4(0u, 0u, 0u, 0u);
+          if (r < p.m) x = *reinterpret_cast<const uint4*>(ab + (size_t)r * p.lda + (size_t)s * 32 + 8 * t);
+          const uint32_t b0[2] = {x.x, x.y}, b1[2] = {x.z, x.w};
+#pragma unroll
+          for (int i = 0; i < MT; ++i) {
+            const uint4 lo = wv[u][i][0], hi = wv[u][i][1];
+            const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
+            mma_bf16_16816(acc[i][j], a0, b0, acc[i][j]);
+            mma_bf16_16816(acc[i][j], a1, b1, acc[i][j]);
+          }
+        }
+      }
+    }
+    if (s0 + kUnroll * n_warps < steps) load_w(s0 + kUnroll * n_warps);
+  }
+  // acc[i][j]: weight rows g, g + 8 of tile i; activation rows 8 j + 2 t, + 1
+  constexpr int kRows = 16 * MT, kCols = 8 * NT;
+  float* mine = red + (size_t)warp * kRows * kCols;
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      mine[(8 * j + 2 * t) * kRows + 16 * i + g] = acc[i][j][0];
+      mine[(8 * j + 2 * t + 1) * kRows + 16 * i + g] = acc[i][j][1];
+      mine[(8 * j + 2 * t) * kRows + 16 * i + g + 8] = acc[i][j][2];
+      mine[(8 * j + 2 * t + 1) * kRows + 16 * i + g + 8] = acc[i][j][3];
+    }
+  __syncthreads();
+  const int out_rows = glu ? 16 : kRows;  // output columns this CTA produces
+  for (int e = threadIdx.x; e < out_rows * kCols; e += blockDim.x) {
+    const int c = e % out_rows, r = m0 + e / out_rows;
+    if (r >= p.m) continue;
+    float v = 0.0f, u = 0.0f;
+    for (int w = 0; w < n_warps; ++w) {
+      const float* q = red + ((size_t)w * kCols + e / out_rows) * kRows;
+      v += q[c];
+      if (glu) u += q[c + 16];
+    }
+    const int wrow = row0[0] + c;  // consecutive rows across the MT tiles when not gated
+    if (wrow >= p.n) continue;
+    if (glu) {
+      if (p.bias) { v += p.bias[wrow]; u += p.bias[wrow + 32]; }
+      const float y = p.epi == LG_EPI_GLU_CLAMP ? glu_clamp(v, u, p.p0, p.p1, p.p2) : v / (1.0f + __expf(-v)) * u;
+      const int oc = (wrow >> 6) * 32 + (wrow & 31);
+      reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)blockIdx.z * p.out_stride + (size_t)r * p.ldc + oc] = __float2bfloat16_rn(y);
+      continue;
+    }
+    if (p.bias) v += p.bias[wrow];
+    const size_t o = (size_t)blockIdx.z * p.out_stride + (size_t)r * p.ldc + wrow;
+    if (p.epi == LG_EPI_BF16) reinterpret_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16_rn(v);
+    else if (p.epi == LG_EPI_RESID_F32) reinterpret_cast<float*>(p.out)[o] += v;
+    else reinterpret_cast<float*>(p.out)[o] = p.p0 > 0.0f ? p.p0 * tanhf(v / p.p0) : v;
+  }
+}
+
+template <int MT, int NT>
+uint32_t launch_small(const SmallArgs& a, int batch, int warps, cudaStream_t s) {
+  const bool glu = a.epi == LG_EPI_SWIGLU || a.epi == LG_EPI_GLU_CLAMP;
+  const size_t smem = (size_t)warps * 16 * MT * 8 * NT * 4;
+  auto kern = linear_small_kernel<MT, NT>;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+  }
+  const int tiles = glu ? a.n / 32 : (a.n + 16 * MT - 1) / (16 * MT);
+  lg::launch(kern, dim3((unsigned)tiles, (unsigned)((a.m + 8 * NT - 1) / (8 * NT)), (unsigned)batch), dim3(32 * warps), smem, s, a);
+  return lg::launch_status();
+}
+
+// ---- fp32 activations -----------------------------------------------------------------------------
+// 64 x 64 tile, 256 threads, 4 x 4 outputs per thread: rows 4 ty .. + 3; columns 2 tx, 2 tx + 1 and the
+// same + 32, so that a thread holds a gate column and its matching up column. fp32 products and sums.
+struct F32Args {
+  const float* a;
+  const __nv_bfloat16* w;
+  const float* bias;
+  float* out;
+  int m, n, k, lda, ldc, epi;
+  int64_t a_stride, w_stride, out_stride;
+  float p0, p1, p2;
+};
+
+__global__ void __launch_bounds__(256)
+linear_f32_kernel(F32Args p) {
+  lg::pdl_prologue();
+  __shared__ float as[16][68], ws[16][68];
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const int n0 = blockIdx.x * 64, m0 = blockIdx.y * 64;
+  const float* A = p.a + (size_t)blockIdx.z * p.a_stride;
+  const __nv_bfloat16* W = p.w + (size_t)blockIdx.z * p.w_stride;
+  float acc[4][4] = {};
+  const int lr = tid >> 2, lk = (tid & 3) * 4;
+  for (int k0 = 0; k0 < p.k; k0 += 16) {
+    float4 av = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (m0 + lr < p.m) av = *reinterpret_cast<const float4*>(A + (size_t)(m0 + lr) * p.lda + k0 + lk);
+    float wv[4] = {0.f, 0.f, 0.f, 0.f};
+    if (n0 + lr < p.n) {
+      const uint2 u = __ldg(reinterpret_cast<const uint2*>(W + (size_t)(n0 + lr) * p.k + k0 + lk));
+      const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+      wv[0] = a.x; wv[1] = a.y; wv[2] = b.x; wv[3] = b.y;
+    }
+    as[lk][lr] = av.x; as[lk + 1][lr] = av.y; as[lk + 2][lr] = av.z; as[lk + 3][lr] = av.w;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) ws[lk + i][lr] = wv[i];
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < 16; ++kk) {
+      float x[4], y[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i] = as[kk][4 * ty + i];
+      y[0] = ws[kk][2 * tx]; y[1] = ws[kk][2 * tx + 1]; y[2] = ws[kk][32 + 2 * tx]; y[3] = ws[kk][33 + 2 * tx];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], y[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+  float* out = p.out + (size_t)blockIdx.z * p.out_stride;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = m0 + 4 * ty + i;
+    if (r >= p.m) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = n0 + (j >> 1) * 32 + 2 * tx + (j & 1);
+      if (c < p.n && p.bias) acc[i][j] += p.bias[c];
+    }
+    if (p.epi == LG_EPI_GLU_CLAMP) {
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        if (n0 + 2 * tx + j >= p.n) continue;
+        const float g = fminf(acc[i][j], p.p1), u = fminf(fmaxf(acc[i][j + 2], -p.p1), p.p1);
+        out[(size_t)r * p.ldc + (n0 >> 1) + 2 * tx + j] = g / (1.0f + expf(-p.p0 * g)) * (u + p.p2);
+      }
+      continue;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = n0 + (j >> 1) * 32 + 2 * tx + (j & 1);
+      if (c >= p.n) continue;
+      float* o = out + (size_t)r * p.ldc + c;
+      if (p.epi == LG_EPI_RESID_F32) *o += acc[i][j];
+      else *o = p.p0 > 0.0f ? p.p0 * tanhf(acc[i][j] / p.p0) : acc[i][j];
+    }
+  }
+}
+
+}  // namespace
+
+extern "C" {
+
+uint32_t logismos_launch_linear_small_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k,
+                                           int32_t lda, int32_t ldc, int32_t batch, int64_t a_stride, int64_t w_stride,
+                                           int64_t out_stride, int32_t epilogue, float p0, float p1, float p2, void* stream) {
+  lg::LaunchScope launch_scope_;
+  epilogue &= ~LG_EPI_STATIC_W;
+  const bool glu = epilogue == LG_EPI_SWIGLU || epilogue == LG_EPI_GLU_CLAMP;
+  if (m <= 0 || n <= 0 || k <= 0 || (k % 32) || batch <= 0 || batch > 65535 || (lda % 8) || lda < k || (a_stride % 8) || (w_stride % 8) ||
+      (glu && (n % 64)) || ldc < (glu ? n / 2 : n) || (((uintptr_t)a | (uintptr_t)w) & 15) || !out || (m + 7) / 8 > 65535)
+    return lg::kInvalidValue;
+  if (epilogue != LG_EPI_BF16 && epilogue != LG_EPI_RESID_F32 && epilogue != LG_EPI_F32 && !glu) return lg::kInvalidValue;
+  const SmallArgs p{(const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (const float*)bias, out, m, n, k, lda, ldc, epilogue,
+                    a_stride, w_stride, out_stride, p0, p1, p2};
+  cudaStream_t s = (cudaStream_t)stream;
+  // two m16 tiles per CTA once that still leaves two CTAs per SM (the activations are then read half as often)
+  const int64_t ctas2 = (int64_t)((n + 31) / 32) * batch;
+  const bool two = glu || ctas2 >= 296;
+  const int steps = k / 32;
+  int warps = steps < 8 ? steps : 8;
+  if (steps >= 128 && !two) warps = 16;
+  const int nt = m <= 8 ? 1 : m <= 16 ? 2 : m <= 32 ? 4 : 8;
+  if (two) {
+    if (nt == 1) return launch_small<2, 1>(p, batch, warps, s);
+    if (nt == 2) return launch_small<2, 2>(p, batch, warps, s);
+    if (nt == 4) return launch_small<2, 4>(p, batch, warps, s);
+    return launch_small<2, 8>(p, batch, warps, s);
+  }
+  if (nt == 1) return launch_small<1, 1>(p, batch, warps, s);
+  if (nt == 2) return launch_small<1, 2>(p, batch, warps, s);
+  if (nt == 4) return launch_small<1, 4>(p, batch, warps, s);
+  return launch_small<1, 8>(p, batch, warps, s);
+}
+
+uint32_t logismos_launch_linear_f32(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k,
+                                    int32_t lda, int32_t ldc, int32_t batch, int64_t a_stride, int64_t w_stride, int64_t out_stride,
+                                    int32_t epilogue, float p0, float p1, float p2, void* stream) {
+  lg::LaunchScope launch_scope_;
+  epilogue &= ~LG_EPI_STATIC_W;
+  const bool glu = epilogue == LG_EPI_GLU_CLAMP;
+  if (m <= 0 || n <= 0 || k <= 0 || (k % 16) || batch <= 0 || batch > 65535 || (lda % 4) || lda < k || (a_stride % 4) || (w_stride % 4) ||
+      (glu && (n % 64)) || ldc < (glu ? n / 2 : n) || ((uintptr_t)a & 15) || ((uintptr_t)w & 7) || !out || (m + 63) / 64 > 65535)
+    return lg::kInvalidValue;
+  if (epilogue != LG_EPI_RESID_F32 && epilogue != LG_EPI_F32 && !glu) return lg::kInvalidValue;
+  const F32Args p{(const float*)a, (const __nv_bfloat16*)w, (const float*)bias, (float*)out, m, n, k, lda, ldc, epilogue,
+                  a_stride, w_stride, out_stride, p0, p1, p2};
+  lg::launch(linear_f32_kernel, dim3((unsigned)((n + 63) / 64), (unsigned)((m + 63) / 64), (unsigned)batch), dim3(256), 0, (cudaStream_t)stream, p);
+  return lg::launch_status();
+}
+
+}  // extern "C"

@@ -26,11 +26,13 @@ struct StepLimits {
   int max_blocks_per_seq = 0, n_pool_blocks = 0, max_step_tokens = 0, max_step_seqs = 0;
   int n_state_slots = 0;       // 0: the executor keeps no per-sequence state
   size_t prefix_cap_tokens = 0;  // keys one gather may hold
+  size_t extra_bytes = 0;      // room at the end of the block for arrays of the executor's own
 };
 
 struct StepBatch {
   StepLimits lim;
   uint8_t* pinned = nullptr;
+  size_t capacity = 0;          // bytes of `pinned`
   // packed order: decode rows first, prefill rows after them (host views into `pinned`)
   uint32_t* ids = nullptr;      // [T]
   int32_t* pos = nullptr;       // [T]
@@ -45,6 +47,8 @@ struct StepBatch {
   int32_t* pre_kv = nullptr;    // [prefill sequences] keys of each
   int32_t* state = nullptr;     // [n_seqs] state slots
   uint8_t* fresh = nullptr;     // [n_seqs] 1: the sequence starts here
+  uint8_t* phase = nullptr;     // [n_seqs] filled by executors whose states alternate between two copies
+  uint8_t* extra = nullptr;     // [extra_bytes], 8-byte aligned
   int T = 0, n_dec = 0, n_pre = 0, n_seqs = 0, max_pre_len = 0, run_count = 0;
   bool has_prefix = false;      // some prefill chunk continues a cached sequence
   std::vector<int> order;       // packed sequence -> caller's sequence
@@ -54,8 +58,8 @@ struct StepBatch {
   bool alloc(const StepLimits& l) {
     lim = l;
     const size_t T_ = (size_t)l.max_step_tokens, S = (size_t)l.max_step_seqs, MB = (size_t)l.max_blocks_per_seq;
-    const size_t bytes = T_ * 20 + (S + 1) * 4 * 4 + S * MB * 4 + S * 4 * 3 + S + 64;
-    return cudaMallocHost((void**)&pinned, bytes) == cudaSuccess;
+    capacity = T_ * 20 + (S + 1) * 4 * 4 + S * MB * 4 + S * 4 * 3 + S * 2 + l.extra_bytes + 64;
+    return cudaMallocHost((void**)&pinned, capacity) == cudaSuccess;
   }
   void release() {
     if (pinned) cudaFreeHost(pinned);
@@ -108,6 +112,9 @@ struct StepBatch {
     pre_kv = (int32_t*)carve((size_t)n * 4);
     state = (int32_t*)carve((size_t)n * 4);
     fresh = carve((size_t)n);
+    phase = carve((size_t)n);
+    extra = carve(0) + ((8 - ((uintptr_t)pp & 7)) & 7);
+    std::memset(phase, 0, (size_t)n);
     cached.assign((size_t)n, 0);
     newl.assign((size_t)n, 0);
     int64_t t = 0;
@@ -155,6 +162,17 @@ struct StepBatch {
       runs.push_back(r);
     }
     return LG_EMB_OK;
+  }
+
+  // rows[i] = packed row of the caller's token i, for all T tokens of the step
+  void caller_rows(int32_t* rows) const {
+    std::vector<int> at((size_t)n_seqs);  // caller's sequence -> packed sequence
+    for (int s = 0; s < n_seqs; ++s) at[(size_t)order[(size_t)s]] = s;
+    int32_t t = 0;
+    for (int i = 0; i < n_seqs; ++i) {
+      const int s = at[(size_t)i];
+      for (int r = cu[s]; r < cu[s + 1]; ++r) rows[t++] = r;
+    }
   }
 };
 
