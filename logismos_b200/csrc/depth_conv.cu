@@ -229,7 +229,7 @@ uint32_t logismos_launch_norm_conv(const void* x_f32, const void* inv_rms_f32, c
                                    const void* state_slots_i32, const void* fresh_u8, const void* phase_u8, const void* seq_ids_i32,
                                    const void* cu_seqlens_i32, int32_t rows, int32_t ld, int32_t taps, void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!x_f32 || !inv_rms_f32 || !gain_f32 || !o1 || rows <= 0 || ld <= 0 || ld % 4 || taps < 1 || taps > kMaxTaps || !state_f32)
+  if (!x_f32 || !inv_rms_f32 || !gain_f32 || !o1 || rows <= 0 || ld <= 0 || ld % 4 || taps < 1 || taps > kMaxTaps || (taps > 1 && !state_f32))
     return lg::kInvalidValue;
   const ConvArgs c{(const float*)gain_f32, (const float*)w1_f32, (const float*)w2_f32, o1, o2, (float*)state_f32, (const int*)state_slots_i32,
                    (const uint8_t*)fresh_u8, (const uint8_t*)phase_u8, taps};
@@ -257,7 +257,7 @@ uint32_t logismos_launch_depth_mix_conv_decode(const void* hist_f32, int64_t his
                                                const void* phase_u8, int32_t rows, int32_t n, int32_t ld, float eps, int32_t taps,
                                                void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!mix_ok(hist_f32, n_hist, coef_f32, rows, n, ld) || !x_f32 || !gain_f32 || !o1 || taps < 1 || taps > kMaxTaps || !state_f32)
+  if (!mix_ok(hist_f32, n_hist, coef_f32, rows, n, ld) || !x_f32 || !gain_f32 || !o1 || taps < 1 || taps > kMaxTaps || (taps > 1 && !state_f32))
     return lg::kInvalidValue;
   const MixArgs p{(const float*)hist_f32, hist_stride, n_hist, (const float*)coef_f32, nullptr, rows, (float*)x_f32, nullptr,
                   nullptr, nullptr, rows, n, ld, out_f32, eps, nullptr};

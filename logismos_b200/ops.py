@@ -538,3 +538,169 @@ def greedy(logits, sync=True):
         check(lib.logismos_launch_greedy_argmax(_p(logits), int(logits.dtype == torch.float32), _p(out), logits.shape[0], logits.shape[1], _stream()), "greedy_argmax")
         _done(sync)
     return out
+
+
+# ---- parallel-block decoders with latent attention ---------------------------------------------
+
+EPI_F32, EPI_GLU_CLAMP = 3, 4
+_ACT_DTYPE = {EPI_BF16: torch.bfloat16, EPI_SWIGLU: torch.bfloat16, EPI_GLU_CLAMP: torch.bfloat16, EPI_F32: torch.float32}
+
+
+def linear_act(a, w, bias=None, epilogue=EPI_F32, p=(0.0, 0.0, 0.0), residual=None, small=False, batch=1, sync=True):
+    """C = A W^T (+bias) with a parametrised epilogue (EPI_F32 with soft cap p[0], EPI_GLU_CLAMP with alpha, limit,
+    shift) or one of linear_t's. a bf16: the tcgen05 kernel, or with ``small`` the weight-streaming kernel for
+    few rows; a fp32: fp32 products and sums. batch > 1 (small or fp32): a [m, batch, k], w [batch, n, k] ->
+    [m, batch, n]."""
+    f32 = a.dtype == torch.float32
+    _req(a, "a", torch.float32 if f32 else torch.bfloat16); _req(w, "w", torch.bfloat16)
+    m, k, n = a.shape[0], a.shape[-1], w.shape[-2]
+    if w.shape[-1] != k or (batch > 1 and (a.shape[1] != batch or w.shape[0] != batch or not (small or f32))):
+        raise InvalidOp("linear_act: shapes")
+    cols = n // 2 if epilogue in (EPI_SWIGLU, EPI_GLU_CLAMP) else n
+    if residual is not None:
+        _req(residual, "residual", torch.float32, 2)
+        out, epilogue = residual, EPI_RESID_F32
+    else:
+        shape = (m, batch, cols) if batch > 1 else (m, cols)
+        out = torch.empty(shape, dtype=torch.float32 if f32 else _ACT_DTYPE[epilogue], device=a.device)
+    status = torch.zeros(1, dtype=torch.int32, device=a.device)
+    with torch.cuda.device(a.device):
+        if f32 or small:
+            fn = lib.logismos_launch_linear_f32 if f32 else lib.logismos_launch_linear_small_bf16
+            check(fn(_p(a), _p(w), _p(bias), _p(out), m, n, k, k * batch, cols * batch, batch, k, n * k, cols, epilogue, *p, _stream()), "linear_act")
+        else:
+            check(lib.logismos_launch_linear_t_act_bf16(_p(a), _p(w), _p(bias), _p(out), m, n, k, k, cols, epilogue, *p, _p(status), _stream()), "linear_act")
+        _done(sync)
+        if sync and int(status.item()) != 0:
+            raise InvalidOp("linear_act: a bounded wait expired")
+    return out
+
+
+def depth_mix(hist, coef, gain, n, eps, row_idx=None, out_f32=True, sync=True):
+    """hist fp32 [snapshots, tokens, ld] -> (x, 1 / rms, normed x) of sum_j coef[j] hist[j]."""
+    _req(hist, "hist", torch.float32, 3); _req(coef, "coef", torch.float32, 1)
+    j, t, ld = hist.shape
+    rows = t if row_idx is None else row_idx.numel()
+    x = torch.empty((rows, ld), dtype=torch.float32, device=hist.device)
+    inv = torch.empty(rows, dtype=torch.float32, device=hist.device)
+    y = torch.empty((rows, ld), dtype=torch.float32 if out_f32 else torch.bfloat16, device=hist.device)
+    status = torch.zeros(1, dtype=torch.int32, device=hist.device)
+    with torch.cuda.device(hist.device):
+        check(lib.logismos_launch_depth_mix_f32(_p(hist), t * ld, j, _p(coef), _p(row_idx), t, _p(x), _p(inv), _p(gain), _p(y), int(out_f32), rows, n,
+                                                ld, float(eps), _p(status), _stream()), "depth_mix")
+        _done(sync)
+        if sync and int(status.item()) != 0:
+            raise InvalidOp("depth_mix: a row index outside the snapshots")
+    return x, inv, y
+
+
+def norm_conv(x, inv_rms, gain, w1, w2, state, state_slots, fresh, phase, seq_ids, cu_seqlens, out_f32=True, sync=True):
+    """Input convolutions of a ragged batch; ``state`` fp32 [slots, 2, taps - 1, ld] is updated in place."""
+    _req(x, "x", torch.float32, 2); _req(state, "state", torch.float32, 4)
+    rows, ld = x.shape
+    taps = state.shape[2] + 1
+    o = [torch.empty((rows, ld), dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device) for _ in range(2)]
+    with torch.cuda.device(x.device):
+        check(lib.logismos_launch_norm_conv(_p(x), _p(inv_rms), _p(gain), _p(w1), _p(w2), _p(o[0]), _p(o[1]), int(out_f32), _p(state), _p(state_slots),
+                                            _p(fresh), _p(phase), _p(seq_ids), _p(cu_seqlens), rows, ld, taps, _stream()), "norm_conv")
+        _done(sync)
+    return o[0], o[1]
+
+
+def depth_mix_conv_decode(hist, coef, gain, w1, w2, state, state_slots, fresh, phase, n, eps, out_f32=True, sync=True):
+    """depth_mix and norm_conv in one launch for one token per sequence -> (x, o1, o2)."""
+    _req(hist, "hist", torch.float32, 3); _req(state, "state", torch.float32, 4)
+    j, rows, ld = hist.shape
+    x = torch.empty((rows, ld), dtype=torch.float32, device=hist.device)
+    o = [torch.empty((rows, ld), dtype=torch.float32 if out_f32 else torch.bfloat16, device=hist.device) for _ in range(2)]
+    with torch.cuda.device(hist.device):
+        check(lib.logismos_launch_depth_mix_conv_decode(_p(hist), rows * ld, j, _p(coef), _p(x), _p(gain), _p(w1), _p(w2), _p(o[0]), _p(o[1]),
+                                                        int(out_f32), _p(state), _p(state_slots), _p(fresh), _p(phase), rows, n, ld, float(eps),
+                                                        state.shape[2] + 1, _stream()), "depth_mix_conv_decode")
+        _done(sync)
+    return x, o[0], o[1]
+
+
+def latent_norm_store(raw, gain_q, gain_c, pool, slot_mapping, q_n, c_n, eps, sync=True):
+    """raw fp32 [rows, q width + c width] -> normed query latents; the normed key/value latents go to ``pool``
+    [blocks, 16, c width] (bf16 or fp32, which also sets the type of the result)."""
+    _req(raw, "raw", torch.float32, 2); _req(slot_mapping, "slot_mapping", torch.int64, 1)
+    rows, qw, cw = raw.shape[0], gain_q.numel(), gain_c.numel()
+    cq = torch.empty((rows, qw), dtype=pool.dtype, device=raw.device)
+    status = torch.zeros(1, dtype=torch.int32, device=raw.device)
+    with torch.cuda.device(raw.device):
+        check(lib.logismos_launch_latent_norm_store(_p(raw), raw.shape[1], _p(gain_q), _p(gain_c), _p(cq), _p(pool), _p(slot_mapping), rows, qw, q_n,
+                                                    cw, c_n, float(eps), pool.shape[0] * 16, int(pool.dtype == torch.float32), _p(status), _stream()),
+              "latent_norm_store")
+        _done(sync)
+        if sync and int(status.item()) != 0:
+            raise InvalidOp("latent_norm_store: slot outside the pool")
+    return cq
+
+
+def latent_gather(pool, block_tables, kv_lens, kv_lens_host, sync=True):
+    """-> (rows bf16 [gather rows, width], kv_start int32 [n_seqs])."""
+    _req(pool, "pool", torch.bfloat16, 3); _req(block_tables, "block_tables", torch.int32, 2)
+    total, n, mx = int(sum(kv_lens_host)), len(kv_lens_host), int(max(kv_lens_host))
+    out = torch.empty((lib.logismos_latent_gather_rows(total, n), pool.shape[2]), dtype=torch.bfloat16, device=pool.device)
+    start = torch.empty(n, dtype=torch.int32, device=pool.device)
+    status = torch.zeros(1, dtype=torch.int32, device=pool.device)
+    with torch.cuda.device(pool.device):
+        check(lib.logismos_launch_latent_gather_bf16(_p(pool), _p(block_tables), block_tables.shape[1], pool.shape[0], _p(kv_lens), _p(out), _p(start),
+                                                     total, n, mx, pool.shape[2], _p(status), _stream()), "latent_gather")
+        _done(sync)
+        if sync and int(status.item()) != 0:
+            raise InvalidOp("latent_gather: a block id fell outside the pool")
+    return out, start
+
+
+def attention_kv(q, k, v_t, cu_seqlens_q, kv_lens, kv_start, n_heads, n_kv_heads, head_dim, scale, max_q_len, sync=True):
+    """Causal attention over contiguous keys [rows, n_kv_heads * head_dim] and transposed values."""
+    _req(q, "q", torch.bfloat16, 2); _req(k, "k", torch.bfloat16, 2); _req(v_t, "v_t", torch.bfloat16, 2)
+    out = torch.empty((q.shape[0], n_heads * head_dim), dtype=torch.bfloat16, device=q.device)
+    status = torch.zeros(1, dtype=torch.int32, device=q.device)
+    with torch.cuda.device(q.device):
+        check(lib.logismos_launch_varlen_attention_kv_tc_bf16(_p(q), q.shape[1], _p(cu_seqlens_q), _p(kv_lens), _p(kv_start), _p(k), _p(v_t), k.shape[0],
+                                                              _p(out), out.shape[1], q.shape[0], kv_lens.numel(), max_q_len, n_heads, n_kv_heads,
+                                                              head_dim, float(scale), _p(status), _stream()), "attention_kv")
+        _done(sync)
+        if sync and int(status.item()) != 0:
+            raise InvalidOp(f"attention_kv: device status {int(status.item())}")
+    return out
+
+
+def latent_decode(q, pool, block_tables, context_lens, context_lens_host, scale, chunk_tokens=0, scratch=None, sync=True):
+    """q bf16 [rows, heads, rank] over cached latents bf16 [blocks, 16, rank]; chunk_tokens 0: the library's choice."""
+    _req(q, "q", torch.bfloat16, 3); _req(pool, "pool", torch.bfloat16, 3); _req(block_tables, "block_tables", torch.int32, 2)
+    rows, heads, rank = q.shape
+    cl = torch.as_tensor(context_lens_host, dtype=torch.int32).contiguous()
+    chunk = chunk_tokens or int(lib.logismos_pick_latent_chunk(C.c_void_p(cl.data_ptr()), rows, heads))
+    off, total = build_decode_chunks(cl, chunk)
+    off = off.to(q.device)
+    out = torch.empty_like(q)
+    if scratch is None:
+        scratch = torch.empty(lib.logismos_latent_decode_scratch_bytes(total, heads, rank), dtype=torch.uint8, device=q.device)
+    status = torch.zeros(1, dtype=torch.int32, device=q.device)
+    with torch.cuda.device(q.device):
+        check(lib.logismos_launch_latent_decode_bf16(_p(q), _p(pool), _p(block_tables), _p(context_lens), _p(off), _p(out), _p(scratch), rows, total,
+                                                     chunk, block_tables.shape[1], pool.shape[0], heads, rank, float(scale), _p(status), _stream()),
+              "latent_decode")
+        _done(sync)
+        if sync and int(status.item()) != 0:
+            raise InvalidOp("latent_decode: a block id fell outside the pool")
+    return out
+
+
+def latent_attention_f32(q, pool, block_tables, seq_ids, positions, scale, sync=True):
+    """fp32 [rows, heads, rank]; row t of sequence seq_ids[t] sees keys 0 .. positions[t]."""
+    _req(q, "q", torch.float32, 3); _req(pool, "pool", torch.float32, 3)
+    out = torch.empty_like(q)
+    status = torch.zeros(1, dtype=torch.int32, device=q.device)
+    with torch.cuda.device(q.device):
+        check(lib.logismos_launch_latent_attention_f32(_p(q), _p(pool), _p(block_tables), _p(seq_ids), _p(positions), _p(out), q.shape[0],
+                                                       block_tables.shape[1], pool.shape[0], q.shape[1], q.shape[2], float(scale), _p(status), _stream()),
+              "latent_attention_f32")
+        _done(sync)
+        if sync and int(status.item()) != 0:
+            raise InvalidOp("latent_attention_f32: a block id fell outside the pool")
+    return out
