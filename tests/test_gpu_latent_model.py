@@ -78,9 +78,9 @@ class Harness:
             at += len(t)
         return z
 
-    def compare(self, z, ref, what, scale=None):
+    def compare(self, z, ref, what, scale=None, factor=1.0):
         err = np.sqrt(np.mean((z - ref) ** 2, axis=1)) / np.sqrt(np.mean((ref if scale is None else scale) ** 2))
-        assert err.max() <= TOLS[self.dtype], (what, int(err.argmax()), float(err.max()))
+        assert err.max() <= factor * TOLS[self.dtype], (what, int(err.argmax()), float(err.max()))
 
     def drop(self, sid):
         self.blocks.release(sid); self.slots.release(sid); self.hist.pop(sid)
@@ -120,7 +120,7 @@ def test_prompt_portions_and_decoding_agree(name, dtype):
     h.drop("one")
     for t in range(40):
         z = h.run([("d", prompt[t:t + 1])])
-        h.compare(z, whole[t:t + 1], ("decoded against prompt", t), whole)
+        h.compare(z, whole[t:t + 1], ("decoded against prompt", t), whole, factor=2.0)   # both sides are rounded
     h.drop("w")
     for k, cuts in enumerate(([2] * 10 + [130], [15, 1, 1, 16, 17, 3, 97], [63, 2, 64, 21], [128, 2, 20], [149, 1])):
         at = 0
