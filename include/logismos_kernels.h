@@ -543,7 +543,9 @@ uint32_t logismos_launch_norm_conv(const void* x_f32, const void* inv_rms_f32, c
                                    void* state_f32, const void* state_slots_i32, const void* fresh_u8,
                                    const void* phase_u8, const void* seq_ids_i32, const void* cu_seqlens_i32,
                                    int32_t rows, int32_t ld, int32_t taps, void* stream);
-/* Both of the above in one launch for a step whose sequences bring one token each (row = sequence). */
+/* Both of the above in one launch for a step whose sequences bring one token each (row = sequence). gain, w1,
+ * w2, the state and the three index arrays must not be written by work still in flight on the stream (they
+ * may be read ahead of the dependency wait). */
 uint32_t logismos_launch_depth_mix_conv_decode(const void* hist_f32, int64_t hist_stride, int32_t n_hist,
                                                const void* coef_f32, void* x_f32, const void* gain_f32,
                                                const void* w1_f32, const void* w2_f32, void* o1, void* o2,
@@ -573,7 +575,9 @@ uint32_t logismos_launch_latent_gather_bf16(const void* pool, const void* block_
  * c_j over the first context_lens[r] cached rows. q, out bf16 [rows, heads, rank]; rank % 64 == 0, rank <=
  * 1024. chunk_offsets as for the paged decode kernel, with chunk_tokens % 64 == 0
  * (logismos_pick_latent_chunk, whose choice leaves at most logismos_latent_max_chunks(rows) chunks). scratch:
- * logismos_latent_decode_scratch_bytes(total_chunks, heads, rank). A second launch merges split contexts. */
+ * logismos_latent_decode_scratch_bytes(total_chunks, heads, rank). A second launch merges split contexts. The
+ * index arrays, and every cached row but the last of each context, must not be written by work still in
+ * flight on the stream (they may be read ahead of the dependency wait). */
 int32_t logismos_pick_latent_chunk(const int32_t* host_context_lens, int32_t n_seqs, int32_t heads);
 int32_t logismos_latent_max_chunks(int32_t max_rows);
 size_t logismos_latent_decode_scratch_bytes(int32_t total_chunks, int32_t heads, int32_t rank);

@@ -115,7 +115,7 @@ LG_DEVINL float block_max(float v, float* red) {
 LG_DEVINL float glu_clamp(float g, float u, float alpha, float limit, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return g / (1.0f + __expf(-alpha * g)) * (u + shift);
+  return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + shift);
 }
 
 LG_DEVINL uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }

@@ -14,7 +14,7 @@ namespace {
 
 using namespace lg;
 
-constexpr int kMaxVec = 8;   // float4 per thread and row
+constexpr int kMaxThreads = 512, kMaxVec = 8;   // float4 per thread and row: 1, 2, 4 or 8
 constexpr int kMaxTaps = 8;
 
 LG_DEVINL float4 fma4(float a, float4 x, float4 c) { return make_float4(fmaf(a, x.x, c.x), fmaf(a, x.y, c.y), fmaf(a, x.z, c.z), fmaf(a, x.w, c.w)); }
@@ -41,28 +41,40 @@ struct MixArgs {
   int* status;
 };
 
-// the row sum of one CTA: acc[i] holds float4 tid + i * blockDim of the row
-LG_DEVINL void mix_row(const MixArgs& p, int src, float4 (&acc)[kMaxVec], float& ss) {
+// the row sum of one CTA: acc[i] holds float4 tid + i * blockDim of the row; about eight loads in flight per thread
+template <int NV>
+LG_DEVINL void mix_row(const MixArgs& p, int src, float4 (&acc)[NV], float& ss) {
+  constexpr int kAhead = NV >= 8 ? 1 : 8 / NV;
   const int nv = p.ld >> 2;
 #pragma unroll
-  for (int i = 0; i < kMaxVec; ++i) acc[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int i = 0; i < NV; ++i) acc[i] = make_float4(0.f, 0.f, 0.f, 0.f);
   const float* base = p.hist + (size_t)src * p.ld;
-#pragma unroll 4
-  for (int j = 0; j < p.n_hist; ++j) {
-    const float c = __ldg(p.coef + j);
-    const float4* row = reinterpret_cast<const float4*>(base + (size_t)j * p.hist_stride);
+  for (int j0 = 0; j0 < p.n_hist; j0 += kAhead) {
+    float4 x[kAhead][NV];
+    float c[kAhead];
 #pragma unroll
-    for (int i = 0; i < kMaxVec; ++i) {
-      const int v = threadIdx.x + i * blockDim.x;
-      if (v < nv) acc[i] = fma4(c, row[v], acc[i]);
+    for (int a = 0; a < kAhead; ++a) {
+      const bool in = j0 + a < p.n_hist;
+      c[a] = in ? __ldg(p.coef + j0 + a) : 0.0f;
+      const float4* row = reinterpret_cast<const float4*>(base + (size_t)(j0 + a) * p.hist_stride);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+        x[a][i] = in && v < nv ? row[v] : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
     }
+#pragma unroll
+    for (int a = 0; a < kAhead; ++a)
+#pragma unroll
+      for (int i = 0; i < NV; ++i) acc[i] = fma4(c[a], x[a][i], acc[i]);
   }
   ss = 0.0f;
 #pragma unroll
-  for (int i = 0; i < kMaxVec; ++i) ss += acc[i].x * acc[i].x + acc[i].y * acc[i].y + acc[i].z * acc[i].z + acc[i].w * acc[i].w;
+  for (int i = 0; i < NV; ++i) ss += acc[i].x * acc[i].x + acc[i].y * acc[i].y + acc[i].z * acc[i].z + acc[i].w * acc[i].w;
 }
 
-__global__ void __launch_bounds__(512)
+template <int NV>
+__global__ void __launch_bounds__(kMaxThreads)
 depth_mix_kernel(MixArgs p) {
   lg::pdl_prologue();
   __shared__ float red[32];
@@ -72,13 +84,13 @@ depth_mix_kernel(MixArgs p) {
     if (threadIdx.x == 0 && p.status) atomicExch(p.status, 1);
     src = 0;
   }
-  float4 acc[kMaxVec];
+  float4 acc[NV];
   float ss;
-  mix_row(p, src, acc, ss);
+  mix_row<NV>(p, src, acc, ss);
   const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.n + p.eps);
   if (p.inv_rms && threadIdx.x == 0) p.inv_rms[r] = inv;
 #pragma unroll
-  for (int i = 0; i < kMaxVec; ++i) {
+  for (int i = 0; i < NV; ++i) {
     const int v = threadIdx.x + i * blockDim.x;
     if (v >= nv) continue;
     if (p.x) reinterpret_cast<float4*>(p.x)[(size_t)r * nv + v] = acc[i];
@@ -99,37 +111,54 @@ struct ConvArgs {
   int taps;
 };
 
-// Depth average, norm and convolution of a step whose sequences bring one token each (row r = sequence r).
-__global__ void __launch_bounds__(512)
+// Depth average, norm and convolution of a step whose sequences bring one token each (row r = sequence r). Gains,
+// filters and the state (left by an earlier step) do not depend on the kernels before this one in the step, so
+// with one float4 per thread they are read ahead of the dependency wait.
+template <int NV, int TAPS>
+__global__ void __launch_bounds__(kMaxThreads)
 depth_mix_conv_decode_kernel(MixArgs p, ConvArgs c) {
-  lg::pdl_prologue();
+  lg::pdl_trigger();
+  constexpr int HN = TAPS - 1;
   __shared__ float red[32];
-  const int r = blockIdx.x, nv = p.ld >> 2, hist = c.taps - 1;
-  float4 acc[kMaxVec];
-  float ss;
-  mix_row(p, r, acc, ss);
-  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.n + p.eps);
+  const int r = blockIdx.x, nv = p.ld >> 2;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   const bool fresh = c.fresh[r] != 0;
-  float4* slot = reinterpret_cast<float4*>(c.state) + (size_t)c.state_slots[r] * 2 * hist * nv;
+  float4* slot = reinterpret_cast<float4*>(c.state) + (size_t)c.state_slots[r] * 2 * HN * nv;
   const int ph = c.phase[r] & 1;
-  const float4* old = slot + (size_t)ph * hist * nv;
-  float4* next = slot + (size_t)(1 - ph) * hist * nv;
+  const float4* old = slot + (size_t)ph * HN * nv;
+  float4* next = slot + (size_t)(1 - ph) * HN * nv;
+  float4 gain = zero, w1[TAPS], w2[TAPS], prev[HN > 0 ? HN : 1];
+  auto fetch = [&](int v) {
+    gain = __ldg(reinterpret_cast<const float4*>(c.gain) + v);
 #pragma unroll
-  for (int i = 0; i < kMaxVec; ++i) {
+    for (int j = 0; j < TAPS; ++j) {
+      w1[j] = c.w1 ? __ldg(reinterpret_cast<const float4*>(c.w1) + (size_t)j * nv + v) : zero;
+      w2[j] = c.w2 ? __ldg(reinterpret_cast<const float4*>(c.w2) + (size_t)j * nv + v) : zero;
+    }
+#pragma unroll
+    for (int j = 0; j < HN; ++j) prev[j] = fresh ? zero : old[(size_t)j * nv + v];
+  };
+  if (NV == 1 && (int)threadIdx.x < nv) fetch(threadIdx.x);
+  lg::pdl_wait();
+  float4 acc[NV];
+  float ss;
+  mix_row<NV>(p, r, acc, ss);
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.n + p.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
     const int v = threadIdx.x + i * blockDim.x;
     if (v >= nv) continue;
+    if (NV > 1) fetch(v);
     reinterpret_cast<float4*>(p.x)[(size_t)r * nv + v] = acc[i];
-    const float4 h = mul4(inv, acc[i], __ldg(reinterpret_cast<const float4*>(c.gain) + v));
-    float4 y1 = h, y2 = h;
-    if (c.w1) y1 = fma4(__ldg(reinterpret_cast<const float4*>(c.w1) + (size_t)hist * nv + v), h, y1);
-    if (c.w2) y2 = fma4(__ldg(reinterpret_cast<const float4*>(c.w2) + (size_t)hist * nv + v), h, y2);
-    for (int j = 0; j < hist; ++j) {
-      const float4 q = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : old[(size_t)j * nv + v];
-      if (c.w1) y1 = fma4(__ldg(reinterpret_cast<const float4*>(c.w1) + (size_t)j * nv + v), q, y1);
-      if (c.w2) y2 = fma4(__ldg(reinterpret_cast<const float4*>(c.w2) + (size_t)j * nv + v), q, y2);
-      if (j > 0) next[(size_t)(j - 1) * nv + v] = q;
+    const float4 h = mul4(inv, acc[i], gain);
+    float4 y1 = fma4(w1[TAPS - 1], h, h), y2 = fma4(w2[TAPS - 1], h, h);
+#pragma unroll
+    for (int j = 0; j < HN; ++j) {
+      y1 = fma4(w1[j], prev[j], y1);
+      y2 = fma4(w2[j], prev[j], y2);
+      if (j > 0) next[(size_t)(j - 1) * nv + v] = prev[j];
     }
-    if (hist > 0) next[(size_t)(hist - 1) * nv + v] = h;
+    if (HN > 0) next[(size_t)(HN > 0 ? HN - 1 : 0) * nv + v] = h;
     store4(c.o1, (size_t)r * nv + v, y1, p.f32);
     if (c.o2) store4(c.o2, (size_t)r * nv + v, y2, p.f32);
   }
@@ -198,13 +227,34 @@ norm_conv_kernel(const float* __restrict__ x, const float* __restrict__ inv_rms,
   }
 }
 
-int mix_threads(int ld) {
-  const int nv = ld / 4;
-  return nv <= 128 * 2 ? 128 : nv <= 256 * kMaxVec ? 256 : 512;
+// threads of a row and float4 per thread
+struct MixShape { int threads, nv; };
+MixShape mix_shape(int ld) {
+  const int v = ld / 4;
+  for (int nv = 1;; nv *= 2)
+    if (v <= kMaxThreads * nv) return {((v + nv - 1) / nv + 31) / 32 * 32, nv};
+}
+
+template <int NV>
+uint32_t launch_decode(const MixArgs& p, const ConvArgs& c, int threads, cudaStream_t s) {
+  auto go = [&](auto kern) {
+    lg::launch(kern, dim3((unsigned)p.rows), dim3((unsigned)threads), 0, s, p, c);
+    return lg::launch_status();
+  };
+  switch (c.taps) {
+    case 1: return go(depth_mix_conv_decode_kernel<NV, 1>);
+    case 2: return go(depth_mix_conv_decode_kernel<NV, 2>);
+    case 3: return go(depth_mix_conv_decode_kernel<NV, 3>);
+    case 4: return go(depth_mix_conv_decode_kernel<NV, 4>);
+    case 5: return go(depth_mix_conv_decode_kernel<NV, 5>);
+    case 6: return go(depth_mix_conv_decode_kernel<NV, 6>);
+    case 7: return go(depth_mix_conv_decode_kernel<NV, 7>);
+    default: return go(depth_mix_conv_decode_kernel<NV, 8>);
+  }
 }
 
 bool mix_ok(const void* hist, int n_hist, const void* coef, int rows, int n, int ld) {
-  return hist && coef && n_hist > 0 && rows > 0 && n > 0 && ld >= n && ld % 4 == 0 && ld / 4 <= 512 * kMaxVec;
+  return hist && coef && n_hist > 0 && rows > 0 && n > 0 && ld >= n && ld % 4 == 0 && ld / 4 <= kMaxThreads * kMaxVec;
 }
 
 }  // namespace
@@ -220,8 +270,12 @@ uint32_t logismos_launch_depth_mix_f32(const void* hist_f32, int64_t hist_stride
     return lg::kInvalidValue;
   const MixArgs p{(const float*)hist_f32, hist_stride, n_hist, (const float*)coef_f32, (const int*)row_idx_i32, n_src_rows, (float*)x_f32,
                   (float*)inv_rms_f32, (const float*)gain_f32, norm_out, rows, n, ld, out_f32, eps, (int*)status_i32};
-  lg::launch(depth_mix_kernel, dim3((unsigned)rows), dim3((unsigned)mix_threads(ld)), 0, (cudaStream_t)stream, p);
-  return lg::launch_status();
+  const MixShape sh = mix_shape(ld);
+  auto go = [&](auto kern) {
+    lg::launch(kern, dim3((unsigned)rows), dim3((unsigned)sh.threads), 0, (cudaStream_t)stream, p);
+    return lg::launch_status();
+  };
+  return sh.nv == 1 ? go(depth_mix_kernel<1>) : sh.nv == 2 ? go(depth_mix_kernel<2>) : sh.nv == 4 ? go(depth_mix_kernel<4>) : go(depth_mix_kernel<8>);
 }
 
 uint32_t logismos_launch_norm_conv(const void* x_f32, const void* inv_rms_f32, const void* gain_f32, const void* w1_f32,
@@ -263,8 +317,10 @@ uint32_t logismos_launch_depth_mix_conv_decode(const void* hist_f32, int64_t his
                   nullptr, nullptr, rows, n, ld, out_f32, eps, nullptr};
   const ConvArgs c{(const float*)gain_f32, (const float*)w1_f32, (const float*)w2_f32, o1, o2, (float*)state_f32, (const int*)state_slots_i32,
                    (const uint8_t*)fresh_u8, (const uint8_t*)phase_u8, taps};
-  lg::launch(depth_mix_conv_decode_kernel, dim3((unsigned)rows), dim3((unsigned)mix_threads(ld)), 0, (cudaStream_t)stream, p, c);
-  return lg::launch_status();
+  const MixShape sh = mix_shape(ld);
+  cudaStream_t s = (cudaStream_t)stream;
+  return sh.nv == 1 ? launch_decode<1>(p, c, sh.threads, s) : sh.nv == 2 ? launch_decode<2>(p, c, sh.threads, s)
+       : sh.nv == 4 ? launch_decode<4>(p, c, sh.threads, s) : launch_decode<8>(p, c, sh.threads, s);
 }
 
 }  // extern "C"

@@ -45,6 +45,17 @@ struct Cfg {
 
 LG_DEVINL float silu_f(float x) { return x / (1.0f + __expf(-x)); }
 
+// eight bias values (the same for every lane); vec: the pointer is 16-byte aligned
+LG_DEVINL void load_bias8(const float* __restrict__ bias, bool vec, float (&b)[8]) {
+  if (vec) {
+    const float4 x = __ldg(reinterpret_cast<const float4*>(bias)), y = __ldg(reinterpret_cast<const float4*>(bias) + 1);
+    b[0] = x.x; b[1] = x.y; b[2] = x.z; b[3] = x.w; b[4] = y.x; b[5] = y.y; b[6] = y.z; b[7] = y.w;
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) b[i] = __ldg(bias + i);
+  }
+}
+
 // constants of the parametrised epilogues (see LG_EPI_F32 and LG_EPI_GLU_CLAMP)
 struct EpiParams { float p0, p1, p2; };
 
@@ -169,6 +180,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
     uint8_t* slabs = smem_gen + C::kStages * C::kStage + q * 2 * 4096;
     const uint32_t slabs_a = epi_base + q * 2 * 4096;
     int it = 0, n_store = 0;
+    const bool bias_vec = (reinterpret_cast<uintptr_t>(bias) & 15) == 0;
     bool ok = true;
     // hands the slab just written to the TMA engine; the slab used two stores ago must have been read
     auto slab_acquire = [&]() -> int {
@@ -281,12 +293,16 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
               uint32_t w[4];
+              float bg[8] = {}, bu[8] = {};
+              if (bias) {
+                load_bias8(bias + ncol + j * 8, bias_vec, bg);
+                load_bias8(bias + ncol + 32 + j * 8, bias_vec, bu);
+              }
 #pragma unroll
               for (int i = 0; i < 4; ++i) {
                 const int e = j * 8 + i * 2;
-                float g0 = __uint_as_float(g[e]), g1 = __uint_as_float(g[e + 1]);
-                float u0 = __uint_as_float(u[e]), u1 = __uint_as_float(u[e + 1]);
-                if (bias) { g0 += bias[ncol + e]; g1 += bias[ncol + e + 1]; u0 += bias[ncol + 32 + e]; u1 += bias[ncol + 32 + e + 1]; }
+                const float g0 = __uint_as_float(g[e]) + bg[2 * i], g1 = __uint_as_float(g[e + 1]) + bg[2 * i + 1];
+                const float u0 = __uint_as_float(u[e]) + bu[2 * i], u1 = __uint_as_float(u[e + 1]) + bu[2 * i + 1];
                 if (EPI == LG_EPI_GLU_CLAMP) w[i] = pack_bf16x2(lg::glu_clamp(g0, u0, ep.p0, ep.p1, ep.p2), lg::glu_clamp(g1, u1, ep.p0, ep.p1, ep.p2));
                 else w[i] = pack_bf16x2(silu_f(g0) * u0, silu_f(g1) * u1);
               }

@@ -431,7 +431,7 @@ uint32_t lg_hybrid_step(void* model, const uint32_t* host_ids, const int32_t* ca
   for (int k = 0; k < n_seqs; ++k) next_tokens[B.order[k]] = toks[k];
   if (const int dev_status = lg_hybrid_device_status(m)) {
     m->acc_dirty = true;
-    char buf[160];
+    char buf[256];
     std::snprintf(buf, sizeof(buf), "device status 0x%x after a step of %d tokens in %d sequences (low byte 1: a range check failed, 2: a bounded wait expired in kernel family <next byte>, 3: a peer did not arrive)",
                   dev_status, (int)total, n_seqs);
     set_error(buf);

@@ -7,19 +7,32 @@
 //   latent_decode       one query token per sequence in the latent space: with q'_h = W_uk,h^T q_h the
 //                       score of a key is q'_h . c and the output is W_uv,h (sum_j p_j c_j), so every head
 //                       shares the same rank-wide key = value row and a cached row is read once for all
-// latent_decode splits the contexts in chunks; CTA = (chunk, group of 16 * MT heads), 8 warps, tiles of
-// TK tokens in a two-stage cp.async ring (16-byte chunks XOR-swizzled by row). Per tile: S = Q' C^T
-// (mma.sync, a warp per 8 tokens), running maximum and sum in fp32 (exp2 domain), P rounded to bf16,
-// O += P C (a warp per rank / 8 columns, C through ldmatrix.trans). Partial results are merged by a
-// second kernel; a context that is one chunk is finished in place.
+// latent_decode splits the contexts in chunks; CTA = (chunk, group of 16 * MT heads), 8 warps, tiles of TK tokens. A cache block (16 tokens) arrives as rank / 64 TMA boxes of 16 rows
+// x 128 bytes (128-byte swizzle) in a ring of stages, so ldmatrix reads are conflict-free and no thread computes
+// addresses of cached rows; warp 0 refills the stage of the previous tile once every warp has passed the
+// current tile's first barrier. Per tile: partial scores S = Q' C^T (mma.sync; a warp takes half of the tokens and a
+// quarter of the rank, its query fragments stay in registers), summed in shared memory in a fixed order; running
+// maximum and sum in fp32 (exp2 domain); P rounded to bf16; O += P C (a warp per slice of the rank, C through
+// ldmatrix.trans). Partial results are merged by a second kernel; a context that is one chunk is finished in
+// place. Every mbarrier wait is bounded: on expiry the status word is raised and the kernel returns.
+#include <cuda.h>
+
 #include "common.cuh"
 #include "logismos_kernels.h"
+#include "tcgen05.cuh"
 
 namespace {
 
 using namespace lg;
+using namespace lg::tc;
 
 constexpr float kLog2e = 1.4426950408889634f;
+
+LG_DEVINL float fast_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
 constexpr int kBlockTokens = 16;
 constexpr int kThreads = 256;
 
@@ -65,46 +78,38 @@ latent_norm_store_kernel(const float* __restrict__ raw, int ld, const float* __r
 LG_DEVINL int round8(int v) { return (v + 7) & ~7; }
 
 // rows of sequence s -> out[pstart[s] ..], every sequence starting at a multiple of 8 rows, padding and
-// the rows after the last sequence zeroed up to tp. Grid (row blocks of 64, sequences).
+// the rows after the last sequence zeroed up to tp. Grid (cache blocks, sequences); a warp copies two rows.
 __global__ void __launch_bounds__(kThreads)
 latent_gather_kernel(const __nv_bfloat16* __restrict__ pool, const int* __restrict__ tables, int max_blocks, int n_pool_blocks,
                      const int* __restrict__ kv_lens, __nv_bfloat16* __restrict__ out, int* __restrict__ pstart, int n_seqs, int tp,
                      int rw, int* __restrict__ status) {
   lg::pdl_prologue();
-  __shared__ int p0_s;
-  const int tb = blockIdx.x, s = blockIdx.y, tid = threadIdx.x;
-  if (tid < 32) {
-    int part = 0;
-    for (int i = tid; i < s; i += 32) part += round8(max(kv_lens[i], 0));
+  const int tb = blockIdx.x, s = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int len = max(kv_lens[s], 0), plen = round8(len), cw = rw >> 3;
+  const bool tail = tb == 0 && s == n_seqs - 1;
+  if (tb * kBlockTokens >= plen && !tail && tb > 0) return;
+  int p0 = 0;
+  for (int i = lane; i < s; i += 32) p0 += round8(max(kv_lens[i], 0));
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) part += __shfl_xor_sync(0xffffffffu, part, o);
-    if (tid == 0) p0_s = part;
-  }
-  __syncthreads();
-  const int p0 = p0_s, len = max(kv_lens[s], 0), plen = round8(len), cw = rw >> 3;
+  for (int o = 16; o > 0; o >>= 1) p0 += __shfl_xor_sync(0xffffffffu, p0, o);
   if (p0 + plen > tp) {
-    if (tid == 0 && status) atomicExch(status, 1);
+    if (threadIdx.x == 0 && status) atomicExch(status, 1);
     return;
   }
-  if (tb == 0 && tid == 0) pstart[s] = p0;
-  if (tb == 0 && s == n_seqs - 1)
-    for (int64_t u = tid; u < (int64_t)(tp - p0 - plen) * cw; u += kThreads)
+  if (tb == 0 && threadIdx.x == 0) pstart[s] = p0;
+  if (tail)
+    for (int64_t u = threadIdx.x; u < (int64_t)(tp - p0 - plen) * cw; u += kThreads)
       reinterpret_cast<uint4*>(out)[(size_t)(p0 + plen) * cw + u] = make_uint4(0u, 0u, 0u, 0u);
-  if (tb * 64 >= plen) return;
-  for (int u = tid; u < 64 * cw; u += kThreads) {
-    const int t = tb * 64 + u / cw, ch = u % cw;
+  const int blk = tb < max_blocks && tb * kBlockTokens < len ? __ldg(tables + (size_t)s * max_blocks + tb) : -1;
+  const bool ok = blk >= 0 && blk < n_pool_blocks;
+  if (!ok && tb * kBlockTokens < len && threadIdx.x == 0 && status) atomicExch(status, 1);
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int r = warp * 2 + h, t = tb * kBlockTokens + r;
     if (t >= plen) break;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (t < len) {
-      const int bi = t / kBlockTokens;
-      const int blk = bi < max_blocks ? __ldg(tables + (size_t)s * max_blocks + bi) : -1;
-      if (blk < 0 || blk >= n_pool_blocks) {
-        if (ch == 0 && status) atomicExch(status, 1);
-      } else {
-        v = reinterpret_cast<const uint4*>(pool)[((size_t)blk * kBlockTokens + t % kBlockTokens) * cw + ch];
-      }
-    }
-    reinterpret_cast<uint4*>(out)[(size_t)(p0 + t) * cw + ch] = v;
+    uint4* dst = reinterpret_cast<uint4*>(out) + (size_t)(p0 + t) * cw;
+    const uint4* src = reinterpret_cast<const uint4*>(pool) + ((size_t)(ok ? blk : 0) * kBlockTokens + r) * cw;
+    for (int c = lane; c < cw; c += 32) dst[c] = ok && t < len ? src[c] : make_uint4(0u, 0u, 0u, 0u);
   }
 }
 
@@ -122,194 +127,279 @@ struct DecodeArgs {
   int* status;
 };
 
-// row r with chunk_offsets[r] <= chunk < chunk_offsets[r + 1]
-LG_DEVINL int find_row(const int* __restrict__ off, int rows, int chunk) {
-  int lo = 0, hi = rows - 1;
-  while (lo < hi) {
-    const int mid = (lo + hi + 1) >> 1;
-    if (__ldg(off + mid) <= chunk) lo = mid;
-    else hi = mid - 1;
-  }
-  return lo;
+constexpr int kMaxStages = 4;
+constexpr int kWarps = 8;
+constexpr int kDecodeThreads = 32 * kWarps;
+
+// shared memory besides the ring: query rows (when they do not stay in registers), partial scores, P, row state
+template <int MT, int TK, bool QREG>
+__host__ __device__ constexpr size_t decode_fixed_smem(int rank) {
+  return (QREG ? 0 : (size_t)16 * MT * rank * 2) + (size_t)4 * 16 * MT * (TK + 8) * 4 + (size_t)16 * MT * (TK + 8) * 2 + (size_t)16 * MT * 3 * 4 +
+         8 * (kMaxStages + 2) + 1024;
 }
 
-template <int MT, int TK>
-__host__ __device__ constexpr size_t decode_smem(int rank) {
-  return (size_t)(16 * MT + 2 * TK) * rank * 2 + (size_t)16 * MT * (TK + 4) * 4 + (size_t)16 * MT * (TK + 8) * 2 + (size_t)16 * MT * 3 * 4;
-}
-
-template <int MT, int MAXNT, int TK>
-__global__ void __launch_bounds__(kThreads)
-latent_decode_kernel(DecodeArgs p) {
-  lg::pdl_prologue();
-  extern __shared__ __align__(128) uint8_t smem[];
-  constexpr int kRows = 16 * MT;
-  const int R = p.rank, cw = R >> 3, row_bytes = R * 2, nt_n = R >> 6;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
-  const uint32_t sq = smem_u32(smem), sc = sq + (uint32_t)kRows * row_bytes;
-  uint8_t* after = smem + (size_t)(kRows + 2 * TK) * row_bytes;
-  float* s_s = reinterpret_cast<float*>(after);                             // [kRows][TK + 4]
-  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_s + kRows * (TK + 4));  // [kRows][TK + 8]
+// MAXKS >= rank / 64: k16 steps of one rank quarter; also the 64-column slabs
+template <int MT, int MAXKS, int TK, bool QREG>
+__global__ void __launch_bounds__(kDecodeThreads, MT == 1 && MAXKS <= 8 ? 2 : 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p, int stages) {
+  lg::pdl_trigger();
+  extern __shared__ uint8_t smem_raw[];
+  constexpr int kRows = 16 * MT, NTS = TK / 16;               // n8 tiles of a token half
+  constexpr int MAXU = (MAXKS * 4 + kWarps - 1) / kWarps;     // 16-column units of the rank per warp
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* gen = smem_raw + (base - smem_u32(smem_raw));
+  const int R = p.rank, slabs = R >> 6, tile_bytes = TK * R * 2;
+  uint8_t* after = gen + (size_t)stages * tile_bytes;
+  const uint32_t sq = smem_u32(after);                        // [kRows][R] swizzled, when !QREG
+  float* s_part = reinterpret_cast<float*>(after + (QREG ? 0 : (size_t)kRows * R * 2));  // [4][kRows][TK + 8]
+  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_part + 4 * kRows * (TK + 8));   // [kRows][TK + 8]
   float* s_m = reinterpret_cast<float*>(s_p + kRows * (TK + 8));
   float* s_l = s_m + kRows;
   float* s_a = s_l + kRows;
-  const uint32_t sp = smem_u32(s_p);
-  auto swz = [&](uint32_t base, int row, int chunk) { return base + (uint32_t)row * row_bytes + (uint32_t)((chunk ^ (row & 7)) << 4); };
-
+  uint8_t* bars_gen = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(s_a + kRows) + 7) & ~(uintptr_t)7);
+  const uint32_t bars = smem_u32(bars_gen);
+  auto full_bar = [&](int i) { return bars + 8u * i; };
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars_gen + 8 * kMaxStages);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < stages; ++i) mbar_init(full_bar(i), 1);
+    *abort_flag = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+    asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+  }
+  // Index arrays date from before the step's first kernel, and so do all cached rows but this step's new token
+  // (the last of each context): both are read ahead of the dependency wait.
   const int chunk = blockIdx.x, h0 = blockIdx.y * kRows;
-  const int r = find_row(p.chunk_offsets, p.rows, chunk);
-  const int c_idx = chunk - __ldg(p.chunk_offsets + r), c_cnt = __ldg(p.chunk_offsets + r + 1) - __ldg(p.chunk_offsets + r);
-  const int ctx = p.ctx[r];
+  int r = 0;  // chunk_offsets[r] <= chunk < chunk_offsets[r + 1]
+  for (int i0 = 0; i0 < p.rows; i0 += kDecodeThreads) {
+    const int i = i0 + threadIdx.x;
+    r += __syncthreads_count(i < p.rows && __ldg(p.chunk_offsets + i + 1) <= chunk);
+  }
+  const int c0 = __ldg(p.chunk_offsets + r), c_idx = chunk - c0, c_cnt = __ldg(p.chunk_offsets + r + 1) - c0;
+  const int ctx = __ldg(p.ctx + r);
   const int k0 = c_idx * p.chunk_tokens, k1 = min(ctx, k0 + p.chunk_tokens);
   const int tiles = (k1 - k0 + TK - 1) / TK;
+  // Tile ti of the chunk into its stage (warp 0, tiles in order): lane = 64-column slab of the rank. Lane b holds the
+  // id of the tile's block b, read one tile ahead.
   const int* table = p.tables + (size_t)r * p.max_blocks;
-
-  // query rows of this head group (heads beyond the last are zero rows)
-  for (int u = threadIdx.x; u < kRows * cw; u += kThreads) {
-    const int hr = u / cw, ch = u % cw;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (h0 + hr < p.heads) v = *reinterpret_cast<const uint4*>(p.q + ((size_t)r * p.heads + h0 + hr) * R + ch * 8);
-    *reinterpret_cast<uint4*>(smem + (swz(sq, hr, ch) - sq)) = v;
-  }
-  for (int i = threadIdx.x; i < kRows; i += kThreads) { s_m[i] = -1e30f; s_l[i] = 0.0f; }
-
-  auto load_tile = [&](int ti) {
-    const uint32_t base = sc + (uint32_t)(ti & 1) * TK * row_bytes;
-    for (int u = threadIdx.x; u < TK * cw; u += kThreads) {
-      const int kr = u / cw, ch = u % cw, key = k0 + ti * TK + kr;
-      const uint32_t dst = swz(base, kr, ch);
-      int blk = -1;
-      if (key < k1) {
-        const int bi = key / kBlockTokens;
-        blk = bi < p.max_blocks ? __ldg(table + bi) : -1;
-        if (blk < 0 || blk >= p.n_pool_blocks) {
-          if (ch == 0 && p.status) atomicExch(p.status, 1);
-          blk = -1;
-        }
-      }
-      if (blk >= 0) cp_async16(dst, p.pool + ((size_t)blk * kBlockTokens + key % kBlockTokens) * R + ch * 8);
-      else *reinterpret_cast<uint4*>(smem + (dst - sq)) = make_uint4(0u, 0u, 0u, 0u);
-    }
-    cp_async_commit();
+  auto block_id = [&](int ti) {
+    const int bi = (k0 + ti * TK) / kBlockTokens + lane;
+    return lane < TK / kBlockTokens && bi < p.max_blocks && bi * kBlockTokens < k1 ? __ldg(table + bi) : -1;
   };
-
-  float acc[MT][MAXNT][4];
-#pragma unroll
-  for (int i = 0; i < MT; ++i)
-#pragma unroll
-    for (int j = 0; j < MAXNT; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.0f;
-
-  load_tile(0);
-  for (int ti = 0; ti < tiles; ++ti) {
-    if (ti + 1 < tiles) {
-      load_tile(ti + 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
+  int ids = warp == 0 ? block_id(0) : -1;
+  auto fetch = [&](int ti) {
+    const int st = ti % stages, nb = min(TK, k1 - (k0 + ti * TK) + kBlockTokens - 1) / kBlockTokens;
+    if (lane == 0) mbar_expect_tx(full_bar(st), (uint32_t)(nb * kBlockTokens * R * 2));
+    __syncwarp();
+    if (lane < nb && (ids < 0 || ids >= p.n_pool_blocks)) {
+      if (p.status) atomicExch(p.status, 1);
+      ids = p.n_pool_blocks;  // beyond the pool: the copy fills zeros
     }
-    __syncthreads();
-    const uint32_t tile = sc + (uint32_t)(ti & 1) * TK * row_bytes;
-    // S = Q' C^T
-    if (warp < TK / 8) {
-      float s0[MT][4], s1[MT][4];
+#pragma unroll
+    for (int b = 0; b < TK / kBlockTokens; ++b) {
+      const int blk = __shfl_sync(0xffffffffu, ids, b);
+      if (b < nb && lane < slabs)
+        tma_load_2d(base + (uint32_t)st * tile_bytes + (uint32_t)lane * (TK * 128) + (uint32_t)b * (kBlockTokens * 128), &map_pool, full_bar(st), lane * 64,
+                    blk * kBlockTokens);
+    }
+    ids = block_id(ti + 1);
+  };
+  int fetched = 0;  // warp 0
+  auto prefetch = [&](bool all) {
+    while (fetched < stages && fetched < tiles && (all || k0 + (fetched + 1) * TK < ctx)) fetch(fetched++);
+  };
+  if (warp == 0) prefetch(false);
+  lg::pdl_wait();
+  if (warp == 0) prefetch(true);
+  if (threadIdx.x < kRows) { s_m[threadIdx.x] = -1e30f; s_l[threadIdx.x] = 0.0f; }
+  if (!QREG) {
+    const int cw = R >> 3;
+    for (int u = threadIdx.x; u < kRows * cw; u += kDecodeThreads) {
+      const int hr = u / cw, ch = u % cw;
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (h0 + hr < p.heads) v = *reinterpret_cast<const uint4*>(p.q + ((size_t)r * p.heads + h0 + hr) * R + ch * 8);
+      *reinterpret_cast<uint4*>(after + (size_t)hr * R * 2 + ((ch ^ (hr & 7)) << 4)) = v;
+    }
+  }
+  __syncthreads();
+
+  {
+    const int half = warp & 1, quarter = warp >> 1;
+    // query fragments of this warp's rank quarter
+    uint32_t qf[QREG ? MT : 1][QREG ? MAXKS : 1][4];
+    if (QREG) {
+#pragma unroll
+      for (int i = 0; i < (QREG ? MT : 1); ++i)
+#pragma unroll
+        for (int ks = 0; ks < (QREG ? MAXKS : 1); ++ks) {
+          const int col = (quarter * slabs + ks) * 16 + 2 * t4, ha = h0 + 16 * i + g;
+          const __nv_bfloat16* q0 = p.q + ((size_t)r * p.heads + ha) * R + col;
+          const bool in = ks < slabs;
+          qf[i][ks][0] = in && ha < p.heads ? *reinterpret_cast<const uint32_t*>(q0) : 0u;
+          qf[i][ks][1] = in && ha + 8 < p.heads ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)8 * R) : 0u;
+          qf[i][ks][2] = in && ha < p.heads ? *reinterpret_cast<const uint32_t*>(q0 + 8) : 0u;
+          qf[i][ks][3] = in && ha + 8 < p.heads ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)8 * R + 8) : 0u;
+        }
+    }
+    const int units = slabs * 4, u_per = (units + kWarps - 1) / kWarps, u0 = warp * u_per, u_n = max(0, min(units - u0, u_per));
+    float acc[MT][2 * MAXU][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int j = 0; j < 2 * MAXU; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.0f;
+    bool ok = true;
+    for (int ti = 0; ti < tiles; ++ti) {
+      const int st = ti % stages;
+      mbar_wait_warp(full_bar(st), (uint32_t)((ti / stages) & 1), abort_flag);  // a wait that expires sets the flag
+      const uint32_t tile = base + (uint32_t)st * tile_bytes;
+      // partial S = Q' C^T over this warp's quarter of the rank, half of the tokens
+      float s[MT][NTS][4];
 #pragma unroll
       for (int i = 0; i < MT; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) { s0[i][e] = 0.0f; s1[i][e] = 0.0f; }
-      for (int ks = 0; ks < (R >> 5); ++ks) {
-        uint32_t b[4];
-        ldmatrix_x4(b, swz(tile, 8 * warp + (lane & 7), 4 * ks + (lane >> 3)));
-        const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
+        for (int j = 0; j < NTS; ++j)
 #pragma unroll
-        for (int i = 0; i < MT; ++i) {
-          const int mat = lane >> 3, row = 16 * i + (lane & 7) + 8 * (mat & 1);
-          uint32_t a0[4], a1[4];
-          ldmatrix_x4(a0, swz(sq, row, 4 * ks + (mat >> 1)));
-          ldmatrix_x4(a1, swz(sq, row, 4 * ks + 2 + (mat >> 1)));
-          mma_bf16_16816(s0[i], a0, b0, s0[i]);
-          mma_bf16_16816(s1[i], a1, b1, s1[i]);
-        }
-      }
-      const int col = 8 * warp + 2 * t4, key = k0 + ti * TK + col;
-      const bool v0 = key < k1, v1 = key + 1 < k1;
+          for (int e = 0; e < 4; ++e) s[i][j][e] = 0.0f;
 #pragma unroll
-      for (int i = 0; i < MT; ++i) {
-        float* d0 = s_s + (16 * i + g) * (TK + 4) + col;
-        float* d1 = d0 + 8 * (TK + 4);
-        d0[0] = v0 ? (s0[i][0] + s1[i][0]) * p.sl2 : -1e30f;
-        d0[1] = v1 ? (s0[i][1] + s1[i][1]) * p.sl2 : -1e30f;
-        d1[0] = v0 ? (s0[i][2] + s1[i][2]) * p.sl2 : -1e30f;
-        d1[1] = v1 ? (s0[i][3] + s1[i][3]) * p.sl2 : -1e30f;
-      }
-    }
-    __syncthreads();
-    // running maximum and sum; a tile always holds at least one visible key, so the maximum is a real score
-    for (int row = warp; row < kRows; row += kThreads / 32) {
-      const float a = s_s[row * (TK + 4) + lane], b = TK > 32 ? s_s[row * (TK + 4) + 32 + lane] : -1e30f;
-      const float m_old = s_m[row], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
-      const float pa = exp2f(a - m_new), pb = TK > 32 ? exp2f(b - m_new) : 0.0f;
-      const float sum = warp_sum(pa + pb), alpha = exp2f(m_old - m_new);
-      s_p[row * (TK + 8) + lane] = __float2bfloat16_rn(pa);
-      if (TK > 32) s_p[row * (TK + 8) + 32 + lane] = __float2bfloat16_rn(pb);
-      __syncwarp();
-      if (lane == 0) { s_m[row] = m_new; s_l[row] = s_l[row] * alpha + sum; s_a[row] = alpha; }
-    }
-    __syncthreads();
-    // O = O * alpha + P C
-#pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const float a0 = s_a[16 * i + g], a1 = s_a[16 * i + g + 8];
-      if (a0 != 1.0f || a1 != 1.0f) {
-#pragma unroll
-        for (int j = 0; j < MAXNT; ++j) { acc[i][j][0] *= a0; acc[i][j][1] *= a0; acc[i][j][2] *= a1; acc[i][j][3] *= a1; }
-      }
-    }
-#pragma unroll
-    for (int ks = 0; ks < TK / 16; ++ks) {
-      uint32_t pa[MT][4];
-#pragma unroll
-      for (int i = 0; i < MT; ++i) {
-        const int mat = lane >> 3, row = 16 * i + (lane & 7) + 8 * (mat & 1);
-        ldmatrix_x4(pa[i], sp + (uint32_t)(row * (TK + 8) + 16 * ks + 8 * (mat >> 1)) * 2);
-      }
-#pragma unroll
-      for (int j = 0; j < MAXNT; j += 2) {
-        if (j < nt_n) {
-          const int ct = warp * nt_n + j + (lane >> 4);  // column tile; the odd one out is read but not used
-          uint32_t b[4];
-          ldmatrix_x4_trans(b, swz(tile, 16 * ks + (lane & 7) + 8 * ((lane >> 3) & 1), min(ct, cw - 1)));
-          const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
+      for (int ks = 0; ks < MAXKS; ++ks) {
+        if (ks < slabs) {
+          const int k16 = quarter * slabs + ks;
+          uint32_t a[MT][4];
 #pragma unroll
           for (int i = 0; i < MT; ++i) {
-            mma_bf16_16816(acc[i][j], pa[i], b0, acc[i][j]);
-            if (j + 1 < MAXNT && j + 1 < nt_n) mma_bf16_16816(acc[i][j + 1 < MAXNT ? j + 1 : j], pa[i], b1, acc[i][j + 1 < MAXNT ? j + 1 : j]);
+            if (QREG) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e) a[i][e] = qf[QREG ? i : 0][QREG ? ks : 0][e];
+            } else {
+              const int mat = lane >> 3, row = 16 * i + (lane & 7) + 8 * (mat & 1);
+              ldmatrix_x4(a[i], sq + (uint32_t)row * R * 2 + (uint32_t)(((2 * k16 + (mat >> 1)) ^ (row & 7)) << 4));
+            }
+          }
+#pragma unroll
+          for (int j = 0; j < NTS; j += 2) {
+            const int key = half * (TK / 2) + 8 * (j + (lane >> 4)) + (lane & 7);
+            const int ch = 2 * (k16 & 3) + ((lane >> 3) & 1);
+            uint32_t b[4];
+            ldmatrix_x4(b, tile + (uint32_t)(k16 >> 2) * (TK * 128) + (uint32_t)key * 128 + (uint32_t)((ch ^ (key & 7)) << 4));
+            const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
+#pragma unroll
+            for (int i = 0; i < MT; ++i) {
+              mma_bf16_16816(s[i][j], a[i], b0, s[i][j]);
+              mma_bf16_16816(s[i][j + 1], a[i], b1, s[i][j + 1]);
+            }
           }
         }
       }
-    }
-    __syncthreads();
-  }
 #pragma unroll
-  for (int i = 0; i < MT; ++i)
+      for (int i = 0; i < MT; ++i)
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int hr = 16 * i + g + 8 * half, h = h0 + hr;
-      if (h >= p.heads) continue;
-      const float inv = 1.0f / s_l[hr];
+        for (int j = 0; j < NTS; ++j) {
+          float* d = s_part + ((size_t)quarter * kRows + 16 * i + g) * (TK + 8) + half * (TK / 2) + 8 * j + 2 * t4;
+          *reinterpret_cast<float2*>(d) = make_float2(s[i][j][0], s[i][j][1]);
+          *reinterpret_cast<float2*>(d + 8 * (TK + 8)) = make_float2(s[i][j][2], s[i][j][3]);
+        }
+      __syncthreads();
+      if (*abort_flag) ok = false;  // set before this barrier or not at all during this tile: the same for every warp
+      if (warp == 0 && ti > 0 && ti - 1 + stages < tiles) fetch(ti - 1 + stages);
+      // running maximum and sum; a tile always holds at least one visible key, so the maximum is a real score
+      const int first = k0 + ti * TK;
 #pragma unroll
-      for (int j = 0; j < MAXNT; ++j) {
-        if (j >= nt_n) continue;
-        const int col = (warp * nt_n + j) * 8 + 2 * t4;
-        const float x = acc[i][j][2 * half], y = acc[i][j][2 * half + 1];
-        if (c_cnt == 1)
-          *reinterpret_cast<uint32_t*>(p.out + ((size_t)r * p.heads + h) * R + col) = pack_bf16x2(x * inv, y * inv);
-        else
-          *reinterpret_cast<float2*>(p.part_o + ((size_t)chunk * p.heads + h) * R + col) = make_float2(x, y);
+      for (int rr = 0; rr < 2 * MT; ++rr) {
+        const int row = warp + kWarps * rr;
+        float v[TK / 32];
+        float mx = -1e30f;
+#pragma unroll
+        for (int e = 0; e < TK / 32; ++e) {
+          const float* d = s_part + (size_t)row * (TK + 8) + 32 * e + lane;
+          const float x = (d[0] + d[kRows * (TK + 8)]) + (d[2 * kRows * (TK + 8)] + d[3 * kRows * (TK + 8)]);
+          v[e] = first + 32 * e + lane < k1 ? x * p.sl2 : -1e30f;
+          mx = fmaxf(mx, v[e]);
+        }
+        const float m_old = s_m[row], m_new = fmaxf(m_old, warp_max(mx));
+        float sum = 0.0f;
+#pragma unroll
+        for (int e = 0; e < TK / 32; ++e) {
+          const float x = fast_exp2(v[e] - m_new);
+          sum += x;
+          s_p[row * (TK + 8) + 32 * e + lane] = __float2bfloat16_rn(x);
+        }
+        sum = warp_sum(sum);
+        if (lane == 0) {
+          const float alpha = fast_exp2(m_old - m_new);
+          s_m[row] = m_new;
+          s_l[row] = s_l[row] * alpha + sum;
+          s_a[row] = alpha;
+        }
       }
-      if (c_cnt > 1 && warp == 0 && t4 == 0) p.part_ml[(size_t)chunk * p.heads + h] = make_float2(s_m[hr], s_l[hr]);
+      __syncthreads();
+      // O = O * alpha + P C; cache blocks past the end of the chunk were not fetched and are skipped
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        const float a0 = s_a[16 * i + g], a1 = s_a[16 * i + g + 8];
+        if (__any_sync(0xffffffffu, a0 != 1.0f || a1 != 1.0f)) {
+#pragma unroll
+          for (int j = 0; j < 2 * MAXU; ++j) { acc[i][j][0] *= a0; acc[i][j][1] *= a0; acc[i][j][2] *= a1; acc[i][j][3] *= a1; }
+        }
+      }
+      const int nb = min(TK, k1 - first + kBlockTokens - 1) / kBlockTokens;
+#pragma unroll
+      for (int ks = 0; ks < TK / 16; ++ks) {
+        if (ks < nb) {
+          uint32_t pa[MT][4];
+#pragma unroll
+          for (int i = 0; i < MT; ++i) {
+            const int mat = lane >> 3, row = 16 * i + (lane & 7) + 8 * (mat & 1);
+            ldmatrix_x4(pa[i], smem_u32(s_p) + (uint32_t)(row * (TK + 8) + 16 * ks + 8 * (mat >> 1)) * 2);
+          }
+          const int key = 16 * ks + (lane & 7) + 8 * ((lane >> 3) & 1);
+#pragma unroll
+          for (int j = 0; j < MAXU; ++j) {
+            if (j < u_n) {
+              const int u = u0 + j, ch = 2 * (u & 3) + (lane >> 4);
+              uint32_t b[4];
+              ldmatrix_x4_trans(b, tile + (uint32_t)(u >> 2) * (TK * 128) + (uint32_t)key * 128 + (uint32_t)((ch ^ (key & 7)) << 4));
+              const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
+#pragma unroll
+              for (int i = 0; i < MT; ++i) {
+                mma_bf16_16816(acc[i][2 * j], pa[i], b0, acc[i][2 * j]);
+                mma_bf16_16816(acc[i][2 * j + 1], pa[i], b1, acc[i][2 * j + 1]);
+              }
+            }
+          }
+        }
+      }
+      if (!ok) break;
     }
+    if (ok) {
+#pragma unroll
+      for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int hh = 0; hh < 2; ++hh) {
+          const int hr = 16 * i + g + 8 * hh, h = h0 + hr;
+          if (h >= p.heads) continue;
+          const float inv = 1.0f / s_l[hr];
+#pragma unroll
+          for (int j = 0; j < 2 * MAXU; ++j) {
+            if ((j >> 1) >= u_n) continue;
+            const int col = (u0 + (j >> 1)) * 16 + (j & 1) * 8 + 2 * t4;
+            const float x = acc[i][j][2 * hh], y = acc[i][j][2 * hh + 1];
+            if (c_cnt == 1)
+              *reinterpret_cast<uint32_t*>(p.out + ((size_t)r * p.heads + h) * R + col) = pack_bf16x2(x * inv, y * inv);
+            else
+              *reinterpret_cast<float2*>(p.part_o + ((size_t)chunk * p.heads + h) * R + col) = make_float2(x, y);
+          }
+          if (c_cnt > 1 && warp == 0 && t4 == 0) p.part_ml[(size_t)chunk * p.heads + h] = make_float2(s_m[hr], s_l[hr]);
+        }
+    }
+  }
+  __syncthreads();
+  if (*abort_flag) {
+    // a wait expired: give copies that may still be in flight time to land before the shared memory is released
+    for (int i = 0; i < 2000; ++i) __nanosleep(1000);
+    if (threadIdx.x == 0 && p.status) atomicExch(p.status, 2 | (4 << 8));
+  }
 }
 
 // CTA = (row, head): the chunks of a context that was split
@@ -433,23 +523,31 @@ uint32_t logismos_launch_latent_gather_bf16(const void* pool, const void* block_
   if (!pool || !out || !kv_start_i32 || total_kv_tokens <= 0 || n_seqs <= 0 || n_seqs > 65535 || max_kv_len <= 0 || max_kv_len > total_kv_tokens ||
       width <= 0 || (width % 8) || max_blocks <= 0 || n_pool_blocks <= 0 || (((uintptr_t)pool | (uintptr_t)out) & 15))
     return lg::kInvalidValue;
-  lg::launch(latent_gather_kernel, dim3((unsigned)((max_kv_len + 63) / 64), (unsigned)n_seqs), dim3(kThreads), 0, (cudaStream_t)stream,
+  lg::launch(latent_gather_kernel, dim3((unsigned)((max_kv_len + kBlockTokens - 1) / kBlockTokens), (unsigned)n_seqs), dim3(kThreads), 0, (cudaStream_t)stream,
              (const __nv_bfloat16*)pool, (const int*)block_tables_i32, max_blocks, n_pool_blocks, (const int*)kv_lens_i32, (__nv_bfloat16*)out,
              (int*)kv_start_i32, n_seqs, logismos_latent_gather_rows(total_kv_tokens, n_seqs), width, (int*)status_i32);
   return lg::launch_status();
 }
 
+// Chunk length by an estimate in token times: the work of all chunks (a start-up and a merge share each) over
+// the CTA slots, plus half a chunk of imbalance at the end.
 int32_t logismos_pick_latent_chunk(const int32_t* context_lens, int32_t n_seqs, int32_t heads) {
+  const int64_t groups = (heads + 63) / 64, slots = 296;
   int64_t total = 0;
   for (int32_t i = 0; i < n_seqs; ++i) total += context_lens[i] > 0 ? context_lens[i] : 0;
-  const int32_t groups = (heads + 63) / 64;
-  const int64_t per = (total * groups + 295) / 296;  // about two CTAs per SM
-  int64_t chunk = (per + 63) / 64 * 64;
-  if (chunk < 256) chunk = 256;
-  return (int32_t)(chunk > (1 << 20) ? (1 << 20) : chunk);
+  int32_t best = 0;
+  int64_t best_cost = 0;
+  for (int32_t c = 128; c <= (1 << 20); c += c < 1024 ? 64 : c) {
+    int64_t n = 0;
+    for (int32_t i = 0; i < n_seqs; ++i) n += (context_lens[i] + c - 1) / c;
+    if (n > logismos_latent_max_chunks(n_seqs)) continue;
+    const int64_t cost = (total + 96 * n) * groups / slots + c / 2;
+    if (best == 0 || cost < best_cost) { best = c; best_cost = cost; }
+  }
+  return best > 0 ? best : 1 << 20;
 }
 
-int32_t logismos_latent_max_chunks(int32_t max_rows) { return max_rows + 300; }
+int32_t logismos_latent_max_chunks(int32_t max_rows) { return max_rows + 1200; }
 
 size_t logismos_latent_decode_scratch_bytes(int32_t total_chunks, int32_t heads, int32_t rank) {
   if (total_chunks < 0 || heads <= 0 || rank <= 0) return 0;
@@ -462,7 +560,7 @@ uint32_t logismos_launch_latent_decode_bf16(const void* q, const void* pool, con
                                             float scale, void* status_i32, void* stream) {
   lg::LaunchScope launch_scope_;
   if (!q || !pool || !out || !scratch || rows <= 0 || rows > 65535 || total_chunks < rows || chunk_tokens <= 0 || (chunk_tokens % 64) || max_blocks <= 0 ||
-      n_pool_blocks <= 0 || heads <= 0 || rank <= 0 || (rank % 64) || rank > 1024 ||
+      n_pool_blocks <= 0 || heads <= 0 || rank <= 0 || (rank % 64) || rank > 1024 || (int64_t)n_pool_blocks * kBlockTokens > 0x7fffffff - 64 ||
       (((uintptr_t)q | (uintptr_t)pool | (uintptr_t)out | (uintptr_t)scratch) & 15))
     return lg::kInvalidValue;
   cudaStream_t s = (cudaStream_t)stream;
@@ -470,29 +568,26 @@ uint32_t logismos_launch_latent_decode_bf16(const void* q, const void* pool, con
                (const int*)chunk_offsets_i32, (__nv_bfloat16*)out, (float*)scratch, nullptr, rows, heads, rank, chunk_tokens, max_blocks,
                n_pool_blocks, scale * kLog2e, (int*)status_i32};
   p.part_ml = (float2*)(p.part_o + (size_t)total_chunks * heads * rank);
-  auto go = [&](auto kern, int mt, size_t smem) -> uint32_t {
+  CUtensorMap map;
+  if (!make_map(&map, pool, (uint64_t)n_pool_blocks * kBlockTokens, (uint64_t)rank, (uint64_t)rank, kBlockTokens)) return lg::kInvalidValue;
+  // stages: up to four, within what lets the kernel's CTAs share an SM (per_sm)
+  auto go = [&](auto kern, int mt, int tk, size_t fixed, int per_sm) -> uint32_t {
+    const size_t tile = (size_t)tk * rank * 2, room = (size_t)(227 / per_sm) * 1024 - (per_sm > 1 ? 1024 : 0);
+    int stages = kMaxStages;
+    while (stages > 2 && fixed + stages * tile > room) --stages;
+    const size_t smem = fixed + stages * tile;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (uint32_t)e;
-    lg::launch(kern, dim3((unsigned)total_chunks, (unsigned)((heads + 16 * mt - 1) / (16 * mt))), dim3(kThreads), smem, s, p);
+    lg::launch(kern, dim3((unsigned)total_chunks, (unsigned)((heads + 16 * mt - 1) / (16 * mt))), dim3(kDecodeThreads), smem, s, map, p, stages);
     return lg::launch_status();
   };
   uint32_t rc;
-  if (rank <= 128) {
-    if (heads <= 16) rc = go(latent_decode_kernel<1, 2, 64>, 1, decode_smem<1, 64>(rank));
-    else if (heads <= 32) rc = go(latent_decode_kernel<2, 2, 64>, 2, decode_smem<2, 64>(rank));
-    else rc = go(latent_decode_kernel<4, 2, 64>, 4, decode_smem<4, 64>(rank));
-  } else if (rank <= 256) {
-    if (heads <= 16) rc = go(latent_decode_kernel<1, 4, 64>, 1, decode_smem<1, 64>(rank));
-    else if (heads <= 32) rc = go(latent_decode_kernel<2, 4, 64>, 2, decode_smem<2, 64>(rank));
-    else rc = go(latent_decode_kernel<4, 4, 64>, 4, decode_smem<4, 64>(rank));
-  } else if (rank <= 512) {
-    if (heads <= 16) rc = go(latent_decode_kernel<1, 8, 64>, 1, decode_smem<1, 64>(rank));
-    else if (heads <= 32) rc = go(latent_decode_kernel<2, 8, 64>, 2, decode_smem<2, 64>(rank));
-    else rc = go(latent_decode_kernel<4, 8, 64>, 4, decode_smem<4, 64>(rank));
-  } else {
-    if (heads <= 16) rc = go(latent_decode_kernel<1, 16, 32>, 1, decode_smem<1, 32>(rank));
-    else rc = go(latent_decode_kernel<2, 16, 32>, 2, decode_smem<2, 32>(rank));
-  }
+#define LG_DECODE(MT, KS, TK, QREG) go(latent_decode_kernel<MT, KS, TK, QREG>, MT, TK, decode_fixed_smem<MT, TK, QREG>(rank), MT == 1 && KS <= 8 ? 2 : 1)
+  if (rank <= 128) rc = heads <= 16 ? LG_DECODE(1, 2, 64, true) : heads <= 32 ? LG_DECODE(2, 2, 64, true) : LG_DECODE(4, 2, 64, true);
+  else if (rank <= 256) rc = heads <= 16 ? LG_DECODE(1, 4, 64, true) : heads <= 32 ? LG_DECODE(2, 4, 64, true) : LG_DECODE(4, 4, 64, true);
+  else if (rank <= 512) rc = heads <= 16 ? LG_DECODE(1, 8, 32, true) : heads <= 32 ? LG_DECODE(2, 8, 64, true) : LG_DECODE(4, 8, 32, false);
+  else rc = heads <= 16 ? LG_DECODE(1, 16, 32, true) : LG_DECODE(2, 16, 32, false);
+#undef LG_DECODE
   if (rc || total_chunks == rows) return rc;
   lg::launch(latent_merge_kernel, dim3((unsigned)heads, (unsigned)rows), dim3(128), 0, s, (const float*)p.part_o, (const float2*)p.part_ml,
              p.chunk_offsets, p.out, heads, rank);

@@ -468,7 +468,7 @@ uint32_t lg_latent_step(void* model, const uint32_t* host_ids, const int32_t* ca
   if (n_out > 0) LG_TRY(cudaMemcpyAsync(next_tokens, m->tokens.p, (size_t)n_out * 4, cudaMemcpyDeviceToHost, s), "D2H tokens");
   LG_TRY(cudaStreamSynchronize(s), "stream synchronize");
   if (const int dev_status = lg_latent_device_status(m)) {
-    char buf[160];
+    char buf[256];
     std::snprintf(buf, sizeof(buf), "device status 0x%x after a step of %d tokens in %d sequences (low byte 1: a range check failed, 2: a bounded wait expired in kernel family <next byte>)",
                   dev_status, B.T, (int)n_seqs);
     set_error(buf);
