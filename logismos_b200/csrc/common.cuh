@@ -118,6 +118,12 @@ LG_DEVINL float glu_clamp(float g, float u, float alpha, float limit, float shif
   return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + shift);
 }
 
+LG_DEVINL float fast_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
+
 LG_DEVINL uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
 LG_DEVINL uint32_t pack_bf16x2(float lo, float hi) {

@@ -9,8 +9,8 @@
 //                       shares the same rank-wide key = value row and a cached row is read once for all
 // latent_decode splits the contexts in chunks; CTA = (chunk, group of 16 * MT heads), 8 warps, tiles of TK tokens. A cache block (16 tokens) arrives as rank / 64 TMA boxes of 16 rows
 // x 128 bytes (128-byte swizzle) in a ring of stages, so ldmatrix reads are conflict-free and no thread computes
-// addresses of cached rows; warp 0 refills the stage of the previous tile once every warp has passed the
-// current tile's first barrier. Per tile: partial scores S = Q' C^T (mma.sync; a warp takes half of the tokens and a
+// addresses of cached rows; the stage of the previous tile is refilled once every warp has passed the current
+// tile's first barrier. Per tile: partial scores S = Q' C^T (mma.sync; a warp takes half of the tokens and a
 // quarter of the rank, its query fragments stay in registers), summed in shared memory in a fixed order; running
 // maximum and sum in fp32 (exp2 domain); P rounded to bf16; O += P C (a warp per slice of the rank, C through
 // ldmatrix.trans). Partial results are merged by a second kernel; a context that is one chunk is finished in
@@ -28,13 +28,14 @@ using namespace lg::tc;
 
 constexpr float kLog2e = 1.4426950408889634f;
 
-LG_DEVINL float fast_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
-  return y;
-}
 constexpr int kBlockTokens = 16;
 constexpr int kThreads = 256;
+
+LG_DEVINL float redux_max(float x) {
+  float y;
+  asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;\n" : "=f"(y) : "f"(x));
+  return y;
+}
 
 LG_DEVINL void store4(void* p, size_t i4, float4 v, bool f32) {
   if (f32) reinterpret_cast<float4*>(p)[i4] = v;
@@ -127,9 +128,7 @@ struct DecodeArgs {
   int* status;
 };
 
-constexpr int kMaxStages = 4;
-constexpr int kWarps = 8;
-constexpr int kDecodeThreads = 32 * kWarps;
+constexpr int kMaxStages = 4, kWarps = 8, kDecodeThreads = 32 * kWarps;
 
 // shared memory besides the ring: query rows (when they do not stay in registers), partial scores, P, row state
 template <int MT, int TK, bool QREG>
@@ -144,7 +143,7 @@ __global__ void __launch_bounds__(kDecodeThreads, MT == 1 && MAXKS <= 8 ? 2 : 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p, int stages) {
   lg::pdl_trigger();
   extern __shared__ uint8_t smem_raw[];
-  constexpr int kRows = 16 * MT, NTS = TK / 16;               // n8 tiles of a token half
+  constexpr int kRows = 16 * MT, NTS = TK / 16, kRowsPerWarp = kRows / kWarps;  // NTS: n8 tiles of a token half
   constexpr int MAXU = (MAXKS * 4 + kWarps - 1) / kWarps;     // 16-column units of the rank per warp
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* gen = smem_raw + (base - smem_u32(smem_raw));
@@ -179,39 +178,37 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
   const int ctx = __ldg(p.ctx + r);
   const int k0 = c_idx * p.chunk_tokens, k1 = min(ctx, k0 + p.chunk_tokens);
   const int tiles = (k1 - k0 + TK - 1) / TK;
-  // Tile ti of the chunk into its stage (warp 0, tiles in order): lane = 64-column slab of the rank. Lane b holds the
-  // id of the tile's block b, read one tile ahead.
+  // Tile ti of the chunk into its stage (all warps, tiles in order): warp w copies the 64-column slabs w, w + 8, .. of the
+  // rank, lane b the boxes of block b (boxes issued by one warp go out one after the other). Lane b holds the id of the
+  // tile's block b, read one tile ahead.
   const int* table = p.tables + (size_t)r * p.max_blocks;
   auto block_id = [&](int ti) {
     const int bi = (k0 + ti * TK) / kBlockTokens + lane;
     return lane < TK / kBlockTokens && bi < p.max_blocks && bi * kBlockTokens < k1 ? __ldg(table + bi) : -1;
   };
-  int ids = warp == 0 ? block_id(0) : -1;
+  int ids = block_id(0);
   auto fetch = [&](int ti) {
     const int st = ti % stages, nb = min(TK, k1 - (k0 + ti * TK) + kBlockTokens - 1) / kBlockTokens;
-    if (lane == 0) mbar_expect_tx(full_bar(st), (uint32_t)(nb * kBlockTokens * R * 2));
+    if (threadIdx.x == 0) mbar_expect_tx(full_bar(st), (uint32_t)(nb * kBlockTokens * R * 2));
+    if (lane < nb) {
+      if (ids < 0 || ids >= p.n_pool_blocks) {
+        if (p.status) atomicExch(p.status, 1);
+        ids = p.n_pool_blocks;  // beyond the pool: the copy fills zeros
+      }
+      for (int sl = warp; sl < slabs; sl += kWarps)
+        tma_load_2d(base + (uint32_t)st * tile_bytes + (uint32_t)sl * (TK * 128) + (uint32_t)lane * (kBlockTokens * 128), &map_pool, full_bar(st), sl * 64,
+                    ids * kBlockTokens);
+    }
     __syncwarp();
-    if (lane < nb && (ids < 0 || ids >= p.n_pool_blocks)) {
-      if (p.status) atomicExch(p.status, 1);
-      ids = p.n_pool_blocks;  // beyond the pool: the copy fills zeros
-    }
-#pragma unroll
-    for (int b = 0; b < TK / kBlockTokens; ++b) {
-      const int blk = __shfl_sync(0xffffffffu, ids, b);
-      if (b < nb && lane < slabs)
-        tma_load_2d(base + (uint32_t)st * tile_bytes + (uint32_t)lane * (TK * 128) + (uint32_t)b * (kBlockTokens * 128), &map_pool, full_bar(st), lane * 64,
-                    blk * kBlockTokens);
-    }
     ids = block_id(ti + 1);
   };
-  int fetched = 0;  // warp 0
+  int fetched = 0;
   auto prefetch = [&](bool all) {
     while (fetched < stages && fetched < tiles && (all || k0 + (fetched + 1) * TK < ctx)) fetch(fetched++);
   };
-  if (warp == 0) prefetch(false);
+  prefetch(false);
   lg::pdl_wait();
-  if (warp == 0) prefetch(true);
-  if (threadIdx.x < kRows) { s_m[threadIdx.x] = -1e30f; s_l[threadIdx.x] = 0.0f; }
+  prefetch(true);
   if (!QREG) {
     const int cw = R >> 3;
     for (int u = threadIdx.x; u < kRows * cw; u += kDecodeThreads) {
@@ -249,12 +246,17 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
       for (int j = 0; j < 2 * MAXU; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.0f;
-    bool ok = true;
-    for (int ti = 0; ti < tiles; ++ti) {
+    // softmax state of the rows warp, warp + 8, ..: the running maximum (the same in every lane) and this lane's share of
+    // the sum (lane = token slot of a tile)
+    float m_run[kRowsPerWarp], l_run[kRowsPerWarp];
+#pragma unroll
+    for (int rr = 0; rr < kRowsPerWarp; ++rr) { m_run[rr] = -1e30f; l_run[rr] = 0.0f; }
+
+    // partial S = Q' C^T of tile ti over this warp's quarter of the rank, half of the tokens -> s_part
+    auto scores = [&](int ti) {
       const int st = ti % stages;
       mbar_wait_warp(full_bar(st), (uint32_t)((ti / stages) & 1), abort_flag);  // a wait that expires sets the flag
       const uint32_t tile = base + (uint32_t)st * tile_bytes;
-      // partial S = Q' C^T over this warp's quarter of the rank, half of the tokens
       float s[MT][NTS][4];
 #pragma unroll
       for (int i = 0; i < MT; ++i)
@@ -300,13 +302,18 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
           *reinterpret_cast<float2*>(d) = make_float2(s[i][j][0], s[i][j][1]);
           *reinterpret_cast<float2*>(d + 8 * (TK + 8)) = make_float2(s[i][j][2], s[i][j][3]);
         }
+    };
+
+    bool ok = true;
+    scores(0);
+    for (int ti = 0; ti < tiles; ++ti) {
       __syncthreads();
-      if (*abort_flag) ok = false;  // set before this barrier or not at all during this tile: the same for every warp
-      if (warp == 0 && ti > 0 && ti - 1 + stages < tiles) fetch(ti - 1 + stages);
+      if (*abort_flag) ok = false;  // set before this barrier or not at all until the next one: the same for every warp
+      if (ti > 0 && ti - 1 + stages < tiles) fetch(ti - 1 + stages);
       // running maximum and sum; a tile always holds at least one visible key, so the maximum is a real score
       const int first = k0 + ti * TK;
 #pragma unroll
-      for (int rr = 0; rr < 2 * MT; ++rr) {
+      for (int rr = 0; rr < kRowsPerWarp; ++rr) {
         const int row = warp + kWarps * rr;
         float v[TK / 32];
         float mx = -1e30f;
@@ -317,24 +324,22 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
           v[e] = first + 32 * e + lane < k1 ? x * p.sl2 : -1e30f;
           mx = fmaxf(mx, v[e]);
         }
-        const float m_old = s_m[row], m_new = fmaxf(m_old, warp_max(mx));
-        float sum = 0.0f;
+        const float m_new = fmaxf(m_run[rr], redux_max(mx)), alpha = fast_exp2(m_run[rr] - m_new);
+        m_run[rr] = m_new;
+        l_run[rr] *= alpha;
 #pragma unroll
         for (int e = 0; e < TK / 32; ++e) {
           const float x = fast_exp2(v[e] - m_new);
-          sum += x;
+          l_run[rr] += x;
           s_p[row * (TK + 8) + 32 * e + lane] = __float2bfloat16_rn(x);
         }
-        sum = warp_sum(sum);
-        if (lane == 0) {
-          const float alpha = fast_exp2(m_old - m_new);
-          s_m[row] = m_new;
-          s_l[row] = s_l[row] * alpha + sum;
-          s_a[row] = alpha;
-        }
+        if (lane == 0) s_a[row] = alpha;
       }
       __syncthreads();
-      // O = O * alpha + P C; cache blocks past the end of the chunk were not fetched and are skipped
+      // the next tile's scores and this tile's O = O * alpha + P C are independent; cache blocks past the end of the
+      // chunk were not fetched and are skipped
+      if (ti + 1 < tiles) scores(ti + 1);
+      const uint32_t tile = base + (uint32_t)(ti % stages) * tile_bytes;
 #pragma unroll
       for (int i = 0; i < MT; ++i) {
         const float a0 = s_a[16 * i + g], a1 = s_a[16 * i + g + 8];
@@ -372,6 +377,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
       }
       if (!ok) break;
     }
+#pragma unroll
+    for (int rr = 0; rr < kRowsPerWarp; ++rr) {
+      const float l = warp_sum(l_run[rr]);
+      if (lane == 0) { s_m[warp + kWarps * rr] = m_run[rr]; s_l[warp + kWarps * rr] = l; }
+    }
+    __syncthreads();
     if (ok) {
 #pragma unroll
       for (int i = 0; i < MT; ++i)
@@ -402,29 +413,50 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
   }
 }
 
-// CTA = (row, head): the chunks of a context that was split
+// CTA = (row, head): the chunks of a context that was split. Their weights are computed by all threads at once, the rows
+// are then summed with several loads in flight.
+constexpr int kMergeTile = 256;
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml, const int* __restrict__ chunk_offsets,
                     __nv_bfloat16* __restrict__ out, int heads, int rank) {
   lg::pdl_prologue();
-  const int h = blockIdx.x, r = blockIdx.y;
+  __shared__ float red[32], w[kMergeTile];
+  const int h = blockIdx.x, r = blockIdx.y, tid = threadIdx.x;
   const int c0 = chunk_offsets[r], c1 = chunk_offsets[r + 1];
   if (c1 - c0 <= 1) return;
-  float m = -1e30f, l = 0.0f;
-  for (int c = c0; c < c1; ++c) m = fmaxf(m, part_ml[(size_t)c * heads + h].x);
-  for (int c = c0; c < c1; ++c) {
-    const float2 ml = part_ml[(size_t)c * heads + h];
-    l += ml.y * exp2f(ml.x - m);
-  }
-  const float inv = 1.0f / l;
-  for (int v = threadIdx.x; v < rank / 4; v += 128) {
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int c = c0; c < c1; ++c) {
-      const float w = exp2f(part_ml[(size_t)c * heads + h].x - m) * inv;
-      const float4 o = reinterpret_cast<const float4*>(part_o + ((size_t)c * heads + h) * rank)[v];
-      a.x += w * o.x; a.y += w * o.y; a.z += w * o.z; a.w += w * o.w;
+  float m = -1e30f;
+  for (int c = c0 + tid; c < c1; c += 128) m = fmaxf(m, part_ml[(size_t)c * heads + h].x);
+  m = block_max(m, red);
+  float l = 0.0f;
+  float4 acc[2] = {make_float4(0.f, 0.f, 0.f, 0.f), make_float4(0.f, 0.f, 0.f, 0.f)};  // rank <= 1024: two float4 per thread
+  for (int cb = c0; cb < c1; cb += kMergeTile) {
+    const int n = min(kMergeTile, c1 - cb);
+    __syncthreads();
+    for (int c = tid; c < n; c += 128) {
+      const float2 ml = part_ml[(size_t)(cb + c) * heads + h];
+      w[c] = exp2f(ml.x - m);
+      l += ml.y * w[c];
     }
-    store4(out, ((size_t)r * heads + h) * (rank / 4) + v, a, false);
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int v = tid + i * 128;
+      if (v >= rank / 4) continue;
+      const float4* src = reinterpret_cast<const float4*>(part_o + ((size_t)cb * heads + h) * rank) + v;
+      const size_t step = (size_t)heads * rank / 4;
+#pragma unroll 8
+      for (int c = 0; c < n; ++c) {
+        const float4 o = src[c * step];
+        acc[i].x = fmaf(w[c], o.x, acc[i].x); acc[i].y = fmaf(w[c], o.y, acc[i].y);
+        acc[i].z = fmaf(w[c], o.z, acc[i].z); acc[i].w = fmaf(w[c], o.w, acc[i].w);
+      }
+    }
+  }
+  const float inv = 1.0f / block_sum(l, red);
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int v = tid + i * 128;
+    if (v < rank / 4) store4(out, ((size_t)r * heads + h) * (rank / 4) + v, make_float4(acc[i].x * inv, acc[i].y * inv, acc[i].z * inv, acc[i].w * inv), false);
   }
 }
 
@@ -529,19 +561,25 @@ uint32_t logismos_launch_latent_gather_bf16(const void* pool, const void* block_
   return lg::launch_status();
 }
 
-// Chunk length by an estimate in token times: the work of all chunks (a start-up and a merge share each) over
-// the CTA slots, plus half a chunk of imbalance at the end.
+// Chunk length by an estimate in token times: full chunks run in waves over the CTA slots (one CTA per SM, two with few
+// heads), the remainders of the contexts fit the last wave's idle slots or take further waves; a chunk costs a start and a merge share.
 int32_t logismos_pick_latent_chunk(const int32_t* context_lens, int32_t n_seqs, int32_t heads) {
-  const int64_t groups = (heads + 63) / 64, slots = 296;
-  int64_t total = 0;
-  for (int32_t i = 0; i < n_seqs; ++i) total += context_lens[i] > 0 ? context_lens[i] : 0;
+  static const int32_t cands[] = {128, 192, 256, 320, 384, 448, 512, 640, 768, 896, 1024, 1280, 1536, 1792, 2048, 3072, 4096, 8192, 16384, 1 << 20};
+  const int64_t groups = (heads + 63) / 64, slots = heads <= 16 ? 296 : 148, start = 96;
   int32_t best = 0;
   int64_t best_cost = 0;
-  for (int32_t c = 128; c <= (1 << 20); c += c < 1024 ? 64 : c) {
-    int64_t n = 0;
-    for (int32_t i = 0; i < n_seqs; ++i) n += (context_lens[i] + c - 1) / c;
-    if (n > logismos_latent_max_chunks(n_seqs)) continue;
-    const int64_t cost = (total + 96 * n) * groups / slots + c / 2;
+  for (int32_t c : cands) {
+    int64_t full = 0, parts = 0, longest = 0;
+    for (int32_t i = 0; i < n_seqs; ++i) {
+      const int32_t f = context_lens[i] / c, r = context_lens[i] - f * c;
+      full += f;
+      parts += r > 0;
+      if (r > longest) longest = r;
+    }
+    if (full + parts > logismos_latent_max_chunks(n_seqs)) continue;
+    const int64_t waves = (full * groups + slots - 1) / slots, all_waves = ((full + parts) * groups + slots - 1) / slots;
+    int64_t cost = waves * (c + start) + (all_waves - waves) * (longest + start);
+    cost += (full + parts) * 16 / slots;
     if (best == 0 || cost < best_cost) { best = c; best_cost = cost; }
   }
   return best > 0 ? best : 1 << 20;
@@ -589,7 +627,9 @@ uint32_t logismos_launch_latent_decode_bf16(const void* q, const void* pool, con
   else rc = heads <= 16 ? LG_DECODE(1, 16, 32, true) : LG_DECODE(2, 16, 32, false);
 #undef LG_DECODE
   if (rc || total_chunks == rows) return rc;
-  lg::launch(latent_merge_kernel, dim3((unsigned)heads, (unsigned)rows), dim3(128), 0, s, (const float*)p.part_o, (const float2*)p.part_ml,
+  // an ordinary launch: with the early one the next projection's CTAs moved in ahead of these and a decode step of 8
+  // sequences took 1.86 instead of 1.42 ms
+  lg::launch_ordered(latent_merge_kernel, dim3((unsigned)heads, (unsigned)rows), dim3(128), 0, s, (const float*)p.part_o, (const float2*)p.part_ml,
              p.chunk_offsets, p.out, heads, rank);
   return lg::launch_status();
 }

@@ -33,8 +33,14 @@ namespace {
 
 using namespace lgm;
 
-// rows up to which a projection streams its weights (linear_small) instead of running on the tcgen05 tiles
-constexpr int kSmallRows = 32;
+// Whether a projection of few rows streams its weights (linear_small) instead of running on the tcgen05 tiles. Measured
+// (us, small / tiles): accumulating into the residual, where the tiles split k, 2048 x 10240 at 1 / 8 / 32 rows 14.6 /
+// 12.6, 15.6 / 12.6, 29.0 / 12.6; gated 16384 x 2048 at 8 / 16 / 32 rows 17.8 / 22.7, 19.0 / 22.0, 28.5 / 17.9; head 32768
+// x 2048 at 16 / 32 rows 39.5 / 41.5, 57.2 / 41.1; 1536 x 2048 at 8 / 32 / 64 rows 5.7 / 17.4, 11.6 / 18.2, 20.8 / 19.1.
+inline bool stream_weights(int rows, int n, int k, int epi) {
+  if (epi == LG_EPI_RESID_F32) return logismos_get_deterministic() && rows <= 32;
+  return rows <= ((int64_t)n * k >= (1 << 23) ? 16 : 32);
+}
 
 inline int r64(int v) { return (v + 63) & ~63; }
 
@@ -71,7 +77,7 @@ uint32_t linear(Latent* m, const Lin& l, int rows, cudaStream_t s) {
   if (m->cfg.is_f32)
     return logismos_launch_linear_f32(l.a, l.w->p, b, l.out, rows, l.n, l.k, l.lda, l.ldc, 1, 0, 0, 0, l.epi == LG_EPI_BF16 ? LG_EPI_F32 : l.epi,
                                       l.p0, l.p1, l.p2, s);
-  if (rows <= kSmallRows)
+  if (stream_weights(rows, l.n, l.k, l.epi))
     return logismos_launch_linear_small_bf16(l.a, l.w->p, b, l.out, rows, l.n, l.k, l.lda, l.ldc, 1, 0, 0, 0, l.epi, l.p0, l.p1, l.p2, s);
   return logismos_launch_linear_t_act_bf16(l.a, l.w->p, b, l.out, rows, l.n, l.k, l.lda, l.ldc, l.epi | LG_EPI_STATIC_W, l.p0, l.p1, l.p2,
                                            m->status.p, s);
