@@ -184,3 +184,177 @@ def measure(sizes, iters, peaks, seqs=(8, 64), ctx=2048, prefill=(4, 1024)):
             torch.cuda.empty_cache()
         out.append(row)
     return out
+
+
+# ---- kernels -------------------------------------------------------------------------------------
+
+def _graph_us(calls, reps=6):
+    """Device time per call: the calls (different operands) captured once, replayed."""
+    import torch
+    from ctypes import c_void_p
+    s = torch.cuda.Stream()
+    torch.cuda.synchronize()  # the operands were made on another stream
+    with torch.cuda.stream(s):
+        for c in calls:
+            assert c(c_void_p(s.cuda_stream)) == 0
+        torch.cuda.synchronize()
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g, stream=s):
+            for c in calls:
+                c(c_void_p(s.cuda_stream))
+        for _ in range(3):
+            g.replay()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(s)
+        for _ in range(reps):
+            g.replay()
+        e1.record(s)
+        torch.cuda.synchronize()
+    return 1e3 * e0.elapsed_time(e1) / reps / len(calls)
+
+
+def kernel_table(z, peaks, T=4096, seqs=64, ctx=8192):
+    """Every kernel of the latent-attention decoder at one size, and the like kernel of the int4 decoder, each against
+    its roofline (the slower of bytes over the measured copy bandwidth and FLOPs over the measured bf16 peak).
+    Operands rotate over copies that exceed L2 together."""
+    import ctypes as C
+    import torch
+    from logismos_b200 import ops
+    from logismos_b200._lib import lib
+    dev = "cuda"
+    P = lambda t: C.c_void_p(t.data_ptr() if t is not None else 0)
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    H, heads, D, Q, R, F = z["width"], z["heads"], z["dim"], z["q_rank"], z["kv_rank"], z["ff"]
+    HD = heads * D
+    rows = []
+    bf = lambda *s: (torch.randn(s, device=dev, dtype=torch.bfloat16) * 0.02)
+    f32 = lambda *s: torch.randn(s, device=dev)
+    i32 = lambda a: torch.as_tensor(np.asarray(a, np.int32)).to(dev)
+
+    def copies(nbytes):
+        return max(2, min(12, int(3e8 // max(nbytes, 1)) + 1))
+
+    def add(phase, name, calls, nbytes, flops=0.0, like=None):
+        us = _graph_us(calls)
+        if int(st.item()):
+            raise RuntimeError("%s / %s: device status 0x%x" % (phase, name, int(st.item())))
+        roof = max(nbytes / peaks["hbm"] / 1e3, flops / peaks["tf_burst"] / 1e6)
+        rows.append({"phase": phase, "kernel": name, "us": us, "roofline_us": roof, "frac": roof / us, "bound": "hbm" if nbytes / peaks["hbm"] / 1e3 >= flops / peaks["tf_burst"] / 1e6 else "tensor",
+                     "like": like})
+        return us
+
+    def gemm(phase, name, m, n, k, epi, small=False, like=None):
+        """bf16 projection through the tcgen05 kernel or the weight-streaming one."""
+        w_bytes = 2.0 * n * k
+        nw = copies(w_bytes)
+        ws, a = [bf(n, k) for _ in range(nw)], bf(m, k)
+        glu = epi in (2, 4)
+        cols = n // 2 if glu else n
+        out = torch.zeros((m, cols), device=dev, dtype=torch.float32 if epi in (1, 3) else torch.bfloat16)
+        bias = torch.zeros(n, device=dev)
+        p = (1.702, 7.0, 1.0) if epi == 4 else (0.0, 0.0, 0.0)
+        if small:
+            calls = [lambda s, w=w: lib.logismos_launch_linear_small_bf16(P(a), P(w), P(bias), P(out), m, n, k, k, cols, 1, 0, 0, 0, epi, *p, s) for w in ws]
+        else:
+            calls = [lambda s, w=w: lib.logismos_launch_linear_t_act_bf16(P(a), P(w), P(bias), P(out), m, n, k, k, cols, epi | 0x100, *p, P(st), s) for w in ws]
+        add(phase, name, calls, w_bytes + 2.0 * m * k + m * cols * out.element_size() * (2 if epi == 1 else 1), 2.0 * m * n * k, like)
+
+    def qlin(phase, name, m, n, k):
+        w_bytes = 0.5625 * n * k
+        nw = copies(w_bytes)
+        codes = [torch.randint(0, 256, (n, k // 2), dtype=torch.uint8, device=dev) for _ in range(nw)]
+        scales = [(torch.rand((n, k // 32), device=dev) * 0.02).to(torch.float16) for _ in range(nw)]
+        a, acc = bf(m, k), torch.zeros((m, n), device=dev)
+        add(phase, name, [lambda s, i=i: lib.logismos_launch_qlinear_int4_g32_acc_f32_static(P(a), P(codes[i]), P(scales[i]), P(acc), m, n, k, k, n, P(st), s) for i in range(nw)],
+            w_bytes + 2.0 * m * k + 8.0 * m * n, 2.0 * m * n * k)
+
+    gain = torch.ones(H, device=dev)
+    # ---- prefill of T tokens in sequences of 1024
+    nq = T // 1024
+    hist, coef, x, inv = f32(9, T, H), torch.ones(9, device=dev), f32(T, H), torch.ones(T, device=dev)
+    add("prefill", "depth_mix (9 snapshots)", [lambda s: lib.logismos_launch_depth_mix_f32(P(hist), T * H, 9, P(coef), P(None), T, P(x), P(inv), P(None), P(None), 0, T, H, H, 1e-6, P(st), s)] * 2,
+        10.0 * T * H * 4, like="rms_norm")
+    w4, o1, o2 = torch.ones((4, H), device=dev), bf(T, H), bf(T, H)
+    state, slots = torch.zeros((64, 2, 3, H), device=dev), i32(range(seqs))
+    zero8, seq_ids, cu = torch.zeros(seqs, dtype=torch.uint8, device=dev), i32(np.repeat(np.arange(nq), 1024)), i32(np.arange(nq + 1) * 1024)
+    xs = [f32(T, H) for _ in range(copies(T * H * 4))]
+    add("prefill", "norm_conv", [lambda s, y=y: lib.logismos_launch_norm_conv(P(y), P(inv), P(gain), P(w4), P(w4), P(o1), P(o2), 0, P(state), P(slots), P(zero8), P(zero8), P(seq_ids), P(cu), T, H, 4, s)
+                                     for y in xs], 8.0 * T * H, like="rms_norm")
+    gemm("prefill", "latent projections", T, Q + R, H, 3, like="qkv GEMM")
+    raws, pool = [f32(T, Q + R) for _ in range(copies(T * (Q + R) * 4))], bf(seqs * (ctx // 16 + 1), 16, R)
+    cq, gq, gc, slot64 = bf(T, Q), torch.ones(Q, device=dev), torch.ones(R, device=dev), torch.randperm(T, device=dev)
+    add("prefill", "latent_norm_store", [lambda s, y=y: lib.logismos_launch_latent_norm_store(P(y), Q + R, P(gq), P(gc), P(cq), P(pool), P(slot64), T, Q, Q, R, R, 1e-6, pool.shape[0] * 16, 0, 0, P(st), s)
+                                             for y in raws], 6.0 * T * (Q + R), like="rms_norm")
+    gemm("prefill", "queries", T, HD, Q, 0, like="qkv GEMM")
+    nblk = 1024 // 16
+    tabs = i32(np.random.default_rng(0).permutation(nq * nblk).reshape(nq, nblk))
+    kv_lens, tp = i32([1024] * nq), int(lib.logismos_latent_gather_rows(T, nq))
+    lat, start = bf(tp, R), i32(np.arange(nq) * 1024)
+    pools = [bf(nq * nblk, 16, R) for _ in range(copies(2 * T * R * 4))]
+    add("prefill", "latent_gather", [lambda s, y=y: lib.logismos_launch_latent_gather_bf16(P(y), P(tabs), nblk, nq * nblk, P(kv_lens), P(lat), P(start), T, nq, 1024, R, P(st), s) for y in pools],
+        4.0 * T * R, like="transpose_v")
+    gemm("prefill", "keys (values: the transposed product)", tp, HD, R, 0, like="qkv GEMM")
+    qs, ks, vts, att = bf(T, HD), bf(tp, HD), bf(HD, tp), bf(T, HD)
+    add("prefill", "attention", [lambda s: lib.logismos_launch_varlen_attention_kv_tc_bf16(P(qs), HD, P(cu), P(kv_lens), P(start), P(ks), P(vts), tp, P(att), HD, T, nq, 1024, heads, heads, D, 0.09, P(st), s)] * 3,
+        2.0 * T * HD * 4, 4.0 * HD * nq * 1024 * 1025 / 2, like="attention")
+    gemm("prefill", "gated feed-forward", T, 2 * F, H, 4, like="gate/up GEMM")
+    gemm("prefill", "output projection [W_o | W_down]", T, H, HD + F, 1, like="down GEMM")
+    # like kernels of the int4 decoder
+    KV = HD // 4
+    add("prefill", "= rms_norm", [lambda s, y=y: lib.logismos_launch_rms_norm_f32(P(y), P(gain), P(o1), T, H, 1e-6, 0, s) for y in xs], 6.0 * T * H)
+    gemm("prefill", "= qkv GEMM", T, HD + 2 * KV, H, 0)
+    gemm("prefill", "= gate/up GEMM", T, 2 * F, H, 2)
+    gemm("prefill", "= down GEMM", T, H, F, 1)
+    qkv = bf(T, HD + 2 * KV)
+    scr = torch.empty(lib.logismos_varlen_attention_tc_scratch_bytes(T, nq, heads // 4, D), dtype=torch.uint8, device=dev)
+    add("prefill", "= attention (with transpose_v)", [lambda s: lib.logismos_launch_varlen_attention_tc_bf16(P(qkv), P(cu), P(att), P(scr), T, nq, 1024, heads, heads // 4, D, HD + 2 * KV, HD, HD + KV, 1, P(st), s)] * 3,
+        2.0 * T * HD * 2 + 4.0 * T * KV, 4.0 * HD * nq * 1024 * 1025 / 2)
+    del hist, xs, raws, pools, qs, ks, vts
+    # ---- decode of `seqs` sequences with `ctx` tokens each, and of 8 for the projections
+    nb = ctx // 16 + 1
+    dh = f32(9, seqs, H)
+    dx = f32(seqs, H)
+    add("decode", "depth_mix_conv_decode (9 snapshots)", [lambda s: lib.logismos_launch_depth_mix_conv_decode(P(dh), seqs * H, 9, P(coef), P(dx), P(gain), P(w4), P(w4), P(o1), P(o2), 0, P(state), P(slots), P(zero8), P(zero8), seqs, H, H, 1e-6, 4, s)] * 4,
+        seqs * H * (10 * 4 + 6 * 4 + 4.0), like="rms_norm")
+    for m in (8, seqs):
+        small = m <= 32
+        gemm("decode %d" % m, "latent projections", m, Q + R, H, 3 if small else 1, small, like="int4 linear qkv")
+        gemm("decode %d" % m, "queries", m, HD, Q, 0, small, like="int4 linear qkv")
+        gemm("decode %d" % m, "gated feed-forward", m, 2 * F, H, 4, m <= 16, like="int4 linear gate/up")
+        gemm("decode %d" % m, "output projection [W_o | W_down]", m, H, HD + F, 1, like="int4 linear down")
+        gemm("decode %d" % m, "head", m, VOCAB, H, 3, m <= 16, like="int4 linear down")
+        wk = [bf(heads, R, D) for _ in range(copies(2 * heads * R * D))]
+        aq, oq = bf(m, heads, D), bf(m, heads, R)
+        add("decode %d" % m, "latent queries (per head)", [lambda s, w=w: lib.logismos_launch_linear_small_bf16(P(aq), P(w), P(None), P(oq), m, R, D, HD, heads * R, heads, D, R * D, R, 0, 0.0, 0.0, 0.0, s) for w in wk],
+            2.0 * heads * (R * D + m * (R + D)), 2.0 * m * heads * R * D, like="int4 linear qkv")
+        if m == 8:
+            qlin("decode 8", "= int4 linear qkv", m, HD + 2 * KV, H)
+            qlin("decode 8", "= int4 linear gate/up", m, 2 * F, H)
+            qlin("decode 8", "= int4 linear down", m, H, F)
+        else:
+            gemm("decode %d" % m, "= qkv GEMM (bf16 copy)", m, HD + 2 * KV, H, 0)
+            gemm("decode %d" % m, "= gate/up GEMM (bf16 copy)", m, 2 * F, H, 2)
+            gemm("decode %d" % m, "= down GEMM (bf16 copy)", m, H, F, 1)
+    cl = torch.full((seqs,), ctx, dtype=torch.int32)
+    tab = i32(np.random.default_rng(1).permutation(seqs * nb).reshape(seqs, nb))
+    qd, od, cg = bf(seqs, heads, R), bf(seqs, heads, R), cl.to(dev)
+    chunk = int(lib.logismos_pick_latent_chunk(C.c_void_p(cl.data_ptr()), seqs, heads))
+    off, total = ops.build_decode_chunks(cl, chunk)
+    off = off.to(dev)
+    scr = torch.empty(lib.logismos_latent_decode_scratch_bytes(total, heads, R), dtype=torch.uint8, device=dev)
+    add("decode", "latent_decode + merge (ctx %d)" % ctx, [lambda s: lib.logismos_launch_latent_decode_bf16(P(qd), P(pool), P(tab), P(cg), P(off), P(od), P(scr), seqs, total, chunk, nb, seqs * nb, heads, R, 0.05, P(st), s)] * 3,
+        seqs * (ctx * R * 2.0 + heads * R * 4.0), 4.0 * seqs * ctx * heads * R, like="paged_decode")
+    del pool
+    nkv = heads // 4
+    kp, vp = bf(seqs * nb, 16, nkv * D), bf(seqs * nb, 16, nkv * D)
+    qp, op = bf(seqs, HD), bf(seqs, HD)
+    pc = ops.pick_decode_chunk(cl, nkv, D)
+    off2, total2 = ops.build_decode_chunks(cl, pc)
+    off2 = off2.to(dev)
+    scr2 = torch.empty(lib.logismos_paged_decode_scratch_bytes(total2, heads, D), dtype=torch.uint8, device=dev)
+    add("decode", "= paged_decode + merge (ctx %d)" % ctx, [lambda s: lib.logismos_launch_paged_attention_decode_bf16(P(qp), P(kp), P(vp), P(None), P(None), P(tab), P(cg), P(off2), P(op), P(scr2), P(st), seqs, total2, pc, nb, seqs * nb, heads, nkv, D, s)] * 3,
+        seqs * ctx * nkv * D * 4.0, 4.0 * seqs * ctx * HD)
+    dxs = f32(seqs, H)
+    add("decode", "= rms_norm", [lambda s: lib.logismos_launch_rms_norm_f32(P(dxs), P(gain), P(o1), seqs, H, 1e-6, 0, s)] * 4, 6.0 * seqs * H)
+    return rows

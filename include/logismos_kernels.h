@@ -558,12 +558,14 @@ uint32_t logismos_launch_depth_mix_conv_decode(const void* hist_f32, int64_t his
  * norm_store: raw f32 [rows, ld] holds the query latent in columns 0 .. q_width and the key/value latent in
  * q_width .. q_width + c_width; both are RMS-normed (means over the first q_n and c_n columns) with their
  * gains; the first goes to q_latent [rows, q_width], the second to the pool at slot_mapping[row] (a slot
- * outside the pool is skipped and raises status to 1). is_f32 selects the type of both. */
-uint32_t logismos_launch_latent_norm_store(const void* raw_f32, int32_t ld, const void* gain_q_f32,
+ * outside the pool is skipped and raises status to 1). is_f32 selects the type of both. zero_raw != 0 leaves
+ * raw zeroed, ready to be accumulated into again. */
+uint32_t logismos_launch_latent_norm_store(void* raw_f32, int32_t ld, const void* gain_q_f32,
                                            const void* gain_c_f32, void* q_latent, void* pool,
                                            const void* slot_mapping_i64, int32_t rows, int32_t q_width,
                                            int32_t q_n, int32_t c_width, int32_t c_n, float eps,
-                                           int64_t n_pool_slots, int32_t is_f32, void* status_i32, void* stream);
+                                           int64_t n_pool_slots, int32_t is_f32, int32_t zero_raw,
+                                           void* status_i32, void* stream);
 /* The cached rows of whole sequences made contiguous: out bf16 [logismos_latent_gather_rows(total, n_seqs),
  * width], sequence s at kv_start[s] (written, a multiple of 8), gaps zeroed. */
 int32_t logismos_latent_gather_rows(int32_t total_kv_tokens, int32_t n_seqs);

@@ -141,7 +141,7 @@ def _declare(l, partial=False):
         "logismos_launch_depth_mix_f32": [vp, i64, i32, vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, vp],
         "logismos_launch_norm_conv": [vp, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, vp],
         "logismos_launch_depth_mix_conv_decode": [vp, i64, i32, vp, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp],
-        "logismos_launch_latent_norm_store": [vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i64, i32, vp, vp],
+        "logismos_launch_latent_norm_store": [vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i64, i32, i32, vp, vp],
         "logismos_launch_latent_gather_bf16": [vp, vp, i32, i32, vp, vp, vp, i32, i32, i32, i32, vp, vp],
         "logismos_launch_latent_decode_bf16": [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp],
         "logismos_launch_latent_attention_f32": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, vp],

@@ -44,14 +44,14 @@ LG_DEVINL void store4(void* p, size_t i4, float4 v, bool f32) {
 
 // warp = (row, half): half 0 the query latent (columns 0 .. qw), half 1 the key/value latent (qw .. qw + rw)
 __global__ void __launch_bounds__(kThreads)
-latent_norm_store_kernel(const float* __restrict__ raw, int ld, const float* __restrict__ gain_q, const float* __restrict__ gain_c,
+latent_norm_store_kernel(float* __restrict__ raw, int ld, const float* __restrict__ gain_q, const float* __restrict__ gain_c,
                          void* __restrict__ cq, void* __restrict__ pool, const int64_t* __restrict__ slots, int rows, int qw, int q_n,
-                         int rw, int r_n, float eps, int64_t n_pool_slots, int f32, int* __restrict__ status) {
+                         int rw, int r_n, float eps, int64_t n_pool_slots, int f32, int zero, int* __restrict__ status) {
   lg::pdl_prologue();
   const int id = (blockIdx.x * kThreads + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   const int row = id >> 1, half = id & 1;
   if (row >= rows) return;
-  const float4* src = reinterpret_cast<const float4*>(raw + (size_t)row * ld + (half ? qw : 0));
+  float4* src = reinterpret_cast<float4*>(raw + (size_t)row * ld + (half ? qw : 0));
   const int nv = (half ? rw : qw) >> 2;
   float ss = 0.0f;
   for (int v = lane; v < nv; v += 32) {
@@ -73,6 +73,7 @@ latent_norm_store_kernel(const float* __restrict__ raw, int ld, const float* __r
   for (int v = lane; v < nv; v += 32) {
     const float4 a = src[v], g = __ldg(gain + v);
     store4(out, dst + v, make_float4(a.x * inv * g.x, a.y * inv * g.y, a.z * inv * g.z, a.w * inv * g.w), f32 != 0);
+    if (zero) src[v] = make_float4(0.f, 0.f, 0.f, 0.f);
   }
 }
 
@@ -531,18 +532,18 @@ latent_attention_f32_kernel(const float* __restrict__ q, const float* __restrict
 
 extern "C" {
 
-uint32_t logismos_launch_latent_norm_store(const void* raw_f32, int32_t ld, const void* gain_q_f32, const void* gain_c_f32, void* q_latent,
+uint32_t logismos_launch_latent_norm_store(void* raw_f32, int32_t ld, const void* gain_q_f32, const void* gain_c_f32, void* q_latent,
                                            void* pool, const void* slot_mapping_i64, int32_t rows, int32_t q_width, int32_t q_n,
                                            int32_t c_width, int32_t c_n, float eps, int64_t n_pool_slots, int32_t is_f32,
-                                           void* status_i32, void* stream) {
+                                           int32_t zero_raw, void* status_i32, void* stream) {
   lg::LaunchScope launch_scope_;
   if (!raw_f32 || rows <= 0 || q_width <= 0 || c_width <= 0 || (q_width % 4) || (c_width % 4) || q_n <= 0 || q_n > q_width || c_n <= 0 ||
       c_n > c_width || ld < q_width + c_width || (ld % 4) || rows > 0x3fffffff)
     return lg::kInvalidValue;
   const int64_t blocks = ((int64_t)rows * 2 + kThreads / 32 - 1) / (kThreads / 32);
-  lg::launch(latent_norm_store_kernel, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, (const float*)raw_f32, ld,
+  lg::launch(latent_norm_store_kernel, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, (float*)raw_f32, ld,
              (const float*)gain_q_f32, (const float*)gain_c_f32, q_latent, pool, (const int64_t*)slot_mapping_i64, rows, q_width, q_n,
-             c_width, c_n, eps, n_pool_slots, is_f32, (int*)status_i32);
+             c_width, c_n, eps, n_pool_slots, is_f32, zero_raw, (int*)status_i32);
   return lg::launch_status();
 }
 

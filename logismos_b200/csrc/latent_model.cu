@@ -42,6 +42,8 @@ inline bool stream_weights(int rows, int n, int k, int epi) {
   return rows <= ((int64_t)n * k >= (1 << 23) ? 16 : 32);
 }
 
+constexpr int kAccRows = 512;
+
 inline int r64(int v) { return (v + 63) & ~63; }
 
 struct LLayer {
@@ -58,13 +60,17 @@ struct Latent {
   int device = 0, Hp = 0;
   Buf embed, final_gain, head, one;
   std::vector<LLayer> layers;
-  Buf hist, h1, h2, raw, cq, q, qlat, olat, cat, last, logits, tokens, status, inv_rms;
+  Buf hist, h1, h2, raw, raw_acc, cq, q, qlat, olat, cat, last, logits, tokens, status, inv_rms;
   Buf lat, kbuf, vt, kv_start, dec_scratch, dev_batch;
   StepBatch batch;
   std::vector<uint8_t> slot_phase;  // per state slot: the copy that holds its state
   cudaStream_t stream = nullptr;
   std::mutex mu;
   int n_out = 0, total_chunks = 0, chunk_tokens = 64, launches = 0;
+  // `raw_acc` is all zero between its uses (the kernel that reads it zeroes it); a step that failed part-way may have left
+  // sums there, so the next one clears it
+  bool acc_dirty = true;
+  size_t acc_bytes = 0;
   bool ready = false;               // a step's indices are on the device (replay)
   template <typename T> T* dev(T* host) const { return (T*)((uint8_t*)dev_batch.p + ((uint8_t*)host - batch.pinned)); }
 };
@@ -138,6 +144,10 @@ uint32_t run_device(Latent* m, cudaStream_t s) {
   float* hist = (float*)m->hist.p;
   void* st = m->status.p;
   m->launches = 1;
+  if (m->acc_dirty) {
+    LG_TRY(cudaMemsetAsync(m->raw_acc.p, 0, m->acc_bytes, s), "clear accumulation workspace");
+    m->acc_dirty = false;
+  }
   LG_TRY(logismos_launch_embed_lookup_bf16(m->embed.p, m->dev(B.ids), hist, T, Hp, c.vocab, s), "embed_lookup");
   const Buf* coef = &m->one;
   for (int l = 0; l < c.n_layers; ++l) {
@@ -157,9 +167,12 @@ uint32_t run_device(Latent* m, cudaStream_t s) {
                                        m->dev(B.phase), m->dev(B.seq_ids), m->dev(B.cu), T, Hp, c.conv_taps, s), "norm and convolution");
       m->launches += 2;
     }
-    LG_TRY(linear(m, {m->h1.p, Hp, &L.w_in, L.Qp + L.Rp, Hp, nullptr, m->raw.p, L.Qp + L.Rp, LG_EPI_F32}, T, s), "latent projections");
-    LG_TRY(logismos_launch_latent_norm_store(m->raw.p, L.Qp + L.Rp, L.gain_q.p, L.gain_c.p, m->cq.p, L.pool.p, m->dev(B.slots), T, L.Qp, L.c.q_rank,
-                                             L.Rp, L.c.kv_rank, c.rms_eps, (int64_t)c.n_pool_blocks * kKvBlock, f32, st, s), "latent norm and store");
+    // a few dozen rows: the narrow projection is accumulated, so that the tiles split its reduction over the idle SMs
+    const bool acc = !f32 && T > 32 && T <= kAccRows && !logismos_get_deterministic();
+    float* raw = (float*)(acc ? m->raw_acc.p : m->raw.p);
+    LG_TRY(linear(m, {m->h1.p, Hp, &L.w_in, L.Qp + L.Rp, Hp, nullptr, raw, L.Qp + L.Rp, acc ? LG_EPI_RESID_F32 : LG_EPI_F32}, T, s), "latent projections");
+    LG_TRY(logismos_launch_latent_norm_store(raw, L.Qp + L.Rp, L.gain_q.p, L.gain_c.p, m->cq.p, L.pool.p, m->dev(B.slots), T, L.Qp, L.c.q_rank,
+                                             L.Rp, L.c.kv_rank, c.rms_eps, (int64_t)c.n_pool_blocks * kKvBlock, f32, acc, st, s), "latent norm and store");
     m->launches += 1;
     LG_TRY(linear(m, {m->cq.p, L.Qp, &L.w_uq, HD, L.Qp, nullptr, m->q.p, HD, LG_EPI_BF16}, T, s), "queries");
     if (uint32_t rc = attention(m, L, s)) return rc;
@@ -349,7 +362,8 @@ uint32_t lg_latent_create(int32_t device, const lg_latent_config_t* cfg, const l
   lim.n_state_slots = c.n_state_slots;
   lim.prefix_cap_tokens = MB * kKvBlock > T ? MB * kKvBlock : T;
   lim.extra_bytes = (size_t)c.max_out_rows * 4;
-  ok = ok && m->hist.alloc((size_t)(c.n_layers + 1) * T * Hp * 4) && m->h1.alloc(T * Hp * esz) && m->h2.alloc(T * Hp * esz) && m->raw.alloc(T * in_w * 4) &&
+  m->acc_bytes = (T < (size_t)kAccRows ? T : (size_t)kAccRows) * in_w * 4;
+  ok = ok && m->hist.alloc((size_t)(c.n_layers + 1) * T * Hp * 4) && m->h1.alloc(T * Hp * esz) && m->h2.alloc(T * Hp * esz) && m->raw.alloc(T * in_w * 4) && m->raw_acc.alloc(m->acc_bytes) &&
        m->cq.alloc(T * q_w * esz) && m->q.alloc(T * hd_w * esz) && m->qlat.alloc(lat_rows * hr_w * esz) && m->olat.alloc(lat_rows * hr_w * esz) &&
        m->cat.alloc(T * cat_w * esz) && m->last.alloc((size_t)c.max_out_rows * Hp * esz) && m->logits.alloc((size_t)c.max_out_rows * c.vocab * 4) &&
        m->tokens.alloc((size_t)c.max_out_rows * 4) && m->status.alloc(4) && m->inv_rms.alloc(T * 4);
@@ -414,7 +428,7 @@ void lg_latent_destroy(void* model) {
   if (!model) return;
   Latent* m = static_cast<Latent*>(model);
   cudaSetDevice(m->device);
-  Buf* bufs[] = {&m->embed, &m->final_gain, &m->head, &m->one, &m->hist, &m->h1, &m->h2, &m->raw, &m->cq, &m->q, &m->qlat, &m->olat, &m->cat,
+  Buf* bufs[] = {&m->embed, &m->final_gain, &m->head, &m->one, &m->hist, &m->h1, &m->h2, &m->raw, &m->raw_acc, &m->cq, &m->q, &m->qlat, &m->olat, &m->cat,
                  &m->last, &m->logits, &m->tokens, &m->status, &m->inv_rms, &m->lat, &m->kbuf, &m->vt, &m->kv_start, &m->dec_scratch, &m->dev_batch};
   for (Buf* b : bufs) b->release();
   for (LLayer& L : m->layers) {
@@ -470,10 +484,11 @@ uint32_t lg_latent_step(void* model, const uint32_t* host_ids, const int32_t* ca
   LG_TRY(cudaMemsetAsync(m->status.p, 0, 4, s), "clear status");
   LG_TRY(cudaMemcpyAsync(m->dev_batch.p, B.pinned, (size_t)((uint8_t*)(rows + n_out) - B.pinned), cudaMemcpyHostToDevice, s), "H2D step");
   m->ready = true;
-  if (uint32_t rc = run_device(m, s)) return rc;
+  if (uint32_t rc = run_device(m, s)) { m->acc_dirty = true; return rc; }
   if (n_out > 0) LG_TRY(cudaMemcpyAsync(next_tokens, m->tokens.p, (size_t)n_out * 4, cudaMemcpyDeviceToHost, s), "D2H tokens");
   LG_TRY(cudaStreamSynchronize(s), "stream synchronize");
   if (const int dev_status = lg_latent_device_status(m)) {
+    m->acc_dirty = true;
     char buf[256];
     std::snprintf(buf, sizeof(buf), "device status 0x%x after a step of %d tokens in %d sequences (low byte 1: a range check failed, 2: a bounded wait expired in kernel family <next byte>)",
                   dev_status, B.T, (int)n_seqs);

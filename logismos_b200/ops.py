@@ -621,7 +621,7 @@ def depth_mix_conv_decode(hist, coef, gain, w1, w2, state, state_slots, fresh, p
     return x, o[0], o[1]
 
 
-def latent_norm_store(raw, gain_q, gain_c, pool, slot_mapping, q_n, c_n, eps, sync=True):
+def latent_norm_store(raw, gain_q, gain_c, pool, slot_mapping, q_n, c_n, eps, zero_raw=False, sync=True):
     """raw fp32 [rows, q width + c width] -> normed query latents; the normed key/value latents go to ``pool``
     [blocks, 16, c width] (bf16 or fp32, which also sets the type of the result)."""
     _req(raw, "raw", torch.float32, 2); _req(slot_mapping, "slot_mapping", torch.int64, 1)
@@ -630,8 +630,8 @@ def latent_norm_store(raw, gain_q, gain_c, pool, slot_mapping, q_n, c_n, eps, sy
     status = torch.zeros(1, dtype=torch.int32, device=raw.device)
     with torch.cuda.device(raw.device):
         check(lib.logismos_launch_latent_norm_store(_p(raw), raw.shape[1], _p(gain_q), _p(gain_c), _p(cq), _p(pool), _p(slot_mapping), rows, qw, q_n,
-                                                    cw, c_n, float(eps), pool.shape[0] * 16, int(pool.dtype == torch.float32), _p(status), _stream()),
-              "latent_norm_store")
+                                                    cw, c_n, float(eps), pool.shape[0] * 16, int(pool.dtype == torch.float32), int(zero_raw),
+                                                    _p(status), _stream()), "latent_norm_store")
         _done(sync)
         if sync and int(status.item()) != 0:
             raise InvalidOp("latent_norm_store: slot outside the pool")

@@ -177,6 +177,9 @@ def test_latent_norm_and_store(dtype, tol, qn, qw, cn, cw):
     assert row_rel(flat[slots, :cn], R.rms_norm(raw[:, qw:qw + cn], gc[:cn], eps)) <= tol and not flat[slots, cn:].any()
     rest = np.setdiff1d(np.arange(blocks * 16), slots)
     assert (flat[rest] == 3.0).all()
+    acc = f32(raw)
+    assert np.array_equal(to_np(ops.latent_norm_store(acc, f32(gq), f32(gc), pool, torch.from_numpy(slots.astype(np.int64)).to(DEV), qn, cn, eps, zero_raw=True)), cq)
+    assert not to_np(acc).any()
     with pytest.raises(ops.InvalidOp):
         ops.latent_norm_store(f32(raw[:1]), f32(gq), f32(gc), pool, torch.tensor([blocks * 16], device=DEV), qn, cn, eps)
 
