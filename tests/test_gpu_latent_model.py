@@ -10,6 +10,7 @@ import numpy as np
 import pytest
 
 import latent_reference as R
+from latent_weights import TINY_LATENT, config, layer, pack
 from logismos_b200.cache import BlockAllocator, SlotAllocator
 from logismos_b200.embed import ComputeError, InputTooLong
 from logismos_b200.generate import generate, sampling_chain
@@ -21,17 +22,6 @@ pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 
-def layer(heads, dim, vdim, q_rank, kv_rank, ff, limit=1.0, scale=None):
-    return {"type": "latent_attention",
-            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": scale or 1.7 / np.sqrt(dim)},
-            "mlp": {"kind": "dense", "ff": ff, "limit": limit} if ff else None}
-
-
-def config(vocab, width, taps, layers, eps=1e-5, cap=6.0):
-    return {"architecture": "Vofosun", "vocab": vocab, "width": width, "canon": {"taps": taps}, "norm": {"eps": eps}, "logit_softcap": cap,
-            "layers": layers}
-
-
 CONFIGS = {
     # unequal layers: value size above and below the query size, a layer without feed-forward, nothing a multiple of 64
     "uneven": config(301, 136, 3, [layer(5, 24, 40, 72, 80, 200, 1.3), layer(3, 80, 16, 40, 200, 0), layer(2, 130, 70, 50, 144, 90, 0.6)]),
@@ -39,7 +29,7 @@ CONFIGS = {
     "heads": config(97, 64, 1, [layer(36, 16, 16, 96, 576, 64, 2.0), layer(18, 64, 64, 64, 320, 128, 0.4)], eps=0.05, cap=3.0),
     # one head of one latent, six taps
     "narrow": config(64, 40, 6, [layer(1, 8, 12, 16, 24, 48, 1.0), layer(2, 12, 8, 8, 16, 0), layer(1, 16, 16, 24, 40, 33, 0.8)], cap=20.0),
-    "plain": config(200, 128, 4, [layer(4, 32, 32, 64, 64, 256, 1.2)] * 2),
+    "plain": TINY_LATENT,
 }
 TOLS = {"float32": 2e-4, "bfloat16": 4e-2}
 
@@ -84,22 +74,6 @@ class Harness:
 
     def drop(self, sid):
         self.blocks.release(sid); self.slots.release(sid); self.hist.pop(sid)
-
-
-def pack(cfg, w):
-    b = {k: R.bf16_bits(v) for k, v in w.items()}
-    out = {"embed": b["embed"], "final_norm": b["final.norm"], "head": b["head"], "layers": []}
-    for i, lc in enumerate(cfg["layers"]):
-        p = "l%d." % i
-        y = {"norm1": b[p + "norm1"], "conv1": b[p + "canon1"], "dwa": b[p + "dwa"]}
-        for n in ("dq", "dq.norm", "uq", "dkv", "dkv.norm", "uk", "uv", "o"):
-            y[n.replace(".", "_")] = b[p + "mix." + n]
-        if lc["mlp"]:
-            y["conv2"] = b[p + "canon2"]
-            for n in ("gate", "up", "down"):
-                y[n], y[n + "_b"] = b[p + "mlp." + n], b[p + "mlp." + n + ".b"]
-        out["layers"].append(y)
-    return out
 
 
 def tokens(rng, cfg, n):
