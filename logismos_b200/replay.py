@@ -29,6 +29,7 @@ class Replay:
     def step(self, entries: List[dict]) -> np.ndarray:
         """Runs the tokens of all entries as one batch; the logits at their wanted places, fp32 [wanted, vocab]."""
         ids, cached, new, tables, slots, want = [], [], [], [], [], []
+        entries = [e for e in entries if e["tokens"]]
         for e in entries:
             rid, toks = e["id"], e["tokens"]
             done = self.cached.get(rid, 0)

@@ -131,7 +131,7 @@ def random_weights(cfg, seed):
     for name, shape in tensor_shapes(cfg).items():
         z = rng.standard_normal(shape)
         leaf = name.split(".", 1)[1] if "." in name else name
-        if leaf in ("norm1", "norm"):                   # stored around zero
+        if leaf in ("norm1", "norm"):                   # offsets from 1
             v = 0.3 * z
         elif name.endswith((".dq.norm", ".dkv.norm")):  # plain gains
             v = 1.0 + 0.3 * z
