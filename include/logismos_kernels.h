@@ -114,6 +114,8 @@ uint32_t logismos_launch_linear_t_bf16(const void* a_bf16, const void* w_bf16,
  *                     clamp(up, -limit, limit), alpha = p0, limit = p1, shift = p2; rows (and bias)
  *                     interleaved as for LG_EPI_SWIGLU, n % 64 == 0 */
 enum { LG_EPI_F32 = 3, LG_EPI_GLU_CLAMP = 4 };
+/*   LG_EPI_RELU2      out bf16 [m, n]      = max(acc + bias, 0)^2 */
+enum { LG_EPI_RELU2 = 5 };
 uint32_t logismos_launch_linear_t_act_bf16(const void* a_bf16, const void* w_bf16, const void* bias_f32,
                                            void* out, int32_t m, int32_t n, int32_t k, int32_t lda,
                                            int32_t ldc, int32_t epilogue, float p0, float p1, float p2,
@@ -121,15 +123,39 @@ uint32_t logismos_launch_linear_t_act_bf16(const void* a_bf16, const void* w_bf1
 /* The same contract for few rows (decode steps): the weights are streamed once and shared by up to 64
  * rows, the reduction order is fixed. W must be static (it is requested before the preceding kernel has
  * finished: LG_EPI_STATIC_W is implied). batch independent products are done in one launch, entry b at
- * a + b * a_stride, w + b * w_stride, out + b * out_stride (elements). All five epilogues; k % 32 == 0,
+ * a + b * a_stride, w + b * w_stride, out + b * out_stride (elements). All six epilogues; k % 32 == 0,
  * lda % 8 == 0, strides of a and w multiples of 8; a and w 16-byte aligned. */
 uint32_t logismos_launch_linear_small_bf16(const void* a_bf16, const void* w_bf16, const void* bias_f32,
                                            void* out, int32_t m, int32_t n, int32_t k, int32_t lda,
                                            int32_t ldc, int32_t batch, int64_t a_stride, int64_t w_stride,
                                            int64_t out_stride, int32_t epilogue, float p0, float p1,
                                            float p2, void* stream);
+/* Several projections of the same rows in one launch, each block of columns with its own input: columns
+ * [end[g - 1], end[g]) of the output are rows of W applied to activation copy g, copy g standing at a + g * m *
+ * lda. Columns below n_main go to out (bf16 [m, n_main], row stride ldc), the others to tail (fp32, row stride
+ * ld_tail), with a soft cap tail_cap tanh(. / tail_cap) when tail_cap > 0. The ends and n_main are multiples of
+ * 128 (the last end is n), n a multiple of 16. The three launchers take the routes of the three above: tcgen05
+ * tiles, weights streamed once for few rows, and fp32 (out and tail fp32). */
+#define LG_MAX_LINEAR_GROUPS 8
+typedef struct lg_linear_groups {
+  int32_t n_groups;
+  int32_t end[LG_MAX_LINEAR_GROUPS];
+  int32_t n_main;
+  void* tail;
+  int32_t ld_tail;
+  float tail_cap;
+} lg_linear_groups_t;
+uint32_t logismos_launch_linear_groups_tc_bf16(const void* a_bf16, const void* w_bf16, void* out, int32_t m, int32_t n,
+                                               int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
+                                               void* status_i32, void* stream);
+uint32_t logismos_launch_linear_groups_small_bf16(const void* a_bf16, const void* w_bf16, void* out, int32_t m, int32_t n,
+                                                  int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
+                                                  void* stream);
+uint32_t logismos_launch_linear_groups_f32(const void* a_f32, const void* w_bf16, void* out_f32, int32_t m, int32_t n,
+                                           int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
+                                           void* stream);
 /* The batched contract with fp32 activations and outputs, true fp32 products and sums over the bf16
- * weights (which fp32 represents exactly). Epilogues LG_EPI_F32, LG_EPI_RESID_F32, LG_EPI_GLU_CLAMP (fp32
+ * weights (which fp32 represents exactly). Epilogues LG_EPI_F32, LG_EPI_RESID_F32, LG_EPI_GLU_CLAMP, LG_EPI_RELU2 (fp32
  * out); k % 16 == 0, lda % 4 == 0, strides of a and w multiples of 4. */
 uint32_t logismos_launch_linear_f32(const void* a_f32, const void* w_bf16, const void* bias_f32, void* out_f32,
                                     int32_t m, int32_t n, int32_t k, int32_t lda, int32_t ldc, int32_t batch,
@@ -657,6 +683,133 @@ int32_t logismos_build_decode_chunks(const int32_t* host_context_lens, int32_t n
  * least 32768 / head_dim CTAs (chunks x kv heads); 512 otherwise. Host-side, no device work. */
 int32_t logismos_pick_decode_chunk(const int32_t* host_context_lens, int32_t n_seqs,
                                    int32_t n_kv_heads, int32_t head_dim);
+
+/* ---- decoder stacks of state-space and parallel attention / time-mixing layers ------------------------------ */
+
+/* Output norm of a sublayer: x f32 [rows, ld] += layer_norm(src) * w + b over n columns; h (may be NULL) receives
+ * the new row in the activation format (bf16, or fp32 with out_f32). x NULL: h = layer_norm(src row) alone.
+ * w NULL: no norm, h = x. row_idx_i32 (may be NULL) selects the rows of src. zero_src: src is cleared once read (an
+ * accumulation buffer). */
+uint32_t logismos_launch_post_norm(void* src_f32, int32_t zero_src, const void* row_idx_i32, int32_t n_src_rows,
+                                   void* x_f32, const void* w_f32, const void* b_f32, void* h, int32_t out_f32,
+                                   int32_t rows, int32_t n, int32_t ld, float eps, void* status_i32, void* stream);
+/* The same for one token per sequence, with the mixes of the next sublayer: copy 0 of h [1 + n_mix][rows][ld] is x,
+ * copy s is x + (x' - x) * mu[s - 1] with x' the previous token's row (state f32 [slots][2][ld]; the copy `phase`
+ * names is read, the other written). */
+uint32_t logismos_launch_post_norm_shift_decode(void* src_f32, int32_t zero_src, void* x_f32, const void* w_f32,
+                                                const void* b_f32, void* h, int32_t out_f32, const void* mu_f32,
+                                                int32_t n_mix, void* state_f32, const void* state_slots_i32,
+                                                const void* fresh_u8, const void* phase_u8, int32_t rows, int32_t n,
+                                                int32_t ld, float eps, void* stream);
+/* The mixes of ragged sequences from x (seq_ids [rows], cu_seqlens). */
+uint32_t logismos_launch_token_shift(const void* x_f32, void* h, int32_t out_f32, const void* mu_f32, int32_t n_mix,
+                                     void* state_f32, const void* state_slots_i32, const void* fresh_u8,
+                                     const void* phase_u8, const void* seq_ids_i32, const void* cu_seqlens_i32,
+                                     int32_t rows, int32_t ld, void* stream);
+/* fp32 [rows, n] (row stride ld) -> bf16 [rows, 2 width]: rounded values, then what rounding dropped: a GEMM over
+ * [W | W] then sees the input to about 16 bits. */
+uint32_t logismos_launch_split_bf16(const void* in_f32, int32_t ld, void* out_bf16, int32_t rows, int32_t n,
+                                    int32_t width, void* stream);
+
+/* Time mixing with a data-dependent decay per key channel, heads padded to dp = 32, 64, 128 or 256 with zeros:
+ *   o_t = (S + diag(u) k_t v_t^T)^T r_t;  S <- diag(exp(-exp(z_t))) S + k_t v_t^T
+ *   out = o / rms(o) * gain * silu(g) * scale          (rms over the d true channels)
+ * proj holds r, k, v, g of head h at columns off_* + h * dp. z f32 [rows, ld_z] or, when NULL, z = W2 low + w0 with
+ * low f32 [rows, ld_low] and w2 bf16 [heads * dp, ld_w2] (rank columns, a multiple of 32). Sequence i owns rows
+ * cu[i] .. cu[i + 1] and state slot state_slots[i] of state f32 [slots][heads][dp][dp]; fresh[i]: it starts here. */
+typedef struct lg_time_mix {
+  const void* proj;
+  int32_t ld, off_r, off_k, off_v, off_g;
+  const void* z;
+  int32_t ld_z;
+  const void* low;
+  int32_t ld_low;
+  const void* w2;
+  int32_t ld_w2, rank;
+  const void *w0, *u, *gain;    /* f32 [heads * dp] */
+  void* state;
+  const void *state_slots, *fresh, *cu;
+  void* out;
+  int32_t ld_out, heads, d, dp;
+  float scale, eps;
+} lg_time_mix_t;
+/* Token by token: decode steps, fp32, any dp. */
+uint32_t logismos_launch_time_mix_step(const lg_time_mix_t* args, int32_t n_seqs, int32_t is_f32, void* stream);
+
+/* State-space mixer with a scalar decay per head; np and vp are powers of two in 16 .. 256 with zero padding:
+ *   x, B, C <- silu(conv);  dt <- softplus(dt + dt_bias)
+ *   S <- exp(-exp(log_a) dt) S + dt B x^T;  y = S^T C + skip x
+ * proj holds z [heads * vp] | x [heads * vp] | B [groups * np] | C [groups * np]; dt f32 [rows, ld_dt]. conv_w f32
+ * [taps][channels], channels = heads * vp + 2 groups * np; conv_state f32 [slots][2][taps - 1][channels] (phase as
+ * above); state f32 [slots][heads][np][vp]. */
+typedef struct lg_ssd {
+  const void* proj;
+  int32_t ld;
+  const void* dt;
+  int32_t ld_dt;
+  const void *conv_w, *conv_b;
+  void* conv_state;
+  int32_t taps;
+  const void *dt_bias, *log_a, *skip;
+  void* state;
+  const void *state_slots, *fresh, *phase, *cu;
+  void* y;
+  int32_t ld_y, heads, groups, np, vp;
+  void* xbc;                    /* chunked form: bf16 [rows, ld_xbc], the convolved channels */
+  int32_t ld_xbc;
+} lg_ssd_t;
+/* Token by token, convolution included: decode steps, fp32, any size. */
+uint32_t logismos_launch_ssd_step(const lg_ssd_t* args, int32_t n_seqs, int32_t is_f32, void* stream);
+/* out = y silu(z), divided in `parts` equal parts of the heads * v true channels by each part's root mean square,
+ * times gain. Rows are laid out [heads][vp]. */
+uint32_t logismos_launch_gated_group_norm(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32,
+                                          void* out, int32_t ld_out, int32_t is_f32, int32_t rows, int32_t heads,
+                                          int32_t v, int32_t vp, int32_t parts, float eps, void* stream);
+
+/* Attention whose scores are capped and biased by distance: score = cap tanh(q . k scale / cap) + bias(i - j), with
+ * queries and keys of unit root mean square and an output gate. bias f32 [n_heads][far + 1] in units of log2, the
+ * entry `far` standing for every larger distance; cap 0: no cap. gate: activation format, head h of a row at h *
+ * head_dim; the output is multiplied by sigmoid(gate) * gate_scale. */
+typedef struct lg_score_bias {
+  float scale, cap;
+  const void* bias;
+  int32_t far;
+  float max_abs_bias;           /* largest |bias|, natural units */
+  const void* gate;
+  int32_t ld_gate;
+  float gate_scale;
+} lg_score_bias_t;
+/* Queries (in place) and keys of packed rows q [n_heads * head_dim] | k [n_kv * head_dim] | v are divided by their
+ * root mean square over dim channels, queries multiplied by 1 + coef ln(floor((pos + 1) / every) + 1) (coef 0:
+ * none); keys and values go to their cache slots. head_dim 64, 128 or 256. */
+uint32_t logismos_launch_unit_qk_store(void* qkv, int32_t ld, void* k_pool, void* v_pool, const void* slot_mapping_i64,
+                                       const void* positions_i32, int32_t rows, int32_t n_heads, int32_t n_kv_heads,
+                                       int32_t head_dim, int32_t dim, float eps, float coef, float every,
+                                       int64_t n_pool_slots, int32_t is_f32, void* status_i32, void* stream);
+/* Decode rows (one query per sequence; q row stride ld_q): the cache already holds the new token. Scratch as
+ * logismos_paged_decode_scratch_bytes; any number of query heads per key head. */
+uint32_t logismos_launch_bias_attention_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool,
+                                                    const void* block_tables, const void* context_lens,
+                                                    const void* chunk_offsets, void* out, int32_t ld_out, void* scratch,
+                                                    int32_t n_seqs, int32_t total_chunks, int32_t chunk_tokens,
+                                                    int32_t max_blocks, int32_t n_pool_blocks, int32_t n_heads,
+                                                    int32_t n_kv_heads, int32_t head_dim, const lg_score_bias_t* score,
+                                                    void* status_i32, void* stream);
+/* Prompt rows over their sequences' cached keys (gathered through the block tables into scratch,
+ * logismos_paged_prefix_attention_scratch_bytes), causal, on the tcgen05 tiles. */
+uint32_t logismos_launch_bias_attention_prefix_bf16(const void* q, int32_t ld_q, const void* cu_seqlens_q, const void* kv_lens,
+                                                    const void* k_pool, const void* v_pool, const void* block_tables,
+                                                    int32_t max_blocks, int32_t n_pool_blocks, void* out, int32_t ld_out,
+                                                    void* scratch, int32_t n_q_tokens, int32_t total_kv_tokens,
+                                                    int32_t n_seqs, int32_t max_q_len, int32_t max_kv_len, int32_t n_heads,
+                                                    int32_t n_kv_heads, int32_t head_dim, const lg_score_bias_t* score,
+                                                    void* status_i32, void* stream);
+/* Every row over its sequence's cached keys in fp32 (seq_ids, positions per row). */
+uint32_t logismos_launch_bias_attention_f32(const void* q_f32, int32_t ld_q, const void* k_pool, const void* v_pool,
+                                            const void* block_tables, const void* seq_ids_i32, const void* positions_i32,
+                                            void* out_f32, int32_t ld_out, int32_t rows, int32_t max_blocks,
+                                            int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
+                                            const lg_score_bias_t* score, void* status_i32, void* stream);
 
 #ifdef __cplusplus
 }

@@ -320,6 +320,79 @@ int32_t lg_latent_launches_last_step(const void* model);
 int32_t lg_latent_device_status(void* model);
 
 /* ====================================================================================
+ * Decoder step over a stack of state-space and parallel (attention beside time mixing) layers (Katadra), post-norm.
+ * No reference counterpart; the contract is that of lg_decoder_step. Weights are bf16, dense.
+ *   x = embed[id];  x += norm1(mixer(x));  with a feed-forward x += norm2(W_down max(W_up x, 0)^2);  logits = head norm(x)
+ *   norms: layer norms with weight and bias
+ *   LG_MIXER_SSD: [z | x | B | C | dt] = W_in h, convolution, scalar-decay recurrence, gate, norm in parts, W_o
+ *     (lg_ssd_t, logismos_launch_gated_group_norm)
+ *   LG_MIXER_PARALLEL: left_scale * attention(h) + right_scale * time_mixing(h); attention without positions, unit
+ *     queries and keys, capped scores, a learned bias by distance bucket, a query temperature and an output gate
+ *     (lg_score_bias_t); time mixing with token shift and a low-rank data-dependent decay (lg_time_mix_t)
+ * A layer may use the tensors of another one (weights_of), with a cache and states of its own. is_f32 as for
+ * lg_latent_config_t; in both formats the residual stream, norms, scores, decays, step sizes and states are fp32.
+ * ==================================================================================== */
+enum { LG_MIXER_SSD = 0, LG_MIXER_PARALLEL = 1 };
+typedef struct lg_mixer_layer_config {
+  int32_t kind;
+  int32_t weights_of;           /* layer whose tensors are used; its own index: its own */
+  int32_t ff;                   /* 0: no feed-forward */
+  /* state-space */
+  int32_t ssd_heads, ssd_vdim, ssd_state, ssd_groups, ssd_norm_groups, ssd_taps;
+  /* attention: sizes <= 256; bias_rows rows of the bias table, distances from bias_max on share the last one */
+  int32_t heads, kv_heads, dim, vdim, bias_rows, bias_max;
+  float scale, softcap, temp_coef, temp_every;
+  /* time mixing */
+  int32_t tm_heads, tm_dim, tm_rank;
+  float left_scale, right_scale;
+} lg_mixer_layer_config_t;
+typedef struct lg_mixer_config {
+  int32_t vocab, width, n_layers;
+  float norm_eps;
+  int32_t is_f32;
+  int32_t n_pool_blocks;        /* cache blocks of 16 tokens per attention layer */
+  int32_t max_blocks_per_seq, max_step_tokens, max_step_seqs;
+  int32_t n_state_slots;        /* recurrent, convolution and shift states */
+  int32_t max_out_rows;
+  int32_t keep_layers;          /* != 0: the stream after every layer is kept (lg_mixer_snapshot) */
+  const lg_mixer_layer_config_t* layers;
+} lg_mixer_config_t;
+/* bf16 values on the host, [out, in]; entries of the other kind of mixer, of a missing feed-forward and of a layer
+ * with weights_of are NULL. mu [5] in the order r, k, v, g, w. */
+typedef struct lg_mixer_layer_weights {
+  const void *norm1, *norm1_b, *norm2, *norm2_b, *up, *down;
+  const void *in, *conv, *conv_b, *dt_bias, *A_log, *D, *norm, *o;
+  const void *left_q, *left_k, *left_v, *left_rel, *left_g, *left_o;
+  const void* mu[5];
+  const void *right_r, *right_k, *right_v, *right_g, *right_w1, *right_w2, *right_w0, *right_u, *right_norm, *right_o;
+} lg_mixer_layer_weights_t;
+typedef struct lg_mixer_weights {
+  const void *embed, *final_norm, *final_norm_b, *head;
+  const lg_mixer_layer_weights_t* layers;
+} lg_mixer_weights_t;
+
+uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_mixer_weights_t* w, void** model);
+/* The same from a bf16 safetensors file with exactly these tensors: embed, final.norm, head and, per layer i that
+ * owns tensors, l<i>.norm1, with a feed-forward l<i>.norm2, l<i>.mlp.{up,down}; l<i>.mix.{in,conv,conv.b,dt_bias,
+ * A_log,D,norm,o} or l<i>.mix.left.{q,k,v,rel,g,o} and l<i>.mix.right.{mu.r,mu.k,mu.v,mu.g,mu.w,r,k,v,g,w1,w2,w0,u,
+ * norm,o}; every norm of the stack also as .b. bias_rows and tm_rank are taken from the tensors. */
+uint32_t lg_mixer_load(int32_t device, const char* path, const lg_mixer_config_t* cfg, void** model);
+void lg_mixer_destroy(void* model);
+/* Step, logits and diagnostics as for lg_latent_*. Recurrent states are updated in place: a step that failed part-way
+ * leaves those of its sequences undefined, and lg_mixer_replay_device (timing) moves them on. */
+uint32_t lg_mixer_step(void* model, const uint32_t* host_ids, const int32_t* host_cached_lens, const int32_t* host_new_lens,
+                       int32_t n_seqs, const int32_t* host_block_tables, const int32_t* host_state_slots,
+                       const int32_t* host_out_rows, int32_t n_out, uint32_t* host_next_tokens);
+uint32_t lg_mixer_replay_device(void* model, void* stream);
+uint32_t lg_mixer_last_logits(void* model, int32_t n_out, float* host_out);
+void* lg_mixer_logits_device(void* model);
+/* The stream of the last step before the first layer (j = 0) and after layer j - 1, fp32 [tokens, width], rows in the
+ * order of host_ids; needs keep_layers. */
+uint32_t lg_mixer_snapshot(void* model, int32_t j, int32_t n_tokens, float* host_out);
+int32_t lg_mixer_launches_last_step(const void* model);
+int32_t lg_mixer_device_status(void* model);
+
+/* ====================================================================================
  * Tensor-parallel exchange over NVLink peer memory (ranks = processes on different GPUs of one node).
  * No reference counterpart (the reference is single-device, README.md:19-21). One kernel per rank
  * writes the local partial sum into every peer's receive buffer with plain peer stores, raises a

@@ -151,6 +151,28 @@ def _declare(l, partial=False):
         "lg_latent_replay_device": [vp, vp],
         "lg_latent_last_logits": [vp, i32, vp],
         "lg_latent_snapshot": [vp, i32, i32, vp],
+        # state-space / parallel decoder
+        "logismos_launch_linear_groups_tc_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp, vp],
+        "logismos_launch_linear_groups_small_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
+        "logismos_launch_linear_groups_f32": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
+        "logismos_launch_post_norm": [vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, vp],
+        "logismos_launch_post_norm_shift_decode": [vp, i32, vp, vp, vp, vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, f32, vp],
+        "logismos_launch_token_shift": [vp, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, vp],
+        "logismos_launch_split_bf16": [vp, i32, vp, i32, i32, i32, vp],
+        "logismos_launch_time_mix_step": [vp, i32, i32, vp],
+        "logismos_launch_ssd_step": [vp, i32, i32, vp],
+        "logismos_launch_gated_group_norm": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp],
+        "logismos_launch_unit_qk_store": [vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, f32, f32, i64, i32, vp, vp],
+        "logismos_launch_bias_attention_decode_bf16": [vp, i32, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
+        "logismos_launch_bias_attention_prefix_bf16": [vp, i32, vp, vp, vp, vp, vp, i32, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32,
+                                                       vp, vp, vp],
+        "logismos_launch_bias_attention_f32": [vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
+        "lg_mixer_create": [i32, vp, vp, C.POINTER(vp)],
+        "lg_mixer_load": [i32, C.c_char_p, vp, C.POINTER(vp)],
+        "lg_mixer_step": [vp, vp, vp, vp, i32, vp, vp, vp, i32, vp],
+        "lg_mixer_replay_device": [vp, vp],
+        "lg_mixer_last_logits": [vp, i32, vp],
+        "lg_mixer_snapshot": [vp, i32, i32, vp],
     }
     # everything that does not return a status
     other = {
@@ -192,6 +214,10 @@ def _declare(l, partial=False):
         "lg_latent_device_status": ([vp], i32),
         "lg_latent_destroy": ([vp], None),
         "lg_latent_logits_device": ([vp], vp),
+        "lg_mixer_launches_last_step": ([vp], i32),
+        "lg_mixer_device_status": ([vp], i32),
+        "lg_mixer_destroy": ([vp], None),
+        "lg_mixer_logits_device": ([vp], vp),
         "logismos_latent_gather_rows": ([i32, i32], i32),
         "logismos_pick_latent_chunk": ([vp, i32, i32], i32),
         "logismos_latent_max_chunks": ([i32], i32),

@@ -16,6 +16,7 @@
 
 #include "common.cuh"
 #include "logismos_kernels.h"
+#include "score_bias.cuh"
 
 namespace {
 
@@ -283,7 +284,8 @@ LG_DEVINL void stage_block(uint32_t sbase, const __nv_bfloat16* kpool, const __n
   }
 }
 
-template <int HD, int kDecWarps, int kDecStages>
+// EXT: capped and biased scores, gated output, and 16 query heads of a key head per CTA (ScoreExt)
+template <int HD, int kDecWarps, int kDecStages, bool EXT = false>
 __global__ void __launch_bounds__(kDecWarps * 32)
 paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ kpool,
                     __nv_bfloat16* __restrict__ vpool, const __nv_bfloat16* __restrict__ new_k,
@@ -291,13 +293,16 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
                     const int* __restrict__ ctx_lens, const int* __restrict__ chunk_offsets,
                     __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
                     int* __restrict__ status, int n_seqs, int chunk_tokens, int max_blocks, int n_pool_blocks,
-                    int n_heads, int n_kv, float sl2) {
+                    int n_heads, int n_kv, float sl2, ScoreExt ext) {
   lg::pdl_prologue();
   extern __shared__ __align__(128) uint8_t smem[];
-  const int chunk_id = blockIdx.x, kvh = blockIdx.y;
+  const int groups = EXT ? (n_heads / n_kv + 15) / 16 : 1;
+  const int chunk_id = blockIdx.x, kvh = blockIdx.y / groups, r_base = (blockIdx.y % groups) * 16;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, c = lane & 3;
-  const int n_rep = n_heads / n_kv;
+  const int n_rep = EXT ? min(16, n_heads / n_kv - r_base) : n_heads / n_kv;  // query heads of this CTA
+  const int head0 = kvh * (n_heads / n_kv) + r_base;
+  const int64_t q_stride = EXT ? ext.ld_q : (int64_t)n_heads * HD;
   constexpr int D = HD, kRowBytes = HD * 2, DT = HD / 8, CH = HD / 8;
   constexpr int kDecStageBytes = DecCfg<HD, kDecWarps, kDecStages>::kStageBytes;
   const int row_elems = n_kv * D;
@@ -342,7 +347,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
   for (int u = tid; u < 16 * CH; u += kDecWarps * 32) {
     const int row = u / CH, chunk = u % CH;
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (row < n_rep) v = __ldg(reinterpret_cast<const uint4*>(q + ((int64_t)seq * n_heads + kvh * n_rep + row) * D + chunk * 8));
+    if (row < n_rep) v = __ldg(reinterpret_cast<const uint4*>(q + seq * q_stride + (head0 + row) * D + chunk * 8));
     *reinterpret_cast<uint4*>(sq + (tile_addr<HD>(sq_a, row, chunk) - sq_a)) = v;
   }
   __syncthreads();
@@ -355,6 +360,14 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
 #pragma unroll
     for (int i = 0; i < 4; ++i) o[j][i] = 0.0f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+  const float *bias0 = nullptr, *bias1 = nullptr;
+  float far0 = 0.0f, far1 = 0.0f;  // bias of every distance >= far
+  if (EXT) {
+    bias0 = ext.bias + (int64_t)(head0 + min(g, n_rep - 1)) * (ext.far + 1);
+    bias1 = ext.bias + (int64_t)(head0 + min(g + 8, n_rep - 1)) * (ext.far + 1);
+    far0 = __ldg(bias0 + ext.far);
+    far1 = __ldg(bias1 + ext.far);
+  }
 
   // ---- per-warp pipeline over this warp's blocks: blk = first + warp, + kDecWarps, ... ----
   const int blk_begin = tok_begin / kBlock, blk_end = (tok_end + kBlock - 1) / kBlock;
@@ -388,6 +401,18 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
     float s[2][4];
     if (valid_block) {
       qk_tile<2, HD>(qf, sb, 0, lane, s);
+      if (EXT) {
+        const int d0 = ctx - 1 - blk * kBlock;  // distance of the block's first key
+        const bool near = d0 - (kBlock - 1) < ext.far;
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int dist = min(max(d0 - 8 * t - 2 * c - e, 0), ext.far);
+            s[t][e] = ext.score(s[t][e], near ? __ldg(bias0 + dist) : far0);
+            if (n_rep > 8) s[t][2 + e] = ext.score(s[t][2 + e], near ? __ldg(bias1 + dist) : far1);
+          }
+      }
     } else {
 #pragma unroll
       for (int t = 0; t < 2; ++t)
@@ -452,13 +477,16 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
       f[w] = (mw == -INFINITY) ? 0.0f : exp2f((mw - M) * sl2);
       L += sml[(w * 16 + r) * 2 + 1] * f[w];
     }
-    const int head = kvh * n_rep + r;
+    const int head = head0 + r;
 #pragma unroll
     for (int d = tid; d < D; d += kDecWarps * 32) {
       float acc = 0.0f;
 #pragma unroll
       for (int w = 0; w < kDecWarps; ++w) acc += so[(w * 16 + r) * D + d] * f[w];
-      if (n_chunks == 1) out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
+      if (EXT && n_chunks == 1)
+        out[(int64_t)seq * ext.ld_out + head * D + d] =
+            __float2bfloat16_rn(ext.gated(acc / L, __bfloat162float(ext.gate[(int64_t)seq * ext.ld_gate + head * D + d])));
+      else if (n_chunks == 1) out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
       else part_o[((int64_t)chunk_id * n_heads + head) * D + d] = acc;
     }
     if (n_chunks != 1 && tid == 0) {
@@ -469,9 +497,10 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
 }
 
 // merges the per-chunk partial results of sequences that were split into several chunks
+template <bool EXT = false>
 __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                           const int* __restrict__ chunk_offsets, __nv_bfloat16* __restrict__ out,
-                                          int n_heads, int D, float sl2) {
+                                          int n_heads, int D, float sl2, ScoreExt ext) {
   lg::pdl_prologue();
   const int seq = blockIdx.x, head = blockIdx.y, d = threadIdx.x;
   const int c0 = chunk_offsets[seq], c1 = chunk_offsets[seq + 1];
@@ -485,7 +514,10 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o, cons
     L += part_ml[((int64_t)ck * n_heads + head) * 2 + 1] * f;
     acc += part_o[((int64_t)ck * n_heads + head) * D + d] * f;
   }
-  out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
+  if (EXT)
+    out[(int64_t)seq * ext.ld_out + head * D + d] = __float2bfloat16_rn(ext.gated(acc / L, __bfloat162float(ext.gate[(int64_t)seq * ext.ld_gate + head * D + d])));
+  else
+    out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
 }
 
 // ================================ paged KV store / gather ======================================
@@ -583,7 +615,7 @@ uint32_t logismos_launch_paged_attention_decode_bf16(
         (const __nv_bfloat16*)q, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, (const __nv_bfloat16*)new_k,
         (const __nv_bfloat16*)new_v, (const int*)block_tables, (const int*)context_lens, (const int*)chunk_offsets,
         (__nv_bfloat16*)out, part_o, part_ml, (int*)status, n_seqs, chunk_tokens, max_blocks, n_pool_blocks, n_heads,
-        n_kv_heads, sl2);
+        n_kv_heads, sl2, ScoreExt{});
     return lg::launch_status();
   };
   uint32_t rc;
@@ -600,11 +632,42 @@ uint32_t logismos_launch_paged_attention_decode_bf16(
   if (rc) return rc;
   if (total_chunks > n_seqs) {  // at least one sequence spans several chunks
     dim3 mgrid(n_seqs, n_heads);
-    lg::launch(paged_decode_merge_kernel, mgrid, dim3(head_dim), 0, (cudaStream_t)stream, part_o, part_ml, (const int*)chunk_offsets,
-                                                                           (__nv_bfloat16*)out, n_heads, head_dim, sl2);
+    lg::launch(paged_decode_merge_kernel<false>, mgrid, dim3(head_dim), 0, (cudaStream_t)stream, part_o, part_ml, (const int*)chunk_offsets,
+                                                                           (__nv_bfloat16*)out, n_heads, head_dim, sl2, ScoreExt{});
     rc = lg::launch_status();
   }
   return rc;
+}
+
+uint32_t logismos_launch_bias_attention_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables,
+                                                    const void* context_lens, const void* chunk_offsets, void* out, int32_t ld_out, void* scratch,
+                                                    int32_t n_seqs, int32_t total_chunks, int32_t chunk_tokens, int32_t max_blocks,
+                                                    int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
+                                                    const lg_score_bias_t* score, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (n_seqs <= 0 || total_chunks < n_seqs || chunk_tokens <= 0 || (chunk_tokens % 64) || max_blocks <= 0 || n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 ||
+      (n_heads % n_kv_heads) || (head_dim != 64 && head_dim != 128 && head_dim != 256) || (ld_q % 8) || ld_q < n_heads * head_dim || ld_out < n_heads * head_dim ||
+      !q || !k_pool || !v_pool || !out || !scratch || (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)scratch) & 15) || !score_ok(score, n_heads * head_dim))
+    return lg::kInvalidValue;
+  float* part_o = (float*)scratch;
+  float* part_ml = part_o + (size_t)total_chunks * n_heads * head_dim;
+  const ScoreExt ext = score_ext(score, ld_q, ld_out);
+  const dim3 grid((unsigned)total_chunks, (unsigned)(n_kv_heads * ((n_heads / n_kv_heads + 15) / 16)));
+  auto launch = [&](auto kern, int warps, int smem) -> uint32_t {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+    lg::launch(kern, grid, dim3(warps * 32), smem, (cudaStream_t)stream, (const __nv_bfloat16*)q, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool,
+               (const __nv_bfloat16*)nullptr, (const __nv_bfloat16*)nullptr, (const int*)block_tables, (const int*)context_lens, (const int*)chunk_offsets,
+               (__nv_bfloat16*)out, part_o, part_ml, (int*)status, n_seqs, chunk_tokens, max_blocks, n_pool_blocks, n_heads, n_kv_heads, 1.0f, ext);
+    return lg::launch_status();
+  };
+  uint32_t rc = head_dim == 64 ? launch(paged_decode_kernel<64, 4, 4, true>, 4, DecCfg<64, 4, 4>::kSmem)
+              : head_dim == 128 ? launch(paged_decode_kernel<128, 4, 2, true>, 4, DecCfg<128, 4, 2>::kSmem)
+                                : launch(paged_decode_kernel<256, 3, 2, true>, 3, DecCfg<256, 3, 2>::kSmem);
+  if (rc || total_chunks == n_seqs) return rc;
+  lg::launch(paged_decode_merge_kernel<true>, dim3((unsigned)n_seqs, (unsigned)n_heads), dim3((unsigned)head_dim), 0, (cudaStream_t)stream, (const float*)part_o,
+             (const float*)part_ml, (const int*)chunk_offsets, (__nv_bfloat16*)out, n_heads, head_dim, 1.0f, ext);
+  return lg::launch_status();
 }
 
 uint32_t logismos_launch_paged_kv_store_bf16(const void* k, const void* v, int32_t src_row_stride, void* k_pool,

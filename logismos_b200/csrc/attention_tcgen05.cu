@@ -24,6 +24,7 @@
 
 #include "common.cuh"
 #include "logismos_kernels.h"
+#include "score_bias.cuh"
 #include "tcgen05.cuh"
 #include "turbo3.cuh"
 
@@ -320,12 +321,19 @@ gather_paged_kv_turbo3_kernel(const uint8_t* __restrict__ kpool, const uint8_t* 
   }
 }
 
-template <bool CAUSAL, int HD>
+// Scores of the kernel below: the plain product; capped and biased by distance, with the running maximum; or
+// the same where cap and biases bound every score so tightly that exp2 of it neither over- nor underflows, and no
+// maximum is kept (one pass over the scores, the output never rescaled).
+enum { kPlain = 0, kBiased = 1, kBounded = 2 };
+constexpr int kBiasWindow = 160;  // distances between the 32 rows of a warp and 128 keys
+constexpr float kBoundedLog2 = 80.0f;
+
+template <bool CAUSAL, int HD, int SCORE = kPlain>
 __global__ void __launch_bounds__(192, HD <= 128 ? 2 : 1)
 attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_vt, const int* __restrict__ cu, const int* __restrict__ pstart,
                     const int* __restrict__ kv_lens, __nv_bfloat16* __restrict__ out, int out_stride, int n_heads, int n_kv, int k_off,
-                    float sl2, int* __restrict__ status) {
+                    float sl2, const ScoreExt ext, int* __restrict__ status) {
   lg::pdl_prologue();
   using C = Attn<HD>;
   constexpr int kQBytes = C::kQBytes, kKBytes = C::kKBytes, kVBytes = C::kVBytes, kVTile = C::kVTile;
@@ -432,9 +440,25 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int row = q * 32 + lane;
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const uint32_t t_s = tmem_base + lane_off + kColS, t_o = tmem_base + lane_off + kColO;
-    float m = -1e30f, l = 0.0f;
+    float m = SCORE == kBounded ? 0.0f : -1e30f, l = 0.0f;
     bool ok = true;
+    // biased scores: the table entries of this warp's rows and the block's keys, distance first + w - 127 at window[w]
+    float* window = reinterpret_cast<float*>(bars_gen + 8 * kBars + 16) + q * kBiasWindow;
+    const float* bias = SCORE != kPlain ? ext.bias + (size_t)h * (ext.far + 1) : nullptr;
+    const float far_bias = SCORE != kPlain ? __ldg(bias + ext.far) : 0.0f;
     for (int j = 0; j < nb; ++j) {
+      bool near = false;
+      if (SCORE != kPlain) {
+        const int first = q_off + q0 + q * 32 - j * 128;
+        near = first - 127 < ext.far;
+        if (near) {
+          __syncwarp();
+#pragma unroll
+          for (int w = 0; w < kBiasWindow; w += 32) window[w + lane] = __ldg(bias + min(max(first + w + lane - 127, 0), ext.far));
+          __syncwarp();
+        }
+      }
+      auto score = [&](uint32_t raw, int key) { return ext.score(__uint_as_float(raw), near ? window[lane + 127 - key] : far_bias); };
       if (!mbar_wait_warp(s_full, (uint32_t)j & 1u, abort_flag)) { ok = false; break; }
       tc_fence_after();
       // keys this row may see in this block: [0, lim)
@@ -442,13 +466,20 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       if (CAUSAL) lim = min(lim, q_off + q0 + row + 1 - j * 128);
       const bool full = lim >= 128;
       float mx = -1e30f;
+      if (SCORE != kBounded)
 #pragma unroll
       for (int c2 = 0; c2 < 2; ++c2) {
         uint32_t ra[32], rb[32];
         tc_ld32(t_s + c2 * 64, ra);
         tc_ld32(t_s + c2 * 64 + 32, rb);
         tc_wait_ld();
-        if (full) {
+        if (SCORE == kBiased) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            if (c2 * 64 + i < lim) mx = fmaxf(mx, score(ra[i], c2 * 64 + i));
+            if (c2 * 64 + 32 + i < lim) mx = fmaxf(mx, score(rb[i], c2 * 64 + 32 + i));
+          }
+        } else if (full) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fmaxf(__uint_as_float(ra[i]), __uint_as_float(rb[i])));
         } else {
@@ -461,9 +492,9 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       }
       // The maximum only moves when it would grow by more than 2^8: P then stays below 256 (exact
       // enough in bf16, summed in fp32) and O is rescaled far less often.
-      const float cand = mx * sl2;
+      const float cand = SCORE == kPlain ? mx * sl2 : mx;
       float alpha = 1.0f;
-      if (cand > m + 8.0f) { alpha = fast_exp2(m - cand); m = cand; }
+      if (SCORE != kBounded && cand > m + 8.0f) { alpha = fast_exp2(m - cand); m = cand; }
       float sum = 0.0f;
 #pragma unroll
       for (int c2 = 0; c2 < 2; ++c2) {
@@ -471,7 +502,20 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         tc_ld32(t_s + c2 * 64, ra);
         tc_ld32(t_s + c2 * 64 + 32, rb);
         tc_wait_ld();
-        if (full) {
+        if (SCORE != kPlain) {
+          auto prob = [&](uint32_t raw, int key) {
+            const float e = fast_exp2(SCORE == kBounded ? score(raw, key) : score(raw, key) - m);
+            return full || key < lim ? e : 0.0f;
+          };
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) {
+            const int ka = c2 * 64 + i, kb = ka + 32;
+            const float a0 = prob(ra[i], ka), a1 = prob(ra[i + 1], ka + 1), b0 = prob(rb[i], kb), b1 = prob(rb[i + 1], kb + 1);
+            sum += (a0 + a1) + (b0 + b1);
+            v[i >> 1] = pack_bf16x2(a0, a1);
+            v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
+          }
+        } else if (full) {
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
             const float a0 = fast_exp2(fmaf(__uint_as_float(ra[i]), sl2, -m)), a1 = fast_exp2(fmaf(__uint_as_float(ra[i + 1]), sl2, -m));
@@ -499,7 +543,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       }
       l = l * alpha + sum;
       // S(j) complete means PV(j-1) is complete: O may be rescaled in place
-      if (j > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
+      if (SCORE != kBounded && j > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
 #pragma unroll
         for (int c = 0; c < HD / 32; ++c) {
           uint32_t r[32];
@@ -526,6 +570,20 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         tc_ld32(t_o + c * 32, r);
         tc_wait_ld();
         if (store) {
+          if (SCORE != kPlain) {  // the output gate
+            const uint4* gp = reinterpret_cast<const uint4*>(ext.gate + (size_t)(t0 + q0 + row) * ext.ld_gate + h * HD + c * 32);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const uint4 gv = __ldg(gp + i);
+              const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+              for (int k = 0; k < 4; ++k) {
+                const float2 gf = unpack_bf16x2(gw[k]);
+                r[8 * i + 2 * k] = __float_as_uint(ext.gated(__uint_as_float(r[8 * i + 2 * k]), gf.x));
+                r[8 * i + 2 * k + 1] = __float_as_uint(ext.gated(__uint_as_float(r[8 * i + 2 * k + 1]), gf.y));
+              }
+            }
+          }
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             uint4 w;
@@ -611,7 +669,7 @@ static uint32_t launch_attn_tc(const void* qkv, const void* cu_seqlens, void* ou
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (uint32_t)e;
     lg::launch(kern, grid, dim3(192), smem, s, map_qk, map_qk, map_vt, (const int*)cu_seqlens, pstart, (const int*)nullptr, (__nv_bfloat16*)out,
-                                 n_heads * D, n_heads, n_kv_heads, k_off, sl2, (int*)status);
+                                 n_heads * D, n_heads, n_kv_heads, k_off, sl2, ScoreExt{}, (int*)status);
     return lg::launch_status();
   };
   if (D == 128) return causal ? launch(attn_tcgen05_kernel<true, 128>, Attn<128>::kSmem) : launch(attn_tcgen05_kernel<false, 128>, Attn<128>::kSmem);
@@ -642,7 +700,7 @@ uint32_t logismos_launch_rope_varlen_attention_tc_bf16(void* qkv, const void* co
 }
 
 size_t logismos_paged_prefix_attention_scratch_bytes(int32_t total_kv_tokens, int32_t n_seqs, int32_t n_kv_heads, int32_t head_dim) {
-  if (total_kv_tokens < 0 || n_seqs < 0 || n_kv_heads <= 0 || (head_dim != 128 && head_dim != 256)) return 0;
+  if (total_kv_tokens < 0 || n_seqs < 0 || n_kv_heads <= 0 || (head_dim != 64 && head_dim != 128 && head_dim != 256)) return 0;
   return pstart_bytes(n_seqs) + 2 * (size_t)n_kv_heads * head_dim * (size_t)padded_tokens(total_kv_tokens, n_seqs) * 2;
 }
 
@@ -650,10 +708,10 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
                                    const void* v_pool, const void* block_tables, int32_t max_blocks, int32_t n_pool_blocks, void* out,
                                    void* scratch, int32_t n_q_tokens, int32_t total_kv_tokens, int32_t n_seqs, int32_t max_q_len,
                                    int32_t max_kv_len, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, bool turbo3, void* status,
-                                   void* stream) {
+                                   void* stream, const ScoreExt* ext = nullptr, bool bounded = false) {
   const int D = head_dim;
   if (n_q_tokens < 0 || total_kv_tokens < 0 || n_seqs < 0 || max_q_len < 0 || max_kv_len < 0 || max_blocks <= 0 ||
-      n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 || (D != 128 && D != 256) || (n_heads % n_kv_heads) ||
+      n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 || (D != 128 && D != 256 && !(D == 64 && ext)) || (n_heads % n_kv_heads) ||
       (q_row_stride % 8) || n_heads * D > q_row_stride || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
       ((uintptr_t)k_pool & (turbo3 ? 7 : 15)) || ((uintptr_t)v_pool & (turbo3 ? 7 : 15)) || !scratch || ((uintptr_t)scratch & 255) || !kv_lens ||
       !block_tables || max_kv_len > total_kv_tokens)
@@ -682,7 +740,8 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
       if (D == 128) go(gather_paged_kv_turbo3_kernel<128>, (const uint8_t*)k_pool, (const uint8_t*)v_pool);
       else go(gather_paged_kv_turbo3_kernel<256>, (const uint8_t*)k_pool, (const uint8_t*)v_pool);
     } else {
-      if (D == 128) go(gather_paged_kv_kernel<128>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool);
+      if (D == 64) go(gather_paged_kv_kernel<64>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool);
+      else if (D == 128) go(gather_paged_kv_kernel<128>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool);
       else go(gather_paged_kv_kernel<256>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool);
     }
     uint32_t rc = lg::launch_status();
@@ -694,9 +753,19 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (uint32_t)e;
     lg::launch(kern, grid, dim3(192), smem, s, map_q, map_k, map_vt, (const int*)cu_seqlens_q, pstart, (const int*)kv_lens, (__nv_bfloat16*)out,
-                                 n_heads * D, n_heads, n_kv_heads, 0, sl2, (int*)status);
+                                 ext ? ext->ld_out : n_heads * D, n_heads, n_kv_heads, 0, sl2, ext ? *ext : ScoreExt{}, (int*)status);
     return lg::launch_status();
   };
+  if (ext) {
+    constexpr size_t kWindow = 4 * kBiasWindow * 4;
+    if (bounded)
+      return D == 64 ? launch(attn_tcgen05_kernel<true, 64, kBounded>, Attn<64>::kSmem + kWindow)
+           : D == 128 ? launch(attn_tcgen05_kernel<true, 128, kBounded>, Attn<128>::kSmem + kWindow)
+                      : launch(attn_tcgen05_kernel<true, 256, kBounded>, Attn<256>::kSmem + kWindow);
+    return D == 64 ? launch(attn_tcgen05_kernel<true, 64, kBiased>, Attn<64>::kSmem + kWindow)
+         : D == 128 ? launch(attn_tcgen05_kernel<true, 128, kBiased>, Attn<128>::kSmem + kWindow)
+                    : launch(attn_tcgen05_kernel<true, 256, kBiased>, Attn<256>::kSmem + kWindow);
+  }
   if (D == 128) return launch(attn_tcgen05_kernel<true, 128>, Attn<128>::kSmem);
   return launch(attn_tcgen05_kernel<true, 256>, Attn<256>::kSmem);
 }
@@ -724,6 +793,20 @@ uint32_t logismos_launch_paged_prefix_attention_turbo3_bf16(const void* q, int32
                             stream);
 }
 
+uint32_t logismos_launch_bias_attention_prefix_bf16(const void* q, int32_t ld_q, const void* cu_seqlens_q, const void* kv_lens, const void* k_pool,
+                                                    const void* v_pool, const void* block_tables, int32_t max_blocks, int32_t n_pool_blocks,
+                                                    void* out, int32_t ld_out, void* scratch, int32_t n_q_tokens, int32_t total_kv_tokens,
+                                                    int32_t n_seqs, int32_t max_q_len, int32_t max_kv_len, int32_t n_heads, int32_t n_kv_heads,
+                                                    int32_t head_dim, const lg_score_bias_t* score, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (n_heads <= 0 || !score_ok(score, n_heads * head_dim) || (ld_out % 8) || ld_out < n_heads * head_dim || (score->ld_gate % 8) || ((uintptr_t)score->gate & 15))
+    return lg::kInvalidValue;
+  const ScoreExt ext = score_ext(score, ld_q, ld_out);
+  const bool bounded = ext.capped && (score->cap + score->max_abs_bias) * 1.4426950408889634f <= kBoundedLog2;
+  return launch_prefix_attn(q, ld_q, cu_seqlens_q, kv_lens, k_pool, v_pool, block_tables, max_blocks, n_pool_blocks, out, scratch, n_q_tokens,
+                            total_kv_tokens, n_seqs, max_q_len, max_kv_len, n_heads, n_kv_heads, head_dim, false, status, stream, &ext, bounded);
+}
+
 uint32_t logismos_launch_varlen_attention_kv_tc_bf16(const void* q, int32_t q_row_stride, const void* cu_seqlens_q, const void* kv_lens,
                                                      const void* kv_start, const void* k, const void* v_t, int32_t n_kv_rows, void* out,
                                                      int32_t out_row_stride, int32_t n_q_tokens, int32_t n_seqs, int32_t max_q_len,
@@ -748,7 +831,7 @@ uint32_t logismos_launch_varlen_attention_kv_tc_bf16(const void* q, int32_t q_ro
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (uint32_t)e;
     lg::launch(kern, grid, dim3(192), smem, (cudaStream_t)stream, map_q, map_k, map_vt, (const int*)cu_seqlens_q, (const int*)kv_start, (const int*)kv_lens,
-               (__nv_bfloat16*)out, out_row_stride, n_heads, n_kv_heads, 0, scale * 1.4426950408889634f, (int*)status);
+               (__nv_bfloat16*)out, out_row_stride, n_heads, n_kv_heads, 0, scale * 1.4426950408889634f, ScoreExt{}, (int*)status);
     return lg::launch_status();
   };
   if (D == 64) return launch(attn_tcgen05_kernel<true, 64>, Attn<64>::kSmem);

@@ -1,0 +1,170 @@
+// What the capped, distance-biased attention needs around the shared attention kernels: unit queries and keys with
+// the cache store, and the fp32 form of the attention itself.
+#include "common.cuh"
+#include "logismos_kernels.h"
+#include "recurrent.cuh"
+#include "score_bias.cuh"
+
+namespace {
+
+using namespace lg;
+
+constexpr int kBlockTokens = 16, kThreads = 256;
+
+struct QkArgs {
+  void* qkv;
+  int ld;
+  void* kpool;
+  void* vpool;
+  const int64_t* slots;
+  const int* pos;
+  int rows, heads, n_kv, dim;
+  float eps, coef, every;
+  int64_t n_slots;
+  int* status;
+};
+
+// warp = one head of one row: q (in place), k or v (to the cache); a lane holds HD / 32 neighbouring channels
+template <typename T, int HD>
+__global__ void __launch_bounds__(kThreads)
+unit_qk_store_kernel(QkArgs p) {
+  lg::pdl_prologue();
+  constexpr int E = HD / 32;
+  struct alignas(E * sizeof(T)) Vec { T v[E]; };
+  const int per_row = p.heads + 2 * p.n_kv;
+  const int64_t item = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+  if (item >= (int64_t)p.rows * per_row) return;
+  const int row = (int)(item / per_row), h = (int)(item % per_row), lane = threadIdx.x & 31;
+  T* src = reinterpret_cast<T*>(p.qkv) + (size_t)row * p.ld + h * HD + lane * E;
+  Vec x = *reinterpret_cast<const Vec*>(src);
+  const bool is_v = h >= p.heads + p.n_kv;
+  if (!is_v) {
+    float f[E], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < E; ++i) { f[i] = rec::Io<T>::load(&x.v[i]); ss += f[i] * f[i]; }
+    float m = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+    if (h < p.heads && p.coef != 0.0f) m *= 1.0f + p.coef * logf(floorf(__fdiv_rn((float)(p.pos[row] + 1), p.every)) + 1.0f);
+#pragma unroll
+    for (int i = 0; i < E; ++i) rec::Io<T>::store(&x.v[i], f[i] * m);
+  }
+  if (h < p.heads) {
+    *reinterpret_cast<Vec*>(src) = x;
+    return;
+  }
+  const int64_t slot = p.slots[row];
+  if (slot < 0 || slot >= p.n_slots) {
+    if (lane == 0 && p.status) atomicExch(p.status, 1);
+    return;
+  }
+  const int kvh = h - p.heads - (is_v ? p.n_kv : 0);
+  T* pool = reinterpret_cast<T*>(is_v ? p.vpool : p.kpool);
+  *reinterpret_cast<Vec*>(pool + (size_t)slot * p.n_kv * HD + kvh * HD + lane * E) = x;
+}
+
+// CTA = (row, head), keys in tiles of 64
+constexpr int kTile = 64, kAttnThreads = 128;
+__global__ void __launch_bounds__(kAttnThreads)
+bias_attention_f32_kernel(const float* __restrict__ q, const float* __restrict__ kpool, const float* __restrict__ vpool, const int* __restrict__ tables,
+                          int max_blocks, int n_pool_blocks, const int* __restrict__ seq_ids, const int* __restrict__ pos, float* __restrict__ out,
+                          int n_kv, int hd, float scale, float cap, const float* __restrict__ gate, ScoreExt ext, int* __restrict__ status) {
+  lg::pdl_prologue();
+  __shared__ float sq[256], ss[kTile], red[32];
+  __shared__ int blk_s[kTile / kBlockTokens];
+  const int r = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int kvh = h / (gridDim.y / n_kv), n_keys = pos[r] + 1;
+  const int* table = tables + (size_t)seq_ids[r] * max_blocks;
+  const float* bias = ext.bias + (size_t)h * (ext.far + 1);
+  const size_t row_w = (size_t)n_kv * hd;
+  for (int i = tid; i < hd; i += kAttnThreads) sq[i] = q[(size_t)r * ext.ld_q + h * hd + i];
+  float m = -1e30f, l = 0.0f, acc[2] = {0.f, 0.f};
+  for (int k0 = 0; k0 < n_keys; k0 += kTile) {
+    const int n = min(kTile, n_keys - k0);
+    __syncthreads();
+    if (tid < kTile / kBlockTokens) {
+      const int bi = k0 / kBlockTokens + tid;
+      int b = tid * kBlockTokens < n && bi < max_blocks ? __ldg(table + bi) : -1;
+      if (tid * kBlockTokens < n && (b < 0 || b >= n_pool_blocks)) {
+        if (status) atomicExch(status, 1);
+        b = -1;
+      }
+      blk_s[tid] = b;
+    }
+    __syncthreads();
+    for (int k = warp; k < kTile; k += kAttnThreads / 32) {
+      const int b = blk_s[k / kBlockTokens];
+      float s = 0.0f;
+      if (k < n && b >= 0) {
+        const float* c = kpool + ((size_t)b * kBlockTokens + k % kBlockTokens) * row_w + kvh * hd;
+        for (int i = lane; i < hd; i += 32) s = fmaf(sq[i], c[i], s);
+      }
+      s = warp_sum(s) * scale;
+      if (cap > 0.0f) s = cap * tanhf(s / cap);
+      if (lane == 0) ss[k] = k < n && b >= 0 ? s * 1.4426950408889634f + bias[min(n_keys - 1 - (k0 + k), ext.far)] : -1e30f;
+    }
+    __syncthreads();
+    const float mine = tid < kTile ? ss[tid] : -1e30f;
+    const float m_new = fmaxf(m, block_max(mine, red));
+    const float alpha = exp2f(m - m_new), e = tid < n ? exp2f(mine - m_new) : 0.0f;
+    l = l * alpha + block_sum(e, red);
+    m = m_new;
+    if (tid < kTile) ss[tid] = e;
+    __syncthreads();
+    acc[0] *= alpha;
+    acc[1] *= alpha;
+    for (int k = 0; k < n; ++k) {
+      const int b = blk_s[k / kBlockTokens];
+      if (b < 0) continue;
+      const float* c = vpool + ((size_t)b * kBlockTokens + k % kBlockTokens) * row_w + kvh * hd;
+      if (tid < hd) acc[0] = fmaf(ss[k], c[tid], acc[0]);
+      if (tid + kAttnThreads < hd) acc[1] = fmaf(ss[k], c[tid + kAttnThreads], acc[1]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int d = tid + i * kAttnThreads;
+    if (d < hd) out[(size_t)r * ext.ld_out + h * hd + d] = acc[i] / l * (ext.gate_scale * rec::sigmoid_f(gate[(size_t)r * ext.ld_gate + h * hd + d]));
+  }
+}
+
+}  // namespace
+
+extern "C" {
+
+uint32_t logismos_launch_unit_qk_store(void* qkv, int32_t ld, void* k_pool, void* v_pool, const void* slot_mapping_i64, const void* positions_i32,
+                                       int32_t rows, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, int32_t dim, float eps, float coef,
+                                       float every, int64_t n_pool_slots, int32_t is_f32, void* status_i32, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!qkv || !k_pool || !v_pool || !slot_mapping_i64 || !positions_i32 || rows <= 0 || n_heads <= 0 || n_kv_heads <= 0 || dim <= 0 || dim > head_dim ||
+      (head_dim != 64 && head_dim != 128 && head_dim != 256) || ld < (n_heads + 2 * n_kv_heads) * head_dim || (ld % 8) ||
+      (((uintptr_t)qkv | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15) || (coef != 0.0f && !(every > 0.0f)))
+    return lg::kInvalidValue;
+  const QkArgs p{qkv, ld, k_pool, v_pool, (const int64_t*)slot_mapping_i64, (const int*)positions_i32, rows, n_heads, n_kv_heads, dim, eps, coef, every,
+                 n_pool_slots, (int*)status_i32};
+  const int64_t blocks = ((int64_t)rows * (n_heads + 2 * n_kv_heads) + kThreads / 32 - 1) / (kThreads / 32);
+  if (blocks > 0x7fffffff) return lg::kInvalidValue;
+  auto go = [&](auto kern) {
+    lg::launch(kern, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, p);
+    return lg::launch_status();
+  };
+  if (is_f32) return head_dim == 64 ? go(unit_qk_store_kernel<float, 64>) : head_dim == 128 ? go(unit_qk_store_kernel<float, 128>) : go(unit_qk_store_kernel<float, 256>);
+  return head_dim == 64 ? go(unit_qk_store_kernel<__nv_bfloat16, 64>) : head_dim == 128 ? go(unit_qk_store_kernel<__nv_bfloat16, 128>)
+                                                                                       : go(unit_qk_store_kernel<__nv_bfloat16, 256>);
+}
+
+uint32_t logismos_launch_bias_attention_f32(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables,
+                                            const void* seq_ids_i32, const void* positions_i32, void* out, int32_t ld_out, int32_t rows,
+                                            int32_t max_blocks, int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
+                                            const lg_score_bias_t* score, void* status_i32, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!q || !k_pool || !v_pool || !block_tables || !seq_ids_i32 || !positions_i32 || !out || rows <= 0 || max_blocks <= 0 || n_pool_blocks <= 0 || n_heads <= 0 ||
+      n_heads > 65535 || n_kv_heads <= 0 || n_heads % n_kv_heads || head_dim <= 0 || head_dim > 256 || ld_q < n_heads * head_dim || ld_out < n_heads * head_dim ||
+      !score_ok(score, n_heads * head_dim))
+    return lg::kInvalidValue;
+  const ScoreExt ext = score_ext(score, ld_q, ld_out);
+  lg::launch(bias_attention_f32_kernel, dim3((unsigned)rows, (unsigned)n_heads), dim3(kAttnThreads), 0, (cudaStream_t)stream, (const float*)q, (const float*)k_pool,
+             (const float*)v_pool, (const int*)block_tables, max_blocks, n_pool_blocks, (const int*)seq_ids_i32, (const int*)positions_i32, (float*)out, n_kv_heads,
+             head_dim, score->scale, score->cap, (const float*)score->gate, ext, (int*)status_i32);
+  return lg::launch_status();
+}
+
+}  // extern "C"

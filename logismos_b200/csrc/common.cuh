@@ -111,6 +111,16 @@ LG_DEVINL float block_max(float v, float* red) {
   return t;
 }
 
+// host-side shape rules of lg_linear_groups_t (logismos_kernels.h)
+template <typename Groups>
+inline bool groups_ok(const Groups* g, int n, int ldc) {
+  if (!g || g->n_groups < 1 || g->n_groups > 8 || g->n_main < 0 || g->n_main > n || (g->n_main < n && (g->n_main % 128)) || ldc < g->n_main) return false;
+  for (int i = 0; i < g->n_groups; ++i) {
+    if (g->end[i] <= (i ? g->end[i - 1] : 0) || (i + 1 < g->n_groups && g->end[i] % 128)) return false;
+  }
+  return g->end[g->n_groups - 1] == n && (g->n_main == n || (g->tail && g->ld_tail >= n - g->n_main));
+}
+
 // clamped gated unit: g' = min(g, limit), u' = clamp(u, -limit, limit); g' sigmoid(alpha g') (u' + shift)
 LG_DEVINL float glu_clamp(float g, float u, float alpha, float limit, float shift) {
   g = fminf(g, limit);

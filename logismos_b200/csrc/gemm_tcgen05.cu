@@ -59,12 +59,23 @@ LG_DEVINL void load_bias8(const float* __restrict__ bias, bool vec, float (&b)[8
 // constants of the parametrised epilogues (see LG_EPI_F32 and LG_EPI_GLU_CLAMP)
 struct EpiParams { float p0, p1, p2; };
 
+// internal epilogue of the grouped projections (lg_linear_groups_t): bf16 columns, then an fp32 tail
+constexpr int kEpiGroups = 6;
+
+// activation copy of the tile that starts at column c
+LG_DEVINL int group_of(const lg_linear_groups_t& g, int c) {
+  int i = 0;
+#pragma unroll
+  for (int j = 0; j < LG_MAX_LINEAR_GROUPS - 1; ++j) i += (j + 1 < g.n_groups && c >= g.end[j]) ? 1 : 0;
+  return i;
+}
+
 template <int BN, int EPI>
 __global__ void __launch_bounds__(kThreads, 1)
 linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                         const __grid_constant__ CUtensorMap map_out, const float* __restrict__ bias,
                         void* __restrict__ out, int M, int N, int K, int ldc, int splits, int w_static,
-                        EpiParams ep, int* __restrict__ status) {
+                        EpiParams ep, const lg_linear_groups_t groups, int* __restrict__ status) {
   using C = Cfg<BN>;
   lg::pdl_trigger();
   extern __shared__ uint8_t smem_raw[];
@@ -130,12 +141,14 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
         const int ot = tile % out_tiles, sp = tile / out_tiles;
         const int m_blk = ot % m_tiles, n_blk = ot / m_tiles;
         const int kb0 = sp * kb_per, kb1 = min(all_kb, kb0 + kb_per);
+        // a tile lies in one group of columns; rows beyond M read the next copy's and are not stored
+        const int a_row = m_blk * BM + (EPI == kEpiGroups ? group_of(groups, n_blk * BN) * M : 0);
         for (int kb = kb0; kb < kb1; ++kb) {
           if (!mbar_wait(empty_bar(stage), phase ^ 1u, abort_flag)) { ok = false; break; }
           const bool have_w = pre_w > 0;  // requested before the dependency wait (first stages of the first tile)
           if (!have_w) mbar_expect_tx(full_bar(stage), (uint32_t)C::kStage);
           const uint32_t sa = smem_base + stage * C::kStage;
-          tma_load_2d(sa, &map_a, full_bar(stage), kb * BK, m_blk * BM);
+          tma_load_2d(sa, &map_a, full_bar(stage), kb * BK, a_row);
           if (!have_w) tma_load_2d(sa + C::kStageA, &map_w, full_bar(stage), kb * BK, n_blk * BN);
           else --pre_w;
           if (++stage == C::kStages) { stage = 0; phase ^= 1u; }
@@ -228,12 +241,23 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
           }
           slab_release(b, ncol, row0, ncol < N && row0 < M);
         }
-      } else if (EPI == LG_EPI_BF16) {
+      } else if (EPI == LG_EPI_BF16 || EPI == LG_EPI_RELU2 || EPI == kEpiGroups) {
         for (int c = 0; c < BN; c += 32) {
           uint32_t r[32];
           tc_ld32(t_row + c, r);
           tc_wait_ld();
           const int ncol = n_blk * BN + c;
+          if (EPI == kEpiGroups && ncol >= groups.n_main) {
+            if (row < M) {
+              float* dst = reinterpret_cast<float*>(groups.tail) + (size_t)row * groups.ld_tail + (ncol - groups.n_main);
+#pragma unroll
+              for (int j = 0; j < 32; ++j) {
+                const float v = __uint_as_float(r[j]);
+                if (ncol + j < N) dst[j] = groups.tail_cap > 0.0f ? groups.tail_cap * tanhf(v / groups.tail_cap) : v;
+              }
+            }
+            continue;
+          }
           if (row < M) {
               __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * ldc + ncol;
 #pragma unroll
@@ -245,6 +269,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                     const int e = j * 8 + i * 2;
                     float a = __uint_as_float(r[e]), b = __uint_as_float(r[e + 1]);
                     if (bias) { a += bias[ncol + e]; b += bias[ncol + e + 1]; }
+                    if (EPI == LG_EPI_RELU2) { a = fmaxf(a, 0.0f); b = fmaxf(b, 0.0f); a *= a; b *= b; }
                     w[i] = pack_bf16x2(a, b);
                   }
                   *reinterpret_cast<uint4*>(dst + j * 8) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -356,9 +381,10 @@ __global__ void linear_t_naive_kernel(const __nv_bfloat16* __restrict__ a, const
 
 template <int BN, int EPI>
 uint32_t launch_cfg(const void* a, const void* w, const float* bias, void* out, int m, int n, int k, int lda,
-                    int ldc, int w_static, EpiParams ep, int* status, cudaStream_t stream) {
+                    int ldc, int w_static, EpiParams ep, int* status, cudaStream_t stream, const lg_linear_groups_t& groups = {}) {
   CUtensorMap ma, mw, mo;
-  if (!make_map(&ma, a, (uint64_t)m, (uint64_t)k, (uint64_t)lda, BM)) return lg::kInvalidValue;
+  const int copies = EPI == kEpiGroups ? groups.n_groups : 1;
+  if (!make_map(&ma, a, (uint64_t)m * copies, (uint64_t)k, (uint64_t)lda, BM)) return lg::kInvalidValue;
   if (!make_map(&mw, w, (uint64_t)n, (uint64_t)k, (uint64_t)k, BN)) return lg::kInvalidValue;
   if (EPI == LG_EPI_RESID_F32) {  // fp32 [m, n] in 32 x 32 boxes for the reduce-add epilogue
     if (!make_map(&mo, out, (uint64_t)m, (uint64_t)n, (uint64_t)ldc, 32, true)) return lg::kInvalidValue;
@@ -383,13 +409,13 @@ uint32_t launch_cfg(const void* a, const void* w, const float* bias, void* out, 
   }
   const int items = tiles * splits;
   const int grid = items < sm_count() ? items : sm_count();
-  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, mo, bias, out, m, n, k, ldc, splits, w_static, ep, status);
+  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, mo, bias, out, m, n, k, ldc, splits, w_static, ep, groups, status);
   return lg::launch_status();
 }
 
 template <int EPI>
 uint32_t launch_epi(const void* a, const void* w, const float* bias, void* out, int m, int n, int k, int lda,
-                    int ldc, int w_static, EpiParams ep, int* status, cudaStream_t stream) {
+                    int ldc, int w_static, EpiParams ep, int* status, cudaStream_t stream, const lg_linear_groups_t& groups = {}) {
   // tile width by wave quantisation: time ~ waves(BN) * BN; ties go to the wider tile
   const int sms = sm_count();
   const int mt = (m + BM - 1) / BM;
@@ -398,14 +424,19 @@ uint32_t launch_epi(const void* a, const void* w, const float* bias, void* out, 
   const int cands[3] = {256, 192, 128};
   for (int i = 0; i < 3; ++i) {
     const int bn = cands[i];
+    if (EPI == kEpiGroups) {  // a tile must not straddle two groups
+      bool fits = groups.n_main % bn == 0 || groups.n_main == n;
+      for (int g = 0; g + 1 < groups.n_groups; ++g) fits = fits && groups.end[g] % bn == 0;
+      if (!fits) continue;
+    }
     const long tiles = (long)mt * ((n + bn - 1) / bn);
     const long waves = (tiles + sms - 1) / sms;
     const long cost = waves * bn;
     if (best_cost < 0 || cost < best_cost) { best_cost = cost; best_bn = bn; }
   }
-  if (best_bn == 256) return launch_cfg<256, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream);
-  if (best_bn == 192) return launch_cfg<192, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream);
-  return launch_cfg<128, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream);
+  if (best_bn == 256) return launch_cfg<256, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream, groups);
+  if (best_bn == 192) return launch_cfg<192, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream, groups);
+  return launch_cfg<128, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream, groups);
 }
 
 }  // namespace
@@ -435,8 +466,18 @@ uint32_t logismos_launch_linear_t_act_bf16(const void* a, const void* w, const v
     case LG_EPI_SWIGLU: return launch_epi<LG_EPI_SWIGLU>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
     case LG_EPI_F32: return launch_epi<LG_EPI_F32>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
     case LG_EPI_GLU_CLAMP: return launch_epi<LG_EPI_GLU_CLAMP>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
+    case LG_EPI_RELU2: return launch_epi<LG_EPI_RELU2>(a, w, b, out, m, n, k, lda, ldc, w_static, ep, st, s);
     default: return lg::kInvalidValue;
   }
+}
+
+uint32_t logismos_launch_linear_groups_tc_bf16(const void* a, const void* w, void* out, int32_t m, int32_t n, int32_t k, int32_t lda,
+                                               int32_t ldc, const lg_linear_groups_t* groups, void* status_i32, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (m <= 0 || n <= 0 || k <= 0 || (k % BK) || (n % 16) || (lda % 8) || lda < k || (((uintptr_t)a | (uintptr_t)w | (uintptr_t)out) & 15) ||
+      (ldc % 8) || !lg::groups_ok(groups, n, ldc))
+    return lg::kInvalidValue;
+  return launch_epi<kEpiGroups>(a, w, nullptr, out, m, n, k, lda, ldc, 1, EpiParams{}, (int*)status_i32, (cudaStream_t)stream, *groups);
 }
 
 uint32_t logismos_launch_linear_t_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m,

@@ -28,23 +28,13 @@
 #include "model_util.h"
 #include "safetensors.h"
 #include "step_batch.h"
+#include "weight_pack.h"
 
 namespace {
 
 using namespace lgm;
 
-// Whether a projection of few rows streams its weights (linear_small) instead of running on the tcgen05 tiles. Measured
-// (us, small / tiles): accumulating into the residual, where the tiles split k, 2048 x 10240 at 1 / 8 / 32 rows 14.6 /
-// 12.6, 15.6 / 12.6, 29.0 / 12.6; gated 16384 x 2048 at 8 / 16 / 32 rows 17.8 / 22.7, 19.0 / 22.0, 28.5 / 17.9; head 32768
-// x 2048 at 16 / 32 rows 39.5 / 41.5, 57.2 / 41.1; 1536 x 2048 at 8 / 32 / 64 rows 5.7 / 17.4, 11.6 / 18.2, 20.8 / 19.1.
-inline bool stream_weights(int rows, int n, int k, int epi) {
-  if (epi == LG_EPI_RESID_F32) return logismos_get_deterministic() && rows <= 32;
-  return rows <= ((int64_t)n * k >= (1 << 23) ? 16 : 32);
-}
-
 constexpr int kAccRows = 512;
-
-inline int r64(int v) { return (v + 63) & ~63; }
 
 struct LLayer {
   lg_latent_layer_config_t c{};
@@ -191,45 +181,6 @@ uint32_t run_device(Latent* m, cudaStream_t s) {
   }
   return 0;
 }
-
-// ---- weights: bf16 on the host, read bytewise (file data may be unaligned) -------------------------
-
-inline uint16_t bf_at(const void* p, size_t i) {
-  uint16_t v;
-  std::memcpy(&v, (const uint8_t*)p + 2 * i, 2);
-  return v;
-}
-inline float f_at(const void* p, size_t i) {
-  const uint32_t u = (uint32_t)bf_at(p, i) << 16;
-  float f;
-  std::memcpy(&f, &u, 4);
-  return f;
-}
-
-// offset + w over n values, zero in the padding
-bool upload_vec(Buf& b, const void* src, int n, int padded, float offset) {
-  std::vector<float> v((size_t)padded, 0.0f);
-  for (int i = 0; i < n; ++i) v[(size_t)i] = offset + f_at(src, (size_t)i);
-  return b.upload(v.data(), v.size() * 4);
-}
-
-// filters [n, taps] -> fp32 [taps, padded]
-bool upload_conv(Buf& b, const void* src, int n, int padded, int taps) {
-  std::vector<float> v((size_t)taps * padded, 0.0f);
-  for (int i = 0; i < n; ++i)
-    for (int j = 0; j < taps; ++j) v[(size_t)j * padded + i] = f_at(src, (size_t)i * taps + j);
-  return b.upload(v.data(), v.size() * 4);
-}
-
-struct Mat {  // zero-initialised bf16 matrix under construction
-  int ld;
-  std::vector<uint16_t> v;
-  Mat(int rows, int cols) : ld(cols), v((size_t)rows * cols, 0) {}
-  void row(int dst_row, int dst_col, const void* src, size_t src_elem, int n) {
-    std::memcpy(v.data() + (size_t)dst_row * ld + dst_col, (const uint8_t*)src + 2 * src_elem, (size_t)n * 2);
-  }
-  bool up(Buf& b) { return b.upload(v.data(), v.size() * 2); }
-};
 
 bool upload_layer(Latent* m, LLayer& L, const lg_latent_layer_weights_t& w, int index) {
   const lg_latent_config_t& c = m->cfg;
@@ -457,18 +408,8 @@ uint32_t lg_latent_step(void* model, const uint32_t* host_ids, const int32_t* ca
   m->ready = false;
   if (uint32_t rc = B.build("lg_latent_step", host_ids, cached, newl, n_seqs, tables, state_slots, false)) return rc;
   for (int s = 0; s < n_seqs; ++s) B.phase[s] = m->slot_phase[(size_t)B.state[s]];
-  // wanted rows: caller's token index -> packed row
   int32_t* rows = (int32_t*)B.extra;
-  std::vector<int32_t> packed_row((size_t)B.T);
-  B.caller_rows(packed_row.data());
-  int64_t off = 0;
-  for (int i = 0; i < n_out; ++i) {
-    int64_t t;
-    if (out_rows) t = out_rows[i];
-    else { off += newl[i]; t = off - 1; }
-    if (t < 0 || t >= B.T) { set_error("lg_latent_step: an output row lies outside the step"); return LG_EMB_COMPUTE; }
-    rows[i] = packed_row[(size_t)t];
-  }
+  if (!B.select_rows(out_rows, n_out, newl, rows)) { set_error("lg_latent_step: an output row lies outside the step"); return LG_EMB_COMPUTE; }
   if (!c.is_f32 && B.n_dec > 0) {
     int heads = 1;
     for (const LLayer& L : m->layers) if (L.c.heads > heads) heads = L.c.heads;
@@ -521,13 +462,8 @@ uint32_t lg_latent_snapshot(void* model, int32_t j, int32_t n_tokens, float* hos
   Latent* m = static_cast<Latent*>(model);
   if (!m || !m->ready || j < 0 || j > m->cfg.n_layers || n_tokens != m->batch.T) { set_error("lg_latent_snapshot: bad arguments"); return LG_EMB_COMPUTE; }
   cudaSetDevice(m->device);
-  const size_t Hp = (size_t)m->Hp, W = (size_t)m->cfg.width;
-  std::vector<float> tmp((size_t)n_tokens * Hp);
-  std::vector<int32_t> packed_row((size_t)n_tokens);
-  m->batch.caller_rows(packed_row.data());
   LG_TRY(cudaDeviceSynchronize(), "device synchronize");
-  LG_TRY(cudaMemcpy(tmp.data(), (float*)m->hist.p + (size_t)j * m->cfg.max_step_tokens * Hp, tmp.size() * 4, cudaMemcpyDeviceToHost), "D2H snapshot");
-  for (int t = 0; t < n_tokens; ++t) std::memcpy(host_out + (size_t)t * W, tmp.data() + (size_t)packed_row[(size_t)t] * Hp, W * 4);
+  LG_TRY(m->batch.rows_to_host((const float*)m->hist.p + (size_t)j * m->cfg.max_step_tokens * m->Hp, m->Hp, m->cfg.width, host_out), "D2H snapshot");
   return LG_EMB_OK;
 }
 

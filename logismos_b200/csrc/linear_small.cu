@@ -22,7 +22,19 @@ struct SmallArgs {
   int m, n, k, lda, ldc, epi;
   int64_t a_stride, w_stride, out_stride;  // per batch entry (elements)
   float p0, p1, p2;
+  lg_linear_groups_t groups;               // with kEpiGroups
 };
+
+// internal epilogue of the grouped projections (lg_linear_groups_t): main columns, then an fp32 tail
+constexpr int kEpiGroups = 6;
+
+// activation copy of a block of columns starting at c
+LG_DEVINL int group_of(const lg_linear_groups_t& g, int c) {
+  int i = 0;
+#pragma unroll
+  for (int j = 0; j < LG_MAX_LINEAR_GROUPS - 1; ++j) i += (j + 1 < g.n_groups && c >= g.end[j]) ? 1 : 0;
+  return i;
+}
 
 LG_DEVINL uint4 ldg16(const void* p) { return __ldg(reinterpret_cast<const uint4*>(p)); }
 
@@ -48,7 +60,7 @@ linear_small_kernel(SmallArgs p) {
   }
   const int m0 = blockIdx.y * 8 * NT;
   const __nv_bfloat16* wb = p.w + (size_t)blockIdx.z * p.w_stride;
-  const __nv_bfloat16* ab = p.a + (size_t)blockIdx.z * p.a_stride;
+  const __nv_bfloat16* ab = p.a + (size_t)blockIdx.z * p.a_stride + (p.epi == kEpiGroups ? (size_t)group_of(p.groups, row0[0]) * p.m * p.lda : 0);
   const __nv_bfloat16* wr[MT][2];
 #pragma unroll
   for (int i = 0; i < MT; ++i)
@@ -131,8 +143,14 @@ linear_small_kernel(SmallArgs p) {
       continue;
     }
     if (p.bias) v += p.bias[wrow];
+    if (p.epi == LG_EPI_RELU2) { v = fmaxf(v, 0.0f); v *= v; }
+    if (p.epi == kEpiGroups && wrow >= p.groups.n_main) {
+      reinterpret_cast<float*>(p.groups.tail)[(size_t)r * p.groups.ld_tail + wrow - p.groups.n_main] =
+          p.groups.tail_cap > 0.0f ? p.groups.tail_cap * tanhf(v / p.groups.tail_cap) : v;
+      continue;
+    }
     const size_t o = (size_t)blockIdx.z * p.out_stride + (size_t)r * p.ldc + wrow;
-    if (p.epi == LG_EPI_BF16) reinterpret_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16_rn(v);
+    if (p.epi == LG_EPI_BF16 || p.epi == LG_EPI_RELU2 || p.epi == kEpiGroups) reinterpret_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16_rn(v);
     else if (p.epi == LG_EPI_RESID_F32) reinterpret_cast<float*>(p.out)[o] += v;
     else reinterpret_cast<float*>(p.out)[o] = p.p0 > 0.0f ? p.p0 * tanhf(v / p.p0) : v;
   }
@@ -163,6 +181,7 @@ struct F32Args {
   int m, n, k, lda, ldc, epi;
   int64_t a_stride, w_stride, out_stride;
   float p0, p1, p2;
+  lg_linear_groups_t groups;
 };
 
 __global__ void __launch_bounds__(256)
@@ -171,7 +190,7 @@ linear_f32_kernel(F32Args p) {
   __shared__ float as[16][68], ws[16][68];
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   const int n0 = blockIdx.x * 64, m0 = blockIdx.y * 64;
-  const float* A = p.a + (size_t)blockIdx.z * p.a_stride;
+  const float* A = p.a + (size_t)blockIdx.z * p.a_stride + (p.epi == kEpiGroups ? (size_t)group_of(p.groups, n0) * p.m * p.lda : 0);
   const __nv_bfloat16* W = p.w + (size_t)blockIdx.z * p.w_stride;
   float acc[4][4] = {};
   const int lr = tid >> 2, lk = (tid & 3) * 4;
@@ -224,6 +243,17 @@ linear_f32_kernel(F32Args p) {
     for (int j = 0; j < 4; ++j) {
       const int c = n0 + (j >> 1) * 32 + 2 * tx + (j & 1);
       if (c >= p.n) continue;
+      if (p.epi == kEpiGroups) {
+        const float v = acc[i][j];
+        if (c < p.groups.n_main) out[(size_t)r * p.ldc + c] = v;
+        else reinterpret_cast<float*>(p.groups.tail)[(size_t)r * p.groups.ld_tail + c - p.groups.n_main] = p.groups.tail_cap > 0.0f ? p.groups.tail_cap * tanhf(v / p.groups.tail_cap) : v;
+        continue;
+      }
+      if (p.epi == LG_EPI_RELU2) {
+        const float v = fmaxf(acc[i][j], 0.0f);
+        out[(size_t)r * p.ldc + c] = v * v;
+        continue;
+      }
       float* o = out + (size_t)r * p.ldc + c;
       if (p.epi == LG_EPI_RESID_F32) *o += acc[i][j];
       else *o = p.p0 > 0.0f ? p.p0 * tanhf(acc[i][j] / p.p0) : acc[i][j];
@@ -235,18 +265,16 @@ linear_f32_kernel(F32Args p) {
 
 extern "C" {
 
-uint32_t logismos_launch_linear_small_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k,
-                                           int32_t lda, int32_t ldc, int32_t batch, int64_t a_stride, int64_t w_stride,
-                                           int64_t out_stride, int32_t epilogue, float p0, float p1, float p2, void* stream) {
-  lg::LaunchScope launch_scope_;
-  epilogue &= ~LG_EPI_STATIC_W;
+static uint32_t small_any(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k, int32_t lda, int32_t ldc,
+                          int32_t batch, int64_t a_stride, int64_t w_stride, int64_t out_stride, int32_t epilogue, float p0, float p1, float p2,
+                          const lg_linear_groups_t& groups, void* stream) {
   const bool glu = epilogue == LG_EPI_SWIGLU || epilogue == LG_EPI_GLU_CLAMP;
   if (m <= 0 || n <= 0 || k <= 0 || (k % 32) || batch <= 0 || batch > 65535 || (lda % 8) || lda < k || (a_stride % 8) || (w_stride % 8) ||
-      (glu && (n % 64)) || ldc < (glu ? n / 2 : n) || (((uintptr_t)a | (uintptr_t)w) & 15) || !out || (m + 7) / 8 > 65535)
+      (glu && (n % 64)) || ldc < (glu ? n / 2 : epilogue == kEpiGroups ? groups.n_main : n) || (((uintptr_t)a | (uintptr_t)w) & 15) || !out ||
+      (m + 7) / 8 > 65535)
     return lg::kInvalidValue;
-  if (epilogue != LG_EPI_BF16 && epilogue != LG_EPI_RESID_F32 && epilogue != LG_EPI_F32 && !glu) return lg::kInvalidValue;
   const SmallArgs p{(const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (const float*)bias, out, m, n, k, lda, ldc, epilogue,
-                    a_stride, w_stride, out_stride, p0, p1, p2};
+                    a_stride, w_stride, out_stride, p0, p1, p2, groups};
   cudaStream_t s = (cudaStream_t)stream;
   // two m16 tiles per CTA once that still leaves two CTAs per SM (the activations are then read half as often)
   const int64_t ctas2 = (int64_t)((n + 31) / 32) * batch;
@@ -267,6 +295,22 @@ uint32_t logismos_launch_linear_small_bf16(const void* a, const void* w, const v
   return launch_small<1, 8>(p, batch, warps, s);
 }
 
+uint32_t logismos_launch_linear_small_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k,
+                                           int32_t lda, int32_t ldc, int32_t batch, int64_t a_stride, int64_t w_stride,
+                                           int64_t out_stride, int32_t epilogue, float p0, float p1, float p2, void* stream) {
+  lg::LaunchScope launch_scope_;
+  epilogue &= ~LG_EPI_STATIC_W;
+  if (epilogue < 0 || epilogue > LG_EPI_RELU2) return lg::kInvalidValue;
+  return small_any(a, w, bias, out, m, n, k, lda, ldc, batch, a_stride, w_stride, out_stride, epilogue, p0, p1, p2, {}, stream);
+}
+
+uint32_t logismos_launch_linear_groups_small_bf16(const void* a, const void* w, void* out, int32_t m, int32_t n, int32_t k, int32_t lda,
+                                                  int32_t ldc, const lg_linear_groups_t* groups, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!lg::groups_ok(groups, n, ldc)) return lg::kInvalidValue;
+  return small_any(a, w, nullptr, out, m, n, k, lda, ldc, 1, 0, 0, 0, kEpiGroups, 0, 0, 0, *groups, stream);
+}
+
 uint32_t logismos_launch_linear_f32(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k,
                                     int32_t lda, int32_t ldc, int32_t batch, int64_t a_stride, int64_t w_stride, int64_t out_stride,
                                     int32_t epilogue, float p0, float p1, float p2, void* stream) {
@@ -276,10 +320,21 @@ uint32_t logismos_launch_linear_f32(const void* a, const void* w, const void* bi
   if (m <= 0 || n <= 0 || k <= 0 || (k % 16) || batch <= 0 || batch > 65535 || (lda % 4) || lda < k || (a_stride % 4) || (w_stride % 4) ||
       (glu && (n % 64)) || ldc < (glu ? n / 2 : n) || ((uintptr_t)a & 15) || ((uintptr_t)w & 7) || !out || (m + 63) / 64 > 65535)
     return lg::kInvalidValue;
-  if (epilogue != LG_EPI_RESID_F32 && epilogue != LG_EPI_F32 && !glu) return lg::kInvalidValue;
+  if (epilogue != LG_EPI_RESID_F32 && epilogue != LG_EPI_F32 && epilogue != LG_EPI_RELU2 && !glu) return lg::kInvalidValue;
   const F32Args p{(const float*)a, (const __nv_bfloat16*)w, (const float*)bias, (float*)out, m, n, k, lda, ldc, epilogue,
-                  a_stride, w_stride, out_stride, p0, p1, p2};
+                  a_stride, w_stride, out_stride, p0, p1, p2, {}};
   lg::launch(linear_f32_kernel, dim3((unsigned)((n + 63) / 64), (unsigned)((m + 63) / 64), (unsigned)batch), dim3(256), 0, (cudaStream_t)stream, p);
+  return lg::launch_status();
+}
+
+uint32_t logismos_launch_linear_groups_f32(const void* a, const void* w, void* out, int32_t m, int32_t n, int32_t k, int32_t lda, int32_t ldc,
+                                           const lg_linear_groups_t* groups, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (m <= 0 || n <= 0 || k <= 0 || (k % 16) || (lda % 4) || lda < k || ((uintptr_t)a & 15) || ((uintptr_t)w & 7) || !out || (m + 63) / 64 > 65535 ||
+      !lg::groups_ok(groups, n, ldc))
+    return lg::kInvalidValue;
+  const F32Args p{(const float*)a, (const __nv_bfloat16*)w, nullptr, (float*)out, m, n, k, lda, ldc, kEpiGroups, 0, 0, 0, 0, 0, 0, *groups};
+  lg::launch(linear_f32_kernel, dim3((unsigned)((n + 63) / 64), (unsigned)((m + 63) / 64)), dim3(256), 0, (cudaStream_t)stream, p);
   return lg::launch_status();
 }
 

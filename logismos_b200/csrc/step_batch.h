@@ -174,6 +174,33 @@ struct StepBatch {
       for (int r = cu[s]; r < cu[s + 1]; ++r) rows[t++] = r;
     }
   }
+
+  // packed rows of the wanted tokens: out_rows [n_out] index the caller's tokens; NULL: the last token of every
+  // sequence. False: an index lies outside the step.
+  bool select_rows(const int32_t* out_rows, int32_t n_out, const int32_t* host_new, int32_t* rows) const {
+    std::vector<int32_t> packed_row((size_t)T);
+    caller_rows(packed_row.data());
+    int64_t off = 0;
+    for (int i = 0; i < n_out; ++i) {
+      int64_t t;
+      if (out_rows) t = out_rows[i];
+      else { off += host_new[i]; t = off - 1; }
+      if (t < 0 || t >= T) return false;
+      rows[i] = packed_row[(size_t)t];
+    }
+    return true;
+  }
+
+  // fp32 rows of the step on the device (row stride ld), in the caller's order, to host_out [T, width]
+  cudaError_t rows_to_host(const float* dev_rows, int ld, int width, float* host_out) const {
+    std::vector<float> tmp((size_t)T * ld);
+    std::vector<int32_t> packed_row((size_t)T);
+    caller_rows(packed_row.data());
+    const cudaError_t e = cudaMemcpy(tmp.data(), dev_rows, tmp.size() * 4, cudaMemcpyDeviceToHost);
+    if (e != cudaSuccess) return e;
+    for (int t = 0; t < T; ++t) std::memcpy(host_out + (size_t)t * width, tmp.data() + (size_t)packed_row[(size_t)t] * ld, (size_t)width * 4);
+    return cudaSuccess;
+  }
 };
 
 }  // namespace lgm
