@@ -735,6 +735,9 @@ typedef struct lg_time_mix {
 } lg_time_mix_t;
 /* Token by token: decode steps, fp32, any dp. */
 uint32_t logismos_launch_time_mix_step(const lg_time_mix_t* args, int32_t n_seqs, int32_t is_f32, void* stream);
+/* Prompts, 64 tokens at a time on the tensor cores: bf16 activations, dp <= 128, z given. */
+int32_t logismos_time_mix_has_chunked(int32_t dp);
+uint32_t logismos_launch_time_mix_chunked_bf16(const lg_time_mix_t* args, int32_t n_seqs, void* stream);
 
 /* State-space mixer with a scalar decay per head; np and vp are powers of two in 16 .. 256 with zero padding:
  *   x, B, C <- silu(conv);  dt <- softplus(dt + dt_bias)
@@ -760,6 +763,11 @@ typedef struct lg_ssd {
 } lg_ssd_t;
 /* Token by token, convolution included: decode steps, fp32, any size. */
 uint32_t logismos_launch_ssd_step(const lg_ssd_t* args, int32_t n_seqs, int32_t is_f32, void* stream);
+/* Prompts: convolution and silu of rows [row0, rows) into xbc (seq_ids [rows]; cu, slots, fresh and phase indexed by
+ * them), then the recurrence 64 tokens at a time on the tensor cores (np 32 .. 128, vp <= 128). */
+int32_t logismos_ssd_has_chunked(int32_t np, int32_t vp);
+uint32_t logismos_launch_ssd_conv_bf16(const lg_ssd_t* args, const void* seq_ids_i32, int32_t row0, int32_t rows, void* stream);
+uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* args, int32_t n_seqs, void* stream);
 /* out = y silu(z), divided in `parts` equal parts of the heads * v true channels by each part's root mean square,
  * times gain. Rows are laid out [heads][vp]. */
 uint32_t logismos_launch_gated_group_norm(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32,

@@ -161,6 +161,9 @@ def _declare(l, partial=False):
         "logismos_launch_split_bf16": [vp, i32, vp, i32, i32, i32, vp],
         "logismos_launch_time_mix_step": [vp, i32, i32, vp],
         "logismos_launch_ssd_step": [vp, i32, i32, vp],
+        "logismos_launch_time_mix_chunked_bf16": [vp, i32, vp],
+        "logismos_launch_ssd_conv_bf16": [vp, vp, i32, i32, vp],
+        "logismos_launch_ssd_chunked_bf16": [vp, i32, vp],
         "logismos_launch_gated_group_norm": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp],
         "logismos_launch_unit_qk_store": [vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, f32, f32, i64, i32, vp, vp],
         "logismos_launch_bias_attention_decode_bf16": [vp, i32, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
@@ -214,6 +217,8 @@ def _declare(l, partial=False):
         "lg_latent_device_status": ([vp], i32),
         "lg_latent_destroy": ([vp], None),
         "lg_latent_logits_device": ([vp], vp),
+        "logismos_time_mix_has_chunked": ([i32], i32),
+        "logismos_ssd_has_chunked": ([i32, i32], i32),
         "lg_mixer_launches_last_step": ([vp], i32),
         "lg_mixer_device_status": ([vp], i32),
         "lg_mixer_destroy": ([vp], None),

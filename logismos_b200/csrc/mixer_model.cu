@@ -153,8 +153,18 @@ uint32_t ssd_mixer(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   a.state_slots = m->dev(B.state); a.fresh = m->dev(B.fresh); a.phase = m->dev(B.phase); a.cu = m->dev(B.cu);
   a.y = m->ffb.p; a.ld_y = inner; a.heads = L.c.ssd_heads; a.groups = L.c.ssd_groups; a.np = L.Np; a.vp = L.Vp;
   a.xbc = m->xbc.p; a.ld_xbc = L.channels;
-  LG_TRY(logismos_launch_ssd_step(&a, B.n_seqs, f32, s), "state-space recurrence");
-  m->launches += 1;
+  const bool chunked = !f32 && B.n_pre > 0 && logismos_ssd_has_chunked(L.Np, L.Vp);
+  const int serial = chunked ? B.n_dec : B.n_seqs;  // sequences that go token by token
+  if (serial > 0) {
+    LG_TRY(logismos_launch_ssd_step(&a, serial, f32, s), "state-space recurrence");
+    m->launches += 1;
+  }
+  if (chunked) {
+    LG_TRY(logismos_launch_ssd_conv_bf16(&a, m->dev(B.seq_ids), B.n_dec, T, s), "state-space convolution");
+    a.state_slots = m->dev(B.state) + B.n_dec; a.fresh = m->dev(B.fresh) + B.n_dec; a.phase = m->dev(B.phase) + B.n_dec; a.cu = m->dev(B.cu) + B.n_dec;
+    LG_TRY(logismos_launch_ssd_chunked_bf16(&a, B.n_pre, s), "state-space recurrence (prompts)");
+    m->launches += 2;
+  }
   LG_TRY(logismos_launch_gated_group_norm(m->ffb.p, inner, m->proj.p, L.groups.n_main, W.gain.p, m->act.p, L.Kout, f32, T, L.c.ssd_heads, L.c.ssd_vdim, L.Vp,
                                           L.c.ssd_norm_groups, c.norm_eps, s), "gate and norm");
   m->launches += 1;
@@ -200,17 +210,30 @@ uint32_t attention(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
 
 uint32_t time_mixing(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   StepBatch& B = m->batch;
-  const int base = (2 * L.c.heads + 2 * L.c.kv_heads) * L.Dh, left = L.c.heads * L.Dh, f32 = m->cfg.is_f32;
+  const int left = L.c.heads * L.Dh, f32 = m->cfg.is_f32;
   lg_time_mix_t a{};
   a.proj = m->proj.p; a.ld = L.groups.n_main;
   a.off_r = L.groups.end[0]; a.off_k = L.groups.end[1]; a.off_v = L.groups.end[2]; a.off_g = L.groups.end[3];
-  (void)base;
   a.low = m->tail.p; a.ld_low = L.groups.ld_tail; a.w2 = W.w2.p; a.ld_w2 = 2 * L.Lr; a.rank = L.Lr; a.w0 = W.w0.p; a.u = W.u.p; a.gain = W.gain.p;
   a.state = L.state.p; a.state_slots = m->dev(B.state); a.fresh = m->dev(B.fresh); a.cu = m->dev(B.cu);
   a.out = (uint8_t*)m->act.p + (size_t)left * (f32 ? 4 : 2); a.ld_out = L.Kout; a.heads = L.c.tm_heads; a.d = L.c.tm_dim; a.dp = L.Dp;
   a.scale = L.c.right_scale; a.eps = m->cfg.norm_eps;
-  LG_TRY(logismos_launch_time_mix_step(&a, B.n_seqs, f32, s), "time mixing");
-  m->launches += 1;
+  const bool chunked = !f32 && B.n_pre > 0 && logismos_time_mix_has_chunked(L.Dp);
+  const int serial = chunked ? B.n_dec : B.n_seqs;  // sequences that go token by token
+  if (serial > 0) {
+    LG_TRY(logismos_launch_time_mix_step(&a, serial, f32, s), "time mixing");
+    m->launches += 1;
+  }
+  if (chunked) {
+    const int rows = B.T - B.n_dec, w = L.Lr;
+    LG_TRY(logismos_launch_split_bf16((const float*)m->tail.p + (size_t)B.n_dec * w, w, m->low2.p, rows, w, w, s), "decay activations");
+    LG_TRY(logismos_launch_linear_t_act_bf16(m->low2.p, W.w2.p, W.w0.p, (float*)m->z.p + (size_t)B.n_dec * L.Rw, rows, L.Rw, 2 * w, 2 * w, L.Rw,
+                                             LG_EPI_F32 | LG_EPI_STATIC_W, 0, 0, 0, m->status.p, s), "decay");
+    a.z = m->z.p; a.ld_z = L.Rw;
+    a.state_slots = m->dev(B.state) + B.n_dec; a.fresh = m->dev(B.fresh) + B.n_dec; a.cu = m->dev(B.cu) + B.n_dec;
+    LG_TRY(logismos_launch_time_mix_chunked_bf16(&a, B.n_pre, s), "time mixing (prompts)");
+    m->launches += 3;
+  }
   return 0;
 }
 

@@ -61,5 +61,62 @@ LG_DEVINL float reduce_load(int cols, const float* red, int c) {
   return s;
 }
 
+// ---- pieces of the chunk-parallel forms: 64 tokens of a sequence at a time, one head per CTA, a warp owns eight
+// value columns and its slice of the state as mma accumulators --------------------------------------------------
+
+constexpr int kChunk = 64;
+
+// transposes an 8 x 8 tile of 16-bit values held one row pair per lane
+LG_DEVINL uint32_t movmatrix_trans(uint32_t v) {
+  uint32_t r;
+  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;\n" : "=r"(r) : "r"(v));
+  return r;
+}
+// two fp32 values as bf16 plus what rounding dropped: together about 16 significant bits
+LG_DEVINL void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(a, b);
+  const float2 h = unpack_bf16x2(hi);
+  lo = pack_bf16x2(a - h.x, b - h.y);
+}
+// accumulators of a 16 (state channels) x 8 (values) tile as the B operand of a product over its channels
+LG_DEVINL void state_operand(const float (&s)[4], uint32_t (&hi)[2], uint32_t (&lo)[2]) {
+  uint32_t h0, l0, h1, l1;
+  split2(s[0], s[1], h0, l0);
+  split2(s[2], s[3], h1, l1);
+  hi[0] = movmatrix_trans(h0); hi[1] = movmatrix_trans(h1);
+  lo[0] = movmatrix_trans(l0); lo[1] = movmatrix_trans(l1);
+}
+// tiles of bf16 rows with a pitch of `pitch` bytes (row length + 16: rows start in different banks)
+// A operand: rows r0 .. r0 + 15, columns k0 .. k0 + 15
+LG_DEVINL void frag_a(uint32_t (&a)[4], uint32_t base, int pitch, int r0, int k0, int lane) {
+  ldmatrix_x4(a, base + (uint32_t)((r0 + (lane & 7) + 8 * ((lane >> 3) & 1)) * pitch + (k0 + 8 * (lane >> 4)) * 2));
+}
+// A operand, the transpose of the tile: rows = columns m0 .. m0 + 15 of it, k = its rows k0 .. k0 + 15
+LG_DEVINL void frag_at(uint32_t (&a)[4], uint32_t base, int pitch, int m0, int k0, int lane) {
+  ldmatrix_x4_trans(a, base + (uint32_t)((k0 + (lane & 7) + 8 * (lane >> 4)) * pitch + (m0 + 8 * ((lane >> 3) & 1)) * 2));
+}
+// B operands of two neighbouring n8 tiles: n = rows n0 .. n0 + 15, k = columns k0 .. k0 + 15; tile i at b[2 i]
+LG_DEVINL void frag_b(uint32_t (&b)[4], uint32_t base, int pitch, int n0, int k0, int lane) {
+  ldmatrix_x4(b, base + (uint32_t)((n0 + (lane & 7) + 8 * (lane >> 4)) * pitch + (k0 + 8 * ((lane >> 3) & 1)) * 2));
+}
+// B operands of one n8 tile for two neighbouring k16 steps: k = rows k0 .. k0 + 31, n = columns n0 .. n0 + 7; step i at b[2 i]
+LG_DEVINL void frag_bt(uint32_t (&b)[4], uint32_t base, int pitch, int k0, int n0, int lane) {
+  ldmatrix_x4_trans(b, base + (uint32_t)((k0 + lane) * pitch + n0 * 2));
+}
+LG_DEVINL void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  const uint32_t b[2] = {b0, b1};
+  mma_bf16_16816(d, a, b, d);
+}
+// rows row0 .. + 63 of a [rows][width] bf16 block at src (row stride ld elements) into a tile; rows >= n are zero
+LG_DEVINL void stage_tile(uint8_t* tile, int pitch, const __nv_bfloat16* src, int64_t ld, int n, int width) {
+  const int pieces = width >> 3;
+  for (int e = threadIdx.x; e < kChunk * pieces; e += blockDim.x) {
+    const int row = e / pieces, piece = e % pieces;
+    uint8_t* dst = tile + row * pitch + piece * 16;
+    if (row < n) cp_async16(smem_u32(dst), src + row * ld + piece * 8);
+    else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
+  }
+}
+
 }  // namespace rec
 }  // namespace lg

@@ -8,6 +8,12 @@
 // phase names and writes the other.
 //
 // ssd_step_kernel: CTA = (head, sequence), tokens one after the other, convolution included. Decode steps, fp32.
+// ssd_conv_kernel, ssd_chunk_kernel: prompts. The chunked form resolves 64 tokens together: with c_i the sum of the
+// log-decays up to token i of the chunk and S the state before it,
+//   P_ij = (C_i . B_j) exp(c_i - c_j) dt_j (j <= i);   y_i = sum_j P_ij x_j + exp(c_i) S^T C_i + D x_i
+//   S <- exp(c_last) S + sum_j B_j (dt_j exp(c_last - c_j) x_j)^T
+// The products run on mma.sync with bf16 operands: B, C and x are bf16 already; the state, P and the weighted x go
+// in as a rounded part and a remainder (two products), so that what is fp32 keeps about 16 bits; sums are fp32.
 #include "common.cuh"
 #include "logismos_kernels.h"
 #include "recurrent.cuh"
@@ -136,6 +142,244 @@ ssd_step_kernel(SsdArgs p) {
   }
 }
 
+// Convolution and silu of ragged prompt rows [row0, rows): a thread owns four channels and a run of consecutive rows.
+constexpr int kRun = 8;
+template <int TAPS>
+__global__ void __launch_bounds__(128)
+ssd_conv_kernel(SsdArgs p, const int* __restrict__ seq_ids, int row0, int rows) {
+  lg::pdl_prologue();
+  constexpr int HN = TAPS - 1;
+  const int all = p.channels(), c0 = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+  if (c0 >= all) return;
+  const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.proj) + p.heads * p.vp + c0;
+  __nv_bfloat16* dst = const_cast<__nv_bfloat16*>(reinterpret_cast<const __nv_bfloat16*>(p.xbc)) + c0;
+  float4 w[TAPS];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) w[j] = __ldg(reinterpret_cast<const float4*>(p.conv_w + (size_t)j * all + c0));
+  const float4 bias = __ldg(reinterpret_cast<const float4*>(p.conv_b + c0));
+  auto load = [&](int t) {
+    const uint2 u = *reinterpret_cast<const uint2*>(src + (size_t)t * p.ld);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+  };
+  auto fma = [](float4 a, float4 x, float4 c) { return make_float4(fmaf(a.x, x.x, c.x), fmaf(a.y, x.y, c.y), fmaf(a.z, x.z, c.z), fmaf(a.w, x.w, c.w)); };
+  auto act = [](float z) { return __fdividef(z, 1.0f + __expf(-z)); };
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  const int first = row0 + blockIdx.x * kRun, last = min(rows, first + kRun);
+  float4 in[kRun], prev[HN > 0 ? HN : 1];
+#pragma unroll
+  for (int i = 0; i < kRun; ++i) in[i] = first + i < last ? load(first + i) : zero;
+  int cur = -1, t0 = 0, len = 0;
+  float* next = nullptr;
+#pragma unroll
+  for (int i = 0; i < kRun; ++i) {
+    const int t = first + i;
+    if (t >= last) break;
+    const int s = seq_ids[t];
+    if (s != cur) {
+      cur = s;
+      t0 = p.cu[s];
+      len = p.cu[s + 1] - t0;
+      const bool fresh = p.fresh[s] != 0;
+      const int ph = p.phase[s] & 1;
+      const float* old = p.conv_state + ((size_t)p.state_slots[s] * 2 + ph) * HN * all + c0;
+      next = p.conv_state + ((size_t)p.state_slots[s] * 2 + 1 - ph) * HN * all + c0;
+#pragma unroll
+      for (int j = 0; j < HN; ++j) {
+        const int idx = t - t0 - HN + j;  // place inside the step's tokens of this sequence; negative: the state
+        if (idx >= 0) prev[j] = load(t0 + idx);
+        else prev[j] = fresh ? zero : *reinterpret_cast<const float4*>(old + (size_t)(HN + idx) * all);
+      }
+      if (t == t0) {  // rows of the old state that stay in the new one
+#pragma unroll
+        for (int j = 0; j < HN; ++j)
+          if (j + len < HN) *reinterpret_cast<float4*>(next + (size_t)j * all) = fresh ? zero : *reinterpret_cast<const float4*>(old + (size_t)(j + len) * all);
+      }
+    }
+    float4 y = fma(w[TAPS - 1], in[i], bias);
+#pragma unroll
+    for (int j = 0; j < HN; ++j) y = fma(w[j], prev[j], y);
+    *reinterpret_cast<uint2*>(dst + (size_t)t * p.ld_xbc) = make_uint2(pack_bf16x2(act(y.x), act(y.y)), pack_bf16x2(act(y.z), act(y.w)));
+    const int keep = HN - (len - (t - t0));  // row of the new state this token becomes, if any
+    if (keep >= 0) *reinterpret_cast<float4*>(next + (size_t)keep * all) = in[i];
+#pragma unroll
+    for (int j = 0; j + 1 < HN; ++j) prev[j] = prev[j + 1];
+    if (HN > 0) prev[HN > 0 ? HN - 1 : 0] = in[i];
+  }
+}
+
+// CTA = (head, sequence), VP / 8 warps; shared memory as laid out by ssd_chunk_smem
+constexpr int kPitchP = kChunk * 2 + 16;
+inline size_t ssd_chunk_smem(int np, int vp) {
+  return (size_t)kChunk * (2 * (2 * (2 * np + 16) + 2 * vp + 16) + 2 * kPitchP) + 2 * kChunk * 4;
+}
+template <int NP>
+__global__ void __launch_bounds__(512)
+ssd_chunk_kernel(SsdArgs p) {
+  lg::pdl_prologue();
+  constexpr int NT = NP / 16, kPitchN = NP * 2 + 16;
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int vp = p.vp, pitch_v = vp * 2 + 16;
+  const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
+  const int g = lane >> 2, t = lane & 3, v0 = 8 * warp;
+  const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
+  if (t1 <= t0) return;
+  const int group = head / (p.heads / p.groups), inner = p.heads * vp;
+  uint8_t *Bt = smem, *Ct = Bt + 2 * kChunk * kPitchN, *Xt = Ct + 2 * kChunk * kPitchN, *Ph = Xt + 2 * kChunk * pitch_v, *Pl = Ph + kChunk * kPitchP;
+  float *cum = reinterpret_cast<float*>(Pl + kChunk * kPitchP), *dts = cum + kChunk;
+  const __nv_bfloat16* xbc = reinterpret_cast<const __nv_bfloat16*>(p.xbc);
+  const __nv_bfloat16 *xs = xbc + head * vp, *bs = xbc + inner + group * NP, *cs = bs + p.groups * NP;
+  __nv_bfloat16* ys = reinterpret_cast<__nv_bfloat16*>(p.y) + head * vp;
+  const float bias = p.dt_bias[head], a2 = expf(p.log_a[head]) * 1.4426950408889634f, skip = p.skip[head];
+  float* st = p.state + ((size_t)p.state_slots[seq] * p.heads + head) * NP * vp;
+  float S[NT][4];   // state channels 16 m + g, + 8; values v0 + 2 t, + 1
+#pragma unroll
+  for (int m = 0; m < NT; ++m) {
+    float2 a = make_float2(0.f, 0.f), b = a;
+    if (!p.fresh[seq]) {
+      a = *reinterpret_cast<const float2*>(st + (size_t)(16 * m + g) * vp + v0 + 2 * t);
+      b = *reinterpret_cast<const float2*>(st + (size_t)(16 * m + g + 8) * vp + v0 + 2 * t);
+    }
+    S[m][0] = a.x; S[m][1] = a.y; S[m][2] = b.x; S[m][3] = b.y;
+  }
+  auto stage = [&](int tb, int buf) {
+    const int n = min(kChunk, t1 - tb);
+    stage_tile(Bt + buf * kChunk * kPitchN, kPitchN, bs + (int64_t)tb * p.ld_xbc, p.ld_xbc, n, NP);
+    stage_tile(Ct + buf * kChunk * kPitchN, kPitchN, cs + (int64_t)tb * p.ld_xbc, p.ld_xbc, n, NP);
+    stage_tile(Xt + buf * kChunk * pitch_v, pitch_v, xs + (int64_t)tb * p.ld_xbc, p.ld_xbc, n, vp);
+    cp_async_commit();
+  };
+  float dt_raw[2] = {0.f, 0.f};
+  auto fetch_dt = [&](int tb) {
+    if (warp != 0) return;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) dt_raw[i] = tb + lane + 32 * i < t1 ? p.dt[(size_t)(tb + lane + 32 * i) * p.ld_dt + head] : 0.0f;
+  };
+  stage(t0, 0);
+  fetch_dt(t0);
+  int buf = 0;
+  for (int tb = t0; tb < t1; tb += kChunk, buf ^= 1) {
+    const int n = min(kChunk, t1 - tb);
+    if (warp == 0) {  // step sizes and log2-decays summed up; tokens past the end take no step
+      const float d0 = lane < n ? softplus_f(dt_raw[0] + bias) : 0.0f, d1 = lane + 32 < n ? softplus_f(dt_raw[1] + bias) : 0.0f;
+      float c0 = -a2 * d0, c1 = -a2 * d1;
+#pragma unroll
+      for (int d = 1; d < 32; d <<= 1) {
+        const float u0 = __shfl_up_sync(0xffffffffu, c0, d), u1 = __shfl_up_sync(0xffffffffu, c1, d);
+        if (lane >= d) { c0 += u0; c1 += u1; }
+      }
+      c1 += __shfl_sync(0xffffffffu, c0, 31);
+      cum[lane] = c0; cum[lane + 32] = c1;
+      dts[lane] = d0; dts[lane + 32] = d1;
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    if (tb + kChunk < t1) {
+      stage(tb + kChunk, buf ^ 1);
+      fetch_dt(tb + kChunk);
+    }
+    const uint32_t B_a = smem_u32(Bt + buf * kChunk * kPitchN), C_a = smem_u32(Ct + buf * kChunk * kPitchN), X_a = smem_u32(Xt + buf * kChunk * pitch_v);
+    // ---- P: sixteen by sixteen blocks on and below the diagonal, dealt to the warps
+    for (int b = warp; b < 10; b += n_warps) {
+      const int I = b < 4 ? 3 : b < 7 ? 2 : b < 9 ? 1 : 0, J = b - (b < 4 ? 0 : b < 7 ? 4 : b < 9 ? 7 : 9);
+      float acc[2][4] = {};
+#pragma unroll
+      for (int ks = 0; ks < NT; ++ks) {
+        uint32_t a[4], bb[4];
+        frag_a(a, C_a, kPitchN, 16 * I, 16 * ks, lane);
+        frag_b(bb, B_a, kPitchN, 16 * J, 16 * ks, lane);
+        mma(acc[0], a, bb[0], bb[1]);
+        mma(acc[1], a, bb[2], bb[3]);
+      }
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int i = 16 * I + g + 8 * h, j = 16 * J + 8 * nt + 2 * t;
+          const float w0 = j <= i ? acc[nt][2 * h] * fast_exp2(cum[i] - cum[j]) * dts[j] : 0.0f;
+          const float w1 = j + 1 <= i ? acc[nt][2 * h + 1] * fast_exp2(cum[i] - cum[j + 1]) * dts[j + 1] : 0.0f;
+          uint32_t hi, lo;
+          split2(w0, w1, hi, lo);
+          *reinterpret_cast<uint32_t*>(Ph + i * kPitchP + j * 2) = hi;
+          *reinterpret_cast<uint32_t*>(Pl + i * kPitchP + j * 2) = lo;
+        }
+    }
+    __syncthreads();
+    // ---- outputs of this warp's eight values
+    float acc[4][4] = {};
+#pragma unroll
+    for (int ks = 0; ks < NT; ++ks) {
+      uint32_t hi[2], lo[2];
+      state_operand(S[ks], hi, lo);
+#pragma unroll
+      for (int mt = 0; mt < 4; ++mt) {
+        uint32_t a[4];
+        frag_a(a, C_a, kPitchN, 16 * mt, 16 * ks, lane);
+        mma(acc[mt], a, hi[0], hi[1]);
+        mma(acc[mt], a, lo[0], lo[1]);
+      }
+    }
+    uint32_t xb[2][4];
+    frag_bt(xb[0], X_a, pitch_v, 0, v0, lane);
+    frag_bt(xb[1], X_a, pitch_v, 32, v0, lane);
+    const uint32_t Ph_a = smem_u32(Ph), Pl_a = smem_u32(Pl);
+#pragma unroll
+    for (int mt = 0; mt < 4; ++mt) {
+      const float e0 = fast_exp2(cum[16 * mt + g]), e1 = fast_exp2(cum[16 * mt + g + 8]);
+      acc[mt][0] *= e0; acc[mt][1] *= e0; acc[mt][2] *= e1; acc[mt][3] *= e1;
+#pragma unroll
+      for (int kt = 0; kt <= mt; ++kt) {
+        uint32_t a[4];
+        frag_a(a, Ph_a, kPitchP, 16 * mt, 16 * kt, lane);
+        mma(acc[mt], a, xb[kt >> 1][2 * (kt & 1)], xb[kt >> 1][2 * (kt & 1) + 1]);
+        frag_a(a, Pl_a, kPitchP, 16 * mt, 16 * kt, lane);
+        mma(acc[mt], a, xb[kt >> 1][2 * (kt & 1)], xb[kt >> 1][2 * (kt & 1) + 1]);
+      }
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {  // D x; the result takes the place of x (columns that only this warp reads)
+        uint32_t* at = reinterpret_cast<uint32_t*>(Xt + buf * kChunk * pitch_v + (16 * mt + g + 8 * h) * pitch_v + (v0 + 2 * t) * 2);
+        const float2 x = unpack_bf16x2(*at);
+        *at = pack_bf16x2(fmaf(skip, x.x, acc[mt][2 * h]), fmaf(skip, x.y, acc[mt][2 * h + 1]));
+      }
+    }
+    // ---- state
+    const float c_last = cum[kChunk - 1], e_last = fast_exp2(c_last);
+#pragma unroll
+    for (int m = 0; m < NT; ++m)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[m][e] *= e_last;
+#pragma unroll
+    for (int kt = 0; kt < 4; ++kt) {
+      uint32_t hi[2], lo[2];
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int j = 16 * kt + 8 * h + 2 * t;
+        const float2 x = unpack_bf16x2(xb[kt >> 1][2 * (kt & 1) + h]);
+        split2(x.x * dts[j] * fast_exp2(c_last - cum[j]), x.y * dts[j + 1] * fast_exp2(c_last - cum[j + 1]), hi[h], lo[h]);
+      }
+#pragma unroll
+      for (int m = 0; m < NT; ++m) {
+        uint32_t a[4];
+        frag_at(a, B_a, kPitchN, 16 * m, 16 * kt, lane);
+        mma(S[m], a, hi[0], hi[1]);
+        mma(S[m], a, lo[0], lo[1]);
+      }
+    }
+    __syncthreads();
+    const int pieces_v = vp >> 3;
+    for (int e = tid; e < n * pieces_v; e += blockDim.x) {
+      const int row = e / pieces_v, piece = e % pieces_v;
+      *reinterpret_cast<uint4*>(ys + (int64_t)(tb + row) * p.ld_y + piece * 8) =
+          *reinterpret_cast<const uint4*>(Xt + buf * kChunk * pitch_v + row * pitch_v + piece * 16);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < NT; ++m) {
+    *reinterpret_cast<float2*>(st + (size_t)(16 * m + g) * vp + v0 + 2 * t) = make_float2(S[m][0], S[m][1]);
+    *reinterpret_cast<float2*>(st + (size_t)(16 * m + g + 8) * vp + v0 + 2 * t) = make_float2(S[m][2], S[m][3]);
+  }
+}
+
 // y silu(z), normalised in equal parts of `width` channels. CTA = (row, part). VEC: channels are contiguous (no
 // padding between heads) and eight of them are moved at once.
 template <typename T, bool VEC>
@@ -236,6 +480,45 @@ uint32_t logismos_launch_ssd_step(const lg_ssd_t* a, int32_t n_seqs, int32_t is_
                    : pt == 16 ? go(ssd_step_kernel<T, 16>) : go(ssd_step_kernel<T, 0>)
   return is_f32 ? (LG_STEP(float)) : (LG_STEP(__nv_bfloat16));
 #undef LG_STEP
+}
+
+int32_t logismos_ssd_has_chunked(int32_t np, int32_t vp) { return pow2(np, 32, 128) && pow2(vp, 16, 128) ? 1 : 0; }
+
+uint32_t logismos_launch_ssd_conv_bf16(const lg_ssd_t* a, const void* seq_ids_i32, int32_t row0, int32_t rows, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!args_ok(a, 1) || !seq_ids_i32 || row0 < 0 || rows <= row0 || !a->xbc || a->ld % 4 || a->ld_xbc % 4 || a->ld_xbc < a->heads * a->vp + 2 * a->groups * a->np)
+    return lg::kInvalidValue;
+  const SsdArgs p = make_args(a);
+  const dim3 grid((unsigned)((rows - row0 + kRun - 1) / kRun), (unsigned)(((a->heads * a->vp + 2 * a->groups * a->np) / 4 + 127) / 128));
+  auto go = [&](auto kern) {
+    lg::launch(kern, grid, dim3(128), 0, (cudaStream_t)stream, p, (const int*)seq_ids_i32, row0, rows);
+    return lg::launch_status();
+  };
+  switch (a->taps) {
+    case 1: return go(ssd_conv_kernel<1>);
+    case 2: return go(ssd_conv_kernel<2>);
+    case 3: return go(ssd_conv_kernel<3>);
+    case 4: return go(ssd_conv_kernel<4>);
+    case 5: return go(ssd_conv_kernel<5>);
+    case 6: return go(ssd_conv_kernel<6>);
+    case 7: return go(ssd_conv_kernel<7>);
+    default: return go(ssd_conv_kernel<8>);
+  }
+}
+
+uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* a, int32_t n_seqs, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!args_ok(a, n_seqs) || !logismos_ssd_has_chunked(a->np, a->vp) || !a->xbc || a->ld_xbc % 8 || a->ld_y % 8 || (((uintptr_t)a->xbc | (uintptr_t)a->y) & 15))
+    return lg::kInvalidValue;
+  const SsdArgs p = make_args(a);
+  const size_t smem = ssd_chunk_smem(a->np, a->vp);
+  auto go = [&](auto kern) -> uint32_t {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3((unsigned)(4 * p.vp)), smem, (cudaStream_t)stream, p);
+    return lg::launch_status();
+  };
+  return a->np == 32 ? go(ssd_chunk_kernel<32>) : a->np == 64 ? go(ssd_chunk_kernel<64>) : go(ssd_chunk_kernel<128>);
 }
 
 uint32_t logismos_launch_gated_group_norm(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32, void* out, int32_t ld_out,

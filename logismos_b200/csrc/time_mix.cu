@@ -6,6 +6,14 @@
 //
 // time_mix_step_kernel: CTA = (head, sequence), tokens one after the other. Decode steps, fp32, head sizes
 // above 128. z comes from a buffer, or is computed from the low-rank activations: z = W2 low + w0.
+//
+// time_mix_chunk_kernel: prompts, CTA = (head, sequence), 64 tokens at a time in four blocks of 16. With c_i the sum
+// of log w inside a block up to its token i, T the block's total and S the state before the block,
+//   R_i = r_i exp(c_(i-1));  K_j = k_j exp(T - c_j)
+//   o_i = S^T R_i + sum_(j < i) (R_i exp(-T) . K_j) v_j + (r_i . u k_i) v_i;   S <- diag(exp(T)) S + sum_j K_j v_j^T
+// R and K need one exponential per element and stay below r and k in size; the product with exp(-T) is taken where
+// exp(T) does not underflow, else the block's coefficients are summed directly. The products run on mma.sync; what
+// is fp32 (R, K, the state, the coefficients) goes in as a rounded bf16 part and a remainder.
 #include "common.cuh"
 #include "logismos_kernels.h"
 #include "recurrent.cuh"
@@ -146,6 +154,225 @@ time_mix_step_kernel(MixArgs p) {
   }
 }
 
+template <int DP> struct ChunkCfg {
+  static constexpr int kThreadsC = 4 * DP, kPitch = DP * 2 + 16, kTile = kChunk * kPitch, kPitchC = DP + 8, kPitchA = 16 * 2 + 16;
+  // r, k, v twice; remainders of R and K; block sums (later the outputs) fp32; coefficients, two parts; totals, bonus
+  static constexpr size_t kSmem = 8 * (size_t)kTile + kChunk * kPitchC * 4 + 2 * kChunk * kPitchA + 4 * DP * 4 + kChunk * 4;
+};
+constexpr float kMaxSpan = 100.0f;  // log2 of the decay over a block up to which exp(-T) is taken
+
+template <int DP>
+__global__ void __launch_bounds__(4 * DP)
+time_mix_chunk_kernel(MixArgs p) {
+  lg::pdl_prologue();
+  using C = ChunkCfg<DP>;
+  constexpr int NT = DP / 16, kOct = DP / 8, kPitch = C::kPitch, kPitchC = C::kPitchC, kPitchA = C::kPitchA;
+  extern __shared__ __align__(16) uint8_t smem[];
+  uint8_t *Rt = smem, *Kt = Rt + 2 * C::kTile, *Vt = Kt + 2 * C::kTile, *Rl = Vt + 2 * C::kTile, *Kl = Rl + C::kTile;
+  float* cs = reinterpret_cast<float*>(Kl + C::kTile);
+  uint8_t *Ah = reinterpret_cast<uint8_t*>(cs + kChunk * kPitchC), *Al = Ah + kChunk * kPitchA;
+  float *tot = reinterpret_cast<float*>(Al + kChunk * kPitchA), *bonus = tot + 4 * DP;
+  const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int g = lane >> 2, t = lane & 3, v0 = 8 * warp, h0 = head * DP;
+  const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
+  if (t1 <= t0) return;
+  const __nv_bfloat16* proj = reinterpret_cast<const __nv_bfloat16*>(p.proj) + h0;
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + h0;
+  float* st = p.state + ((size_t)p.state_slots[seq] * p.heads + head) * DP * DP;
+  float S[NT][4];   // key channels 16 m + g, + 8; values v0 + 2 t, + 1
+#pragma unroll
+  for (int m = 0; m < NT; ++m) {
+    float2 a = make_float2(0.f, 0.f), b = a;
+    if (!p.fresh[seq]) {
+      a = *reinterpret_cast<const float2*>(st + (size_t)(16 * m + g) * DP + v0 + 2 * t);
+      b = *reinterpret_cast<const float2*>(st + (size_t)(16 * m + g + 8) * DP + v0 + 2 * t);
+    }
+    S[m][0] = a.x; S[m][1] = a.y; S[m][2] = b.x; S[m][3] = b.y;
+  }
+  auto stage = [&](int tb, int buf) {
+    const int n = min(kChunk, t1 - tb);
+    const __nv_bfloat16* row = proj + (int64_t)tb * p.ld;
+    stage_tile(Rt + buf * C::kTile, kPitch, row + p.off_r, p.ld, n, DP);
+    stage_tile(Kt + buf * C::kTile, kPitch, row + p.off_k, p.ld, n, DP);
+    stage_tile(Vt + buf * C::kTile, kPitch, row + p.off_v, p.ld, n, DP);
+    cp_async_commit();
+  };
+  const int zc = tid % DP, zb = tid / DP;  // channel and block of 16 tokens whose log-decays this thread sums
+  float z[16];
+  auto fetch_z = [&](int tb) {
+#pragma unroll
+    for (int i = 0; i < 16; ++i) z[i] = tb + 16 * zb + i < t1 ? p.z[(size_t)(tb + 16 * zb + i) * p.ld_z + h0 + zc] : -INFINITY;
+  };
+  stage(t0, 0);
+  fetch_z(t0);
+  int buf = 0;
+  for (int tb = t0; tb < t1; tb += kChunk, buf ^= 1) {
+    const int n = min(kChunk, t1 - tb);
+    {
+      float c = 0.0f;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {  // past the end: no decay
+        c -= expf(z[i]) * 1.4426950408889634f;
+        cs[(16 * zb + i) * kPitchC + zc] = c;
+      }
+      tot[zb * DP + zc] = c;
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    if (tb + kChunk < t1) {
+      stage(tb + kChunk, buf ^ 1);
+      fetch_z(tb + kChunk);
+    }
+    uint8_t *R = Rt + buf * C::kTile, *K = Kt + buf * C::kTile;
+    // ---- R and K in two parts (the rounded ones in place), and r . u k
+    for (int e = tid; e < kChunk * kOct; e += C::kThreadsC) {
+      const int row = e / kOct, d0 = 8 * (e % kOct);
+      const uint4 ru = *reinterpret_cast<const uint4*>(R + row * kPitch + d0 * 2), ku = *reinterpret_cast<const uint4*>(K + row * kPitch + d0 * 2);
+      const uint32_t rw[4] = {ru.x, ru.y, ru.z, ru.w}, kw[4] = {ku.x, ku.y, ku.z, ku.w};
+      uint32_t rh[4], rl[4], kh[4], kl[4];
+      float dot = 0.0f;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const int d = d0 + 2 * q;
+        const float2 r = unpack_bf16x2(rw[q]), k = unpack_bf16x2(kw[q]);
+        const float2 c = *reinterpret_cast<const float2*>(cs + row * kPitchC + d), tt = *reinterpret_cast<const float2*>(tot + (row >> 4) * DP + d);
+        const float2 cp = (row & 15) ? *reinterpret_cast<const float2*>(cs + (row - 1) * kPitchC + d) : make_float2(0.f, 0.f);
+        const float2 u = __ldg(reinterpret_cast<const float2*>(p.u + h0 + d));
+        dot = fmaf(r.x * u.x, k.x, fmaf(r.y * u.y, k.y, dot));
+        split2(r.x * fast_exp2(cp.x), r.y * fast_exp2(cp.y), rh[q], rl[q]);
+        split2(k.x * fast_exp2(tt.x - c.x), k.y * fast_exp2(tt.y - c.y), kh[q], kl[q]);
+      }
+#pragma unroll
+      for (int o = 1; o < kOct; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+      if (d0 == 0) bonus[row] = dot;
+      *reinterpret_cast<uint4*>(R + row * kPitch + d0 * 2) = make_uint4(rh[0], rh[1], rh[2], rh[3]);
+      *reinterpret_cast<uint4*>(Rl + row * kPitch + d0 * 2) = make_uint4(rl[0], rl[1], rl[2], rl[3]);
+      *reinterpret_cast<uint4*>(K + row * kPitch + d0 * 2) = make_uint4(kh[0], kh[1], kh[2], kh[3]);
+      *reinterpret_cast<uint4*>(Kl + row * kPitch + d0 * 2) = make_uint4(kl[0], kl[1], kl[2], kl[3]);
+    }
+    __syncthreads();
+    const uint32_t R_a = smem_u32(R), K_a = smem_u32(K), V_a = smem_u32(Vt + buf * C::kTile), Rl_a = smem_u32(Rl), Kl_a = smem_u32(Kl);
+    // ---- coefficients inside the blocks
+    for (int I = warp; I < 4; I += C::kThreadsC / 32) {
+      float worst = 0.0f;
+      for (int d = lane; d < DP; d += 32) worst = fmaxf(worst, -tot[I * DP + d]);
+      float acc[2][4] = {};
+      if (__all_sync(0xffffffffu, worst <= kMaxSpan)) {
+#pragma unroll
+        for (int ks = 0; ks < NT; ++ks) {
+          uint32_t ah[4], al[4], bh[4], bl[4];
+          frag_a(ah, R_a, kPitch, 16 * I, 16 * ks, lane);
+          frag_a(al, Rl_a, kPitch, 16 * I, 16 * ks, lane);
+          frag_b(bh, K_a, kPitch, 16 * I, 16 * ks, lane);
+          frag_b(bl, Kl_a, kPitch, 16 * I, 16 * ks, lane);
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {  // columns 2 t (+ 8 for q >= 2)
+            const float2 f = *reinterpret_cast<const float2*>(tot + I * DP + 16 * ks + 8 * (q >> 1) + 2 * t);
+            const float2 x = unpack_bf16x2(ah[q]), y = unpack_bf16x2(al[q]);
+            split2((x.x + y.x) * fast_exp2(-f.x), (x.y + y.y) * fast_exp2(-f.y), ah[q], al[q]);
+          }
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) {
+            mma(acc[nt], ah, bh[2 * nt], bh[2 * nt + 1]);
+            mma(acc[nt], al, bh[2 * nt], bh[2 * nt + 1]);
+            mma(acc[nt], ah, bl[2 * nt], bl[2 * nt + 1]);
+          }
+        }
+      } else {  // some channel decays too far: term by term, with exponents c_(i-1) - c_j <= 0
+        const __nv_bfloat16 *rs = proj + p.off_r, *ks_ = proj + p.off_k;
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int i = 16 * I + g + 8 * (e >> 1), j = 16 * I + 8 * nt + 2 * t + (e & 1);
+            if (j >= i || i >= n) continue;
+            float s = 0.0f;
+            for (int d = 0; d < DP; ++d)
+              s = fmaf(__bfloat162float(rs[(int64_t)(tb + i) * p.ld + d]) * __bfloat162float(ks_[(int64_t)(tb + j) * p.ld + d]),
+                       fast_exp2(cs[(i - 1) * kPitchC + d] - cs[j * kPitchC + d]), s);
+            acc[nt][e] = s;
+          }
+      }
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int i = g + 8 * h, j = 8 * nt + 2 * t;
+          const float b = bonus[16 * I + i];
+          uint32_t hi, lo;
+          split2(j < i ? acc[nt][2 * h] : j == i ? b : 0.0f, j + 1 < i ? acc[nt][2 * h + 1] : j + 1 == i ? b : 0.0f, hi, lo);
+          *reinterpret_cast<uint32_t*>(Ah + (16 * I + i) * kPitchA + j * 2) = hi;
+          *reinterpret_cast<uint32_t*>(Al + (16 * I + i) * kPitchA + j * 2) = lo;
+        }
+    }
+    __syncthreads();
+    // ---- outputs of this warp's eight values and the state, block by block
+    uint32_t vb[2][4];
+    frag_bt(vb[0], V_a, kPitch, 0, v0, lane);
+    frag_bt(vb[1], V_a, kPitch, 32, v0, lane);
+    const uint32_t Ah_a = smem_u32(Ah), Al_a = smem_u32(Al);
+#pragma unroll
+    for (int I = 0; I < 4; ++I) {
+      const uint32_t b0 = vb[I >> 1][2 * (I & 1)], b1 = vb[I >> 1][2 * (I & 1) + 1];
+      float acc[4] = {};
+#pragma unroll
+      for (int ks = 0; ks < NT; ++ks) {
+        uint32_t hi[2], lo[2], a[4];
+        state_operand(S[ks], hi, lo);
+        frag_a(a, R_a, kPitch, 16 * I, 16 * ks, lane);
+        mma(acc, a, hi[0], hi[1]);
+        mma(acc, a, lo[0], lo[1]);
+        frag_a(a, Rl_a, kPitch, 16 * I, 16 * ks, lane);
+        mma(acc, a, hi[0], hi[1]);
+      }
+      uint32_t a[4];
+      frag_a(a, Ah_a, kPitchA, 16 * I, 0, lane);
+      mma(acc, a, b0, b1);
+      frag_a(a, Al_a, kPitchA, 16 * I, 0, lane);
+      mma(acc, a, b0, b1);
+      *reinterpret_cast<float2*>(cs + (16 * I + g) * kPitchC + v0 + 2 * t) = make_float2(acc[0], acc[1]);  // the block sums are no longer needed
+      *reinterpret_cast<float2*>(cs + (16 * I + g + 8) * kPitchC + v0 + 2 * t) = make_float2(acc[2], acc[3]);
+#pragma unroll
+      for (int m = 0; m < NT; ++m) {
+        const float e0 = fast_exp2(tot[I * DP + 16 * m + g]), e1 = fast_exp2(tot[I * DP + 16 * m + g + 8]);
+        S[m][0] *= e0; S[m][1] *= e0; S[m][2] *= e1; S[m][3] *= e1;
+        frag_at(a, K_a, kPitch, 16 * m, 16 * I, lane);
+        mma(S[m], a, b0, b1);
+        frag_at(a, Kl_a, kPitch, 16 * m, 16 * I, lane);
+        mma(S[m], a, b0, b1);
+      }
+    }
+    __syncthreads();
+    // ---- norm over the head, gain, gate
+    for (int e = tid; e < kChunk * kOct; e += C::kThreadsC) {
+      const int row = e / kOct, d0 = 8 * (e % kOct);
+      const float4 a = *reinterpret_cast<const float4*>(cs + row * kPitchC + d0), b = *reinterpret_cast<const float4*>(cs + row * kPitchC + d0 + 4);
+      float o[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w}, ss = 0.0f;
+#pragma unroll
+      for (int q = 0; q < 8; ++q) ss = fmaf(o[q], o[q], ss);
+#pragma unroll
+      for (int s = 1; s < kOct; s <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+      if (row >= n) continue;
+      const float inv = p.scale / sqrtf(ss / (float)p.d + p.eps);
+      const uint4 gu = *reinterpret_cast<const uint4*>(proj + (int64_t)(tb + row) * p.ld + p.off_g + d0);
+      const uint32_t gw[4] = {gu.x, gu.y, gu.z, gu.w};
+      uint32_t w[4];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float2 gg = unpack_bf16x2(gw[q]), gn = __ldg(reinterpret_cast<const float2*>(p.gain + h0 + d0 + 2 * q));
+        w[q] = pack_bf16x2(o[2 * q] * inv * gn.x * __fdividef(gg.x, 1.0f + __expf(-gg.x)), o[2 * q + 1] * inv * gn.y * __fdividef(gg.y, 1.0f + __expf(-gg.y)));
+      }
+      *reinterpret_cast<uint4*>(out + (int64_t)(tb + row) * p.ld_out + d0) = make_uint4(w[0], w[1], w[2], w[3]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int m = 0; m < NT; ++m) {
+    *reinterpret_cast<float2*>(st + (size_t)(16 * m + g) * DP + v0 + 2 * t) = make_float2(S[m][0], S[m][1]);
+    *reinterpret_cast<float2*>(st + (size_t)(16 * m + g + 8) * DP + v0 + 2 * t) = make_float2(S[m][2], S[m][3]);
+  }
+}
+
 bool args_ok(const lg_time_mix_t* a, int n_seqs) {
   return a && n_seqs > 0 && n_seqs <= 65535 && a->proj && a->state && a->state_slots && a->fresh && a->cu && a->out && a->u && a->gain && a->heads > 0 &&
          (a->dp == 32 || a->dp == 64 || a->dp == 128 || a->dp == 256) && a->d > 0 && a->d <= a->dp && a->ld_out >= a->heads * a->dp &&
@@ -174,6 +401,24 @@ uint32_t logismos_launch_time_mix_step(const lg_time_mix_t* a, int32_t n_seqs, i
 #define LG_STEP(T) p.dp == 32 ? go(time_mix_step_kernel<T, 1>) : p.dp == 64 ? go(time_mix_step_kernel<T, 4>) : p.dp == 128 ? go(time_mix_step_kernel<T, 16>) : go(time_mix_step_kernel<T, 0>)
   return is_f32 ? (LG_STEP(float)) : (LG_STEP(__nv_bfloat16));
 #undef LG_STEP
+}
+
+int32_t logismos_time_mix_has_chunked(int32_t dp) { return dp == 32 || dp == 64 || dp == 128 ? 1 : 0; }
+
+uint32_t logismos_launch_time_mix_chunked_bf16(const lg_time_mix_t* a, int32_t n_seqs, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!args_ok(a, n_seqs) || !a->z || !logismos_time_mix_has_chunked(a->dp) || ((a->ld | a->ld_out | a->off_r | a->off_k | a->off_v | a->off_g) % 8) ||
+      (((uintptr_t)a->proj | (uintptr_t)a->out) & 15))
+    return lg::kInvalidValue;
+  const MixArgs p = make_args(a);
+  auto go = [&](auto kern, size_t smem) -> uint32_t {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3((unsigned)(4 * p.dp)), smem, (cudaStream_t)stream, p);
+    return lg::launch_status();
+  };
+  return a->dp == 32 ? go(time_mix_chunk_kernel<32>, ChunkCfg<32>::kSmem) : a->dp == 64 ? go(time_mix_chunk_kernel<64>, ChunkCfg<64>::kSmem)
+                                                                              : go(time_mix_chunk_kernel<128>, ChunkCfg<128>::kSmem);
 }
 
 }  // extern "C"
