@@ -10,6 +10,7 @@ every rank holds a full replica and its own batch (request sharding, no collecti
 
   python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference] [--layers L]
   python bench.py --workload ragged_step                    (continuous-batching step of the int4 decoder)
+  python bench.py --workload latent | mixer [--sizes A,B --kernels]   (bf16 decoders beside an int4 one of equal size)
   python bench.py --workload serving_sweep [--requests R --max-seqs S --arrival-rate L --tp T]
                                                             (hybrid decoder under the host scheduler)
 
@@ -632,9 +633,9 @@ def main():
     ap.add_argument("--no-cpu", action="store_true")
     ap.add_argument("--no-extra", action="store_true", help="skip the decode workloads of the default line")
     ap.add_argument("--ref-budget", type=float, default=150.0, help="--impl reference: seconds of timed CPU work (each step is a full batch)")
-    ap.add_argument("--workload", default="stella", choices=["stella", "ragged_step", "serving_sweep", "latent"])
-    ap.add_argument("--sizes", default="", help="latent: comma-separated sizes of bench_latent.SIZES (default all)")
-    ap.add_argument("--kernels", action="store_true", help="latent: also every kernel against its roofline, per size")
+    ap.add_argument("--workload", default="stella", choices=["stella", "ragged_step", "serving_sweep", "latent", "mixer"])
+    ap.add_argument("--sizes", default="", help="latent, mixer: comma-separated sizes of bench_latent.SIZES or bench_mixer.SIZES (default all)")
+    ap.add_argument("--kernels", action="store_true", help="latent, mixer: also every kernel against its roofline, per size")
     ap.add_argument("--requests", type=int, default=96, help="serving_sweep: requests per GPU")
     ap.add_argument("--extra-requests", type=int, default=64, help="requests per GPU of the serving sample inside the default line")
     ap.add_argument("--max-seqs", type=int, default=256, help="serving_sweep: concurrent sequences per GPU")
@@ -684,6 +685,22 @@ def main():
                 "clocks": clocks, "sizes": rows}
         if args.kernels:
             line["kernels"] = {n: bench_latent.kernel_table(bench_latent.SIZES[n], peaks) for n in sizes}
+        print(json.dumps(line))
+    elif args.workload == "mixer":
+        import bench_mixer
+        if world > 1:
+            raise SystemExit("--workload mixer runs on one GPU")
+        peaks, sizes = measured_peaks(), [n for n in args.sizes.split(",") if n] or list(bench_mixer.SIZES)
+        sampler = ClockSampler(local)
+        sampler.start()
+        rows = bench_mixer.measure(sizes, args.steps, peaks)
+        clocks = sampler.stop()
+        line = {"metric": "mixer_decoder_tokens_per_s", "value": rows[0]["mixer"]["prefill"]["tokens_per_s"], "unit": "tokens/s (prefill of the first size)", "n_gpus": 1,
+                "steps": args.steps, "warmup": 3, "higher_is_better": True, "vs_baseline": None, "dtype": "bf16 weights and activations (beside: int4-g32 weights)",
+                "data": "synthetic", "config": {"workload": "state-space / parallel decoder beside the hybrid decoder at equal width, depth, heads and feed-forward", "sizes": sizes},
+                "clocks": clocks, "sizes": rows}
+        if args.kernels:
+            line["kernels"] = {n: bench_mixer.kernel_table(bench_mixer.SIZES[n], peaks) for n in sizes}
         print(json.dumps(line))
     elif args.workload == "ragged_step":
         line = ragged_step_measure(R, steps=args.steps, warmup=args.warmup, layers=args.layers)

@@ -133,7 +133,9 @@ uint32_t logismos_launch_linear_small_bf16(const void* a_bf16, const void* w_bf1
 /* Several projections of the same rows in one launch, each block of columns with its own input: columns
  * [end[g - 1], end[g]) of the output are rows of W applied to activation copy g, copy g standing at a + g * m *
  * lda. Columns below n_main go to out (bf16 [m, n_main], row stride ldc), the others to tail (fp32, row stride
- * ld_tail), with a soft cap tail_cap tanh(. / tail_cap) when tail_cap > 0. The ends and n_main are multiples of
+ * ld_tail), with a soft cap tail_cap tanh(. / tail_cap) when tail_cap > 0, and (bf16 routes) when tail_parts is given
+ * also there as bf16 [m, 2 (n - n_main)]: the rounded values, then what rounding dropped, so that a GEMM over [W | W]
+ * sees them to about 16 bits. The ends and n_main are multiples of
  * 128 (the last end is n), n a multiple of 16. The three launchers take the routes of the three above: tcgen05
  * tiles, weights streamed once for few rows, and fp32 (out and tail fp32). */
 #define LG_MAX_LINEAR_GROUPS 8
@@ -144,6 +146,7 @@ typedef struct lg_linear_groups {
   void* tail;
   int32_t ld_tail;
   float tail_cap;
+  void* tail_parts;
 } lg_linear_groups_t;
 uint32_t logismos_launch_linear_groups_tc_bf16(const void* a_bf16, const void* w_bf16, void* out, int32_t m, int32_t n,
                                                int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
@@ -706,10 +709,6 @@ uint32_t logismos_launch_token_shift(const void* x_f32, void* h, int32_t out_f32
                                      void* state_f32, const void* state_slots_i32, const void* fresh_u8,
                                      const void* phase_u8, const void* seq_ids_i32, const void* cu_seqlens_i32,
                                      int32_t rows, int32_t ld, void* stream);
-/* fp32 [rows, n] (row stride ld) -> bf16 [rows, 2 width]: rounded values, then what rounding dropped: a GEMM over
- * [W | W] then sees the input to about 16 bits. */
-uint32_t logismos_launch_split_bf16(const void* in_f32, int32_t ld, void* out_bf16, int32_t rows, int32_t n,
-                                    int32_t width, void* stream);
 
 /* Time mixing with a data-dependent decay per key channel, heads padded to dp = 32, 64, 128 or 256 with zeros:
  *   o_t = (S + diag(u) k_t v_t^T)^T r_t;  S <- diag(exp(-exp(z_t))) S + k_t v_t^T
@@ -758,15 +757,17 @@ typedef struct lg_ssd {
   const void *state_slots, *fresh, *phase, *cu;
   void* y;
   int32_t ld_y, heads, groups, np, vp;
-  void* xbc;                    /* chunked form: bf16 [rows, ld_xbc], the convolved channels */
+  void* xbc;                    /* activation format [rows, ld_xbc]: the convolved channels x | B | C */
   int32_t ld_xbc;
 } lg_ssd_t;
-/* Token by token, convolution included: decode steps, fp32, any size. */
+/* Convolution and silu of rows [row0, rows) from proj into xbc (seq_ids [rows]; cu, slots, fresh and phase indexed by
+ * them). single: rows are one token per sequence. */
+uint32_t logismos_launch_ssd_conv(const lg_ssd_t* args, const void* seq_ids_i32, int32_t row0, int32_t rows, int32_t single,
+                                  int32_t is_f32, void* stream);
+/* The recurrence over xbc token by token: decode steps, fp32, any size. */
 uint32_t logismos_launch_ssd_step(const lg_ssd_t* args, int32_t n_seqs, int32_t is_f32, void* stream);
-/* Prompts: convolution and silu of rows [row0, rows) into xbc (seq_ids [rows]; cu, slots, fresh and phase indexed by
- * them), then the recurrence 64 tokens at a time on the tensor cores (np 32 .. 128, vp <= 128). */
+/* Prompts: the recurrence 64 tokens at a time on the tensor cores (np 32 .. 128, vp <= 128). */
 int32_t logismos_ssd_has_chunked(int32_t np, int32_t vp);
-uint32_t logismos_launch_ssd_conv_bf16(const lg_ssd_t* args, const void* seq_ids_i32, int32_t row0, int32_t rows, void* stream);
 uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* args, int32_t n_seqs, void* stream);
 /* out = y silu(z), divided in `parts` equal parts of the heads * v true channels by each part's root mean square,
  * times gain. Rows are laid out [heads][vp]. */
@@ -783,6 +784,7 @@ typedef struct lg_score_bias {
   const void* bias;
   int32_t far;
   float max_abs_bias;           /* largest |bias|, natural units */
+  float max_abs_qk;             /* bound of |q . k|, 0: unknown */
   const void* gate;
   int32_t ld_gate;
   float gate_scale;

@@ -158,11 +158,10 @@ def _declare(l, partial=False):
         "logismos_launch_post_norm": [vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, vp],
         "logismos_launch_post_norm_shift_decode": [vp, i32, vp, vp, vp, vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, f32, vp],
         "logismos_launch_token_shift": [vp, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, vp],
-        "logismos_launch_split_bf16": [vp, i32, vp, i32, i32, i32, vp],
         "logismos_launch_time_mix_step": [vp, i32, i32, vp],
         "logismos_launch_ssd_step": [vp, i32, i32, vp],
         "logismos_launch_time_mix_chunked_bf16": [vp, i32, vp],
-        "logismos_launch_ssd_conv_bf16": [vp, vp, i32, i32, vp],
+        "logismos_launch_ssd_conv": [vp, vp, i32, i32, i32, i32, vp],
         "logismos_launch_ssd_chunked_bf16": [vp, i32, vp],
         "logismos_launch_gated_group_norm": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp],
         "logismos_launch_unit_qk_store": [vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, f32, f32, i64, i32, vp, vp],

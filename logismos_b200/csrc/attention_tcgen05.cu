@@ -321,12 +321,42 @@ gather_paged_kv_turbo3_kernel(const uint8_t* __restrict__ kpool, const uint8_t* 
   }
 }
 
-// Scores of the kernel below: the plain product; capped and biased by distance, with the running maximum; or
-// the same where cap and biases bound every score so tightly that exp2 of it neither over- nor underflows, and no
-// maximum is kept (one pass over the scores, the output never rescaled).
-enum { kPlain = 0, kBiased = 1, kBounded = 2 };
+// Scores of the kernel below: the plain product; capped and biased by distance, with the running maximum; the same
+// where cap and biases bound every score so tightly that exp2 of it neither over- nor underflows, and no maximum is
+// kept (one pass over the scores, the output never rescaled); and that with the cap as a polynomial, where the products
+// are known to be small (unit queries and keys): the multiplier units then leave the exponential unit to the softmax.
+enum { kPlain = 0, kBiased = 1, kBounded = 2, kPoly = 3 };
 constexpr int kBiasWindow = 160;  // distances between the 32 rows of a warp and 128 keys
 constexpr float kBoundedLog2 = 80.0f;
+
+// One block's probabilities where no maximum is kept: scores of 128 keys out of TMEM, P back over them; returns the
+// row's sum. NEAR: biases from the window (entry lane + 127 - key), else one bias for all; keys >= lim do not count.
+template <int SCORE, bool NEAR, bool FULL>
+LG_DEVINL float bounded_block(uint32_t t_s, const ScoreExt& ext, const float* window, float far_bias, int lim) {
+  float sum = 0.0f;
+#pragma unroll
+  for (int c2 = 0; c2 < 2; ++c2) {
+    uint32_t ra[32], rb[32], v[32];
+    tc_ld32(t_s + c2 * 64, ra);
+    tc_ld32(t_s + c2 * 64 + 32, rb);
+    tc_wait_ld();
+    auto prob = [&](uint32_t raw, int key) {
+      const float b = NEAR ? window[127 - key] : far_bias, qk = __uint_as_float(raw);
+      const float e = fast_exp2(SCORE == kPoly ? ext.score_poly(qk, b) : ext.score(qk, b));
+      return FULL || key < lim ? e : 0.0f;
+    };
+#pragma unroll
+    for (int i = 0; i < 32; i += 2) {
+      const int ka = c2 * 64 + i, kb = ka + 32;
+      const float a0 = prob(ra[i], ka), a1 = prob(ra[i + 1], ka + 1), b0 = prob(rb[i], kb), b1 = prob(rb[i + 1], kb + 1);
+      sum += (a0 + a1) + (b0 + b1);
+      v[i >> 1] = pack_bf16x2(a0, a1);
+      v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
+    }
+    tc_st32(t_s + c2 * 32, v);
+  }
+  return sum;
+}
 
 template <bool CAUSAL, int HD, int SCORE = kPlain>
 __global__ void __launch_bounds__(192, HD <= 128 ? 2 : 1)
@@ -440,7 +470,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int row = q * 32 + lane;
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const uint32_t t_s = tmem_base + lane_off + kColS, t_o = tmem_base + lane_off + kColO;
-    float m = SCORE == kBounded ? 0.0f : -1e30f, l = 0.0f;
+    float m = -1e30f, l = 0.0f;
     bool ok = true;
     // biased scores: the table entries of this warp's rows and the block's keys, distance first + w - 127 at window[w]
     float* window = reinterpret_cast<float*>(bars_gen + 8 * kBars + 16) + q * kBiasWindow;
@@ -450,7 +480,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       bool near = false;
       if (SCORE != kPlain) {
         const int first = q_off + q0 + q * 32 - j * 128;
-        near = first - 127 < ext.far;
+        near = first - 127 < ext.far || first < 256;  // masked blocks read the window too
         if (near) {
           __syncwarp();
 #pragma unroll
@@ -465,8 +495,19 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       int lim = kv_len - j * 128;
       if (CAUSAL) lim = min(lim, q_off + q0 + row + 1 - j * 128);
       const bool full = lim >= 128;
+      if (SCORE == kBounded || SCORE == kPoly) {
+        constexpr int S = SCORE == kPoly ? kPoly : kBounded;
+        // every lane of a warp takes the same branch: TMEM accesses are warp-wide
+        if (!__all_sync(0xffffffffu, full)) l += bounded_block<S, true, false>(t_s, ext, window + lane, far_bias, lim);
+        else if (near) l += bounded_block<S, true, true>(t_s, ext, window + lane, far_bias, lim);
+        else l += bounded_block<S, false, true>(t_s, ext, window + lane, far_bias, lim);
+        tc_wait_st();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(p_full);
+        continue;
+      }
       float mx = -1e30f;
-      if (SCORE != kBounded)
 #pragma unroll
       for (int c2 = 0; c2 < 2; ++c2) {
         uint32_t ra[32], rb[32];
@@ -494,7 +535,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       // enough in bf16, summed in fp32) and O is rescaled far less often.
       const float cand = SCORE == kPlain ? mx * sl2 : mx;
       float alpha = 1.0f;
-      if (SCORE != kBounded && cand > m + 8.0f) { alpha = fast_exp2(m - cand); m = cand; }
+      if (cand > m + 8.0f) { alpha = fast_exp2(m - cand); m = cand; }
       float sum = 0.0f;
 #pragma unroll
       for (int c2 = 0; c2 < 2; ++c2) {
@@ -504,7 +545,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         tc_wait_ld();
         if (SCORE != kPlain) {
           auto prob = [&](uint32_t raw, int key) {
-            const float e = fast_exp2(SCORE == kBounded ? score(raw, key) : score(raw, key) - m);
+            const float e = fast_exp2(score(raw, key) - m);
             return full || key < lim ? e : 0.0f;
           };
 #pragma unroll
@@ -543,7 +584,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       }
       l = l * alpha + sum;
       // S(j) complete means PV(j-1) is complete: O may be rescaled in place
-      if (SCORE != kBounded && j > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
+      if (j > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
 #pragma unroll
         for (int c = 0; c < HD / 32; ++c) {
           uint32_t r[32];
@@ -708,7 +749,7 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
                                    const void* v_pool, const void* block_tables, int32_t max_blocks, int32_t n_pool_blocks, void* out,
                                    void* scratch, int32_t n_q_tokens, int32_t total_kv_tokens, int32_t n_seqs, int32_t max_q_len,
                                    int32_t max_kv_len, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, bool turbo3, void* status,
-                                   void* stream, const ScoreExt* ext = nullptr, bool bounded = false) {
+                                   void* stream, const ScoreExt* ext = nullptr, int score = kPlain) {
   const int D = head_dim;
   if (n_q_tokens < 0 || total_kv_tokens < 0 || n_seqs < 0 || max_q_len < 0 || max_kv_len < 0 || max_blocks <= 0 ||
       n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 || (D != 128 && D != 256 && !(D == 64 && ext)) || (n_heads % n_kv_heads) ||
@@ -758,7 +799,11 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
   };
   if (ext) {
     constexpr size_t kWindow = 4 * kBiasWindow * 4;
-    if (bounded)
+    if (score == kPoly)
+      return D == 64 ? launch(attn_tcgen05_kernel<true, 64, kPoly>, Attn<64>::kSmem + kWindow)
+           : D == 128 ? launch(attn_tcgen05_kernel<true, 128, kPoly>, Attn<128>::kSmem + kWindow)
+                      : launch(attn_tcgen05_kernel<true, 256, kPoly>, Attn<256>::kSmem + kWindow);
+    if (score == kBounded)
       return D == 64 ? launch(attn_tcgen05_kernel<true, 64, kBounded>, Attn<64>::kSmem + kWindow)
            : D == 128 ? launch(attn_tcgen05_kernel<true, 128, kBounded>, Attn<128>::kSmem + kWindow)
                       : launch(attn_tcgen05_kernel<true, 256, kBounded>, Attn<256>::kSmem + kWindow);
@@ -801,10 +846,11 @@ uint32_t logismos_launch_bias_attention_prefix_bf16(const void* q, int32_t ld_q,
   lg::LaunchScope launch_scope_;
   if (n_heads <= 0 || !score_ok(score, n_heads * head_dim) || (ld_out % 8) || ld_out < n_heads * head_dim || (score->ld_gate % 8) || ((uintptr_t)score->gate & 15))
     return lg::kInvalidValue;
-  const ScoreExt ext = score_ext(score, ld_q, ld_out);
+  ScoreExt ext = score_ext(score, ld_q, ld_out);
   const bool bounded = ext.capped && (score->cap + score->max_abs_bias) * 1.4426950408889634f <= kBoundedLog2;
   return launch_prefix_attn(q, ld_q, cu_seqlens_q, kv_lens, k_pool, v_pool, block_tables, max_blocks, n_pool_blocks, out, scratch, n_q_tokens,
-                            total_kv_tokens, n_seqs, max_q_len, max_kv_len, n_heads, n_kv_heads, head_dim, false, status, stream, &ext, bounded);
+                            total_kv_tokens, n_seqs, max_q_len, max_kv_len, n_heads, n_kv_heads, head_dim, false, status, stream, &ext,
+                            !bounded ? kBiased : fit_score_poly(score, &ext) ? kPoly : kBounded);
 }
 
 uint32_t logismos_launch_varlen_attention_kv_tc_bf16(const void* q, int32_t q_row_stride, const void* cu_seqlens_q, const void* kv_lens,

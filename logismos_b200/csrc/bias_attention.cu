@@ -11,6 +11,10 @@ using namespace lg;
 
 constexpr int kBlockTokens = 16, kThreads = 256;
 
+template <typename T, int HD> struct UnitGeometry {
+  static constexpr int E = HD * sizeof(T) / 16 > 32 ? HD / 32 : 16 / (int)sizeof(T), LANES = HD / E, ITEMS = 4;
+};
+
 struct QkArgs {
   void* qkv;
   int ld;
@@ -24,41 +28,54 @@ struct QkArgs {
   int* status;
 };
 
-// warp = one head of one row: q (in place), k or v (to the cache); a lane holds HD / 32 neighbouring channels
+// A head of a row, q (in place), k or v (to the cache), is held by LANES lanes, sixteen bytes each (fp32 heads of 256:
+// thirty-two); a group of lanes takes ITEMS heads, all requested at once.
 template <typename T, int HD>
 __global__ void __launch_bounds__(kThreads)
 unit_qk_store_kernel(QkArgs p) {
   lg::pdl_prologue();
-  constexpr int E = HD / 32;
+  using G = UnitGeometry<T, HD>;
+  constexpr int E = G::E, LANES = G::LANES, ITEMS = G::ITEMS;
   struct alignas(E * sizeof(T)) Vec { T v[E]; };
-  const int per_row = p.heads + 2 * p.n_kv;
-  const int64_t item = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
-  if (item >= (int64_t)p.rows * per_row) return;
-  const int row = (int)(item / per_row), h = (int)(item % per_row), lane = threadIdx.x & 31;
-  T* src = reinterpret_cast<T*>(p.qkv) + (size_t)row * p.ld + h * HD + lane * E;
-  Vec x = *reinterpret_cast<const Vec*>(src);
-  const bool is_v = h >= p.heads + p.n_kv;
-  if (!is_v) {
+  const int per_row = p.heads + 2 * p.n_kv, lane = threadIdx.x % LANES;
+  const int64_t total = (int64_t)p.rows * per_row, first = ((int64_t)blockIdx.x * kThreads + threadIdx.x) / LANES * ITEMS;
+  Vec x[ITEMS];
+#pragma unroll
+  for (int k = 0; k < ITEMS; ++k) {
+    if (first + k >= total) continue;
+    const int row = (int)((first + k) / per_row), h = (int)((first + k) % per_row);
+    x[k] = *reinterpret_cast<const Vec*>(reinterpret_cast<const T*>(p.qkv) + (size_t)row * p.ld + h * HD + lane * E);
+  }
+#pragma unroll
+  for (int k = 0; k < ITEMS; ++k) {
+    const bool in = first + k < total;
+    const int row = in ? (int)((first + k) / per_row) : 0, h = in ? (int)((first + k) % per_row) : 0;
+    const bool is_v = h >= p.heads + p.n_kv;
     float f[E], ss = 0.0f;
 #pragma unroll
-    for (int i = 0; i < E; ++i) { f[i] = rec::Io<T>::load(&x.v[i]); ss += f[i] * f[i]; }
-    float m = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
-    if (h < p.heads && p.coef != 0.0f) m *= 1.0f + p.coef * logf(floorf(__fdiv_rn((float)(p.pos[row] + 1), p.every)) + 1.0f);
+    for (int i = 0; i < E; ++i) { f[i] = in ? rec::Io<T>::load(&x[k].v[i]) : 0.0f; ss += f[i] * f[i]; }
 #pragma unroll
-    for (int i = 0; i < E; ++i) rec::Io<T>::store(&x.v[i], f[i] * m);
+    for (int o = 1; o < LANES; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!in) continue;
+    if (!is_v) {
+      float m = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
+      if (h < p.heads && p.coef != 0.0f) m *= 1.0f + p.coef * logf(floorf(__fdiv_rn((float)(p.pos[row] + 1), p.every)) + 1.0f);
+#pragma unroll
+      for (int i = 0; i < E; ++i) rec::Io<T>::store(&x[k].v[i], f[i] * m);
+    }
+    if (h < p.heads) {
+      *reinterpret_cast<Vec*>(reinterpret_cast<T*>(p.qkv) + (size_t)row * p.ld + h * HD + lane * E) = x[k];
+      continue;
+    }
+    const int64_t slot = p.slots[row];
+    if (slot < 0 || slot >= p.n_slots) {
+      if (lane == 0 && p.status) atomicExch(p.status, 1);
+      continue;
+    }
+    const int kvh = h - p.heads - (is_v ? p.n_kv : 0);
+    T* pool = reinterpret_cast<T*>(is_v ? p.vpool : p.kpool);
+    *reinterpret_cast<Vec*>(pool + (size_t)slot * p.n_kv * HD + kvh * HD + lane * E) = x[k];
   }
-  if (h < p.heads) {
-    *reinterpret_cast<Vec*>(src) = x;
-    return;
-  }
-  const int64_t slot = p.slots[row];
-  if (slot < 0 || slot >= p.n_slots) {
-    if (lane == 0 && p.status) atomicExch(p.status, 1);
-    return;
-  }
-  const int kvh = h - p.heads - (is_v ? p.n_kv : 0);
-  T* pool = reinterpret_cast<T*>(is_v ? p.vpool : p.kpool);
-  *reinterpret_cast<Vec*>(pool + (size_t)slot * p.n_kv * HD + kvh * HD + lane * E) = x;
 }
 
 // CTA = (row, head), keys in tiles of 64
@@ -140,15 +157,17 @@ uint32_t logismos_launch_unit_qk_store(void* qkv, int32_t ld, void* k_pool, void
     return lg::kInvalidValue;
   const QkArgs p{qkv, ld, k_pool, v_pool, (const int64_t*)slot_mapping_i64, (const int*)positions_i32, rows, n_heads, n_kv_heads, dim, eps, coef, every,
                  n_pool_slots, (int*)status_i32};
-  const int64_t blocks = ((int64_t)rows * (n_heads + 2 * n_kv_heads) + kThreads / 32 - 1) / (kThreads / 32);
-  if (blocks > 0x7fffffff) return lg::kInvalidValue;
-  auto go = [&](auto kern) {
+  const int64_t items = (int64_t)rows * (n_heads + 2 * n_kv_heads);
+  auto go = [&](auto kern, int per_block) -> uint32_t {
+    const int64_t blocks = (items + per_block - 1) / per_block;
+    if (blocks > 0x7fffffff) return lg::kInvalidValue;
     lg::launch(kern, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
-  if (is_f32) return head_dim == 64 ? go(unit_qk_store_kernel<float, 64>) : head_dim == 128 ? go(unit_qk_store_kernel<float, 128>) : go(unit_qk_store_kernel<float, 256>);
-  return head_dim == 64 ? go(unit_qk_store_kernel<__nv_bfloat16, 64>) : head_dim == 128 ? go(unit_qk_store_kernel<__nv_bfloat16, 128>)
-                                                                                       : go(unit_qk_store_kernel<__nv_bfloat16, 256>);
+#define LG_UNIT(T, HD) go(unit_qk_store_kernel<T, HD>, kThreads / UnitGeometry<T, HD>::LANES * UnitGeometry<T, HD>::ITEMS)
+  if (is_f32) return head_dim == 64 ? LG_UNIT(float, 64) : head_dim == 128 ? LG_UNIT(float, 128) : LG_UNIT(float, 256);
+  return head_dim == 64 ? LG_UNIT(__nv_bfloat16, 64) : head_dim == 128 ? LG_UNIT(__nv_bfloat16, 128) : LG_UNIT(__nv_bfloat16, 256);
+#undef LG_UNIT
 }
 
 uint32_t logismos_launch_bias_attention_f32(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables,

@@ -249,11 +249,20 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
           const int ncol = n_blk * BN + c;
           if (EPI == kEpiGroups && ncol >= groups.n_main) {
             if (row < M) {
-              float* dst = reinterpret_cast<float*>(groups.tail) + (size_t)row * groups.ld_tail + (ncol - groups.n_main);
+              const int c0 = ncol - groups.n_main, width = N - groups.n_main;
+              float* dst = reinterpret_cast<float*>(groups.tail) + (size_t)row * groups.ld_tail + c0;
+              __nv_bfloat16* parts = reinterpret_cast<__nv_bfloat16*>(groups.tail_parts) + (size_t)row * 2 * width + c0;
 #pragma unroll
               for (int j = 0; j < 32; ++j) {
-                const float v = __uint_as_float(r[j]);
-                if (ncol + j < N) dst[j] = groups.tail_cap > 0.0f ? groups.tail_cap * tanhf(v / groups.tail_cap) : v;
+                if (ncol + j >= N) continue;
+                float v = __uint_as_float(r[j]);
+                if (groups.tail_cap > 0.0f) v = groups.tail_cap * tanhf(v / groups.tail_cap);
+                dst[j] = v;
+                if (groups.tail_parts) {
+                  const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+                  parts[j] = hi;
+                  parts[width + j] = __float2bfloat16_rn(v - __bfloat162float(hi));
+                }
               }
             }
             continue;
@@ -277,8 +286,28 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
               }
           }
         }
+      } else if (EPI == LG_EPI_F32 && (ldc & 3) == 0) {  // whole 128-byte rows through the staging slabs
+        for (int c = 0; c < BN; c += 32) {
+          uint32_t r[32];
+          tc_ld32(t_row + c, r);
+          tc_wait_ld();
+          const int ncol = n_blk * BN + c;
+          if (ncol >= N) break;
+          const int b = slab_acquire();
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            float v[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              v[i] = __uint_as_float(r[4 * j + i]);
+              if (bias && ncol + 4 * j + i < N) v[i] += bias[ncol + 4 * j + i];
+              if (ep.p0 > 0.0f) v[i] = ep.p0 * tanhf(v[i] / ep.p0);
+            }
+            slab_write(slabs + b * 4096, lane, j, make_uint4(__float_as_uint(v[0]), __float_as_uint(v[1]), __float_as_uint(v[2]), __float_as_uint(v[3])));
+          }
+          slab_release(b, ncol, row0, row0 < M);
+        }
       } else if (EPI == LG_EPI_F32) {
-        const bool vec = (ldc & 3) == 0;
         for (int c = 0; c < BN; c += 32) {
           uint32_t r[32];
           tc_ld32(t_row + c, r);
@@ -295,12 +324,8 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                 if (bias && ncol + j + i < N) v[i] += bias[ncol + j + i];
                 if (ep.p0 > 0.0f) v[i] = ep.p0 * tanhf(v[i] / ep.p0);
               }
-              if (vec && ncol + j + 4 <= N) {
-                *reinterpret_cast<float4*>(dst + j) = make_float4(v[0], v[1], v[2], v[3]);
-              } else {
 #pragma unroll
-                for (int i = 0; i < 4; ++i) if (ncol + j + i < N) dst[j + i] = v[i];
-              }
+              for (int i = 0; i < 4; ++i) if (ncol + j + i < N) dst[j + i] = v[i];
             }
           }
         }
@@ -386,7 +411,7 @@ uint32_t launch_cfg(const void* a, const void* w, const float* bias, void* out, 
   const int copies = EPI == kEpiGroups ? groups.n_groups : 1;
   if (!make_map(&ma, a, (uint64_t)m * copies, (uint64_t)k, (uint64_t)lda, BM)) return lg::kInvalidValue;
   if (!make_map(&mw, w, (uint64_t)n, (uint64_t)k, (uint64_t)k, BN)) return lg::kInvalidValue;
-  if (EPI == LG_EPI_RESID_F32) {  // fp32 [m, n] in 32 x 32 boxes for the reduce-add epilogue
+  if (EPI == LG_EPI_RESID_F32 || (EPI == LG_EPI_F32 && ldc % 4 == 0)) {  // fp32 [m, n] in 32 x 32 boxes
     if (!make_map(&mo, out, (uint64_t)m, (uint64_t)n, (uint64_t)ldc, 32, true)) return lg::kInvalidValue;
   } else {
     mo = ma;  // unused by the direct-store epilogues
@@ -431,7 +456,8 @@ uint32_t launch_epi(const void* a, const void* w, const float* bias, void* out, 
     }
     const long tiles = (long)mt * ((n + bn - 1) / bn);
     const long waves = (tiles + sms - 1) / sms;
-    const long cost = waves * bn;
+    long cost = waves * bn;
+    if (EPI == kEpiGroups && bn == 128) cost += cost / 6;  // the narrow tile runs at about six sevenths of the wide one's rate
     if (best_cost < 0 || cost < best_cost) { best_cost = cost; best_bn = bn; }
   }
   if (best_bn == 256) return launch_cfg<256, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream, groups);

@@ -145,8 +145,14 @@ linear_small_kernel(SmallArgs p) {
     if (p.bias) v += p.bias[wrow];
     if (p.epi == LG_EPI_RELU2) { v = fmaxf(v, 0.0f); v *= v; }
     if (p.epi == kEpiGroups && wrow >= p.groups.n_main) {
-      reinterpret_cast<float*>(p.groups.tail)[(size_t)r * p.groups.ld_tail + wrow - p.groups.n_main] =
-          p.groups.tail_cap > 0.0f ? p.groups.tail_cap * tanhf(v / p.groups.tail_cap) : v;
+      const int tc = wrow - p.groups.n_main, width = p.n - p.groups.n_main;
+      if (p.groups.tail_cap > 0.0f) v = p.groups.tail_cap * tanhf(v / p.groups.tail_cap);
+      reinterpret_cast<float*>(p.groups.tail)[(size_t)r * p.groups.ld_tail + tc] = v;
+      if (p.groups.tail_parts) {
+        __nv_bfloat16* parts = reinterpret_cast<__nv_bfloat16*>(p.groups.tail_parts) + (size_t)r * 2 * width + tc;
+        parts[0] = __float2bfloat16_rn(v);
+        parts[width] = __float2bfloat16_rn(v - __bfloat162float(parts[0]));
+      }
       continue;
     }
     const size_t o = (size_t)blockIdx.z * p.out_stride + (size_t)r * p.ldc + wrow;

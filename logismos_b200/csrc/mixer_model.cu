@@ -4,8 +4,8 @@
 //
 // A step packs decode tokens first and prefill chunks after them (step_batch.h):
 //   embed -> per layer
-//     state-space: one GEMM to [z | x | B | C] and fp32 dt -> decode rows: convolution + recurrence in one launch;
-//       prefill rows: convolution, chunk-parallel recurrence -> gate + norm -> output GEMM
+//     state-space: one GEMM to [z | x | B | C] and fp32 dt -> convolution -> recurrence, token by token for decode
+//       rows, chunk-parallel for prefill rows -> gate + norm -> output GEMM
 //     parallel: one GEMM over the stream and its five token-shift mixes to attention q | k | v | gate, time-mixing
 //       r | k | v | g and the fp32 low-rank activations of the decay -> unit q, k + cache store -> attention with its
 //       gate into the left columns of one activation row; time mixing with its norm and gate into the right ones ->
@@ -16,6 +16,7 @@
 // keeps the padding of every activation zero.
 #include <cuda_runtime.h>
 
+#include <algorithm>
 #include <cmath>
 #include <mutex>
 #include <string>
@@ -92,6 +93,7 @@ uint32_t linear(Mixer* m, const void* a, int lda, const Buf& w, int n, int k, vo
 uint32_t projections(Mixer* m, const MLayer& L, const MWeights& W, int rows, cudaStream_t s) {
   lg_linear_groups_t g = L.groups;
   g.tail = m->tail.p;
+  g.tail_parts = L.c.kind == LG_MIXER_PARALLEL && m->batch.n_pre > 0 ? m->low2.p : nullptr;
   m->launches += 1;
   const int Hp = m->Hp;
   if (m->cfg.is_f32) return logismos_launch_linear_groups_f32(m->h.p, W.w_in.p, m->proj.p, rows, L.N, Hp, Hp, g.n_main, &g, s);
@@ -155,15 +157,17 @@ uint32_t ssd_mixer(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   a.xbc = m->xbc.p; a.ld_xbc = L.channels;
   const bool chunked = !f32 && B.n_pre > 0 && logismos_ssd_has_chunked(L.Np, L.Vp);
   const int serial = chunked ? B.n_dec : B.n_seqs;  // sequences that go token by token
+  if (B.n_dec > 0) LG_TRY(logismos_launch_ssd_conv(&a, m->dev(B.seq_ids), 0, B.n_dec, 1, f32, s), "state-space convolution");
+  if (B.n_pre > 0) LG_TRY(logismos_launch_ssd_conv(&a, m->dev(B.seq_ids), B.n_dec, T, 0, f32, s), "state-space convolution");
+  m->launches += (B.n_dec > 0) + (B.n_pre > 0);
   if (serial > 0) {
     LG_TRY(logismos_launch_ssd_step(&a, serial, f32, s), "state-space recurrence");
     m->launches += 1;
   }
   if (chunked) {
-    LG_TRY(logismos_launch_ssd_conv_bf16(&a, m->dev(B.seq_ids), B.n_dec, T, s), "state-space convolution");
     a.state_slots = m->dev(B.state) + B.n_dec; a.fresh = m->dev(B.fresh) + B.n_dec; a.phase = m->dev(B.phase) + B.n_dec; a.cu = m->dev(B.cu) + B.n_dec;
     LG_TRY(logismos_launch_ssd_chunked_bf16(&a, B.n_pre, s), "state-space recurrence (prompts)");
-    m->launches += 2;
+    m->launches += 1;
   }
   LG_TRY(logismos_launch_gated_group_norm(m->ffb.p, inner, m->proj.p, L.groups.n_main, W.gain.p, m->act.p, L.Kout, f32, T, L.c.ssd_heads, L.c.ssd_vdim, L.Vp,
                                           L.c.ssd_norm_groups, c.norm_eps, s), "gate and norm");
@@ -183,6 +187,12 @@ uint32_t attention(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   m->launches += 1;
   lg_score_bias_t sb{};
   sb.scale = L.c.scale; sb.cap = L.c.softcap; sb.bias = W.bias.p; sb.far = L.c.bias_max; sb.max_abs_bias = W.max_bias;
+  {  // unit queries and keys: |q . k| <= dim times the largest temperature, with room for their rounding
+    int longest = 1;
+    for (int k = 0; k < B.n_seqs; ++k) longest = std::max(longest, B.cached[(size_t)k] + B.newl[(size_t)k]);
+    const float t = L.c.temp_coef != 0.0f ? std::fabs(L.c.temp_coef) * std::log(std::floor(longest / L.c.temp_every) + 1.0f) : 0.0f;
+    sb.max_abs_qk = 1.01f * L.c.dim * (1.0f + t);
+  }
   sb.gate = proj + (size_t)(HD + 2 * GD) * esz; sb.ld_gate = P; sb.gate_scale = L.c.left_scale;
   if (f32) {
     LG_TRY(logismos_launch_bias_attention_f32(proj, P, L.kpool.p, L.vpool.p, m->dev(B.tables), m->dev(B.seq_ids), m->dev(B.pos), out, L.Kout, T, MB,
@@ -226,13 +236,12 @@ uint32_t time_mixing(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   }
   if (chunked) {
     const int rows = B.T - B.n_dec, w = L.Lr;
-    LG_TRY(logismos_launch_split_bf16((const float*)m->tail.p + (size_t)B.n_dec * w, w, m->low2.p, rows, w, w, s), "decay activations");
-    LG_TRY(logismos_launch_linear_t_act_bf16(m->low2.p, W.w2.p, W.w0.p, (float*)m->z.p + (size_t)B.n_dec * L.Rw, rows, L.Rw, 2 * w, 2 * w, L.Rw,
+    LG_TRY(logismos_launch_linear_t_act_bf16((const uint16_t*)m->low2.p + (size_t)B.n_dec * 2 * w, W.w2.p, W.w0.p, (float*)m->z.p + (size_t)B.n_dec * L.Rw, rows, L.Rw, 2 * w, 2 * w, L.Rw,
                                              LG_EPI_F32 | LG_EPI_STATIC_W, 0, 0, 0, m->status.p, s), "decay");
     a.z = m->z.p; a.ld_z = L.Rw;
     a.state_slots = m->dev(B.state) + B.n_dec; a.fresh = m->dev(B.fresh) + B.n_dec; a.cu = m->dev(B.cu) + B.n_dec;
     LG_TRY(logismos_launch_time_mix_chunked_bf16(&a, B.n_pre, s), "time mixing (prompts)");
-    m->launches += 3;
+    m->launches += 2;
   }
   return 0;
 }
@@ -511,11 +520,11 @@ uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_
   lim.extra_bytes = (size_t)c.max_out_rows * 4;
   m->acc_bytes = (T < (size_t)kAccRows ? T : (size_t)kAccRows) * Hp * 4;
   ok = ok && m->x.alloc(T * Hp * 4) && zeroed(m->h, (1 + kMixes) * T * Hp * esz) && zeroed(m->proj, T * proj_w * esz) && m->tail.alloc(T * tail_w * 4) &&
-       zeroed(m->act, T * act_w * esz) && zeroed(m->ffb, T * ff_w * esz) && m->y.alloc(T * Hp * 4) && m->y_acc.alloc(m->acc_bytes) &&
+       zeroed(m->act, T * act_w * esz) && zeroed(m->ffb, T * ff_w * esz) && zeroed(m->xbc, T * xbc_w * esz) && m->y.alloc(T * Hp * 4) && m->y_acc.alloc(m->acc_bytes) &&
        m->last.alloc((size_t)c.max_out_rows * Hp * esz) && m->logits.alloc((size_t)c.max_out_rows * c.vocab * 4) && m->tokens.alloc((size_t)c.max_out_rows * 4) &&
        m->status.alloc(4) && (!c.keep_layers || m->hist.alloc((size_t)(c.n_layers + 1) * T * Hp * 4));
   if (!c.is_f32)
-    ok = ok && m->low2.alloc(T * low_w * 2) && m->z.alloc(T * z_w * 4) && zeroed(m->xbc, T * xbc_w * 2) && m->attn_ws.alloc(ws) && m->dec_scratch.alloc(scratch);
+    ok = ok && m->low2.alloc(T * low_w * 2) && m->z.alloc(T * z_w * 4) && m->attn_ws.alloc(ws) && m->dec_scratch.alloc(scratch);
   ok = ok && cudaMemset(m->status.p, 0, 4) == cudaSuccess && m->batch.alloc(lim) && m->dev_batch.alloc(m->batch.capacity) &&
        cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking) == cudaSuccess;
   m->slot_phase.assign(slots, 0);

@@ -169,18 +169,6 @@ token_shift_kernel(const float* __restrict__ x, const int* __restrict__ seq_ids,
   }
 }
 
-// fp32 [rows, n] -> bf16 [rows, 2 width]: the rounded values, and in the second half what rounding dropped
-__global__ void split_bf16_kernel(const float* __restrict__ in, int ld, __nv_bfloat16* __restrict__ out, int rows, int n, int width) {
-  lg::pdl_prologue();
-  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= (int64_t)rows * width) return;
-  const int r = (int)(i / width), c = (int)(i % width);
-  const float v = c < n ? in[(size_t)r * ld + c] : 0.0f;
-  const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-  out[(size_t)r * 2 * width + c] = hi;
-  out[(size_t)r * 2 * width + width + c] = __float2bfloat16_rn(v - __bfloat162float(hi));
-}
-
 struct Shape { int threads, nv; };
 Shape shape_of(int ld) {
   const int v = ld / 4;
@@ -240,14 +228,6 @@ uint32_t logismos_launch_token_shift(const void* x_f32, void* h, int32_t out_f32
   const dim3 grid((unsigned)((rows + kRun - 1) / kRun), (unsigned)((ld / 4 + 127) / 128));
   lg::launch(token_shift_kernel, grid, dim3(128), 0, (cudaStream_t)stream, (const float*)x_f32, (const int*)seq_ids_i32, (const int*)cu_seqlens_i32, h, c, rows,
              ld, out_f32);
-  return lg::launch_status();
-}
-
-uint32_t logismos_launch_split_bf16(const void* in_f32, int32_t ld, void* out_bf16, int32_t rows, int32_t n, int32_t width, void* stream) {
-  lg::LaunchScope launch_scope_;
-  if (!in_f32 || !out_bf16 || rows <= 0 || n <= 0 || width < n || ld < n) return lg::kInvalidValue;
-  lg::launch(split_bf16_kernel, dim3((unsigned)(((int64_t)rows * width + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, (const float*)in_f32, ld,
-             (__nv_bfloat16*)out_bf16, rows, n, width);
   return lg::launch_status();
 }
 

@@ -1,6 +1,8 @@
 // Scores that are capped and biased by distance, and the output gate, shared by the attention kernels
 // (lg_score_bias_t).
 #pragma once
+#include <cmath>
+
 #include "common.cuh"
 #include "logismos_kernels.h"
 
@@ -15,16 +17,47 @@ struct ScoreExt {
   int far;
   float pre, post;               // capped: post tanh(.) + bias with the exponent pre q . k; else post q . k + bias
   int capped;
+  float poly[5];                 // post tanh(.) as q . k (poly[0] + poly[1] s + ...) with s = (q . k)^2, where products are bounded
   const __nv_bfloat16* gate;
   int ld_gate;
   float gate_scale;
   int ld_q, ld_out;
   LG_DEVINL float score(float qk, float b) const { return fmaf(post, capped ? tanh_from_exp2(qk * pre) : qk, b); }
+  LG_DEVINL float score_poly(float qk, float b) const {
+    const float s = qk * qk;
+    return fmaf(qk, fmaf(fmaf(fmaf(fmaf(poly[4], s, poly[3]), s, poly[2]), s, poly[1]), s, poly[0]), b);
+  }
   LG_DEVINL float gated(float o, float g) const { return o * __fdividef(gate_scale, 1.0f + __expf(-g)); }
 };
 
 inline bool score_ok(const lg_score_bias_t* s, int width) {
   return s && s->scale > 0.0f && s->cap >= 0.0f && s->bias && s->far >= 0 && s->gate && s->ld_gate >= width;
+}
+
+// The polynomial above by interpolation of tanh(x) / x in x^2 at Chebyshev nodes on [0, limit^2]: for limit <= 0.7 within
+// 2e-7 of it. False: products may be too large, and nothing is set.
+inline bool fit_score_poly(const lg_score_bias_t* s, ScoreExt* e) {
+  const double x_max = (double)s->max_abs_qk * s->scale / (s->cap > 0.0f ? s->cap : 1.0f);
+  if (!(s->cap > 0.0f) || !(s->max_abs_qk > 0.0f) || x_max > 0.7) return false;
+  const int n = 5;
+  const double U = x_max * x_max, pi = 3.14159265358979323846;
+  double node[n], coef[n];  // Newton's divided differences
+  for (int i = 0; i < n; ++i) {
+    node[i] = 0.5 * U * (1.0 + std::cos(pi * (2 * i + 1) / (2 * n)));
+    const double x = std::sqrt(node[i]);
+    coef[i] = x > 1e-9 ? std::tanh(x) / x : 1.0;
+  }
+  for (int k = 1; k < n; ++k)
+    for (int i = n - 1; i >= k; --i) coef[i] = (coef[i] - coef[i - 1]) / (node[i] - node[i - k]);
+  double p[n] = {coef[n - 1], 0, 0, 0, 0};  // to powers of u
+  for (int k = n - 2; k >= 0; --k) {
+    for (int i = n - 1; i > 0; --i) p[i] = p[i - 1] - node[k] * p[i];
+    p[0] = coef[k] - node[k] * p[0];
+  }
+  const double a = (double)s->scale / s->cap;  // x = a q.k
+  double f = (double)s->cap * 1.4426950408889634 * a;
+  for (int i = 0; i < n; ++i, f *= a * a) e->poly[i] = (float)(p[i] * f);
+  return true;
 }
 
 inline ScoreExt score_ext(const lg_score_bias_t* s, int ld_q, int ld_out) {

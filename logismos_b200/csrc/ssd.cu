@@ -7,8 +7,9 @@
 // The last taps - 1 inputs of the convolution are its state: a slot holds two copies, a step reads the one its
 // phase names and writes the other.
 //
-// ssd_step_kernel: CTA = (head, sequence), tokens one after the other, convolution included. Decode steps, fp32.
-// ssd_conv_kernel, ssd_chunk_kernel: prompts. The chunked form resolves 64 tokens together: with c_i the sum of the
+// ssd_conv_kernel: convolution and silu of all rows.
+// ssd_step_kernel: CTA = (head, sequence), tokens one after the other. Decode steps, fp32, sizes beyond the next form.
+// ssd_chunk_kernel: prompts. The chunked form resolves 64 tokens together: with c_i the sum of the
 // log-decays up to token i of the chunk and S the state before it,
 //   P_ij = (C_i . B_j) exp(c_i - c_j) dt_j (j <= i);   y_i = sum_j P_ij x_j + exp(c_i) S^T C_i + D x_i
 //   S <- exp(c_last) S + sum_j B_j (dt_j exp(c_last - c_j) x_j)^T
@@ -23,7 +24,7 @@ namespace {
 using namespace lg;
 using namespace lg::rec;
 
-constexpr int kMaxTaps = 8, kMaxChannels = 768;  // VP + 2 NP of a head
+constexpr int kMaxTaps = 8;
 
 struct SsdArgs {
   const void* proj;        // z at 0, x at heads * vp, B, C behind it
@@ -45,33 +46,26 @@ struct SsdArgs {
   void* y;                 // activation format, [rows, ld_y], head h at h * vp
   int ld_y;
   int heads, groups, np, vp;
-  const void* xbc;         // convolved channels (the chunked form)
+  void* xbc;               // convolved channels [rows, ld_xbc], activation format
   int ld_xbc;
-  LG_DEVINL int channels() const { return heads * vp + 2 * groups * np; }
+  __host__ __device__ __forceinline__ int channels() const { return heads * vp + 2 * groups * np; }
 };
 
+// PT up to 4 pieces leave room for four CTAs per SM, whose states are then in flight together
 template <typename T, int PT>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, PT == 0 ? 2 : PT <= 8 ? 4 : 2)
 ssd_step_kernel(SsdArgs p) {
   lg::pdl_trigger();
   constexpr int NP = PT ? PT : 1;
-  extern __shared__ float hist[];   // [taps - 1][local channels] raw inputs
-  __shared__ float act[kMaxChannels], red[8 * 128];
+  __shared__ __align__(16) float xs[256], bs[256], cs[256], red[8 * 128];
   const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
-  const int vp = p.vp, np = p.np, group = head / (p.heads / p.groups), inner = p.heads * vp, nch = vp + 2 * np, all = p.channels();
-  const bool owns_group = head % (p.heads / p.groups) == 0;
+  const int vp = p.vp, np = p.np, group = head / (p.heads / p.groups), inner = p.heads * vp;
   const Tile t(np, vp);
-  const size_t slot = (size_t)p.state_slots[seq];
-  float* st = p.state + (slot * p.heads + head) * np * vp;
+  float* st = p.state + ((size_t)p.state_slots[seq] * p.heads + head) * np * vp;
   const bool fresh = p.fresh[seq] != 0;
-  const int ph = p.phase[seq] & 1, keep = p.taps - 1;
-  const float* old = p.conv_state + (slot * 2 + ph) * keep * all;
-  float* next = p.conv_state + (slot * 2 + 1 - ph) * keep * all;
   const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  // channel of the convolution behind local channel c
-  auto chan = [&](int c) { return c < vp ? head * vp + c : c < vp + np ? inner + group * np + c - vp : inner + (p.groups + group) * np + c - vp - np; };
-  // states of an earlier step and weights do not depend on the kernels before this one
+  // the state of an earlier step and the weights do not depend on the kernels before this one
   float4 S[NP];
   if (PT) {
 #pragma unroll
@@ -80,33 +74,22 @@ ssd_step_kernel(SsdArgs p) {
       S[i] = !fresh && row < np ? *reinterpret_cast<const float4*>(st + (size_t)row * vp + t.c4) : zero;
     }
   }
-  for (int e = tid; e < keep * nch; e += kThreads) hist[e] = fresh ? 0.0f : old[(size_t)(e / nch) * all + chan(e % nch)];
   const float bias = __ldg(p.dt_bias + head), a = expf(__ldg(p.log_a + head)), skip = __ldg(p.skip + head);
   lg::pdl_wait();
-  __syncthreads();
-  int at = 0;  // oldest row of hist
   for (int tok = t0; tok < t1; ++tok) {
-    const T* row = reinterpret_cast<const T*>(p.proj) + (size_t)tok * p.ld + inner;
+    const T* row = reinterpret_cast<const T*>(p.xbc) + (size_t)tok * p.ld_xbc;
     const float dt = softplus_f(p.dt[(size_t)tok * p.ld_dt + head] + bias), decay = expf(-a * dt);
-    for (int c = tid; c < nch; c += kThreads) {  // a thread meets the same channels for every token
-      const int g = chan(c);
-      const float cur = Io<T>::load(row + g);
-      float s = fmaf(__ldg(p.conv_w + (size_t)keep * all + g), cur, __ldg(p.conv_b + g));
-      for (int j = 0; j < keep; ++j) {
-        const int r = at + j < keep ? at + j : at + j - keep;
-        s = fmaf(__ldg(p.conv_w + (size_t)j * all + g), hist[r * nch + c], s);
-      }
-      if (keep > 0) hist[at * nch + c] = cur;
-      act[c] = silu_f(s);
+    if (tid < vp) xs[tid] = Io<T>::load(row + head * vp + tid);
+    if (tid < np) {
+      bs[tid] = dt * Io<T>::load(row + inner + group * np + tid);
+      cs[tid] = Io<T>::load(row + inner + (p.groups + group) * np + tid);
     }
-    if (keep > 0 && ++at == keep) at = 0;
     __syncthreads();
-    const float4 x4 = *reinterpret_cast<const float4*>(act + t.c4);
-    const float4 dx = make_float4(dt * x4.x, dt * x4.y, dt * x4.z, dt * x4.w);
+    const float4 x4 = *reinterpret_cast<const float4*>(xs + t.c4);
     float4 o = zero;
     auto visit = [&](int r, float4& s) {
-      const float b = act[vp + r], c = act[vp + np + r];
-      s = make_float4(fmaf(decay, s.x, b * dx.x), fmaf(decay, s.y, b * dx.y), fmaf(decay, s.z, b * dx.z), fmaf(decay, s.w, b * dx.w));
+      const float b = bs[r], c = cs[r];
+      s = make_float4(fmaf(decay, s.x, b * x4.x), fmaf(decay, s.y, b * x4.y), fmaf(decay, s.z, b * x4.z), fmaf(decay, s.w, b * x4.w));
       o.x = fmaf(c, s.x, o.x); o.y = fmaf(c, s.y, o.y); o.z = fmaf(c, s.z, o.z); o.w = fmaf(c, s.w, o.w);
     };
     if (PT) {
@@ -114,6 +97,13 @@ ssd_step_kernel(SsdArgs p) {
       for (int i = 0; i < NP; ++i) {
         const int r = t.r0 + i * t.step;
         if (r < np) visit(r, S[i]);
+      }
+      if (tok + 1 == t1) {  // the new state is on its way out before the sums meet
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int r = t.r0 + i * t.step;
+          if (r < np) *reinterpret_cast<float4*>(st + (size_t)r * vp + t.c4) = S[i];
+        }
       }
     } else {
       for (int r = t.r0; r < np; r += t.step) {
@@ -125,54 +115,53 @@ ssd_step_kernel(SsdArgs p) {
     }
     reduce_store(t, o, red);
     __syncthreads();
-    if (tid < vp) Io<T>::store(reinterpret_cast<T*>(p.y) + (size_t)tok * p.ld_y + head * vp + tid, reduce_load(vp, red, tid) + skip * act[tid]);
+    if (tid < vp) Io<T>::store(reinterpret_cast<T*>(p.y) + (size_t)tok * p.ld_y + head * vp + tid, reduce_load(vp, red, tid) + skip * xs[tid]);
     if (tok + 1 < t1) __syncthreads();
-  }
-  if (PT) {
-#pragma unroll
-    for (int i = 0; i < NP; ++i) {
-      const int row = t.r0 + i * t.step;
-      if (row < np) *reinterpret_cast<float4*>(st + (size_t)row * vp + t.c4) = S[i];
-    }
-  }
-  __syncthreads();
-  for (int e = tid; e < keep * nch; e += kThreads) {
-    const int j = e / nch, c = e % nch;
-    if (c < vp || owns_group) next[(size_t)j * all + chan(c)] = hist[((at + j) % keep) * nch + c];
   }
 }
 
-// Convolution and silu of ragged prompt rows [row0, rows): a thread owns four channels and a run of consecutive rows.
-constexpr int kRun = 8;
-template <int TAPS>
+// Convolution and silu of ragged rows [row0, rows): a thread owns four channels and a run of RUN consecutive rows.
+template <typename T> struct Raw4;
+template <> struct Raw4<float> { typedef float4 type; };
+template <> struct Raw4<__nv_bfloat16> { typedef uint2 type; };
+LG_DEVINL float4 widen(float4 v) { return v; }
+LG_DEVINL float4 widen(uint2 u) {
+  const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+// z sigmoid(z) where bf16 is the result: sigmoid(z) = (1 + tanh(z / 2)) / 2 with the approximate tanh (relative error 2^-11)
+LG_DEVINL float silu_bf16(float z) {
+  float t;
+  asm("tanh.approx.f32 %0, %1;\n" : "=f"(t) : "f"(0.5f * z));
+  const float h = 0.5f * z;
+  return fmaf(h, t, h);
+}
+
+template <typename T, int TAPS, int RUN>
 __global__ void __launch_bounds__(128)
 ssd_conv_kernel(SsdArgs p, const int* __restrict__ seq_ids, int row0, int rows) {
   lg::pdl_prologue();
+  typedef typename Raw4<T>::type Raw;
   constexpr int HN = TAPS - 1;
   const int all = p.channels(), c0 = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
   if (c0 >= all) return;
-  const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.proj) + p.heads * p.vp + c0;
-  __nv_bfloat16* dst = const_cast<__nv_bfloat16*>(reinterpret_cast<const __nv_bfloat16*>(p.xbc)) + c0;
-  float4 w[TAPS];
+  const T* src = reinterpret_cast<const T*>(p.proj) + p.heads * p.vp + c0;
+  T* dst = reinterpret_cast<T*>(p.xbc) + c0;
+  auto load = [&](int t) { return *reinterpret_cast<const Raw*>(src + (size_t)t * p.ld); };
+  const int first = row0 + blockIdx.x * RUN, last = min(rows, first + RUN);
+  Raw in[RUN];
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) in[i] = load(first + i < last ? first + i : first);
+  float4 w[TAPS], prev[HN > 0 ? HN : 1];
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) w[j] = __ldg(reinterpret_cast<const float4*>(p.conv_w + (size_t)j * all + c0));
   const float4 bias = __ldg(reinterpret_cast<const float4*>(p.conv_b + c0));
-  auto load = [&](int t) {
-    const uint2 u = *reinterpret_cast<const uint2*>(src + (size_t)t * p.ld);
-    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
-    return make_float4(a.x, a.y, b.x, b.y);
-  };
   auto fma = [](float4 a, float4 x, float4 c) { return make_float4(fmaf(a.x, x.x, c.x), fmaf(a.y, x.y, c.y), fmaf(a.z, x.z, c.z), fmaf(a.w, x.w, c.w)); };
-  auto act = [](float z) { return __fdividef(z, 1.0f + __expf(-z)); };
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  const int first = row0 + blockIdx.x * kRun, last = min(rows, first + kRun);
-  float4 in[kRun], prev[HN > 0 ? HN : 1];
-#pragma unroll
-  for (int i = 0; i < kRun; ++i) in[i] = first + i < last ? load(first + i) : zero;
   int cur = -1, t0 = 0, len = 0;
   float* next = nullptr;
 #pragma unroll
-  for (int i = 0; i < kRun; ++i) {
+  for (int i = 0; i < RUN; ++i) {
     const int t = first + i;
     if (t >= last) break;
     const int s = seq_ids[t];
@@ -187,7 +176,7 @@ ssd_conv_kernel(SsdArgs p, const int* __restrict__ seq_ids, int row0, int rows) 
 #pragma unroll
       for (int j = 0; j < HN; ++j) {
         const int idx = t - t0 - HN + j;  // place inside the step's tokens of this sequence; negative: the state
-        if (idx >= 0) prev[j] = load(t0 + idx);
+        if (idx >= 0) prev[j] = widen(load(t0 + idx));
         else prev[j] = fresh ? zero : *reinterpret_cast<const float4*>(old + (size_t)(HN + idx) * all);
       }
       if (t == t0) {  // rows of the old state that stay in the new one
@@ -196,15 +185,38 @@ ssd_conv_kernel(SsdArgs p, const int* __restrict__ seq_ids, int row0, int rows) 
           if (j + len < HN) *reinterpret_cast<float4*>(next + (size_t)j * all) = fresh ? zero : *reinterpret_cast<const float4*>(old + (size_t)(j + len) * all);
       }
     }
-    float4 y = fma(w[TAPS - 1], in[i], bias);
+    const float4 x = widen(in[i]);
+    float4 y = fma(w[TAPS - 1], x, bias);
 #pragma unroll
     for (int j = 0; j < HN; ++j) y = fma(w[j], prev[j], y);
-    *reinterpret_cast<uint2*>(dst + (size_t)t * p.ld_xbc) = make_uint2(pack_bf16x2(act(y.x), act(y.y)), pack_bf16x2(act(y.z), act(y.w)));
+    if constexpr (sizeof(T) == 2)
+      *reinterpret_cast<uint2*>(dst + (size_t)t * p.ld_xbc) = make_uint2(pack_bf16x2(silu_bf16(y.x), silu_bf16(y.y)), pack_bf16x2(silu_bf16(y.z), silu_bf16(y.w)));
+    else
+      *reinterpret_cast<float4*>(dst + (size_t)t * p.ld_xbc) = make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w));
     const int keep = HN - (len - (t - t0));  // row of the new state this token becomes, if any
-    if (keep >= 0) *reinterpret_cast<float4*>(next + (size_t)keep * all) = in[i];
+    if (keep >= 0) *reinterpret_cast<float4*>(next + (size_t)keep * all) = x;
 #pragma unroll
     for (int j = 0; j + 1 < HN; ++j) prev[j] = prev[j + 1];
-    if (HN > 0) prev[HN > 0 ? HN - 1 : 0] = in[i];
+    if (HN > 0) prev[HN > 0 ? HN - 1 : 0] = x;
+  }
+}
+
+template <typename T, int RUN>
+uint32_t launch_conv(const SsdArgs& p, const int* seq_ids, int row0, int rows, cudaStream_t s) {
+  const dim3 grid((unsigned)((rows - row0 + RUN - 1) / RUN), (unsigned)(((p.heads * p.vp + 2 * p.groups * p.np) / 4 + 127) / 128));
+  auto go = [&](auto kern) {
+    lg::launch(kern, grid, dim3(128), 0, s, p, seq_ids, row0, rows);
+    return lg::launch_status();
+  };
+  switch (p.taps) {
+    case 1: return go(ssd_conv_kernel<T, 1, RUN>);
+    case 2: return go(ssd_conv_kernel<T, 2, RUN>);
+    case 3: return go(ssd_conv_kernel<T, 3, RUN>);
+    case 4: return go(ssd_conv_kernel<T, 4, RUN>);
+    case 5: return go(ssd_conv_kernel<T, 5, RUN>);
+    case 6: return go(ssd_conv_kernel<T, 6, RUN>);
+    case 7: return go(ssd_conv_kernel<T, 7, RUN>);
+    default: return go(ssd_conv_kernel<T, 8, RUN>);
   }
 }
 
@@ -380,7 +392,51 @@ ssd_chunk_kernel(SsdArgs p) {
   }
 }
 
-// y silu(z), normalised in equal parts of `width` channels. CTA = (row, part). VEC: channels are contiguous (no
+// y silu(z), normalised in equal parts of `width` contiguous bf16 channels: a warp per (row, part), NV times eight
+// channels per lane.
+template <int NV>
+__global__ void __launch_bounds__(256)
+gated_norm_warp_kernel(const __nv_bfloat16* __restrict__ y, int ld_y, const __nv_bfloat16* __restrict__ z, int ld_z, const float* __restrict__ gain,
+                       __nv_bfloat16* __restrict__ out, int ld_out, int rows, int parts, int width, float eps) {
+  lg::pdl_prologue();
+  const int64_t item = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (item >= (int64_t)rows * parts) return;
+  const int r = (int)(item / parts), c0 = (int)(item % parts) * width, lane = threadIdx.x & 31;
+  uint4 a[NV], b[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = 8 * (lane + 32 * i);
+    a[i] = b[i] = make_uint4(0u, 0u, 0u, 0u);
+    if (c < width) {
+      a[i] = *reinterpret_cast<const uint4*>(y + (size_t)r * ld_y + c0 + c);
+      b[i] = *reinterpret_cast<const uint4*>(z + (size_t)r * ld_z + c0 + c);
+    }
+  }
+  float x[NV][8], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const uint32_t wa[4] = {a[i].x, a[i].y, a[i].z, a[i].w}, wb[4] = {b[i].x, b[i].y, b[i].z, b[i].w};
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 fa = unpack_bf16x2(wa[k]), fb = unpack_bf16x2(wb[k]);
+      x[i][2 * k] = fa.x * silu_bf16(fb.x);
+      x[i][2 * k + 1] = fa.y * silu_bf16(fb.y);
+      ss = fmaf(x[i][2 * k], x[i][2 * k], fmaf(x[i][2 * k + 1], x[i][2 * k + 1], ss));
+    }
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)width + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = 8 * (lane + 32 * i);
+    if (c >= width) continue;
+    const float4 g0 = __ldg(reinterpret_cast<const float4*>(gain + c0 + c)), g1 = __ldg(reinterpret_cast<const float4*>(gain + c0 + c + 4));
+    *reinterpret_cast<uint4*>(out + (size_t)r * ld_out + c0 + c) =
+        make_uint4(pack_bf16x2(x[i][0] * inv * g0.x, x[i][1] * inv * g0.y), pack_bf16x2(x[i][2] * inv * g0.z, x[i][3] * inv * g0.w),
+                   pack_bf16x2(x[i][4] * inv * g1.x, x[i][5] * inv * g1.y), pack_bf16x2(x[i][6] * inv * g1.z, x[i][7] * inv * g1.w));
+  }
+}
+
+// The same for any width and format, a CTA per (row, part). VEC: channels are contiguous (no
 // padding between heads) and eight of them are moved at once.
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(512)
@@ -469,10 +525,10 @@ extern "C" {
 uint32_t logismos_launch_ssd_step(const lg_ssd_t* a, int32_t n_seqs, int32_t is_f32, void* stream) {
   lg::LaunchScope launch_scope_;
   if (!args_ok(a, n_seqs)) return lg::kInvalidValue;
+  if (!a->xbc || a->ld_xbc < make_args(a).channels()) return lg::kInvalidValue;
   const SsdArgs p = make_args(a);
-  const size_t smem = (size_t)(p.taps - 1) * (p.vp + 2 * p.np) * 4;
   auto go = [&](auto kern) {
-    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3(kThreads), smem, (cudaStream_t)stream, p);
+    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3(kThreads), 0, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
   const int pt = pieces(p.np, p.vp);
@@ -484,26 +540,14 @@ uint32_t logismos_launch_ssd_step(const lg_ssd_t* a, int32_t n_seqs, int32_t is_
 
 int32_t logismos_ssd_has_chunked(int32_t np, int32_t vp) { return pow2(np, 32, 128) && pow2(vp, 16, 128) ? 1 : 0; }
 
-uint32_t logismos_launch_ssd_conv_bf16(const lg_ssd_t* a, const void* seq_ids_i32, int32_t row0, int32_t rows, void* stream) {
+uint32_t logismos_launch_ssd_conv(const lg_ssd_t* a, const void* seq_ids_i32, int32_t row0, int32_t rows, int32_t single, int32_t is_f32, void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!args_ok(a, 1) || !seq_ids_i32 || row0 < 0 || rows <= row0 || !a->xbc || a->ld % 4 || a->ld_xbc % 4 || a->ld_xbc < a->heads * a->vp + 2 * a->groups * a->np)
-    return lg::kInvalidValue;
+  if (!args_ok(a, 1) || !seq_ids_i32 || row0 < 0 || rows <= row0 || !a->xbc || a->ld % 4 || a->ld_xbc % 4 || a->ld_xbc < make_args(a).channels()) return lg::kInvalidValue;
   const SsdArgs p = make_args(a);
-  const dim3 grid((unsigned)((rows - row0 + kRun - 1) / kRun), (unsigned)(((a->heads * a->vp + 2 * a->groups * a->np) / 4 + 127) / 128));
-  auto go = [&](auto kern) {
-    lg::launch(kern, grid, dim3(128), 0, (cudaStream_t)stream, p, (const int*)seq_ids_i32, row0, rows);
-    return lg::launch_status();
-  };
-  switch (a->taps) {
-    case 1: return go(ssd_conv_kernel<1>);
-    case 2: return go(ssd_conv_kernel<2>);
-    case 3: return go(ssd_conv_kernel<3>);
-    case 4: return go(ssd_conv_kernel<4>);
-    case 5: return go(ssd_conv_kernel<5>);
-    case 6: return go(ssd_conv_kernel<6>);
-    case 7: return go(ssd_conv_kernel<7>);
-    default: return go(ssd_conv_kernel<8>);
-  }
+  const int* ids = (const int*)seq_ids_i32;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (is_f32) return launch_conv<float, 1>(p, ids, row0, rows, s);
+  return single ? launch_conv<__nv_bfloat16, 1>(p, ids, row0, rows, s) : launch_conv<__nv_bfloat16, 16>(p, ids, row0, rows, s);
 }
 
 uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* a, int32_t n_seqs, void* stream) {
@@ -532,6 +576,15 @@ uint32_t logismos_launch_gated_group_norm(const void* y, int32_t ld_y, const voi
   const bool vec = v == vp && width % 8 == 0 && width <= 4 * 8 * 512 && ld_y % 8 == 0 && ld_z % 8 == 0 && ld_out % 8 == 0;
   int threads = ((vec ? width / 8 : width) + 31) / 32 * 32;
   if (threads > 512) threads = 512;
+  if (!is_f32 && vec && width <= 2048) {
+    auto warp = [&](auto kern) {
+      lg::launch(kern, dim3((unsigned)(((int64_t)rows * parts + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, (const __nv_bfloat16*)y, ld_y, (const __nv_bfloat16*)z, ld_z,
+                 (const float*)gain_f32, (__nv_bfloat16*)out, ld_out, rows, parts, width, eps);
+      return lg::launch_status();
+    };
+    return width <= 256 ? warp(gated_norm_warp_kernel<1>) : width <= 512 ? warp(gated_norm_warp_kernel<2>) : width <= 1024 ? warp(gated_norm_warp_kernel<4>)
+                                                                                                           : warp(gated_norm_warp_kernel<8>);
+  }
   const dim3 grid((unsigned)rows, (unsigned)parts);
   auto go = [&](auto kern, auto* t) {
     using T = std::remove_pointer_t<decltype(t)>;

@@ -46,7 +46,7 @@ struct MixArgs {
 };
 
 template <typename T, int PT>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, PT && PT <= 4 ? 4 : 2)
 time_mix_step_kernel(MixArgs p) {
   lg::pdl_trigger();
   constexpr int NP = PT ? PT : 1;
@@ -131,6 +131,13 @@ time_mix_step_kernel(MixArgs p) {
         const int r = t.r0 + i * t.step;
         if (r < dp) visit(r, S[i]);
       }
+      if (tok + 1 == t1) {  // the new state is on its way out before the sums meet
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int r = t.r0 + i * t.step;
+          if (r < dp) *reinterpret_cast<float4*>(st + (size_t)r * dp + t.c4) = S[i];
+        }
+      }
     } else {
       for (int r = t.r0; r < dp; r += t.step) {
         float4* at = reinterpret_cast<float4*>(st + (size_t)r * dp + t.c4);
@@ -144,13 +151,6 @@ time_mix_step_kernel(MixArgs p) {
     const float oc = tid < dp ? reduce_load(dp, red, tid) : 0.0f;
     const float inv = 1.0f / sqrtf(block_sum(oc * oc, bred) / (float)p.d + p.eps);  // its barriers also free the vectors above
     if (tid < dp) Io<T>::store(reinterpret_cast<T*>(p.out) + (size_t)tok * p.ld_out + h0 + tid, oc * inv * gain * silu_f(g) * p.scale);
-  }
-  if (PT) {
-#pragma unroll
-    for (int i = 0; i < NP; ++i) {
-      const int row = t.r0 + i * t.step;
-      if (row < dp) *reinterpret_cast<float4*>(st + (size_t)row * dp + t.c4) = S[i];
-    }
   }
 }
 
