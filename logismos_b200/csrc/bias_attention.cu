@@ -12,7 +12,7 @@ using namespace lg;
 constexpr int kBlockTokens = 16, kThreads = 256;
 
 template <typename T, int HD> struct UnitGeometry {
-  static constexpr int E = HD * sizeof(T) / 16 > 32 ? HD / 32 : 16 / (int)sizeof(T), LANES = HD / E, ITEMS = 4;
+  static constexpr int E = HD * sizeof(T) / 16 > 32 ? HD / 32 : 16 / (int)sizeof(T), LANES = HD / E;
 };
 
 struct QkArgs {
@@ -30,15 +30,15 @@ struct QkArgs {
 
 // A head of a row, q (in place), k or v (to the cache), is held by LANES lanes, sixteen bytes each (fp32 heads of 256:
 // thirty-two); a group of lanes takes ITEMS heads, all requested at once.
-template <typename T, int HD>
+template <typename T, int HD, int ITEMS>
 __global__ void __launch_bounds__(kThreads)
 unit_qk_store_kernel(QkArgs p) {
   lg::pdl_prologue();
   using G = UnitGeometry<T, HD>;
-  constexpr int E = G::E, LANES = G::LANES, ITEMS = G::ITEMS;
+  constexpr int E = G::E, LANES = G::LANES;
   struct alignas(E * sizeof(T)) Vec { T v[E]; };
-  const int per_row = p.heads + 2 * p.n_kv, lane = threadIdx.x % LANES;
-  const int64_t total = (int64_t)p.rows * per_row, first = ((int64_t)blockIdx.x * kThreads + threadIdx.x) / LANES * ITEMS;
+  const uint32_t per_row = p.heads + 2 * p.n_kv, lane = threadIdx.x % LANES;
+  const uint32_t total = p.rows * per_row, first = (blockIdx.x * kThreads + threadIdx.x) / LANES * ITEMS;
   Vec x[ITEMS];
 #pragma unroll
   for (int k = 0; k < ITEMS; ++k) {
@@ -158,13 +158,16 @@ uint32_t logismos_launch_unit_qk_store(void* qkv, int32_t ld, void* k_pool, void
   const QkArgs p{qkv, ld, k_pool, v_pool, (const int64_t*)slot_mapping_i64, (const int*)positions_i32, rows, n_heads, n_kv_heads, dim, eps, coef, every,
                  n_pool_slots, (int*)status_i32};
   const int64_t items = (int64_t)rows * (n_heads + 2 * n_kv_heads);
+  if (items > 0x3fffffff) return lg::kInvalidValue;
   auto go = [&](auto kern, int per_block) -> uint32_t {
     const int64_t blocks = (items + per_block - 1) / per_block;
     if (blocks > 0x7fffffff) return lg::kInvalidValue;
     lg::launch(kern, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
-#define LG_UNIT(T, HD) go(unit_qk_store_kernel<T, HD>, kThreads / UnitGeometry<T, HD>::LANES * UnitGeometry<T, HD>::ITEMS)
+#define LG_UNIT(T, HD)                                                                             \
+  (items < 20000 ? go(unit_qk_store_kernel<T, HD, 1>, kThreads / UnitGeometry<T, HD>::LANES)       \
+                 : go(unit_qk_store_kernel<T, HD, 4>, kThreads / UnitGeometry<T, HD>::LANES * 4))
   if (is_f32) return head_dim == 64 ? LG_UNIT(float, 64) : head_dim == 128 ? LG_UNIT(float, 128) : LG_UNIT(float, 256);
   return head_dim == 64 ? LG_UNIT(__nv_bfloat16, 64) : head_dim == 128 ? LG_UNIT(__nv_bfloat16, 128) : LG_UNIT(__nv_bfloat16, 256);
 #undef LG_UNIT

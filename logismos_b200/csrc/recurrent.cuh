@@ -1,7 +1,9 @@
-// Pieces shared by the token-serial recurrences whose per-head state is a matrix [rows][cols] in fp32: a CTA of
-// 256 threads holds it as float4 pieces, thread -> four columns and every (1024 / cols)-th row. cols is a power of
-// two from 16 to 1024. PT pieces per thread stay in registers over the tokens of a call; PT = 0: too many for that,
-// the state is read and written in memory for every token.
+// Pieces shared by the kernels of recurrences whose per-head state is a matrix [rows][cols] in fp32.
+//
+// Token-serial forms: a CTA of 256 threads, thread -> four columns (cols: a power of two from 16 to 1024) and every
+// (1024 / cols)-th row. The state waits in shared memory, every thread fetching its own pieces asynchronously and
+// reading back only those: what is in flight takes no registers and needs no barrier, so that many CTAs of a step
+// stream their states at once. A state too large for that is read and written in memory for every token.
 #pragma once
 #include "common.cuh"
 
@@ -34,14 +36,44 @@ struct Tile {
   }
 };
 
-// pieces per thread that hold a state of this size, or 0
-inline int pieces(int rows, int cols) {
-  const int n = (rows * cols + 4 * kThreads - 1) / (4 * kThreads);
-  return n <= 1 ? 1 : n <= 2 ? 2 : n <= 4 ? 4 : n <= 8 ? 8 : n <= 16 ? 16 : 0;
+// shared memory that holds a state, or 0: too large
+inline size_t state_smem(int rows, int cols) {
+  const size_t bytes = ((size_t)rows * cols * 4 + 16 * kThreads - 1) / (16 * kThreads) * (16 * kThreads);
+  return bytes <= 160 * 1024 ? bytes : 0;
 }
 
+// the state of one head: requested (or zeroed) at once, then visited row piece by row piece
+struct State {
+  float4* own;        // this thread's pieces in shared memory, kThreads apart; NULL: in memory
+  float* st;
+  LG_DEVINL State(void* smem, bool in_smem, float* st_) : own(in_smem ? reinterpret_cast<float4*>(smem) + threadIdx.x : nullptr), st(st_) {}
+  LG_DEVINL void request(const Tile& t, bool fresh) {
+    if (!own) return;
+    int i = 0;
+    for (int r = t.r0; r < t.rows; r += t.step, ++i) {
+      if (fresh) own[i * kThreads] = make_float4(0.f, 0.f, 0.f, 0.f);
+      else cp_async16(smem_u32(own + i * kThreads), st + (size_t)r * t.cols + t.c4);
+    }
+    cp_async_commit();
+  }
+  LG_DEVINL void arrived() { if (own) cp_async_wait<0>(); }
+  // f(row, piece) updates each piece; `first`: the first token of a sequence that starts here; `last`: leaves for memory
+  template <typename F>
+  LG_DEVINL void visit(const Tile& t, bool first, bool last, F f) {
+    int i = 0;
+#pragma unroll 4
+    for (int r = t.r0; r < t.rows; r += t.step, ++i) {
+      float4* at = reinterpret_cast<float4*>(st + (size_t)r * t.cols + t.c4);
+      float4 s = own ? own[i * kThreads] : first ? make_float4(0.f, 0.f, 0.f, 0.f) : *at;
+      f(r, s);
+      if (own && !last) own[i * kThreads] = s;
+      else *at = s;
+    }
+  }
+};
+
 // sum over the threads that share columns; the result of column c is in out[c] for every thread after the barrier.
-// red: [8][cols] floats (cols <= 128) or [kThreads / (cols / 4)][cols]
+// red: 1024 floats
 LG_DEVINL int reduce_groups(int cols) { const int nv = cols >> 2; return kThreads / (nv < 32 ? 32 : nv); }
 LG_DEVINL void reduce_store(const Tile& t, float4 v, float* red) {
   const int nv = t.cols >> 2;

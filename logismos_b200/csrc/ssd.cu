@@ -51,29 +51,20 @@ struct SsdArgs {
   __host__ __device__ __forceinline__ int channels() const { return heads * vp + 2 * groups * np; }
 };
 
-// PT up to 4 pieces leave room for four CTAs per SM, whose states are then in flight together
-template <typename T, int PT>
-__global__ void __launch_bounds__(kThreads, PT == 0 ? 2 : PT <= 8 ? 4 : 2)
-ssd_step_kernel(SsdArgs p) {
+template <typename T>
+__global__ void __launch_bounds__(kThreads, 5)
+ssd_step_kernel(SsdArgs p, int in_smem) {
   lg::pdl_trigger();
-  constexpr int NP = PT ? PT : 1;
-  __shared__ __align__(16) float xs[256], bs[256], cs[256], red[8 * 128];
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ __align__(16) float xs[256], bs[256], cs[256], red[1024];
   const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
   const int vp = p.vp, np = p.np, group = head / (p.heads / p.groups), inner = p.heads * vp;
   const Tile t(np, vp);
-  float* st = p.state + ((size_t)p.state_slots[seq] * p.heads + head) * np * vp;
   const bool fresh = p.fresh[seq] != 0;
-  const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
-  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   // the state of an earlier step and the weights do not depend on the kernels before this one
-  float4 S[NP];
-  if (PT) {
-#pragma unroll
-    for (int i = 0; i < NP; ++i) {
-      const int row = t.r0 + i * t.step;
-      S[i] = !fresh && row < np ? *reinterpret_cast<const float4*>(st + (size_t)row * vp + t.c4) : zero;
-    }
-  }
+  State S(smem, in_smem, p.state + ((size_t)p.state_slots[seq] * p.heads + head) * np * vp);
+  S.request(t, fresh);
+  const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
   const float bias = __ldg(p.dt_bias + head), a = expf(__ldg(p.log_a + head)), skip = __ldg(p.skip + head);
   lg::pdl_wait();
   for (int tok = t0; tok < t1; ++tok) {
@@ -85,34 +76,14 @@ ssd_step_kernel(SsdArgs p) {
       cs[tid] = Io<T>::load(row + inner + (p.groups + group) * np + tid);
     }
     __syncthreads();
+    if (tok == t0) S.arrived();
     const float4 x4 = *reinterpret_cast<const float4*>(xs + t.c4);
-    float4 o = zero;
-    auto visit = [&](int r, float4& s) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    S.visit(t, fresh && tok == t0, tok + 1 == t1, [&](int r, float4& s) {
       const float b = bs[r], c = cs[r];
       s = make_float4(fmaf(decay, s.x, b * x4.x), fmaf(decay, s.y, b * x4.y), fmaf(decay, s.z, b * x4.z), fmaf(decay, s.w, b * x4.w));
       o.x = fmaf(c, s.x, o.x); o.y = fmaf(c, s.y, o.y); o.z = fmaf(c, s.z, o.z); o.w = fmaf(c, s.w, o.w);
-    };
-    if (PT) {
-#pragma unroll
-      for (int i = 0; i < NP; ++i) {
-        const int r = t.r0 + i * t.step;
-        if (r < np) visit(r, S[i]);
-      }
-      if (tok + 1 == t1) {  // the new state is on its way out before the sums meet
-#pragma unroll
-        for (int i = 0; i < NP; ++i) {
-          const int r = t.r0 + i * t.step;
-          if (r < np) *reinterpret_cast<float4*>(st + (size_t)r * vp + t.c4) = S[i];
-        }
-      }
-    } else {
-      for (int r = t.r0; r < np; r += t.step) {
-        float4* q = reinterpret_cast<float4*>(st + (size_t)r * vp + t.c4);
-        float4 s = fresh && tok == t0 ? zero : *q;
-        visit(r, s);
-        *q = s;
-      }
-    }
+    });
     reduce_store(t, o, red);
     __syncthreads();
     if (tid < vp) Io<T>::store(reinterpret_cast<T*>(p.y) + (size_t)tok * p.ld_y + head * vp + tid, reduce_load(vp, red, tid) + skip * xs[tid]);
@@ -527,15 +498,14 @@ uint32_t logismos_launch_ssd_step(const lg_ssd_t* a, int32_t n_seqs, int32_t is_
   if (!args_ok(a, n_seqs)) return lg::kInvalidValue;
   if (!a->xbc || a->ld_xbc < make_args(a).channels()) return lg::kInvalidValue;
   const SsdArgs p = make_args(a);
-  auto go = [&](auto kern) {
-    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3(kThreads), 0, (cudaStream_t)stream, p);
+  const size_t smem = state_smem(p.np, p.vp);
+  auto go = [&](auto kern) -> uint32_t {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3(kThreads), smem, (cudaStream_t)stream, p, smem > 0 ? 1 : 0);
     return lg::launch_status();
   };
-  const int pt = pieces(p.np, p.vp);
-#define LG_STEP(T) pt == 1 ? go(ssd_step_kernel<T, 1>) : pt == 2 ? go(ssd_step_kernel<T, 2>) : pt == 4 ? go(ssd_step_kernel<T, 4>) : pt == 8 ? go(ssd_step_kernel<T, 8>) \
-                   : pt == 16 ? go(ssd_step_kernel<T, 16>) : go(ssd_step_kernel<T, 0>)
-  return is_f32 ? (LG_STEP(float)) : (LG_STEP(__nv_bfloat16));
-#undef LG_STEP
+  return is_f32 ? go(ssd_step_kernel<float>) : go(ssd_step_kernel<__nv_bfloat16>);
 }
 
 int32_t logismos_ssd_has_chunked(int32_t np, int32_t vp) { return pow2(np, 32, 128) && pow2(vp, 16, 128) ? 1 : 0; }

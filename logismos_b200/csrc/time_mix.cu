@@ -45,43 +45,26 @@ struct MixArgs {
   float scale, eps;
 };
 
-template <typename T, int PT>
-__global__ void __launch_bounds__(kThreads, PT && PT <= 4 ? 4 : 2)
-time_mix_step_kernel(MixArgs p) {
+template <typename T>
+__global__ void __launch_bounds__(kThreads, 4)
+time_mix_step_kernel(MixArgs p, int in_smem) {
   lg::pdl_trigger();
-  constexpr int NP = PT ? PT : 1;
-  __shared__ float sr[256], sk[256], sv[256], sw[256], red[8 * 128], bred[32];
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ __align__(16) float sr[256], sk[256], sv[256], sw[256], su[256], red[1024], ssq[8];
   const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
   const int dp = p.dp, h0 = head * dp;
   const Tile t(dp, dp);
-  float* st = p.state + ((size_t)p.state_slots[seq] * p.heads + head) * dp * dp;
   const bool fresh = p.fresh[seq] != 0;
-  const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
-  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   // the state, left by an earlier step, and the weights do not depend on the kernels before this one
-  float4 S[NP];
-  if (PT) {
-#pragma unroll
-    for (int i = 0; i < NP; ++i) {
-      const int row = t.r0 + i * t.step;
-      S[i] = !fresh && row < dp ? *reinterpret_cast<const float4*>(st + (size_t)row * dp + t.c4) : zero;
-    }
-  }
-  float uu = 0.0f, w0 = 0.0f, gain = 0.0f;
-  __shared__ float su[256];
-  if (tid < dp) { uu = __ldg(p.u + h0 + tid); w0 = __ldg(p.w0 + h0 + tid); gain = __ldg(p.gain + h0 + tid); su[tid] = uu; }
-  constexpr int kAhead = 4;  // 16-byte pieces of W2 per thread requested ahead: four threads per channel, 64 channels
-  uint4 wv[kAhead];
-  const int ch0 = tid >> 2, part = tid & 3;
-#pragma unroll
-  for (int j = 0; j < kAhead; ++j) {
-    wv[j] = make_uint4(0u, 0u, 0u, 0u);
-    if (!p.z && ch0 < dp && 32 * j < p.rank) wv[j] = __ldg(reinterpret_cast<const uint4*>(p.w2 + (size_t)(h0 + ch0) * p.ld_w2 + 32 * j + 8 * part));
-  }
+  State S(smem, in_smem, p.state + ((size_t)p.state_slots[seq] * p.heads + head) * dp * dp);
+  S.request(t, fresh);
+  const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
+  float w0 = 0.0f, gain = 0.0f;
+  if (tid < dp) { w0 = __ldg(p.w0 + h0 + tid); gain = __ldg(p.gain + h0 + tid); su[tid] = __ldg(p.u + h0 + tid); }
   lg::pdl_wait();
   for (int tok = t0; tok < t1; ++tok) {
     const T* row = reinterpret_cast<const T*>(p.proj) + (size_t)tok * p.ld + h0;
-    float g = 0.0f, z = 0.0f;
+    float z = 0.0f, g = 0.0f;
     if (tid < dp) {
       sr[tid] = Io<T>::load(row + p.off_r + tid);
       sk[tid] = Io<T>::load(row + p.off_k + tid);
@@ -89,34 +72,32 @@ time_mix_step_kernel(MixArgs p) {
       g = Io<T>::load(row + p.off_g + tid);
       if (p.z) z = p.z[(size_t)tok * p.ld_z + h0 + tid];
     }
-    if (!p.z) {
+    if (!p.z) {  // four threads per channel, eight of its columns at a time
       const float* low = p.low + (size_t)tok * p.ld_low;
-      for (int ch = ch0; ch < dp; ch += 64) {
+      for (int ch = tid >> 2; ch < dp; ch += 64) {
+        const __nv_bfloat16* wr = p.w2 + (size_t)(h0 + ch) * p.ld_w2;
         float s = 0.0f;
-        for (int j0 = 0; j0 < p.rank; j0 += 32 * kAhead) {
-#pragma unroll
-          for (int j = 0; j < kAhead; ++j) {
-            const int c = j0 + 32 * j + 8 * part;
-            if (c - 8 * part >= p.rank) break;
-            const uint4 w = ch == ch0 && j0 == 0 ? wv[j] : __ldg(reinterpret_cast<const uint4*>(p.w2 + (size_t)(h0 + ch) * p.ld_w2 + c));
-            const float4 a = *reinterpret_cast<const float4*>(low + c), b = *reinterpret_cast<const float4*>(low + c + 4);
-            const float2 w01 = unpack_bf16x2(w.x), w23 = unpack_bf16x2(w.y), w45 = unpack_bf16x2(w.z), w67 = unpack_bf16x2(w.w);
-            s = fmaf(a.x, w01.x, fmaf(a.y, w01.y, fmaf(a.z, w23.x, fmaf(a.w, w23.y, s))));
-            s = fmaf(b.x, w45.x, fmaf(b.y, w45.y, fmaf(b.z, w67.x, fmaf(b.w, w67.y, s))));
-          }
+#pragma unroll 2
+        for (int c = 8 * (tid & 3); c < p.rank; c += 32) {
+          const uint4 w = __ldg(reinterpret_cast<const uint4*>(wr + c));
+          const float4 a = *reinterpret_cast<const float4*>(low + c), b = *reinterpret_cast<const float4*>(low + c + 4);
+          const float2 w01 = unpack_bf16x2(w.x), w23 = unpack_bf16x2(w.y), w45 = unpack_bf16x2(w.z), w67 = unpack_bf16x2(w.w);
+          s = fmaf(a.x, w01.x, fmaf(a.y, w01.y, fmaf(a.z, w23.x, fmaf(a.w, w23.y, s))));
+          s = fmaf(b.x, w45.x, fmaf(b.y, w45.y, fmaf(b.z, w67.x, fmaf(b.w, w67.y, s))));
         }
         s += __shfl_xor_sync(0xffffffffu, s, 1);
         s += __shfl_xor_sync(0xffffffffu, s, 2);
-        if (part == 0) sw[ch] = s;
+        if ((tid & 3) == 0) sw[ch] = s;
       }
       __syncthreads();
       if (tid < dp) z = sw[tid] + w0;
     }
     if (tid < dp) sw[tid] = expf(-expf(z));
     __syncthreads();
+    if (tok == t0) S.arrived();
     const float4 v4 = *reinterpret_cast<const float4*>(sv + t.c4);
-    float4 o = zero;
-    auto visit = [&](int r, float4& s) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    S.visit(t, fresh && tok == t0, tok + 1 == t1, [&](int r, float4& s) {
       const float kr = sk[r], rr = sr[r], wr = sw[r], ur = su[r];
       const float4 kv = make_float4(kr * v4.x, kr * v4.y, kr * v4.z, kr * v4.w);
       o.x = fmaf(rr, fmaf(ur, kv.x, s.x), o.x);
@@ -124,33 +105,19 @@ time_mix_step_kernel(MixArgs p) {
       o.z = fmaf(rr, fmaf(ur, kv.z, s.z), o.z);
       o.w = fmaf(rr, fmaf(ur, kv.w, s.w), o.w);
       s = make_float4(fmaf(wr, s.x, kv.x), fmaf(wr, s.y, kv.y), fmaf(wr, s.z, kv.z), fmaf(wr, s.w, kv.w));
-    };
-    if (PT) {
-#pragma unroll
-      for (int i = 0; i < NP; ++i) {
-        const int r = t.r0 + i * t.step;
-        if (r < dp) visit(r, S[i]);
-      }
-      if (tok + 1 == t1) {  // the new state is on its way out before the sums meet
-#pragma unroll
-        for (int i = 0; i < NP; ++i) {
-          const int r = t.r0 + i * t.step;
-          if (r < dp) *reinterpret_cast<float4*>(st + (size_t)r * dp + t.c4) = S[i];
-        }
-      }
-    } else {
-      for (int r = t.r0; r < dp; r += t.step) {
-        float4* at = reinterpret_cast<float4*>(st + (size_t)r * dp + t.c4);
-        float4 s = fresh && tok == t0 ? zero : *at;
-        visit(r, s);
-        *at = s;
-      }
-    }
+    });
     reduce_store(t, o, red);
     __syncthreads();
     const float oc = tid < dp ? reduce_load(dp, red, tid) : 0.0f;
-    const float inv = 1.0f / sqrtf(block_sum(oc * oc, bred) / (float)p.d + p.eps);  // its barriers also free the vectors above
-    if (tid < dp) Io<T>::store(reinterpret_cast<T*>(p.out) + (size_t)tok * p.ld_out + h0 + tid, oc * inv * gain * silu_f(g) * p.scale);
+    const float part = warp_sum(oc * oc);
+    if ((tid & 31) == 0) ssq[tid >> 5] = part;
+    __syncthreads();
+    if (tid < dp) {
+      float ss = 0.0f;
+      for (int i = 0; i < dp / 32; ++i) ss += ssq[i];
+      Io<T>::store(reinterpret_cast<T*>(p.out) + (size_t)tok * p.ld_out + h0 + tid, oc * (p.scale / sqrtf(ss / (float)p.d + p.eps)) * gain * silu_f(g));
+    }
+    if (tok + 1 < t1) __syncthreads();
   }
 }
 
@@ -252,11 +219,19 @@ time_mix_chunk_kernel(MixArgs p) {
     }
     __syncthreads();
     const uint32_t R_a = smem_u32(R), K_a = smem_u32(K), V_a = smem_u32(Vt + buf * C::kTile), Rl_a = smem_u32(Rl), Kl_a = smem_u32(Kl);
-    // ---- coefficients inside the blocks
-    for (int I = warp; I < 4; I += C::kThreadsC / 32) {
+    // the gates of the epilogue, requested now
+    uint4 gate[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int e = tid + i * C::kThreadsC, row = e / kOct;
+      gate[i] = row < n ? *reinterpret_cast<const uint4*>(proj + (int64_t)(tb + row) * p.ld + p.off_g + 8 * (e % kOct)) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    // ---- coefficients inside the blocks, eight columns j at a time
+    for (int task = warp; task < 8; task += C::kThreadsC / 32) {
+      const int I = task >> 1, nt = task & 1;
       float worst = 0.0f;
       for (int d = lane; d < DP; d += 32) worst = fmaxf(worst, -tot[I * DP + d]);
-      float acc[2][4] = {};
+      float acc[4] = {}, low1[4] = {}, low2[4] = {};
       if (__all_sync(0xffffffffu, worst <= kMaxSpan)) {
 #pragma unroll
         for (int ks = 0; ks < NT; ++ks) {
@@ -265,45 +240,41 @@ time_mix_chunk_kernel(MixArgs p) {
           frag_a(al, Rl_a, kPitch, 16 * I, 16 * ks, lane);
           frag_b(bh, K_a, kPitch, 16 * I, 16 * ks, lane);
           frag_b(bl, Kl_a, kPitch, 16 * I, 16 * ks, lane);
+          const uint32_t h0 = nt ? bh[2] : bh[0], h1 = nt ? bh[3] : bh[1], l0 = nt ? bl[2] : bl[0], l1 = nt ? bl[3] : bl[1];
 #pragma unroll
           for (int q = 0; q < 4; ++q) {  // columns 2 t (+ 8 for q >= 2)
             const float2 f = *reinterpret_cast<const float2*>(tot + I * DP + 16 * ks + 8 * (q >> 1) + 2 * t);
             const float2 x = unpack_bf16x2(ah[q]), y = unpack_bf16x2(al[q]);
             split2((x.x + y.x) * fast_exp2(-f.x), (x.y + y.y) * fast_exp2(-f.y), ah[q], al[q]);
           }
-#pragma unroll
-          for (int nt = 0; nt < 2; ++nt) {
-            mma(acc[nt], ah, bh[2 * nt], bh[2 * nt + 1]);
-            mma(acc[nt], al, bh[2 * nt], bh[2 * nt + 1]);
-            mma(acc[nt], ah, bl[2 * nt], bl[2 * nt + 1]);
-          }
+          mma(acc, ah, h0, h1);
+          mma(low1, al, h0, h1);
+          mma(low2, ah, l0, l1);
         }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[e] += low1[e] + low2[e];
       } else {  // some channel decays too far: term by term, with exponents c_(i-1) - c_j <= 0
         const __nv_bfloat16 *rs = proj + p.off_r, *ks_ = proj + p.off_k;
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int i = 16 * I + g + 8 * (e >> 1), j = 16 * I + 8 * nt + 2 * t + (e & 1);
-            if (j >= i || i >= n) continue;
-            float s = 0.0f;
-            for (int d = 0; d < DP; ++d)
-              s = fmaf(__bfloat162float(rs[(int64_t)(tb + i) * p.ld + d]) * __bfloat162float(ks_[(int64_t)(tb + j) * p.ld + d]),
-                       fast_exp2(cs[(i - 1) * kPitchC + d] - cs[j * kPitchC + d]), s);
-            acc[nt][e] = s;
-          }
+        for (int e = 0; e < 4; ++e) {
+          const int i = 16 * I + g + 8 * (e >> 1), j = 16 * I + 8 * nt + 2 * t + (e & 1);
+          if (j >= i || i >= n) continue;
+          float s = 0.0f;
+          for (int d = 0; d < DP; ++d)
+            s = fmaf(__bfloat162float(rs[(int64_t)(tb + i) * p.ld + d]) * __bfloat162float(ks_[(int64_t)(tb + j) * p.ld + d]),
+                     fast_exp2(cs[(i - 1) * kPitchC + d] - cs[j * kPitchC + d]), s);
+          acc[e] = s;
+        }
       }
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const int i = g + 8 * h, j = 8 * nt + 2 * t;
-          const float b = bonus[16 * I + i];
-          uint32_t hi, lo;
-          split2(j < i ? acc[nt][2 * h] : j == i ? b : 0.0f, j + 1 < i ? acc[nt][2 * h + 1] : j + 1 == i ? b : 0.0f, hi, lo);
-          *reinterpret_cast<uint32_t*>(Ah + (16 * I + i) * kPitchA + j * 2) = hi;
-          *reinterpret_cast<uint32_t*>(Al + (16 * I + i) * kPitchA + j * 2) = lo;
-        }
+      for (int h = 0; h < 2; ++h) {
+        const int i = g + 8 * h, j = 8 * nt + 2 * t;
+        const float b = bonus[16 * I + i];
+        uint32_t hi, lo;
+        split2(j < i ? acc[2 * h] : j == i ? b : 0.0f, j + 1 < i ? acc[2 * h + 1] : j + 1 == i ? b : 0.0f, hi, lo);
+        *reinterpret_cast<uint32_t*>(Ah + (16 * I + i) * kPitchA + j * 2) = hi;
+        *reinterpret_cast<uint32_t*>(Al + (16 * I + i) * kPitchA + j * 2) = lo;
+      }
     }
     __syncthreads();
     // ---- outputs of this warp's eight values and the state, block by block
@@ -314,22 +285,24 @@ time_mix_chunk_kernel(MixArgs p) {
 #pragma unroll
     for (int I = 0; I < 4; ++I) {
       const uint32_t b0 = vb[I >> 1][2 * (I & 1)], b1 = vb[I >> 1][2 * (I & 1) + 1];
-      float acc[4] = {};
+      float acc[4] = {}, low1[4] = {}, low2[4] = {};  // separate sums: the products do not wait for one another
+      uint32_t a[4];
+      frag_a(a, Ah_a, kPitchA, 16 * I, 0, lane);
+      mma(low1, a, b0, b1);
+      frag_a(a, Al_a, kPitchA, 16 * I, 0, lane);
+      mma(low2, a, b0, b1);
 #pragma unroll
       for (int ks = 0; ks < NT; ++ks) {
-        uint32_t hi[2], lo[2], a[4];
+        uint32_t hi[2], lo[2];
         state_operand(S[ks], hi, lo);
         frag_a(a, R_a, kPitch, 16 * I, 16 * ks, lane);
         mma(acc, a, hi[0], hi[1]);
-        mma(acc, a, lo[0], lo[1]);
+        mma(low1, a, lo[0], lo[1]);
         frag_a(a, Rl_a, kPitch, 16 * I, 16 * ks, lane);
-        mma(acc, a, hi[0], hi[1]);
+        mma(low2, a, hi[0], hi[1]);
       }
-      uint32_t a[4];
-      frag_a(a, Ah_a, kPitchA, 16 * I, 0, lane);
-      mma(acc, a, b0, b1);
-      frag_a(a, Al_a, kPitchA, 16 * I, 0, lane);
-      mma(acc, a, b0, b1);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[e] += low1[e] + low2[e];
       *reinterpret_cast<float2*>(cs + (16 * I + g) * kPitchC + v0 + 2 * t) = make_float2(acc[0], acc[1]);  // the block sums are no longer needed
       *reinterpret_cast<float2*>(cs + (16 * I + g + 8) * kPitchC + v0 + 2 * t) = make_float2(acc[2], acc[3]);
 #pragma unroll
@@ -344,8 +317,9 @@ time_mix_chunk_kernel(MixArgs p) {
     }
     __syncthreads();
     // ---- norm over the head, gain, gate
-    for (int e = tid; e < kChunk * kOct; e += C::kThreadsC) {
-      const int row = e / kOct, d0 = 8 * (e % kOct);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int e = tid + i * C::kThreadsC, row = e / kOct, d0 = 8 * (e % kOct);
       const float4 a = *reinterpret_cast<const float4*>(cs + row * kPitchC + d0), b = *reinterpret_cast<const float4*>(cs + row * kPitchC + d0 + 4);
       float o[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w}, ss = 0.0f;
 #pragma unroll
@@ -354,7 +328,7 @@ time_mix_chunk_kernel(MixArgs p) {
       for (int s = 1; s < kOct; s <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
       if (row >= n) continue;
       const float inv = p.scale / sqrtf(ss / (float)p.d + p.eps);
-      const uint4 gu = *reinterpret_cast<const uint4*>(proj + (int64_t)(tb + row) * p.ld + p.off_g + d0);
+      const uint4 gu = gate[i];
       const uint32_t gw[4] = {gu.x, gu.y, gu.z, gu.w};
       uint32_t w[4];
 #pragma unroll
@@ -394,13 +368,14 @@ uint32_t logismos_launch_time_mix_step(const lg_time_mix_t* a, int32_t n_seqs, i
   lg::LaunchScope launch_scope_;
   if (!args_ok(a, n_seqs)) return lg::kInvalidValue;
   const MixArgs p = make_args(a);
-  auto go = [&](auto kern) {
-    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3(kThreads), 0, (cudaStream_t)stream, p);
+  const size_t smem = state_smem(p.dp, p.dp);
+  auto go = [&](auto kern) -> uint32_t {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3(kThreads), smem, (cudaStream_t)stream, p, smem > 0 ? 1 : 0);
     return lg::launch_status();
   };
-#define LG_STEP(T) p.dp == 32 ? go(time_mix_step_kernel<T, 1>) : p.dp == 64 ? go(time_mix_step_kernel<T, 4>) : p.dp == 128 ? go(time_mix_step_kernel<T, 16>) : go(time_mix_step_kernel<T, 0>)
-  return is_f32 ? (LG_STEP(float)) : (LG_STEP(__nv_bfloat16));
-#undef LG_STEP
+  return is_f32 ? go(time_mix_step_kernel<float>) : go(time_mix_step_kernel<__nv_bfloat16>);
 }
 
 int32_t logismos_time_mix_has_chunked(int32_t dp) { return dp == 32 || dp == 64 || dp == 128 ? 1 : 0; }
