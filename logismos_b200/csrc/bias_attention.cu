@@ -39,17 +39,20 @@ unit_qk_store_kernel(QkArgs p) {
   struct alignas(E * sizeof(T)) Vec { T v[E]; };
   const uint32_t per_row = p.heads + 2 * p.n_kv, lane = threadIdx.x % LANES;
   const uint32_t total = p.rows * per_row, first = (blockIdx.x * kThreads + threadIdx.x) / LANES * ITEMS;
+  const int row0 = (int)(first / per_row), head0 = (int)(first % per_row);
   Vec x[ITEMS];
 #pragma unroll
   for (int k = 0; k < ITEMS; ++k) {
     if (first + k >= total) continue;
-    const int row = (int)((first + k) / per_row), h = (int)((first + k) % per_row);
+    const bool wrap = head0 + k >= (int)per_row;  // ITEMS <= per_row or ITEMS == 1: at most one row further
+    const int row = row0 + wrap, h = head0 + k - (wrap ? (int)per_row : 0);
     x[k] = *reinterpret_cast<const Vec*>(reinterpret_cast<const T*>(p.qkv) + (size_t)row * p.ld + h * HD + lane * E);
   }
 #pragma unroll
   for (int k = 0; k < ITEMS; ++k) {
     const bool in = first + k < total;
-    const int row = in ? (int)((first + k) / per_row) : 0, h = in ? (int)((first + k) % per_row) : 0;
+    const bool wrap = head0 + k >= (int)per_row;
+    const int row = in ? row0 + wrap : 0, h = in ? head0 + k - (wrap ? (int)per_row : 0) : 0;
     const bool is_v = h >= p.heads + p.n_kv;
     float f[E], ss = 0.0f;
 #pragma unroll
@@ -166,7 +169,7 @@ uint32_t logismos_launch_unit_qk_store(void* qkv, int32_t ld, void* k_pool, void
     return lg::launch_status();
   };
 #define LG_UNIT(T, HD)                                                                             \
-  (items < 20000 ? go(unit_qk_store_kernel<T, HD, 1>, kThreads / UnitGeometry<T, HD>::LANES)       \
+  (items < 20000 || n_heads + 2 * n_kv_heads < 4 ? go(unit_qk_store_kernel<T, HD, 1>, kThreads / UnitGeometry<T, HD>::LANES)       \
                  : go(unit_qk_store_kernel<T, HD, 4>, kThreads / UnitGeometry<T, HD>::LANES * 4))
   if (is_f32) return head_dim == 64 ? LG_UNIT(float, 64) : head_dim == 128 ? LG_UNIT(float, 128) : LG_UNIT(float, 256);
   return head_dim == 64 ? LG_UNIT(__nv_bfloat16, 64) : head_dim == 128 ? LG_UNIT(__nv_bfloat16, 128) : LG_UNIT(__nv_bfloat16, 256);
