@@ -139,11 +139,11 @@ LG_DEVINL void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t 
   const uint32_t b[2] = {b0, b1};
   mma_bf16_16816(d, a, b, d);
 }
-// rows row0 .. + 63 of a [rows][width] bf16 block at src (row stride ld elements) into a tile; rows >= n are zero
+// 64 rows of a [rows][width] bf16 block at src (row stride ld elements; width a power of two) into a tile; rows >= n are zero
 LG_DEVINL void stage_tile(uint8_t* tile, int pitch, const __nv_bfloat16* src, int64_t ld, int n, int width) {
-  const int pieces = width >> 3;
+  const int pieces = width >> 3, lg = 31 - __clz(pieces);
   for (int e = threadIdx.x; e < kChunk * pieces; e += blockDim.x) {
-    const int row = e / pieces, piece = e % pieces;
+    const int row = e >> lg, piece = e & (pieces - 1);
     uint8_t* dst = tile + row * pitch + piece * 16;
     if (row < n) cp_async16(smem_u32(dst), src + row * ld + piece * 8);
     else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);

@@ -194,7 +194,7 @@ uint32_t launch_conv(const SsdArgs& p, const int* seq_ids, int row0, int rows, c
 // CTA = (head, sequence), VP / 8 warps; shared memory as laid out by ssd_chunk_smem
 constexpr int kPitchP = kChunk * 2 + 16;
 inline size_t ssd_chunk_smem(int np, int vp) {
-  return (size_t)kChunk * (2 * (2 * (2 * np + 16) + 2 * vp + 16) + 2 * kPitchP) + 2 * kChunk * 4;
+  return (size_t)kChunk * (2 * (2 * (2 * np + 16) + 2 * vp + 16) + 2 * kPitchP) + 4 * kChunk * 4;
 }
 template <int NP>
 __global__ void __launch_bounds__(512)
@@ -209,7 +209,7 @@ ssd_chunk_kernel(SsdArgs p) {
   if (t1 <= t0) return;
   const int group = head / (p.heads / p.groups), inner = p.heads * vp;
   uint8_t *Bt = smem, *Ct = Bt + 2 * kChunk * kPitchN, *Xt = Ct + 2 * kChunk * kPitchN, *Ph = Xt + 2 * kChunk * pitch_v, *Pl = Ph + kChunk * kPitchP;
-  float *cum = reinterpret_cast<float*>(Pl + kChunk * kPitchP), *dts = cum + kChunk;
+  float *cums = reinterpret_cast<float*>(Pl + kChunk * kPitchP), *dtss = cums + 2 * kChunk;
   const __nv_bfloat16* xbc = reinterpret_cast<const __nv_bfloat16*>(p.xbc);
   const __nv_bfloat16 *xs = xbc + head * vp, *bs = xbc + inner + group * NP, *cs = bs + p.groups * NP;
   __nv_bfloat16* ys = reinterpret_cast<__nv_bfloat16*>(p.y) + head * vp;
@@ -234,32 +234,34 @@ ssd_chunk_kernel(SsdArgs p) {
   };
   float dt_raw[2] = {0.f, 0.f};
   auto fetch_dt = [&](int tb) {
-    if (warp != 0) return;
 #pragma unroll
     for (int i = 0; i < 2; ++i) dt_raw[i] = tb + lane + 32 * i < t1 ? p.dt[(size_t)(tb + lane + 32 * i) * p.ld_dt + head] : 0.0f;
   };
-  stage(t0, 0);
-  fetch_dt(t0);
-  int buf = 0;
-  for (int tb = t0; tb < t1; tb += kChunk, buf ^= 1) {
+  // step sizes and log2-decays of a chunk summed up by one warp; tokens past the end take no step
+  auto sum_decays = [&](int tb, int to) {
     const int n = min(kChunk, t1 - tb);
-    if (warp == 0) {  // step sizes and log2-decays summed up; tokens past the end take no step
-      const float d0 = lane < n ? softplus_f(dt_raw[0] + bias) : 0.0f, d1 = lane + 32 < n ? softplus_f(dt_raw[1] + bias) : 0.0f;
-      float c0 = -a2 * d0, c1 = -a2 * d1;
+    const float d0 = lane < n ? softplus_f(dt_raw[0] + bias) : 0.0f, d1 = lane + 32 < n ? softplus_f(dt_raw[1] + bias) : 0.0f;
+    float c0 = -a2 * d0, c1 = -a2 * d1;
 #pragma unroll
-      for (int d = 1; d < 32; d <<= 1) {
-        const float u0 = __shfl_up_sync(0xffffffffu, c0, d), u1 = __shfl_up_sync(0xffffffffu, c1, d);
-        if (lane >= d) { c0 += u0; c1 += u1; }
-      }
-      c1 += __shfl_sync(0xffffffffu, c0, 31);
-      cum[lane] = c0; cum[lane + 32] = c1;
-      dts[lane] = d0; dts[lane + 32] = d1;
+    for (int d = 1; d < 32; d <<= 1) {
+      const float u0 = __shfl_up_sync(0xffffffffu, c0, d), u1 = __shfl_up_sync(0xffffffffu, c1, d);
+      if (lane >= d) { c0 += u0; c1 += u1; }
     }
+    c1 += __shfl_sync(0xffffffffu, c0, 31);
+    cums[to * kChunk + lane] = c0; cums[to * kChunk + lane + 32] = c1;
+    dtss[to * kChunk + lane] = d0; dtss[to * kChunk + lane + 32] = d1;
+  };
+  stage(t0, 0);
+  if (warp == 0) { fetch_dt(t0); sum_decays(t0, 0); }
+  int buf = 0, turn = 0;  // the warp whose turn it is prepares the next chunk's decays
+  for (int tb = t0; tb < t1; tb += kChunk, buf ^= 1, turn = turn + 1 < n_warps ? turn + 1 : 0) {
+    const int n = min(kChunk, t1 - tb);
+    const float *cum = cums + buf * kChunk, *dts = dtss + buf * kChunk;
     cp_async_wait<0>();
     __syncthreads();
     if (tb + kChunk < t1) {
       stage(tb + kChunk, buf ^ 1);
-      fetch_dt(tb + kChunk);
+      if (warp == turn) fetch_dt(tb + kChunk);
     }
     const uint32_t B_a = smem_u32(Bt + buf * kChunk * kPitchN), C_a = smem_u32(Ct + buf * kChunk * kPitchN), X_a = smem_u32(Xt + buf * kChunk * pitch_v);
     // ---- P: sixteen by sixteen blocks on and below the diagonal, dealt to the warps
@@ -348,10 +350,11 @@ ssd_chunk_kernel(SsdArgs p) {
         mma(S[m], a, lo[0], lo[1]);
       }
     }
+    if (warp == turn && tb + kChunk < t1) sum_decays(tb + kChunk, buf ^ 1);
     __syncthreads();
-    const int pieces_v = vp >> 3;
+    const int pieces_v = vp >> 3, lg_v = 31 - __clz(pieces_v);
     for (int e = tid; e < n * pieces_v; e += blockDim.x) {
-      const int row = e / pieces_v, piece = e % pieces_v;
+      const int row = e >> lg_v, piece = e & (pieces_v - 1);
       *reinterpret_cast<uint4*>(ys + (int64_t)(tb + row) * p.ld_y + piece * 8) =
           *reinterpret_cast<const uint4*>(Xt + buf * kChunk * pitch_v + row * pitch_v + piece * 16);
     }

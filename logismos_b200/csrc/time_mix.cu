@@ -123,8 +123,8 @@ time_mix_step_kernel(MixArgs p, int in_smem) {
 
 template <int DP> struct ChunkCfg {
   static constexpr int kThreadsC = 4 * DP, kPitch = DP * 2 + 16, kTile = kChunk * kPitch, kPitchC = DP + 8, kPitchA = 16 * 2 + 16;
-  // r, k, v twice; remainders of R and K; block sums (later the outputs) fp32; coefficients, two parts; totals, bonus
-  static constexpr size_t kSmem = 8 * (size_t)kTile + kChunk * kPitchC * 4 + 2 * kChunk * kPitchA + 4 * DP * 4 + kChunk * 4;
+  // r, k, v twice; remainders of R and K; block sums (later the outputs) fp32; coefficients, two parts; totals, bonus, u, gain
+  static constexpr size_t kSmem = 8 * (size_t)kTile + kChunk * kPitchC * 4 + 2 * kChunk * kPitchA + 4 * DP * 4 + kChunk * 4 + 2 * DP * 4;
 };
 constexpr float kMaxSpan = 100.0f;  // log2 of the decay over a block up to which exp(-T) is taken
 
@@ -138,7 +138,7 @@ time_mix_chunk_kernel(MixArgs p) {
   uint8_t *Rt = smem, *Kt = Rt + 2 * C::kTile, *Vt = Kt + 2 * C::kTile, *Rl = Vt + 2 * C::kTile, *Kl = Rl + C::kTile;
   float* cs = reinterpret_cast<float*>(Kl + C::kTile);
   uint8_t *Ah = reinterpret_cast<uint8_t*>(cs + kChunk * kPitchC), *Al = Ah + kChunk * kPitchA;
-  float *tot = reinterpret_cast<float*>(Al + kChunk * kPitchA), *bonus = tot + 4 * DP;
+  float *tot = reinterpret_cast<float*>(Al + kChunk * kPitchA), *bonus = tot + 4 * DP, *us = bonus + kChunk, *gains = us + DP;
   const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, t = lane & 3, v0 = 8 * warp, h0 = head * DP;
   const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
@@ -172,6 +172,7 @@ time_mix_chunk_kernel(MixArgs p) {
   };
   stage(t0, 0);
   fetch_z(t0);
+  if (tid < DP) { us[tid] = p.u[h0 + tid]; gains[tid] = p.gain[h0 + tid]; }
   int buf = 0;
   for (int tb = t0; tb < t1; tb += kChunk, buf ^= 1) {
     const int n = min(kChunk, t1 - tb);
@@ -179,7 +180,7 @@ time_mix_chunk_kernel(MixArgs p) {
       float c = 0.0f;
 #pragma unroll
       for (int i = 0; i < 16; ++i) {  // past the end: no decay
-        c -= expf(z[i]) * 1.4426950408889634f;
+        c = fmaf(fast_exp2(z[i] * 1.4426950408889634f), -1.4426950408889634f, c);
         cs[(16 * zb + i) * kPitchC + zc] = c;
       }
       tot[zb * DP + zc] = c;
@@ -204,7 +205,7 @@ time_mix_chunk_kernel(MixArgs p) {
         const float2 r = unpack_bf16x2(rw[q]), k = unpack_bf16x2(kw[q]);
         const float2 c = *reinterpret_cast<const float2*>(cs + row * kPitchC + d), tt = *reinterpret_cast<const float2*>(tot + (row >> 4) * DP + d);
         const float2 cp = (row & 15) ? *reinterpret_cast<const float2*>(cs + (row - 1) * kPitchC + d) : make_float2(0.f, 0.f);
-        const float2 u = __ldg(reinterpret_cast<const float2*>(p.u + h0 + d));
+        const float2 u = *reinterpret_cast<const float2*>(us + d);
         dot = fmaf(r.x * u.x, k.x, fmaf(r.y * u.y, k.y, dot));
         split2(r.x * fast_exp2(cp.x), r.y * fast_exp2(cp.y), rh[q], rl[q]);
         split2(k.x * fast_exp2(tt.x - c.x), k.y * fast_exp2(tt.y - c.y), kh[q], kl[q]);
@@ -333,7 +334,7 @@ time_mix_chunk_kernel(MixArgs p) {
       uint32_t w[4];
 #pragma unroll
       for (int q = 0; q < 4; ++q) {
-        const float2 gg = unpack_bf16x2(gw[q]), gn = __ldg(reinterpret_cast<const float2*>(p.gain + h0 + d0 + 2 * q));
+        const float2 gg = unpack_bf16x2(gw[q]), gn = *reinterpret_cast<const float2*>(gains + d0 + 2 * q);
         w[q] = pack_bf16x2(o[2 * q] * inv * gn.x * __fdividef(gg.x, 1.0f + __expf(-gg.x)), o[2 * q + 1] * inv * gn.y * __fdividef(gg.y, 1.0f + __expf(-gg.y)));
       }
       *reinterpret_cast<uint4*>(out + (int64_t)(tb + row) * p.ld_out + d0) = make_uint4(w[0], w[1], w[2], w[3]);
