@@ -323,7 +323,7 @@ int32_t lg_latent_device_status(void* model);
  * Decoder step over a stack of state-space and parallel (attention beside time mixing) layers (Katadra), post-norm.
  * No reference counterpart; the contract is that of lg_decoder_step. Weights are bf16, dense.
  *   x = embed[id];  x += norm1(mixer(x));  with a feed-forward x += norm2(W_down max(W_up x, 0)^2);  logits = head norm(x)
- *   norms: layer norms with weight and bias
+ *   norms: layer norms (gain and offset)
  *   LG_MIXER_SSD: [z | x | B | C | dt] = W_in h, convolution, scalar-decay recurrence, gate, norm in parts, W_o
  *     (lg_ssd_t, logismos_launch_gated_group_norm)
  *   LG_MIXER_PARALLEL: left_scale * attention(h) + right_scale * time_mixing(h); attention without positions, unit
