@@ -284,7 +284,7 @@ def kernel_table(z, peaks, T=4096, seqs=64, ctx=8192):
     gemm("prefill", "latent projections", T, Q + R, H, 3, like="qkv GEMM")
     raws, pool = [f32(T, Q + R) for _ in range(copies(T * (Q + R) * 4))], bf(seqs * (ctx // 16 + 1), 16, R)
     cq, gq, gc, slot64 = bf(T, Q), torch.ones(Q, device=dev), torch.ones(R, device=dev), torch.randperm(T, device=dev)
-    add("prefill", "latent_norm_store", [lambda s, y=y: lib.logismos_launch_latent_norm_store(P(y), Q + R, P(gq), P(gc), P(cq), P(pool), P(slot64), T, Q, Q, R, R, 1e-6, pool.shape[0] * 16, 0, 0, P(st), s)
+    add("prefill", "latent_norm_store", [lambda s, y=y: lib.logismos_launch_latent_norm_store(P(y), Q + R, P(gq), P(gc), P(cq), P(pool), P(slot64), T, Q, Q, R, R, 1e-6, pool.shape[0] * 16, 0, 0, P(None), P(st), s)
                                              for y in raws], 6.0 * T * (Q + R), like="rms_norm")
     gemm("prefill", "queries", T, HD, Q, 0, like="qkv GEMM")
     nblk = 1024 // 16
@@ -296,7 +296,7 @@ def kernel_table(z, peaks, T=4096, seqs=64, ctx=8192):
         4.0 * T * R, like="transpose_v")
     gemm("prefill", "keys (values: the transposed product)", tp, HD, R, 0, like="qkv GEMM")
     qs, ks, vts, att = bf(T, HD), bf(tp, HD), bf(HD, tp), bf(T, HD)
-    add("prefill", "attention", [lambda s: lib.logismos_launch_varlen_attention_kv_tc_bf16(P(qs), HD, P(cu), P(kv_lens), P(start), P(ks), P(vts), tp, P(att), HD, T, nq, 1024, heads, heads, D, 0.09, P(st), s)] * 3,
+    add("prefill", "attention", [lambda s: lib.logismos_launch_varlen_attention_kv_tc_bf16(P(qs), HD, P(cu), P(kv_lens), P(start), P(ks), P(vts), tp, P(att), HD, T, nq, 1024, heads, heads, D, 0.09, P(None), 0, P(st), s)] * 3,
         2.0 * T * HD * 4, 4.0 * HD * nq * 1024 * 1025 / 2, like="attention")
     gemm("prefill", "gated feed-forward", T, 2 * F, H, 4, like="gate/up GEMM")
     gemm("prefill", "output projection [W_o | W_down]", T, H, HD + F, 1, like="down GEMM")
@@ -343,7 +343,7 @@ def kernel_table(z, peaks, T=4096, seqs=64, ctx=8192):
     off, total = ops.build_decode_chunks(cl, chunk)
     off = off.to(dev)
     scr = torch.empty(lib.logismos_latent_decode_scratch_bytes(total, heads, R), dtype=torch.uint8, device=dev)
-    add("decode", "latent_decode + merge (ctx %d)" % ctx, [lambda s: lib.logismos_launch_latent_decode_bf16(P(qd), P(pool), P(tab), P(cg), P(off), P(od), P(scr), seqs, total, chunk, nb, seqs * nb, heads, R, 0.05, P(st), s)] * 3,
+    add("decode", "latent_decode + merge (ctx %d)" % ctx, [lambda s: lib.logismos_launch_latent_decode_bf16(P(qd), P(pool), P(tab), P(cg), P(off), P(od), P(scr), seqs, total, chunk, nb, seqs * nb, heads, R, 0.05, P(None), 0, P(st), s)] * 3,
         seqs * (ctx * R * 2.0 + heads * R * 4.0), 4.0 * seqs * ctx * heads * R, like="paged_decode")
     del pool
     nkv = heads // 4

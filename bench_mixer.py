@@ -184,28 +184,6 @@ def measure(sizes, iters, peaks, seqs=(8, 64), ctx=2048, prefill=(4, 1024)):
 
 # ---- kernels -------------------------------------------------------------------------------------
 
-vp, i32, f32 = C.c_void_p, C.c_int32, C.c_float
-
-
-class TimeMixArgs(C.Structure):
-    _fields_ = [("proj", vp)] + [(n, i32) for n in ("ld", "off_r", "off_k", "off_v", "off_g")] + [("z", vp), ("ld_z", i32), ("low", vp), ("ld_low", i32),
-               ("w2", vp), ("ld_w2", i32), ("rank", i32), ("w0", vp), ("u", vp), ("gain", vp), ("state", vp), ("state_slots", vp), ("fresh", vp), ("cu", vp),
-               ("out", vp), ("ld_out", i32), ("heads", i32), ("d", i32), ("dp", i32), ("scale", f32), ("eps", f32)]
-
-
-class SsdArgs(C.Structure):
-    _fields_ = [("proj", vp), ("ld", i32), ("dt", vp), ("ld_dt", i32), ("conv_w", vp), ("conv_b", vp), ("conv_state", vp), ("taps", i32), ("dt_bias", vp),
-                ("log_a", vp), ("skip", vp), ("state", vp), ("state_slots", vp), ("fresh", vp), ("phase", vp), ("cu", vp), ("y", vp)] + [
-               (n, i32) for n in ("ld_y", "heads", "groups", "np", "vp")] + [("xbc", vp), ("ld_xbc", i32)]
-
-
-class Groups(C.Structure):
-    _fields_ = [("n_groups", i32), ("end", i32 * 8), ("n_main", i32), ("tail", vp), ("ld_tail", i32), ("tail_cap", f32), ("tail_parts", vp)]
-
-
-class ScoreBias(C.Structure):
-    _fields_ = [("scale", f32), ("cap", f32), ("bias", vp), ("far", i32), ("max_abs_bias", f32), ("max_abs_qk", f32), ("gate", vp), ("ld_gate", i32), ("gate_scale", f32)]
-
 
 def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
     """Every kernel of the Katadra decoder at one size, and the like kernel of the hybrid decoder, each against its
@@ -213,7 +191,8 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
     rotate over copies that exceed L2 together."""
     import torch
     from logismos_b200 import ops
-    from logismos_b200._lib import lib
+    from logismos_b200._lib import i32, lib
+    from logismos_b200.structs import Groups, ScoreBias, Ssd, TimeMix
     dev = "cuda"
     P = lambda t: C.c_void_p(t.data_ptr() if t is not None else 0)
     A = lambda t: 0 if t is None else t.data_ptr()
@@ -283,13 +262,13 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
     def ssd_args(m, seqs, xbc, proj, dt, y, state, cstate, slots, cu):
         q = [torch.zeros(z["sh"], device=dev), torch.zeros(z["sh"], device=dev), torch.ones(z["sh"], device=dev), u8(seqs), u8(seqs)]
         keep.append(q)
-        return SsdArgs(A(proj), proj.shape[1], A(dt), z["sh"], A(w4), A(bias_c), A(cstate), 4, A(q[0]), A(q[1]), A(q[2]), A(state), A(slots), A(q[3]), A(q[4]), A(cu), A(y),
+        return Ssd(A(proj), proj.shape[1], A(dt), z["sh"], A(w4), A(bias_c), A(cstate), 4, A(q[0]), A(q[1]), A(q[2]), A(state), A(slots), A(q[3]), A(q[4]), A(cu), A(y),
                        inner, z["sh"], z["groups"], z["state"], z["sv"], A(xbc), ch)
 
     def tm_args(proj, zz, low, w2, state, seqs, slots, cu, out):
         q = [torch.full((TD,), -2.0, device=dev), torch.full((TD,), 0.3, device=dev), u8(seqs)]
         keep.append(q)
-        return TimeMixArgs(A(proj), proj.shape[1], 0, TD, 2 * TD, 3 * TD, A(zz), TD, A(low), R, A(w2), 2 * R, R, A(q[0]), A(q[1]), A(gain_t), A(state), A(slots), A(q[2]), A(cu),
+        return TimeMix(A(proj), proj.shape[1], 0, TD, 2 * TD, 3 * TD, A(zz), TD, A(low), R, A(w2), 2 * R, R, A(q[0]), A(q[1]), A(gain_t), A(state), A(slots), A(q[2]), A(cu),
                            A(out), TD, z["th"], z["td"], z["td"], 1.0, 1e-6)
 
     # ---- prefill of T tokens in sequences of 1024

@@ -147,6 +147,7 @@ typedef struct lg_linear_groups {
   int32_t ld_tail;
   float tail_cap;
   void* tail_parts;
+  const void* bias;             /* f32 [n_main], added to the main columns (NULL: none) */
 } lg_linear_groups_t;
 uint32_t logismos_launch_linear_groups_tc_bf16(const void* a_bf16, const void* w_bf16, void* out, int32_t m, int32_t n,
                                                int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
@@ -157,6 +158,27 @@ uint32_t logismos_launch_linear_groups_small_bf16(const void* a_bf16, const void
 uint32_t logismos_launch_linear_groups_f32(const void* a_f32, const void* w_bf16, void* out_f32, int32_t m, int32_t n,
                                            int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
                                            void* stream);
+/* A stack of matrices, one per group of rows: rows offsets[g] .. offsets[g + 1] of the output are rows of the input
+ * times w[g] (w bf16 [n_groups][n][k]). offsets i32 [n_groups + 1] on the device. row_idx (NULL: none) gives the input row
+ * of every output row. max_group_rows bounds the rows of one group (host value). Epilogues LG_EPI_BF16 and LG_EPI_SWIGLU
+ * (small), LG_EPI_F32 and LG_EPI_GLU_CLAMP (fp32). The first streams the weights of the groups that have rows. */
+uint32_t logismos_launch_linear_experts_small_bf16(const void* a_bf16, const void* w_bf16, void* out, const void* offsets_i32,
+                                                   const void* row_idx_i32, int32_t n_groups, int32_t max_group_rows,
+                                                   int32_t expected_group_rows, int32_t n, int32_t k, int32_t lda, int32_t ldc,
+                                                   int32_t epilogue, void* stream);
+uint32_t logismos_launch_linear_experts_f32(const void* a_f32, const void* w_bf16, void* out_f32, const void* offsets_i32,
+                                            const void* row_idx_i32, int32_t n_groups, int32_t max_group_rows, int32_t n,
+                                            int32_t k, int32_t lda, int32_t ldc, int32_t epilogue, float p0, float p1, float p2,
+                                            void* stream);
+/* The same on the tcgen05 tiles, with the row tiles of 128 listed by logismos_launch_moe_place: tiles i32 [.][4] = group,
+ * first output row, last output row + 1, and -1 - input row for tiles that read a_direct; the others read the rows of a
+ * that they write (with a_direct NULL: all do). n_tiles i32 [1]; both on the device. max_tiles bounds their number.
+ * a [a_rows, lda], a_direct [direct_rows, lda]. */
+uint32_t logismos_launch_linear_experts_tc_bf16(const void* a_bf16, int32_t a_rows, const void* a_direct_bf16,
+                                                int32_t direct_rows, const void* w_bf16, void* out_bf16, const void* tiles_i32,
+                                                const void* n_tiles_i32, int32_t max_tiles, int32_t n_groups, int32_t n,
+                                                int32_t k, int32_t lda, int32_t ldc, int32_t epilogue, void* status_i32,
+                                                void* stream);
 /* The batched contract with fp32 activations and outputs, true fp32 products and sums over the bf16
  * weights (which fp32 represents exactly). Epilogues LG_EPI_F32, LG_EPI_RESID_F32, LG_EPI_GLU_CLAMP, LG_EPI_RELU2 (fp32
  * out); k % 16 == 0, lda % 4 == 0, strides of a and w multiples of 4. */
@@ -271,12 +293,14 @@ uint32_t logismos_launch_paged_prefix_attention_turbo3_bf16(
  * kv_lens[s] keys at rows / columns kv_start[s] .. (kv_start a multiple of 8; what lies between sequences
  * must be finite); query i sees its first kv_lens[s] - new + i + 1 keys. Scores are scaled by `scale` (> 0).
  * out bf16, rows out_row_stride apart. head_dim 64, 128 or 256; n_kv_rows % 8 == 0. One launch of the
- * tcgen05 kernel above. status as there. */
+ * tcgen05 kernel above. status as there. gate (f32 [n_q_tokens, ld_gate], NULL: none): head h of a row is multiplied by
+ * the sigmoid of its column h. */
 uint32_t logismos_launch_varlen_attention_kv_tc_bf16(
     const void* q_bf16, int32_t q_row_stride, const void* cu_seqlens_q_i32, const void* kv_lens_i32,
     const void* kv_start_i32, const void* k_bf16, const void* v_t_bf16, int32_t n_kv_rows, void* out_bf16,
     int32_t out_row_stride, int32_t n_q_tokens, int32_t n_seqs, int32_t max_q_len, int32_t n_heads,
-    int32_t n_kv_heads, int32_t head_dim, float scale, void* status_i32, void* stream);
+    int32_t n_kv_heads, int32_t head_dim, float scale, const void* gate_f32, int32_t ld_gate, void* status_i32,
+    void* stream);
 
 /* mean_pool_masked -> l2_normalize -> linear_t(head) -> l2_normalize (cpu_f32 mod.rs:553-591 as
  * composed by StellaModel::encode_raw, crates/embed/src/stella.rs:231-246), mask all ones.
@@ -588,13 +612,23 @@ uint32_t logismos_launch_depth_mix_conv_decode(const void* hist_f32, int64_t his
  * q_width .. q_width + c_width; both are RMS-normed (means over the first q_n and c_n columns) with their
  * gains; the first goes to q_latent [rows, q_width], the second to the pool at slot_mapping[row] (a slot
  * outside the pool is skipped and raises status to 1). is_f32 selects the type of both. zero_raw != 0 leaves
- * raw zeroed, ready to be accumulated into again. */
+ * raw zeroed, ready to be accumulated into again.
+ * rotary (NULL: none): the key/value latent takes the first `at` of the c_width columns (a multiple of 4, c_n of them not
+ * padding), the next dims columns are one rotated key part; raw columns q_width + c_width .. + n_gate go to gate f32
+ * [rows, ld_gate] as they are. */
+typedef struct lg_latent_rotary {
+  const void* table;            /* f32 [positions][dims / 2][2] */
+  const void* positions;        /* i32 [rows] */
+  int32_t at, dims;
+  void* gate;
+  int32_t n_gate, ld_gate;
+} lg_latent_rotary_t;
 uint32_t logismos_launch_latent_norm_store(void* raw_f32, int32_t ld, const void* gain_q_f32,
                                            const void* gain_c_f32, void* q_latent, void* pool,
                                            const void* slot_mapping_i64, int32_t rows, int32_t q_width,
                                            int32_t q_n, int32_t c_width, int32_t c_n, float eps,
                                            int64_t n_pool_slots, int32_t is_f32, int32_t zero_raw,
-                                           void* status_i32, void* stream);
+                                           const lg_latent_rotary_t* rotary, void* status_i32, void* stream);
 /* The cached rows of whole sequences made contiguous: out bf16 [logismos_latent_gather_rows(total, n_seqs),
  * width], sequence s at kv_start[s] (written, a multiple of 8), gaps zeroed. */
 int32_t logismos_latent_gather_rows(int32_t total_kv_tokens, int32_t n_seqs);
@@ -608,7 +642,8 @@ uint32_t logismos_launch_latent_gather_bf16(const void* pool, const void* block_
  * (logismos_pick_latent_chunk, whose choice leaves at most logismos_latent_max_chunks(rows) chunks). scratch:
  * logismos_latent_decode_scratch_bytes(total_chunks, heads, rank). A second launch merges split contexts. The
  * index arrays, and every cached row but the last of each context, must not be written by work still in
- * flight on the stream (they may be read ahead of the dependency wait). */
+ * flight on the stream (they may be read ahead of the dependency wait). gate (f32 [rows, ld_gate], NULL: none): head h of
+ * a row is multiplied by the sigmoid of its column h. */
 int32_t logismos_pick_latent_chunk(const int32_t* host_context_lens, int32_t n_seqs, int32_t heads);
 int32_t logismos_latent_max_chunks(int32_t max_rows);
 size_t logismos_latent_decode_scratch_bytes(int32_t total_chunks, int32_t heads, int32_t rank);
@@ -616,14 +651,14 @@ uint32_t logismos_launch_latent_decode_bf16(const void* q_bf16, const void* pool
                                             const void* context_lens_i32, const void* chunk_offsets_i32,
                                             void* out_bf16, void* scratch, int32_t rows, int32_t total_chunks,
                                             int32_t chunk_tokens, int32_t max_blocks, int32_t n_pool_blocks,
-                                            int32_t heads, int32_t rank, float scale, void* status_i32,
-                                            void* stream);
+                                            int32_t heads, int32_t rank, float scale, const void* gate_f32,
+                                            int32_t ld_gate, void* status_i32, void* stream);
 /* The fp32 form for any rows of a step: row t of sequence seq_ids[t] sees keys 0 .. positions[t]. */
 uint32_t logismos_launch_latent_attention_f32(const void* q_f32, const void* pool_f32, const void* block_tables_i32,
                                               const void* seq_ids_i32, const void* positions_i32, void* out_f32,
                                               int32_t rows, int32_t max_blocks, int32_t n_pool_blocks,
-                                              int32_t heads, int32_t rank, float scale, void* status_i32,
-                                              void* stream);
+                                              int32_t heads, int32_t rank, float scale, const void* gate_f32,
+                                              int32_t ld_gate, void* status_i32, void* stream);
 
 /* ====================================================================================
  * Sampling chain on the device: the logit processors and the multinomial sampler of
@@ -710,12 +745,15 @@ uint32_t logismos_launch_token_shift(const void* x_f32, void* h, int32_t out_f32
                                      const void* phase_u8, const void* seq_ids_i32, const void* cu_seqlens_i32,
                                      int32_t rows, int32_t ld, void* stream);
 
-/* Time mixing with a data-dependent decay per key channel, heads padded to dp = 32, 64, 128 or 256 with zeros:
- *   o_t = (S + diag(u) k_t v_t^T)^T r_t;  S <- diag(exp(-exp(z_t))) S + k_t v_t^T
- *   out = o / rms(o) * gain * silu(g) * scale          (rms over the d true channels)
- * proj holds r, k, v, g of head h at columns off_* + h * dp. z f32 [rows, ld_z] or, when NULL, z = W2 low + w0 with
+/* Linear attention with a data-dependent decay per key channel; key heads padded to dp, value heads to vp, each 32, 64,
+ * 128 or 256, with zeros:
+ *   LG_DECAY_TIME_MIX  o_t = (S + diag(u) k_t v_t^T)^T r_t;  S <- diag(exp(-exp(z_t))) S + k_t v_t^T     (vp = dp)
+ *   LG_DECAY_GATED     S <- diag(sigmoid(z_t)^(1 / tau)) S + k_t v_t^T;  o_t = q_scale S^T r_t
+ *   out = o / rms(o) * gain * silu(g) * scale          (rms over the d true value channels)
+ * proj holds r, k of head h at columns off_* + h * dp, v, g at off_* + h * vp. z f32 [rows, ld_z] or, when NULL, z = W2 low + w0 with
  * low f32 [rows, ld_low] and w2 bf16 [heads * dp, ld_w2] (rank columns, a multiple of 32). Sequence i owns rows
- * cu[i] .. cu[i + 1] and state slot state_slots[i] of state f32 [slots][heads][dp][dp]; fresh[i]: it starts here. */
+ * cu[i] .. cu[i + 1] and state slot state_slots[i] of state f32 [slots][heads][dp][vp]; fresh[i]: it starts here. */
+enum { LG_DECAY_TIME_MIX = 0, LG_DECAY_GATED = 1 };
 typedef struct lg_time_mix {
   const void* proj;
   int32_t ld, off_r, off_k, off_v, off_g;
@@ -725,17 +763,19 @@ typedef struct lg_time_mix {
   int32_t ld_low;
   const void* w2;
   int32_t ld_w2, rank;
-  const void *w0, *u, *gain;    /* f32 [heads * dp] */
+  const void *w0, *u, *gain;    /* f32 [heads * dp], u only for time mixing; gain [heads * vp] */
   void* state;
   const void *state_slots, *fresh, *cu;
   void* out;
   int32_t ld_out, heads, d, dp;
   float scale, eps;
+  int32_t mode, vp;             /* vp 0: dp */
+  float tau, q_scale;
 } lg_time_mix_t;
 /* Token by token: decode steps, fp32, any dp. */
 uint32_t logismos_launch_time_mix_step(const lg_time_mix_t* args, int32_t n_seqs, int32_t is_f32, void* stream);
-/* Prompts, 64 tokens at a time on the tensor cores: bf16 activations, dp <= 128, z given. */
-int32_t logismos_time_mix_has_chunked(int32_t dp);
+/* Prompts, 64 tokens at a time on the tensor cores: bf16 activations, dp and vp <= 128, z given. */
+int32_t logismos_time_mix_has_chunked(int32_t dp, int32_t vp);
 uint32_t logismos_launch_time_mix_chunked_bf16(const lg_time_mix_t* args, int32_t n_seqs, void* stream);
 
 /* State-space mixer with a scalar decay per head; np and vp are powers of two in 16 .. 256 with zero padding:
@@ -820,6 +860,107 @@ uint32_t logismos_launch_bias_attention_f32(const void* q_f32, int32_t ld_q, con
                                             void* out_f32, int32_t ld_out, int32_t rows, int32_t max_blocks,
                                             int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
                                             const lg_score_bias_t* score, void* status_i32, void* stream);
+
+/* ---- norms without statistics, rotary positions, windows, mixtures of experts ---------------------------------- */
+
+/* tanh(alpha x) w + b, w and b f32 [ld] with zeros in the padding. */
+typedef struct lg_tanh_norm {
+  float alpha;
+  const void *w, *b;
+} lg_tanh_norm_t;
+/* What a mixture of experts returns, rows of the experts still to be summed: sum over the token's n_pairs pairs i of
+ * weights[i] (1 from top on) * rows[pair_row[i]], plus identity[token] times the row of h before this call. pair_row i32
+ * [tokens, n_pairs] (negative: an identity expert). counts i32 [n_counts] are cleared. */
+typedef struct lg_mixture_out {
+  const void* rows;             /* activation format [., ld] */
+  const void *pair_row, *weights, *identity;   /* weights f32 [tokens, top], identity f32 [tokens] */
+  int32_t n_pairs, top;
+  void* counts;
+  int32_t n_counts;
+} lg_mixture_out_t;
+/* x += post(y) (y f32 [rows, ld], with zero_y cleared once read, or the sum `mixture`; post NULL: x stays), then
+ * h = next(x) in the activation format (next NULL: none). row_idx selects rows of x (then post is NULL). */
+uint32_t logismos_launch_tanh_norm(void* y_f32, int32_t zero_y, const lg_mixture_out_t* mixture, const void* row_idx_i32,
+                                   int32_t n_src_rows, void* x_f32, const lg_tanh_norm_t* post, void* h,
+                                   const lg_tanh_norm_t* next, int32_t out_f32, int32_t rows, int32_t ld, void* status_i32,
+                                   void* stream);
+
+/* Rotary positions in the interleaved layout: channels 2 i, 2 i + 1 of the first dims channels of a vector turn by the
+ * angle whose amplitude-scaled cosine and sine are table[position][i] (f32 [positions][dims / 2][2]). */
+
+/* Packed rows q [n_heads * head_dim] | k [n_kv * head_dim] | v [n_kv * head_dim]: all of q (and all of k) is divided by
+ * its root mean square over its n_* * dim channels, times gain f32 [n_* * head_dim], and its heads are rotated; q in
+ * place, keys and values to their cache slots. head_dim % 8 == 0. */
+uint32_t logismos_launch_qk_norm_rotary_store(void* qkv, int32_t ld, void* k_pool, void* v_pool, const void* slot_mapping_i64,
+                                              const void* positions_i32, int32_t rows, int32_t n_heads, int32_t n_kv_heads,
+                                              int32_t head_dim, int32_t dim, const void* gain_q_f32, const void* gain_k_f32,
+                                              float eps, const void* table_f32, int32_t rot_dims, int64_t n_pool_slots,
+                                              int32_t is_f32, void* status_i32, void* stream);
+/* Channels at .. at + dims of every head (head_dim apart, at % 8 == 0), in place. */
+uint32_t logismos_launch_rotary_heads(void* q, int32_t ld, const void* positions_i32, int32_t rows, int32_t n_heads,
+                                      int32_t head_dim, int32_t at, const void* table_f32, int32_t dims, int32_t is_f32,
+                                      void* stream);
+
+/* Attention over a window: a query at position i sees the keys j <= i with i - j < size or j < keep_first (size 0: all).
+ * sink: one is added to the softmax denominator. gate f32 [rows, ld_gate]: head h of a row is multiplied by the sigmoid of
+ * its column h (NULL: none). Scores are scaled by scale (> 0). */
+typedef struct lg_window {
+  float scale;
+  int32_t size, keep_first, sink;
+  const void* gate;
+  int32_t ld_gate;
+} lg_window_t;
+/* Decode launches split what a query sees, the kept blocks and the window's, as one context of this length. */
+int32_t logismos_window_context(int32_t context_len, int32_t size, int32_t keep_first);
+/* Keys that the prompt launch gathers for a sequence of kv_len keys whose last new_len are its queries. */
+int32_t logismos_window_keys(int32_t kv_len, int32_t new_len, int32_t size, int32_t keep_first);
+/* As logismos_launch_bias_attention_decode_bf16 (chunk_offsets over logismos_window_context of the context lengths),
+ * logismos_launch_bias_attention_prefix_bf16 (total_keys and max_keys over logismos_window_keys) and
+ * logismos_launch_bias_attention_f32. */
+uint32_t logismos_launch_window_attention_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool,
+                                                      const void* block_tables, const void* context_lens,
+                                                      const void* chunk_offsets, void* out, int32_t ld_out, void* scratch,
+                                                      int32_t n_seqs, int32_t total_chunks, int32_t chunk_tokens,
+                                                      int32_t max_blocks, int32_t n_pool_blocks, int32_t n_heads,
+                                                      int32_t n_kv_heads, int32_t head_dim, const lg_window_t* window,
+                                                      void* status_i32, void* stream);
+uint32_t logismos_launch_window_attention_prefix_bf16(const void* q, int32_t ld_q, const void* cu_seqlens_q, const void* kv_lens,
+                                                      const void* k_pool, const void* v_pool, const void* block_tables,
+                                                      int32_t max_blocks, int32_t n_pool_blocks, void* out, int32_t ld_out,
+                                                      void* scratch, int32_t n_q_tokens, int32_t total_keys, int32_t n_seqs,
+                                                      int32_t max_q_len, int32_t max_keys, int32_t n_heads, int32_t n_kv_heads,
+                                                      int32_t head_dim, const lg_window_t* window, void* status_i32,
+                                                      void* stream);
+uint32_t logismos_launch_window_attention_f32(const void* q_f32, int32_t ld_q, const void* k_pool, const void* v_pool,
+                                              const void* block_tables, const void* seq_ids_i32, const void* positions_i32,
+                                              void* out_f32, int32_t ld_out, int32_t rows, int32_t max_blocks,
+                                              int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
+                                              const lg_window_t* window, void* status_i32, void* stream);
+
+/* Router of a mixture of experts: scores s = softmax over the n_experts + n_identity logits of a token (f32 [tokens, ld]),
+ * the `top` largest s + correction are chosen, with the weights s / (sum of the chosen s + 1e-20). n_always further
+ * experts (a shared one) take every token with weight 1; together n_experts + n_always groups of rows. Identity experts
+ * have no rows: their weights add up in identity [tokens].
+ * pair i of a token (top + n_always of them) has its row of the groups in pair_row i32 [tokens, top + n_always] (-1: identity).
+ * logits are cleared with zero_logits. One launch for few tokens: offsets i32 [groups + 1], row_token i32 [pairs] included.
+ * Many tokens: route (counts i32 [n_experts], zero on entry) and then place, which also copies the tokens' rows of h (bf16
+ * [tokens, ld]) of the chosen experts to gathered [., ld] and lists the row tiles (logismos_launch_linear_experts_tc_bf16;
+ * the tiles of the n_always groups read h itself). At most 512 router outputs, top <= 32. */
+typedef struct lg_moe_route {
+  void* logits;
+  int32_t ld, zero_logits;
+  const void* correction;       /* f32 [n_experts + n_identity] */
+  int32_t n_experts, n_identity, top, n_always;
+  void *weights, *pair_row, *identity;
+  void *offsets, *row_token;    /* few tokens, fp32 */
+  void *counts, *pair_expert;   /* many tokens; pair_expert i32 [tokens, top] */
+  void *tiles, *n_tiles;
+} lg_moe_route_t;
+int32_t logismos_moe_few_tokens(void);  /* largest number of tokens of the one-launch form */
+int32_t logismos_moe_max_tiles(int32_t tokens, int32_t top, int32_t n_experts, int32_t n_always);
+uint32_t logismos_launch_moe_route(const lg_moe_route_t* args, int32_t tokens, void* stream);
+uint32_t logismos_launch_moe_place(const lg_moe_route_t* args, const void* h_bf16, void* gathered_bf16, int32_t ld,
+                                   int32_t tokens, void* stream);
 
 #ifdef __cplusplus
 }

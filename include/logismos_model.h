@@ -320,31 +320,53 @@ int32_t lg_latent_launches_last_step(const void* model);
 int32_t lg_latent_device_status(void* model);
 
 /* ====================================================================================
- * Decoder step over a stack of state-space and parallel (attention beside time mixing) layers (Katadra), post-norm.
- * No reference counterpart; the contract is that of lg_decoder_step. Weights are bf16, dense.
- *   x = embed[id];  x += norm1(mixer(x));  with a feed-forward x += norm2(W_down max(W_up x, 0)^2);  logits = head norm(x)
- *   norms: layer norms (gain and offset)
+ * Decoder step over a stack of layers, each a mixer and a feed-forward of its own kind. No reference counterpart; the
+ * contract is that of lg_decoder_step. Weights are bf16, dense. Sizes may differ from layer to layer; a layer may use the
+ * tensors of another one (weights_of), with a cache and states of its own. is_f32 as for lg_latent_config_t; in both
+ * formats the residual stream, norms, scores, routers, decays, step sizes and states are fp32.
+ *   x = embed[id];  per layer x += mixer, x += feed-forward, normed as the stack's `norm` says:
+ *   LG_NORM_LAYER_POST (Katadra)  x += norm(f(x)), layer norms (gain and offset); logits = head norm(x)
+ *   LG_NORM_TANH_AROUND (Vugedra) x += norm_b(f(norm_a(x))), norms tanh(alpha x) w + b; logits = head norm(x)
+ * Mixers:
  *   LG_MIXER_SSD: [z | x | B | C | dt] = W_in h, convolution, scalar-decay recurrence, gate, norm in parts, W_o
  *     (lg_ssd_t, logismos_launch_gated_group_norm)
- *   LG_MIXER_PARALLEL: left_scale * attention(h) + right_scale * time_mixing(h); attention without positions, unit
- *     queries and keys, capped scores, a learned bias by distance bucket, a query temperature and an output gate
- *     (lg_score_bias_t); time mixing with token shift and a low-rank data-dependent decay (lg_time_mix_t)
- * A layer may use the tensors of another one (weights_of), with a cache and states of its own. is_f32 as for
- * lg_latent_config_t; in both formats the residual stream, norms, scores, decays, step sizes and states are fp32.
+ *   LG_MIXER_PARALLEL (in a post-norm stack): left_scale * attention(h) + right_scale * time_mixing(h); attention without
+ *     positions, unit queries and keys, capped scores, a learned bias by distance bucket, a query temperature and an output
+ *     gate (lg_score_bias_t); time mixing with token shift and a low-rank data-dependent decay (lg_time_mix_t)
+ *   LG_MIXER_ATTENTION: q, k, v with biases, q and k normed over the whole projection and rotated; a window with kept first
+ *     keys, one added to the softmax denominator, an output gate per head (lg_window_t); W_o
+ *   LG_MIXER_GLA: gated linear attention, a decay per key channel (lg_time_mix_t, LG_DECAY_GATED); W_o
+ *   LG_MIXER_LATENT: queries W_uq rms(W_dq h), per head dim unrotated and rot_dims rotated channels; W_dkv h is the latent
+ *     (normed, cached) and one rotated key part for all heads; keys W_uk c, values W_uv c; causal, a gate per head; W_o
+ * Feed-forwards:
+ *   LG_FF_RELU2: W_down max(W_up h, 0)^2
+ *   LG_FF_GATED: W_down (silu(W_gate h) * (W_up h))
+ *   LG_FF_MIXTURE: `top` of experts + identity experts of the latter form by a softmax router with a correction for the
+ *     choice alone (lg_moe_route_t); identity experts return h; a shared expert is added (shared_ff 0: none)
  * ==================================================================================== */
-enum { LG_MIXER_SSD = 0, LG_MIXER_PARALLEL = 1 };
+enum { LG_MIXER_SSD = 0, LG_MIXER_PARALLEL = 1, LG_MIXER_ATTENTION = 2, LG_MIXER_GLA = 3, LG_MIXER_LATENT = 4 };
+enum { LG_FF_RELU2 = 0, LG_FF_GATED = 1, LG_FF_MIXTURE = 2 };
+enum { LG_NORM_LAYER_POST = 0, LG_NORM_TANH_AROUND = 1 };
 typedef struct lg_mixer_layer_config {
   int32_t kind;
   int32_t weights_of;           /* layer whose tensors are used; its own index: its own */
-  int32_t ff;                   /* 0: no feed-forward */
+  int32_t ff;                   /* 0: no feed-forward; a mixture: of one expert */
   /* state-space */
   int32_t ssd_heads, ssd_vdim, ssd_state, ssd_groups, ssd_norm_groups, ssd_taps;
-  /* attention: sizes <= 256; bias_rows rows of the bias table, distances from bias_max on share the last one */
+  /* attention of any kind and gated linear attention: sizes <= 256. Parallel layers: bias_rows rows of the bias table,
+   * distances from bias_max on share the last one */
   int32_t heads, kv_heads, dim, vdim, bias_rows, bias_max;
   float scale, softcap, temp_coef, temp_every;
-  /* time mixing */
+  /* time mixing; tm_rank (of the decay) also for gated linear attention */
   int32_t tm_heads, tm_dim, tm_rank;
   float left_scale, right_scale;
+  int32_t ff_kind;
+  int32_t experts, identity, top, shared_ff;   /* a mixture */
+  int32_t window, keep_first;   /* attention; window 0: all keys */
+  int32_t q_rank, kv_rank;      /* latent attention: kv_rank + rot_dims <= 1024 */
+  int32_t rot_dims;             /* rotated channels per head, interleaved pairs */
+  float tau;                    /* gated linear attention */
+  double rot_base, rot_factor, rot_original, rot_fast, rot_slow;   /* YaRN interpolation; rot_factor 0: none */
 } lg_mixer_layer_config_t;
 typedef struct lg_mixer_config {
   int32_t vocab, width, n_layers;
@@ -356,26 +378,35 @@ typedef struct lg_mixer_config {
   int32_t max_out_rows;
   int32_t keep_layers;          /* != 0: the stream after every layer is kept (lg_mixer_snapshot) */
   const lg_mixer_layer_config_t* layers;
+  int32_t norm;
 } lg_mixer_config_t;
-/* bf16 values on the host, [out, in]; entries of the other kind of mixer, of a missing feed-forward and of a layer
- * with weights_of are NULL. mu [5] in the order r, k, v, g, w. */
+/* bf16 values on the host, [out, in]; entries of other kinds of mixer, of a missing feed-forward and of a layer
+ * with weights_of are NULL. mu [5] in the order r, k, v, g, w. experts [3 * experts]: gate, up, down of each. */
 typedef struct lg_mixer_layer_weights {
   const void *norm1, *norm1_b, *norm2, *norm2_b, *up, *down;
   const void *in, *conv, *conv_b, *dt_bias, *A_log, *D, *norm, *o;
   const void *left_q, *left_k, *left_v, *left_rel, *left_g, *left_o;
   const void* mu[5];
   const void *right_r, *right_k, *right_v, *right_g, *right_w1, *right_w2, *right_w0, *right_u, *right_norm, *right_o;
+  const void *norm1_alpha, *norm1b, *norm1b_b, *norm1b_alpha, *norm2_alpha, *norm2b, *norm2b_b, *norm2b_alpha;
+  const void *q, *q_b, *q_norm, *k, *k_b, *k_norm, *v, *v_b, *g, *a1, *a2, *a2_b;
+  const void *dq, *dq_norm, *uq, *dkv, *dkv_norm, *uk, *uv;
+  const void *gate, *router, *correction, *shared_gate, *shared_up, *shared_down;
+  const void* const* experts;
 } lg_mixer_layer_weights_t;
 typedef struct lg_mixer_weights {
   const void *embed, *final_norm, *final_norm_b, *head;
   const lg_mixer_layer_weights_t* layers;
+  const void* final_norm_alpha; /* tanh norms */
 } lg_mixer_weights_t;
 
 uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_mixer_weights_t* w, void** model);
-/* The same from a bf16 safetensors file with exactly these tensors: embed, final.norm, head and, per layer i that
- * owns tensors, l<i>.norm1, with a feed-forward l<i>.norm2, l<i>.mlp.{up,down}; l<i>.mix.{in,conv,conv.b,dt_bias,
- * A_log,D,norm,o} or l<i>.mix.left.{q,k,v,rel,g,o} and l<i>.mix.right.{mu.r,mu.k,mu.v,mu.g,mu.w,r,k,v,g,w1,w2,w0,u,
- * norm,o}; every norm of the stack also as .b. bias_rows and tm_rank are taken from the tensors. */
+/* The same from a bf16 safetensors file with exactly these tensors: embed, final.norm, head and, per layer i that owns
+ * tensors, l<i>.norm1 and with a feed-forward l<i>.norm2 (tanh norms: also l<i>.norm1b, l<i>.norm2b), every one of them with
+ * .b (and .alpha); under l<i>.mix.: {in,conv,conv.b,dt_bias,A_log,D,norm,o}, left.{q,k,v,rel,g,o} and right.{mu.r,mu.k,mu.v,
+ * mu.g,mu.w,r,k,v,g,w1,w2,w0,u,norm,o}, {q,k,v,g,o} with {q,k,v}.b and {q,k}.norm, {q,k,v,g,o,norm,a1,a2,a2.b}, or {dq,
+ * dq.norm,uq,dkv,dkv.norm,uk,uv,g,o}; under l<i>.mlp.: {up,down}, {gate,up,down}, or {router,correction} with {e<j>,shared}.
+ * {gate,up,down}. bias_rows and tm_rank are taken from the tensors. */
 uint32_t lg_mixer_load(int32_t device, const char* path, const lg_mixer_config_t* cfg, void** model);
 void lg_mixer_destroy(void* model);
 /* Step, logits and diagnostics as for lg_latent_*. Recurrent states are updated in place: a step that failed part-way

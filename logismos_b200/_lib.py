@@ -137,14 +137,14 @@ def _declare(l, partial=False):
         "logismos_launch_linear_t_act_bf16": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp, vp],
         "logismos_launch_linear_small_bf16": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i64, i64, i64, i32, f32, f32, f32, vp],
         "logismos_launch_linear_f32": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i64, i64, i64, i32, f32, f32, f32, vp],
-        "logismos_launch_varlen_attention_kv_tc_bf16": [vp, i32, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp],
+        "logismos_launch_varlen_attention_kv_tc_bf16": [vp, i32, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
         "logismos_launch_depth_mix_f32": [vp, i64, i32, vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, vp],
         "logismos_launch_norm_conv": [vp, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, vp],
         "logismos_launch_depth_mix_conv_decode": [vp, i64, i32, vp, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp],
-        "logismos_launch_latent_norm_store": [vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i64, i32, i32, vp, vp],
+        "logismos_launch_latent_norm_store": [vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i64, i32, i32, vp, vp, vp],
         "logismos_launch_latent_gather_bf16": [vp, vp, i32, i32, vp, vp, vp, i32, i32, i32, i32, vp, vp],
-        "logismos_launch_latent_decode_bf16": [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp],
-        "logismos_launch_latent_attention_f32": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, vp],
+        "logismos_launch_latent_decode_bf16": [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
+        "logismos_launch_latent_attention_f32": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
         "lg_latent_create": [i32, vp, vp, C.POINTER(vp)],
         "lg_latent_load": [i32, C.c_char_p, vp, C.POINTER(vp)],
         "lg_latent_step": [vp, vp, vp, vp, i32, vp, vp, vp, i32, vp],
@@ -169,6 +169,19 @@ def _declare(l, partial=False):
         "logismos_launch_bias_attention_prefix_bf16": [vp, i32, vp, vp, vp, vp, vp, i32, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32,
                                                        vp, vp, vp],
         "logismos_launch_bias_attention_f32": [vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
+        # norms without statistics, rotary positions, windows, mixtures of experts
+        "logismos_launch_tanh_norm": [vp, i32, vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, vp, vp],
+        "logismos_launch_qk_norm_rotary_store": [vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp, f32, vp, i32, i64, i32, vp, vp],
+        "logismos_launch_rotary_heads": [vp, i32, vp, i32, i32, i32, i32, vp, i32, i32, vp],
+        "logismos_launch_window_attention_decode_bf16": [vp, i32, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
+        "logismos_launch_window_attention_prefix_bf16": [vp, i32, vp, vp, vp, vp, vp, i32, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32,
+                                                         vp, vp, vp],
+        "logismos_launch_window_attention_f32": [vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
+        "logismos_launch_moe_route": [vp, i32, vp],
+        "logismos_launch_moe_place": [vp, vp, vp, i32, i32, vp],
+        "logismos_launch_linear_experts_small_bf16": [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp],
+        "logismos_launch_linear_experts_f32": [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp],
+        "logismos_launch_linear_experts_tc_bf16": [vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp],
         "lg_mixer_create": [i32, vp, vp, C.POINTER(vp)],
         "lg_mixer_load": [i32, C.c_char_p, vp, C.POINTER(vp)],
         "lg_mixer_step": [vp, vp, vp, vp, i32, vp, vp, vp, i32, vp],
@@ -216,12 +229,16 @@ def _declare(l, partial=False):
         "lg_latent_device_status": ([vp], i32),
         "lg_latent_destroy": ([vp], None),
         "lg_latent_logits_device": ([vp], vp),
-        "logismos_time_mix_has_chunked": ([i32], i32),
+        "logismos_time_mix_has_chunked": ([i32, i32], i32),
         "logismos_ssd_has_chunked": ([i32, i32], i32),
         "lg_mixer_launches_last_step": ([vp], i32),
         "lg_mixer_device_status": ([vp], i32),
         "lg_mixer_destroy": ([vp], None),
         "lg_mixer_logits_device": ([vp], vp),
+        "logismos_window_context": ([i32, i32, i32], i32),
+        "logismos_window_keys": ([i32, i32, i32, i32], i32),
+        "logismos_moe_few_tokens": ([], i32),
+        "logismos_moe_max_tiles": ([i32, i32, i32, i32], i32),
         "logismos_latent_gather_rows": ([i32, i32], i32),
         "logismos_pick_latent_chunk": ([vp, i32, i32], i32),
         "logismos_latent_max_chunks": ([i32], i32),

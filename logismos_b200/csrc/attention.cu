@@ -284,8 +284,13 @@ LG_DEVINL void stage_block(uint32_t sbase, const __nv_bfloat16* kpool, const __n
   }
 }
 
-// EXT: capped and biased scores, gated output, and 16 query heads of a key head per CTA (ScoreExt)
-template <int HD, int kDecWarps, int kDecStages, bool EXT = false>
+// What a decode kernel does beyond the plain softmax; both forms take 16 query heads of a key head per CTA. kWindowed: the
+// blocks that a query sees, kept ones and the window's, are numbered through ("virtual" blocks) and split in chunks.
+enum { kPlain = 0, kBiased = 1, kWindowed = 2 };
+template <int MODE> struct ExtOf { using type = ScoreExt; };
+template <> struct ExtOf<kWindowed> { using type = WindowExt; };
+
+template <int HD, int kDecWarps, int kDecStages, int MODE = kPlain>
 __global__ void __launch_bounds__(kDecWarps * 32)
 paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ kpool,
                     __nv_bfloat16* __restrict__ vpool, const __nv_bfloat16* __restrict__ new_k,
@@ -293,8 +298,9 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
                     const int* __restrict__ ctx_lens, const int* __restrict__ chunk_offsets,
                     __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
                     int* __restrict__ status, int n_seqs, int chunk_tokens, int max_blocks, int n_pool_blocks,
-                    int n_heads, int n_kv, float sl2, ScoreExt ext) {
+                    int n_heads, int n_kv, float sl2, typename ExtOf<MODE>::type ext) {
   lg::pdl_prologue();
+  constexpr bool EXT = MODE != kPlain;
   extern __shared__ __align__(128) uint8_t smem[];
   const int groups = EXT ? (n_heads / n_kv + 15) / 16 : 1;
   const int chunk_id = blockIdx.x, kvh = blockIdx.y / groups, r_base = (blockIdx.y % groups) * 16;
@@ -302,7 +308,8 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
   const int g = lane >> 2, c = lane & 3;
   const int n_rep = EXT ? min(16, n_heads / n_kv - r_base) : n_heads / n_kv;  // query heads of this CTA
   const int head0 = kvh * (n_heads / n_kv) + r_base;
-  const int64_t q_stride = EXT ? ext.ld_q : (int64_t)n_heads * HD;
+  int64_t q_stride = (int64_t)n_heads * HD;
+  if constexpr (EXT) q_stride = ext.ld_q;
   constexpr int D = HD, kRowBytes = HD * 2, DT = HD / 8, CH = HD / 8;
   constexpr int kDecStageBytes = DecCfg<HD, kDecWarps, kDecStages>::kStageBytes;
   const int row_elems = n_kv * D;
@@ -317,8 +324,10 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
   const int chunk_in_seq = chunk_id - chunk_offsets[seq];
   const int n_chunks = chunk_offsets[seq + 1] - chunk_offsets[seq];
   const int ctx = ctx_lens[seq];
+  int gap = 0, kept_blocks = 0;  // a virtual block from kept_blocks on stands for the block `gap` further
+  if constexpr (MODE == kWindowed) { gap = window_gap_blocks(ctx, ext.size, ext.keep); kept_blocks = (ext.keep + kBlock - 1) / kBlock; }
   const int tok_begin = chunk_in_seq * chunk_tokens;
-  const int tok_end = min(ctx, tok_begin + chunk_tokens);
+  const int tok_end = min(ctx - gap * kBlock, tok_begin + chunk_tokens);
   const int* table = tables + (int64_t)seq * max_blocks;
 
   // ---- fused append: the CTA of the last chunk stores the new token's K/V slice first ----
@@ -362,7 +371,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
   const float *bias0 = nullptr, *bias1 = nullptr;
   float far0 = 0.0f, far1 = 0.0f;  // bias of every distance >= far
-  if (EXT) {
+  if constexpr (MODE == kBiased) {
     bias0 = ext.bias + (int64_t)(head0 + min(g, n_rep - 1)) * (ext.far + 1);
     bias1 = ext.bias + (int64_t)(head0 + min(g + 8, n_rep - 1)) * (ext.far + 1);
     far0 = __ldg(bias0 + ext.far);
@@ -375,9 +384,10 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
   const int my_first = blk_begin + warp;
   const int my_count = my_first < blk_end ? (blk_end - my_first + kDecWarps - 1) / kDecWarps : 0;
 
+  auto place = [&](int vb) { return MODE == kWindowed && vb >= kept_blocks ? vb + gap : vb; };
   auto issue = [&](int i) {  // i-th block of this warp; always commits a group (possibly empty)
     if (i < my_count) {
-      const int bidx = my_first + i * kDecWarps;
+      const int bidx = place(my_first + i * kDecWarps);
       const int pb = bidx < max_blocks ? table[bidx] : -1;
       if (pb >= 0 && pb < n_pool_blocks) {
         stage_block<HD>(wbase + (i % kDecStages) * kDecStageBytes, kpool, vpool, pb, row_elems, kvh, lane);
@@ -394,14 +404,24 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
     issue(i + kDecStages - 1);
     cp_async_wait<kDecStages - 1>();
     __syncwarp();
-    const int blk = my_first + i * kDecWarps;
-    const int pb = blk < max_blocks ? table[blk] : -1;
+    const int blk = my_first + i * kDecWarps, real = place(blk);
+    const int pb = real < max_blocks ? table[real] : -1;
     const bool valid_block = pb >= 0 && pb < n_pool_blocks;
     const uint32_t sb = wbase + (i % kDecStages) * kDecStageBytes;
     float s[2][4];
     if (valid_block) {
       qk_tile<2, HD>(qf, sb, 0, lane, s);
-      if (EXT) {
+      if constexpr (MODE == kWindowed) {
+        const int first = real * kBlock;
+        if (ctx - 1 - first >= ext.size && first + kBlock > ext.keep) {  // some key may lie outside
+#pragma unroll
+          for (int t = 0; t < 2; ++t)
+#pragma unroll
+            for (int e = 0; e < 2; ++e)
+              if (!ext.sees(ctx - 1, first + 8 * t + 2 * c + e)) s[t][e] = s[t][2 + e] = -INFINITY;
+        }
+      }
+      if constexpr (MODE == kBiased) {
         const int d0 = ctx - 1 - blk * kBlock;  // distance of the block's first key
         const bool near = d0 - (kBlock - 1) < ext.far;
 #pragma unroll
@@ -470,23 +490,29 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, sml[(w * 16 + r) * 2]);
-    float L = 0.0f, f[kDecWarps];
+    float L = 0.0f, f[kDecWarps], gate = 1.0f;
+    const int head = head0 + r;
+    if constexpr (MODE == kWindowed) {
+      gate = ext.head_gate(seq, head);
+      if (ext.sink && n_chunks == 1) { M = fmaxf(M, 0.0f); L = exp2f(-M * sl2); }
+    }
 #pragma unroll
     for (int w = 0; w < kDecWarps; ++w) {
       const float mw = sml[(w * 16 + r) * 2];
       f[w] = (mw == -INFINITY) ? 0.0f : exp2f((mw - M) * sl2);
       L += sml[(w * 16 + r) * 2 + 1] * f[w];
     }
-    const int head = head0 + r;
 #pragma unroll
     for (int d = tid; d < D; d += kDecWarps * 32) {
       float acc = 0.0f;
 #pragma unroll
       for (int w = 0; w < kDecWarps; ++w) acc += so[(w * 16 + r) * D + d] * f[w];
-      if (EXT && n_chunks == 1)
-        out[(int64_t)seq * ext.ld_out + head * D + d] =
-            __float2bfloat16_rn(ext.gated(acc / L, __bfloat162float(ext.gate[(int64_t)seq * ext.ld_gate + head * D + d])));
-      else if (n_chunks == 1) out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
+      if (EXT && n_chunks == 1) {
+        if constexpr (MODE == kBiased)
+          out[(int64_t)seq * ext.ld_out + head * D + d] =
+              __float2bfloat16_rn(ext.gated(acc / L, __bfloat162float(ext.gate[(int64_t)seq * ext.ld_gate + head * D + d])));
+        if constexpr (MODE == kWindowed) out[(int64_t)seq * ext.ld_out + head * D + d] = __float2bfloat16_rn(acc / L * gate);
+      } else if (n_chunks == 1) out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
       else part_o[((int64_t)chunk_id * n_heads + head) * D + d] = acc;
     }
     if (n_chunks != 1 && tid == 0) {
@@ -497,10 +523,10 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
 }
 
 // merges the per-chunk partial results of sequences that were split into several chunks
-template <bool EXT = false>
+template <int MODE = kPlain>
 __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                           const int* __restrict__ chunk_offsets, __nv_bfloat16* __restrict__ out,
-                                          int n_heads, int D, float sl2, ScoreExt ext) {
+                                          int n_heads, int D, float sl2, typename ExtOf<MODE>::type ext) {
   lg::pdl_prologue();
   const int seq = blockIdx.x, head = blockIdx.y, d = threadIdx.x;
   const int c0 = chunk_offsets[seq], c1 = chunk_offsets[seq + 1];
@@ -508,14 +534,18 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o, cons
   float M = -INFINITY;
   for (int ck = c0; ck < c1; ++ck) M = fmaxf(M, part_ml[((int64_t)ck * n_heads + head) * 2]);
   float L = 0.0f, acc = 0.0f;
+  if constexpr (MODE == kWindowed)
+    if (ext.sink) { M = fmaxf(M, 0.0f); L = exp2f(-M * sl2); }
   for (int ck = c0; ck < c1; ++ck) {
     const float mw = part_ml[((int64_t)ck * n_heads + head) * 2];
     const float f = (mw == -INFINITY) ? 0.0f : exp2f((mw - M) * sl2);
     L += part_ml[((int64_t)ck * n_heads + head) * 2 + 1] * f;
     acc += part_o[((int64_t)ck * n_heads + head) * D + d] * f;
   }
-  if (EXT)
+  if constexpr (MODE == kBiased)
     out[(int64_t)seq * ext.ld_out + head * D + d] = __float2bfloat16_rn(ext.gated(acc / L, __bfloat162float(ext.gate[(int64_t)seq * ext.ld_gate + head * D + d])));
+  else if constexpr (MODE == kWindowed)
+    out[(int64_t)seq * ext.ld_out + head * D + d] = __float2bfloat16_rn(acc / L * ext.head_gate(seq, head));
   else
     out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
 }
@@ -632,12 +662,45 @@ uint32_t logismos_launch_paged_attention_decode_bf16(
   if (rc) return rc;
   if (total_chunks > n_seqs) {  // at least one sequence spans several chunks
     dim3 mgrid(n_seqs, n_heads);
-    lg::launch(paged_decode_merge_kernel<false>, mgrid, dim3(head_dim), 0, (cudaStream_t)stream, part_o, part_ml, (const int*)chunk_offsets,
+    lg::launch(paged_decode_merge_kernel<kPlain>, mgrid, dim3(head_dim), 0, (cudaStream_t)stream, part_o, part_ml, (const int*)chunk_offsets,
                                                                            (__nv_bfloat16*)out, n_heads, head_dim, sl2, ScoreExt{});
     rc = lg::launch_status();
   }
   return rc;
 }
+
+// the two extended forms of the decode kernel; the cache already holds the new tokens
+}  // extern "C"
+template <int MODE, typename Ext>
+static uint32_t launch_ext_decode(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables, const void* context_lens,
+                                  const void* chunk_offsets, void* out, int32_t ld_out, void* scratch, int32_t n_seqs, int32_t total_chunks,
+                                  int32_t chunk_tokens, int32_t max_blocks, int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
+                                  float sl2, const Ext& ext, void* status, void* stream) {
+  if (n_seqs <= 0 || total_chunks < n_seqs || chunk_tokens <= 0 || (chunk_tokens % 64) || max_blocks <= 0 || n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 ||
+      (n_heads % n_kv_heads) || (head_dim != 64 && head_dim != 128 && head_dim != 256) || (ld_q % 8) || ld_q < n_heads * head_dim || ld_out < n_heads * head_dim ||
+      !q || !k_pool || !v_pool || !out || !scratch || (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)scratch) & 15))
+    return lg::kInvalidValue;
+  float* part_o = (float*)scratch;
+  float* part_ml = part_o + (size_t)total_chunks * n_heads * head_dim;
+  const dim3 grid((unsigned)total_chunks, (unsigned)(n_kv_heads * ((n_heads / n_kv_heads + 15) / 16)));
+  auto launch = [&](auto kern, int warps, int smem) -> uint32_t {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+    lg::launch(kern, grid, dim3(warps * 32), smem, (cudaStream_t)stream, (const __nv_bfloat16*)q, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool,
+               (const __nv_bfloat16*)nullptr, (const __nv_bfloat16*)nullptr, (const int*)block_tables, (const int*)context_lens, (const int*)chunk_offsets,
+               (__nv_bfloat16*)out, part_o, part_ml, (int*)status, n_seqs, chunk_tokens, max_blocks, n_pool_blocks, n_heads, n_kv_heads, sl2, ext);
+    return lg::launch_status();
+  };
+  uint32_t rc = head_dim == 64 ? launch(paged_decode_kernel<64, 4, 4, MODE>, 4, DecCfg<64, 4, 4>::kSmem)
+              : head_dim == 128 ? launch(paged_decode_kernel<128, 4, 2, MODE>, 4, DecCfg<128, 4, 2>::kSmem)
+                                : launch(paged_decode_kernel<256, 3, 2, MODE>, 3, DecCfg<256, 3, 2>::kSmem);
+  if (rc || total_chunks == n_seqs) return rc;
+  lg::launch(paged_decode_merge_kernel<MODE>, dim3((unsigned)n_seqs, (unsigned)n_heads), dim3((unsigned)head_dim), 0, (cudaStream_t)stream, (const float*)part_o,
+             (const float*)part_ml, (const int*)chunk_offsets, (__nv_bfloat16*)out, n_heads, head_dim, sl2, ext);
+  return lg::launch_status();
+}
+
+extern "C" {
 
 uint32_t logismos_launch_bias_attention_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables,
                                                     const void* context_lens, const void* chunk_offsets, void* out, int32_t ld_out, void* scratch,
@@ -645,29 +708,27 @@ uint32_t logismos_launch_bias_attention_decode_bf16(const void* q, int32_t ld_q,
                                                     int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
                                                     const lg_score_bias_t* score, void* status, void* stream) {
   lg::LaunchScope launch_scope_;
-  if (n_seqs <= 0 || total_chunks < n_seqs || chunk_tokens <= 0 || (chunk_tokens % 64) || max_blocks <= 0 || n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 ||
-      (n_heads % n_kv_heads) || (head_dim != 64 && head_dim != 128 && head_dim != 256) || (ld_q % 8) || ld_q < n_heads * head_dim || ld_out < n_heads * head_dim ||
-      !q || !k_pool || !v_pool || !out || !scratch || (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)scratch) & 15) || !score_ok(score, n_heads * head_dim))
-    return lg::kInvalidValue;
-  float* part_o = (float*)scratch;
-  float* part_ml = part_o + (size_t)total_chunks * n_heads * head_dim;
-  const ScoreExt ext = score_ext(score, ld_q, ld_out);
-  const dim3 grid((unsigned)total_chunks, (unsigned)(n_kv_heads * ((n_heads / n_kv_heads + 15) / 16)));
-  auto launch = [&](auto kern, int warps, int smem) -> uint32_t {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return (uint32_t)e;
-    lg::launch(kern, grid, dim3(warps * 32), smem, (cudaStream_t)stream, (const __nv_bfloat16*)q, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool,
-               (const __nv_bfloat16*)nullptr, (const __nv_bfloat16*)nullptr, (const int*)block_tables, (const int*)context_lens, (const int*)chunk_offsets,
-               (__nv_bfloat16*)out, part_o, part_ml, (int*)status, n_seqs, chunk_tokens, max_blocks, n_pool_blocks, n_heads, n_kv_heads, 1.0f, ext);
-    return lg::launch_status();
-  };
-  uint32_t rc = head_dim == 64 ? launch(paged_decode_kernel<64, 4, 4, true>, 4, DecCfg<64, 4, 4>::kSmem)
-              : head_dim == 128 ? launch(paged_decode_kernel<128, 4, 2, true>, 4, DecCfg<128, 4, 2>::kSmem)
-                                : launch(paged_decode_kernel<256, 3, 2, true>, 3, DecCfg<256, 3, 2>::kSmem);
-  if (rc || total_chunks == n_seqs) return rc;
-  lg::launch(paged_decode_merge_kernel<true>, dim3((unsigned)n_seqs, (unsigned)n_heads), dim3((unsigned)head_dim), 0, (cudaStream_t)stream, (const float*)part_o,
-             (const float*)part_ml, (const int*)chunk_offsets, (__nv_bfloat16*)out, n_heads, head_dim, 1.0f, ext);
-  return lg::launch_status();
+  if (!score_ok(score, n_heads * head_dim)) return lg::kInvalidValue;
+  return launch_ext_decode<kBiased>(q, ld_q, k_pool, v_pool, block_tables, context_lens, chunk_offsets, out, ld_out, scratch, n_seqs, total_chunks, chunk_tokens,
+                                    max_blocks, n_pool_blocks, n_heads, n_kv_heads, head_dim, 1.0f, score_ext(score, ld_q, ld_out), status, stream);
+}
+
+int32_t logismos_window_context(int32_t context_len, int32_t size, int32_t keep_first) {
+  return context_len - kBlock * window_gap_blocks(context_len, size ? size : 0x7fffffff, keep_first);
+}
+int32_t logismos_window_keys(int32_t kv_len, int32_t new_len, int32_t size, int32_t keep_first) {
+  return kv_len - window_gap_keys(kv_len, new_len, size ? size : 0x7fffffff, keep_first);
+}
+
+uint32_t logismos_launch_window_attention_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables,
+                                                      const void* context_lens, const void* chunk_offsets, void* out, int32_t ld_out, void* scratch,
+                                                      int32_t n_seqs, int32_t total_chunks, int32_t chunk_tokens, int32_t max_blocks,
+                                                      int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
+                                                      const lg_window_t* window, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!window_ok(window, n_heads)) return lg::kInvalidValue;
+  return launch_ext_decode<kWindowed>(q, ld_q, k_pool, v_pool, block_tables, context_lens, chunk_offsets, out, ld_out, scratch, n_seqs, total_chunks, chunk_tokens,
+                                      max_blocks, n_pool_blocks, n_heads, n_kv_heads, head_dim, window->scale * kLog2e, window_ext(window, ld_q, ld_out), status, stream);
 }
 
 uint32_t logismos_launch_paged_kv_store_bf16(const void* k, const void* v, int32_t src_row_stride, void* k_pool,

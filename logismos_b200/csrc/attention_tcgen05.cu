@@ -163,13 +163,21 @@ transpose_v_kernel(const __nv_bfloat16* __restrict__ qkv, const int* __restrict_
 // zeroed). Token t of sequence s is read from block tables[s * max_blocks + t / 16], slot t % 16 of
 // k_pool / v_pool [n_pool_blocks, 16, n_kv * HD] (the row layout of FlatKvCache,
 // crates/cache/src/flat.rs:36-69; the read is KvCache::get, :254-304). A block id outside the pool
-// yields zero rows and raises the status word. Grid (key blocks of 64, kv heads, sequences).
+// yields zero rows and raises the status word. Grid (key blocks of 64, kv heads, sequences). With a window the keys between
+// the kept ones and the first query's window are left out (window_gap_keys): rows from tile kept_tiles on stand `gap` keys
+// further in the sequence.
+struct GatherWindow {
+  const int* cu;     // query offsets (NULL: all keys are gathered)
+  int size, keep;
+  LG_DEVINL int gap(int s, int kv_len) const { return cu ? window_gap_keys(kv_len, cu[s + 1] - cu[s], size, keep) : 0; }
+};
+
 template <int HD>
 __global__ void __launch_bounds__(256)
 gather_paged_kv_kernel(const __nv_bfloat16* __restrict__ kpool, const __nv_bfloat16* __restrict__ vpool,
                        const int* __restrict__ tables, int max_blocks, int n_pool_blocks, const int* __restrict__ kv_lens,
                        __nv_bfloat16* __restrict__ kbuf, __nv_bfloat16* __restrict__ vt, int* __restrict__ pstart, int n_seqs,
-                       int tp, int tx, int n_kv, int* __restrict__ status) {
+                       int tp, int tx, int n_kv, GatherWindow win, int* __restrict__ status) {
   lg::pdl_prologue();
   __shared__ __align__(16) __nv_bfloat16 tile[64][HD + 8];
   constexpr int kParts = 256 / HD, kChunks = HD / 8;
@@ -178,7 +186,7 @@ gather_paged_kv_kernel(const __nv_bfloat16* __restrict__ kpool, const __nv_bfloa
   const int tb = (int)blockIdx.x % tx, kvh = ((int)blockIdx.x / tx) % n_kv, s = (int)blockIdx.x / (tx * n_kv);
   if (tid < 32) {
     int part = 0;
-    for (int i = tid; i < s; i += 32) part += round8(max(kv_lens[i], 0));
+    for (int i = tid; i < s; i += 32) part += round8(max(kv_lens[i] - win.gap(i, kv_lens[i]), 0));
     part += __shfl_xor_sync(0xffffffffu, part, 16);
     part += __shfl_xor_sync(0xffffffffu, part, 8);
     part += __shfl_xor_sync(0xffffffffu, part, 4);
@@ -188,7 +196,8 @@ gather_paged_kv_kernel(const __nv_bfloat16* __restrict__ kpool, const __nv_bfloa
   }
   __syncthreads();
   const int p0 = p0_s;
-  const int len = max(kv_lens[s], 0), plen = round8(len);
+  const int gap = win.gap(s, kv_lens[s]), kept_rows = (win.keep + 127) / 128 * 128;
+  const int len = max(kv_lens[s] - gap, 0), plen = round8(len);
   const int row_w = n_kv * HD;
   if (p0 + plen > tp) {  // the caller's total does not cover these lengths: nothing is written
     if (tid == 0 && status) atomicExch(status, 1);
@@ -207,12 +216,12 @@ gather_paged_kv_kernel(const __nv_bfloat16* __restrict__ kpool, const __nv_bfloa
     const int r = u / kChunks, ch = u % kChunks, t = tb * 64 + r;
     uint4 kq = make_uint4(0u, 0u, 0u, 0u), vq = kq;
     if (t < len) {
-      const int bi = t >> 4;
+      const int at = t < kept_rows ? t : t + gap, bi = at >> 4;
       const int blk = bi < max_blocks ? __ldg(tables + (size_t)s * max_blocks + bi) : -1;
       if (blk < 0 || blk >= n_pool_blocks) {
         if (ch == 0 && status) atomicExch(status, 1);
       } else {
-        const size_t src = ((size_t)blk * 16 + (t & 15)) * row_w + kvh * HD + ch * 8;
+        const size_t src = ((size_t)blk * 16 + (at & 15)) * row_w + kvh * HD + ch * 8;
         kq = __ldg(reinterpret_cast<const uint4*>(kpool + src));
         vq = __ldg(reinterpret_cast<const uint4*>(vpool + src));
       }
@@ -325,7 +334,11 @@ gather_paged_kv_turbo3_kernel(const uint8_t* __restrict__ kpool, const uint8_t* 
 // where cap and biases bound every score so tightly that exp2 of it neither over- nor underflows, and no maximum is
 // kept (one pass over the scores, the output never rescaled); and that with the cap as a polynomial, where the products
 // are known to be small (unit queries and keys): the multiplier units then leave the exponential unit to the softmax.
-enum { kPlain = 0, kBiased = 1, kBounded = 2, kPoly = 3 };
+// kWindowed: a window with kept first keys and a softmax denominator with one added, where asked for, and a gate per head;
+// only the key tiles that some query of the CTA sees are visited.
+enum { kPlain = 0, kBiased = 1, kBounded = 2, kPoly = 3, kWindowed = 4 };
+template <int SCORE> struct ExtOf { using type = ScoreExt; };
+template <> struct ExtOf<kWindowed> { using type = WindowExt; };
 constexpr int kBiasWindow = 160;  // distances between the 32 rows of a warp and 128 keys
 constexpr float kBoundedLog2 = 80.0f;
 
@@ -363,8 +376,9 @@ __global__ void __launch_bounds__(192, HD <= 128 ? 2 : 1)
 attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_vt, const int* __restrict__ cu, const int* __restrict__ pstart,
                     const int* __restrict__ kv_lens, __nv_bfloat16* __restrict__ out, int out_stride, int n_heads, int n_kv, int k_off,
-                    float sl2, const ScoreExt ext, int* __restrict__ status) {
+                    float sl2, const typename ExtOf<SCORE>::type ext, int* __restrict__ status) {
   lg::pdl_prologue();
+  constexpr bool BIASED = SCORE == kBiased || SCORE == kBounded || SCORE == kPoly;
   using C = Attn<HD>;
   constexpr int kQBytes = C::kQBytes, kKBytes = C::kKBytes, kVBytes = C::kVBytes, kVTile = C::kVTile;
   constexpr uint32_t kTmemCols = C::kTmemCols;
@@ -384,7 +398,17 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   const int k_row0 = kv_lens ? pstart[s] : t0;
   const int kvh = h / (n_heads / n_kv);
   const int kv_len = CAUSAL ? min(kv_total, q_off + q0 + 128) : kv_total;
-  const int nb = (kv_len + 127) >> 7;
+  int nb = (kv_len + 127) >> 7;
+  // windows: the tiles [0, kept) and [kept + skip, ..) are visited, gathered rows of the latter standing `gap` keys further
+  int kept = 0, skip = 0, gap = 0;
+  if constexpr (SCORE == kWindowed) {
+    gap = kv_lens ? window_gap_keys(kv_total, len, ext.size, ext.keep) : 0;
+    nb = (kv_len - gap + 127) >> 7;
+    kept = min((ext.keep + 127) >> 7, nb);
+    const int first = q_off + q0 - ext.size + 1 - gap;  // gathered row of the first key in the window of the tile's first query
+    if (ext.size <= q_off + q0 && (first >> 7) > kept) skip = (first >> 7) - kept;
+    nb -= skip;
+  }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
   extern __shared__ uint8_t smem_raw[];
@@ -423,14 +447,15 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       const int pv = pstart[s];
       for (int j = 0; j < nb; ++j) {
         const uint32_t phase = (uint32_t)j & 1u;
+        const int jt = SCORE == kWindowed && j >= kept ? j + skip : j;
         if (!mbar_wait(k_empty, phase ^ 1u, abort_flag)) break;
         mbar_expect_tx(k_full, (uint32_t)kKBytes);
 #pragma unroll
-        for (int i = 0; i < HD / 64; ++i) tma_load_2d(k_smem + i * kTileBytes, &map_k, k_full, k_off + kvh * HD + i * 64, k_row0 + j * 128);
+        for (int i = 0; i < HD / 64; ++i) tma_load_2d(k_smem + i * kTileBytes, &map_k, k_full, k_off + kvh * HD + i * 64, k_row0 + jt * 128);
         if (!mbar_wait(v_empty, phase ^ 1u, abort_flag)) break;
         mbar_expect_tx(v_full, (uint32_t)kVBytes);
-        tma_load_2d(v_smem, &map_vt, v_full, pv + j * 128, kvh * HD);
-        tma_load_2d(v_smem + kVTile, &map_vt, v_full, pv + j * 128 + 64, kvh * HD);
+        tma_load_2d(v_smem, &map_vt, v_full, pv + jt * 128, kvh * HD);
+        tma_load_2d(v_smem + kVTile, &map_vt, v_full, pv + jt * 128 + 64, kvh * HD);
       }
     }
   } else if (warp == 1) {
@@ -474,11 +499,17 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     bool ok = true;
     // biased scores: the table entries of this warp's rows and the block's keys, distance first + w - 127 at window[w]
     float* window = reinterpret_cast<float*>(bars_gen + 8 * kBars + 16) + q * kBiasWindow;
-    const float* bias = SCORE != kPlain ? ext.bias + (size_t)h * (ext.far + 1) : nullptr;
-    const float far_bias = SCORE != kPlain ? __ldg(bias + ext.far) : 0.0f;
+    const float* bias = nullptr;
+    float far_bias = 0.0f;
+    if constexpr (BIASED) {
+      bias = ext.bias + (size_t)h * (ext.far + 1);
+      far_bias = __ldg(bias + ext.far);
+    }
+    if constexpr (SCORE == kWindowed)
+      if (ext.sink) { m = 0.0f; l = 1.0f; }  // a further score of 0, without a value
     for (int j = 0; j < nb; ++j) {
       bool near = false;
-      if (SCORE != kPlain) {
+      if constexpr (BIASED) {
         const int first = q_off + q0 + q * 32 - j * 128;
         near = first - 127 < ext.far || first < 256;  // masked blocks read the window too
         if (near) {
@@ -488,14 +519,26 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           __syncwarp();
         }
       }
-      auto score = [&](uint32_t raw, int key) { return ext.score(__uint_as_float(raw), near ? window[lane + 127 - key] : far_bias); };
+      auto score = [&](uint32_t raw, int key) {
+        if constexpr (BIASED) return ext.score(__uint_as_float(raw), near ? window[lane + 127 - key] : far_bias);
+        else return 0.0f;
+      };
       if (!mbar_wait_warp(s_full, (uint32_t)j & 1u, abort_flag)) { ok = false; break; }
       tc_fence_after();
       // keys this row may see in this block: [0, lim)
       int lim = kv_len - j * 128;
       if (CAUSAL) lim = min(lim, q_off + q0 + row + 1 - j * 128);
-      const bool full = lim >= 128;
-      if (SCORE == kBounded || SCORE == kPoly) {
+      bool full = lim >= 128;
+      int lo = 0, keep = 0;  // and of these [lo, lim) and [0, keep)
+      if constexpr (SCORE == kWindowed) {
+        const int jt = j >= kept ? j + skip : j, base = jt * 128 + (jt >= kept ? gap : 0), at = q_off + q0 + row;  // key 0's position
+        lim = min(kv_len, at + 1) - base;
+        lo = ext.size <= at ? at - ext.size + 1 - base : 0;
+        keep = ext.keep - base;
+        full = lim >= 128 && (lo <= 0 || keep >= 128);
+      }
+      auto seen = [&](int key) { return key < lim && (SCORE != kWindowed || key >= lo || key < keep); };
+      if constexpr (SCORE == kBounded || SCORE == kPoly) {
         constexpr int S = SCORE == kPoly ? kPoly : kBounded;
         // every lane of a warp takes the same branch: TMEM accesses are warp-wide
         if (!__all_sync(0xffffffffu, full)) l += bounded_block<S, true, false>(t_s, ext, window + lane, far_bias, lim);
@@ -526,14 +569,14 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            if (c2 * 64 + i < lim) mx = fmaxf(mx, __uint_as_float(ra[i]));
-            if (c2 * 64 + 32 + i < lim) mx = fmaxf(mx, __uint_as_float(rb[i]));
+            if (seen(c2 * 64 + i)) mx = fmaxf(mx, __uint_as_float(ra[i]));
+            if (seen(c2 * 64 + 32 + i)) mx = fmaxf(mx, __uint_as_float(rb[i]));
           }
         }
       }
       // The maximum only moves when it would grow by more than 2^8: P then stays below 256 (exact
       // enough in bf16, summed in fp32) and O is rescaled far less often.
-      const float cand = SCORE == kPlain ? mx * sl2 : mx;
+      const float cand = BIASED ? mx : mx * sl2;
       float alpha = 1.0f;
       if (cand > m + 8.0f) { alpha = fast_exp2(m - cand); m = cand; }
       float sum = 0.0f;
@@ -543,7 +586,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         tc_ld32(t_s + c2 * 64, ra);
         tc_ld32(t_s + c2 * 64 + 32, rb);
         tc_wait_ld();
-        if (SCORE != kPlain) {
+        if (BIASED) {
           auto prob = [&](uint32_t raw, int key) {
             const float e = fast_exp2(score(raw, key) - m);
             return full || key < lim ? e : 0.0f;
@@ -569,10 +612,10 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
             const int ka = c2 * 64 + i, kb = ka + 32;
-            const float a0 = ka < lim ? fast_exp2(fmaf(__uint_as_float(ra[i]), sl2, -m)) : 0.0f;
-            const float a1 = ka + 1 < lim ? fast_exp2(fmaf(__uint_as_float(ra[i + 1]), sl2, -m)) : 0.0f;
-            const float b0 = kb < lim ? fast_exp2(fmaf(__uint_as_float(rb[i]), sl2, -m)) : 0.0f;
-            const float b1 = kb + 1 < lim ? fast_exp2(fmaf(__uint_as_float(rb[i + 1]), sl2, -m)) : 0.0f;
+            const float a0 = seen(ka) ? fast_exp2(fmaf(__uint_as_float(ra[i]), sl2, -m)) : 0.0f;
+            const float a1 = seen(ka + 1) ? fast_exp2(fmaf(__uint_as_float(ra[i + 1]), sl2, -m)) : 0.0f;
+            const float b0 = seen(kb) ? fast_exp2(fmaf(__uint_as_float(rb[i]), sl2, -m)) : 0.0f;
+            const float b1 = seen(kb + 1) ? fast_exp2(fmaf(__uint_as_float(rb[i + 1]), sl2, -m)) : 0.0f;
             sum += (a0 + a1) + (b0 + b1);
             v[i >> 1] = pack_bf16x2(a0, a1);
             v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
@@ -602,8 +645,10 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     }
     if (ok && mbar_wait_warp(o_done, 0u, abort_flag)) {
       tc_fence_after();
-      const float inv = 1.0f / l;
+      float inv = 1.0f / l;
       const bool store = q0 + row < len;
+      if constexpr (SCORE == kWindowed)
+        if (store) inv *= ext.head_gate((size_t)(t0 + q0 + row), h);
       __nv_bfloat16* dst = out + (size_t)(t0 + q0 + row) * (size_t)out_stride + h * HD;
 #pragma unroll
       for (int c = 0; c < HD / 32; ++c) {
@@ -611,7 +656,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         tc_ld32(t_o + c * 32, r);
         tc_wait_ld();
         if (store) {
-          if (SCORE != kPlain) {  // the output gate
+          if constexpr (BIASED) {  // the output gate
             const uint4* gp = reinterpret_cast<const uint4*>(ext.gate + (size_t)(t0 + q0 + row) * ext.ld_gate + h * HD + c * 32);
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
@@ -749,10 +794,10 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
                                    const void* v_pool, const void* block_tables, int32_t max_blocks, int32_t n_pool_blocks, void* out,
                                    void* scratch, int32_t n_q_tokens, int32_t total_kv_tokens, int32_t n_seqs, int32_t max_q_len,
                                    int32_t max_kv_len, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, bool turbo3, void* status,
-                                   void* stream, const ScoreExt* ext = nullptr, int score = kPlain) {
+                                   void* stream, const ScoreExt* ext = nullptr, int score = kPlain, const WindowExt* win = nullptr, float scale = 0.0f) {
   const int D = head_dim;
   if (n_q_tokens < 0 || total_kv_tokens < 0 || n_seqs < 0 || max_q_len < 0 || max_kv_len < 0 || max_blocks <= 0 ||
-      n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 || (D != 128 && D != 256 && !(D == 64 && ext)) || (n_heads % n_kv_heads) ||
+      n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 || (D != 128 && D != 256 && !(D == 64 && (ext || win))) || (n_heads % n_kv_heads) ||
       (q_row_stride % 8) || n_heads * D > q_row_stride || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
       ((uintptr_t)k_pool & (turbo3 ? 7 : 15)) || ((uintptr_t)v_pool & (turbo3 ? 7 : 15)) || !scratch || ((uintptr_t)scratch & 255) || !kv_lens ||
       !block_tables || max_kv_len > total_kv_tokens)
@@ -773,30 +818,37 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
   const int64_t blocks = (int64_t)tx * n_kv_heads * n_seqs;
   if (blocks > 0x7fffffff) return lg::kInvalidValue;
   if (blocks > 0) {
-    auto go = [&](auto kern, auto* kp, auto* vp) {
+    auto go = [&](auto kern, auto* kp, auto* vp, auto... more) {
       lg::launch(kern, dim3((unsigned)blocks), dim3(256), 0, s, kp, vp, (const int*)block_tables, max_blocks, n_pool_blocks, (const int*)kv_lens, kbuf, vt, pstart,
-                                            n_seqs, tp, tx, n_kv_heads, (int*)status);
+                                            n_seqs, tp, tx, n_kv_heads, more..., (int*)status);
     };
+    const GatherWindow gw = win ? GatherWindow{(const int*)cu_seqlens_q, win->size, win->keep} : GatherWindow{};
     if (turbo3) {
       if (D == 128) go(gather_paged_kv_turbo3_kernel<128>, (const uint8_t*)k_pool, (const uint8_t*)v_pool);
       else go(gather_paged_kv_turbo3_kernel<256>, (const uint8_t*)k_pool, (const uint8_t*)v_pool);
     } else {
-      if (D == 64) go(gather_paged_kv_kernel<64>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool);
-      else if (D == 128) go(gather_paged_kv_kernel<128>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool);
-      else go(gather_paged_kv_kernel<256>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool);
+      if (D == 64) go(gather_paged_kv_kernel<64>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, gw);
+      else if (D == 128) go(gather_paged_kv_kernel<128>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, gw);
+      else go(gather_paged_kv_kernel<256>, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, gw);
     }
     uint32_t rc = lg::launch_status();
     if (rc) return rc;
   }
-  const float sl2 = 1.4426950408889634f / sqrtf((float)D);
+  const float sl2 = win ? 1.4426950408889634f * scale : 1.4426950408889634f / sqrtf((float)D);
+  const int ld_out = win ? win->ld_out : ext ? ext->ld_out : n_heads * D;
   dim3 grid((max_q_len + 127) / 128, n_heads, n_seqs);
-  auto launch = [&](auto kern, size_t smem) -> uint32_t {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (uint32_t)e;
-    lg::launch(kern, grid, dim3(192), smem, s, map_q, map_k, map_vt, (const int*)cu_seqlens_q, pstart, (const int*)kv_lens, (__nv_bfloat16*)out,
-                                 ext ? ext->ld_out : n_heads * D, n_heads, n_kv_heads, 0, sl2, ext ? *ext : ScoreExt{}, (int*)status);
+  auto launch_ext = [&](auto kern, size_t smem, const auto& e) -> uint32_t {
+    cudaError_t rc = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (rc != cudaSuccess) return (uint32_t)rc;
+    lg::launch(kern, grid, dim3(192), smem, s, map_q, map_k, map_vt, (const int*)cu_seqlens_q, pstart, (const int*)kv_lens, (__nv_bfloat16*)out, ld_out, n_heads,
+               n_kv_heads, 0, sl2, e, (int*)status);
     return lg::launch_status();
   };
+  auto launch = [&](auto kern, size_t smem) { return launch_ext(kern, smem, ext ? *ext : ScoreExt{}); };
+  if (win)
+    return D == 64 ? launch_ext(attn_tcgen05_kernel<true, 64, kWindowed>, Attn<64>::kSmem, *win)
+         : D == 128 ? launch_ext(attn_tcgen05_kernel<true, 128, kWindowed>, Attn<128>::kSmem, *win)
+                    : launch_ext(attn_tcgen05_kernel<true, 256, kWindowed>, Attn<256>::kSmem, *win);
   if (ext) {
     constexpr size_t kWindow = 4 * kBiasWindow * 4;
     if (score == kPoly)
@@ -853,16 +905,28 @@ uint32_t logismos_launch_bias_attention_prefix_bf16(const void* q, int32_t ld_q,
                             !bounded ? kBiased : fit_score_poly(score, &ext) ? kPoly : kBounded);
 }
 
+uint32_t logismos_launch_window_attention_prefix_bf16(const void* q, int32_t ld_q, const void* cu_seqlens_q, const void* kv_lens, const void* k_pool,
+                                                      const void* v_pool, const void* block_tables, int32_t max_blocks, int32_t n_pool_blocks, void* out,
+                                                      int32_t ld_out, void* scratch, int32_t n_q_tokens, int32_t total_keys, int32_t n_seqs,
+                                                      int32_t max_q_len, int32_t max_keys, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
+                                                      const lg_window_t* window, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (n_heads <= 0 || !window_ok(window, n_heads) || (ld_out % 8) || ld_out < n_heads * head_dim) return lg::kInvalidValue;
+  const WindowExt win = window_ext(window, ld_q, ld_out);
+  return launch_prefix_attn(q, ld_q, cu_seqlens_q, kv_lens, k_pool, v_pool, block_tables, max_blocks, n_pool_blocks, out, scratch, n_q_tokens, total_keys, n_seqs,
+                            max_q_len, max_keys, n_heads, n_kv_heads, head_dim, false, status, stream, nullptr, kPlain, &win, window->scale);
+}
+
 uint32_t logismos_launch_varlen_attention_kv_tc_bf16(const void* q, int32_t q_row_stride, const void* cu_seqlens_q, const void* kv_lens,
                                                      const void* kv_start, const void* k, const void* v_t, int32_t n_kv_rows, void* out,
                                                      int32_t out_row_stride, int32_t n_q_tokens, int32_t n_seqs, int32_t max_q_len,
-                                                     int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, float scale, void* status,
-                                                     void* stream) {
+                                                     int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, float scale, const void* gate,
+                                                     int32_t ld_gate, void* status, void* stream) {
   lg::LaunchScope launch_scope_;
   const int D = head_dim;
   if (n_q_tokens < 0 || n_seqs < 0 || max_q_len < 0 || n_kv_rows <= 0 || (n_kv_rows % 8) || n_heads <= 0 || n_kv_heads <= 0 ||
       (n_heads % n_kv_heads) || (D != 64 && D != 128 && D != 256) || (q_row_stride % 8) || n_heads * D > q_row_stride ||
-      (out_row_stride % 8) || n_heads * D > out_row_stride || !(scale > 0.0f) || !q || !k || !v_t || !out || !cu_seqlens_q || !kv_lens ||
+      (out_row_stride % 8) || n_heads * D > out_row_stride || !(scale > 0.0f) || (gate && ld_gate < n_heads) || !q || !k || !v_t || !out || !cu_seqlens_q || !kv_lens ||
       !kv_start || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v_t | (uintptr_t)out) & 15))
     return lg::kInvalidValue;
   if (n_seqs == 0 || max_q_len == 0 || n_q_tokens == 0) return 0;
@@ -873,16 +937,23 @@ uint32_t logismos_launch_varlen_attention_kv_tc_bf16(const void* q, int32_t q_ro
       !make_map(&map_vt, v_t, (uint64_t)row_w, (uint64_t)n_kv_rows, (uint64_t)n_kv_rows, (uint32_t)D))
     return lg::kInvalidValue;
   dim3 grid((max_q_len + 127) / 128, n_heads, n_seqs);
-  auto launch = [&](auto kern, size_t smem) -> uint32_t {
+  auto launch = [&](auto kern, size_t smem, const auto& ext) -> uint32_t {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (uint32_t)e;
     lg::launch(kern, grid, dim3(192), smem, (cudaStream_t)stream, map_q, map_k, map_vt, (const int*)cu_seqlens_q, (const int*)kv_start, (const int*)kv_lens,
-               (__nv_bfloat16*)out, out_row_stride, n_heads, n_kv_heads, 0, scale * 1.4426950408889634f, ScoreExt{}, (int*)status);
+               (__nv_bfloat16*)out, out_row_stride, n_heads, n_kv_heads, 0, scale * 1.4426950408889634f, ext, (int*)status);
     return lg::launch_status();
   };
-  if (D == 64) return launch(attn_tcgen05_kernel<true, 64>, Attn<64>::kSmem);
-  if (D == 128) return launch(attn_tcgen05_kernel<true, 128>, Attn<128>::kSmem);
-  return launch(attn_tcgen05_kernel<true, 256>, Attn<256>::kSmem);
+  if (gate) {
+    const WindowExt all{0x7fffffff, 0, 0, (const float*)gate, ld_gate, q_row_stride, out_row_stride};
+    if (D == 64) return launch(attn_tcgen05_kernel<true, 64, kWindowed>, Attn<64>::kSmem, all);
+    if (D == 128) return launch(attn_tcgen05_kernel<true, 128, kWindowed>, Attn<128>::kSmem, all);
+    return launch(attn_tcgen05_kernel<true, 256, kWindowed>, Attn<256>::kSmem, all);
+  }
+  const ScoreExt none{};
+  if (D == 64) return launch(attn_tcgen05_kernel<true, 64>, Attn<64>::kSmem, none);
+  if (D == 128) return launch(attn_tcgen05_kernel<true, 128>, Attn<128>::kSmem, none);
+  return launch(attn_tcgen05_kernel<true, 256>, Attn<256>::kSmem, none);
 }
 
 }  // extern "C"

@@ -1,5 +1,5 @@
-// What the capped, distance-biased attention needs around the shared attention kernels: unit queries and keys with
-// the cache store, and the fp32 form of the attention itself.
+// What the extended forms of attention (score_bias.cuh) need around the shared attention kernels: unit queries and keys
+// with the cache store, and the fp32 attention, capped and biased by distance or over a window.
 #include "common.cuh"
 #include "logismos_kernels.h"
 #include "recurrent.cuh"
@@ -83,21 +83,24 @@ unit_qk_store_kernel(QkArgs p) {
 
 // CTA = (row, head), keys in tiles of 64
 constexpr int kTile = 64, kAttnThreads = 128;
+template <bool WINDOW>
 __global__ void __launch_bounds__(kAttnThreads)
-bias_attention_f32_kernel(const float* __restrict__ q, const float* __restrict__ kpool, const float* __restrict__ vpool, const int* __restrict__ tables,
-                          int max_blocks, int n_pool_blocks, const int* __restrict__ seq_ids, const int* __restrict__ pos, float* __restrict__ out,
-                          int n_kv, int hd, float scale, float cap, const float* __restrict__ gate, ScoreExt ext, int* __restrict__ status) {
+attention_f32_kernel(const float* __restrict__ q, const float* __restrict__ kpool, const float* __restrict__ vpool, const int* __restrict__ tables,
+                     int max_blocks, int n_pool_blocks, const int* __restrict__ seq_ids, const int* __restrict__ pos, float* __restrict__ out,
+                     int n_kv, int hd, float scale, float cap, const float* __restrict__ gate, ScoreExt ext, WindowExt win, int* __restrict__ status) {
   lg::pdl_prologue();
   __shared__ float sq[256], ss[kTile], red[32];
   __shared__ int blk_s[kTile / kBlockTokens];
   const int r = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int kvh = h / (gridDim.y / n_kv), n_keys = pos[r] + 1;
   const int* table = tables + (size_t)seq_ids[r] * max_blocks;
-  const float* bias = ext.bias + (size_t)h * (ext.far + 1);
+  const float* bias = WINDOW ? nullptr : ext.bias + (size_t)h * (ext.far + 1);
   const size_t row_w = (size_t)n_kv * hd;
-  for (int i = tid; i < hd; i += kAttnThreads) sq[i] = q[(size_t)r * ext.ld_q + h * hd + i];
-  float m = -1e30f, l = 0.0f, acc[2] = {0.f, 0.f};
+  for (int i = tid; i < hd; i += kAttnThreads) sq[i] = q[(size_t)r * (WINDOW ? win.ld_q : ext.ld_q) + h * hd + i];
+  const bool sink = WINDOW && win.sink;  // a further score of 0
+  float m = sink ? 0.0f : -1e30f, l = sink ? 1.0f : 0.0f, acc[2] = {0.f, 0.f};
   for (int k0 = 0; k0 < n_keys; k0 += kTile) {
+    if (WINDOW && k0 >= win.keep && n_keys - 1 - (k0 + kTile - 1) >= win.size) continue;  // a tile that is not seen
     const int n = min(kTile, n_keys - k0);
     __syncthreads();
     if (tid < kTile / kBlockTokens) {
@@ -118,6 +121,10 @@ bias_attention_f32_kernel(const float* __restrict__ q, const float* __restrict__
         for (int i = lane; i < hd; i += 32) s = fmaf(sq[i], c[i], s);
       }
       s = warp_sum(s) * scale;
+      if (WINDOW) {
+        if (lane == 0) ss[k] = k < n && b >= 0 && win.sees(n_keys - 1, k0 + k) ? s * 1.4426950408889634f : -INFINITY;
+        continue;
+      }
       if (cap > 0.0f) s = cap * tanhf(s / cap);
       if (lane == 0) ss[k] = k < n && b >= 0 ? s * 1.4426950408889634f + bias[min(n_keys - 1 - (k0 + k), ext.far)] : -1e30f;
     }
@@ -139,10 +146,16 @@ bias_attention_f32_kernel(const float* __restrict__ q, const float* __restrict__
       if (tid + kAttnThreads < hd) acc[1] = fmaf(ss[k], c[tid + kAttnThreads], acc[1]);
     }
   }
+  if constexpr (WINDOW) {
+    const float g = win.gate ? rec::sigmoid_f(win.gate[(size_t)r * win.ld_gate + h]) : 1.0f;
+    if (tid < hd) out[(size_t)r * win.ld_out + h * hd + tid] = acc[0] / l * g;
+    if (tid + kAttnThreads < hd) out[(size_t)r * win.ld_out + h * hd + tid + kAttnThreads] = acc[1] / l * g;
+  } else {
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int d = tid + i * kAttnThreads;
-    if (d < hd) out[(size_t)r * ext.ld_out + h * hd + d] = acc[i] / l * (ext.gate_scale * rec::sigmoid_f(gate[(size_t)r * ext.ld_gate + h * hd + d]));
+    for (int i = 0; i < 2; ++i) {
+      const int d = tid + i * kAttnThreads;
+      if (d < hd) out[(size_t)r * ext.ld_out + h * hd + d] = acc[i] / l * (ext.gate_scale * rec::sigmoid_f(gate[(size_t)r * ext.ld_gate + h * hd + d]));
+    }
   }
 }
 
@@ -186,9 +199,24 @@ uint32_t logismos_launch_bias_attention_f32(const void* q, int32_t ld_q, const v
       !score_ok(score, n_heads * head_dim))
     return lg::kInvalidValue;
   const ScoreExt ext = score_ext(score, ld_q, ld_out);
-  lg::launch(bias_attention_f32_kernel, dim3((unsigned)rows, (unsigned)n_heads), dim3(kAttnThreads), 0, (cudaStream_t)stream, (const float*)q, (const float*)k_pool,
+  lg::launch(attention_f32_kernel<false>, dim3((unsigned)rows, (unsigned)n_heads), dim3(kAttnThreads), 0, (cudaStream_t)stream, (const float*)q, (const float*)k_pool,
              (const float*)v_pool, (const int*)block_tables, max_blocks, n_pool_blocks, (const int*)seq_ids_i32, (const int*)positions_i32, (float*)out, n_kv_heads,
-             head_dim, score->scale, score->cap, (const float*)score->gate, ext, (int*)status_i32);
+             head_dim, score->scale, score->cap, (const float*)score->gate, ext, WindowExt{}, (int*)status_i32);
+  return lg::launch_status();
+}
+
+uint32_t logismos_launch_window_attention_f32(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables,
+                                              const void* seq_ids_i32, const void* positions_i32, void* out, int32_t ld_out, int32_t rows,
+                                              int32_t max_blocks, int32_t n_pool_blocks, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim,
+                                              const lg_window_t* window, void* status_i32, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!q || !k_pool || !v_pool || !block_tables || !seq_ids_i32 || !positions_i32 || !out || rows <= 0 || max_blocks <= 0 || n_pool_blocks <= 0 || n_heads <= 0 ||
+      n_heads > 65535 || n_kv_heads <= 0 || n_heads % n_kv_heads || head_dim <= 0 || head_dim > 256 || ld_q < n_heads * head_dim || ld_out < n_heads * head_dim ||
+      !window_ok(window, n_heads))
+    return lg::kInvalidValue;
+  lg::launch(attention_f32_kernel<true>, dim3((unsigned)rows, (unsigned)n_heads), dim3(kAttnThreads), 0, (cudaStream_t)stream, (const float*)q, (const float*)k_pool,
+             (const float*)v_pool, (const int*)block_tables, max_blocks, n_pool_blocks, (const int*)seq_ids_i32, (const int*)positions_i32, (float*)out, n_kv_heads,
+             head_dim, window->scale, 0.0f, (const float*)nullptr, ScoreExt{}, window_ext(window, ld_q, ld_out), (int*)status_i32);
   return lg::launch_status();
 }
 

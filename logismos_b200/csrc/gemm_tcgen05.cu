@@ -18,6 +18,8 @@
 // No cluster launch and no multicast is used: each CTA fetches its own tiles.
 #include <cuda.h>
 
+#include <algorithm>
+
 #include "common.cuh"
 #include "logismos_kernels.h"
 #include "tcgen05.cuh"
@@ -70,12 +72,20 @@ LG_DEVINL int group_of(const lg_linear_groups_t& g, int c) {
   return i;
 }
 
-template <int BN, int EPI>
+// One matrix per group of rows (EXPERTS): the row tiles are listed on the device; map_out then describes the activations
+// that some groups read directly.
+struct RowTiles {
+  const int4* tiles;   // group, first output row, last + 1, -1 - input row of map_out or any other value: the input row is the output row
+  const int* n_tiles;
+  int direct;          // 0: no group reads map_out
+};
+
+template <int BN, int EPI, bool EXPERTS = false>
 __global__ void __launch_bounds__(kThreads, 1)
 linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                         const __grid_constant__ CUtensorMap map_out, const float* __restrict__ bias,
                         void* __restrict__ out, int M, int N, int K, int ldc, int splits, int w_static,
-                        EpiParams ep, const lg_linear_groups_t groups, int* __restrict__ status) {
+                        EpiParams ep, const lg_linear_groups_t groups, const RowTiles row_tiles, int* __restrict__ status) {
   using C = Cfg<BN>;
   lg::pdl_trigger();
   extern __shared__ uint8_t smem_raw[];
@@ -93,7 +103,8 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
   volatile int* abort_flag = reinterpret_cast<volatile int*>(bars_gen + 8 * (2 * C::kStages + 4) + 8);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int m_tiles = (M + BM - 1) / BM, n_tiles = (N + BN - 1) / BN;
+  if (EXPERTS) lg::pdl_wait();  // the tile list is the work of a kernel of this step
+  const int m_tiles = EXPERTS ? *row_tiles.n_tiles : (M + BM - 1) / BM, n_tiles = (N + BN - 1) / BN;
   // a work item is (k slice, output tile); slices of k exist only for the accumulating epilogue, whose
   // reduce-add makes them meet in the output
   const int out_tiles = m_tiles * n_tiles;
@@ -121,7 +132,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
       tma_load_2d(smem_base + pre_w * C::kStage + C::kStageA, &map_w, full_bar(pre_w), kb * BK, n_blk * BN);
     }
   }
-  lg::pdl_wait();  // everything before this touched shared memory or read the static weights only
+  if (!EXPERTS) lg::pdl_wait();  // everything before this touched shared memory or read the static weights only
   if (warp == 1) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_u32((const void*)tmem_slot)), "r"((uint32_t)C::kTmemCols) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
@@ -142,14 +153,22 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
         const int m_blk = ot % m_tiles, n_blk = ot / m_tiles;
         const int kb0 = sp * kb_per, kb1 = min(all_kb, kb0 + kb_per);
         // a tile lies in one group of columns; rows beyond M read the next copy's and are not stored
-        const int a_row = m_blk * BM + (EPI == kEpiGroups ? group_of(groups, n_blk * BN) * M : 0);
+        int a_row = m_blk * BM + (EPI == kEpiGroups ? group_of(groups, n_blk * BN) * M : 0), w_row = n_blk * BN;
+        const CUtensorMap* a_map = &map_a;
+        if (EXPERTS) {
+          const int4 rt = row_tiles.tiles[m_blk];
+          w_row += rt.x * N;
+          const bool direct = row_tiles.direct && rt.w < 0;
+          a_row = direct ? -1 - rt.w : rt.y;
+          if (direct) a_map = &map_out;
+        }
         for (int kb = kb0; kb < kb1; ++kb) {
           if (!mbar_wait(empty_bar(stage), phase ^ 1u, abort_flag)) { ok = false; break; }
           const bool have_w = pre_w > 0;  // requested before the dependency wait (first stages of the first tile)
           if (!have_w) mbar_expect_tx(full_bar(stage), (uint32_t)C::kStage);
           const uint32_t sa = smem_base + stage * C::kStage;
-          tma_load_2d(sa, &map_a, full_bar(stage), kb * BK, a_row);
-          if (!have_w) tma_load_2d(sa + C::kStageA, &map_w, full_bar(stage), kb * BK, n_blk * BN);
+          tma_load_2d(sa, a_map, full_bar(stage), kb * BK, a_row);
+          if (!have_w) tma_load_2d(sa + C::kStageA, &map_w, full_bar(stage), kb * BK, w_row);
           else --pre_w;
           if (++stage == C::kStages) { stage = 0; phase ^= 1u; }
         }
@@ -222,8 +241,9 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
       const uint32_t acc_phase = (uint32_t)(it >> 1) & 1u;
       if (!mbar_wait_warp(tfull_bar(buf), acc_phase, abort_flag)) { ok = false; break; }
       tc_fence_after();
-      const int row0 = m_blk * BM + q * 32;  // first output row of this warp's slab
-      const int row = row0 + lane;
+      const int4 rt = EXPERTS ? row_tiles.tiles[m_blk] : make_int4(0, m_blk * BM, M, 0);
+      const int row0 = rt.y + q * 32;  // first output row of this warp's slab
+      const int row = row0 + lane, row_end = rt.z;
       const uint32_t t_row = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(buf * BN);
       if (EPI == LG_EPI_RESID_F32) {
         for (int c = 0; c < BN; c += 32) {
@@ -248,7 +268,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
           tc_wait_ld();
           const int ncol = n_blk * BN + c;
           if (EPI == kEpiGroups && ncol >= groups.n_main) {
-            if (row < M) {
+            if (row < row_end) {
               const int c0 = ncol - groups.n_main, width = N - groups.n_main;
               float* dst = reinterpret_cast<float*>(groups.tail) + (size_t)row * groups.ld_tail + c0;
               __nv_bfloat16* parts = reinterpret_cast<__nv_bfloat16*>(groups.tail_parts) + (size_t)row * 2 * width + c0;
@@ -267,7 +287,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
             }
             continue;
           }
-          if (row < M) {
+          if (row < row_end) {
               __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * ldc + ncol;
 #pragma unroll
               for (int j = 0; j < 4; ++j) {
@@ -313,7 +333,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
           tc_ld32(t_row + c, r);
           tc_wait_ld();
           const int ncol = n_blk * BN + c;
-          if (row < M) {
+          if (row < row_end) {
             float* dst = reinterpret_cast<float*>(out) + (size_t)row * ldc + ncol;
 #pragma unroll
             for (int j = 0; j < 32; j += 4) {
@@ -338,7 +358,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
           tc_wait_ld();
           const int ncol = n_blk * BN + c;        // column of the gate block in W-row space
           const int ocol = ncol >> 1;             // output column
-          if (row < M && ncol < N) {
+          if (row < row_end && ncol < N) {
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * ldc + ocol;
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
@@ -434,7 +454,7 @@ uint32_t launch_cfg(const void* a, const void* w, const float* bias, void* out, 
   }
   const int items = tiles * splits;
   const int grid = items < sm_count() ? items : sm_count();
-  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, mo, bias, out, m, n, k, ldc, splits, w_static, ep, groups, status);
+  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, mo, bias, out, m, n, k, ldc, splits, w_static, ep, groups, RowTiles{}, status);
   return lg::launch_status();
 }
 
@@ -465,9 +485,62 @@ uint32_t launch_epi(const void* a, const void* w, const float* bias, void* out, 
   return launch_cfg<128, EPI>(a, w, bias, out, m, n, k, lda, ldc, w_static, ep, status, stream, groups);
 }
 
+struct ExpertRows {
+  const void* a;
+  int a_rows;
+  const void* direct;
+  int direct_rows;
+  RowTiles tiles;
+  int max_tiles, groups;
+};
+
+template <int BN, int EPI>
+uint32_t launch_experts(const ExpertRows& x, const void* w, void* out, int n, int k, int lda, int ldc, int* status, cudaStream_t stream) {
+  CUtensorMap ma, md, mw;
+  if (!make_map(&ma, x.a, (uint64_t)x.a_rows, (uint64_t)k, (uint64_t)lda, BM)) return lg::kInvalidValue;
+  if (x.direct) {
+    if (!make_map(&md, x.direct, (uint64_t)x.direct_rows, (uint64_t)k, (uint64_t)lda, BM)) return lg::kInvalidValue;
+  } else {
+    md = ma;
+  }
+  if (!make_map(&mw, w, (uint64_t)n * x.groups, (uint64_t)k, (uint64_t)k, BN)) return lg::kInvalidValue;
+  auto kern = linear_t_tcgen05_kernel<BN, EPI, true>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg<BN>::kSmem);
+  if (e != cudaSuccess) return (uint32_t)e;
+  const int64_t items = (int64_t)x.max_tiles * ((n + BN - 1) / BN);
+  const int grid = items < sm_count() ? (int)items : sm_count();
+  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, md, (const float*)nullptr, out, x.a_rows, n, k, ldc, 1, 0, EpiParams{}, lg_linear_groups_t{},
+             x.tiles, status);
+  return lg::launch_status();
+}
+
+// tile width as in launch_epi; the number of row tiles is only bounded here, about half of the partial ones are counted
+template <int EPI>
+uint32_t launch_experts_epi(const ExpertRows& x, const void* w, void* out, int n, int k, int lda, int ldc, int* status, cudaStream_t stream) {
+  const int64_t mt = std::max(1, x.max_tiles - x.groups / 2), sms = sm_count();
+  auto cost = [&](int bn) { return (mt * ((n + bn - 1) / bn) + sms - 1) / sms * bn; };
+  return cost(128) < cost(256) ? launch_experts<128, EPI>(x, w, out, n, k, lda, ldc, status, stream) : launch_experts<256, EPI>(x, w, out, n, k, lda, ldc, status, stream);
+}
+
 }  // namespace
 
 extern "C" {
+
+uint32_t logismos_launch_linear_experts_tc_bf16(const void* a, int32_t a_rows, const void* a_direct, int32_t direct_rows, const void* w, void* out,
+                                                const void* tiles, const void* n_tiles, int32_t max_tiles, int32_t n_groups, int32_t n, int32_t k,
+                                                int32_t lda, int32_t ldc, int32_t epilogue, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  epilogue &= ~LG_EPI_STATIC_W;
+  const bool glu = epilogue == LG_EPI_SWIGLU;
+  if (!a || a_rows <= 0 || !w || !out || !tiles || !n_tiles || max_tiles <= 0 || n_groups <= 0 || n <= 0 || n % (glu ? 64 : 16) || k <= 0 || k % BK || lda < k || lda % 8 ||
+      ldc % 8 || ldc < (glu ? n / 2 : n) || (a_direct && direct_rows <= 0) || (int64_t)n * n_groups > 0x7fffffff ||
+      (((uintptr_t)a | (uintptr_t)a_direct | (uintptr_t)w | (uintptr_t)out | (uintptr_t)tiles) & 15))
+    return lg::kInvalidValue;
+  const ExpertRows x{a, a_rows, a_direct, direct_rows, RowTiles{(const int4*)tiles, (const int*)n_tiles, a_direct ? 1 : 0}, max_tiles, n_groups};
+  if (glu) return launch_experts_epi<LG_EPI_SWIGLU>(x, w, out, n, k, lda, ldc, (int*)status, (cudaStream_t)stream);
+  if (epilogue == LG_EPI_BF16) return launch_experts_epi<LG_EPI_BF16>(x, w, out, n, k, lda, ldc, (int*)status, (cudaStream_t)stream);
+  return lg::kInvalidValue;
+}
 
 uint32_t logismos_launch_linear_t_act_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m,
                                            int32_t n, int32_t k, int32_t lda, int32_t ldc, int32_t epilogue, float p0,
@@ -503,7 +576,7 @@ uint32_t logismos_launch_linear_groups_tc_bf16(const void* a, const void* w, voi
   if (m <= 0 || n <= 0 || k <= 0 || (k % BK) || (n % 16) || (lda % 8) || lda < k || (((uintptr_t)a | (uintptr_t)w | (uintptr_t)out) & 15) ||
       (ldc % 8) || !lg::groups_ok(groups, n, ldc))
     return lg::kInvalidValue;
-  return launch_epi<kEpiGroups>(a, w, nullptr, out, m, n, k, lda, ldc, 1, EpiParams{}, (int*)status_i32, (cudaStream_t)stream, *groups);
+  return launch_epi<kEpiGroups>(a, w, (const float*)groups->bias, out, m, n, k, lda, ldc, 1, EpiParams{}, (int*)status_i32, (cudaStream_t)stream, *groups);
 }
 
 uint32_t logismos_launch_linear_t_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m,

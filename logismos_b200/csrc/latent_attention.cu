@@ -1,7 +1,7 @@
-// Latent attention (keys and values are linear images of one cached row c of `rank` values per token, no
-// rotated part): the cache side and the decode side.
+// Latent attention (keys and values are linear images of one cached row c of `rank` values per token; a rotated key part
+// that all heads share is more columns of that row): the cache side and the decode side.
 //   latent_norm_store   RMS norms of the query latent and of the key/value latent from the fp32
-//                       projection; the latter goes to its paged-cache slot
+//                       projection; the latter goes to its paged-cache slot, with its rotated columns
 //   latent_gather       cached rows of whole sequences made contiguous (prefill expands them to keys and
 //                       values with GEMMs and runs the tcgen05 attention kernel)
 //   latent_decode       one query token per sequence in the latent space: with q'_h = W_uk,h^T q_h the
@@ -42,17 +42,25 @@ LG_DEVINL void store4(void* p, size_t i4, float4 v, bool f32) {
   else reinterpret_cast<uint2*>(p)[i4] = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
 }
 
+struct RotaryArgs {
+  const float2* table;   // [positions][pairs], NULL: no rotated columns
+  const int* pos;
+  int at, pairs;         // first rotated column of the key/value row (a multiple of 4)
+  float* gate;
+  int n_gate, ld_gate;
+};
+
 // warp = (row, half): half 0 the query latent (columns 0 .. qw), half 1 the key/value latent (qw .. qw + rw)
 __global__ void __launch_bounds__(kThreads)
 latent_norm_store_kernel(float* __restrict__ raw, int ld, const float* __restrict__ gain_q, const float* __restrict__ gain_c,
                          void* __restrict__ cq, void* __restrict__ pool, const int64_t* __restrict__ slots, int rows, int qw, int q_n,
-                         int rw, int r_n, float eps, int64_t n_pool_slots, int f32, int zero, int* __restrict__ status) {
+                         int rw, int r_n, float eps, int64_t n_pool_slots, int f32, int zero, RotaryArgs rot, int* __restrict__ status) {
   lg::pdl_prologue();
   const int id = (blockIdx.x * kThreads + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   const int row = id >> 1, half = id & 1;
   if (row >= rows) return;
   float4* src = reinterpret_cast<float4*>(raw + (size_t)row * ld + (half ? qw : 0));
-  const int nv = (half ? rw : qw) >> 2;
+  const int all = (half ? rw : qw) >> 2, nv = half && rot.table ? rot.at >> 2 : all;  // float4s, and the normed ones of them
   float ss = 0.0f;
   for (int v = lane; v < nv; v += 32) {
     const float4 a = src[v];
@@ -70,6 +78,21 @@ latent_norm_store_kernel(float* __restrict__ raw, int ld, const float* __restric
   }
   const float4* gain = reinterpret_cast<const float4*>(half ? gain_c : gain_q);
   void* out = half ? pool : cq;
+  if (half && rot.table) {
+    const float2* angles = rot.table + (size_t)rot.pos[row] * rot.pairs;
+    for (int v = nv + lane; v < all; v += 32) {
+      const int i = 2 * (v - nv);
+      const float4 a = src[v];
+      const float2 c0 = i < rot.pairs ? __ldg(angles + i) : make_float2(0.f, 0.f), c1 = i + 1 < rot.pairs ? __ldg(angles + i + 1) : make_float2(0.f, 0.f);
+      store4(out, dst + v, make_float4(a.x * c0.x - a.y * c0.y, a.y * c0.x + a.x * c0.y, a.z * c1.x - a.w * c1.y, a.w * c1.x + a.z * c1.y), f32 != 0);
+      if (zero) src[v] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    float* g = raw + (size_t)row * ld + qw + rw;
+    for (int h = lane; h < rot.n_gate; h += 32) {
+      rot.gate[(size_t)row * rot.ld_gate + h] = g[h];
+      if (zero) g[h] = 0.0f;
+    }
+  }
   for (int v = lane; v < nv; v += 32) {
     const float4 a = src[v], g = __ldg(gain + v);
     store4(out, dst + v, make_float4(a.x * inv * g.x, a.y * inv * g.y, a.z * inv * g.z, a.w * inv * g.w), f32 != 0);
@@ -126,8 +149,12 @@ struct DecodeArgs {
   float2* part_ml;            // [chunks, heads]
   int rows, heads, rank, chunk_tokens, max_blocks, n_pool_blocks;
   float sl2;
+  const float* gate;          // [rows, ld_gate], NULL: none
+  int ld_gate;
   int* status;
 };
+
+LG_DEVINL float head_gate(const float* gate, size_t row, int ld, int head) { return gate ? 1.0f / (1.0f + __expf(-gate[row * ld + head])) : 1.0f; }
 
 constexpr int kMaxStages = 4, kWarps = 8, kDecodeThreads = 32 * kWarps;
 
@@ -391,7 +418,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
         for (int hh = 0; hh < 2; ++hh) {
           const int hr = 16 * i + g + 8 * hh, h = h0 + hr;
           if (h >= p.heads) continue;
-          const float inv = 1.0f / s_l[hr];
+          const float inv = c_cnt == 1 ? head_gate(p.gate, r, p.ld_gate, h) / s_l[hr] : 0.0f;
 #pragma unroll
           for (int j = 0; j < 2 * MAXU; ++j) {
             if ((j >> 1) >= u_n) continue;
@@ -419,7 +446,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
 constexpr int kMergeTile = 256;
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml, const int* __restrict__ chunk_offsets,
-                    __nv_bfloat16* __restrict__ out, int heads, int rank) {
+                    __nv_bfloat16* __restrict__ out, int heads, int rank, const float* __restrict__ gate, int ld_gate) {
   lg::pdl_prologue();
   __shared__ float red[32], w[kMergeTile];
   const int h = blockIdx.x, r = blockIdx.y, tid = threadIdx.x;
@@ -453,7 +480,7 @@ latent_merge_kernel(const float* __restrict__ part_o, const float2* __restrict__
       }
     }
   }
-  const float inv = 1.0f / block_sum(l, red);
+  const float inv = head_gate(gate, r, ld_gate, h) / block_sum(l, red);
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int v = tid + i * 128;
@@ -466,7 +493,7 @@ constexpr int kF32Tile = 64;
 __global__ void __launch_bounds__(128)
 latent_attention_f32_kernel(const float* __restrict__ q, const float* __restrict__ pool, const int* __restrict__ tables, int max_blocks,
                             int n_pool_blocks, const int* __restrict__ seq_ids, const int* __restrict__ pos, float* __restrict__ out,
-                            int heads, int rank, float sl2, int* __restrict__ status) {
+                            int heads, int rank, float sl2, const float* __restrict__ gate, int ld_gate, int* __restrict__ status) {
   lg::pdl_prologue();
   extern __shared__ float fs[];  // q [rank], scores [kF32Tile]
   __shared__ float red[32];
@@ -522,7 +549,7 @@ latent_attention_f32_kernel(const float* __restrict__ q, const float* __restrict
         if (tid + i * 128 < rank) acc[i] = fmaf(w, c[tid + i * 128], acc[i]);
     }
   }
-  const float inv = 1.0f / l;
+  const float inv = (gate ? 1.0f / (1.0f + expf(-gate[(size_t)t * ld_gate + h])) : 1.0f) / l;
 #pragma unroll
   for (int i = 0; i < 8; ++i)
     if (tid + i * 128 < rank) out[row + tid + i * 128] = acc[i] * inv;
@@ -535,15 +562,22 @@ extern "C" {
 uint32_t logismos_launch_latent_norm_store(void* raw_f32, int32_t ld, const void* gain_q_f32, const void* gain_c_f32, void* q_latent,
                                            void* pool, const void* slot_mapping_i64, int32_t rows, int32_t q_width, int32_t q_n,
                                            int32_t c_width, int32_t c_n, float eps, int64_t n_pool_slots, int32_t is_f32,
-                                           int32_t zero_raw, void* status_i32, void* stream) {
+                                           int32_t zero_raw, const lg_latent_rotary_t* rotary, void* status_i32, void* stream) {
   lg::LaunchScope launch_scope_;
+  if (rotary && (!rotary->table || !rotary->positions || rotary->at <= 0 || rotary->at % 4 || c_n > rotary->at || rotary->dims <= 0 || rotary->dims % 2 ||
+                 rotary->at + rotary->dims > c_width || rotary->n_gate < 0 || (rotary->n_gate && (!rotary->gate || rotary->ld_gate < rotary->n_gate)) ||
+                 ld < q_width + c_width + rotary->n_gate || ((uintptr_t)rotary->table & 7)))
+    return lg::kInvalidValue;
+  const RotaryArgs rot = rotary ? RotaryArgs{(const float2*)rotary->table, (const int*)rotary->positions, rotary->at, rotary->dims / 2, (float*)rotary->gate, rotary->n_gate,
+                                             rotary->ld_gate}
+                                : RotaryArgs{};
   if (!raw_f32 || rows <= 0 || q_width <= 0 || c_width <= 0 || (q_width % 4) || (c_width % 4) || q_n <= 0 || q_n > q_width || c_n <= 0 ||
       c_n > c_width || ld < q_width + c_width || (ld % 4) || rows > 0x3fffffff)
     return lg::kInvalidValue;
   const int64_t blocks = ((int64_t)rows * 2 + kThreads / 32 - 1) / (kThreads / 32);
   lg::launch(latent_norm_store_kernel, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, (float*)raw_f32, ld,
              (const float*)gain_q_f32, (const float*)gain_c_f32, q_latent, pool, (const int64_t*)slot_mapping_i64, rows, q_width, q_n,
-             c_width, c_n, eps, n_pool_slots, is_f32, zero_raw, (int*)status_i32);
+             c_width, c_n, eps, n_pool_slots, is_f32, zero_raw, rot, (int*)status_i32);
   return lg::launch_status();
 }
 
@@ -596,16 +630,16 @@ size_t logismos_latent_decode_scratch_bytes(int32_t total_chunks, int32_t heads,
 uint32_t logismos_launch_latent_decode_bf16(const void* q, const void* pool, const void* block_tables_i32, const void* context_lens_i32,
                                             const void* chunk_offsets_i32, void* out, void* scratch, int32_t rows, int32_t total_chunks,
                                             int32_t chunk_tokens, int32_t max_blocks, int32_t n_pool_blocks, int32_t heads, int32_t rank,
-                                            float scale, void* status_i32, void* stream) {
+                                            float scale, const void* gate_f32, int32_t ld_gate, void* status_i32, void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!q || !pool || !out || !scratch || rows <= 0 || rows > 65535 || total_chunks < rows || chunk_tokens <= 0 || (chunk_tokens % 64) || max_blocks <= 0 ||
+  if ((gate_f32 && ld_gate < heads) || !q || !pool || !out || !scratch || rows <= 0 || rows > 65535 || total_chunks < rows || chunk_tokens <= 0 || (chunk_tokens % 64) || max_blocks <= 0 ||
       n_pool_blocks <= 0 || heads <= 0 || rank <= 0 || (rank % 64) || rank > 1024 || (int64_t)n_pool_blocks * kBlockTokens > 0x7fffffff - 64 ||
       (((uintptr_t)q | (uintptr_t)pool | (uintptr_t)out | (uintptr_t)scratch) & 15))
     return lg::kInvalidValue;
   cudaStream_t s = (cudaStream_t)stream;
   DecodeArgs p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, (const int*)block_tables_i32, (const int*)context_lens_i32,
                (const int*)chunk_offsets_i32, (__nv_bfloat16*)out, (float*)scratch, nullptr, rows, heads, rank, chunk_tokens, max_blocks,
-               n_pool_blocks, scale * kLog2e, (int*)status_i32};
+               n_pool_blocks, scale * kLog2e, (const float*)gate_f32, ld_gate, (int*)status_i32};
   p.part_ml = (float2*)(p.part_o + (size_t)total_chunks * heads * rank);
   CUtensorMap map;
   if (!make_map(&map, pool, (uint64_t)n_pool_blocks * kBlockTokens, (uint64_t)rank, (uint64_t)rank, kBlockTokens)) return lg::kInvalidValue;
@@ -625,26 +659,27 @@ uint32_t logismos_launch_latent_decode_bf16(const void* q, const void* pool, con
   if (rank <= 128) rc = heads <= 16 ? LG_DECODE(1, 2, 64, true) : heads <= 32 ? LG_DECODE(2, 2, 64, true) : LG_DECODE(4, 2, 64, true);
   else if (rank <= 256) rc = heads <= 16 ? LG_DECODE(1, 4, 64, true) : heads <= 32 ? LG_DECODE(2, 4, 64, true) : LG_DECODE(4, 4, 64, true);
   else if (rank <= 512) rc = heads <= 16 ? LG_DECODE(1, 8, 32, true) : heads <= 32 ? LG_DECODE(2, 8, 64, true) : LG_DECODE(4, 8, 32, false);
+  else if (rank <= 640) rc = heads <= 16 ? LG_DECODE(1, 10, 32, true) : heads <= 32 ? LG_DECODE(2, 10, 32, true) : LG_DECODE(4, 10, 32, false);
   else rc = heads <= 16 ? LG_DECODE(1, 16, 32, true) : LG_DECODE(2, 16, 32, false);
 #undef LG_DECODE
   if (rc || total_chunks == rows) return rc;
   // an ordinary launch: with the early one the next projection's CTAs moved in ahead of these and a decode step of 8
   // sequences took 1.86 instead of 1.42 ms
   lg::launch_ordered(latent_merge_kernel, dim3((unsigned)heads, (unsigned)rows), dim3(128), 0, s, (const float*)p.part_o, (const float2*)p.part_ml,
-             p.chunk_offsets, p.out, heads, rank);
+             p.chunk_offsets, p.out, heads, rank, p.gate, ld_gate);
   return lg::launch_status();
 }
 
 uint32_t logismos_launch_latent_attention_f32(const void* q_f32, const void* pool_f32, const void* block_tables_i32, const void* seq_ids_i32,
                                               const void* positions_i32, void* out_f32, int32_t rows, int32_t max_blocks,
-                                              int32_t n_pool_blocks, int32_t heads, int32_t rank, float scale, void* status_i32,
-                                              void* stream) {
+                                              int32_t n_pool_blocks, int32_t heads, int32_t rank, float scale, const void* gate_f32,
+                                              int32_t ld_gate, void* status_i32, void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!q_f32 || !pool_f32 || !out_f32 || rows <= 0 || max_blocks <= 0 || n_pool_blocks <= 0 || heads <= 0 || heads > 65535 || rank <= 0 || rank > 1024)
+  if ((gate_f32 && ld_gate < heads) || !q_f32 || !pool_f32 || !out_f32 || rows <= 0 || max_blocks <= 0 || n_pool_blocks <= 0 || heads <= 0 || heads > 65535 || rank <= 0 || rank > 1024)
     return lg::kInvalidValue;
   lg::launch(latent_attention_f32_kernel, dim3((unsigned)rows, (unsigned)heads), dim3(128), (size_t)(rank + kF32Tile) * 4, (cudaStream_t)stream,
              (const float*)q_f32, (const float*)pool_f32, (const int*)block_tables_i32, max_blocks, n_pool_blocks, (const int*)seq_ids_i32,
-             (const int*)positions_i32, (float*)out_f32, heads, rank, scale * kLog2e, (int*)status_i32);
+             (const int*)positions_i32, (float*)out_f32, heads, rank, scale * kLog2e, (const float*)gate_f32, ld_gate, (int*)status_i32);
   return lg::launch_status();
 }
 

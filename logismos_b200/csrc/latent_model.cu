@@ -95,7 +95,7 @@ uint32_t attention(Latent* m, LLayer& L, cudaStream_t s) {
   if (c.is_f32) {
     LG_TRY(head_linear(m, m->q.p, HD, L.w_ukt, L.c.heads, L.Rp, L.D, m->qlat.p, HR, B.T, s), "latent queries");
     LG_TRY(logismos_launch_latent_attention_f32(m->qlat.p, L.pool.p, m->dev(B.tables), m->dev(B.seq_ids), m->dev(B.pos), m->olat.p, B.T, MB,
-                                                c.n_pool_blocks, L.c.heads, L.Rp, L.c.scale, st, s), "latent attention");
+                                                c.n_pool_blocks, L.c.heads, L.Rp, L.c.scale, nullptr, 0, st, s), "latent attention");
     m->launches += 1;
     LG_TRY(head_linear(m, m->olat.p, HR, L.w_uv, L.c.heads, L.D, L.Rp, m->cat.p, L.Cw, B.T, s), "latent values");
     return 0;
@@ -103,7 +103,7 @@ uint32_t attention(Latent* m, LLayer& L, cudaStream_t s) {
   if (B.n_dec > 0) {
     LG_TRY(head_linear(m, m->q.p, HD, L.w_ukt, L.c.heads, L.Rp, L.D, m->qlat.p, HR, B.n_dec, s), "latent queries");
     LG_TRY(logismos_launch_latent_decode_bf16(m->qlat.p, L.pool.p, m->dev(B.tables), m->dev(B.ctx), m->dev(B.chunks), m->olat.p, m->dec_scratch.p,
-                                              B.n_dec, m->total_chunks, m->chunk_tokens, MB, c.n_pool_blocks, L.c.heads, L.Rp, L.c.scale, st, s),
+                                              B.n_dec, m->total_chunks, m->chunk_tokens, MB, c.n_pool_blocks, L.c.heads, L.Rp, L.c.scale, nullptr, 0, st, s),
            "latent decode");
     m->launches += m->total_chunks > B.n_dec ? 2 : 1;
     LG_TRY(head_linear(m, m->olat.p, HR, L.w_uv, L.c.heads, L.D, L.Rp, m->cat.p, L.Cw, B.n_dec, s), "latent values");
@@ -119,7 +119,7 @@ uint32_t attention(Latent* m, LLayer& L, cudaStream_t s) {
                                              st, s), "keys");
     LG_TRY(logismos_launch_linear_t_act_bf16(L.w_uv.p, m->lat.p, nullptr, m->vt.p, HD, tp, L.Rp, L.Rp, tp, LG_EPI_BF16, 0, 0, 0, st, s), "values");
     LG_TRY(logismos_launch_varlen_attention_kv_tc_bf16(q, HD, m->dev(B.cu_pre) + r.s0, kv_lens, m->kv_start.p, m->kbuf.p, m->vt.p, tp, out, L.Cw,
-                                                       B.T - B.n_dec, ns, r.max_q, L.c.heads, L.c.heads, L.D, L.c.scale, st, s), "attention");
+                                                       B.T - B.n_dec, ns, r.max_q, L.c.heads, L.c.heads, L.D, L.c.scale, nullptr, 0, st, s), "attention");
     m->launches += 4;
   }
   return 0;
@@ -162,7 +162,7 @@ uint32_t run_device(Latent* m, cudaStream_t s) {
     float* raw = (float*)(acc ? m->raw_acc.p : m->raw.p);
     LG_TRY(linear(m, {m->h1.p, Hp, &L.w_in, L.Qp + L.Rp, Hp, nullptr, raw, L.Qp + L.Rp, acc ? LG_EPI_RESID_F32 : LG_EPI_F32}, T, s), "latent projections");
     LG_TRY(logismos_launch_latent_norm_store(raw, L.Qp + L.Rp, L.gain_q.p, L.gain_c.p, m->cq.p, L.pool.p, m->dev(B.slots), T, L.Qp, L.c.q_rank,
-                                             L.Rp, L.c.kv_rank, c.rms_eps, (int64_t)c.n_pool_blocks * kKvBlock, f32, acc, st, s), "latent norm and store");
+                                             L.Rp, L.c.kv_rank, c.rms_eps, (int64_t)c.n_pool_blocks * kKvBlock, f32, acc, nullptr, st, s), "latent norm and store");
     m->launches += 1;
     LG_TRY(linear(m, {m->cq.p, L.Qp, &L.w_uq, HD, L.Qp, nullptr, m->q.p, HD, LG_EPI_BF16}, T, s), "queries");
     if (uint32_t rc = attention(m, L, s)) return rc;

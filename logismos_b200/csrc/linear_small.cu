@@ -23,6 +23,8 @@ struct SmallArgs {
   int64_t a_stride, w_stride, out_stride;  // per batch entry (elements)
   float p0, p1, p2;
   lg_linear_groups_t groups;               // with kEpiGroups
+  const int* offsets;                      // EXPERTS: batch entry b has the output rows offsets[b] .. offsets[b + 1]
+  const int* row_idx;                      // and reads these input rows (NULL: the same)
 };
 
 // internal epilogue of the grouped projections (lg_linear_groups_t): main columns, then an fp32 tail
@@ -38,10 +40,17 @@ LG_DEVINL int group_of(const lg_linear_groups_t& g, int c) {
 
 LG_DEVINL uint4 ldg16(const void* p) { return __ldg(reinterpret_cast<const uint4*>(p)); }
 
-template <int MT, int NT>
+template <int MT, int NT, bool EXPERTS = false>
 __global__ void __launch_bounds__(512)
 linear_small_kernel(SmallArgs p) {
   lg::pdl_trigger();
+  int first = 0;
+  if (EXPERTS) {  // which rows a matrix has is the work of a kernel of this step
+    lg::pdl_wait();
+    first = p.offsets[blockIdx.z];
+    p.m = p.offsets[blockIdx.z + 1] - first;
+    if ((int)blockIdx.y * 8 * NT >= p.m) return;
+  }
   constexpr int kUnroll = MT * NT >= 8 ? 2 : 4;
   extern __shared__ float red[];  // [warps][16 * MT][8 * NT]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
@@ -86,7 +95,15 @@ linear_small_kernel(SmallArgs p) {
     }
   };
   load_w(warp);      // the weights are static: requested before the dependency wait
-  lg::pdl_wait();
+  if (!EXPERTS) lg::pdl_wait();
+  int src[NT];       // EXPERTS: input rows of this lane
+  if (EXPERTS) {
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int r = m0 + 8 * j + g;
+      src[j] = r < p.m ? (p.row_idx ? p.row_idx[first + r] : first + r) : 0;
+    }
+  }
   for (int s0 = warp; s0 < steps; s0 += kUnroll * n_warps) {
 #pragma unroll
     for (int u = 0; u < kUnroll; ++u) {
@@ -96,7 +113,7 @@ linear_small_kernel(SmallArgs p) {
         for (int j = 0; j < NT; ++j) {
           const int r = m0 + 8 * j + g;
           uint4 x = make_uint4(0u, 0u, 0u, 0u);
-          if (r < p.m) x = *reinterpret_cast<const uint4*>(ab + (size_t)r * p.lda + (size_t)s * 32 + 8 * t);
+          if (r < p.m) x = *reinterpret_cast<const uint4*>(ab + (size_t)(EXPERTS ? src[j] : r) * p.lda + (size_t)s * 32 + 8 * t);
           const uint32_t b0[2] = {x.x, x.y}, b1[2] = {x.z, x.w};
 #pragma unroll
           for (int i = 0; i < MT; ++i) {
@@ -124,6 +141,7 @@ linear_small_kernel(SmallArgs p) {
     }
   __syncthreads();
   const int out_rows = glu ? 16 : kRows;  // output columns this CTA produces
+  if (EXPERTS) p.out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)first * p.ldc;
   for (int e = threadIdx.x; e < out_rows * kCols; e += blockDim.x) {
     const int c = e % out_rows, r = m0 + e / out_rows;
     if (r >= p.m) continue;
@@ -142,7 +160,7 @@ linear_small_kernel(SmallArgs p) {
       reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)blockIdx.z * p.out_stride + (size_t)r * p.ldc + oc] = __float2bfloat16_rn(y);
       continue;
     }
-    if (p.bias) v += p.bias[wrow];
+    if (p.bias && (p.epi != kEpiGroups || wrow < p.groups.n_main)) v += p.bias[wrow];
     if (p.epi == LG_EPI_RELU2) { v = fmaxf(v, 0.0f); v *= v; }
     if (p.epi == kEpiGroups && wrow >= p.groups.n_main) {
       const int tc = wrow - p.groups.n_main, width = p.n - p.groups.n_main;
@@ -176,6 +194,20 @@ uint32_t launch_small(const SmallArgs& a, int batch, int warps, cudaStream_t s) 
   return lg::launch_status();
 }
 
+template <int NT>
+uint32_t launch_small_experts(const SmallArgs& a, int n_groups, int max_rows, int warps, cudaStream_t s) {
+  const bool glu = a.epi == LG_EPI_SWIGLU;
+  const size_t smem = (size_t)warps * 32 * 8 * NT * 4;
+  auto kern = linear_small_kernel<2, NT, true>;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (uint32_t)e;
+  }
+  const int tiles = glu ? a.n / 32 : (a.n + 31) / 32;
+  lg::launch(kern, dim3((unsigned)tiles, (unsigned)((max_rows + 8 * NT - 1) / (8 * NT)), (unsigned)n_groups), dim3(32 * warps), smem, s, a);
+  return lg::launch_status();
+}
+
 // ---- fp32 activations -----------------------------------------------------------------------------
 // 64 x 64 tile, 256 threads, 4 x 4 outputs per thread: rows 4 ty .. + 3; columns 2 tx, 2 tx + 1 and the
 // same + 32, so that a thread holds a gate column and its matching up column. fp32 products and sums.
@@ -188,21 +220,31 @@ struct F32Args {
   int64_t a_stride, w_stride, out_stride;
   float p0, p1, p2;
   lg_linear_groups_t groups;
+  const int* offsets;      // as for SmallArgs (NULL: one range of rows)
+  const int* row_idx;
 };
 
 __global__ void __launch_bounds__(256)
 linear_f32_kernel(F32Args p) {
   lg::pdl_prologue();
   __shared__ float as[16][68], ws[16][68];
+  int first = 0;
+  if (p.offsets) {
+    first = p.offsets[blockIdx.z];
+    p.m = p.offsets[blockIdx.z + 1] - first;
+    if ((int)blockIdx.y * 64 >= p.m) return;
+  }
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   const int n0 = blockIdx.x * 64, m0 = blockIdx.y * 64;
   const float* A = p.a + (size_t)blockIdx.z * p.a_stride + (p.epi == kEpiGroups ? (size_t)group_of(p.groups, n0) * p.m * p.lda : 0);
   const __nv_bfloat16* W = p.w + (size_t)blockIdx.z * p.w_stride;
   float acc[4][4] = {};
   const int lr = tid >> 2, lk = (tid & 3) * 4;
+  int a_row = m0 + lr;
+  if (p.offsets && a_row < p.m) a_row = p.row_idx ? p.row_idx[first + a_row] : first + a_row;
   for (int k0 = 0; k0 < p.k; k0 += 16) {
     float4 av = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (m0 + lr < p.m) av = *reinterpret_cast<const float4*>(A + (size_t)(m0 + lr) * p.lda + k0 + lk);
+    if (m0 + lr < p.m) av = *reinterpret_cast<const float4*>(A + (size_t)a_row * p.lda + k0 + lk);
     float wv[4] = {0.f, 0.f, 0.f, 0.f};
     if (n0 + lr < p.n) {
       const uint2 u = __ldg(reinterpret_cast<const uint2*>(W + (size_t)(n0 + lr) * p.k + k0 + lk));
@@ -226,7 +268,7 @@ linear_f32_kernel(F32Args p) {
     }
     __syncthreads();
   }
-  float* out = p.out + (size_t)blockIdx.z * p.out_stride;
+  float* out = p.out + (size_t)blockIdx.z * p.out_stride + (size_t)first * p.ldc;
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int r = m0 + 4 * ty + i;
@@ -234,7 +276,7 @@ linear_f32_kernel(F32Args p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int c = n0 + (j >> 1) * 32 + 2 * tx + (j & 1);
-      if (c < p.n && p.bias) acc[i][j] += p.bias[c];
+      if (c < p.n && p.bias && (p.epi != kEpiGroups || c < p.groups.n_main)) acc[i][j] += p.bias[c];
     }
     if (p.epi == LG_EPI_GLU_CLAMP) {
 #pragma unroll
@@ -314,7 +356,7 @@ uint32_t logismos_launch_linear_groups_small_bf16(const void* a, const void* w, 
                                                   int32_t ldc, const lg_linear_groups_t* groups, void* stream) {
   lg::LaunchScope launch_scope_;
   if (!lg::groups_ok(groups, n, ldc)) return lg::kInvalidValue;
-  return small_any(a, w, nullptr, out, m, n, k, lda, ldc, 1, 0, 0, 0, kEpiGroups, 0, 0, 0, *groups, stream);
+  return small_any(a, w, groups->bias, out, m, n, k, lda, ldc, 1, 0, 0, 0, kEpiGroups, 0, 0, 0, *groups, stream);
 }
 
 uint32_t logismos_launch_linear_f32(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k,
@@ -339,8 +381,41 @@ uint32_t logismos_launch_linear_groups_f32(const void* a, const void* w, void* o
   if (m <= 0 || n <= 0 || k <= 0 || (k % 16) || (lda % 4) || lda < k || ((uintptr_t)a & 15) || ((uintptr_t)w & 7) || !out || (m + 63) / 64 > 65535 ||
       !lg::groups_ok(groups, n, ldc))
     return lg::kInvalidValue;
-  const F32Args p{(const float*)a, (const __nv_bfloat16*)w, nullptr, (float*)out, m, n, k, lda, ldc, kEpiGroups, 0, 0, 0, 0, 0, 0, *groups};
+  const F32Args p{(const float*)a, (const __nv_bfloat16*)w, (const float*)groups->bias, (float*)out, m, n, k, lda, ldc, kEpiGroups, 0, 0, 0, 0, 0, 0, *groups};
   lg::launch(linear_f32_kernel, dim3((unsigned)((n + 63) / 64), (unsigned)((m + 63) / 64)), dim3(256), 0, (cudaStream_t)stream, p);
+  return lg::launch_status();
+}
+
+uint32_t logismos_launch_linear_experts_small_bf16(const void* a, const void* w, void* out, const void* offsets, const void* row_idx, int32_t n_groups,
+                                                   int32_t max_group_rows, int32_t expected_group_rows, int32_t n, int32_t k, int32_t lda, int32_t ldc,
+                                                   int32_t epilogue, void* stream) {
+  lg::LaunchScope launch_scope_;
+  epilogue &= ~LG_EPI_STATIC_W;
+  const bool glu = epilogue == LG_EPI_SWIGLU;
+  if (!a || !w || !out || !offsets || n_groups <= 0 || n_groups > 65535 || max_group_rows <= 0 || max_group_rows > (1 << 19) || n <= 0 || n % (glu ? 64 : 16) || k <= 0 ||
+      k % 32 || lda < k || lda % 8 || ldc < (glu ? n / 2 : n) || (((uintptr_t)a | (uintptr_t)w) & 15) || (!glu && epilogue != LG_EPI_BF16))
+    return lg::kInvalidValue;
+  SmallArgs p{(const __nv_bfloat16*)a, (const __nv_bfloat16*)w, nullptr, out, 0, n, k, lda, ldc, epilogue, 0, (int64_t)n * k, 0, 0, 0, 0, {}, (const int*)offsets,
+              (const int*)row_idx};
+  const int steps = k / 32, warps = steps < 8 ? steps : 8, rows = expected_group_rows < max_group_rows ? expected_group_rows : max_group_rows;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (rows <= 8) return launch_small_experts<1>(p, n_groups, max_group_rows, warps, s);
+  if (rows <= 16) return launch_small_experts<2>(p, n_groups, max_group_rows, warps, s);
+  return launch_small_experts<4>(p, n_groups, max_group_rows, warps, s);
+}
+
+uint32_t logismos_launch_linear_experts_f32(const void* a, const void* w, void* out, const void* offsets, const void* row_idx, int32_t n_groups,
+                                            int32_t max_group_rows, int32_t n, int32_t k, int32_t lda, int32_t ldc, int32_t epilogue, float p0, float p1,
+                                            float p2, void* stream) {
+  lg::LaunchScope launch_scope_;
+  epilogue &= ~LG_EPI_STATIC_W;
+  const bool glu = epilogue == LG_EPI_GLU_CLAMP;
+  if (!a || !w || !out || !offsets || n_groups <= 0 || n_groups > 65535 || max_group_rows <= 0 || (max_group_rows + 63) / 64 > 65535 || n <= 0 || (glu && n % 64) || k <= 0 ||
+      k % 16 || lda < k || lda % 4 || ldc < (glu ? n / 2 : n) || ((uintptr_t)a & 15) || ((uintptr_t)w & 7) || (!glu && epilogue != LG_EPI_F32))
+    return lg::kInvalidValue;
+  const F32Args p{(const float*)a, (const __nv_bfloat16*)w, nullptr, (float*)out, 0, n, k, lda, ldc, epilogue, 0, (int64_t)n * k, 0, p0, p1, p2, {}, (const int*)offsets,
+                  (const int*)row_idx};
+  lg::launch(linear_f32_kernel, dim3((unsigned)((n + 63) / 64), (unsigned)((max_group_rows + 63) / 64), (unsigned)n_groups), dim3(256), 0, (cudaStream_t)stream, p);
   return lg::launch_status();
 }
 

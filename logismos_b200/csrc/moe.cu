@@ -1,0 +1,259 @@
+// Router of a mixture of experts (lg_moe_route_t): the choice of experts per token and the grouping of rows by expert.
+//   few tokens    one CTA: choice, counts, offsets and row lists; the expert products read their rows through the list
+//   many tokens   choice with per-CTA histograms (a row's rank in its group is unique, its order is not fixed; rows of a
+//                 group are independent), then a second launch that places the rows, copies them and lists the row tiles
+// Logits, softmax, choice and weights are fp32. A warp handles a token, a lane the experts lane, lane + 32, ...
+#include "common.cuh"
+#include "logismos_kernels.h"
+
+namespace {
+
+using namespace lg;
+
+constexpr int kMaxOut = 512, kMaxTop = 32, kMaxAlways = 64, kMaxGroups = kMaxOut + kMaxAlways;
+constexpr int kFewThreads = 1024, kRouteThreads = 256, kRouteTokens = 32;
+
+struct RouteArgs {
+  float* logits;
+  int ld, zero;
+  const float* correction;
+  int experts, identity, top, always;
+  float* weights;
+  int* pair_row;
+  float* id_weight;
+  int* offsets;
+  int* row_token;
+  int* counts;
+  int* pair_expert;
+  int4* tiles;
+  int* n_tiles;
+  int tokens;
+};
+
+// float -> integer of the same order
+LG_DEVINL uint32_t ordered(float x) {
+  const uint32_t u = __float_as_uint(x);
+  return u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+
+// The token's experts: lane i < top receives the i-th choice and its weight. R: logits per lane.
+template <int R>
+LG_DEVINL void choose(const RouteArgs& p, int token, int lane, int& expert, float& weight) {
+  const int n = p.experts + p.identity;
+  float* z = p.logits + (size_t)token * p.ld;
+  float s[R], c[R], mx = -INFINITY, sum = 0.0f;
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    s[i] = lane + 32 * i < n ? z[lane + 32 * i] : -INFINITY;
+    mx = fmaxf(mx, s[i]);
+  }
+  mx = warp_max(mx);
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    s[i] = expf(s[i] - mx);
+    sum += s[i];
+  }
+  sum = warp_sum(sum);
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    s[i] /= sum;
+    c[i] = lane + 32 * i < n ? s[i] + __ldg(p.correction + lane + 32 * i) : -INFINITY;
+    if (p.zero && lane + 32 * i < n) z[lane + 32 * i] = 0.0f;
+  }
+  expert = -1;
+  float picked = 0.0f, total = 0.0f;
+  for (int k = 0; k < p.top; ++k) {
+    float best = -INFINITY;
+    int at = 0;
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+      if (c[i] > best) { best = c[i]; at = i; }
+    const uint32_t key = ordered(best), top_key = __reduce_max_sync(0xffffffffu, key);
+    const int id = __reduce_min_sync(0xffffffffu, key == top_key ? lane + 32 * at : kMaxOut);  // equal scores: the first
+    float score = 0.0f;
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+      if (id == lane + 32 * i) { score = s[i]; c[i] = -INFINITY; }
+    score = __shfl_sync(0xffffffffu, score, id & 31);
+    total += score;
+    if (lane == k) { expert = id; picked = score; }
+  }
+  weight = picked / (total + 1e-20f);
+}
+
+// weights, the identity experts' share, and the group of each pair (-1: none)
+LG_DEVINL int store_choice(const RouteArgs& p, int token, int lane, int expert, float weight) {
+  const bool in = lane < p.top, none = in && expert >= p.experts;
+  const float id = warp_sum(none ? weight : 0.0f);
+  if (in) p.weights[(size_t)token * p.top + lane] = weight;
+  if (lane == 0) p.id_weight[token] = id;
+  return in && !none ? expert : -1;
+}
+
+// exclusive prefix of count[0 .. n) into start[0 .. n]; all threads of the CTA, n <= kMaxGroups
+LG_DEVINL void prefix(const int* count, int* start, int n) {
+  if (threadIdx.x < 32) {
+    int base = 0;
+    for (int g0 = 0; g0 < n; g0 += 32) {
+      const int g = g0 + (int)threadIdx.x, own = g < n ? count[g] : 0;
+      int x = own;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int y = __shfl_up_sync(0xffffffffu, x, o);
+        if ((int)threadIdx.x >= o) x += y;
+      }
+      if (g < n) start[g] = base + x - own;
+      base += __shfl_sync(0xffffffffu, x, 31);
+    }
+    if (threadIdx.x == 0) start[n] = base;
+  }
+  __syncthreads();
+}
+
+template <int R>
+__global__ void __launch_bounds__(kFewThreads)
+moe_route_few_kernel(RouteArgs p) {
+  lg::pdl_prologue();
+  __shared__ int count[kMaxGroups], start[kMaxGroups + 1];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, groups = p.experts + p.always, pairs = p.top + p.always;
+  for (int g = tid; g < groups; g += kFewThreads) count[g] = g < p.experts ? 0 : p.tokens;
+  __syncthreads();
+  for (int t = warp; t < p.tokens; t += kFewThreads / 32) {
+    int expert;
+    float weight;
+    choose<R>(p, t, lane, expert, weight);
+    const int g = store_choice(p, t, lane, expert, weight);
+    // the rank in the group goes to pair_row for now, the group rides in its high bits
+    if (lane < p.top) p.pair_row[(size_t)t * pairs + lane] = g < 0 ? -1 : atomicAdd(&count[g], 1) | (g << 20);
+  }
+  __syncthreads();
+  prefix(count, start, groups);
+  for (int g = tid; g <= groups; g += kFewThreads) p.offsets[g] = start[g];
+  for (int i = tid; i < p.tokens * pairs; i += kFewThreads) {
+    const int t = i / pairs, k = i - t * pairs;
+    int row;
+    if (k >= p.top) row = start[p.experts + k - p.top] + t;
+    else {
+      const int v = p.pair_row[i];
+      if (v < 0) continue;
+      row = start[v >> 20] + (v & 0xfffff);
+    }
+    p.pair_row[i] = row;
+    p.row_token[row] = t;
+  }
+}
+
+template <int R>
+__global__ void __launch_bounds__(kRouteThreads)
+moe_route_kernel(RouteArgs p) {
+  lg::pdl_prologue();
+  __shared__ int count[kMaxOut], base[kMaxOut], group_s[kRouteTokens * kMaxTop], rank_s[kRouteTokens * kMaxTop];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, pairs = p.top + p.always;
+  const int t0 = blockIdx.x * kRouteTokens, n = min(kRouteTokens, p.tokens - t0);
+  for (int g = tid; g < p.experts; g += kRouteThreads) count[g] = 0;
+  __syncthreads();
+  for (int t = warp; t < n; t += kRouteThreads / 32) {
+    int expert;
+    float weight;
+    choose<R>(p, t0 + t, lane, expert, weight);
+    const int g = store_choice(p, t0 + t, lane, expert, weight);
+    if (lane < p.top) {
+      group_s[t * p.top + lane] = g;
+      rank_s[t * p.top + lane] = g < 0 ? 0 : atomicAdd(&count[g], 1);
+    }
+  }
+  __syncthreads();
+  for (int g = tid; g < p.experts; g += kRouteThreads) base[g] = count[g] ? atomicAdd(p.counts + g, count[g]) : 0;
+  __syncthreads();
+  for (int i = tid; i < n * p.top; i += kRouteThreads) {
+    const int t = i / p.top, k = i - t * p.top, g = group_s[i];
+    p.pair_expert[(size_t)(t0 + t) * p.top + k] = g;
+    p.pair_row[(size_t)(t0 + t) * pairs + k] = g < 0 ? -1 : base[g] + rank_s[i];  // rank in the group, placed by the next launch
+  }
+}
+
+// A warp per (token, pair): final rows, and the copy of the token's row for the chosen experts. CTA 0 also lists the tiles.
+__global__ void __launch_bounds__(kRouteThreads)
+moe_place_kernel(RouteArgs p, const uint4* h, uint4* gathered, int vecs) {
+  lg::pdl_prologue();
+  __shared__ int count[kMaxGroups], start[kMaxGroups + 1], first[kMaxGroups + 1];
+  const int tid = threadIdx.x, lane = tid & 31, groups = p.experts + p.always, pairs = p.top + p.always;
+  for (int g = tid; g < groups; g += kRouteThreads) count[g] = g < p.experts ? p.counts[g] : p.tokens;
+  __syncthreads();
+  prefix(count, start, groups);
+  const int64_t total = (int64_t)p.tokens * pairs;
+  for (int64_t i = (int64_t)blockIdx.x * (kRouteThreads / 32) + (tid >> 5); i < total; i += (int64_t)gridDim.x * (kRouteThreads / 32)) {
+    const int t = (int)(i / pairs), k = (int)(i - (int64_t)t * pairs);
+    if (k >= p.top) {
+      if (lane == 0) p.pair_row[i] = start[p.experts + k - p.top] + t;
+      continue;
+    }
+    const int g = p.pair_expert[(size_t)t * p.top + k];
+    if (g < 0) continue;
+    const int row = start[g] + p.pair_row[i];
+    __syncwarp();
+    if (lane == 0) p.pair_row[i] = row;
+    for (int v = lane; v < vecs; v += 32) gathered[(size_t)row * vecs + v] = h[(size_t)t * vecs + v];
+  }
+  if (blockIdx.x) return;
+  for (int g = tid; g < groups; g += kRouteThreads) count[g] = (count[g] + 127) >> 7;
+  __syncthreads();
+  prefix(count, first, groups);
+  for (int g = tid; g < groups; g += kRouteThreads)
+    for (int i = 0; i < count[g]; ++i) {
+      const int row = start[g] + 128 * i;
+      p.tiles[first[g] + i] = make_int4(g, row, start[g + 1], g < p.experts ? row : -1 - 128 * i);
+    }
+  if (tid == 0) *p.n_tiles = first[groups];
+}
+
+bool route_ok(const lg_moe_route_t* a, int tokens) {
+  return a && tokens > 0 && tokens < (1 << 20) && a->logits && a->correction && a->weights && a->pair_row && a->identity && a->n_experts > 0 &&
+         a->n_identity >= 0 && a->n_experts + a->n_identity <= kMaxOut && a->ld >= a->n_experts + a->n_identity && a->top > 0 && a->top <= kMaxTop &&
+         a->top <= a->n_experts + a->n_identity && a->n_always >= 0 && a->n_always <= kMaxAlways;
+}
+RouteArgs route_args(const lg_moe_route_t* a, int tokens) {
+  return RouteArgs{(float*)a->logits, a->ld, a->zero_logits, (const float*)a->correction, a->n_experts, a->n_identity, a->top, a->n_always, (float*)a->weights,
+                   (int*)a->pair_row, (float*)a->identity, (int*)a->offsets, (int*)a->row_token, (int*)a->counts, (int*)a->pair_expert, (int4*)a->tiles,
+                   (int*)a->n_tiles, tokens};
+}
+
+}  // namespace
+
+extern "C" {
+
+int32_t logismos_moe_few_tokens(void) { return 128; }
+
+int32_t logismos_moe_max_tiles(int32_t tokens, int32_t top, int32_t n_experts, int32_t n_always) {
+  return (int32_t)((int64_t)tokens * top / 128) + n_experts + (tokens + 127) / 128 * n_always;
+}
+
+// one launch when offsets are given, else the first of two
+uint32_t logismos_launch_moe_route(const lg_moe_route_t* a, int32_t tokens, void* stream) {
+  lg::LaunchScope launch_scope_;
+  const bool few = a && a->offsets;
+  if (!route_ok(a, tokens) || (few ? !a->row_token : !a->counts || !a->pair_expert)) return lg::kInvalidValue;
+  const RouteArgs p = route_args(a, tokens);
+  const dim3 grid(few ? 1u : (unsigned)((tokens + kRouteTokens - 1) / kRouteTokens)), block(few ? kFewThreads : kRouteThreads);
+  auto go = [&](auto kern) -> uint32_t {
+    lg::launch(kern, grid, block, 0, (cudaStream_t)stream, p);
+    return lg::launch_status();
+  };
+  const int n = p.experts + p.identity;
+#define LG_ROUTE(R) (few ? go(moe_route_few_kernel<R>) : go(moe_route_kernel<R>))
+  return n <= 32 ? LG_ROUTE(1) : n <= 64 ? LG_ROUTE(2) : n <= 128 ? LG_ROUTE(4) : n <= 256 ? LG_ROUTE(8) : LG_ROUTE(16);
+#undef LG_ROUTE
+}
+
+uint32_t logismos_launch_moe_place(const lg_moe_route_t* a, const void* h, void* gathered, int32_t ld, int32_t tokens, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!route_ok(a, tokens) || !a->counts || !a->pair_expert || !a->tiles || !a->n_tiles || !h || !gathered || ld <= 0 || ld % 8 ||
+      (((uintptr_t)h | (uintptr_t)gathered | (uintptr_t)a->tiles) & 15))
+    return lg::kInvalidValue;
+  const RouteArgs p = route_args(a, tokens);
+  const int64_t warps = (int64_t)tokens * (p.top + p.always), ctas = (warps + kRouteThreads / 32 - 1) / (kRouteThreads / 32);
+  lg::launch(moe_place_kernel, dim3((unsigned)(ctas < 148 * 8 ? ctas : 148 * 8)), dim3(kRouteThreads), 0, (cudaStream_t)stream, p, (const uint4*)h, (uint4*)gathered, ld / 8);
+  return lg::launch_status();
+}
+
+}  // extern "C"

@@ -1,5 +1,6 @@
-// Scores that are capped and biased by distance, and the output gate, shared by the attention kernels
-// (lg_score_bias_t).
+// What the attention kernels share beyond the plain softmax: scores that are capped and biased by distance, with an
+// output gate per channel (lg_score_bias_t), and windows with kept first keys, one added to the softmax denominator and an
+// output gate per head (lg_window_t).
 #pragma once
 #include <cmath>
 
@@ -29,6 +30,38 @@ struct ScoreExt {
   }
   LG_DEVINL float gated(float o, float g) const { return o * __fdividef(gate_scale, 1.0f + __expf(-g)); }
 };
+
+// The window form: where a query at position i looks, and what becomes of its output
+struct WindowExt {
+  int size, keep, sink;          // size INT_MAX: all keys
+  const float* gate;             // [rows, ld_gate], NULL: none
+  int ld_gate;
+  int ld_q, ld_out;
+  LG_DEVINL bool sees(int i, int j) const { return j <= i && (i - j < size || j < keep); }
+  LG_DEVINL float head_gate(size_t row, int head) const { return gate ? 1.0f / (1.0f + __expf(-gate[row * ld_gate + head])) : 1.0f; }
+};
+
+// Blocks of 16 tokens between the kept ones and the first of the window, for the last of `ctx` tokens
+__host__ __device__ inline int window_gap_blocks(int ctx, int size, int keep) {
+  if (size >= ctx) return 0;
+  const int first = (ctx - size) / 16, kept = (keep + 15) / 16;
+  return first > kept ? first - kept : 0;
+}
+// Keys left out of a prompt launch's gather, for queries at the last q_len of kv_len positions: between the kept keys,
+// rounded up to tiles of 128, and the first query's window, rounded down to a multiple of 8
+__host__ __device__ inline int window_gap_keys(int kv_len, int q_len, int size, int keep) {
+  const int cached = kv_len - q_len;
+  if (cached < size) return 0;
+  const int first = (cached - size + 1) & ~7, kept = (keep + 127) / 128 * 128;
+  return first > kept ? first - kept : 0;
+}
+
+inline bool window_ok(const lg_window_t* w, int heads) {
+  return w && w->scale > 0.0f && w->size >= 0 && w->keep_first >= 0 && w->keep_first < (1 << 30) && (!w->gate || w->ld_gate >= heads);
+}
+inline WindowExt window_ext(const lg_window_t* w, int ld_q, int ld_out) {
+  return WindowExt{w->size ? w->size : 0x7fffffff, w->keep_first, w->sink, (const float*)w->gate, w->ld_gate, ld_q, ld_out};
+}
 
 inline bool score_ok(const lg_score_bias_t* s, int width) {
   return s && s->scale > 0.0f && s->cap >= 0.0f && s->bias && s->far >= 0 && s->gate && s->ld_gate >= width;

@@ -631,7 +631,7 @@ def latent_norm_store(raw, gain_q, gain_c, pool, slot_mapping, q_n, c_n, eps, ze
     with torch.cuda.device(raw.device):
         check(lib.logismos_launch_latent_norm_store(_p(raw), raw.shape[1], _p(gain_q), _p(gain_c), _p(cq), _p(pool), _p(slot_mapping), rows, qw, q_n,
                                                     cw, c_n, float(eps), pool.shape[0] * 16, int(pool.dtype == torch.float32), int(zero_raw),
-                                                    _p(status), _stream()), "latent_norm_store")
+                                                    None, _p(status), _stream()), "latent_norm_store")
         _done(sync)
         if sync and int(status.item()) != 0:
             raise InvalidOp("latent_norm_store: slot outside the pool")
@@ -662,7 +662,7 @@ def attention_kv(q, k, v_t, cu_seqlens_q, kv_lens, kv_start, n_heads, n_kv_heads
     with torch.cuda.device(q.device):
         check(lib.logismos_launch_varlen_attention_kv_tc_bf16(_p(q), q.shape[1], _p(cu_seqlens_q), _p(kv_lens), _p(kv_start), _p(k), _p(v_t), k.shape[0],
                                                               _p(out), out.shape[1], q.shape[0], kv_lens.numel(), max_q_len, n_heads, n_kv_heads,
-                                                              head_dim, float(scale), _p(status), _stream()), "attention_kv")
+                                                              head_dim, float(scale), None, 0, _p(status), _stream()), "attention_kv")
         _done(sync)
         if sync and int(status.item()) != 0:
             raise InvalidOp(f"attention_kv: device status {int(status.item())}")
@@ -683,7 +683,7 @@ def latent_decode(q, pool, block_tables, context_lens, context_lens_host, scale,
     status = torch.zeros(1, dtype=torch.int32, device=q.device)
     with torch.cuda.device(q.device):
         check(lib.logismos_launch_latent_decode_bf16(_p(q), _p(pool), _p(block_tables), _p(context_lens), _p(off), _p(out), _p(scratch), rows, total,
-                                                     chunk, block_tables.shape[1], pool.shape[0], heads, rank, float(scale), _p(status), _stream()),
+                                                     chunk, block_tables.shape[1], pool.shape[0], heads, rank, float(scale), None, 0, _p(status), _stream()),
               "latent_decode")
         _done(sync)
         if sync and int(status.item()) != 0:
@@ -698,7 +698,7 @@ def latent_attention_f32(q, pool, block_tables, seq_ids, positions, scale, sync=
     status = torch.zeros(1, dtype=torch.int32, device=q.device)
     with torch.cuda.device(q.device):
         check(lib.logismos_launch_latent_attention_f32(_p(q), _p(pool), _p(block_tables), _p(seq_ids), _p(positions), _p(out), q.shape[0],
-                                                       block_tables.shape[1], pool.shape[0], q.shape[1], q.shape[2], float(scale), _p(status), _stream()),
+                                                       block_tables.shape[1], pool.shape[0], q.shape[1], q.shape[2], float(scale), None, 0, _p(status), _stream()),
               "latent_attention_f32")
         _done(sync)
         if sync and int(status.item()) != 0:

@@ -8,32 +8,11 @@ import torch
 import katadra_reference as R
 from logismos_b200 import ops
 from logismos_b200._lib import check, lib
+from logismos_b200.structs import Groups, ScoreBias, Ssd, TimeMix
 
 pytestmark = pytest.mark.gpu
 DEV = "cuda:0"
 vp, i32, f32 = C.c_void_p, C.c_int32, C.c_float
-
-
-class TimeMix(C.Structure):
-    _fields_ = [("proj", vp)] + [(n, i32) for n in ("ld", "off_r", "off_k", "off_v", "off_g")] + [("z", vp), ("ld_z", i32), ("low", vp), ("ld_low", i32),
-               ("w2", vp), ("ld_w2", i32), ("rank", i32), ("w0", vp), ("u", vp), ("gain", vp), ("state", vp), ("state_slots", vp), ("fresh", vp), ("cu", vp),
-               ("out", vp), ("ld_out", i32), ("heads", i32), ("d", i32), ("dp", i32), ("scale", f32), ("eps", f32)]
-
-
-class Ssd(C.Structure):
-    _fields_ = [("proj", vp), ("ld", i32), ("dt", vp), ("ld_dt", i32), ("conv_w", vp), ("conv_b", vp), ("conv_state", vp), ("taps", i32), ("dt_bias", vp),
-                ("log_a", vp), ("skip", vp), ("state", vp), ("state_slots", vp), ("fresh", vp), ("phase", vp), ("cu", vp), ("y", vp)] + [
-               (n, i32) for n in ("ld_y", "heads", "groups", "np", "vp")] + [("xbc", vp), ("ld_xbc", i32)]
-
-
-class Groups(C.Structure):
-    _fields_ = [("n_groups", i32), ("end", i32 * 8), ("n_main", i32), ("tail", vp), ("ld_tail", i32), ("tail_cap", f32), ("tail_parts", vp)]
-
-
-class ScoreBias(C.Structure):
-    _fields_ = [("scale", f32), ("cap", f32), ("bias", vp), ("far", i32), ("max_abs_bias", f32), ("max_abs_qk", f32), ("gate", vp), ("ld_gate", i32), ("gate_scale", f32)]
-
-
 P = lambda t: vp(0 if t is None else t.data_ptr())
 A = lambda t: 0 if t is None else t.data_ptr()
 stream = lambda: vp(torch.cuda.current_stream().cuda_stream)
@@ -220,7 +199,7 @@ def run_time_mix(form, heads, d, lens, seed, fp32=False, z_lo=-6.0, z_hi=1.0, sp
 @pytest.mark.parametrize("form", ["step", "low", "chunked"])
 def test_time_mixing(form, heads, d):
     if form == "chunked" and d > 128:
-        assert not lib.logismos_time_mix_has_chunked(256)
+        assert not lib.logismos_time_mix_has_chunked(256, 256)
         return
     lens = [1, 1, 1] if form == "low" else [1, 2, 15, 16, 17, 63, 64, 65, 130]
     o, want, st, ends = run_time_mix(form, heads, d, lens, 3)
