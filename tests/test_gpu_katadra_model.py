@@ -10,80 +10,21 @@ import numpy as np
 import pytest
 
 import katadra_reference as R
+import stack_harness
 from katadra_weights import CONFIGS, SIZES, again, config, pack, parallel, ssd, weights
-from logismos_b200.cache import BlockAllocator, SlotAllocator
 from logismos_b200.embed import ComputeError, InputTooLong
 from logismos_b200.generate import generate, sampling_chain
 from logismos_b200.mixer import MixerModel, parse_config
 from logismos_b200.registry import Limits, load_model
 from logismos_b200.replay import Replay
+from stack_harness import TOLS, greedy_reference, tokens
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-TOLS = {"float32": 2e-5, "bfloat16": 6e-2}
 
 
-class Harness:
-    def __init__(self, cfg, w, dtype, pool_tokens=1024, max_seqs=6, step_tokens=700, block_seed=3, keep_layers=False):
-        self.cfg, self.w, self.dtype = cfg, w, dtype
-        n = pool_tokens // 16
-        self.model = MixerModel(parse_config(cfg), pack(cfg, w), n, n, step_tokens, max_seqs, max_seqs, dtype=dtype, max_out_rows=step_tokens, keep_layers=keep_layers)
-        self.blocks, self.slots, self.hist, self.ref = BlockAllocator(n, n, seed=block_seed), SlotAllocator(max_seqs), {}, {}
-        self.seen = self.over = 0
-
-    def expect(self, sid):
-        """Reference logits of a sequence's whole history (computed once per history)."""
-        h = tuple(self.hist[sid])
-        known, z = self.ref.get(sid, ((), None))
-        if known[:len(h)] != h:
-            z = R.forward(self.cfg, self.w, h)
-            self.ref[sid] = (h, z)
-        return z[:len(h)]
-
-    def run(self, entries, check=True):
-        """entries: (sequence, tokens); every new token's logits are compared."""
-        ids, cached, new, tabs, sl = [], [], [], [], []
-        for sid, toks in entries:
-            prev = self.hist.setdefault(sid, [])
-            cached.append(len(prev)); new.append(len(toks)); ids.extend(int(t) for t in toks)
-            prev.extend(int(t) for t in toks)
-            tabs.append(self.blocks.ensure(sid, len(prev))); sl.append(self.slots.get(sid))
-        toks = self.model.step(ids, cached, new, np.stack(tabs), sl, out_rows=range(len(ids)))
-        assert self.model.device_status() == 0
-        z, at = self.model.last_logits(), 0
-        assert np.array_equal(toks, z.argmax(1))
-        for (sid, t) in entries:
-            if check:
-                ref = self.expect(sid)
-                self.compare(z[at:at + len(t)], ref[len(ref) - len(t):], (sid, len(ref)), ref)
-            at += len(t)
-        return z
-
-    def compare(self, z, ref, what, scale=None, factor=1.0):
-        """fp32: every position. bf16: a position whose output is nearly zero before a norm can be moved far by rounding
-        alone, so single ones may exceed the limit (``close`` counts them over the whole test)."""
-        err = np.sqrt(np.mean((z - ref) ** 2, axis=1)) / np.sqrt(np.mean((ref if scale is None else scale) ** 2))
-        bound = factor * TOLS[self.dtype]
-        self.seen += err.size
-        self.over += int((err > bound).sum())
-        assert err.max() <= (bound if self.dtype == "float32" else 6 * bound), (what, int(err.argmax()), float(err.max()))
-
-    def close(self):
-        self.model.close()
-        assert self.over <= 0.02 * self.seen, (self.over, self.seen)
-
-    def known(self, sid, tokens):
-        """Computes the reference of a sequence's full history once, before it is fed in parts."""
-        self.hist[sid] = [int(t) for t in tokens]
-        self.expect(sid)
-        self.hist[sid] = []
-
-    def drop(self, sid):
-        self.blocks.release(sid); self.slots.release(sid); self.hist.pop(sid)
-
-
-def tokens(rng, cfg, n):
-    return rng.integers(0, cfg["vocab"], n)
+def Harness(cfg, w, dtype, **kw):
+    return stack_harness.Harness(MixerModel, pack, R.forward, cfg, w, dtype, **kw)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -261,24 +202,13 @@ def test_logits_do_not_depend_on_the_batch():
         assert np.sqrt(np.mean((got[0] - got[1]) ** 2)) <= tol * np.sqrt(np.mean(got[0] ** 2))
 
 
-def greedy_reference(cfg, w, prompt, n):
-    h = list(prompt)
-    margins = []
-    for _ in range(n):
-        z = R.forward(cfg, w, h)[-1]
-        top = np.sort(z)[-2:]
-        margins.append(top[1] - top[0])
-        h.append(int(z.argmax()))
-    return h[len(prompt):], min(margins)
-
-
 def test_greedy_generation_through_scheduler_and_command_line(tmp_path):
     """Prompts fed in chunks beside decoding sequences, more requests than slots, from a model folder."""
     cfg, w = CONFIGS["uneven"], weights("uneven", 41)
     R.write_checkpoint(tmp_path, cfg, w)
     rng = np.random.default_rng(6)
     prompts = [tokens(rng, cfg, n).tolist() for n in (40, 1, 17, 64, 2)]
-    want = [greedy_reference(cfg, w, p, 10) for p in prompts]
+    want = [greedy_reference(R.forward, cfg, w, p, 10) for p in prompts]
     assert min(m for _, m in want) > 1e-3      # no near ties: the continuation is defined
     served = load_model(str(tmp_path), Limits(192, 3, max_step_tokens=30), "float32")
     got = generate(served, prompts, 10, prefill_token_budget=24)
