@@ -633,9 +633,9 @@ def main():
     ap.add_argument("--no-cpu", action="store_true")
     ap.add_argument("--no-extra", action="store_true", help="skip the decode workloads of the default line")
     ap.add_argument("--ref-budget", type=float, default=150.0, help="--impl reference: seconds of timed CPU work (each step is a full batch)")
-    ap.add_argument("--workload", default="stella", choices=["stella", "ragged_step", "serving_sweep", "latent", "mixer"])
-    ap.add_argument("--sizes", default="", help="latent, mixer: comma-separated sizes of bench_latent.SIZES or bench_mixer.SIZES (default all)")
-    ap.add_argument("--kernels", action="store_true", help="latent, mixer: also every kernel against its roofline, per size")
+    ap.add_argument("--workload", default="stella", choices=["stella", "ragged_step", "serving_sweep", "latent", "mixer", "vugedra"])
+    ap.add_argument("--sizes", default="", help="latent, mixer, vugedra: comma-separated sizes of the workload's SIZES (default all)")
+    ap.add_argument("--kernels", action="store_true", help="latent, mixer, vugedra: also every kernel against its roofline, per size")
     ap.add_argument("--requests", type=int, default=96, help="serving_sweep: requests per GPU")
     ap.add_argument("--extra-requests", type=int, default=64, help="requests per GPU of the serving sample inside the default line")
     ap.add_argument("--max-seqs", type=int, default=256, help="serving_sweep: concurrent sequences per GPU")
@@ -701,6 +701,22 @@ def main():
                 "clocks": clocks, "sizes": rows}
         if args.kernels:
             line["kernels"] = {n: bench_mixer.kernel_table(bench_mixer.SIZES[n], peaks) for n in sizes}
+        print(json.dumps(line))
+    elif args.workload == "vugedra":
+        import bench_vugedra
+        if world > 1:
+            raise SystemExit("--workload vugedra runs on one GPU")
+        peaks, sizes = measured_peaks(), [n for n in args.sizes.split(",") if n] or list(bench_vugedra.SIZES)
+        sampler = ClockSampler(local)
+        sampler.start()
+        rows = bench_vugedra.measure(sizes, args.steps, peaks)
+        clocks = sampler.stop()
+        line = {"metric": "vugedra_decoder_tokens_per_s", "value": rows[0]["vugedra"]["prefill"]["tokens_per_s"], "unit": "tokens/s (prefill of the first size)", "n_gpus": 1,
+                "steps": args.steps, "warmup": 3, "higher_is_better": True, "vs_baseline": None, "dtype": "bf16 weights and activations",
+                "data": "synthetic", "config": {"workload": "Vugedra decoder beside the Katadra decoder at equal width, depth and attention heads", "sizes": sizes},
+                "clocks": clocks, "sizes": rows}
+        if args.kernels:
+            line["kernels"] = {n: bench_vugedra.kernel_table(bench_vugedra.SIZES[n], peaks) for n in sizes}
         print(json.dumps(line))
     elif args.workload == "ragged_step":
         line = ragged_step_measure(R, steps=args.steps, warmup=args.warmup, layers=args.layers)

@@ -71,18 +71,21 @@ class Engine:
         self.seqs, self.ctx = seqs, ctx
         mb = (ctx + 64) // 16 + 1
         pool = seqs * mb + 4
-        if which == "mixer":
-            from logismos_b200.mixer import MixerModel
-            cfg = mixer_config(z)
-            self.model = MixerModel(cfg, mixer_weights(cfg, z, seed), pool, mb, step_tokens, seqs, seqs, device=device)
-        else:
-            from logismos_b200.hybrid import HybridModel, random_int4_weights
-            cfg = hybrid_config(z)
-            self.model = HybridModel(cfg, random_int4_weights(cfg, seed), pool, mb, step_tokens, seqs, seqs, device=device)
+        cfg, self.model = self.make(which, z, pool, mb, step_tokens, seqs, device, seed)
         alloc = BlockAllocator(pool, mb, seed=1)
         self.tables = np.stack([alloc.ensure(i, ctx + 1) for i in range(seqs)])
         self.rng = np.random.Generator(np.random.PCG64(9))
         self.vocab, self.step_tokens = cfg["vocab"], step_tokens
+
+    def make(self, which, z, pool, mb, step_tokens, seqs, device, seed):
+        """The configuration and the executor."""
+        if which == "mixer":
+            from logismos_b200.mixer import MixerModel
+            cfg = mixer_config(z)
+            return cfg, MixerModel(cfg, mixer_weights(cfg, z, seed), pool, mb, step_tokens, seqs, seqs, device=device)
+        from logismos_b200.hybrid import HybridModel, random_int4_weights
+        cfg = hybrid_config(z)
+        return cfg, HybridModel(cfg, random_int4_weights(cfg, seed), pool, mb, step_tokens, seqs, seqs, device=device)
 
     def step(self, idx, cached, new):
         ids = self.rng.integers(0, self.vocab, int(sum(new)), dtype=np.uint32)

@@ -953,7 +953,7 @@ typedef struct lg_moe_route {
   int32_t n_experts, n_identity, top, n_always;
   void *weights, *pair_row, *identity;
   void *offsets, *row_token;    /* few tokens, fp32 */
-  void *counts, *pair_expert;   /* many tokens; pair_expert i32 [tokens, top] */
+  void *counts, *pair_expert;   /* many tokens; pair_expert i32 [tokens, top]: group << 20 | rank in the group, -1: identity */
   void *tiles, *n_tiles;
 } lg_moe_route_t;
 int32_t logismos_moe_few_tokens(void);  /* largest number of tokens of the one-launch form */

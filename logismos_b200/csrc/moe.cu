@@ -148,7 +148,7 @@ __global__ void __launch_bounds__(kRouteThreads)
 moe_route_kernel(RouteArgs p) {
   lg::pdl_prologue();
   __shared__ int count[kMaxOut], base[kMaxOut], group_s[kRouteTokens * kMaxTop], rank_s[kRouteTokens * kMaxTop];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, pairs = p.top + p.always;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int t0 = blockIdx.x * kRouteTokens, n = min(kRouteTokens, p.tokens - t0);
   for (int g = tid; g < p.experts; g += kRouteThreads) count[g] = 0;
   __syncthreads();
@@ -167,8 +167,7 @@ moe_route_kernel(RouteArgs p) {
   __syncthreads();
   for (int i = tid; i < n * p.top; i += kRouteThreads) {
     const int t = i / p.top, k = i - t * p.top, g = group_s[i];
-    p.pair_expert[(size_t)(t0 + t) * p.top + k] = g;
-    p.pair_row[(size_t)(t0 + t) * pairs + k] = g < 0 ? -1 : base[g] + rank_s[i];  // rank in the group, placed by the next launch
+    p.pair_expert[(size_t)(t0 + t) * p.top + k] = g < 0 ? -1 : (base[g] + rank_s[i]) | (g << 20);
   }
 }
 
@@ -188,12 +187,10 @@ moe_place_kernel(RouteArgs p, const uint4* h, uint4* gathered, int vecs) {
       if (lane == 0) p.pair_row[i] = start[p.experts + k - p.top] + t;
       continue;
     }
-    const int g = p.pair_expert[(size_t)t * p.top + k];
-    if (g < 0) continue;
-    const int row = start[g] + p.pair_row[i];
-    __syncwarp();
+    const int v = p.pair_expert[(size_t)t * p.top + k], row = v < 0 ? -1 : start[v >> 20] + (v & 0xfffff);
     if (lane == 0) p.pair_row[i] = row;
-    for (int v = lane; v < vecs; v += 32) gathered[(size_t)row * vecs + v] = h[(size_t)t * vecs + v];
+    if (row < 0) continue;
+    for (int c = lane; c < vecs; c += 32) gathered[(size_t)row * vecs + c] = h[(size_t)t * vecs + c];
   }
   if (blockIdx.x) return;
   for (int g = tid; g < groups; g += kRouteThreads) count[g] = (count[g] + 127) >> 7;
