@@ -343,7 +343,7 @@ def kernel_table(z, peaks, T=4096, seqs=64, ctx=8192):
     off, total = ops.build_decode_chunks(cl, chunk)
     off = off.to(dev)
     scr = torch.empty(lib.logismos_latent_decode_scratch_bytes(total, heads, R), dtype=torch.uint8, device=dev)
-    add("decode", "latent_decode + merge (ctx %d)" % ctx, [lambda s: lib.logismos_launch_latent_decode_bf16(P(qd), P(pool), P(tab), P(cg), P(off), P(od), P(scr), seqs, total, chunk, nb, seqs * nb, heads, R, 0.05, P(None), 0, P(st), s)] * 3,
+    add("decode", "latent_decode + merge (ctx %d)" % ctx, [lambda s: lib.logismos_launch_latent_decode_bf16(P(qd), P(pool), P(tab), P(cg), P(off), P(od), P(scr), seqs, total, chunk, nb, seqs * nb, heads, R, 0.05, P(None), 0, P(None), 0, 0, P(st), s)] * 3,
         seqs * (ctx * R * 2.0 + heads * R * 4.0), 4.0 * seqs * ctx * heads * R, like="paged_decode")
     del pool
     nkv = heads // 4

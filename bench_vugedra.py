@@ -212,6 +212,13 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
 
     def grouped(phase, name, m, n_main, n_tail, parts=False, copies_in=1, like=None):
         n = n_main + n_tail
+        if copies_in == 1 and 32 < m <= 512 and up(n, 128) // 128 * (up(m, 128) // 128) <= 74:   # summed over slices of k, then finished
+            ws, a, acc = [bf(n, H) for _ in range(copies(2.0 * n * H))], bf(m, H), zf(m, n)
+            out, tail = torch.zeros((m, n_main), device=dev, dtype=torch.bfloat16), zf(m, n_tail)
+            g = Groups(1, (i32 * 8)(n), n_main, A(tail), n_tail, 0.0, 0, 0)
+            keep.append((g, tail))
+            both = lambda s, w: lib.logismos_launch_linear_t_act_bf16(P(a), P(w), P(None), P(acc), m, n, H, H, n, 0x101, 0, 0, 0, P(st), s) or lib.logismos_launch_linear_groups_finish(P(acc), P(out), m, n, n, n_main, C.byref(g), s)
+            return add(phase, name + " (with finish)", [lambda s, w=w: both(s, w) for w in ws], 2.0 * n * H + 2.0 * m * H + 2.0 * m * n_main + 4.0 * m * n_tail, 2.0 * m * n * H, like)
         ws, a = [bf(n, H) for _ in range(copies(2.0 * n * H))], bf(copies_in, m, H)
         out, tail = torch.zeros((m, n_main), device=dev, dtype=torch.bfloat16), zf(m, n_tail)
         pt = torch.zeros((m, 2 * n_tail), device=dev, dtype=torch.bfloat16) if parts else None
@@ -230,7 +237,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
 
     def mixture(ph, m):
         """The router, the experts' products and the sum, with even choices."""
-        few = m <= lib.logismos_moe_few_tokens()
+        few = lib.logismos_moe_streams(m, TOP, EXPERTS, IDENTITY, 1, H, F)
         ld = up(EXPERTS + IDENTITY, 16)
         logits, corr, h = rf(m, ld), zf(ld), bf(m, H)
         wts, prow, ident, off, tok = zf(m, TOP), it(m, pairs), zf(m), it(groups + 1), it(m * pairs)
@@ -243,7 +250,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         else:
             r.counts, r.pair_expert, r.tiles, r.n_tiles = A(counts), A(pe), A(tiles), A(nt)
         keep.append((r, logits, corr, wts, prow, ident, off, tok, counts, pe, tiles, nt))
-        gemm(ph, "router", m, ld, H, 1 if 32 < m <= 512 else 3, like="latent projections")
+        gemm(ph, "router", m, ld, H, 1 if m > 32 else 3, like="latent projections")
         # by even chances: rows of the experts, and experts that have any
         n_rows, used = m * (active_experts() + 1), active_experts(m) + 1
         nw = max(2, min(6, int(3e8 // (6.0 * F * H * groups)) + 1))
@@ -253,7 +260,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         db, dl = 2.0 * used * F * H + 2.0 * n_rows * F + 2.0 * n_rows * H, 2.0 * n_rows * F * H
         if few:
             add(ph, "choice of experts", [lambda s: lib.logismos_launch_moe_route(Y(r), m, s)] * 4, m * (ld * 4.0 + 12.0 * pairs), like="post_norm")
-            ex = -(-m * TOP // EXPERTS)
+            ex = 8 if m <= 8 else 16
             add(ph, "experts, gate and up", [lambda s, w=w: lib.logismos_launch_linear_experts_small_bf16(P(h), P(w), P(mid), P(off), P(tok), groups, m, ex, 2 * F, H, H, F, 2, s) for w in wu], ub, ul, "gate/up")
             add(ph, "experts, down", [lambda s, w=w: lib.logismos_launch_linear_experts_small_bf16(P(mid), P(w), P(out), P(off), P(None), groups, m, ex, H, F, F, H, 0, s) for w in wd], db, dl, "down")
         else:
@@ -417,7 +424,6 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         lp2 = bf(m * nb, 16, R)
         add(ph, "= latent_norm_store", [lambda s: lib.logismos_launch_latent_norm_store(P(raw), NL, P(ones), P(ones), P(cqm), P(lp2), P(s1), m, Q, Q, R, R, 1e-6, m * nb * 16, 0, 1, None, P(st), s)] * 4, m * 10.0 * (Q + R))
         qd, ql, ol = bf(m, HD), bf(m, heads * Rp), bf(m, heads * Rp)
-        add(ph, "rotation of the queries", [lambda s: lib.logismos_launch_rotary_heads(P(qd), HD, P(ps), m, heads, DIM, NOPE, P(table), ROT, 0, s)] * 4, 4.0 * m * heads * ROT, like="unit_qk_store")
         for rr, name, like in ((Rp, "", "latent decoder"), (R, "= ", None)):
             wk = [bf(heads, rr, DIM) for _ in range(copies(2.0 * heads * rr * DIM))]
             tagged = lambda n: name + n + (" (latent decoder)" if name else "")
@@ -433,7 +439,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
             lscr = torch.empty(lib.logismos_latent_decode_scratch_bytes(lt, heads, rr), dtype=torch.uint8, device=dev)
             used = R + ROT if rr == Rp else R
             pl, g = (lpool, gd) if rr == Rp else (lp2, None)
-            add(ph, tagged("latent decode + merge (ctx %d)" % ctx), [lambda s: lib.logismos_launch_latent_decode_bf16(P(ql), P(pl), P(tab), P(cg), P(lo), P(ol), P(lscr), m, lt, ck, nb, m * nb, heads, rr, 0.05, P(g), hg, P(st), s)] * 3,
+            add(ph, tagged("latent decode + merge (ctx %d)" % ctx), [lambda s: lib.logismos_launch_latent_decode_bf16(P(ql), P(pl), P(tab), P(cg), P(lo), P(ol), P(lscr), m, lt, ck, nb, m * nb, heads, rr, 0.05, P(g), hg, P(table if rr == Rp else None), R, ROT, P(st), s)] * 3,
                 2.0 * m * ctx * used, 2.0 * m * ctx * heads * (used + R), like and "latent decode + merge (latent decoder)")
         del lpool, lp2
     return rows

@@ -155,6 +155,10 @@ uint32_t logismos_launch_linear_groups_tc_bf16(const void* a_bf16, const void* w
 uint32_t logismos_launch_linear_groups_small_bf16(const void* a_bf16, const void* w_bf16, void* out, int32_t m, int32_t n,
                                                   int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
                                                   void* stream);
+/* The same of one group from its sums acc f32 [m, ldc] over all n columns (which are cleared): bias, rounding and the tail.
+ * For a number of rows at which accumulating over slices of k is faster than whole tiles. */
+uint32_t logismos_launch_linear_groups_finish(void* acc_f32, void* out_bf16, int32_t m, int32_t n, int32_t ld_acc, int32_t ldc,
+                                              const lg_linear_groups_t* groups, void* stream);
 uint32_t logismos_launch_linear_groups_f32(const void* a_f32, const void* w_bf16, void* out_f32, int32_t m, int32_t n,
                                            int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
                                            void* stream);
@@ -643,7 +647,8 @@ uint32_t logismos_launch_latent_gather_bf16(const void* pool, const void* block_
  * logismos_latent_decode_scratch_bytes(total_chunks, heads, rank). A second launch merges split contexts. The
  * index arrays, and every cached row but the last of each context, must not be written by work still in
  * flight on the stream (they may be read ahead of the dependency wait). gate (f32 [rows, ld_gate], NULL: none): head h of
- * a row is multiplied by the sigmoid of its column h. */
+ * a row is multiplied by the sigmoid of its column h. rot_table (NULL: none; f32 [positions][rot_dims / 2][2]): channels
+ * rot_at .. rot_at + rot_dims (rot_at % 8 == 0) of q are turned by the angles of position context_lens - 1 as they are read. */
 int32_t logismos_pick_latent_chunk(const int32_t* host_context_lens, int32_t n_seqs, int32_t heads);
 int32_t logismos_latent_max_chunks(int32_t max_rows);
 size_t logismos_latent_decode_scratch_bytes(int32_t total_chunks, int32_t heads, int32_t rank);
@@ -652,7 +657,8 @@ uint32_t logismos_launch_latent_decode_bf16(const void* q_bf16, const void* pool
                                             void* out_bf16, void* scratch, int32_t rows, int32_t total_chunks,
                                             int32_t chunk_tokens, int32_t max_blocks, int32_t n_pool_blocks,
                                             int32_t heads, int32_t rank, float scale, const void* gate_f32,
-                                            int32_t ld_gate, void* status_i32, void* stream);
+                                            int32_t ld_gate, const void* rot_table_f32, int32_t rot_at, int32_t rot_dims,
+                                            void* status_i32, void* stream);
 /* The fp32 form for any rows of a step: row t of sequence seq_ids[t] sees keys 0 .. positions[t]. */
 uint32_t logismos_launch_latent_attention_f32(const void* q_f32, const void* pool_f32, const void* block_tables_i32,
                                               const void* seq_ids_i32, const void* positions_i32, void* out_f32,
@@ -956,7 +962,9 @@ typedef struct lg_moe_route {
   void *counts, *pair_expert;   /* many tokens; pair_expert i32 [tokens, top]: group << 20 | rank in the group, -1: identity */
   void *tiles, *n_tiles;
 } lg_moe_route_t;
-int32_t logismos_moe_few_tokens(void);  /* largest number of tokens of the one-launch form */
+/* 1: so few tokens are best served by the one-launch form and products that stream the experts' weights. */
+int32_t logismos_moe_streams(int32_t tokens, int32_t top, int32_t n_experts, int32_t n_identity, int32_t n_always, int32_t width,
+                             int32_t ff);
 int32_t logismos_moe_max_tiles(int32_t tokens, int32_t top, int32_t n_experts, int32_t n_always);
 uint32_t logismos_launch_moe_route(const lg_moe_route_t* args, int32_t tokens, void* stream);
 uint32_t logismos_launch_moe_place(const lg_moe_route_t* args, const void* h_bf16, void* gathered_bf16, int32_t ld,

@@ -143,7 +143,7 @@ def _declare(l, partial=False):
         "logismos_launch_depth_mix_conv_decode": [vp, i64, i32, vp, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp],
         "logismos_launch_latent_norm_store": [vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i64, i32, i32, vp, vp, vp],
         "logismos_launch_latent_gather_bf16": [vp, vp, i32, i32, vp, vp, vp, i32, i32, i32, i32, vp, vp],
-        "logismos_launch_latent_decode_bf16": [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
+        "logismos_launch_latent_decode_bf16": [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, i32, vp, vp],
         "logismos_launch_latent_attention_f32": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
         "lg_latent_create": [i32, vp, vp, C.POINTER(vp)],
         "lg_latent_load": [i32, C.c_char_p, vp, C.POINTER(vp)],
@@ -154,6 +154,7 @@ def _declare(l, partial=False):
         # state-space / parallel decoder
         "logismos_launch_linear_groups_tc_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp, vp],
         "logismos_launch_linear_groups_small_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
+        "logismos_launch_linear_groups_finish": [vp, vp, i32, i32, i32, i32, vp, vp],
         "logismos_launch_linear_groups_f32": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
         "logismos_launch_post_norm": [vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, vp],
         "logismos_launch_post_norm_shift_decode": [vp, i32, vp, vp, vp, vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, f32, vp],
@@ -237,7 +238,7 @@ def _declare(l, partial=False):
         "lg_mixer_logits_device": ([vp], vp),
         "logismos_window_context": ([i32, i32, i32], i32),
         "logismos_window_keys": ([i32, i32, i32, i32], i32),
-        "logismos_moe_few_tokens": ([], i32),
+        "logismos_moe_streams": ([i32] * 7, i32),
         "logismos_moe_max_tiles": ([i32, i32, i32, i32], i32),
         "logismos_latent_gather_rows": ([i32, i32], i32),
         "logismos_pick_latent_chunk": ([vp, i32, i32], i32),

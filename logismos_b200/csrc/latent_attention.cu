@@ -151,8 +151,18 @@ struct DecodeArgs {
   float sl2;
   const float* gate;          // [rows, ld_gate], NULL: none
   int ld_gate;
+  const float2* rot;          // [positions][rot_pairs], NULL: none
+  int rot_at, rot_pairs;
   int* status;
 };
+
+// channels col, col + 1 of a query (col even), turned if they are a rotated pair
+LG_DEVINL uint32_t rotate_pair(uint32_t u, int col, const DecodeArgs& p, int pos) {
+  const int pr = (col - p.rot_at) >> 1;
+  if (!p.rot || col < p.rot_at || pr >= p.rot_pairs) return u;
+  const float2 x = unpack_bf16x2(u), cs = __ldg(p.rot + (size_t)pos * p.rot_pairs + pr);
+  return pack_bf16x2(x.x * cs.x - x.y * cs.y, x.y * cs.x + x.x * cs.y);
+}
 
 LG_DEVINL float head_gate(const float* gate, size_t row, int ld, int head) { return gate ? 1.0f / (1.0f + __expf(-gate[row * ld + head])) : 1.0f; }
 
@@ -243,6 +253,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
       const int hr = u / cw, ch = u % cw;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
       if (h0 + hr < p.heads) v = *reinterpret_cast<const uint4*>(p.q + ((size_t)r * p.heads + h0 + hr) * R + ch * 8);
+      if (p.rot && ch * 8 >= p.rot_at)
+        v = make_uint4(rotate_pair(v.x, ch * 8, p, ctx - 1), rotate_pair(v.y, ch * 8 + 2, p, ctx - 1), rotate_pair(v.z, ch * 8 + 4, p, ctx - 1), rotate_pair(v.w, ch * 8 + 6, p, ctx - 1));
       *reinterpret_cast<uint4*>(after + (size_t)hr * R * 2 + ((ch ^ (hr & 7)) << 4)) = v;
     }
   }
@@ -264,6 +276,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_pool, DecodeArgs p,
           qf[i][ks][1] = in && ha + 8 < p.heads ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)8 * R) : 0u;
           qf[i][ks][2] = in && ha < p.heads ? *reinterpret_cast<const uint32_t*>(q0 + 8) : 0u;
           qf[i][ks][3] = in && ha + 8 < p.heads ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)8 * R + 8) : 0u;
+          if (p.rot && in && col + 8 >= p.rot_at) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) qf[i][ks][e] = rotate_pair(qf[i][ks][e], col + 8 * (e >> 1), p, ctx - 1);
+          }
         }
     }
     const int units = slabs * 4, u_per = (units + kWarps - 1) / kWarps, u0 = warp * u_per, u_n = max(0, min(units - u0, u_per));
@@ -630,16 +646,17 @@ size_t logismos_latent_decode_scratch_bytes(int32_t total_chunks, int32_t heads,
 uint32_t logismos_launch_latent_decode_bf16(const void* q, const void* pool, const void* block_tables_i32, const void* context_lens_i32,
                                             const void* chunk_offsets_i32, void* out, void* scratch, int32_t rows, int32_t total_chunks,
                                             int32_t chunk_tokens, int32_t max_blocks, int32_t n_pool_blocks, int32_t heads, int32_t rank,
-                                            float scale, const void* gate_f32, int32_t ld_gate, void* status_i32, void* stream) {
+                                            float scale, const void* gate_f32, int32_t ld_gate, const void* rot_table, int32_t rot_at, int32_t rot_dims,
+                                            void* status_i32, void* stream) {
   lg::LaunchScope launch_scope_;
-  if ((gate_f32 && ld_gate < heads) || !q || !pool || !out || !scratch || rows <= 0 || rows > 65535 || total_chunks < rows || chunk_tokens <= 0 || (chunk_tokens % 64) || max_blocks <= 0 ||
+  if ((gate_f32 && ld_gate < heads) || (rot_table && (rot_at < 0 || rot_at % 8 || rot_dims <= 0 || rot_dims % 2 || rot_at + rot_dims > rank || ((uintptr_t)rot_table & 7))) || !q || !pool || !out || !scratch || rows <= 0 || rows > 65535 || total_chunks < rows || chunk_tokens <= 0 || (chunk_tokens % 64) || max_blocks <= 0 ||
       n_pool_blocks <= 0 || heads <= 0 || rank <= 0 || (rank % 64) || rank > 1024 || (int64_t)n_pool_blocks * kBlockTokens > 0x7fffffff - 64 ||
       (((uintptr_t)q | (uintptr_t)pool | (uintptr_t)out | (uintptr_t)scratch) & 15))
     return lg::kInvalidValue;
   cudaStream_t s = (cudaStream_t)stream;
   DecodeArgs p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, (const int*)block_tables_i32, (const int*)context_lens_i32,
                (const int*)chunk_offsets_i32, (__nv_bfloat16*)out, (float*)scratch, nullptr, rows, heads, rank, chunk_tokens, max_blocks,
-               n_pool_blocks, scale * kLog2e, (const float*)gate_f32, ld_gate, (int*)status_i32};
+               n_pool_blocks, scale * kLog2e, (const float*)gate_f32, ld_gate, (const float2*)rot_table, rot_at, rot_dims / 2, (int*)status_i32};
   p.part_ml = (float2*)(p.part_o + (size_t)total_chunks * heads * rank);
   CUtensorMap map;
   if (!make_map(&map, pool, (uint64_t)n_pool_blocks * kBlockTokens, (uint64_t)rank, (uint64_t)rank, kBlockTokens)) return lg::kInvalidValue;

@@ -103,7 +103,7 @@ uint32_t attention(Latent* m, LLayer& L, cudaStream_t s) {
   if (B.n_dec > 0) {
     LG_TRY(head_linear(m, m->q.p, HD, L.w_ukt, L.c.heads, L.Rp, L.D, m->qlat.p, HR, B.n_dec, s), "latent queries");
     LG_TRY(logismos_launch_latent_decode_bf16(m->qlat.p, L.pool.p, m->dev(B.tables), m->dev(B.ctx), m->dev(B.chunks), m->olat.p, m->dec_scratch.p,
-                                              B.n_dec, m->total_chunks, m->chunk_tokens, MB, c.n_pool_blocks, L.c.heads, L.Rp, L.c.scale, nullptr, 0, st, s),
+                                              B.n_dec, m->total_chunks, m->chunk_tokens, MB, c.n_pool_blocks, L.c.heads, L.Rp, L.c.scale, nullptr, 0, nullptr, 0, 0, st, s),
            "latent decode");
     m->launches += m->total_chunks > B.n_dec ? 2 : 1;
     LG_TRY(head_linear(m, m->olat.p, HR, L.w_uv, L.c.heads, L.D, L.Rp, m->cat.p, L.Cw, B.n_dec, s), "latent values");

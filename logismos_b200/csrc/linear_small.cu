@@ -309,9 +309,48 @@ linear_f32_kernel(F32Args p) {
   }
 }
 
+// ---- sums over slices of k -> the outputs of a grouped projection -----------------------------------
+__global__ void __launch_bounds__(256)
+groups_finish_kernel(float* __restrict__ acc, __nv_bfloat16* __restrict__ out, int m, int n, int ld_acc, int ldc, lg_linear_groups_t g) {
+  lg::pdl_prologue();
+  const int c = 4 * (blockIdx.x * 256 + threadIdx.x), r = blockIdx.y;
+  if (c >= n) return;
+  float4* src = reinterpret_cast<float4*>(acc + (size_t)r * ld_acc + c);
+  float4 v = *src;
+  *src = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (c < g.n_main) {
+    if (g.bias) {
+      const float4 b = __ldg(reinterpret_cast<const float4*>(reinterpret_cast<const float*>(g.bias) + c));
+      v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+    }
+    *reinterpret_cast<uint2*>(out + (size_t)r * ldc + c) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+    return;
+  }
+  const int t = c - g.n_main, width = n - g.n_main;
+  const float cap = g.tail_cap;
+  if (cap > 0.0f) { v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap); v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap); }
+  *reinterpret_cast<float4*>(reinterpret_cast<float*>(g.tail) + (size_t)r * g.ld_tail + t) = v;
+  if (!g.tail_parts) return;
+  __nv_bfloat16* parts = reinterpret_cast<__nv_bfloat16*>(g.tail_parts) + (size_t)r * 2 * width + t;
+  const uint2 hi = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+  const float2 a = unpack_bf16x2(hi.x), b = unpack_bf16x2(hi.y);
+  *reinterpret_cast<uint2*>(parts) = hi;
+  *reinterpret_cast<uint2*>(parts + width) = make_uint2(pack_bf16x2(v.x - a.x, v.y - a.y), pack_bf16x2(v.z - b.x, v.w - b.y));
+}
+
 }  // namespace
 
 extern "C" {
+
+uint32_t logismos_launch_linear_groups_finish(void* acc, void* out, int32_t m, int32_t n, int32_t ld_acc, int32_t ldc, const lg_linear_groups_t* groups, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!acc || !out || m <= 0 || m > 65535 || n <= 0 || n % 4 || ld_acc < n || ld_acc % 4 || ldc % 4 || !lg::groups_ok(groups, n, ldc) || groups->n_groups != 1 ||
+      groups->n_main % 4 || (groups->n_main < n && groups->ld_tail % 4) || (((uintptr_t)acc | (uintptr_t)groups->bias | (uintptr_t)groups->tail) & 15) ||
+      (((uintptr_t)out | (uintptr_t)groups->tail_parts) & 7))
+    return lg::kInvalidValue;
+  lg::launch(groups_finish_kernel, dim3((unsigned)((n / 4 + 255) / 256), (unsigned)m), dim3(256), 0, (cudaStream_t)stream, (float*)acc, (__nv_bfloat16*)out, m, n, ld_acc, ldc, *groups);
+  return lg::launch_status();
+}
 
 static uint32_t small_any(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k, int32_t lda, int32_t ldc,
                           int32_t batch, int64_t a_stride, int64_t w_stride, int64_t out_stride, int32_t epilogue, float p0, float p1, float p2,

@@ -108,8 +108,13 @@ uint32_t latent_attention(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s
   LG_TRY(logismos_launch_latent_norm_store(raw, L.N, W.gain_q.p, W.gain_k.p, m->cq.p, L.kpool.p, m->dev(B.slots), T, L.Qp, L.c.q_rank, L.Rp, L.c.kv_rank, c.norm_eps,
                                            (int64_t)c.n_pool_blocks * kKvBlock, f32, acc, &rot, st, s), "latent norm and store");
   LG_TRY(linear(m, m->cq.p, L.Qp, W.w_uq, HD, L.Qp, m->proj.p, HD, LG_EPI_BF16, T, s), "queries");
-  LG_TRY(logismos_launch_rotary_heads(m->proj.p, HD, m->dev(B.pos), T, heads, L.Dh, L.Dn, angles, L.c.rot_dims, f32, s), "rotation of the queries");
-  m->launches += 2;
+  m->launches += 1;
+  const int turned = f32 ? 0 : B.n_dec;  // decode rows are turned by the decode kernel, in the latent space
+  if (T > turned) {
+    LG_TRY(logismos_launch_rotary_heads((uint8_t*)m->proj.p + (size_t)turned * HD * (f32 ? 4 : 2), HD, m->dev(B.pos) + turned, T - turned, heads, L.Dh, L.Dn, angles, L.c.rot_dims, f32, s),
+           "rotation of the queries");
+    m->launches += 1;
+  }
   const float* gate = (const float*)m->gate.p;
   if (f32) {
     LG_TRY(head_linear(m, m->proj.p, HD, W.w_ukt, heads, L.Rp, L.Dh, m->qlat.p, HR, T, s), "latent queries");
@@ -122,7 +127,7 @@ uint32_t latent_attention(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s
   if (B.n_dec > 0) {
     LG_TRY(head_linear(m, m->proj.p, HD, W.w_ukt, heads, L.Rp, L.Dh, m->qlat.p, HR, B.n_dec, s), "latent queries");
     LG_TRY(logismos_launch_latent_decode_bf16(m->qlat.p, L.kpool.p, m->dev(B.tables), m->dev(B.ctx), m->dev(V.chunks), m->olat.p, m->dec_scratch.p, B.n_dec, V.total,
-                                              V.chunk_tokens, MB, c.n_pool_blocks, heads, L.Rp, L.c.scale, gate, LG, st, s), "latent decode");
+                                              V.chunk_tokens, MB, c.n_pool_blocks, heads, L.Rp, L.c.scale, gate, LG, angles, L.Rc, L.c.rot_dims, st, s), "latent decode");
     m->launches += V.total > B.n_dec ? 2 : 1;
     LG_TRY(head_linear(m, m->olat.p, HR, W.w_uv, heads, L.Dh, L.Rp, m->act.p, L.Kout, B.n_dec, s), "latent values");
   }
@@ -160,7 +165,8 @@ uint32_t run_gated_kinds(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s)
 uint32_t run_mixture(Mixer* m, const MLayer& L, const MWeights& W, lg_mixture_out_t* out, cudaStream_t s) {
   const lg_mixer_layer_config_t& y = L.c;
   const int T = m->batch.T, Hp = m->Hp, n_routed = y.experts + y.identity, groups = y.experts + L.always, pairs = y.top + L.always, f32 = m->cfg.is_f32;
-  const bool few = f32 || T <= logismos_moe_few_tokens(), acc = T > 32 && m->accumulates(T);
+  const bool few = f32 || logismos_moe_streams(T, y.top, y.experts, y.identity, L.always, Hp, L.Fp);
+  const bool acc = T > 32 && !f32 && !logismos_get_deterministic();  // the narrow product is split over k whatever the rows
   void *logits = acc ? m->route_acc.p : m->route.p, *st = m->status.p;
   LG_TRY(linear(m, m->h.p, Hp, W.w_router, L.route_ld, Hp, logits, L.route_ld, acc ? LG_EPI_RESID_F32 : LG_EPI_F32, T, s), "router");
   lg_moe_route_t r{};
@@ -171,7 +177,7 @@ uint32_t run_mixture(Mixer* m, const MLayer& L, const MWeights& W, lg_mixture_ou
   if (few) {
     r.offsets = m->offsets.p; r.row_token = m->row_token.p;
     LG_TRY(logismos_launch_moe_route(&r, T, s), "choice of experts");
-    const int expected = (T * y.top + y.experts - 1) / y.experts;
+    const int expected = T <= 8 ? 8 : 16;
     if (f32) {
       LG_TRY(logismos_launch_linear_experts_f32(m->h.p, W.w_up.p, m->ffb.p, r.offsets, r.row_token, groups, T, 2 * L.Fp, Hp, Hp, L.Fp, LG_EPI_GLU_CLAMP, 1.0f, INFINITY,
                                                 0.0f, s), "experts, gate and up");

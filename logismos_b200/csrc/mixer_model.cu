@@ -41,6 +41,10 @@ uint32_t head_linear(Mixer* m, const void* a, int lda, const Buf& w, int heads, 
   return logismos_launch_linear_small_bf16(a, w.p, nullptr, out, rows, n, k, lda, ldc, heads, k, (int64_t)n * k, n, LG_EPI_BF16, 0, 0, 0, s);
 }
 
+// Whether an input projection of a few dozen rows is summed over slices of k, with a launch that finishes it: its tiles alone
+// would leave most SMs idle (3088 x 2048 at 64 rows: 16.1 us in tiles; summed 5.2, finished 2.5)
+bool splits_projections(const MLayer& L, int rows) { return L.groups.n_groups == 1 && rows > 32 && rows <= kAccRows && (L.N + 127) / 128 * ((rows + 127) / 128) <= 74; }
+
 uint32_t projections(Mixer* m, const MLayer& L, const MWeights& W, bool tail_parts, cudaStream_t s) {
   lg_linear_groups_t g = L.groups;
   g.tail = m->tail.p;
@@ -49,6 +53,11 @@ uint32_t projections(Mixer* m, const MLayer& L, const MWeights& W, bool tail_par
   m->launches += 1;
   const int Hp = m->Hp, rows = m->batch.T;
   if (m->cfg.is_f32) return logismos_launch_linear_groups_f32(m->h.p, W.w_in.p, m->proj.p, rows, L.N, Hp, Hp, g.n_main, &g, s);
+  if (splits_projections(L, rows) && m->accumulates(rows)) {
+    m->launches += 1;
+    if (uint32_t rc = logismos_launch_linear_t_act_bf16(m->h.p, W.w_in.p, nullptr, m->raw_acc.p, rows, L.N, Hp, Hp, L.N, LG_EPI_RESID_F32 | LG_EPI_STATIC_W, 0, 0, 0, m->status.p, s)) return rc;
+    return logismos_launch_linear_groups_finish(m->raw_acc.p, m->proj.p, rows, L.N, L.N, g.n_main, &g, s);
+  }
   if (stream_weights(rows, L.N, Hp, LG_EPI_BF16))
     return logismos_launch_linear_groups_small_bf16(m->h.p, W.w_in.p, m->proj.p, rows, L.N, Hp, Hp, g.n_main, &g, s);
   return logismos_launch_linear_groups_tc_bf16(m->h.p, W.w_in.p, m->proj.p, rows, L.N, Hp, Hp, g.n_main, &g, m->status.p, s);
@@ -397,6 +406,7 @@ uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_
     L.table = table_of(m, L.c);
     grow(z.proj, (size_t)L.groups.n_main);
     grow(z.tail, (size_t)L.groups.ld_tail);
+    if (splits_projections(L, 33)) grow(z.raw, (size_t)L.N);
     grow(z.act, (size_t)L.Kout);
     size_feed_forward(L, z);
     ok = ok && L.table != -2 && (is_gated_kind(L.c.kind) ? alloc_gated_kinds(m, L, z) : alloc_parallel_kinds(m, L, z));
@@ -412,17 +422,17 @@ uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_
   lim.extra_bytes = ((size_t)c.max_out_rows + m->views.size() * (S + 1)) * 4;
   m->acc_bytes = acc_rows * Hp * 4;
   m->raw_acc_bytes = c.is_f32 ? 0 : acc_rows * z.raw * 4;
-  m->route_acc_bytes = c.is_f32 ? 0 : acc_rows * z.route * 4;
+  m->route_acc_bytes = c.is_f32 ? 0 : T * z.route * 4;
   m->counts_bytes = z.groups * 4;
   ok = ok && m->x.alloc(T * Hp * 4) && zeroed(m->h, copies * T * Hp * esz) && zeroed(m->proj, T * z.proj * esz) && m->tail.alloc(T * z.tail * 4) &&
-       zeroed(m->act, T * z.act * esz) && zeroed(m->ffb, T * z.ff * esz) && zeroed(m->xbc, T * z.xbc * esz) && m->y.alloc(T * Hp * 4) && m->y_acc.alloc(m->acc_bytes) &&
+       zeroed(m->act, T * z.act * esz) && zeroed(m->ffb, T * z.ff * esz) && zeroed(m->xbc, T * z.xbc * esz) && m->y.alloc(T * Hp * 4) && m->y_acc.alloc(m->acc_bytes) && m->raw_acc.alloc(m->raw_acc_bytes) &&
        m->last.alloc((size_t)c.max_out_rows * Hp * esz) && m->logits.alloc((size_t)c.max_out_rows * c.vocab * 4) && m->tokens.alloc((size_t)c.max_out_rows * 4) &&
        m->status.alloc(4) && (!c.keep_layers || m->hist.alloc((size_t)(c.n_layers + 1) * T * Hp * 4));
   if (!c.is_f32)
     ok = ok && m->low2.alloc(T * z.low * 2) && m->z.alloc(T * z.z * 4) && m->attn_ws.alloc(z.attn_ws) && m->dec_scratch.alloc(z.scratch);
-  if (z.raw) {  // latent attention
+  if (z.lat) {  // latent attention
     const size_t rows = c.is_f32 ? T : S;    // that attend in the latent space
-    ok = ok && m->raw_acc.alloc(m->raw_acc_bytes) && m->cq.alloc(T * z.cq * esz) && m->gate.alloc(T * z.heads * 4) && m->qlat.alloc(rows * z.lat_q * esz) &&
+    ok = ok && m->cq.alloc(T * z.cq * esz) && m->gate.alloc(T * z.heads * 4) && m->qlat.alloc(rows * z.lat_q * esz) &&
          m->olat.alloc(rows * z.lat_q * esz);
     if (!c.is_f32) {
       const size_t tp = (size_t)logismos_latent_gather_rows((int32_t)lim.prefix_cap_tokens, c.max_step_seqs);

@@ -87,7 +87,8 @@ struct Mixer {
   std::vector<DecodeView> views;
   std::vector<RotationTable> tables;
   Buf x, h, proj, tail, low2, z, xbc, act, ffb, y, y_acc, hist, last, logits, tokens, status, attn_ws, dec_scratch, dev_batch;
-  Buf raw_acc, cq, gate, qlat, olat, lat, kbuf, vt, kv_start;                                                      // latent attention
+  Buf raw_acc;                          // sums of input projections over slices of k
+  Buf cq, gate, qlat, olat, lat, kbuf, vt, kv_start;                                                      // latent attention
   Buf route, route_acc, pair_w, pair_row, pair_expert, identity, offsets, row_token, counts, tiles, gathered, expert_rows;  // mixture
   StepBatch batch;
   std::vector<uint8_t> slot_phase;      // per state slot: the copy that holds its convolution and shift states
@@ -105,7 +106,8 @@ struct Mixer {
 // largest sizes over the layers, per token unless said otherwise (elements)
 struct Sizes {
   size_t proj = 0, tail = 0, act = 0, ff = 0, z = 0, low = 0, xbc = 0, attn_ws = 0, scratch = 0;   // the last two in bytes
-  size_t raw = 0, cq = 0, heads = 0, lat_q = 0, lat = 0, lat_heads = 0;                             // latent attention
+  size_t raw = 0;                                                                                    // of summed input projections
+  size_t cq = 0, heads = 0, lat_q = 0, lat = 0, lat_heads = 0;                             // latent attention
   size_t route = 0, pairs = 0, top = 0, groups = 0, expert_ff = 0;                                  // mixture
 };
 inline void grow(size_t& a, size_t b) { if (b > a) a = b; }

@@ -219,7 +219,15 @@ RouteArgs route_args(const lg_moe_route_t* a, int tokens) {
 
 extern "C" {
 
-int32_t logismos_moe_few_tokens(void) { return 128; }
+// Measured (us, choice included, streamed / tiles; experts, top, width x ff): 16, 2, 1024 x 512 at 64 / 96 tokens 30 / 31, 35 /
+// 31; 16, 2, 2048 x 1024 at 16 / 32 / 64 59 / 62, 63 / 61, 76 / 63; 16, 2, 4096 x 2048 at 4 / 8 / 16 102 / 112, 113 / 105, 159 /
+// 139; 64, 8, 2048 x 512 at 8 / 16 79 / 80, 105 / 89: the tiles win once the experts in use hold some 200 MB.
+int32_t logismos_moe_streams(int32_t tokens, int32_t top, int32_t n_experts, int32_t n_identity, int32_t n_always, int32_t width, int32_t ff) {
+  if (tokens > 64) return 0;
+  double idle = 1.0;
+  for (int32_t i = 0; i < tokens; ++i) idle *= 1.0 - (double)top / (n_experts + n_identity);
+  return (n_experts * (1.0 - idle) + n_always) * 6.0 * width * ff < 2e8 ? 1 : 0;
+}
 
 int32_t logismos_moe_max_tiles(int32_t tokens, int32_t top, int32_t n_experts, int32_t n_always) {
   return (int32_t)((int64_t)tokens * top / 128) + n_experts + (tokens + 127) / 128 * n_always;

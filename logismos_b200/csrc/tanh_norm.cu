@@ -81,19 +81,35 @@ tanh_norm_kernel(Args p) {
     if (!MIX && p.post.w) y[i] = p.y[(size_t)r * p.nv + v];
   }
   if (MIX) {
+    // four experts of every row at a time: first where their rows are, then all of these at once
+    constexpr int kBatch = 4;
 #pragma unroll
     for (int i = 0; i < RUN; ++i) {
       const int r = r0 + i;
-      if (r >= p.rows) continue;
-      const float id = p.identity[r];
+      const float id = r < p.rows ? p.identity[r] : 0.0f;
       if (id != 0.0f) add_scaled(y[i], id, load4(p.h, (size_t)r * p.nv + v, p.f32));
-      const int* rows = p.pair_row + (size_t)r * p.n_pairs;
-#pragma unroll 4
-      for (int k = 0; k < p.n_pairs; ++k) {
-        const int row = rows[k];
-        const float w = k < p.top ? p.weights[(size_t)r * p.top + k] : 1.0f;
-        if (row >= 0) add_scaled(y[i], w, load4(p.expert_rows, (size_t)row * p.nv + v, p.f32));
-      }
+    }
+    for (int k0 = 0; k0 < p.n_pairs; k0 += kBatch) {
+      int row[RUN][kBatch];
+      float w[RUN][kBatch];
+#pragma unroll
+      for (int i = 0; i < RUN; ++i)
+#pragma unroll
+        for (int j = 0; j < kBatch; ++j) {
+          const int r = r0 + i, k = k0 + j;
+          const bool ok = r < p.rows && k < p.n_pairs;
+          row[i][j] = ok ? p.pair_row[(size_t)r * p.n_pairs + k] : -1;
+          w[i][j] = ok && k < p.top ? p.weights[(size_t)r * p.top + k] : 1.0f;
+        }
+      float4 e[RUN][kBatch];
+#pragma unroll
+      for (int i = 0; i < RUN; ++i)
+#pragma unroll
+        for (int j = 0; j < kBatch; ++j) e[i][j] = row[i][j] >= 0 ? load4(p.expert_rows, (size_t)row[i][j] * p.nv + v, p.f32) : zero;
+#pragma unroll
+      for (int i = 0; i < RUN; ++i)
+#pragma unroll
+        for (int j = 0; j < kBatch; ++j) add_scaled(y[i], w[i][j], e[i][j]);
     }
   }
 #pragma unroll
@@ -140,6 +156,6 @@ extern "C" uint32_t logismos_launch_tanh_norm(void* y, int32_t zero_y, const lg_
     lg::launch(kern, dim3((unsigned)cols, (unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
-  if (mix) return run ? go(tanh_norm_kernel<true, 4>, 4) : go(tanh_norm_kernel<true, 1>, 1);
+  if (mix) return run ? go(tanh_norm_kernel<true, 2>, 2) : go(tanh_norm_kernel<true, 1>, 1);
   return run ? go(tanh_norm_kernel<false, 4>, 4) : go(tanh_norm_kernel<false, 1>, 1);
 }

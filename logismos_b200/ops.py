@@ -683,7 +683,7 @@ def latent_decode(q, pool, block_tables, context_lens, context_lens_host, scale,
     status = torch.zeros(1, dtype=torch.int32, device=q.device)
     with torch.cuda.device(q.device):
         check(lib.logismos_launch_latent_decode_bf16(_p(q), _p(pool), _p(block_tables), _p(context_lens), _p(off), _p(out), _p(scratch), rows, total,
-                                                     chunk, block_tables.shape[1], pool.shape[0], heads, rank, float(scale), None, 0, _p(status), _stream()),
+                                                     chunk, block_tables.shape[1], pool.shape[0], heads, rank, float(scale), None, 0, None, 0, 0, _p(status), _stream()),
               "latent_decode")
         _done(sync)
         if sync and int(status.item()) != 0:

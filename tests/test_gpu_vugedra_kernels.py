@@ -480,6 +480,59 @@ def test_grouped_projections_add_their_bias_to_the_main_columns():
         close(host(t), want[:, n_main:], 1e-5)
 
 
+@pytest.mark.parametrize("parts", [False, True])
+def test_finishing_a_summed_projection(parts):
+    rng = np.random.default_rng(3)
+    m, n_main, tail = 50, 384, 32
+    acc, b = rng.standard_normal((m, n_main + tail + 4)), rng.standard_normal(n_main)
+    ad, bd, out, t = fl(acc), fl(b), act(np.zeros((m, n_main)), False), fl(np.zeros((m, tail)))
+    tp = act(np.zeros((m, 2 * tail)), False) if parts else None
+    g = Groups(1, (i32 * 8)(n_main + tail), n_main, A(t), tail, 2.0 if parts else 0.0, A(tp), A(bd))
+    check(lib.logismos_launch_linear_groups_finish(P(ad), P(out), m, n_main + tail, n_main + tail + 4, n_main, C.byref(g), stream()), "finish")
+    want = acc[:, n_main:n_main + tail]
+    want = 2.0 * np.tanh(want / 2.0) if parts else want
+    close(host(out), acc[:, :n_main] + b, 3e-3)
+    close(host(t), want, 1e-6)
+    assert not ad[:, :n_main + tail].any()
+    if parts:
+        close(host(tp)[:, :tail], want, 3e-3)
+        close(host(tp)[:, :tail] + host(tp)[:, tail:], want, 2e-5)
+
+
+@pytest.mark.parametrize("heads,rank,at,dims", [(3, 64, 24, 6), (16, 576, 512, 64), (20, 128, 40, 88), (40, 640, 8, 2), (64, 576, 512, 32)])
+def test_latent_decode_turns_its_queries_and_gates_its_heads(heads, rank, at, dims):
+    rng = np.random.default_rng(rank)
+    lens = [1, 17, 64, 200]
+    n, mb = len(lens), 14
+    rot = {"dims": dims, "base": 500.0}
+    nb = sum(-(-v // 16) for v in lens)
+    tables, perm, used = -np.ones((n, mb), np.int32), rng.permutation(nb), 0
+    pool = 0.5 * rng.standard_normal((nb, 16, rank))
+    pd = act(pool, False)
+    pool = host(pd)
+    for s, v in enumerate(lens):
+        b = -(-v // 16)
+        tables[s, :b] = perm[used:used + b]
+        used += b
+    qd, gate = act(rng.standard_normal((n, heads, rank)), False), rng.standard_normal((n, heads + 3))
+    q, gd, tab, td, cl = host(qd), fl(gate), angles(rot, 256), ints(tables), ints(lens)
+    for chunk in (64, 1024):
+        off = np.concatenate([[0], np.cumsum([-(-v // chunk) for v in lens])]).astype(np.int32)
+        od, out, st = ints(off), act(np.zeros((n, heads, rank)), False), status()
+        scr = torch.empty(lib.logismos_latent_decode_scratch_bytes(int(off[-1]), heads, rank), dtype=torch.uint8, device=DEV)
+        check(lib.logismos_launch_latent_decode_bf16(P(qd), P(pd), P(td), P(cl), P(od), P(out), P(scr), n, int(off[-1]), chunk, mb, nb, heads, rank, 0.08, P(gd), heads + 3, P(tab), at,
+                                                     dims, P(st), stream()), "decode")
+        want = np.zeros((n, heads, rank))
+        for s, v in enumerate(lens):
+            c = pool[tables[s, np.arange(v) // 16], np.arange(v) % 16]
+            x = q[s:s + 1].copy()
+            x[..., at:at + dims] = R.rotate(x[..., at:at + dims], [v - 1], rot)
+            for a in range(heads):
+                want[s, a] = R.softmax(x[0, a] @ c.T * 0.08) @ c * R.sigmoid(gate[s, a])
+        close(host(out), want, 8e-3)
+        assert st.item() == 0
+
+
 def test_launchers_reject_what_they_cannot_address():
     x, st = fl(np.zeros((4, 64))), status()
     one = fl(np.ones(64))
