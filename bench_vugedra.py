@@ -250,7 +250,13 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         else:
             r.counts, r.pair_expert, r.tiles, r.n_tiles = A(counts), A(pe), A(tiles), A(nt)
         keep.append((r, logits, corr, wts, prow, ident, off, tok, counts, pe, tiles, nt))
-        gemm(ph, "router", m, ld, H, 1 if m > 32 else 3, like="latent projections")
+        fused = few and m * (EXPERTS + IDENTITY) * H <= 1 << 22
+        if fused:
+            wr, arrived = bf(ld, H), it(1)
+            r.h, r.w, r.width, r.arrived = A(h), A(wr), H, A(arrived)
+            keep.append((wr, arrived))
+        else:
+            gemm(ph, "router", m, ld, H, 1 if m > 32 else 3, like="latent projections")
         # by even chances: rows of the experts, and experts that have any
         n_rows, used = m * (active_experts() + 1), active_experts(m) + 1
         nw = max(2, min(6, int(3e8 // (6.0 * F * H * groups)) + 1))
@@ -259,7 +265,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         ub, ul = 2.0 * used * 2 * F * H + 2.0 * m * H + 2.0 * n_rows * F, 4.0 * n_rows * F * H
         db, dl = 2.0 * used * F * H + 2.0 * n_rows * F + 2.0 * n_rows * H, 2.0 * n_rows * F * H
         if few:
-            add(ph, "choice of experts", [lambda s: lib.logismos_launch_moe_route(Y(r), m, s)] * 4, m * (ld * 4.0 + 12.0 * pairs), like="post_norm")
+            add(ph, "router and choice of experts" if fused else "choice of experts", [lambda s: lib.logismos_launch_moe_route(Y(r), m, s)] * 4, m * (2.0 * H if fused else ld * 4.0) + 12.0 * m * pairs, like="post_norm")
             ex = 8 if m <= 8 else 16
             add(ph, "experts, gate and up", [lambda s, w=w: lib.logismos_launch_linear_experts_small_bf16(P(h), P(w), P(mid), P(off), P(tok), groups, m, ex, 2 * F, H, H, F, 2, s) for w in wu], ub, ul, "gate/up")
             add(ph, "experts, down", [lambda s, w=w: lib.logismos_launch_linear_experts_small_bf16(P(mid), P(w), P(out), P(off), P(None), groups, m, ex, H, F, F, H, 0, s) for w in wd], db, dl, "down")
@@ -369,6 +375,11 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         gemm(ph, "latent projections", m, NL, H, 1 if acc else 3, like="latent projections (latent decoder)")
         gemm(ph, "= latent projections (latent decoder)", m, Q + R, H, 1 if acc else 3)
         gemm(ph, "queries", m, HD, Q, 0, like="queries (latent decoder)")
+        if m <= 16:
+            ws, a, xo, ho = [bf(H, HD) for _ in range(copies(2.0 * H * HD))], bf(m, HD), rf(m, H), bf(m, H)
+            add(ph, "output projection with tanh norms", [lambda s, w=w: lib.logismos_launch_linear_small_tanh_norm(P(a), P(w), P(xo), Y(norm), P(ho), Y(norm), m, H, HD, HD, H, s) for w in ws],
+                2.0 * H * HD + 2.0 * m * HD + 10.0 * m * H, 2.0 * m * H * HD, "output projection (parallel layer)")
+            del ws
         gemm(ph, "output projection", m, H, HD, 1, like="output projection (parallel layer)")
         gemm(ph, "= output projection (parallel layer)", m, H, HD + tdw, 1)
         gemm(ph, "head", m, VOCAB, H, 3, like="gate/up")
@@ -398,6 +409,8 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         # windows rotate over shifted tables, so that the keys seen exceed L2 together
         vc = torch.full((m,), lib.logismos_window_context(ctx, WINDOW, KEEP), dtype=torch.int32)
         chunk = ops.pick_decode_chunk(vc, kv, DIM)
+        while chunk <= 512 and chunk > 64 and -(-int(vc[0]) // chunk) * m * kv < 256:
+            chunk //= 2
         offs, total = ops.build_decode_chunks(vc, chunk)
         offs = offs.to(dev)
         scr = torch.empty(max(16, lib.logismos_paged_decode_scratch_bytes(total, heads, DIM)), dtype=torch.uint8, device=dev)

@@ -130,6 +130,13 @@ uint32_t logismos_launch_linear_small_bf16(const void* a_bf16, const void* w_bf1
                                            int32_t ldc, int32_t batch, int64_t a_stride, int64_t w_stride,
                                            int64_t out_stride, int32_t epilogue, float p0, float p1,
                                            float p2, void* stream);
+/* The same for an output projection whose norms need no statistics: x f32 [m, ld] += post(a W^T), then h bf16 [m, ld] =
+ * next(x) (next NULL: none); n <= ld columns (lg_tanh_norm_t below). */
+struct lg_tanh_norm;
+uint32_t logismos_launch_linear_small_tanh_norm(const void* a_bf16, const void* w_bf16, void* x_f32,
+                                                const struct lg_tanh_norm* post, void* h_bf16,
+                                                const struct lg_tanh_norm* next, int32_t m, int32_t n, int32_t k,
+                                                int32_t lda, int32_t ld, void* stream);
 /* Several projections of the same rows in one launch, each block of columns with its own input: columns
  * [end[g - 1], end[g]) of the output are rows of W applied to activation copy g, copy g standing at a + g * m *
  * lda. Columns below n_main go to out (bf16 [m, n_main], row stride ldc), the others to tail (fp32, row stride
@@ -961,6 +968,9 @@ typedef struct lg_moe_route {
   void *offsets, *row_token;    /* few tokens, fp32 */
   void *counts, *pair_expert;   /* many tokens; pair_expert i32 [tokens, top]: group << 20 | rank in the group, -1: identity */
   void *tiles, *n_tiles;
+  const void *h, *w;            /* few tokens: the logits are w h (bf16 [outputs, width], [tokens, width], fp32 sums) instead */
+  int32_t width;
+  void* arrived;                /* i32, zero on entry and on return */
 } lg_moe_route_t;
 /* 1: so few tokens are best served by the one-launch form and products that stream the experts' weights. */
 int32_t logismos_moe_streams(int32_t tokens, int32_t top, int32_t n_experts, int32_t n_identity, int32_t n_always, int32_t width,

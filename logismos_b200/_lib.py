@@ -154,6 +154,7 @@ def _declare(l, partial=False):
         # state-space / parallel decoder
         "logismos_launch_linear_groups_tc_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp, vp],
         "logismos_launch_linear_groups_small_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
+        "logismos_launch_linear_small_tanh_norm": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp],
         "logismos_launch_linear_groups_finish": [vp, vp, i32, i32, i32, i32, vp, vp],
         "logismos_launch_linear_groups_f32": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
         "logismos_launch_post_norm": [vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, vp],

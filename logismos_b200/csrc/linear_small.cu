@@ -25,10 +25,16 @@ struct SmallArgs {
   lg_linear_groups_t groups;               // with kEpiGroups
   const int* offsets;                      // EXPERTS: batch entry b has the output rows offsets[b] .. offsets[b + 1]
   const int* row_idx;                      // and reads these input rows (NULL: the same)
+  // kEpiTanhNorm: out is the residual stream
+  float post_alpha, next_alpha;
+  const float *post_w, *post_b, *next_w, *next_b;
+  void* h;
 };
 
 // internal epilogue of the grouped projections (lg_linear_groups_t): main columns, then an fp32 tail
 constexpr int kEpiGroups = 6;
+// an output projection with the norms around the residual (lg_tanh_norm_t)
+constexpr int kEpiTanhNorm = 7;
 
 // activation copy of a block of columns starting at c
 LG_DEVINL int group_of(const lg_linear_groups_t& g, int c) {
@@ -174,6 +180,13 @@ linear_small_kernel(SmallArgs p) {
       continue;
     }
     const size_t o = (size_t)blockIdx.z * p.out_stride + (size_t)r * p.ldc + wrow;
+    if (p.epi == kEpiTanhNorm) {
+      float* xs = reinterpret_cast<float*>(p.out) + o;
+      const float x = *xs + fmaf(tanhf(p.post_alpha * v), __ldg(p.post_w + wrow), __ldg(p.post_b + wrow));
+      *xs = x;
+      if (p.next_w) reinterpret_cast<__nv_bfloat16*>(p.h)[o] = __float2bfloat16_rn(fmaf(tanhf(p.next_alpha * x), __ldg(p.next_w + wrow), __ldg(p.next_b + wrow)));
+      continue;
+    }
     if (p.epi == LG_EPI_BF16 || p.epi == LG_EPI_RELU2 || p.epi == kEpiGroups) reinterpret_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16_rn(v);
     else if (p.epi == LG_EPI_RESID_F32) reinterpret_cast<float*>(p.out)[o] += v;
     else reinterpret_cast<float*>(p.out)[o] = p.p0 > 0.0f ? p.p0 * tanhf(v / p.p0) : v;
@@ -309,6 +322,29 @@ linear_f32_kernel(F32Args p) {
   }
 }
 
+// the instantiation for a number of rows
+uint32_t small_by_rows(const SmallArgs& p, int batch, cudaStream_t s) {
+  const int m = p.m, n = p.n, k = p.k;
+  const bool glu = p.epi == LG_EPI_SWIGLU || p.epi == LG_EPI_GLU_CLAMP;
+  // two m16 tiles per CTA once that still leaves two CTAs per SM (the activations are then read half as often)
+  const int64_t ctas2 = (int64_t)((n + 31) / 32) * batch;
+  const bool two = glu || ctas2 >= 296;
+  const int steps = k / 32;
+  int warps = steps < 8 ? steps : 8;
+  if (steps >= 128 && !two) warps = 16;
+  const int nt = m <= 8 ? 1 : m <= 16 ? 2 : m <= 32 ? 4 : 8;
+  if (two) {
+    if (nt == 1) return launch_small<2, 1>(p, batch, warps, s);
+    if (nt == 2) return launch_small<2, 2>(p, batch, warps, s);
+    if (nt == 4) return launch_small<2, 4>(p, batch, warps, s);
+    return launch_small<2, 8>(p, batch, warps, s);
+  }
+  if (nt == 1) return launch_small<1, 1>(p, batch, warps, s);
+  if (nt == 2) return launch_small<1, 2>(p, batch, warps, s);
+  if (nt == 4) return launch_small<1, 4>(p, batch, warps, s);
+  return launch_small<1, 8>(p, batch, warps, s);
+}
+
 // ---- sums over slices of k -> the outputs of a grouped projection -----------------------------------
 __global__ void __launch_bounds__(256)
 groups_finish_kernel(float* __restrict__ acc, __nv_bfloat16* __restrict__ out, int m, int n, int ld_acc, int ldc, lg_linear_groups_t g) {
@@ -362,24 +398,19 @@ static uint32_t small_any(const void* a, const void* w, const void* bias, void* 
     return lg::kInvalidValue;
   const SmallArgs p{(const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (const float*)bias, out, m, n, k, lda, ldc, epilogue,
                     a_stride, w_stride, out_stride, p0, p1, p2, groups};
-  cudaStream_t s = (cudaStream_t)stream;
-  // two m16 tiles per CTA once that still leaves two CTAs per SM (the activations are then read half as often)
-  const int64_t ctas2 = (int64_t)((n + 31) / 32) * batch;
-  const bool two = glu || ctas2 >= 296;
-  const int steps = k / 32;
-  int warps = steps < 8 ? steps : 8;
-  if (steps >= 128 && !two) warps = 16;
-  const int nt = m <= 8 ? 1 : m <= 16 ? 2 : m <= 32 ? 4 : 8;
-  if (two) {
-    if (nt == 1) return launch_small<2, 1>(p, batch, warps, s);
-    if (nt == 2) return launch_small<2, 2>(p, batch, warps, s);
-    if (nt == 4) return launch_small<2, 4>(p, batch, warps, s);
-    return launch_small<2, 8>(p, batch, warps, s);
-  }
-  if (nt == 1) return launch_small<1, 1>(p, batch, warps, s);
-  if (nt == 2) return launch_small<1, 2>(p, batch, warps, s);
-  if (nt == 4) return launch_small<1, 4>(p, batch, warps, s);
-  return launch_small<1, 8>(p, batch, warps, s);
+  return small_by_rows(p, batch, (cudaStream_t)stream);
+}
+
+uint32_t logismos_launch_linear_small_tanh_norm(const void* a, const void* w, void* x, const lg_tanh_norm_t* post, void* h, const lg_tanh_norm_t* next, int32_t m,
+                                                int32_t n, int32_t k, int32_t lda, int32_t ld, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!a || !w || !x || !post || !post->w || !post->b || (next && (!h || !next->w || !next->b)) || m <= 0 || (m + 7) / 8 > 65535 || n <= 0 || n > ld || k <= 0 || k % 32 || lda < k ||
+      lda % 8 || (((uintptr_t)a | (uintptr_t)w) & 15))
+    return lg::kInvalidValue;
+  SmallArgs p{(const __nv_bfloat16*)a, (const __nv_bfloat16*)w, nullptr, x, m, n, k, lda, ld, kEpiTanhNorm, 0, 0, 0, 0, 0, 0, {}};
+  p.post_alpha = post->alpha; p.post_w = (const float*)post->w; p.post_b = (const float*)post->b;
+  if (next) { p.next_alpha = next->alpha; p.next_w = (const float*)next->w; p.next_b = (const float*)next->b; p.h = h; }
+  return small_by_rows(p, 1, (cudaStream_t)stream);
 }
 
 uint32_t logismos_launch_linear_small_bf16(const void* a, const void* w, const void* bias, void* out, int32_t m, int32_t n, int32_t k,

@@ -168,8 +168,11 @@ uint32_t run_mixture(Mixer* m, const MLayer& L, const MWeights& W, lg_mixture_ou
   const bool few = f32 || logismos_moe_streams(T, y.top, y.experts, y.identity, L.always, Hp, L.Fp);
   const bool acc = T > 32 && !f32 && !logismos_get_deterministic();  // the narrow product is split over k whatever the rows
   void *logits = acc ? m->route_acc.p : m->route.p, *st = m->status.p;
-  LG_TRY(linear(m, m->h.p, Hp, W.w_router, L.route_ld, Hp, logits, L.route_ld, acc ? LG_EPI_RESID_F32 : LG_EPI_F32, T, s), "router");
+  // a step of a few tokens with a small router: the product rides on the choice
+  const bool fused = few && !f32 && (int64_t)T * n_routed * Hp <= 1 << 22;
+  if (!fused) LG_TRY(linear(m, m->h.p, Hp, W.w_router, L.route_ld, Hp, logits, L.route_ld, acc ? LG_EPI_RESID_F32 : LG_EPI_F32, T, s), "router");
   lg_moe_route_t r{};
+  if (fused) { r.h = m->h.p; r.w = W.w_router.p; r.width = Hp; r.arrived = (uint8_t*)m->counts.p + m->counts_bytes - 4; }
   r.logits = logits; r.ld = L.route_ld; r.zero_logits = acc; r.correction = W.correction.p;
   r.n_experts = y.experts; r.n_identity = n_routed - y.experts; r.top = y.top; r.n_always = L.always;
   r.weights = m->pair_w.p; r.pair_row = m->pair_row.p; r.identity = m->identity.p;

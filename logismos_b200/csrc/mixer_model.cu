@@ -123,6 +123,15 @@ uint32_t tanh_norms(Mixer* m, void* y, bool zero_y, const lg_mixture_out_t* mix,
                                    m->status.p, s);
 }
 
+// the norm of a sublayer's output, and that of the next sublayer's input (NULL: none)
+void norms_after(Mixer* m, int l, bool second, const TanhNorm** post, const TanhNorm** next) {
+  const MWeights& W = m->weights[(size_t)m->layers[(size_t)l].owner];
+  *post = second ? &W.post2 : &W.post1;
+  *next = !second && m->layers[(size_t)l].c.ff > 0 ? &W.pre2 : l + 1 < m->cfg.n_layers ? &m->weights[(size_t)m->layers[(size_t)l + 1].owner].pre1 : nullptr;
+}
+
+constexpr int kFusedNormRows = 16;   // up to so many rows the norms around the residual ride on the output projection
+
 // What follows a sublayer of layer l: the norm of its output y, the residual, and the input of the next sublayer.
 // second: the feed-forward; mix: instead of y.
 uint32_t finish_sublayer(Mixer* m, int l, bool second, void* y, bool zero_y, const lg_mixture_out_t* mix, cudaStream_t s) {
@@ -132,14 +141,23 @@ uint32_t finish_sublayer(Mixer* m, int l, bool second, void* y, bool zero_y, con
   const int next = l + 1 < c.n_layers ? l + 1 : kNone;
   if (c.norm == LG_NORM_LAYER_POST)
     return norm_and_inputs(m, y, zero_y, second ? &W.norm2 : &W.norm1, second ? &W.norm2_b : &W.norm1_b, ff_next ? kPlain : next, s);
-  const TanhNorm* in = ff_next ? &W.pre2 : next != kNone ? &m->weights[(size_t)m->layers[(size_t)next].owner].pre1 : nullptr;
-  return tanh_norms(m, y, zero_y, mix, second ? &W.post2 : &W.post1, in, s);
+  const TanhNorm *post, *in;
+  norms_after(m, l, second, &post, &in);
+  return tanh_norms(m, y, zero_y, mix, post, in, s);
 }
 
 uint32_t output_projection(Mixer* m, int l, bool second, const void* a, int k, const Buf& w, cudaStream_t s) {
   const int T = m->batch.T, Hp = m->Hp;
   const bool acc = m->accumulates(T);
   void* y = acc ? m->y_acc.p : m->y.p;
+  if (m->cfg.norm == LG_NORM_TANH_AROUND && !m->cfg.is_f32 && T <= kFusedNormRows) {  // the norms in the product's epilogue
+    const TanhNorm *post, *next;
+    norms_after(m, l, second, &post, &next);
+    const lg_tanh_norm_t p = post->view(), n = next ? next->view() : lg_tanh_norm_t{};
+    m->launches += 1;
+    LG_TRY(logismos_launch_linear_small_tanh_norm(a, w.p, m->x.p, &p, m->h.p, next ? &n : nullptr, T, Hp, k, k, Hp, s), "output projection with norms");
+    return 0;
+  }
   LG_TRY(linear(m, a, k, w, Hp, k, y, Hp, acc ? LG_EPI_RESID_F32 : LG_EPI_F32, T, s), "output projection");
   LG_TRY(finish_sublayer(m, l, second, y, acc, nullptr, s), "output norm");
   return 0;
@@ -221,6 +239,14 @@ bool split_contexts(Mixer* m) {
     if (m->cfg.is_f32 || B.n_dec == 0) continue;
     for (int i = 0; i < B.n_dec; ++i) ctx[(size_t)i] = logismos_window_context(B.ctx[i], V.window, V.keep_first);
     V.chunk_tokens = V.latent ? logismos_pick_latent_chunk(ctx.data(), B.n_dec, V.heads) : logismos_pick_decode_chunk(ctx.data(), B.n_dec, V.kv, V.hd);
+    if (V.window && V.chunk_tokens == 512) {  // few sequences: what a window shows is cut in smaller pieces, down to a block per warp
+      auto pieces = [&](int c) {
+        int64_t n = 0;
+        for (int32_t v : ctx) n += (v + c - 1) / c;
+        return n;
+      };
+      while (V.chunk_tokens > 64 && pieces(V.chunk_tokens) * V.kv < 32768 / V.hd) V.chunk_tokens /= 2;
+    }
     V.total = logismos_build_decode_chunks(ctx.data(), B.n_dec, V.chunk_tokens, V.chunks);
     if (V.total < 0 || V.total > V.max_chunks) return false;
   }
@@ -308,7 +334,12 @@ int view_of(Mixer* m, const MLayer& L) {
     v.latent = latent;
     v.window = window;
     v.keep_first = keep;
-    v.max_chunks = latent ? logismos_latent_max_chunks(seqs) : seqs * ((m->cfg.max_blocks_per_seq * kKvBlock + 511) / 512);
+    const int longest = m->cfg.max_blocks_per_seq * kKvBlock;
+    v.max_chunks = latent ? logismos_latent_max_chunks(seqs) : seqs * ((longest + 511) / 512);
+    if (!latent && window) {  // cut in pieces of 64 while these are too few to fill the GPU
+      const int64_t seen = std::min((int64_t)longest, (int64_t)window + keep + 2 * kKvBlock);
+      v.max_chunks = std::max(v.max_chunks, (int)std::min((int64_t)seqs * ((seen + 63) / 64), (int64_t)seqs + 2048));
+    }
     m->views.push_back(v);
   }
   DecodeView& V = m->views[(size_t)i];
@@ -423,7 +454,7 @@ uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_
   m->acc_bytes = acc_rows * Hp * 4;
   m->raw_acc_bytes = c.is_f32 ? 0 : acc_rows * z.raw * 4;
   m->route_acc_bytes = c.is_f32 ? 0 : T * z.route * 4;
-  m->counts_bytes = z.groups * 4;
+  m->counts_bytes = z.groups ? (z.groups + 1) * 4 : 0;  // the last one counts the router's finished tokens
   ok = ok && m->x.alloc(T * Hp * 4) && zeroed(m->h, copies * T * Hp * esz) && zeroed(m->proj, T * z.proj * esz) && m->tail.alloc(T * z.tail * 4) &&
        zeroed(m->act, T * z.act * esz) && zeroed(m->ffb, T * z.ff * esz) && zeroed(m->xbc, T * z.xbc * esz) && m->y.alloc(T * Hp * 4) && m->y_acc.alloc(m->acc_bytes) && m->raw_acc.alloc(m->raw_acc_bytes) &&
        m->last.alloc((size_t)c.max_out_rows * Hp * esz) && m->logits.alloc((size_t)c.max_out_rows * c.vocab * 4) && m->tokens.alloc((size_t)c.max_out_rows * 4) &&

@@ -1,5 +1,6 @@
 // Router of a mixture of experts (lg_moe_route_t): the choice of experts per token and the grouping of rows by expert.
-//   few tokens    one CTA: choice, counts, offsets and row lists; the expert products read their rows through the list
+//   few tokens    one CTA: choice, counts, offsets and row lists; the expert products read their rows through the list. Or a
+//                 CTA per token that computes the token's logits too, the last one to finish then groups the rows
 //   many tokens   choice with per-CTA histograms (a row's rank in its group is unique, its order is not fixed; rows of a
 //                 group are independent), then a second launch that places the rows, copies them and lists the row tiles
 // Logits, softmax, choice and weights are fp32. A warp handles a token, a lane the experts lane, lane + 32, ...
@@ -28,6 +29,10 @@ struct RouteArgs {
   int4* tiles;
   int* n_tiles;
   int tokens;
+  const __nv_bfloat16* h;     // with the product: [tokens, width]
+  const __nv_bfloat16* w;     // [experts + identity, width]
+  int width;
+  int* arrived;
 };
 
 // float -> integer of the same order
@@ -36,11 +41,10 @@ LG_DEVINL uint32_t ordered(float x) {
   return u & 0x80000000u ? ~u : u | 0x80000000u;
 }
 
-// The token's experts: lane i < top receives the i-th choice and its weight. R: logits per lane.
+// The experts by a token's logits z: lane i < top receives the i-th choice and its weight. R: logits per lane.
 template <int R>
-LG_DEVINL void choose(const RouteArgs& p, int token, int lane, int& expert, float& weight) {
+LG_DEVINL void choose(const RouteArgs& p, float* z, int lane, int& expert, float& weight) {
   const int n = p.experts + p.identity;
-  float* z = p.logits + (size_t)token * p.ld;
   float s[R], c[R], mx = -INFINITY, sum = 0.0f;
 #pragma unroll
   for (int i = 0; i < R; ++i) {
@@ -110,26 +114,12 @@ LG_DEVINL void prefix(const int* count, int* start, int n) {
   __syncthreads();
 }
 
-template <int R>
-__global__ void __launch_bounds__(kFewThreads)
-moe_route_few_kernel(RouteArgs p) {
-  lg::pdl_prologue();
-  __shared__ int count[kMaxGroups], start[kMaxGroups + 1];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, groups = p.experts + p.always, pairs = p.top + p.always;
-  for (int g = tid; g < groups; g += kFewThreads) count[g] = g < p.experts ? 0 : p.tokens;
-  __syncthreads();
-  for (int t = warp; t < p.tokens; t += kFewThreads / 32) {
-    int expert;
-    float weight;
-    choose<R>(p, t, lane, expert, weight);
-    const int g = store_choice(p, t, lane, expert, weight);
-    // the rank in the group goes to pair_row for now, the group rides in its high bits
-    if (lane < p.top) p.pair_row[(size_t)t * pairs + lane] = g < 0 ? -1 : atomicAdd(&count[g], 1) | (g << 20);
-  }
-  __syncthreads();
+// the groups of all pairs, rank | group << 20 in pair_row (-1: none), counted in `count` -> offsets, rows and their tokens
+LG_DEVINL void group_rows(const RouteArgs& p, const int* count, int* start) {
+  const int groups = p.experts + p.always, pairs = p.top + p.always;
   prefix(count, start, groups);
-  for (int g = tid; g <= groups; g += kFewThreads) p.offsets[g] = start[g];
-  for (int i = tid; i < p.tokens * pairs; i += kFewThreads) {
+  for (int g = threadIdx.x; g <= groups; g += blockDim.x) p.offsets[g] = start[g];
+  for (int i = threadIdx.x; i < p.tokens * pairs; i += blockDim.x) {
     const int t = i / pairs, k = i - t * pairs;
     int row;
     if (k >= p.top) row = start[p.experts + k - p.top] + t;
@@ -144,6 +134,75 @@ moe_route_few_kernel(RouteArgs p) {
 }
 
 template <int R>
+__global__ void __launch_bounds__(kFewThreads)
+moe_route_few_kernel(RouteArgs p) {
+  lg::pdl_prologue();
+  __shared__ int count[kMaxGroups], start[kMaxGroups + 1];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, groups = p.experts + p.always, pairs = p.top + p.always;
+  for (int g = tid; g < groups; g += kFewThreads) count[g] = g < p.experts ? 0 : p.tokens;
+  __syncthreads();
+  for (int t = warp; t < p.tokens; t += kFewThreads / 32) {
+    int expert;
+    float weight;
+    choose<R>(p, p.logits + (size_t)t * p.ld, lane, expert, weight);
+    const int g = store_choice(p, t, lane, expert, weight);
+    if (lane < p.top) p.pair_row[(size_t)t * pairs + lane] = g < 0 ? -1 : atomicAdd(&count[g], 1) | (g << 20);
+  }
+  __syncthreads();
+  group_rows(p, count, start);
+}
+
+// CTA = token: its logits (a warp per router row, fp32 sums in a fixed order), its choice; the last CTA groups the rows
+template <int R>
+__global__ void __launch_bounds__(kRouteThreads)
+moe_router_kernel(RouteArgs p) {
+  lg::pdl_prologue();
+  __shared__ float z[kMaxOut];
+  __shared__ int count[kMaxGroups], start[kMaxGroups + 1], last;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, t = blockIdx.x, n = p.experts + p.identity, pairs = p.top + p.always;
+  const uint4* h = reinterpret_cast<const uint4*>(p.h + (size_t)t * p.width);
+  for (int e = warp; e < n; e += kRouteThreads / 32) {
+    const uint4* w = reinterpret_cast<const uint4*>(p.w + (size_t)e * p.width);
+    float s = 0.0f;
+#pragma unroll 4
+    for (int c = lane; c < p.width / 8; c += 32) {
+      const uint4 a = h[c], b = __ldg(w + c);
+      const uint32_t aw[4] = {a.x, a.y, a.z, a.w}, bw[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 x = unpack_bf16x2(aw[i]), y = unpack_bf16x2(bw[i]);
+        s = fmaf(x.x, y.x, fmaf(x.y, y.y, s));
+      }
+    }
+    s = warp_sum(s);
+    if (lane == 0) z[e] = s;
+  }
+  __syncthreads();
+  if (warp == 0) {
+    int expert;
+    float weight;
+    choose<R>(p, z, lane, expert, weight);
+    const int g = store_choice(p, t, lane, expert, weight);
+    if (lane < p.top) p.pair_row[(size_t)t * pairs + lane] = g;
+    __threadfence();
+    if (lane == 0) last = atomicAdd(p.arrived, 1) == (int)gridDim.x - 1;
+  }
+  __syncthreads();
+  if (!last) return;
+  __threadfence();
+  if (tid == 0) *p.arrived = 0;
+  for (int g = tid; g < p.experts + p.always; g += kRouteThreads) count[g] = g < p.experts ? 0 : p.tokens;
+  __syncthreads();
+  volatile int* groups = p.pair_row;
+  for (int i = tid; i < p.tokens * p.top; i += kRouteThreads) {
+    const int at = i / p.top * pairs + i % p.top, g = groups[at];
+    if (g >= 0) groups[at] = atomicAdd(&count[g], 1) | (g << 20);
+  }
+  __syncthreads();
+  group_rows(p, count, start);
+}
+
+template <int R>
 __global__ void __launch_bounds__(kRouteThreads)
 moe_route_kernel(RouteArgs p) {
   lg::pdl_prologue();
@@ -155,7 +214,7 @@ moe_route_kernel(RouteArgs p) {
   for (int t = warp; t < n; t += kRouteThreads / 32) {
     int expert;
     float weight;
-    choose<R>(p, t0 + t, lane, expert, weight);
+    choose<R>(p, p.logits + (size_t)(t0 + t) * p.ld, lane, expert, weight);
     const int g = store_choice(p, t0 + t, lane, expert, weight);
     if (lane < p.top) {
       group_s[t * p.top + lane] = g;
@@ -205,14 +264,14 @@ moe_place_kernel(RouteArgs p, const uint4* h, uint4* gathered, int vecs) {
 }
 
 bool route_ok(const lg_moe_route_t* a, int tokens) {
-  return a && tokens > 0 && tokens < (1 << 20) && a->logits && a->correction && a->weights && a->pair_row && a->identity && a->n_experts > 0 &&
-         a->n_identity >= 0 && a->n_experts + a->n_identity <= kMaxOut && a->ld >= a->n_experts + a->n_identity && a->top > 0 && a->top <= kMaxTop &&
+  return a && tokens > 0 && tokens < (1 << 20) && (a->logits || a->h) && a->correction && a->weights && a->pair_row && a->identity && a->n_experts > 0 &&
+         a->n_identity >= 0 && a->n_experts + a->n_identity <= kMaxOut && (a->h || a->ld >= a->n_experts + a->n_identity) && a->top > 0 && a->top <= kMaxTop &&
          a->top <= a->n_experts + a->n_identity && a->n_always >= 0 && a->n_always <= kMaxAlways;
 }
 RouteArgs route_args(const lg_moe_route_t* a, int tokens) {
   return RouteArgs{(float*)a->logits, a->ld, a->zero_logits, (const float*)a->correction, a->n_experts, a->n_identity, a->top, a->n_always, (float*)a->weights,
                    (int*)a->pair_row, (float*)a->identity, (int*)a->offsets, (int*)a->row_token, (int*)a->counts, (int*)a->pair_expert, (int4*)a->tiles,
-                   (int*)a->n_tiles, tokens};
+                   (int*)a->n_tiles, tokens, (const __nv_bfloat16*)a->h, (const __nv_bfloat16*)a->w, a->width, (int*)a->arrived};
 }
 
 }  // namespace
@@ -238,14 +297,16 @@ uint32_t logismos_launch_moe_route(const lg_moe_route_t* a, int32_t tokens, void
   lg::LaunchScope launch_scope_;
   const bool few = a && a->offsets;
   if (!route_ok(a, tokens) || (few ? !a->row_token : !a->counts || !a->pair_expert)) return lg::kInvalidValue;
-  const RouteArgs p = route_args(a, tokens);
-  const dim3 grid(few ? 1u : (unsigned)((tokens + kRouteTokens - 1) / kRouteTokens)), block(few ? kFewThreads : kRouteThreads);
+  if (a->h && (!few || !a->w || !a->arrived || a->width <= 0 || a->width % 8 || (((uintptr_t)a->h | (uintptr_t)a->w) & 15))) return lg::kInvalidValue;
+  RouteArgs p = route_args(a, tokens);
+  if (p.h) p.zero = 0;
+  const dim3 grid(p.h ? (unsigned)tokens : few ? 1u : (unsigned)((tokens + kRouteTokens - 1) / kRouteTokens)), block(few && !p.h ? kFewThreads : kRouteThreads);
   auto go = [&](auto kern) -> uint32_t {
     lg::launch(kern, grid, block, 0, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
   const int n = p.experts + p.identity;
-#define LG_ROUTE(R) (few ? go(moe_route_few_kernel<R>) : go(moe_route_kernel<R>))
+#define LG_ROUTE(R) (p.h ? go(moe_router_kernel<R>) : few ? go(moe_route_few_kernel<R>) : go(moe_route_kernel<R>))
   return n <= 32 ? LG_ROUTE(1) : n <= 64 ? LG_ROUTE(2) : n <= 128 ? LG_ROUTE(4) : n <= 256 ? LG_ROUTE(8) : LG_ROUTE(16);
 #undef LG_ROUTE
 }

@@ -49,4 +49,4 @@ class MixtureOut(C.Structure):
 
 class MoeRoute(C.Structure):
     _fields_ = [("logits", vp)] + _ints("ld", "zero_logits") + [("correction", vp)] + _ints("n_experts", "n_identity", "top", "n_always") + _pointers(
-               "weights", "pair_row", "identity", "offsets", "row_token", "counts", "pair_expert", "tiles", "n_tiles")
+               "weights", "pair_row", "identity", "offsets", "row_token", "counts", "pair_expert", "tiles", "n_tiles", "h", "w") + [("width", i32), ("arrived", vp)]

@@ -383,7 +383,7 @@ def plain_mixture(h, z, corr, top, E, up, down, always):
 
 
 @pytest.mark.parametrize("E,I,top,always,F,H", MIXTURES)
-@pytest.mark.parametrize("tokens,form", [(1, "few"), (7, "few"), (100, "few"), (130, "many"), (400, "many"), (33, "many"), (2500, "many"), (50, "f32")])
+@pytest.mark.parametrize("tokens,form", [(1, "few"), (7, "few"), (100, "few"), (130, "many"), (400, "many"), (33, "many"), (2500, "many"), (50, "f32"), (1, "router"), (9, "router"), (60, "router")])
 def test_mixture_of_experts(E, I, top, always, F, H, tokens, form):
     if tokens > 1000 and E != 5:
         return
@@ -395,8 +395,14 @@ def test_mixture_of_experts(E, I, top, always, F, H, tokens, form):
     if I == 300:
         corr[:E] -= 2.0       # every choice an identity expert: groups without rows
     z, corr = z.astype(np.float32), corr.astype(np.float32)
+    wr = R.bf16(2 * rng.standard_normal((n, H)) / np.sqrt(H))
     hd = act(rng.standard_normal((tokens, H)), fp32)
     h = host(hd)
+    if form == "router":      # the logits are a product of the rows: no close calls
+        z[:, :n] = h @ wr.T
+        ranked = -np.sort(-(R.softmax(z[:, :n].astype(np.float64)) + corr), axis=1)
+        if top < n:
+            corr = (corr + np.where((ranked[:, top - 1] - ranked[:, top]).min() < 1e-6, 1e-4 * rng.standard_normal(n), 0)).astype(np.float32)
     up = R.bf16(rng.standard_normal((G, 2, F, H)) / np.sqrt(H))
     down = R.bf16(rng.standard_normal((G, H, F)) / np.sqrt(F))
     wu = np.stack([np.concatenate([np.concatenate([up[g, 0, i:i + 32], up[g, 1, i:i + 32]]) for i in range(0, F, 32)]) for g in range(G)])
@@ -409,6 +415,11 @@ def test_mixture_of_experts(E, I, top, always, F, H, tokens, form):
     if form != "many":
         off, tok = it(G + 1), it(tokens * pairs)
         r.offsets, r.row_token = A(off), A(tok)
+        if form == "router":
+            wrd, arrived = dev(wr, torch.bfloat16), torch.zeros(1, dtype=torch.int32, device=DEV)
+            r.logits, r.h, r.w, r.width, r.arrived = 0, A(hd), A(wrd), H, A(arrived)
+            check(lib.logismos_launch_moe_route(C.byref(r), tokens, stream()), "route")     # twice: it leaves its counter cleared
+            assert not arrived.any()
         check(lib.logismos_launch_moe_route(C.byref(r), tokens, stream()), "route")
         if fp32:
             check(lib.logismos_launch_linear_experts_f32(P(hd), P(keep[2]), P(mid), P(off), P(tok), G, tokens, 2 * F, H, H, F, 4, 1.0, float("inf"), 0.0, stream()), "up")
@@ -435,7 +446,7 @@ def test_mixture_of_experts(E, I, top, always, F, H, tokens, form):
     # the choice itself: exact, and every pair has a row of its own
     chosen, weight = R.route(z[:, :n].astype(np.float64), corr.astype(np.float64), top)
     pr = prow.cpu().numpy()
-    assert np.array_equal(pr[:, :top] < 0, chosen >= E) and not keep[0][:, :n].any()
+    assert np.array_equal(pr[:, :top] < 0, chosen >= E) and (form == "router" or not keep[0][:, :n].any())
     close(host(wts), weight, 1e-5)
     close(host(ident) + 1e-3, np.where(chosen >= E, weight, 0).sum(1) + 1e-3, 1e-5)
     used = pr[pr >= 0]
@@ -478,6 +489,26 @@ def test_grouped_projections_add_their_bias_to_the_main_columns():
         want = host(x) @ w.T
         close(host(out), want[:, :n_main] + b, 1e-5 if route == "f32" else 3e-3)
         close(host(t), want[:, n_main:], 1e-5)
+
+
+@pytest.mark.parametrize("m,n,k", [(1, 64, 64), (7, 192, 256), (16, 1024, 512), (12, 4096, 4096)])
+@pytest.mark.parametrize("last", [False, True])
+def test_output_projection_with_its_norms(m, n, k, last):
+    rng = np.random.default_rng(n)
+    ld = n + 64
+    a, w = act(rng.standard_normal((m, k)), False), R.bf16(rng.standard_normal((n, k)) / np.sqrt(k))
+    post, nxt, x = tanh_vectors(rng, n, ld), tanh_vectors(rng, n, ld), 2 * rng.standard_normal((m, ld))
+    keep = [[fl(v) for v in p[1:]] for p in (post, nxt)]
+    tp, tn = (TanhNorm(p[0], A(k_[0]), A(k_[1])) for p, k_ in zip((post, nxt), keep))
+    xd, hd, wd = fl(x), act(np.zeros((m, ld)), False), dev(w, torch.bfloat16)
+    check(lib.logismos_launch_linear_small_tanh_norm(P(a), P(wd), P(xd), C.byref(tp), P(hd), None if last else C.byref(tn), m, n, k, k, ld, stream()), "projection")
+    want = x[:, :n] + R.tanh_norm(host(a) @ w.T, post[0], post[1][:n], post[2][:n])
+    close(host(xd)[:, :n], want, 2e-6)
+    assert np.array_equal(host(xd)[:, n:], x[:, n:].astype(np.float32)) and (host(hd)[:, n:] == 0).all()
+    if last:
+        assert not hd.any()
+    else:
+        close(host(hd)[:, :n], R.tanh_norm(want, nxt[0], nxt[1][:n], nxt[2][:n]), 3e-3)
 
 
 @pytest.mark.parametrize("parts", [False, True])
