@@ -40,6 +40,7 @@ struct Args {
   NormVec post, next;
   void* h;
   int f32, rows, nv;
+  unsigned cols;  // CTAs per row
   // mixture
   const void* expert_rows;
   const int* pair_row;
@@ -51,19 +52,22 @@ struct Args {
   int* status;
 };
 
+// The sum over experts waits for rows at scattered places: as many threads as the SM takes, few rows in flight in each.
 template <bool MIX, int RUN>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, MIX ? 16 : 1)
 tanh_norm_kernel(Args p) {
   lg::pdl_trigger();
-  const int v = blockIdx.x * kThreads + threadIdx.x, r0 = blockIdx.y * RUN;
+  const int v = (int)(blockIdx.x % p.cols) * kThreads + threadIdx.x, r0 = (int)(blockIdx.x / p.cols) * RUN;
   const bool in = v < p.nv;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  // the vectors of the norms do not depend on the kernels before this one
   float4 w1 = zero, b1 = zero, w2 = zero, b2 = zero;
-  if (in && p.post.w) { w1 = __ldg(p.post.w + v); b1 = __ldg(p.post.b + v); }
-  if (in && p.next.w) { w2 = __ldg(p.next.w + v); b2 = __ldg(p.next.b + v); }
+  const auto vectors = [&] {
+    if (p.post.w) { w1 = __ldg(p.post.w + v); b1 = __ldg(p.post.b + v); }
+    if (p.next.w) { w2 = __ldg(p.next.w + v); b2 = __ldg(p.next.b + v); }
+  };
+  if (!MIX && in) vectors();  // they do not depend on the kernels before this one
   lg::pdl_wait();
-  if (MIX && blockIdx.x == 0 && blockIdx.y == 0 && p.counts)
+  if (MIX && blockIdx.x == 0 && p.counts)
     for (int g = threadIdx.x; g < p.n_counts; g += kThreads) p.counts[g] = 0;
   if (!in) return;
   float4 x[RUN], y[RUN];
@@ -81,8 +85,8 @@ tanh_norm_kernel(Args p) {
     if (!MIX && p.post.w) y[i] = p.y[(size_t)r * p.nv + v];
   }
   if (MIX) {
-    // four experts of every row at a time: first where their rows are, then all of these at once
-    constexpr int kBatch = 4;
+    // three experts of every row at a time: first where their rows are, then all of these at once
+    constexpr int kBatch = 3;
 #pragma unroll
     for (int i = 0; i < RUN; ++i) {
       const int r = r0 + i;
@@ -111,6 +115,7 @@ tanh_norm_kernel(Args p) {
 #pragma unroll
         for (int j = 0; j < kBatch; ++j) add_scaled(y[i], w[i][j], e[i][j]);
     }
+    vectors();
   }
 #pragma unroll
   for (int i = 0; i < RUN; ++i) {
@@ -141,21 +146,20 @@ extern "C" uint32_t logismos_launch_tanh_norm(void* y, int32_t zero_y, const lg_
                                                                               mix->top < 0 || mix->top > mix->n_pairs)) ||
       (((uintptr_t)x | (uintptr_t)y | (uintptr_t)h) & 15))
     return lg::kInvalidValue;
-  Args p{(float4*)y, zero_y, (const int*)row_idx, n_src_rows, (float4*)x, vec(post), vec(next), h, out_f32, rows, ld / 4};
+  Args p{(float4*)y, zero_y, (const int*)row_idx, n_src_rows, (float4*)x, vec(post), vec(next), h, out_f32, rows, ld / 4, (unsigned)(ld / 4 + kThreads - 1) / kThreads};
   p.status = (int*)status;
   if (mix) {
     p.expert_rows = mix->rows; p.pair_row = (const int*)mix->pair_row; p.weights = (const float*)mix->weights; p.identity = (const float*)mix->identity;
     p.n_pairs = mix->n_pairs; p.top = mix->top; p.counts = (int*)mix->counts; p.n_counts = mix->n_counts;
   }
-  const int cols = (p.nv + kThreads - 1) / kThreads;
   // several rows per thread once that still leaves a few CTAs per SM
-  const bool run = (int64_t)cols * rows >= 148 * 16;
+  const bool run = (int64_t)p.cols * rows >= 148 * 16;
   auto go = [&](auto kern, int per) -> uint32_t {
-    const int64_t blocks = ((int64_t)rows + per - 1) / per;
-    if (blocks > 65535) return lg::kInvalidValue;
-    lg::launch(kern, dim3((unsigned)cols, (unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, p);
+    const int64_t blocks = ((int64_t)rows + per - 1) / per * p.cols;
+    if (blocks > INT32_MAX) return lg::kInvalidValue;
+    lg::launch(kern, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
-  if (mix) return run ? go(tanh_norm_kernel<true, 2>, 2) : go(tanh_norm_kernel<true, 1>, 1);
+  if (mix) return go(tanh_norm_kernel<true, 1>, 1);
   return run ? go(tanh_norm_kernel<false, 4>, 4) : go(tanh_norm_kernel<false, 1>, 1);
 }
