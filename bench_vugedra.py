@@ -167,7 +167,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
     bandwidth and FLOPs over the measured bf16 peak). Operands rotate over copies that exceed L2 together."""
     import torch
     from logismos_b200 import ops
-    from logismos_b200._lib import i32, lib
+    from logismos_b200._lib import check, i32, lib
     from logismos_b200.structs import Groups, LatentRotary, MixtureOut, MoeRoute, ScoreBias, TanhNorm, TimeMix, Window
     dev, rows, keep = "cuda", [], []
     P = lambda t: C.c_void_p(t.data_ptr() if t is not None else 0)
@@ -236,7 +236,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
     Y = lambda n: C.byref(n)
 
     def mixture(ph, m):
-        """The router, the experts' products and the sum, with even choices."""
+        """The router, the experts' products and the sum."""
         few = lib.logismos_moe_streams(m, TOP, EXPERTS, IDENTITY, 1, H, F)
         ld = up(EXPERTS + IDENTITY, 16)
         logits, corr, h = rf(m, ld), zf(ld), bf(m, H)
@@ -257,8 +257,10 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
             keep.append((wr, arrived))
         else:
             gemm(ph, "router", m, ld, H, 1 if m > 32 else 3, like="latent projections")
-        # by even chances: rows of the experts, and experts that have any
-        n_rows, used = m * (active_experts() + 1), active_experts(m) + 1
+        # rows of the experts, and experts that have any
+        check(lib.logismos_launch_moe_route(Y(r), m, torch.cuda.current_stream().cuda_stream), "moe_route")
+        rows_of = (off[1:] - off[:-1] if few else counts).cpu().numpy()
+        n_rows, used = int(rows_of.sum()) + (0 if few else m), int((rows_of > 0).sum()) + (0 if few else 1)
         nw = max(2, min(6, int(3e8 // (6.0 * F * H * groups)) + 1))
         wu, wd = [bf(groups, 2 * F, H) for _ in range(nw)], [bf(groups, H, F) for _ in range(nw)]
         mid, out = bf(m * pairs, F), bf(m * pairs, H)
@@ -274,7 +276,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
                 counts.zero_()
                 return lib.logismos_launch_moe_route(Y(r), m, s)
             add(ph, "choice of experts (with clearing)", [choose] * 4, m * (ld * 4.0 + 12.0 * pairs), like="post_norm")
-            add(ph, "rows by expert", [lambda s: lib.logismos_launch_moe_place(Y(r), P(h), P(gat), H, m, s)] * 4, m * H * 2.0 * (1 + active_experts()), like="latent_gather")
+            add(ph, "rows by expert", [lambda s: lib.logismos_launch_moe_place(Y(r), P(h), P(gat), H, m, s)] * 4, 2.0 * H * n_rows, like="latent_gather")
             add(ph, "experts, gate and up", [lambda s, w=w: lib.logismos_launch_linear_experts_tc_bf16(P(gat), m * pairs, P(h), m, P(w), P(mid), P(tiles), P(nt), mt, groups, 2 * F, H, H, F, 2, P(st), s) for w in wu], ub, ul, "gate/up")
             add(ph, "experts, down", [lambda s, w=w: lib.logismos_launch_linear_experts_tc_bf16(P(mid), m * pairs, P(None), 0, P(w), P(out), P(tiles), P(nt), mt, groups, H, F, F, H, 0, P(st), s) for w in wd], db, dl, "down")
         del wu, wd

@@ -52,10 +52,12 @@ struct Args {
   int* status;
 };
 
-// The sum over experts waits for rows at scattered places: as many threads as the SM takes, few rows in flight in each.
-template <bool MIX, int RUN>
-__global__ void __launch_bounds__(kThreads, MIX ? 16 : 1)
+// BATCH: 0, or rows of experts that a thread has in flight. They lie at scattered places, so many rows of tokens want as
+// many threads as the SM takes (MANY) rather than many requests in each.
+template <int BATCH, bool MANY, int RUN>
+__global__ void __launch_bounds__(kThreads, BATCH && MANY ? 16 : 1)
 tanh_norm_kernel(Args p) {
+  constexpr bool MIX = BATCH != 0;
   lg::pdl_trigger();
   const int v = (int)(blockIdx.x % p.cols) * kThreads + threadIdx.x, r0 = (int)(blockIdx.x / p.cols) * RUN;
   const bool in = v < p.nv;
@@ -65,7 +67,7 @@ tanh_norm_kernel(Args p) {
     if (p.post.w) { w1 = __ldg(p.post.w + v); b1 = __ldg(p.post.b + v); }
     if (p.next.w) { w2 = __ldg(p.next.w + v); b2 = __ldg(p.next.b + v); }
   };
-  if (!MIX && in) vectors();  // they do not depend on the kernels before this one
+  if (!(MIX && MANY) && in) vectors();  // they do not depend on the kernels before this one
   lg::pdl_wait();
   if (MIX && blockIdx.x == 0 && p.counts)
     for (int g = threadIdx.x; g < p.n_counts; g += kThreads) p.counts[g] = 0;
@@ -85,8 +87,8 @@ tanh_norm_kernel(Args p) {
     if (!MIX && p.post.w) y[i] = p.y[(size_t)r * p.nv + v];
   }
   if (MIX) {
-    // three experts of every row at a time: first where their rows are, then all of these at once
-    constexpr int kBatch = 3;
+    // a few experts of every row at a time: first where their rows are, then all of these at once
+    constexpr int kBatch = BATCH ? BATCH : 1;
 #pragma unroll
     for (int i = 0; i < RUN; ++i) {
       const int r = r0 + i;
@@ -115,7 +117,7 @@ tanh_norm_kernel(Args p) {
 #pragma unroll
         for (int j = 0; j < kBatch; ++j) add_scaled(y[i], w[i][j], e[i][j]);
     }
-    vectors();
+    if (MANY) vectors();
   }
 #pragma unroll
   for (int i = 0; i < RUN; ++i) {
@@ -152,14 +154,13 @@ extern "C" uint32_t logismos_launch_tanh_norm(void* y, int32_t zero_y, const lg_
     p.expert_rows = mix->rows; p.pair_row = (const int*)mix->pair_row; p.weights = (const float*)mix->weights; p.identity = (const float*)mix->identity;
     p.n_pairs = mix->n_pairs; p.top = mix->top; p.counts = (int*)mix->counts; p.n_counts = mix->n_counts;
   }
-  // several rows per thread once that still leaves a few CTAs per SM
-  const bool run = (int64_t)p.cols * rows >= 148 * 16;
+  const bool many = (int64_t)p.cols * rows >= 148 * 16;
   auto go = [&](auto kern, int per) -> uint32_t {
     const int64_t blocks = ((int64_t)rows + per - 1) / per * p.cols;
     if (blocks > INT32_MAX) return lg::kInvalidValue;
     lg::launch(kern, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
-  if (mix) return go(tanh_norm_kernel<true, 1>, 1);
-  return run ? go(tanh_norm_kernel<false, 4>, 4) : go(tanh_norm_kernel<false, 1>, 1);
+  if (mix) return many ? go(tanh_norm_kernel<3, true, 1>, 1) : go(tanh_norm_kernel<4, false, 1>, 1);
+  return many ? go(tanh_norm_kernel<0, true, 4>, 4) : go(tanh_norm_kernel<0, false, 1>, 1);
 }
