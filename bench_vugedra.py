@@ -269,16 +269,16 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         if few:
             add(ph, "router and choice of experts" if fused else "choice of experts", [lambda s: lib.logismos_launch_moe_route(Y(r), m, s)] * 4, m * (2.0 * H if fused else ld * 4.0) + 12.0 * m * pairs, like="post_norm")
             ex = 8 if m <= 8 else 16
-            add(ph, "experts, gate and up", [lambda s, w=w: lib.logismos_launch_linear_experts_small_bf16(P(h), P(w), P(mid), P(off), P(tok), groups, m, ex, 2 * F, H, H, F, 2, s) for w in wu], ub, ul, "gate/up")
-            add(ph, "experts, down", [lambda s, w=w: lib.logismos_launch_linear_experts_small_bf16(P(mid), P(w), P(out), P(off), P(None), groups, m, ex, H, F, F, H, 0, s) for w in wd], db, dl, "down")
+            add(ph, "experts, gate and up", [lambda s, w=w: lib.logismos_launch_linear_experts_small_bf16(P(h), P(w), P(mid), P(off), P(tok), groups, m, ex, 2 * F, H, H, F, 2, 0, 0, 0, s) for w in wu], ub, ul, "gate/up")
+            add(ph, "experts, down", [lambda s, w=w: lib.logismos_launch_linear_experts_small_bf16(P(mid), P(w), P(out), P(off), P(None), groups, m, ex, H, F, F, H, 0, 0, 0, 0, s) for w in wd], db, dl, "down")
         else:
             def choose(s):
                 counts.zero_()
                 return lib.logismos_launch_moe_route(Y(r), m, s)
             add(ph, "choice of experts (with clearing)", [choose] * 4, m * (ld * 4.0 + 12.0 * pairs), like="post_norm")
             add(ph, "rows by expert", [lambda s: lib.logismos_launch_moe_place(Y(r), P(h), P(gat), H, m, s)] * 4, 2.0 * H * n_rows, like="latent_gather")
-            add(ph, "experts, gate and up", [lambda s, w=w: lib.logismos_launch_linear_experts_tc_bf16(P(gat), m * pairs, P(h), m, P(w), P(mid), P(tiles), P(nt), mt, groups, 2 * F, H, H, F, 2, P(st), s) for w in wu], ub, ul, "gate/up")
-            add(ph, "experts, down", [lambda s, w=w: lib.logismos_launch_linear_experts_tc_bf16(P(mid), m * pairs, P(None), 0, P(w), P(out), P(tiles), P(nt), mt, groups, H, F, F, H, 0, P(st), s) for w in wd], db, dl, "down")
+            add(ph, "experts, gate and up", [lambda s, w=w: lib.logismos_launch_linear_experts_tc_bf16(P(gat), m * pairs, P(h), m, P(w), P(mid), P(tiles), P(nt), mt, groups, 2 * F, H, H, F, 2, 0, 0, 0, P(st), s) for w in wu], ub, ul, "gate/up")
+            add(ph, "experts, down", [lambda s, w=w: lib.logismos_launch_linear_experts_tc_bf16(P(mid), m * pairs, P(None), 0, P(w), P(out), P(tiles), P(nt), mt, groups, H, F, F, H, 0, 0, 0, 0, P(st), s) for w in wd], db, dl, "down")
         del wu, wd
         x, outs = rf(m, H), [bf(m * pairs, H) for _ in range(copies(2.0 * m * pairs * H))]
         mo = [MixtureOut(A(o), A(prow), A(wts), A(ident), pairs, TOP, 0, 0) for o in outs]

@@ -155,6 +155,7 @@ typedef struct lg_linear_groups {
   float tail_cap;
   void* tail_parts;
   const void* bias;             /* f32 [n_main], added to the main columns (NULL: none) */
+  int32_t silu_begin, silu_end; /* main columns that leave as z sigmoid(z); multiples of 32 (equal: none) */
 } lg_linear_groups_t;
 uint32_t logismos_launch_linear_groups_tc_bf16(const void* a_bf16, const void* w_bf16, void* out, int32_t m, int32_t n,
                                                int32_t k, int32_t lda, int32_t ldc, const lg_linear_groups_t* groups,
@@ -171,12 +172,13 @@ uint32_t logismos_launch_linear_groups_f32(const void* a_f32, const void* w_bf16
                                            void* stream);
 /* A stack of matrices, one per group of rows: rows offsets[g] .. offsets[g + 1] of the output are rows of the input
  * times w[g] (w bf16 [n_groups][n][k]). offsets i32 [n_groups + 1] on the device. row_idx (NULL: none) gives the input row
- * of every output row. max_group_rows bounds the rows of one group (host value). Epilogues LG_EPI_BF16 and LG_EPI_SWIGLU
- * (small), LG_EPI_F32 and LG_EPI_GLU_CLAMP (fp32). The first streams the weights of the groups that have rows. */
+ * of every output row. max_group_rows bounds the rows of one group (host value). Epilogues LG_EPI_BF16, LG_EPI_SWIGLU and
+ * LG_EPI_GLU_CLAMP (small), LG_EPI_F32 and LG_EPI_GLU_CLAMP (fp32), with the constants p0, p1, p2 of the last. The first
+ * streams the weights of the groups that have rows. */
 uint32_t logismos_launch_linear_experts_small_bf16(const void* a_bf16, const void* w_bf16, void* out, const void* offsets_i32,
                                                    const void* row_idx_i32, int32_t n_groups, int32_t max_group_rows,
                                                    int32_t expected_group_rows, int32_t n, int32_t k, int32_t lda, int32_t ldc,
-                                                   int32_t epilogue, void* stream);
+                                                   int32_t epilogue, float p0, float p1, float p2, void* stream);
 uint32_t logismos_launch_linear_experts_f32(const void* a_f32, const void* w_bf16, void* out_f32, const void* offsets_i32,
                                             const void* row_idx_i32, int32_t n_groups, int32_t max_group_rows, int32_t n,
                                             int32_t k, int32_t lda, int32_t ldc, int32_t epilogue, float p0, float p1, float p2,
@@ -188,8 +190,8 @@ uint32_t logismos_launch_linear_experts_f32(const void* a_f32, const void* w_bf1
 uint32_t logismos_launch_linear_experts_tc_bf16(const void* a_bf16, int32_t a_rows, const void* a_direct_bf16,
                                                 int32_t direct_rows, const void* w_bf16, void* out_bf16, const void* tiles_i32,
                                                 const void* n_tiles_i32, int32_t max_tiles, int32_t n_groups, int32_t n,
-                                                int32_t k, int32_t lda, int32_t ldc, int32_t epilogue, void* status_i32,
-                                                void* stream);
+                                                int32_t k, int32_t lda, int32_t ldc, int32_t epilogue, float p0, float p1,
+                                                float p2, void* status_i32, void* stream);
 /* The batched contract with fp32 activations and outputs, true fp32 products and sums over the bf16
  * weights (which fp32 represents exactly). Epilogues LG_EPI_F32, LG_EPI_RESID_F32, LG_EPI_GLU_CLAMP, LG_EPI_RELU2 (fp32
  * out); k % 16 == 0, lda % 4 == 0, strides of a and w multiples of 4. */
@@ -812,6 +814,9 @@ typedef struct lg_ssd {
   int32_t ld_y, heads, groups, np, vp;
   void* xbc;                    /* activation format [rows, ld_xbc]: the convolved channels x | B | C */
   int32_t ld_xbc;
+  /* given: f32 [heads], log2 of a fixed decay per head. Every step then has size one, S <- decay S + B x^T, y = S^T C (linear
+   * attention: x, B, C its values, keys and queries); only xbc, state and its indices, y and the sizes are used. */
+  const void* log2_decay;
 } lg_ssd_t;
 /* Convolution and silu of rows [row0, rows) from proj into xbc (seq_ids [rows]; cu, slots, fresh and phase indexed by
  * them). single: rows are one token per sequence. */
@@ -827,6 +832,11 @@ uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* args, int32_t n_seqs, 
 uint32_t logismos_launch_gated_group_norm(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32,
                                           void* out, int32_t ld_out, int32_t is_f32, int32_t rows, int32_t heads,
                                           int32_t v, int32_t vp, int32_t parts, float eps, void* stream);
+
+/* out = y / rms(y) * gain * sigmoid(z) over the heads * v true channels, laid out [heads][vp]. */
+uint32_t logismos_launch_norm_gate(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32,
+                                   void* out, int32_t ld_out, int32_t is_f32, int32_t rows, int32_t heads, int32_t v,
+                                   int32_t vp, float eps, void* stream);
 
 /* Attention whose scores are capped and biased by distance: score = cap tanh(q . k scale / cap) + bias(i - j), with
  * queries and keys of unit root mean square and an output gate. bias f32 [n_heads][far + 1] in units of log2, the
@@ -914,21 +924,32 @@ uint32_t logismos_launch_rotary_heads(void* q, int32_t ld, const void* positions
                                       int32_t head_dim, int32_t at, const void* table_f32, int32_t dims, int32_t is_f32,
                                       void* stream);
 
-/* Attention over a window: a query at position i sees the keys j <= i with i - j < size or j < keep_first (size 0: all).
- * sink: one is added to the softmax denominator. gate f32 [rows, ld_gate]: head h of a row is multiplied by the sigmoid of
- * its column h (NULL: none). Scores are scaled by scale (> 0). */
+/* Attention over a window: a query at position i sees the keys j <= i with i - j < size or j < keep_first (size 0: all);
+ * chunked: those in its own chunk of `size` positions, counted from 0. sink: one is added to the softmax denominator. gate
+ * f32 [rows, ld_gate]: head h of a row is multiplied by the sigmoid of its column h (NULL: none). Scores are scaled by scale
+ * (> 0).
+ * pool > 0: besides its window a query sees one key and value for each block of `pool` positions (b pool .. b pool + pool - 1)
+ * that lies wholly before it. They are rows of k_mean and v_mean [n_pool_blocks][ceil(16 / pool)], as wide as the cache's:
+ * block b is kept with the cache block that holds its last token, the blocks ending there one after the other
+ * (logismos_launch_pool_blocks). */
 typedef struct lg_window {
   float scale;
   int32_t size, keep_first, sink;
   const void* gate;
   int32_t ld_gate;
+  int32_t chunked, pool;        /* of these and keep_first at most one */
+  const void *k_mean, *v_mean;
+  int32_t out_f32;              /* the output is fp32 whatever the queries are */
 } lg_window_t;
-/* Decode launches split what a query sees, the kept blocks and the window's, as one context of this length. */
+/* Decode launches split what a query sees, leading and window blocks, as one context of this length; keys that the prompt
+ * launch gathers for a sequence of kv_len keys whose last new_len are its queries. */
+int32_t logismos_window_view_context(const lg_window_t* window, int32_t context_len);
+int32_t logismos_window_view_keys(const lg_window_t* window, int32_t kv_len, int32_t new_len);
+/* The same of a sliding window with kept keys. */
 int32_t logismos_window_context(int32_t context_len, int32_t size, int32_t keep_first);
-/* Keys that the prompt launch gathers for a sequence of kv_len keys whose last new_len are its queries. */
 int32_t logismos_window_keys(int32_t kv_len, int32_t new_len, int32_t size, int32_t keep_first);
-/* As logismos_launch_bias_attention_decode_bf16 (chunk_offsets over logismos_window_context of the context lengths),
- * logismos_launch_bias_attention_prefix_bf16 (total_keys and max_keys over logismos_window_keys) and
+/* As logismos_launch_bias_attention_decode_bf16 (chunk_offsets over logismos_window_view_context of the context lengths),
+ * logismos_launch_bias_attention_prefix_bf16 (total_keys and max_keys over logismos_window_view_keys) and
  * logismos_launch_bias_attention_f32. */
 uint32_t logismos_launch_window_attention_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool,
                                                       const void* block_tables, const void* context_lens,
@@ -958,11 +979,14 @@ uint32_t logismos_launch_window_attention_f32(const void* q_f32, int32_t ld_q, c
  * logits are cleared with zero_logits. One launch for few tokens: offsets i32 [groups + 1], row_token i32 [pairs] included.
  * Many tokens: route (counts i32 [n_experts], zero on entry) and then place, which also copies the tokens' rows of h (bf16
  * [tokens, ld]) of the chosen experts to gathered [., ld] and lists the row tiles (logismos_launch_linear_experts_tc_bf16;
- * the tiles of the n_always groups read h itself). At most 512 router outputs, top <= 32. */
+ * the tiles of the n_always groups read h itself). At most 512 router outputs, top <= 32.
+ * scoring LG_ROUTE_SIGMOID: s = sigmoid(logit). groups > 0: the outputs form that many equal groups of neighbours, a group
+ * scores the sum of its two largest s + correction, and only the outputs of the best keep_groups groups are chosen from. */
+enum { LG_ROUTE_SOFTMAX = 0, LG_ROUTE_SIGMOID = 1 };
 typedef struct lg_moe_route {
   void* logits;
   int32_t ld, zero_logits;
-  const void* correction;       /* f32 [n_experts + n_identity] */
+  const void* correction;       /* f32 [n_experts + n_identity], NULL: none */
   int32_t n_experts, n_identity, top, n_always;
   void *weights, *pair_row, *identity;
   void *offsets, *row_token;    /* few tokens, fp32 */
@@ -971,6 +995,7 @@ typedef struct lg_moe_route {
   const void *h, *w;            /* few tokens: the logits are w h (bf16 [outputs, width], [tokens, width], fp32 sums) instead */
   int32_t width;
   void* arrived;                /* i32, zero on entry and on return */
+  int32_t scoring, groups, keep_groups;
 } lg_moe_route_t;
 /* 1: so few tokens are best served by the one-launch form and products that stream the experts' weights. */
 int32_t logismos_moe_streams(int32_t tokens, int32_t top, int32_t n_experts, int32_t n_identity, int32_t n_always, int32_t width,
@@ -979,6 +1004,66 @@ int32_t logismos_moe_max_tiles(int32_t tokens, int32_t top, int32_t n_experts, i
 uint32_t logismos_launch_moe_route(const lg_moe_route_t* args, int32_t tokens, void* stream);
 uint32_t logismos_launch_moe_place(const lg_moe_route_t* args, const void* h_bf16, void* gathered_bf16, int32_t ld,
                                    int32_t tokens, void* stream);
+
+/* ---- per-head norms, pooled blocks, differences of two attentions, gated residuals -------------------------------- */
+
+/* Packed rows q [heads * maps * hd] | k [n_kv * maps * hd] | v [n_kv * maps * hd]: every one of the q and k pieces of hd
+ * channels (a multiple of 8, at most 256) is divided by its root mean square over dim of them, times gain f32 [hd], and
+ * rotated; keys and values go to their cache slots. maps 1: queries in place. maps 2: the pieces of q are ordered by key
+ * head, map, query head of the key head; they go to q_out [rows][heads * 2][2 hd], each to the half of its map and zeros to
+ * the other, so that one attention over keys [map 1 | map 2] gives both maps' scores.
+ * pool > 0: for the rows below pool_rows (one per sequence, in the order of the tables) whose token ends a block of `pool`
+ * positions, the means of the block's cached keys and values go to k_mean and v_mean (lg_window_t). */
+typedef struct lg_head_norm {
+  void* qkv;
+  int32_t ld, rows, heads, n_kv, maps, hd, dim;
+  const void *gain_q, *gain_k;
+  float eps;
+  const void* table;            /* rotation (NULL: none) */
+  int32_t rot_dims;
+  void* q_out;
+  int32_t ld_q;
+  void *k_pool, *v_pool;
+  const void *slots_i64, *positions_i32;
+  int64_t n_pool_slots;
+  int32_t pool, pool_rows;
+  void *k_mean, *v_mean;
+  const void *tables_i32, *seq_ids_i32;
+  int32_t max_blocks, n_pool_blocks;
+} lg_head_norm_t;
+uint32_t logismos_launch_head_norm_store(const lg_head_norm_t* args, int32_t is_f32, void* status_i32, void* stream);
+/* The means for the rows from pool_rows on, once all rows of the step are stored. */
+uint32_t logismos_launch_pool_blocks(const lg_head_norm_t* args, int32_t is_f32, void* status_i32, void* stream);
+
+/* Difference of two attentions over the same values: a f32 [rows, ld_a] holds heads * 2 outputs of vp channels ordered by key
+ * head, map, query head of the key head; out = (a1 - lambda a2) / rms over the v true channels * scale, [rows, ld_out] with
+ * head h at h * vp. */
+uint32_t logismos_launch_attention_difference(const void* a_f32, int32_t ld_a, void* out, int32_t ld_out, int32_t is_f32,
+                                              int32_t rows, int32_t heads, int32_t n_kv, int32_t v, int32_t vp,
+                                              float lambda, float scale, float eps, void* stream);
+
+/* Residual stream with RMS norms of one gain and gated sublayers, one launch between two sublayers:
+ *   y = branch[0] (one branch), half the sum of both, each divided by its root mean square, times its gain, or a mixture
+ *   x += y sigmoid(gate);   kept = x;   x += embed[ids] + step;   h = x / rms(x) * gain
+ * whatever is NULL is left out. branch f32 [rows, ld], cleared once read with zero_branches; gate in the activation format;
+ * embed bf16. n true columns, ld a multiple of 4, padding zero throughout. row_idx selects rows of x (no sublayer then). */
+typedef struct lg_gated_residual {
+  void* x;
+  void* branch[2];
+  int32_t zero_branches;
+  const void* branch_gain[2];   /* f32 [ld], of two branches */
+  const lg_mixture_out_t* mixture;
+  const void* gate;
+  int32_t ld_gate;
+  void* kept;
+  const void *embed, *ids, *step;
+  int32_t vocab;
+  void* h;
+  float gain, eps;
+  const void* row_idx;
+  int32_t n_src_rows, rows, n, ld, is_f32;
+} lg_gated_residual_t;
+uint32_t logismos_launch_gated_residual(const lg_gated_residual_t* args, void* status_i32, void* stream);
 
 #ifdef __cplusplus
 }

@@ -327,6 +327,8 @@ int32_t lg_latent_device_status(void* model);
  *   x = embed[id];  per layer x += mixer, x += feed-forward, normed as the stack's `norm` says:
  *   LG_NORM_LAYER_POST (Katadra)  x += norm(f(x)), layer norms (gain and offset); logits = head norm(x)
  *   LG_NORM_TANH_AROUND (Vugedra) x += norm_b(f(norm_a(x))), norms tanh(alpha x) w + b; logits = head norm(x)
+ *   LG_NORM_RMS_GATED (Zetalorn)  h = norm(x); x += f(h) sigmoid(W_rg h + b), norms x / rms(x) * g with one gain g; logits =
+ *     logit_scale head norm(x)
  * Mixers:
  *   LG_MIXER_SSD: [z | x | B | C | dt] = W_in h, convolution, scalar-decay recurrence, gate, norm in parts, W_o
  *     (lg_ssd_t, logismos_launch_gated_group_norm)
@@ -336,17 +338,27 @@ int32_t lg_latent_device_status(void* model);
  *   LG_MIXER_ATTENTION: q, k, v with biases, q and k normed over the whole projection and rotated; a window with kept first
  *     keys, one added to the softmax denominator, an output gate per head (lg_window_t); W_o
  *   LG_MIXER_GLA: gated linear attention, a decay per key channel (lg_time_mix_t, LG_DECAY_GATED); W_o
+ *   LG_MIXER_DIFF (in a gated RMS stack): differential attention over chunks. Every head has two maps of queries and keys, q
+ *     and k normed per head and map and rotated, over one set of values; out = (a1 - lambda a2) / rms * (1 - diff) with lambda =
+ *     exp(lq1 . lk1) - exp(lq2 . lk2) + diff; W_o
+ *   LG_MIXER_PAIR (in a gated RMS stack): half the sum of two branches, each with its W_o, then normed over the width with a
+ *     gain. Left: attention over a sliding window and, before it, pooled blocks (lg_window_t), q and k normed per head and
+ *     rotated. Right: linear attention with a fixed decay per head, q, k, v with silu; normed over all heads, times sigmoid(W_g h)
  *   LG_MIXER_LATENT: queries W_uq rms(W_dq h), per head dim unrotated and rot_dims rotated channels; W_dkv h is the latent
  *     (normed, cached) and one rotated key part for all heads; keys W_uk c, values W_uv c; causal, a gate per head; W_o
  * Feed-forwards:
  *   LG_FF_RELU2: W_down max(W_up h, 0)^2
  *   LG_FF_GATED: W_down (silu(W_gate h) * (W_up h))
  *   LG_FF_MIXTURE: `top` of experts + identity experts of the latter form by a softmax router with a correction for the
- *     choice alone (lg_moe_route_t); identity experts return h; a shared expert is added (shared_ff 0: none)
+ *     choice alone (lg_moe_route_t); identity experts return h; a shared expert is added (shared_ff 0: none). Also with sigmoid
+ *     scores, a choice among the best groups, and clamped gated units (LG_EPI_GLU_CLAMP)
+ * Layers may be repeated: a run of them is listed once per pass, those of later passes with weights_of, and the first of each
+ * pass names it: x += embed[id] (not in the first), x += loop_step[pass], before its norm.
  * ==================================================================================== */
-enum { LG_MIXER_SSD = 0, LG_MIXER_PARALLEL = 1, LG_MIXER_ATTENTION = 2, LG_MIXER_GLA = 3, LG_MIXER_LATENT = 4 };
+enum { LG_MIXER_SSD = 0, LG_MIXER_PARALLEL = 1, LG_MIXER_ATTENTION = 2, LG_MIXER_GLA = 3, LG_MIXER_LATENT = 4,
+       LG_MIXER_DIFF = 5, LG_MIXER_PAIR = 6 };
 enum { LG_FF_RELU2 = 0, LG_FF_GATED = 1, LG_FF_MIXTURE = 2 };
-enum { LG_NORM_LAYER_POST = 0, LG_NORM_TANH_AROUND = 1 };
+enum { LG_NORM_LAYER_POST = 0, LG_NORM_TANH_AROUND = 1, LG_NORM_RMS_GATED = 2 };
 typedef struct lg_mixer_layer_config {
   int32_t kind;
   int32_t weights_of;           /* layer whose tensors are used; its own index: its own */
@@ -366,7 +378,17 @@ typedef struct lg_mixer_layer_config {
   int32_t q_rank, kv_rank;      /* latent attention: kv_rank + rot_dims <= 1024 */
   int32_t rot_dims;             /* rotated channels per head, interleaved pairs */
   float tau;                    /* gated linear attention */
-  double rot_base, rot_factor, rot_original, rot_fast, rot_slow;   /* YaRN interpolation; rot_factor 0: none */
+  double rot_base, rot_factor, rot_original, rot_fast, rot_slow;   /* YaRN interpolation; rot_factor 0: none, rot_original 0: linear */
+  int32_t rot_halves;           /* pairs (i, i + rot_dims / 2) instead; differential and paired attention */
+  int32_t chunked, pool;        /* the window is a chunk; pooled blocks before it */
+  float diff;
+  int32_t lin_heads, lin_dim, lin_vdim;        /* linear attention of a pair: sizes <= 256 */
+  const double* decay;          /* [lin_heads], in (0, 1]; read while the model is made */
+  float glu_alpha, glu_limit, glu_shift;       /* of the experts; glu_limit 0: silu(gate) * up */
+  int32_t scoring, route_groups, keep_groups;  /* LG_ROUTE_*; route_groups 0: none */
+  int32_t no_correction;
+  int32_t file_layer;           /* 1 + the layer's number in tensor names, 0: its own index */
+  int32_t pass;                 /* 1 + the pass that begins with this layer, 0: none */
 } lg_mixer_layer_config_t;
 typedef struct lg_mixer_config {
   int32_t vocab, width, n_layers;
@@ -379,6 +401,8 @@ typedef struct lg_mixer_config {
   int32_t keep_layers;          /* != 0: the stream after every layer is kept (lg_mixer_snapshot) */
   const lg_mixer_layer_config_t* layers;
   int32_t norm;
+  int32_t passes;               /* over repeated layers, 0: none are */
+  float logit_scale;            /* gated RMS stack */
 } lg_mixer_config_t;
 /* bf16 values on the host, [out, in]; entries of other kinds of mixer, of a missing feed-forward and of a layer
  * with weights_of are NULL. mu [5] in the order r, k, v, g, w. experts [3 * experts]: gate, up, down of each. */
@@ -393,11 +417,15 @@ typedef struct lg_mixer_layer_weights {
   const void *dq, *dq_norm, *uq, *dkv, *dkv_norm, *uk, *uv;
   const void *gate, *router, *correction, *shared_gate, *shared_up, *shared_down;
   const void* const* experts;
+  const void *rg1, *rg1_b, *rg2, *rg2_b;        /* gated residual; norm1 and norm2 are then single values */
+  const void *lq1, *lk1, *lq2, *lk2;            /* differential attention: also q, k, v, o, q_norm and k_norm [dim] */
+  const void *left_q_norm, *left_k_norm, *left_out, *right_q, *right_out;   /* a pair: also left_* q, k, v, o, right_* k, v, g, norm, o */
 } lg_mixer_layer_weights_t;
 typedef struct lg_mixer_weights {
   const void *embed, *final_norm, *final_norm_b, *head;
   const lg_mixer_layer_weights_t* layers;
   const void* final_norm_alpha; /* tanh norms */
+  const void* loop_step;        /* [passes, width] */
 } lg_mixer_weights_t;
 
 uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_mixer_weights_t* w, void** model);
@@ -406,7 +434,9 @@ uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_
  * .b (and .alpha); under l<i>.mix.: {in,conv,conv.b,dt_bias,A_log,D,norm,o}, left.{q,k,v,rel,g,o} and right.{mu.r,mu.k,mu.v,
  * mu.g,mu.w,r,k,v,g,w1,w2,w0,u,norm,o}, {q,k,v,g,o} with {q,k,v}.b and {q,k}.norm, {q,k,v,g,o,norm,a1,a2,a2.b}, or {dq,
  * dq.norm,uq,dkv,dkv.norm,uk,uv,g,o}; under l<i>.mlp.: {up,down}, {gate,up,down}, or {router,correction} with {e<j>,shared}.
- * {gate,up,down}. bias_rows and tm_rank are taken from the tensors. */
+ * {gate,up,down}. bias_rows and tm_rank are taken from the tensors. A gated RMS stack: norms of one value without .b, l<i>.rg1,
+ * l<i>.rg2 with .b, l<i>.mix.{q,k,v,q.norm,k.norm,lq1,lk1,lq2,lk2,o}, or left.{q,k,v,q.norm,k.norm,o,out} and right.{q,k,v,g,
+ * norm,o,out}, no mlp.correction, and loop.step when layers are repeated. */
 uint32_t lg_mixer_load(int32_t device, const char* path, const lg_mixer_config_t* cfg, void** model);
 void lg_mixer_destroy(void* model);
 /* Step, logits and diagnostics as for lg_latent_*. Recurrent states are updated in place: a step that failed part-way

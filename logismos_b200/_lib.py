@@ -166,6 +166,11 @@ def _declare(l, partial=False):
         "logismos_launch_ssd_conv": [vp, vp, i32, i32, i32, i32, vp],
         "logismos_launch_ssd_chunked_bf16": [vp, i32, vp],
         "logismos_launch_gated_group_norm": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp],
+        "logismos_launch_norm_gate": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp],
+        "logismos_launch_head_norm_store": [vp, i32, vp, vp],
+        "logismos_launch_pool_blocks": [vp, i32, vp, vp],
+        "logismos_launch_attention_difference": [vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp],
+        "logismos_launch_gated_residual": [vp, vp, vp],
         "logismos_launch_unit_qk_store": [vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, f32, f32, i64, i32, vp, vp],
         "logismos_launch_bias_attention_decode_bf16": [vp, i32, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
         "logismos_launch_bias_attention_prefix_bf16": [vp, i32, vp, vp, vp, vp, vp, i32, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32,
@@ -181,9 +186,9 @@ def _declare(l, partial=False):
         "logismos_launch_window_attention_f32": [vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
         "logismos_launch_moe_route": [vp, i32, vp],
         "logismos_launch_moe_place": [vp, vp, vp, i32, i32, vp],
-        "logismos_launch_linear_experts_small_bf16": [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp],
+        "logismos_launch_linear_experts_small_bf16": [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp],
         "logismos_launch_linear_experts_f32": [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp],
-        "logismos_launch_linear_experts_tc_bf16": [vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp],
+        "logismos_launch_linear_experts_tc_bf16": [vp, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp, vp],
         "lg_mixer_create": [i32, vp, vp, C.POINTER(vp)],
         "lg_mixer_load": [i32, C.c_char_p, vp, C.POINTER(vp)],
         "lg_mixer_step": [vp, vp, vp, vp, i32, vp, vp, vp, i32, vp],
@@ -238,6 +243,8 @@ def _declare(l, partial=False):
         "lg_mixer_destroy": ([vp], None),
         "lg_mixer_logits_device": ([vp], vp),
         "logismos_window_context": ([i32, i32, i32], i32),
+        "logismos_window_view_context": ([vp, i32], i32),
+        "logismos_window_view_keys": ([vp, i32, i32], i32),
         "logismos_window_keys": ([i32, i32, i32, i32], i32),
         "logismos_moe_streams": ([i32] * 7, i32),
         "logismos_moe_max_tiles": ([i32, i32, i32, i32], i32),

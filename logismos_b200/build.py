@@ -28,7 +28,7 @@ CU_SOURCES = ["cudacore.cu", "legacy_fp16.cu", "elementwise.cu", "gemv_int4.cu",
               "attention.cu", "attention_tcgen05.cu", "gdn.cu", "gdn_chunk.cu", "sampling.cu", "kvquant.cu", "stella_model.cu", "decoder_model.cu", "hybrid_model.cu", "tp_comm.cu",
               "linear_small.cu", "depth_conv.cu", "latent_attention.cu", "latent_model.cu",
               "post_norm.cu", "tanh_norm.cu", "time_mix.cu", "ssd.cu", "bias_attention.cu", "rotary.cu", "moe.cu", "mixer_parallel.cu",
-              "mixer_gated.cu", "mixer_model.cu"]
+              "gated_residual.cu", "mixer_gated.cu", "mixer_paired.cu", "mixer_model.cu"]
 CPP_SOURCES = ["sched.cpp", "loader.cpp", "checkpoints.cpp"]
 
 # what one model family needs: the sources of a library that serves it alone
@@ -37,7 +37,7 @@ GROUPS = {
                "latent_attention.cu", "latent_model.cu", "sampling.cu", "sched.cpp", "loader.cpp"],
     "mixer": ["cudacore.cu", "elementwise.cu", "gemm_tcgen05.cu", "attention.cu", "attention_tcgen05.cu", "linear_small.cu", "post_norm.cu",
               "tanh_norm.cu", "time_mix.cu", "ssd.cu", "bias_attention.cu", "latent_attention.cu", "rotary.cu", "moe.cu", "mixer_parallel.cu",
-              "mixer_gated.cu", "mixer_model.cu", "sampling.cu", "sched.cpp", "loader.cpp"],
+              "gated_residual.cu", "mixer_gated.cu", "mixer_paired.cu", "mixer_model.cu", "sampling.cu", "sched.cpp", "loader.cpp"],
 }
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-std=c++17", "-lineinfo",

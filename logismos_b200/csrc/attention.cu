@@ -284,8 +284,22 @@ LG_DEVINL void stage_block(uint32_t sbase, const __nv_bfloat16* kpool, const __n
   }
 }
 
+// the same of sixteen pooled rows: lane r < 16 holds the number of row r
+template <int HD>
+LG_DEVINL void stage_means(uint32_t sbase, const __nv_bfloat16* kmean, const __nv_bfloat16* vmean, uint32_t number, int row_elems, int kvh, int lane) {
+  constexpr int CH = HD / 8;
+#pragma unroll
+  for (int i = 0; i < (kBlock * CH) / 32; ++i) {
+    const int u = lane + 32 * i;
+    const int row = u / CH, chunk = u % CH;
+    const int64_t at = (int64_t)__shfl_sync(0xffffffffu, number, row) * row_elems + kvh * HD + chunk * 8;
+    cp_async16(tile_addr<HD>(sbase, row, chunk), kmean + at);
+    cp_async16(tile_addr<HD>(sbase + kBlock * HD * 2, row, chunk), vmean + at);
+  }
+}
+
 // What a decode kernel does beyond the plain softmax; both forms take 16 query heads of a key head per CTA. kWindowed: the
-// blocks that a query sees, kept ones and the window's, are numbered through ("virtual" blocks) and split in chunks.
+// blocks that a query sees, leading ones and the window's, are numbered through ("virtual" blocks) and split in chunks.
 enum { kPlain = 0, kBiased = 1, kWindowed = 2 };
 template <int MODE> struct ExtOf { using type = ScoreExt; };
 template <> struct ExtOf<kWindowed> { using type = WindowExt; };
@@ -324,8 +338,14 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
   const int chunk_in_seq = chunk_id - chunk_offsets[seq];
   const int n_chunks = chunk_offsets[seq + 1] - chunk_offsets[seq];
   const int ctx = ctx_lens[seq];
-  int gap = 0, kept_blocks = 0;  // a virtual block from kept_blocks on stands for the block `gap` further
-  if constexpr (MODE == kWindowed) { gap = window_gap_blocks(ctx, ext.size, ext.keep); kept_blocks = (ext.keep + kBlock - 1) / kBlock; }
+  int gap = 0, kept_blocks = 0;  // a virtual block from kept_blocks on stands for the block `gap` further; those before it may be of pooled keys
+  int n_means = 0, win_first = 0;
+  if constexpr (MODE == kWindowed) {
+    gap = ext.gap_blocks(ctx);
+    kept_blocks = ext.lead_blocks(ctx);
+    n_means = ext.pooled(ctx - 1);
+    win_first = ext.first(ctx - 1);
+  }
   const int tok_begin = chunk_in_seq * chunk_tokens;
   const int tok_end = min(ctx - gap * kBlock, tok_begin + chunk_tokens);
   const int* table = tables + (int64_t)seq * max_blocks;
@@ -387,6 +407,20 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
   auto place = [&](int vb) { return MODE == kWindowed && vb >= kept_blocks ? vb + gap : vb; };
   auto issue = [&](int i) {  // i-th block of this warp; always commits a group (possibly empty)
     if (i < my_count) {
+      if (MODE == kWindowed && my_first + i * kDecWarps < kept_blocks && n_means > 0) {
+        if constexpr (MODE == kWindowed) {  // sixteen pooled rows, each with its own place; past the last one it is repeated
+          const int b = min((my_first + i * kDecWarps) * kBlock + (lane & 15), n_means - 1), page = ext.mean_block(b);
+          int pb = page < max_blocks ? table[page] : -1;
+          if (pb < 0 || pb >= n_pool_blocks) {
+            if (status) atomicExch(status, 1);
+            pb = 0;
+          }
+          stage_means<HD>(wbase + (i % kDecStages) * kDecStageBytes, (const __nv_bfloat16*)ext.kmean, (const __nv_bfloat16*)ext.vmean,
+                          (uint32_t)(pb * ext.mean_rows() + ext.mean_row(b)), row_elems, kvh, lane);
+        }
+        cp_async_commit();
+        return;
+      }
       const int bidx = place(my_first + i * kDecWarps);
       const int pb = bidx < max_blocks ? table[bidx] : -1;
       if (pb >= 0 && pb < n_pool_blocks) {
@@ -405,20 +439,23 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
     cp_async_wait<kDecStages - 1>();
     __syncwarp();
     const int blk = my_first + i * kDecWarps, real = place(blk);
-    const int pb = real < max_blocks ? table[real] : -1;
+    const bool means = MODE == kWindowed && blk < kept_blocks && n_means > 0;
+    const int pb = means ? 0 : real < max_blocks ? table[real] : -1;
     const bool valid_block = pb >= 0 && pb < n_pool_blocks;
     const uint32_t sb = wbase + (i % kDecStages) * kDecStageBytes;
     float s[2][4];
     if (valid_block) {
       qk_tile<2, HD>(qf, sb, 0, lane, s);
       if constexpr (MODE == kWindowed) {
-        const int first = real * kBlock;
-        if (ctx - 1 - first >= ext.size && first + kBlock > ext.keep) {  // some key may lie outside
+        const int first = means ? blk * kBlock : real * kBlock;
+        if (means ? first + kBlock > n_means : first < win_first && first + kBlock > ext.keep) {  // some key may lie outside
 #pragma unroll
           for (int t = 0; t < 2; ++t)
 #pragma unroll
-            for (int e = 0; e < 2; ++e)
-              if (!ext.sees(ctx - 1, first + 8 * t + 2 * c + e)) s[t][e] = s[t][2 + e] = -INFINITY;
+            for (int e = 0; e < 2; ++e) {
+              const int j = first + 8 * t + 2 * c + e;
+              if (means ? j >= n_means : j < win_first && j >= ext.keep) s[t][e] = s[t][2 + e] = -INFINITY;
+            }
         }
       }
       if constexpr (MODE == kBiased) {
@@ -511,7 +548,11 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
         if constexpr (MODE == kBiased)
           out[(int64_t)seq * ext.ld_out + head * D + d] =
               __float2bfloat16_rn(ext.gated(acc / L, __bfloat162float(ext.gate[(int64_t)seq * ext.ld_gate + head * D + d])));
-        if constexpr (MODE == kWindowed) out[(int64_t)seq * ext.ld_out + head * D + d] = __float2bfloat16_rn(acc / L * gate);
+        if constexpr (MODE == kWindowed) {
+          const int64_t at = (int64_t)seq * ext.ld_out + head * D + d;
+          if (ext.raw) reinterpret_cast<float*>(out)[at] = acc / L * gate;
+          else out[at] = __float2bfloat16_rn(acc / L * gate);
+        }
       } else if (n_chunks == 1) out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
       else part_o[((int64_t)chunk_id * n_heads + head) * D + d] = acc;
     }
@@ -544,9 +585,11 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o, cons
   }
   if constexpr (MODE == kBiased)
     out[(int64_t)seq * ext.ld_out + head * D + d] = __float2bfloat16_rn(ext.gated(acc / L, __bfloat162float(ext.gate[(int64_t)seq * ext.ld_gate + head * D + d])));
-  else if constexpr (MODE == kWindowed)
-    out[(int64_t)seq * ext.ld_out + head * D + d] = __float2bfloat16_rn(acc / L * ext.head_gate(seq, head));
-  else
+  else if constexpr (MODE == kWindowed) {
+    const int64_t at = (int64_t)seq * ext.ld_out + head * D + d;
+    if (ext.raw) reinterpret_cast<float*>(out)[at] = acc / L * ext.head_gate(seq, head);
+    else out[at] = __float2bfloat16_rn(acc / L * ext.head_gate(seq, head));
+  } else
     out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
 }
 
@@ -713,11 +756,19 @@ uint32_t logismos_launch_bias_attention_decode_bf16(const void* q, int32_t ld_q,
                                     max_blocks, n_pool_blocks, n_heads, n_kv_heads, head_dim, 1.0f, score_ext(score, ld_q, ld_out), status, stream);
 }
 
+int32_t logismos_window_view_context(const lg_window_t* window, int32_t context_len) { return context_len - kBlock * window_ext(window, 0, 0).gap_blocks(context_len); }
+int32_t logismos_window_view_keys(const lg_window_t* window, int32_t kv_len, int32_t new_len) { return kv_len - window_ext(window, 0, 0).gap_keys(kv_len, new_len); }
 int32_t logismos_window_context(int32_t context_len, int32_t size, int32_t keep_first) {
-  return context_len - kBlock * window_gap_blocks(context_len, size ? size : 0x7fffffff, keep_first);
+  lg_window_t w{};
+  w.size = size;
+  w.keep_first = keep_first;
+  return logismos_window_view_context(&w, context_len);
 }
 int32_t logismos_window_keys(int32_t kv_len, int32_t new_len, int32_t size, int32_t keep_first) {
-  return kv_len - window_gap_keys(kv_len, new_len, size ? size : 0x7fffffff, keep_first);
+  lg_window_t w{};
+  w.size = size;
+  w.keep_first = keep_first;
+  return logismos_window_view_keys(&w, kv_len, new_len);
 }
 
 uint32_t logismos_launch_window_attention_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables,

@@ -164,12 +164,13 @@ transpose_v_kernel(const __nv_bfloat16* __restrict__ qkv, const int* __restrict_
 // k_pool / v_pool [n_pool_blocks, 16, n_kv * HD] (the row layout of FlatKvCache,
 // crates/cache/src/flat.rs:36-69; the read is KvCache::get, :254-304). A block id outside the pool
 // yields zero rows and raises the status word. Grid (key blocks of 64, kv heads, sequences). With a window the keys between
-// the kept ones and the first query's window are left out (window_gap_keys): rows from tile kept_tiles on stand `gap` keys
-// further in the sequence.
+// the leading ones and the first query's window are left out (gap_keys): rows after the leading tiles stand `gap` keys
+// further in the sequence. Leading rows may be pooled blocks, the rest of their last tile is zero.
 struct GatherWindow {
   const int* cu;     // query offsets (NULL: all keys are gathered)
-  int size, keep;
-  LG_DEVINL int gap(int s, int kv_len) const { return cu ? window_gap_keys(kv_len, cu[s + 1] - cu[s], size, keep) : 0; }
+  WindowExt w;
+  LG_DEVINL int gap(int s, int kv_len) const { return cu ? w.gap_keys(kv_len, cu[s + 1] - cu[s]) : 0; }
+  LG_DEVINL int lead(int kv_len) const { return cu ? w.lead_keys(kv_len) : 0; }
 };
 
 template <int HD>
@@ -196,7 +197,8 @@ gather_paged_kv_kernel(const __nv_bfloat16* __restrict__ kpool, const __nv_bfloa
   }
   __syncthreads();
   const int p0 = p0_s;
-  const int gap = win.gap(s, kv_lens[s]), kept_rows = (win.keep + 127) / 128 * 128;
+  const int gap = win.gap(s, kv_lens[s]), kept_rows = win.lead(kv_lens[s]), n_means = win.cu ? win.w.pooled(kv_lens[s] - 1) : 0;
+  const bool pools = win.cu && win.w.pool;
   const int len = max(kv_lens[s] - gap, 0), plen = round8(len);
   const int row_w = n_kv * HD;
   if (p0 + plen > tp) {  // the caller's total does not cover these lengths: nothing is written
@@ -215,15 +217,16 @@ gather_paged_kv_kernel(const __nv_bfloat16* __restrict__ kpool, const __nv_bfloa
   for (int u = tid; u < 64 * kChunks; u += 256) {
     const int r = u / kChunks, ch = u % kChunks, t = tb * 64 + r;
     uint4 kq = make_uint4(0u, 0u, 0u, 0u), vq = kq;
-    if (t < len) {
-      const int at = t < kept_rows ? t : t + gap, bi = at >> 4;
+    const bool mean = pools && t < kept_rows;
+    if (t < len && (!mean || t < n_means)) {
+      const int at = t < kept_rows ? t : t + gap, bi = mean ? win.w.mean_block(t) : at >> 4;
       const int blk = bi < max_blocks ? __ldg(tables + (size_t)s * max_blocks + bi) : -1;
       if (blk < 0 || blk >= n_pool_blocks) {
         if (ch == 0 && status) atomicExch(status, 1);
       } else {
-        const size_t src = ((size_t)blk * 16 + (at & 15)) * row_w + kvh * HD + ch * 8;
-        kq = __ldg(reinterpret_cast<const uint4*>(kpool + src));
-        vq = __ldg(reinterpret_cast<const uint4*>(vpool + src));
+        const size_t src = (mean ? (size_t)blk * win.w.mean_rows() + win.w.mean_row(t) : (size_t)blk * 16 + (at & 15)) * row_w + kvh * HD + ch * 8;
+        kq = __ldg(reinterpret_cast<const uint4*>((mean ? (const __nv_bfloat16*)win.w.kmean : kpool) + src));
+        vq = __ldg(reinterpret_cast<const uint4*>((mean ? (const __nv_bfloat16*)win.w.vmean : vpool) + src));
       }
     }
     if (t < plen) *reinterpret_cast<uint4*>(kbuf + (size_t)(p0 + t) * row_w + kvh * HD + ch * 8) = kq;
@@ -334,8 +337,8 @@ gather_paged_kv_turbo3_kernel(const uint8_t* __restrict__ kpool, const uint8_t* 
 // where cap and biases bound every score so tightly that exp2 of it neither over- nor underflows, and no maximum is
 // kept (one pass over the scores, the output never rescaled); and that with the cap as a polynomial, where the products
 // are known to be small (unit queries and keys): the multiplier units then leave the exponential unit to the softmax.
-// kWindowed: a window with kept first keys and a softmax denominator with one added, where asked for, and a gate per head;
-// only the key tiles that some query of the CTA sees are visited.
+// kWindowed: a window, sliding or a chunk, with kept first keys or pooled blocks ahead of it, a softmax denominator with one
+// added, where asked for, and a gate per head; only the key tiles that some query of the CTA sees are visited.
 enum { kPlain = 0, kBiased = 1, kBounded = 2, kPoly = 3, kWindowed = 4 };
 template <int SCORE> struct ExtOf { using type = ScoreExt; };
 template <> struct ExtOf<kWindowed> { using type = WindowExt; };
@@ -402,11 +405,11 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   // windows: the tiles [0, kept) and [kept + skip, ..) are visited, gathered rows of the latter standing `gap` keys further
   int kept = 0, skip = 0, gap = 0;
   if constexpr (SCORE == kWindowed) {
-    gap = kv_lens ? window_gap_keys(kv_total, len, ext.size, ext.keep) : 0;
+    gap = kv_lens ? ext.gap_keys(kv_total, len) : 0;
     nb = (kv_len - gap + 127) >> 7;
-    kept = min((ext.keep + 127) >> 7, nb);
-    const int first = q_off + q0 - ext.size + 1 - gap;  // gathered row of the first key in the window of the tile's first query
-    if (ext.size <= q_off + q0 && (first >> 7) > kept) skip = (first >> 7) - kept;
+    kept = min(((ext.pool ? ext.pooled(kv_len - 1) : ext.keep) + 127) >> 7, nb);
+    const int first = ext.first(q_off + q0) - gap;  // gathered row of the first key in the window of the tile's first query
+    if ((first >> 7) > kept) skip = (first >> 7) - kept;
     nb -= skip;
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -505,8 +508,12 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       bias = ext.bias + (size_t)h * (ext.far + 1);
       far_bias = __ldg(bias + ext.far);
     }
-    if constexpr (SCORE == kWindowed)
+    int seen_from = 0, seen_means = 0;  // first key of this row's window, pooled blocks before it
+    if constexpr (SCORE == kWindowed) {
       if (ext.sink) { m = 0.0f; l = 1.0f; }  // a further score of 0, without a value
+      seen_from = ext.first(q_off + q0 + row);
+      seen_means = ext.pooled(q_off + q0 + row);
+    }
     for (int j = 0; j < nb; ++j) {
       bool near = false;
       if constexpr (BIASED) {
@@ -532,9 +539,13 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       int lo = 0, keep = 0;  // and of these [lo, lim) and [0, keep)
       if constexpr (SCORE == kWindowed) {
         const int jt = j >= kept ? j + skip : j, base = jt * 128 + (jt >= kept ? gap : 0), at = q_off + q0 + row;  // key 0's position
-        lim = min(kv_len, at + 1) - base;
-        lo = ext.size <= at ? at - ext.size + 1 - base : 0;
-        keep = ext.keep - base;
+        if (ext.pool && j < kept) {
+          lim = seen_means - jt * 128;
+        } else {
+          lim = min(kv_len, at + 1) - base;
+          lo = seen_from - base;
+          keep = ext.keep - base;
+        }
         full = lim >= 128 && (lo <= 0 || keep >= 128);
       }
       auto seen = [&](int key) { return key < lim && (SCORE != kWindowed || key >= lo || key < keep); };
@@ -668,6 +679,15 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 r[8 * i + 2 * k] = __float_as_uint(ext.gated(__uint_as_float(r[8 * i + 2 * k]), gf.x));
                 r[8 * i + 2 * k + 1] = __float_as_uint(ext.gated(__uint_as_float(r[8 * i + 2 * k + 1]), gf.y));
               }
+            }
+          }
+          if constexpr (SCORE == kWindowed) {
+            if (ext.raw) {
+              float4* to = reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + (size_t)(t0 + q0 + row) * (size_t)out_stride + h * HD + c * 32);
+#pragma unroll
+              for (int i = 0; i < 8; ++i)
+                to[i] = make_float4(__uint_as_float(r[4 * i]) * inv, __uint_as_float(r[4 * i + 1]) * inv, __uint_as_float(r[4 * i + 2]) * inv, __uint_as_float(r[4 * i + 3]) * inv);
+              continue;
             }
           }
 #pragma unroll
@@ -822,7 +842,7 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
       lg::launch(kern, dim3((unsigned)blocks), dim3(256), 0, s, kp, vp, (const int*)block_tables, max_blocks, n_pool_blocks, (const int*)kv_lens, kbuf, vt, pstart,
                                             n_seqs, tp, tx, n_kv_heads, more..., (int*)status);
     };
-    const GatherWindow gw = win ? GatherWindow{(const int*)cu_seqlens_q, win->size, win->keep} : GatherWindow{};
+    const GatherWindow gw = win ? GatherWindow{(const int*)cu_seqlens_q, *win} : GatherWindow{};
     if (turbo3) {
       if (D == 128) go(gather_paged_kv_turbo3_kernel<128>, (const uint8_t*)k_pool, (const uint8_t*)v_pool);
       else go(gather_paged_kv_turbo3_kernel<256>, (const uint8_t*)k_pool, (const uint8_t*)v_pool);
@@ -945,7 +965,11 @@ uint32_t logismos_launch_varlen_attention_kv_tc_bf16(const void* q, int32_t q_ro
     return lg::launch_status();
   };
   if (gate) {
-    const WindowExt all{0x7fffffff, 0, 0, (const float*)gate, ld_gate, q_row_stride, out_row_stride};
+    WindowExt all{0x7fffffff};
+    all.gate = (const float*)gate;
+    all.ld_gate = ld_gate;
+    all.ld_q = q_row_stride;
+    all.ld_out = out_row_stride;
     if (D == 64) return launch(attn_tcgen05_kernel<true, 64, kWindowed>, Attn<64>::kSmem, all);
     if (D == 128) return launch(attn_tcgen05_kernel<true, 128, kWindowed>, Attn<128>::kSmem, all);
     return launch(attn_tcgen05_kernel<true, 256, kWindowed>, Attn<256>::kSmem, all);

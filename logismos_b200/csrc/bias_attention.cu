@@ -90,7 +90,7 @@ attention_f32_kernel(const float* __restrict__ q, const float* __restrict__ kpoo
                      int n_kv, int hd, float scale, float cap, const float* __restrict__ gate, ScoreExt ext, WindowExt win, int* __restrict__ status) {
   lg::pdl_prologue();
   __shared__ float sq[256], ss[kTile], red[32];
-  __shared__ int blk_s[kTile / kBlockTokens];
+  __shared__ int64_t row_s[kTile];  // cache row of every key of the tile, -1: not seen; pooled rows lie in pools of their own
   const int r = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int kvh = h / (gridDim.y / n_kv), n_keys = pos[r] + 1;
   const int* table = tables + (size_t)seq_ids[r] * max_blocks;
@@ -99,34 +99,41 @@ attention_f32_kernel(const float* __restrict__ q, const float* __restrict__ kpoo
   for (int i = tid; i < hd; i += kAttnThreads) sq[i] = q[(size_t)r * (WINDOW ? win.ld_q : ext.ld_q) + h * hd + i];
   const bool sink = WINDOW && win.sink;  // a further score of 0
   float m = sink ? 0.0f : -1e30f, l = sink ? 1.0f : 0.0f, acc[2] = {0.f, 0.f};
-  for (int k0 = 0; k0 < n_keys; k0 += kTile) {
-    if (WINDOW && k0 >= win.keep && n_keys - 1 - (k0 + kTile - 1) >= win.size) continue;  // a tile that is not seen
-    const int n = min(kTile, n_keys - k0);
+  const int n_means = WINDOW ? win.pooled(n_keys - 1) : 0, mean_tiles = (n_means + kTile - 1) / kTile * kTile;
+  for (int at = 0; at < mean_tiles + n_keys; at += kTile) {
+    const bool means = WINDOW && at < mean_tiles;
+    const int k0 = means ? at : at - mean_tiles, n = min(kTile, (means ? n_means : n_keys) - k0);
+    if (WINDOW && !means && k0 >= win.keep && k0 + kTile - 1 < win.first(n_keys - 1)) continue;  // a tile that is not seen
     __syncthreads();
-    if (tid < kTile / kBlockTokens) {
-      const int bi = k0 / kBlockTokens + tid;
-      int b = tid * kBlockTokens < n && bi < max_blocks ? __ldg(table + bi) : -1;
-      if (tid * kBlockTokens < n && (b < 0 || b >= n_pool_blocks)) {
-        if (status) atomicExch(status, 1);
-        b = -1;
+    if (tid < kTile) {
+      const int k = k0 + tid, bi = means ? win.mean_block(k) : k / kBlockTokens;
+      int64_t row = -1;
+      if (tid < n && (!WINDOW || means || win.sees(n_keys - 1, k))) {
+        const int b = bi < max_blocks ? __ldg(table + bi) : -1;
+        if (b < 0 || b >= n_pool_blocks) {
+          if (status) atomicExch(status, 1);
+        } else {
+          row = means ? (int64_t)b * win.mean_rows() + win.mean_row(k) : (int64_t)b * kBlockTokens + k % kBlockTokens;
+        }
       }
-      blk_s[tid] = b;
+      row_s[tid] = row;
     }
     __syncthreads();
+    const float *keys = means ? (const float*)win.kmean : kpool, *values = means ? (const float*)win.vmean : vpool;
     for (int k = warp; k < kTile; k += kAttnThreads / 32) {
-      const int b = blk_s[k / kBlockTokens];
+      const int64_t row = row_s[k];
       float s = 0.0f;
-      if (k < n && b >= 0) {
-        const float* c = kpool + ((size_t)b * kBlockTokens + k % kBlockTokens) * row_w + kvh * hd;
+      if (row >= 0) {
+        const float* c = keys + row * row_w + kvh * hd;
         for (int i = lane; i < hd; i += 32) s = fmaf(sq[i], c[i], s);
       }
       s = warp_sum(s) * scale;
       if (WINDOW) {
-        if (lane == 0) ss[k] = k < n && b >= 0 && win.sees(n_keys - 1, k0 + k) ? s * 1.4426950408889634f : -INFINITY;
+        if (lane == 0) ss[k] = row >= 0 ? s * 1.4426950408889634f : -INFINITY;
         continue;
       }
       if (cap > 0.0f) s = cap * tanhf(s / cap);
-      if (lane == 0) ss[k] = k < n && b >= 0 ? s * 1.4426950408889634f + bias[min(n_keys - 1 - (k0 + k), ext.far)] : -1e30f;
+      if (lane == 0) ss[k] = row >= 0 ? s * 1.4426950408889634f + bias[min(n_keys - 1 - (k0 + k), ext.far)] : -1e30f;
     }
     __syncthreads();
     const float mine = tid < kTile ? ss[tid] : -1e30f;
@@ -139,9 +146,8 @@ attention_f32_kernel(const float* __restrict__ q, const float* __restrict__ kpoo
     acc[0] *= alpha;
     acc[1] *= alpha;
     for (int k = 0; k < n; ++k) {
-      const int b = blk_s[k / kBlockTokens];
-      if (b < 0) continue;
-      const float* c = vpool + ((size_t)b * kBlockTokens + k % kBlockTokens) * row_w + kvh * hd;
+      if (row_s[k] < 0) continue;
+      const float* c = values + row_s[k] * row_w + kvh * hd;
       if (tid < hd) acc[0] = fmaf(ss[k], c[tid], acc[0]);
       if (tid + kAttnThreads < hd) acc[1] = fmaf(ss[k], c[tid + kAttnThreads], acc[1]);
     }

@@ -114,7 +114,8 @@ LG_DEVINL float block_max(float v, float* red) {
 // host-side shape rules of lg_linear_groups_t (logismos_kernels.h)
 template <typename Groups>
 inline bool groups_ok(const Groups* g, int n, int ldc) {
-  if (!g || g->n_groups < 1 || g->n_groups > 8 || g->n_main < 0 || g->n_main > n || (g->n_main < n && (g->n_main % 128)) || ldc < g->n_main) return false;
+  if (!g || g->silu_begin < 0 || g->silu_begin % 32 || g->silu_end % 32 || g->silu_end < g->silu_begin || g->silu_end > g->n_main) return false;
+  if (g->n_groups < 1 || g->n_groups > 8 || g->n_main < 0 || g->n_main > n || (g->n_main < n && (g->n_main % 128)) || ldc < g->n_main) return false;
   for (int i = 0; i < g->n_groups; ++i) {
     if (g->end[i] <= (i ? g->end[i - 1] : 0) || (i + 1 < g->n_groups && g->end[i] % 128)) return false;
   }
@@ -127,6 +128,8 @@ LG_DEVINL float glu_clamp(float g, float u, float alpha, float limit, float shif
   u = fminf(fmaxf(u, -limit), limit);
   return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + shift);
 }
+
+LG_DEVINL float silu_fast(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 
 LG_DEVINL float fast_exp2(float x) {
   float y;

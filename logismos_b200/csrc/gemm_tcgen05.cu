@@ -287,6 +287,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
             }
             continue;
           }
+          const bool silu = EPI == kEpiGroups && ncol >= groups.silu_begin && ncol < groups.silu_end;
           if (row < row_end) {
               __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * ldc + ncol;
 #pragma unroll
@@ -299,6 +300,7 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                     float a = __uint_as_float(r[e]), b = __uint_as_float(r[e + 1]);
                     if (bias) { a += bias[ncol + e]; b += bias[ncol + e + 1]; }
                     if (EPI == LG_EPI_RELU2) { a = fmaxf(a, 0.0f); b = fmaxf(b, 0.0f); a *= a; b *= b; }
+                    if (silu) { a = lg::silu_fast(a); b = lg::silu_fast(b); }
                     w[i] = pack_bf16x2(a, b);
                   }
                   *reinterpret_cast<uint4*>(dst + j * 8) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -495,7 +497,7 @@ struct ExpertRows {
 };
 
 template <int BN, int EPI>
-uint32_t launch_experts(const ExpertRows& x, const void* w, void* out, int n, int k, int lda, int ldc, int* status, cudaStream_t stream) {
+uint32_t launch_experts(const ExpertRows& x, const void* w, void* out, int n, int k, int lda, int ldc, EpiParams ep, int* status, cudaStream_t stream) {
   CUtensorMap ma, md, mw;
   if (!make_map(&ma, x.a, (uint64_t)x.a_rows, (uint64_t)k, (uint64_t)lda, BM)) return lg::kInvalidValue;
   if (x.direct) {
@@ -509,17 +511,17 @@ uint32_t launch_experts(const ExpertRows& x, const void* w, void* out, int n, in
   if (e != cudaSuccess) return (uint32_t)e;
   const int64_t items = (int64_t)x.max_tiles * ((n + BN - 1) / BN);
   const int grid = items < sm_count() ? (int)items : sm_count();
-  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, md, (const float*)nullptr, out, x.a_rows, n, k, ldc, 1, 0, EpiParams{}, lg_linear_groups_t{},
+  lg::launch(kern, dim3(grid), dim3(kThreads), Cfg<BN>::kSmem, stream, ma, mw, md, (const float*)nullptr, out, x.a_rows, n, k, ldc, 1, 0, ep, lg_linear_groups_t{},
              x.tiles, status);
   return lg::launch_status();
 }
 
 // tile width as in launch_epi; the number of row tiles is only bounded here, about half of the partial ones are counted
 template <int EPI>
-uint32_t launch_experts_epi(const ExpertRows& x, const void* w, void* out, int n, int k, int lda, int ldc, int* status, cudaStream_t stream) {
+uint32_t launch_experts_epi(const ExpertRows& x, const void* w, void* out, int n, int k, int lda, int ldc, EpiParams ep, int* status, cudaStream_t stream) {
   const int64_t mt = std::max(1, x.max_tiles - x.groups / 2), sms = sm_count();
   auto cost = [&](int bn) { return (mt * ((n + bn - 1) / bn) + sms - 1) / sms * bn; };
-  return cost(128) < cost(256) ? launch_experts<128, EPI>(x, w, out, n, k, lda, ldc, status, stream) : launch_experts<256, EPI>(x, w, out, n, k, lda, ldc, status, stream);
+  return cost(128) < cost(256) ? launch_experts<128, EPI>(x, w, out, n, k, lda, ldc, ep, status, stream) : launch_experts<256, EPI>(x, w, out, n, k, lda, ldc, ep, status, stream);
 }
 
 }  // namespace
@@ -528,17 +530,19 @@ extern "C" {
 
 uint32_t logismos_launch_linear_experts_tc_bf16(const void* a, int32_t a_rows, const void* a_direct, int32_t direct_rows, const void* w, void* out,
                                                 const void* tiles, const void* n_tiles, int32_t max_tiles, int32_t n_groups, int32_t n, int32_t k,
-                                                int32_t lda, int32_t ldc, int32_t epilogue, void* status, void* stream) {
+                                                int32_t lda, int32_t ldc, int32_t epilogue, float p0, float p1, float p2, void* status, void* stream) {
   lg::LaunchScope launch_scope_;
   epilogue &= ~LG_EPI_STATIC_W;
-  const bool glu = epilogue == LG_EPI_SWIGLU;
+  const bool glu = epilogue == LG_EPI_SWIGLU || epilogue == LG_EPI_GLU_CLAMP;
+  const EpiParams ep{p0, p1, p2};
   if (!a || a_rows <= 0 || !w || !out || !tiles || !n_tiles || max_tiles <= 0 || n_groups <= 0 || n <= 0 || n % (glu ? 64 : 16) || k <= 0 || k % BK || lda < k || lda % 8 ||
       ldc % 8 || ldc < (glu ? n / 2 : n) || (a_direct && direct_rows <= 0) || (int64_t)n * n_groups > 0x7fffffff ||
       (((uintptr_t)a | (uintptr_t)a_direct | (uintptr_t)w | (uintptr_t)out | (uintptr_t)tiles) & 15))
     return lg::kInvalidValue;
   const ExpertRows x{a, a_rows, a_direct, direct_rows, RowTiles{(const int4*)tiles, (const int*)n_tiles, a_direct ? 1 : 0}, max_tiles, n_groups};
-  if (glu) return launch_experts_epi<LG_EPI_SWIGLU>(x, w, out, n, k, lda, ldc, (int*)status, (cudaStream_t)stream);
-  if (epilogue == LG_EPI_BF16) return launch_experts_epi<LG_EPI_BF16>(x, w, out, n, k, lda, ldc, (int*)status, (cudaStream_t)stream);
+  if (epilogue == LG_EPI_SWIGLU) return launch_experts_epi<LG_EPI_SWIGLU>(x, w, out, n, k, lda, ldc, ep, (int*)status, (cudaStream_t)stream);
+  if (epilogue == LG_EPI_GLU_CLAMP) return launch_experts_epi<LG_EPI_GLU_CLAMP>(x, w, out, n, k, lda, ldc, ep, (int*)status, (cudaStream_t)stream);
+  if (epilogue == LG_EPI_BF16) return launch_experts_epi<LG_EPI_BF16>(x, w, out, n, k, lda, ldc, ep, (int*)status, (cudaStream_t)stream);
   return lg::kInvalidValue;
 }
 

@@ -168,6 +168,7 @@ linear_small_kernel(SmallArgs p) {
     }
     if (p.bias && (p.epi != kEpiGroups || wrow < p.groups.n_main)) v += p.bias[wrow];
     if (p.epi == LG_EPI_RELU2) { v = fmaxf(v, 0.0f); v *= v; }
+    if (p.epi == kEpiGroups && wrow >= p.groups.silu_begin && wrow < p.groups.silu_end) v = silu_fast(v);
     if (p.epi == kEpiGroups && wrow >= p.groups.n_main) {
       const int tc = wrow - p.groups.n_main, width = p.n - p.groups.n_main;
       if (p.groups.tail_cap > 0.0f) v = p.groups.tail_cap * tanhf(v / p.groups.tail_cap);
@@ -209,7 +210,7 @@ uint32_t launch_small(const SmallArgs& a, int batch, int warps, cudaStream_t s) 
 
 template <int NT>
 uint32_t launch_small_experts(const SmallArgs& a, int n_groups, int max_rows, int warps, cudaStream_t s) {
-  const bool glu = a.epi == LG_EPI_SWIGLU;
+  const bool glu = a.epi == LG_EPI_SWIGLU || a.epi == LG_EPI_GLU_CLAMP;
   const size_t smem = (size_t)warps * 32 * 8 * NT * 4;
   auto kern = linear_small_kernel<2, NT, true>;
   if (smem > 48 * 1024) {
@@ -306,7 +307,7 @@ linear_f32_kernel(F32Args p) {
       if (c >= p.n) continue;
       if (p.epi == kEpiGroups) {
         const float v = acc[i][j];
-        if (c < p.groups.n_main) out[(size_t)r * p.ldc + c] = v;
+        if (c < p.groups.n_main) out[(size_t)r * p.ldc + c] = c >= p.groups.silu_begin && c < p.groups.silu_end ? v / (1.0f + expf(-v)) : v;
         else reinterpret_cast<float*>(p.groups.tail)[(size_t)r * p.groups.ld_tail + c - p.groups.n_main] = p.groups.tail_cap > 0.0f ? p.groups.tail_cap * tanhf(v / p.groups.tail_cap) : v;
         continue;
       }
@@ -359,6 +360,7 @@ groups_finish_kernel(float* __restrict__ acc, __nv_bfloat16* __restrict__ out, i
       const float4 b = __ldg(reinterpret_cast<const float4*>(reinterpret_cast<const float*>(g.bias) + c));
       v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
     }
+    if (c >= g.silu_begin && c < g.silu_end) v = make_float4(silu_fast(v.x), silu_fast(v.y), silu_fast(v.z), silu_fast(v.w));
     *reinterpret_cast<uint2*>(out + (size_t)r * ldc + c) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
     return;
   }
@@ -458,14 +460,14 @@ uint32_t logismos_launch_linear_groups_f32(const void* a, const void* w, void* o
 
 uint32_t logismos_launch_linear_experts_small_bf16(const void* a, const void* w, void* out, const void* offsets, const void* row_idx, int32_t n_groups,
                                                    int32_t max_group_rows, int32_t expected_group_rows, int32_t n, int32_t k, int32_t lda, int32_t ldc,
-                                                   int32_t epilogue, void* stream) {
+                                                   int32_t epilogue, float p0, float p1, float p2, void* stream) {
   lg::LaunchScope launch_scope_;
   epilogue &= ~LG_EPI_STATIC_W;
-  const bool glu = epilogue == LG_EPI_SWIGLU;
+  const bool glu = epilogue == LG_EPI_SWIGLU || epilogue == LG_EPI_GLU_CLAMP;
   if (!a || !w || !out || !offsets || n_groups <= 0 || n_groups > 65535 || max_group_rows <= 0 || max_group_rows > (1 << 19) || n <= 0 || n % (glu ? 64 : 16) || k <= 0 ||
       k % 32 || lda < k || lda % 8 || ldc < (glu ? n / 2 : n) || (((uintptr_t)a | (uintptr_t)w) & 15) || (!glu && epilogue != LG_EPI_BF16))
     return lg::kInvalidValue;
-  SmallArgs p{(const __nv_bfloat16*)a, (const __nv_bfloat16*)w, nullptr, out, 0, n, k, lda, ldc, epilogue, 0, (int64_t)n * k, 0, 0, 0, 0, {}, (const int*)offsets,
+  SmallArgs p{(const __nv_bfloat16*)a, (const __nv_bfloat16*)w, nullptr, out, 0, n, k, lda, ldc, epilogue, 0, (int64_t)n * k, 0, p0, p1, p2, {}, (const int*)offsets,
               (const int*)row_idx};
   const int steps = k / 32, warps = steps < 8 ? steps : 8, rows = expected_group_rows < max_group_rows ? expected_group_rows : max_group_rows;
   cudaStream_t s = (cudaStream_t)stream;

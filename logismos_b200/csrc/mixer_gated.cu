@@ -18,50 +18,19 @@ namespace {
 
 constexpr uint16_t kOne = 0x3f80;  // 1.0 in bf16
 
-lg_window_t window_of(const MLayer& L, const void* gate, int ld_gate) { return lg_window_t{L.c.scale, L.c.window, L.c.keep_first, 1, gate, ld_gate}; }
-
 uint32_t attention(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   const lg_mixer_config_t& c = m->cfg;
   StepBatch& B = m->batch;
-  const DecodeView& V = m->views[(size_t)L.view];
-  const int T = B.T, MB = c.max_blocks_per_seq, P = L.groups.n_main, f32 = c.is_f32;
-  const size_t esz = f32 ? 4 : 2;
-  void* st = m->status.p;
-  uint8_t *proj = (uint8_t*)m->proj.p, *out = (uint8_t*)m->act.p;
+  const int T = B.T, P = L.groups.n_main, f32 = c.is_f32;
+  void *st = m->status.p, *proj = m->proj.p;
   LG_TRY(projections(m, L, W, false, s), "input projections");
   LG_TRY(logismos_launch_qk_norm_rotary_store(proj, P, L.kpool.p, L.vpool.p, m->dev(B.slots), m->dev(B.pos), T, L.c.heads, L.c.kv_heads, L.Dh, L.c.dim, W.gain_q.p,
                                               W.gain_k.p, c.norm_eps, L.table < 0 ? nullptr : m->tables[(size_t)L.table].angles.p, L.c.rot_dims,
                                               (int64_t)c.n_pool_blocks * kKvBlock, f32, st, s), "queries, keys and cache store");
   m->launches += 1;
-  lg_window_t w = window_of(L, m->tail.p, L.groups.ld_tail);
-  if (f32) {
-    LG_TRY(logismos_launch_window_attention_f32(proj, P, L.kpool.p, L.vpool.p, m->dev(B.tables), m->dev(B.seq_ids), m->dev(B.pos), out, L.Kout, T, MB,
-                                                c.n_pool_blocks, L.c.heads, L.c.kv_heads, L.Dh, &w, st, s), "attention");
-    m->launches += 1;
-    return 0;
-  }
-  if (B.n_dec > 0) {
-    LG_TRY(logismos_launch_window_attention_decode_bf16(proj, P, L.kpool.p, L.vpool.p, m->dev(B.tables), m->dev(B.ctx), m->dev(V.chunks), out, L.Kout,
-                                                        m->dec_scratch.p, B.n_dec, V.total, V.chunk_tokens, MB, c.n_pool_blocks, L.c.heads, L.c.kv_heads,
-                                                        L.Dh, &w, st, s), "decode attention");
-    m->launches += V.total > B.n_dec ? 2 : 1;
-  }
-  const size_t row0 = (size_t)B.n_dec;
-  w.gate = (const float*)w.gate + row0 * w.ld_gate;
-  for (const PrefixRun& r : B.runs) {
-    int total = 0, longest = 0;
-    for (int k = r.s0; k < r.s1; ++k) {
-      const int n = logismos_window_keys(B.pre_kv[k], B.newl[row0 + (size_t)k], L.c.window, L.c.keep_first);
-      total += n;
-      longest = std::max(longest, n);
-    }
-    LG_TRY(logismos_launch_window_attention_prefix_bf16(proj + row0 * P * esz, P, m->dev(B.cu_pre) + r.s0, m->dev(B.pre_kv) + r.s0, L.kpool.p, L.vpool.p,
-                                                        m->dev(B.tables) + (row0 + r.s0) * MB, MB, c.n_pool_blocks, out + row0 * L.Kout * esz, L.Kout,
-                                                        m->attn_ws.p, T - B.n_dec, total, r.s1 - r.s0, r.max_q, longest, L.c.heads, L.c.kv_heads, L.Dh, &w,
-                                                        st, s), "attention");
-    m->launches += 2;
-  }
-  return 0;
+  lg_window_t w = m->views[(size_t)L.view].shape;
+  w.scale = L.c.scale; w.sink = 1; w.gate = m->tail.p; w.ld_gate = L.groups.ld_tail;
+  return window_attention(m, L, w, proj, P, L.c.heads, L.c.kv_heads, L.Dh, m->act.p, L.Kout, s);
 }
 
 uint32_t gated_linear_attention(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
@@ -158,6 +127,40 @@ void gate_up_rows(Mat& dst, int row0, const void* gate, const void* up, int firs
 
 }  // namespace
 
+uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int ld_q, int heads, int kv, int hd, void* out, int ld_out, cudaStream_t s) {
+  const lg_mixer_config_t& c = m->cfg;
+  StepBatch& B = m->batch;
+  const DecodeView& V = m->views[(size_t)L.view];
+  const int T = B.T, MB = c.max_blocks_per_seq;
+  void* st = m->status.p;
+  if (c.is_f32) {
+    LG_TRY(logismos_launch_window_attention_f32(q, ld_q, L.kpool.p, L.vpool.p, m->dev(B.tables), m->dev(B.seq_ids), m->dev(B.pos), out, ld_out, T, MB, c.n_pool_blocks,
+                                                heads, kv, hd, &w, st, s), "attention");
+    m->launches += 1;
+    return 0;
+  }
+  if (B.n_dec > 0) {
+    LG_TRY(logismos_launch_window_attention_decode_bf16(q, ld_q, L.kpool.p, L.vpool.p, m->dev(B.tables), m->dev(B.ctx), m->dev(V.chunks), out, ld_out, m->dec_scratch.p,
+                                                        B.n_dec, V.total, V.chunk_tokens, MB, c.n_pool_blocks, heads, kv, hd, &w, st, s), "decode attention");
+    m->launches += V.total > B.n_dec ? 2 : 1;
+  }
+  const size_t row0 = (size_t)B.n_dec;
+  if (w.gate) w.gate = (const float*)w.gate + row0 * w.ld_gate;
+  for (const PrefixRun& r : B.runs) {
+    int total = 0, longest = 0;
+    for (int k = r.s0; k < r.s1; ++k) {
+      const int n = logismos_window_view_keys(&w, B.pre_kv[k], B.newl[row0 + (size_t)k]);
+      total += n;
+      longest = std::max(longest, n);
+    }
+    LG_TRY(logismos_launch_window_attention_prefix_bf16((const uint16_t*)q + row0 * ld_q, ld_q, m->dev(B.cu_pre) + r.s0, m->dev(B.pre_kv) + r.s0, L.kpool.p, L.vpool.p,
+                                                        m->dev(B.tables) + (row0 + r.s0) * MB, MB, c.n_pool_blocks, (uint8_t*)out + row0 * ld_out * (w.out_f32 ? 4 : 2),
+                                                        ld_out, m->attn_ws.p, T - B.n_dec, total, r.s1 - r.s0, r.max_q, longest, heads, kv, hd, &w, st, s), "attention");
+    m->launches += 2;
+  }
+  return 0;
+}
+
 uint32_t run_gated_kinds(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   return L.c.kind == LG_MIXER_ATTENTION ? attention(m, L, W, s) : L.c.kind == LG_MIXER_GLA ? gated_linear_attention(m, L, W, s) : latent_attention(m, L, W, s);
 }
@@ -168,12 +171,16 @@ uint32_t run_mixture(Mixer* m, const MLayer& L, const MWeights& W, lg_mixture_ou
   const bool few = f32 || logismos_moe_streams(T, y.top, y.experts, y.identity, L.always, Hp, L.Fp);
   const bool acc = T > 32 && !f32 && !logismos_get_deterministic();  // the narrow product is split over k whatever the rows
   void *logits = acc ? m->route_acc.p : m->route.p, *st = m->status.p;
-  // a step of a few tokens with a small router: the product rides on the choice
-  const bool fused = few && !f32 && (int64_t)T * n_routed * Hp <= 1 << 22;
-  if (!fused) LG_TRY(linear(m, m->h.p, Hp, W.w_router, L.route_ld, Hp, logits, L.route_ld, acc ? LG_EPI_RESID_F32 : LG_EPI_F32, T, s), "router");
+  // a step of a few tokens with a small router: the product rides on the choice; in a gated stack on the gate's
+  const bool gated = m->cfg.norm == LG_NORM_RMS_GATED, fused = !gated && few && !f32 && (int64_t)T * n_routed * Hp <= 1 << 22;
+  if (gated) logits = m->route.p;
+  else if (!fused) LG_TRY(linear(m, m->h.p, Hp, W.w_router, L.route_ld, Hp, logits, L.route_ld, acc ? LG_EPI_RESID_F32 : LG_EPI_F32, T, s), "router");
   lg_moe_route_t r{};
   if (fused) { r.h = m->h.p; r.w = W.w_router.p; r.width = Hp; r.arrived = (uint8_t*)m->counts.p + m->counts_bytes - 4; }
-  r.logits = logits; r.ld = L.route_ld; r.zero_logits = acc; r.correction = W.correction.p;
+  r.logits = logits; r.ld = L.route_ld; r.zero_logits = acc && !gated; r.correction = W.correction.p;
+  r.scoring = y.scoring; r.groups = y.route_groups; r.keep_groups = y.keep_groups;
+  const bool clamped = y.glu_limit > 0.0f;
+  const int glu = clamped ? LG_EPI_GLU_CLAMP : LG_EPI_SWIGLU;
   r.n_experts = y.experts; r.n_identity = n_routed - y.experts; r.top = y.top; r.n_always = L.always;
   r.weights = m->pair_w.p; r.pair_row = m->pair_row.p; r.identity = m->identity.p;
   *out = lg_mixture_out_t{m->expert_rows.p, m->pair_row.p, m->pair_w.p, m->identity.p, pairs, y.top, nullptr, 0};
@@ -182,13 +189,14 @@ uint32_t run_mixture(Mixer* m, const MLayer& L, const MWeights& W, lg_mixture_ou
     LG_TRY(logismos_launch_moe_route(&r, T, s), "choice of experts");
     const int expected = T <= 8 ? 8 : 16;
     if (f32) {
-      LG_TRY(logismos_launch_linear_experts_f32(m->h.p, W.w_up.p, m->ffb.p, r.offsets, r.row_token, groups, T, 2 * L.Fp, Hp, Hp, L.Fp, LG_EPI_GLU_CLAMP, 1.0f, INFINITY,
-                                                0.0f, s), "experts, gate and up");
+      LG_TRY(logismos_launch_linear_experts_f32(m->h.p, W.w_up.p, m->ffb.p, r.offsets, r.row_token, groups, T, 2 * L.Fp, Hp, Hp, L.Fp, LG_EPI_GLU_CLAMP,
+                                                clamped ? y.glu_alpha : 1.0f, clamped ? y.glu_limit : INFINITY, clamped ? y.glu_shift : 0.0f, s), "experts, gate and up");
       LG_TRY(logismos_launch_linear_experts_f32(m->ffb.p, W.w_down.p, m->expert_rows.p, r.offsets, nullptr, groups, T, Hp, L.Fp, L.Fp, Hp, LG_EPI_F32, 0, 0, 0, s), "experts, down");
     } else {
-      LG_TRY(logismos_launch_linear_experts_small_bf16(m->h.p, W.w_up.p, m->ffb.p, r.offsets, r.row_token, groups, T, expected, 2 * L.Fp, Hp, Hp, L.Fp, LG_EPI_SWIGLU, s),
+      LG_TRY(logismos_launch_linear_experts_small_bf16(m->h.p, W.w_up.p, m->ffb.p, r.offsets, r.row_token, groups, T, expected, 2 * L.Fp, Hp, Hp, L.Fp, glu, y.glu_alpha,
+                                                       y.glu_limit, y.glu_shift, s),
              "experts, gate and up");
-      LG_TRY(logismos_launch_linear_experts_small_bf16(m->ffb.p, W.w_down.p, m->expert_rows.p, r.offsets, nullptr, groups, T, expected, Hp, L.Fp, L.Fp, Hp, LG_EPI_BF16, s),
+      LG_TRY(logismos_launch_linear_experts_small_bf16(m->ffb.p, W.w_down.p, m->expert_rows.p, r.offsets, nullptr, groups, T, expected, Hp, L.Fp, L.Fp, Hp, LG_EPI_BF16, 0, 0, 0, s),
              "experts, down");
     }
     m->launches += 3;
@@ -200,9 +208,9 @@ uint32_t run_mixture(Mixer* m, const MLayer& L, const MWeights& W, lg_mixture_ou
   LG_TRY(logismos_launch_moe_route(&r, T, s), "choice of experts");
   LG_TRY(logismos_launch_moe_place(&r, m->h.p, m->gathered.p, Hp, T, s), "rows by expert");
   LG_TRY(logismos_launch_linear_experts_tc_bf16(m->gathered.p, rows, m->h.p, T, W.w_up.p, m->ffb.p, r.tiles, r.n_tiles, max_tiles, groups, 2 * L.Fp, Hp, Hp, L.Fp,
-                                                LG_EPI_SWIGLU, st, s), "experts, gate and up");
+                                                glu, y.glu_alpha, y.glu_limit, y.glu_shift, st, s), "experts, gate and up");
   LG_TRY(logismos_launch_linear_experts_tc_bf16(m->ffb.p, rows, nullptr, 0, W.w_down.p, m->expert_rows.p, r.tiles, r.n_tiles, max_tiles, groups, Hp, L.Fp, L.Fp, Hp,
-                                                LG_EPI_BF16, st, s), "experts, down");
+                                                LG_EPI_BF16, 0, 0, 0, st, s), "experts, down");
   m->launches += 4;
   out->counts = r.counts;
   out->n_counts = y.experts;
@@ -383,6 +391,11 @@ const char* check_feed_forward(const lg_mixer_layer_config_t& y) {
   if (y.ff_kind != LG_FF_MIXTURE) return "kind of feed-forward";
   if (y.experts <= 0 || y.identity < 0 || y.experts + y.identity > 512) return "experts (at most 512 with the identity experts)";
   if (y.top <= 0 || y.top > 32 || y.top > y.experts + y.identity) return "experts per token (at most 32)";
+  if (y.scoring != LG_ROUTE_SOFTMAX && y.scoring != LG_ROUTE_SIGMOID) return "scores of the router";
+  if (y.route_groups < 0 || (y.route_groups > 0 && ((y.experts + y.identity) % y.route_groups || y.keep_groups <= 0 || y.keep_groups > y.route_groups ||
+                                                    y.top > (y.experts + y.identity) / y.route_groups * y.keep_groups)))
+    return "groups of experts";
+  if (!(y.glu_limit >= 0.0f)) return "a limit of the gated units that is negative";
   if (y.shared_ff < 0 || (y.shared_ff + y.ff - 1) / y.ff > 64) return "a shared expert of more than 64 times an expert's size";
   return nullptr;
 }
@@ -416,9 +429,11 @@ bool upload_feed_forward(Mixer* m, const MLayer& L, MWeights& W, const lg_mixer_
         cudaMemcpy((uint8_t*)W.w_down.p + e * down_bytes, d.v.data(), down_bytes, cudaMemcpyHostToDevice) != cudaSuccess)
       return false;
   }
+  if (!c.no_correction && !upload_vec(W.correction, w.correction, n, n, 0.0f)) return false;
+  if (m->cfg.norm == LG_NORM_RMS_GATED) return true;  // the router's rows follow those of the gate
   Mat router(L.route_ld, Hp);
   for (int i = 0; i < n; ++i) router.row(i, 0, w.router, (size_t)i * H, H);
-  return router.up(W.w_router) && upload_vec(W.correction, w.correction, n, n, 0.0f);
+  return router.up(W.w_router);
 }
 
 void size_feed_forward(const MLayer& L, Sizes& z) {
@@ -443,7 +458,7 @@ bool want_feed_forward(Wanted& t, const std::string& mlp, int64_t H, const lg_mi
   for (int e = 0; e < y.experts; ++e)
     if (!unit(mlp + "e" + std::to_string(e) + ".", y.ff, &experts[(size_t)3 * e], &experts[(size_t)3 * e + 1], &experts[(size_t)3 * e + 2])) return false;
   const int64_t n = y.experts + y.identity;
-  return t.get(mlp + "router", {n, H}, &L.router) && t.get(mlp + "correction", {n}, &L.correction) &&
+  return t.get(mlp + "router", {n, H}, &L.router) && (y.no_correction || t.get(mlp + "correction", {n}, &L.correction)) &&
          (!y.shared_ff || unit(mlp + "shared.", y.shared_ff, &L.shared_gate, &L.shared_up, &L.shared_down));
 }
 

@@ -1,6 +1,7 @@
 // The executor of a stack of mixers (lg_mixer_*) as its parts see it: mixer_model.cu holds the step, the norms around the
 // sublayers, creation and loading; mixer_parallel.cu the state-space and the parallel mixers; mixer_gated.cu windowed
-// attention, gated linear attention, latent attention and the gated feed-forwards.
+// attention, gated linear attention, latent attention and the gated feed-forwards; mixer_paired.cu differential attention and
+// pooled-window attention beside linear attention.
 #pragma once
 #include <cuda_runtime.h>
 
@@ -44,6 +45,9 @@ struct MWeights {   // of a layer that owns tensors
   Buf b_in, gain_q, gain_k;                               // windowed attention; latent attention: gains of its latents
   Buf w_uq, w_uk, w_ukt, w_uv;                            // latent attention
   Buf w_router, correction;                               // mixture: w_up, w_down hold its experts one after the other
+  Buf w_gate2, b_gate2;                                   // gated residual: the gate of a feed-forward, then the router's rows
+  Buf w_out2, branch_gain[2], log2_decay;                 // a pair
+  float gain1 = 0.0f, gain2 = 0.0f, lambda = 0.0f;        // norms of one value; differential attention
   float max_bias = 0.0f;
   void release();
 };
@@ -57,14 +61,16 @@ struct MLayer {
   int Dh = 0, Dp = 0, Rw = 0, Lr = 0;   // attention head, linear-attention key head, padded block of its heads, padded rank
   int Qp = 0, Rp = 0, Rc = 0, Dn = 0;   // latent attention: padded latents, first rotated column of a cache row and of a head
   int always = 0, route_ld = 0;         // mixture: experts that every token takes, columns of the router
+  int off_right = 0, off_gate = 0, Kleft = 0;   // first columns of the right branch and of the residual's gate, inputs of the left W_o
+  lg_linear_groups_t gate2{};           // gated residual: the feed-forward's gate and router
   int view = -1, table = -1;            // decode view, rotation table
-  Buf kpool, vpool, shift, conv_state, state;
+  Buf kpool, vpool, kmean, vmean, shift, conv_state, state;
 };
 
 // How decode launches split the contexts of a kind of attention: the same for all layers with one window
 struct DecodeView {
   bool latent = false;
-  int window = 0, keep_first = 0;
+  lg_window_t shape{};                  // window, kept keys, chunks, pooled blocks
   int kv = 1, hd = 64, heads = 1;       // of the widest layer
   int chunk_tokens = 512, total = 0, max_chunks = 0;
   int32_t* chunks = nullptr;            // host, in the step's index block
@@ -80,8 +86,9 @@ struct Mixer {
   lg_mixer_config_t cfg{};
   std::vector<lg_mixer_layer_config_t> layer_cfg;
   int device = 0, Hp = 0;
-  Buf embed, head, final_norm, final_norm_b;
+  Buf embed, head, final_norm, final_norm_b, loop_step;
   TanhNorm final_tanh;
+  float final_gain = 0.0f;
   std::vector<MWeights> weights;
   std::vector<MLayer> layers;
   std::vector<DecodeView> views;
@@ -89,6 +96,7 @@ struct Mixer {
   Buf x, h, proj, tail, low2, z, xbc, act, ffb, y, y_acc, hist, last, logits, tokens, status, attn_ws, dec_scratch, dev_batch;
   Buf raw_acc;                          // sums of input projections over slices of k
   Buf cq, gate, qlat, olat, lat, kbuf, vt, kv_start;                                                      // latent attention
+  Buf qx, maps_out;                     // differential attention: queries of both maps, outputs of both (fp32)
   Buf route, route_acc, pair_w, pair_row, pair_expert, identity, offsets, row_token, counts, tiles, gathered, expert_rows;  // mixture
   StepBatch batch;
   std::vector<uint8_t> slot_phase;      // per state slot: the copy that holds its convolution and shift states
@@ -109,6 +117,7 @@ struct Sizes {
   size_t raw = 0;                                                                                    // of summed input projections
   size_t cq = 0, heads = 0, lat_q = 0, lat = 0, lat_heads = 0;                             // latent attention
   size_t route = 0, pairs = 0, top = 0, groups = 0, expert_ff = 0;                                  // mixture
+  size_t maps = 0;                                                                                   // differential attention
 };
 inline void grow(size_t& a, size_t b) { if (b > a) a = b; }
 
@@ -138,6 +147,10 @@ uint32_t linear(Mixer* m, const void* a, int lda, const Buf& w, int n, int k, vo
 uint32_t head_linear(Mixer* m, const void* a, int lda, const Buf& w, int heads, int n, int k, void* out, int ldc, int rows, cudaStream_t s);
 // input projections of a layer: main columns to proj, fp32 tail to `tail` (and rounded with remainders to low2)
 uint32_t projections(Mixer* m, const MLayer& L, const MWeights& W, bool tail_parts, cudaStream_t s);
+// one grouped projection of the step's rows of h (n columns in all) to m->proj
+uint32_t grouped_projection(Mixer* m, const Buf& w, int n, const lg_linear_groups_t& g, cudaStream_t s);
+// whether a grouped projection is summed over slices of k at this number of rows
+bool splits_projections(const lg_linear_groups_t& g, int n, int rows);
 bool zeroed(Buf& b, size_t bytes);
 
 // rows of head h of src [heads * d, k] -> rows of dst at row0 + h * dp
@@ -146,7 +159,8 @@ void head_rows(Mat& dst, int row0, const void* src, int heads, int d, int dp, in
 void head_cols(Mat& dst, int col0, const void* src, int n, int heads, int d, int dp);
 
 // ---- kinds of mixers: what a layer needs (NULL or 0: fine), its layout, weights, buffers and step ----
-inline bool is_gated_kind(int kind) { return kind >= LG_MIXER_ATTENTION; }
+inline bool is_gated_kind(int kind) { return kind >= LG_MIXER_ATTENTION && kind <= LG_MIXER_LATENT; }
+inline bool is_paired_kind(int kind) { return kind >= LG_MIXER_DIFF; }
 
 const char* check_parallel_kinds(const lg_mixer_layer_config_t& y);
 const char* check_parallel_tensors(const lg_mixer_layer_config_t& y);   // sizes that a file's tensors give
@@ -163,6 +177,16 @@ bool upload_gated_kinds(Mixer* m, const MLayer& L, MWeights& W, const lg_mixer_l
 bool alloc_gated_kinds(Mixer* m, MLayer& L, Sizes& z);
 bool want_gated_kinds(Wanted& t, const std::string& mix, int64_t width, lg_mixer_layer_config_t& y, lg_mixer_layer_weights_t& L);
 uint32_t run_gated_kinds(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s);
+
+// attention over a window from queries and the layer's cache: `heads` query heads of hd channels, kv key heads
+uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int ld_q, int heads, int kv, int hd, void* out, int ld_out, cudaStream_t s);
+
+const char* check_paired_kinds(const lg_mixer_layer_config_t& y);
+void layout_paired_kinds(const Mixer* m, MLayer& L);
+bool upload_paired_kinds(Mixer* m, const MLayer& L, MWeights& W, const lg_mixer_layer_weights_t& w);   // the output projections too
+bool alloc_paired_kinds(Mixer* m, MLayer& L, Sizes& z);
+bool want_paired_kinds(Wanted& t, const std::string& mix, int64_t width, lg_mixer_layer_config_t& y, lg_mixer_layer_weights_t& L);
+uint32_t run_paired_kinds(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s);
 
 // ---- feed-forwards -----------------------------------------------------------------------------------
 const char* check_feed_forward(const lg_mixer_layer_config_t& y);

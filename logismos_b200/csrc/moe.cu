@@ -3,7 +3,8 @@
 //                 CTA per token that computes the token's logits too, the last one to finish then groups the rows
 //   many tokens   choice with per-CTA histograms (a row's rank in its group is unique, its order is not fixed; rows of a
 //                 group are independent), then a second launch that places the rows, copies them and lists the row tiles
-// Logits, softmax, choice and weights are fp32. A warp handles a token, a lane the experts lane, lane + 32, ...
+// Logits, scores (softmax or sigmoid), choice and weights are fp32. A warp handles a token, a lane the experts lane, lane +
+// 32, ... Choice by groups: the experts of all but the best groups are struck out first.
 #include "common.cuh"
 #include "logismos_kernels.h"
 
@@ -33,12 +34,61 @@ struct RouteArgs {
   const __nv_bfloat16* w;     // [experts + identity, width]
   int width;
   int* arrived;
+  int sigmoid, groups, keep_groups;
 };
 
 // float -> integer of the same order
 LG_DEVINL uint32_t ordered(float x) {
   const uint32_t u = __float_as_uint(x);
   return u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+
+// The largest c of a warp and the first output that has it (kMaxOut: all are -inf), struck out of c
+template <int R>
+LG_DEVINL int take_best(float (&c)[R], int lane, float* value) {
+  float best = -INFINITY;
+  int at = 0;
+#pragma unroll
+  for (int i = 0; i < R; ++i)
+    if (c[i] > best) { best = c[i]; at = i; }
+  const uint32_t key = ordered(best), top_key = __reduce_max_sync(0xffffffffu, key);
+  const int id = __reduce_min_sync(0xffffffffu, key == top_key ? lane + 32 * at : kMaxOut);  // equal scores: the first
+  float v = 0.0f;
+#pragma unroll
+  for (int i = 0; i < R; ++i)
+    if (id == lane + 32 * i) { v = c[i]; c[i] = -INFINITY; }
+  *value = __shfl_sync(0xffffffffu, v, id & 31);
+  return id;
+}
+
+// c of the outputs outside the best groups is struck out; a group scores the sum of its two largest
+template <int R>
+LG_DEVINL void keep_best_groups(const RouteArgs& p, float (&c)[R], int lane) {
+  const int n = p.experts + p.identity, size = n / p.groups;
+  float score[R];   // of the groups lane, lane + 32, ...
+#pragma unroll
+  for (int i = 0; i < R; ++i) score[i] = -INFINITY;
+  for (int g = 0; g < p.groups; ++g) {
+    float own[R], sum, second = 0.0f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) own[i] = (lane + 32 * i) / size == g && lane + 32 * i < n ? c[i] : -INFINITY;
+    take_best<R>(own, lane, &sum);
+    if (size > 1) take_best<R>(own, lane, &second);
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+      if (g == lane + 32 * i) score[i] = sum + second;
+  }
+  uint32_t kept = 0;   // of this lane's outputs
+  for (int k = 0; k < p.keep_groups; ++k) {
+    float unused;
+    const int g = take_best<R>(score, lane, &unused);
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+      if ((lane + 32 * i) / size == g) kept |= 1u << i;
+  }
+#pragma unroll
+  for (int i = 0; i < R; ++i)
+    if (!(kept >> i & 1)) c[i] = -INFINITY;
 }
 
 // The experts by a token's logits z: lane i < top receives the i-th choice and its weight. R: logits per lane.
@@ -51,33 +101,34 @@ LG_DEVINL void choose(const RouteArgs& p, float* z, int lane, int& expert, float
     s[i] = lane + 32 * i < n ? z[lane + 32 * i] : -INFINITY;
     mx = fmaxf(mx, s[i]);
   }
-  mx = warp_max(mx);
+  if (p.sigmoid) {
 #pragma unroll
-  for (int i = 0; i < R; ++i) {
-    s[i] = expf(s[i] - mx);
-    sum += s[i];
+    for (int i = 0; i < R; ++i) s[i] = 1.0f / (1.0f + expf(-s[i]));
+  } else {
+    mx = warp_max(mx);
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      s[i] = expf(s[i] - mx);
+      sum += s[i];
+    }
+    sum = warp_sum(sum);
+#pragma unroll
+    for (int i = 0; i < R; ++i) s[i] /= sum;
   }
-  sum = warp_sum(sum);
 #pragma unroll
   for (int i = 0; i < R; ++i) {
-    s[i] /= sum;
-    c[i] = lane + 32 * i < n ? s[i] + __ldg(p.correction + lane + 32 * i) : -INFINITY;
+    c[i] = lane + 32 * i < n ? s[i] + (p.correction ? __ldg(p.correction + lane + 32 * i) : 0.0f) : -INFINITY;
     if (p.zero && lane + 32 * i < n) z[lane + 32 * i] = 0.0f;
   }
+  if (p.groups > 0) keep_best_groups<R>(p, c, lane);
   expert = -1;
   float picked = 0.0f, total = 0.0f;
   for (int k = 0; k < p.top; ++k) {
-    float best = -INFINITY;
-    int at = 0;
+    float unused, score = 0.0f;
+    const int id = take_best<R>(c, lane, &unused);
 #pragma unroll
     for (int i = 0; i < R; ++i)
-      if (c[i] > best) { best = c[i]; at = i; }
-    const uint32_t key = ordered(best), top_key = __reduce_max_sync(0xffffffffu, key);
-    const int id = __reduce_min_sync(0xffffffffu, key == top_key ? lane + 32 * at : kMaxOut);  // equal scores: the first
-    float score = 0.0f;
-#pragma unroll
-    for (int i = 0; i < R; ++i)
-      if (id == lane + 32 * i) { score = s[i]; c[i] = -INFINITY; }
+      if (id == lane + 32 * i) score = s[i];
     score = __shfl_sync(0xffffffffu, score, id & 31);
     total += score;
     if (lane == k) { expert = id; picked = score; }
@@ -264,14 +315,17 @@ moe_place_kernel(RouteArgs p, const uint4* h, uint4* gathered, int vecs) {
 }
 
 bool route_ok(const lg_moe_route_t* a, int tokens) {
-  return a && tokens > 0 && tokens < (1 << 20) && (a->logits || a->h) && a->correction && a->weights && a->pair_row && a->identity && a->n_experts > 0 &&
+  return a && tokens > 0 && tokens < (1 << 20) && (a->logits || a->h) && a->weights && a->pair_row && a->identity && a->n_experts > 0 &&
          a->n_identity >= 0 && a->n_experts + a->n_identity <= kMaxOut && (a->h || a->ld >= a->n_experts + a->n_identity) && a->top > 0 && a->top <= kMaxTop &&
-         a->top <= a->n_experts + a->n_identity && a->n_always >= 0 && a->n_always <= kMaxAlways;
+         a->top <= a->n_experts + a->n_identity && a->n_always >= 0 && a->n_always <= kMaxAlways &&
+         (a->scoring == LG_ROUTE_SOFTMAX || a->scoring == LG_ROUTE_SIGMOID) && a->groups >= 0 &&
+         (a->groups == 0 || ((a->n_experts + a->n_identity) % a->groups == 0 && a->keep_groups > 0 && a->keep_groups <= a->groups &&
+                             a->top <= (a->n_experts + a->n_identity) / a->groups * a->keep_groups));
 }
 RouteArgs route_args(const lg_moe_route_t* a, int tokens) {
   return RouteArgs{(float*)a->logits, a->ld, a->zero_logits, (const float*)a->correction, a->n_experts, a->n_identity, a->top, a->n_always, (float*)a->weights,
                    (int*)a->pair_row, (float*)a->identity, (int*)a->offsets, (int*)a->row_token, (int*)a->counts, (int*)a->pair_expert, (int4*)a->tiles,
-                   (int*)a->n_tiles, tokens, (const __nv_bfloat16*)a->h, (const __nv_bfloat16*)a->w, a->width, (int*)a->arrived};
+                   (int*)a->n_tiles, tokens, (const __nv_bfloat16*)a->h, (const __nv_bfloat16*)a->w, a->width, (int*)a->arrived, a->scoring == LG_ROUTE_SIGMOID, a->groups, a->keep_groups};
 }
 
 }  // namespace

@@ -1,6 +1,7 @@
-// Rotary positions in the interleaved layout, fused with what surrounds them: norms of whole query and key projections
-// and the cache store of a packed q | k | v row, or the rotated part of every query head in place. Angles come from a
-// table of (cos, sin) per position and pair, amplitude included; norms and rotations are fp32.
+// Rotary positions in the interleaved layout, fused with what surrounds them: norms of whole query and key projections, or of
+// every head, and the cache store of a packed q | k | v row, or the rotated part of every query head in place. Angles come
+// from a table of (cos, sin) per position and pair, amplitude included; norms and rotations are fp32. The means of blocks of
+// cached keys and values are made where the last token of a block is stored, or by a launch after it.
 #include "common.cuh"
 #include "logismos_kernels.h"
 #include "recurrent.cuh"
@@ -119,9 +120,176 @@ rotary_heads_kernel(T* __restrict__ q, int ld, const int* __restrict__ pos, int 
   *x = pack<T>(f);
 }
 
+struct HeadArgs {
+  void* qkv;
+  int ld, rows, heads, n_kv, maps, dim;
+  const float *gain_q, *gain_k;
+  float eps;
+  const float2* table;
+  int pairs;
+  void* q_out;
+  int ld_q;
+  void *kpool, *vpool;
+  const int64_t* slots;
+  const int* pos;
+  int64_t n_slots;
+  int pool, pool_rows;
+  void *kmean, *vmean;
+  const int *tables, *seq_ids;
+  int max_blocks, n_pool_blocks;
+  int* status;
+};
+
+// The mean of the block of tokens that ends at position `at`, eight channels of a cache row from channel c0 on
+template <typename T>
+LG_DEVINL void pool_piece(const HeadArgs& p, const T* pool, T* mean, int seq, int at, int row_w, int c0) {
+  const int* table = p.tables + (size_t)seq * p.max_blocks;
+  float sum[8] = {};
+  int page = -1, block = -1;
+#pragma unroll 4
+  for (int j = at + 1 - p.pool; j <= at; ++j) {
+    if (j >> 4 != page) {
+      page = j >> 4;
+      block = page < p.max_blocks ? table[page] : -1;
+      if (block < 0 || block >= p.n_pool_blocks) {
+        if (p.status) atomicExch(p.status, 1);
+        return;
+      }
+    }
+    float f[8];
+    unpack<T>(*reinterpret_cast<const Vec8<T>*>(pool + ((size_t)block * 16 + (j & 15)) * row_w + c0), f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) sum[i] += f[i];
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i) sum[i] /= (float)p.pool;
+  const int b = at / p.pool, rows = (15 + p.pool) / p.pool;
+  *reinterpret_cast<Vec8<T>*>(mean + ((size_t)block * rows + b - (page << 4) / p.pool) * row_w + c0) = pack<T>(sum);
+}
+
+// LANES lanes hold a piece of HD channels, eight each; a group of lanes takes ITEMS pieces, all requested at once
+template <typename T, int LANES, int ITEMS>
+__global__ void __launch_bounds__(kThreads)
+head_norm_store_kernel(HeadArgs p) {
+  lg::pdl_prologue();
+  constexpr int HD = LANES * 8;
+  const uint32_t nq = p.heads * p.maps, nk = p.n_kv * p.maps, per_row = nq + 2 * nk, lane = threadIdx.x % LANES;
+  const uint32_t total = p.rows * per_row, first = (blockIdx.x * kThreads + threadIdx.x) / LANES * ITEMS;
+  const int row_w = (int)nk * HD, c = (int)lane * 8;
+  Vec8<T> x[ITEMS];
+  int row[ITEMS], unit[ITEMS];
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const uint32_t at = min(first + i, total - 1);
+    row[i] = (int)(at / per_row);
+    unit[i] = (int)(at % per_row);
+    x[i] = *reinterpret_cast<const Vec8<T>*>(reinterpret_cast<const T*>(p.qkv) + (size_t)row[i] * p.ld + unit[i] * HD + c);
+  }
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const bool in = first + i < total;
+    const uint32_t u = (uint32_t)unit[i];
+    const int r = row[i], pos = p.pos[r];
+    if (u < nq + nk) {   // the same for all lanes of a piece
+      float f[8], ss = 0.0f;
+      unpack<T>(x[i], f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
+      constexpr int kWidth = LANES;
+      const uint32_t mask = kWidth == 32 ? 0xffffffffu : ((1u << (kWidth & 31)) - 1u) << ((threadIdx.x & 31) / kWidth * kWidth);
+#pragma unroll
+      for (int o = 1; o < LANES; o <<= 1) ss += __shfl_xor_sync(mask, ss, o);
+      const float m = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
+      const float4* gain = reinterpret_cast<const float4*>((u < nq ? p.gain_q : p.gain_k) + c);
+      const float4 g0 = __ldg(gain), g1 = __ldg(gain + 1);
+      const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] *= m * g[j];
+      rotate8(f, c, p.pairs, p.table + (size_t)pos * p.pairs);
+      x[i] = pack<T>(f);
+    }
+    if (!in) continue;
+    if (u < nq) {
+      T* q = reinterpret_cast<T*>(p.q_out) + (size_t)r * p.ld_q + u * p.maps * HD + c;
+      if (p.maps == 1) { *reinterpret_cast<Vec8<T>*>(q) = x[i]; continue; }
+      const int map = (int)(u / (p.heads / p.n_kv)) & 1;
+      const float zero[8] = {};
+      *reinterpret_cast<Vec8<T>*>(q + map * HD) = x[i];
+      *reinterpret_cast<Vec8<T>*>(q + (1 - map) * HD) = pack<T>(zero);
+      continue;
+    }
+    const int64_t slot = p.slots[r];
+    if (slot < 0 || slot >= p.n_slots) {
+      if (lane == 0 && p.status) atomicExch(p.status, 1);
+      continue;
+    }
+    const bool is_v = u >= nq + nk;
+    const int at = (int)(u - nq - (is_v ? nk : 0)) * HD + c;
+    T* pool = reinterpret_cast<T*>(is_v ? p.vpool : p.kpool);
+    *reinterpret_cast<Vec8<T>*>(pool + (size_t)slot * row_w + at) = x[i];
+    if (p.pool && r < p.pool_rows && (pos + 1) % p.pool == 0) pool_piece<T>(p, pool, reinterpret_cast<T*>(is_v ? p.vmean : p.kmean), r, pos, row_w, at);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+pool_blocks_kernel(HeadArgs p, int octs) {
+  lg::pdl_prologue();
+  const uint32_t at = blockIdx.x * kThreads + threadIdx.x;
+  const int r = p.pool_rows + (int)(at / (2 * octs)), piece = (int)(at % (2 * octs));
+  if (r >= p.rows || (p.pos[r] + 1) % p.pool) return;
+  const bool is_v = piece >= octs;
+  pool_piece<T>(p, reinterpret_cast<const T*>(is_v ? p.vpool : p.kpool), reinterpret_cast<T*>(is_v ? p.vmean : p.kmean), p.seq_ids[r], p.pos[r], octs * 8,
+                8 * (is_v ? piece - octs : piece));
+}
+
+bool head_args(const lg_head_norm_t* a, int is_f32, void* status, HeadArgs* p) {
+  if (!a || !a->qkv || !a->gain_q || !a->gain_k || !a->k_pool || !a->v_pool || !a->slots_i64 || !a->positions_i32 || a->rows <= 0 || a->heads <= 0 || a->n_kv <= 0 ||
+      a->heads % a->n_kv || (a->maps != 1 && a->maps != 2) || (a->hd != 32 && a->hd != 64 && a->hd != 128 && a->hd != 256) || a->dim <= 0 || a->dim > a->hd ||
+      a->rot_dims < 0 || a->rot_dims % 2 || a->rot_dims > a->dim || (a->rot_dims && !a->table) || a->ld % 8 || a->ld < a->maps * (a->heads + 2 * a->n_kv) * a->hd ||
+      (a->maps == 2 && (!a->q_out || a->ld_q < 4 * a->heads * a->hd || a->ld_q % 8)) ||
+      (((uintptr_t)a->qkv | (uintptr_t)a->k_pool | (uintptr_t)a->v_pool | (uintptr_t)a->q_out | (uintptr_t)a->k_mean | (uintptr_t)a->v_mean) & (is_f32 ? 31 : 15)) ||
+      (((uintptr_t)a->gain_q | (uintptr_t)a->gain_k) & 15) || ((uintptr_t)a->table & 7) || (int64_t)a->rows * a->maps * (a->heads + 2 * a->n_kv) > (1 << 26))
+    return false;
+  if (a->pool < 0 || (a->pool && (!a->k_mean || !a->v_mean || !a->tables_i32 || !a->seq_ids_i32 || a->pool_rows < 0 || a->max_blocks <= 0 || a->n_pool_blocks <= 0))) return false;
+  *p = HeadArgs{a->qkv, a->ld, a->rows, a->heads, a->n_kv, a->maps, a->dim, (const float*)a->gain_q, (const float*)a->gain_k, a->eps, (const float2*)a->table, a->rot_dims / 2,
+                a->maps == 1 ? a->qkv : a->q_out, a->maps == 1 ? a->ld : a->ld_q, a->k_pool, a->v_pool, (const int64_t*)a->slots_i64, (const int*)a->positions_i32,
+                a->n_pool_slots, a->pool, a->pool_rows, a->k_mean, a->v_mean, (const int*)a->tables_i32, (const int*)a->seq_ids_i32, a->max_blocks, a->n_pool_blocks,
+                (int*)status};
+  return true;
+}
+
 }  // namespace
 
 extern "C" {
+
+uint32_t logismos_launch_head_norm_store(const lg_head_norm_t* a, int32_t is_f32, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  HeadArgs p;
+  if (!head_args(a, is_f32, status, &p)) return lg::kInvalidValue;
+  const int64_t items = (int64_t)a->rows * a->maps * (a->heads + 2 * a->n_kv);
+  auto go = [&](auto kern, int per_block) -> uint32_t {
+    lg::launch(kern, dim3((unsigned)((items + per_block - 1) / per_block)), dim3(kThreads), 0, (cudaStream_t)stream, p);
+    return lg::launch_status();
+  };
+#define LG_HEADS(T, LANES) (items < 20000 ? go(head_norm_store_kernel<T, LANES, 1>, kThreads / LANES) : go(head_norm_store_kernel<T, LANES, 4>, kThreads / LANES * 4))
+  if (is_f32) return a->hd == 32 ? LG_HEADS(float, 4) : a->hd == 64 ? LG_HEADS(float, 8) : a->hd == 128 ? LG_HEADS(float, 16) : LG_HEADS(float, 32);
+  return a->hd == 32 ? LG_HEADS(__nv_bfloat16, 4) : a->hd == 64 ? LG_HEADS(__nv_bfloat16, 8) : a->hd == 128 ? LG_HEADS(__nv_bfloat16, 16) : LG_HEADS(__nv_bfloat16, 32);
+#undef LG_HEADS
+}
+
+uint32_t logismos_launch_pool_blocks(const lg_head_norm_t* a, int32_t is_f32, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  HeadArgs p;
+  if (!head_args(a, is_f32, status, &p) || a->pool <= 0 || a->pool_rows >= a->rows) return lg::kInvalidValue;
+  const int octs = a->n_kv * a->maps * a->hd / 8;
+  const int64_t threads = (int64_t)(a->rows - a->pool_rows) * 2 * octs;
+  if (threads > 0x7fffff00) return lg::kInvalidValue;
+  const dim3 grid((unsigned)((threads + kThreads - 1) / kThreads));
+  if (is_f32) lg::launch(pool_blocks_kernel<float>, grid, dim3(kThreads), 0, (cudaStream_t)stream, p, octs);
+  else lg::launch(pool_blocks_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, (cudaStream_t)stream, p, octs);
+  return lg::launch_status();
+}
 
 uint32_t logismos_launch_qk_norm_rotary_store(void* qkv, int32_t ld, void* k_pool, void* v_pool, const void* slots, const void* positions, int32_t rows,
                                               int32_t n_heads, int32_t n_kv, int32_t head_dim, int32_t dim, const void* gain_q, const void* gain_k, float eps,

@@ -1,6 +1,6 @@
 // What the attention kernels share beyond the plain softmax: scores that are capped and biased by distance, with an
-// output gate per channel (lg_score_bias_t), and windows with kept first keys, one added to the softmax denominator and an
-// output gate per head (lg_window_t).
+// output gate per channel (lg_score_bias_t), and windows: sliding or by chunks, with kept first keys or with blocks of
+// tokens pooled behind them, one added to the softmax denominator and an output gate per head (lg_window_t).
 #pragma once
 #include <cmath>
 
@@ -31,36 +31,47 @@ struct ScoreExt {
   LG_DEVINL float gated(float o, float g) const { return o * __fdividef(gate_scale, 1.0f + __expf(-g)); }
 };
 
-// The window form: where a query at position i looks, and what becomes of its output
+// The window form: where a query at position i looks, and what becomes of its output. What stands ahead of the window, kept
+// first keys or pooled blocks, is numbered through with it: `lead` of them, then the window's keys from a place rounded down.
 struct WindowExt {
-  int size, keep, sink;          // size INT_MAX: all keys
+  int size, keep, sink, chunked, pool;   // size INT_MAX: all keys
   const float* gate;             // [rows, ld_gate], NULL: none
   int ld_gate;
   int ld_q, ld_out;
-  LG_DEVINL bool sees(int i, int j) const { return j <= i && (i - j < size || j < keep); }
+  int raw;                       // the output is fp32
+  const void *kmean, *vmean;     // pooled keys and values, mean_rows() of them per cache block
+  // first key of the window
+  __host__ __device__ int first(int i) const { return chunked ? i - i % size : i < size ? 0 : i - size + 1; }
+  LG_DEVINL bool sees(int i, int j) const { return j <= i && (j >= first(i) || j < keep); }
+  // pooled blocks that lie wholly before the window
+  __host__ __device__ int pooled(int i) const { return pool && i >= size ? (i - size + 1) / pool : 0; }
+  // a pooled block is kept with the cache block that holds its last token
+  __host__ __device__ int mean_rows() const { return (15 + pool) / pool; }
+  LG_DEVINL int mean_block(int b) const { return ((b + 1) * pool - 1) >> 4; }
+  LG_DEVINL int mean_row(int b) const { return b - (mean_block(b) << 4) / pool; }
   LG_DEVINL float head_gate(size_t row, int head) const { return gate ? 1.0f / (1.0f + __expf(-gate[row * ld_gate + head])) : 1.0f; }
+  // leading blocks of 16 for the last of `ctx` tokens, and the distance by which the blocks after them are renumbered
+  __host__ __device__ int lead_blocks(int ctx) const { return ((pool ? pooled(ctx - 1) : keep) + 15) / 16; }
+  __host__ __device__ int gap_blocks(int ctx) const {
+    const int gap = first(ctx - 1) / 16 - lead_blocks(ctx);
+    return pool || gap > 0 ? gap : 0;
+  }
+  // the same of a prompt launch's gather, for queries at the last q_len of kv_len positions: leading rows come in tiles of
+  // 128, the window of the first query begins at a multiple of 8
+  __host__ __device__ int lead_keys(int kv_len) const { return ((pool ? pooled(kv_len - 1) : keep) + 127) / 128 * 128; }
+  __host__ __device__ int gap_keys(int kv_len, int q_len) const {
+    const int gap = (first(kv_len - q_len) & ~7) - lead_keys(kv_len);
+    return pool || gap > 0 ? gap : 0;
+  }
 };
 
-// Blocks of 16 tokens between the kept ones and the first of the window, for the last of `ctx` tokens
-__host__ __device__ inline int window_gap_blocks(int ctx, int size, int keep) {
-  if (size >= ctx) return 0;
-  const int first = (ctx - size) / 16, kept = (keep + 15) / 16;
-  return first > kept ? first - kept : 0;
-}
-// Keys left out of a prompt launch's gather, for queries at the last q_len of kv_len positions: between the kept keys,
-// rounded up to tiles of 128, and the first query's window, rounded down to a multiple of 8
-__host__ __device__ inline int window_gap_keys(int kv_len, int q_len, int size, int keep) {
-  const int cached = kv_len - q_len;
-  if (cached < size) return 0;
-  const int first = (cached - size + 1) & ~7, kept = (keep + 127) / 128 * 128;
-  return first > kept ? first - kept : 0;
-}
-
 inline bool window_ok(const lg_window_t* w, int heads) {
-  return w && w->scale > 0.0f && w->size >= 0 && w->keep_first >= 0 && w->keep_first < (1 << 30) && (!w->gate || w->ld_gate >= heads);
+  return w && w->scale > 0.0f && w->size >= 0 && w->keep_first >= 0 && w->keep_first < (1 << 30) && (!w->gate || w->ld_gate >= heads) && w->pool >= 0 &&
+         (!(w->chunked || w->pool) || (w->size > 0 && !w->keep_first)) && !(w->chunked && w->pool) &&
+         (!w->pool || (w->k_mean && w->v_mean && (((uintptr_t)w->k_mean | (uintptr_t)w->v_mean) & 15) == 0));
 }
 inline WindowExt window_ext(const lg_window_t* w, int ld_q, int ld_out) {
-  return WindowExt{w->size ? w->size : 0x7fffffff, w->keep_first, w->sink, (const float*)w->gate, w->ld_gate, ld_q, ld_out};
+  return WindowExt{w->size ? w->size : 0x7fffffff, w->keep_first, w->sink, w->chunked, w->pool, (const float*)w->gate, w->ld_gate, ld_q, ld_out, w->out_f32, w->k_mean, w->v_mean};
 }
 
 inline bool score_ok(const lg_score_bias_t* s, int width) {

@@ -3,7 +3,8 @@
 // and C pass a causal depthwise convolution and silu; then per head (B, C of its group)
 //   dt <- softplus(dt + bias);  S <- exp(-exp(log_a) dt) S + dt B x^T;  y = S^T C + D x
 // and over the heads y silu(z), each of several equal parts divided by its root mean square, times a gain.
-// State, step sizes, decays, convolution sums and norms are fp32. NP and VP are powers of two with zero padding.
+// A fixed decay per head makes it linear attention over rows x | B | C = values | keys | queries, with every step of size one
+// and no skip. State, step sizes, decays, convolution sums and norms are fp32. NP and VP are powers of two with zero padding.
 // The last taps - 1 inputs of the convolution are its state: a slot holds two copies, a step reads the one its
 // phase names and writes the other.
 //
@@ -48,10 +49,11 @@ struct SsdArgs {
   int heads, groups, np, vp;
   void* xbc;               // convolved channels [rows, ld_xbc], activation format
   int ld_xbc;
+  const float* log2_decay;
   __host__ __device__ __forceinline__ int channels() const { return heads * vp + 2 * groups * np; }
 };
 
-template <typename T>
+template <typename T, bool FIXED>
 __global__ void __launch_bounds__(kThreads, 5)
 ssd_step_kernel(SsdArgs p, int in_smem) {
   lg::pdl_trigger();
@@ -65,11 +67,12 @@ ssd_step_kernel(SsdArgs p, int in_smem) {
   State S(smem, in_smem, p.state + ((size_t)p.state_slots[seq] * p.heads + head) * np * vp);
   S.request(t, fresh);
   const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
-  const float bias = __ldg(p.dt_bias + head), a = expf(__ldg(p.log_a + head)), skip = __ldg(p.skip + head);
+  const float bias = FIXED ? 0.0f : __ldg(p.dt_bias + head), a = FIXED ? 0.0f : expf(__ldg(p.log_a + head)), skip = FIXED ? 0.0f : __ldg(p.skip + head);
+  const float fixed = FIXED ? exp2f(__ldg(p.log2_decay + head)) : 0.0f;
   lg::pdl_wait();
   for (int tok = t0; tok < t1; ++tok) {
     const T* row = reinterpret_cast<const T*>(p.xbc) + (size_t)tok * p.ld_xbc;
-    const float dt = softplus_f(p.dt[(size_t)tok * p.ld_dt + head] + bias), decay = expf(-a * dt);
+    const float dt = FIXED ? 1.0f : softplus_f(p.dt[(size_t)tok * p.ld_dt + head] + bias), decay = FIXED ? fixed : expf(-a * dt);
     if (tid < vp) xs[tid] = Io<T>::load(row + head * vp + tid);
     if (tid < np) {
       bs[tid] = dt * Io<T>::load(row + inner + group * np + tid);
@@ -196,7 +199,7 @@ constexpr int kPitchP = kChunk * 2 + 16;
 inline size_t ssd_chunk_smem(int np, int vp) {
   return (size_t)kChunk * (2 * (2 * (2 * np + 16) + 2 * vp + 16) + 2 * kPitchP) + 4 * kChunk * 4;
 }
-template <int NP>
+template <int NP, bool FIXED>
 __global__ void __launch_bounds__(512)
 ssd_chunk_kernel(SsdArgs p) {
   lg::pdl_prologue();
@@ -213,7 +216,7 @@ ssd_chunk_kernel(SsdArgs p) {
   const __nv_bfloat16* xbc = reinterpret_cast<const __nv_bfloat16*>(p.xbc);
   const __nv_bfloat16 *xs = xbc + head * vp, *bs = xbc + inner + group * NP, *cs = bs + p.groups * NP;
   __nv_bfloat16* ys = reinterpret_cast<__nv_bfloat16*>(p.y) + head * vp;
-  const float bias = p.dt_bias[head], a2 = expf(p.log_a[head]) * 1.4426950408889634f, skip = p.skip[head];
+  const float bias = FIXED ? 0.0f : p.dt_bias[head], a2 = FIXED ? -p.log2_decay[head] : expf(p.log_a[head]) * 1.4426950408889634f, skip = FIXED ? 0.0f : p.skip[head];
   float* st = p.state + ((size_t)p.state_slots[seq] * p.heads + head) * NP * vp;
   float S[NT][4];   // state channels 16 m + g, + 8; values v0 + 2 t, + 1
 #pragma unroll
@@ -235,12 +238,12 @@ ssd_chunk_kernel(SsdArgs p) {
   float dt_raw[2] = {0.f, 0.f};
   auto fetch_dt = [&](int tb) {
 #pragma unroll
-    for (int i = 0; i < 2; ++i) dt_raw[i] = tb + lane + 32 * i < t1 ? p.dt[(size_t)(tb + lane + 32 * i) * p.ld_dt + head] : 0.0f;
+    for (int i = 0; i < 2 && !FIXED; ++i) dt_raw[i] = tb + lane + 32 * i < t1 ? p.dt[(size_t)(tb + lane + 32 * i) * p.ld_dt + head] : 0.0f;
   };
   // step sizes and log2-decays of a chunk summed up by one warp; tokens past the end take no step
   auto sum_decays = [&](int tb, int to) {
     const int n = min(kChunk, t1 - tb);
-    const float d0 = lane < n ? softplus_f(dt_raw[0] + bias) : 0.0f, d1 = lane + 32 < n ? softplus_f(dt_raw[1] + bias) : 0.0f;
+    const float d0 = lane < n ? (FIXED ? 1.0f : softplus_f(dt_raw[0] + bias)) : 0.0f, d1 = lane + 32 < n ? (FIXED ? 1.0f : softplus_f(dt_raw[1] + bias)) : 0.0f;
     float c0 = -a2 * d0, c1 = -a2 * d1;
 #pragma unroll
     for (int d = 1; d < 32; d <<= 1) {
@@ -367,8 +370,8 @@ ssd_chunk_kernel(SsdArgs p) {
 }
 
 // y silu(z), normalised in equal parts of `width` contiguous bf16 channels: a warp per (row, part), NV times eight
-// channels per lane.
-template <int NV>
+// channels per lane. AFTER: y is normalised and then multiplied by sigmoid(z).
+template <int NV, bool AFTER>
 __global__ void __launch_bounds__(256)
 gated_norm_warp_kernel(const __nv_bfloat16* __restrict__ y, int ld_y, const __nv_bfloat16* __restrict__ z, int ld_z, const float* __restrict__ gain,
                        __nv_bfloat16* __restrict__ out, int ld_out, int rows, int parts, int width, float eps) {
@@ -393,8 +396,8 @@ gated_norm_warp_kernel(const __nv_bfloat16* __restrict__ y, int ld_y, const __nv
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       const float2 fa = unpack_bf16x2(wa[k]), fb = unpack_bf16x2(wb[k]);
-      x[i][2 * k] = fa.x * silu_bf16(fb.x);
-      x[i][2 * k + 1] = fa.y * silu_bf16(fb.y);
+      x[i][2 * k] = AFTER ? fa.x : fa.x * silu_bf16(fb.x);
+      x[i][2 * k + 1] = AFTER ? fa.y : fa.y * silu_bf16(fb.y);
       ss = fmaf(x[i][2 * k], x[i][2 * k], fmaf(x[i][2 * k + 1], x[i][2 * k + 1], ss));
     }
   }
@@ -404,6 +407,15 @@ gated_norm_warp_kernel(const __nv_bfloat16* __restrict__ y, int ld_y, const __nv
     const int c = 8 * (lane + 32 * i);
     if (c >= width) continue;
     const float4 g0 = __ldg(reinterpret_cast<const float4*>(gain + c0 + c)), g1 = __ldg(reinterpret_cast<const float4*>(gain + c0 + c + 4));
+    if (AFTER) {
+      const uint32_t wb[4] = {b[i].x, b[i].y, b[i].z, b[i].w};
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 fb = unpack_bf16x2(wb[k]);
+        x[i][2 * k] *= __fdividef(1.0f, 1.0f + __expf(-fb.x));
+        x[i][2 * k + 1] *= __fdividef(1.0f, 1.0f + __expf(-fb.y));
+      }
+    }
     *reinterpret_cast<uint4*>(out + (size_t)r * ld_out + c0 + c) =
         make_uint4(pack_bf16x2(x[i][0] * inv * g0.x, x[i][1] * inv * g0.y), pack_bf16x2(x[i][2] * inv * g0.z, x[i][3] * inv * g0.w),
                    pack_bf16x2(x[i][4] * inv * g1.x, x[i][5] * inv * g1.y), pack_bf16x2(x[i][6] * inv * g1.z, x[i][7] * inv * g1.w));
@@ -412,7 +424,7 @@ gated_norm_warp_kernel(const __nv_bfloat16* __restrict__ y, int ld_y, const __nv
 
 // The same for any width and format, a CTA per (row, part). VEC: channels are contiguous (no
 // padding between heads) and eight of them are moved at once.
-template <typename T, bool VEC>
+template <typename T, bool VEC, bool AFTER>
 __global__ void __launch_bounds__(512)
 gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__ z, int ld_z, const float* __restrict__ gain, T* __restrict__ out,
                         int ld_out, int width, int v, int vp, float eps) {
@@ -423,7 +435,7 @@ gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__
   T* o = out + (size_t)r * ld_out;
   if constexpr (VEC) {
     constexpr int kMax = 4;  // width <= 4 * 8 * 512
-    float x[kMax][8];
+    float x[kMax][8], after[AFTER ? kMax : 1][8];
     float ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < kMax; ++i) {
@@ -443,7 +455,11 @@ gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__
         for (int k = 0; k < 8; ++k) { a[k] = yr[c0 + c + k]; g[k] = zr[c0 + c + k]; }
       }
 #pragma unroll
-      for (int k = 0; k < 8; ++k) { x[i][k] = a[k] * (sizeof(T) == 2 ? __fdividef(g[k], 1.0f + __expf(-g[k])) : silu_f(g[k])); ss += x[i][k] * x[i][k]; }
+      for (int k = 0; k < 8; ++k) {
+        x[i][k] = AFTER ? a[k] : a[k] * (sizeof(T) == 2 ? __fdividef(g[k], 1.0f + __expf(-g[k])) : silu_f(g[k]));
+        if (AFTER) after[AFTER ? i : 0][k] = sigmoid_f(g[k]);
+        ss += x[i][k] * x[i][k];
+      }
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
 #pragma unroll
@@ -451,7 +467,9 @@ gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__
       const int c = 8 * (threadIdx.x + i * blockDim.x);
       if (c >= width) break;
       const float4 g0 = __ldg(reinterpret_cast<const float4*>(gain + c0 + c)), g1 = __ldg(reinterpret_cast<const float4*>(gain + c0 + c + 4));
-      const float w[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+      float w[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+#pragma unroll
+      for (int k = 0; k < 8 && AFTER; ++k) w[k] *= after[AFTER ? i : 0][k];
       if constexpr (sizeof(T) == 2) {
         uint32_t u[4];
 #pragma unroll
@@ -466,13 +484,14 @@ gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__
     auto col = [&](int c) { const int ch = c0 + c; return (ch / v) * vp + ch % v; };
     float ss = 0.0f;
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
-      const float x = Io<T>::load(yr + col(c)) * silu_f(Io<T>::load(zr + col(c)));
+      const float x = Io<T>::load(yr + col(c)) * (AFTER ? 1.0f : silu_f(Io<T>::load(zr + col(c))));
       ss += x * x;
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
       const int k = col(c);
-      Io<T>::store(o + k, Io<T>::load(yr + k) * silu_f(Io<T>::load(zr + k)) * inv * gain[k]);
+      const float g = Io<T>::load(zr + k);
+      Io<T>::store(o + k, Io<T>::load(yr + k) * (AFTER ? sigmoid_f(g) : silu_f(g)) * inv * gain[k]);
     }
   }
 }
@@ -480,6 +499,9 @@ gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__
 bool pow2(int v, int lo, int hi) { return v >= lo && v <= hi && (v & (v - 1)) == 0; }
 
 bool args_ok(const lg_ssd_t* a, int n_seqs) {
+  if (a && a->log2_decay)
+    return n_seqs > 0 && n_seqs <= 65535 && a->xbc && a->state && a->state_slots && a->fresh && a->cu && a->y && a->heads > 0 && a->groups == a->heads && pow2(a->np, 16, 256) &&
+           pow2(a->vp, 16, 256) && a->ld_y >= a->heads * a->vp;
   return a && n_seqs > 0 && n_seqs <= 65535 && a->proj && a->dt && a->conv_w && a->conv_b && a->dt_bias && a->log_a && a->skip && a->state && a->state_slots &&
          a->fresh && a->phase && a->cu && a->y && a->taps >= 1 && a->taps <= kMaxTaps && (a->taps == 1 || a->conv_state) && a->heads > 0 && a->groups > 0 &&
          a->heads % a->groups == 0 && pow2(a->np, 16, 256) && pow2(a->vp, 16, 256) && a->ld >= 2 * a->heads * a->vp + 2 * a->groups * a->np &&
@@ -489,7 +511,36 @@ bool args_ok(const lg_ssd_t* a, int n_seqs) {
 SsdArgs make_args(const lg_ssd_t* a) {
   return SsdArgs{a->proj, a->ld, (const float*)a->dt, a->ld_dt, (const float*)a->conv_w, (const float*)a->conv_b, (float*)a->conv_state, a->taps,
                  (const float*)a->dt_bias, (const float*)a->log_a, (const float*)a->skip, (float*)a->state, (const int*)a->state_slots,
-                 (const uint8_t*)a->fresh, (const uint8_t*)a->phase, (const int*)a->cu, a->y, a->ld_y, a->heads, a->groups, a->np, a->vp, a->xbc, a->ld_xbc};
+                 (const uint8_t*)a->fresh, (const uint8_t*)a->phase, (const int*)a->cu, a->y, a->ld_y, a->heads, a->groups, a->np, a->vp, a->xbc, a->ld_xbc, (const float*)a->log2_decay};
+}
+
+template <bool AFTER>
+uint32_t launch_gated_norm(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32, void* out, int32_t ld_out, int32_t is_f32,
+                           int32_t rows, int32_t heads, int32_t v, int32_t vp, int32_t parts, float eps, void* stream) {
+  if (!y || !z || !gain_f32 || !out || rows <= 0 || heads <= 0 || v <= 0 || vp < v || parts <= 0 || parts > 65535 || (heads * v) % parts || ld_y < heads * vp ||
+      ld_z < heads * vp || ld_out < heads * vp)
+    return lg::kInvalidValue;
+  const int width = heads * v / parts;
+  const bool vec = v == vp && width % 8 == 0 && width <= 4 * 8 * 512 && ld_y % 8 == 0 && ld_z % 8 == 0 && ld_out % 8 == 0;
+  int threads = ((vec ? width / 8 : width) + 31) / 32 * 32;
+  if (threads > 512) threads = 512;
+  if (!is_f32 && vec && width <= 2048) {
+    auto warp = [&](auto kern) {
+      lg::launch(kern, dim3((unsigned)(((int64_t)rows * parts + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, (const __nv_bfloat16*)y, ld_y, (const __nv_bfloat16*)z, ld_z,
+                 (const float*)gain_f32, (__nv_bfloat16*)out, ld_out, rows, parts, width, eps);
+      return lg::launch_status();
+    };
+    return width <= 256 ? warp(gated_norm_warp_kernel<1, AFTER>) : width <= 512 ? warp(gated_norm_warp_kernel<2, AFTER>) : width <= 1024 ? warp(gated_norm_warp_kernel<4, AFTER>)
+                                                                                                           : warp(gated_norm_warp_kernel<8, AFTER>);
+  }
+  const dim3 grid((unsigned)rows, (unsigned)parts);
+  auto go = [&](auto kern, auto* t) {
+    using T = std::remove_pointer_t<decltype(t)>;
+    lg::launch(kern, grid, dim3((unsigned)threads), 0, (cudaStream_t)stream, (const T*)y, ld_y, (const T*)z, ld_z, (const float*)gain_f32, (T*)out, ld_out, width, v, vp, eps);
+    return lg::launch_status();
+  };
+  if (is_f32) return vec ? go(gated_group_norm_kernel<float, true, AFTER>, (float*)nullptr) : go(gated_group_norm_kernel<float, false, AFTER>, (float*)nullptr);
+  return vec ? go(gated_group_norm_kernel<__nv_bfloat16, true, AFTER>, (__nv_bfloat16*)nullptr) : go(gated_group_norm_kernel<__nv_bfloat16, false, AFTER>, (__nv_bfloat16*)nullptr);
 }
 
 }  // namespace
@@ -508,14 +559,15 @@ uint32_t logismos_launch_ssd_step(const lg_ssd_t* a, int32_t n_seqs, int32_t is_
     lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3(kThreads), smem, (cudaStream_t)stream, p, smem > 0 ? 1 : 0);
     return lg::launch_status();
   };
-  return is_f32 ? go(ssd_step_kernel<float>) : go(ssd_step_kernel<__nv_bfloat16>);
+  if (p.log2_decay) return is_f32 ? go(ssd_step_kernel<float, true>) : go(ssd_step_kernel<__nv_bfloat16, true>);
+  return is_f32 ? go(ssd_step_kernel<float, false>) : go(ssd_step_kernel<__nv_bfloat16, false>);
 }
 
 int32_t logismos_ssd_has_chunked(int32_t np, int32_t vp) { return pow2(np, 32, 128) && pow2(vp, 16, 128) ? 1 : 0; }
 
 uint32_t logismos_launch_ssd_conv(const lg_ssd_t* a, const void* seq_ids_i32, int32_t row0, int32_t rows, int32_t single, int32_t is_f32, void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!args_ok(a, 1) || !seq_ids_i32 || row0 < 0 || rows <= row0 || !a->xbc || a->ld % 4 || a->ld_xbc % 4 || a->ld_xbc < make_args(a).channels()) return lg::kInvalidValue;
+  if (!args_ok(a, 1) || a->log2_decay || !seq_ids_i32 || row0 < 0 || rows <= row0 || !a->xbc || a->ld % 4 || a->ld_xbc % 4 || a->ld_xbc < make_args(a).channels()) return lg::kInvalidValue;
   const SsdArgs p = make_args(a);
   const int* ids = (const int*)seq_ids_i32;
   cudaStream_t s = (cudaStream_t)stream;
@@ -535,37 +587,21 @@ uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* a, int32_t n_seqs, voi
     lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3((unsigned)(4 * p.vp)), smem, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
-  return a->np == 32 ? go(ssd_chunk_kernel<32>) : a->np == 64 ? go(ssd_chunk_kernel<64>) : go(ssd_chunk_kernel<128>);
+  if (p.log2_decay) return a->np == 32 ? go(ssd_chunk_kernel<32, true>) : a->np == 64 ? go(ssd_chunk_kernel<64, true>) : go(ssd_chunk_kernel<128, true>);
+  return a->np == 32 ? go(ssd_chunk_kernel<32, false>) : a->np == 64 ? go(ssd_chunk_kernel<64, false>) : go(ssd_chunk_kernel<128, false>);
 }
 
 uint32_t logismos_launch_gated_group_norm(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32, void* out, int32_t ld_out,
                                           int32_t is_f32, int32_t rows, int32_t heads, int32_t v, int32_t vp, int32_t parts, float eps,
                                           void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!y || !z || !gain_f32 || !out || rows <= 0 || heads <= 0 || v <= 0 || vp < v || parts <= 0 || parts > 65535 || (heads * v) % parts || ld_y < heads * vp ||
-      ld_z < heads * vp || ld_out < heads * vp)
-    return lg::kInvalidValue;
-  const int width = heads * v / parts;
-  const bool vec = v == vp && width % 8 == 0 && width <= 4 * 8 * 512 && ld_y % 8 == 0 && ld_z % 8 == 0 && ld_out % 8 == 0;
-  int threads = ((vec ? width / 8 : width) + 31) / 32 * 32;
-  if (threads > 512) threads = 512;
-  if (!is_f32 && vec && width <= 2048) {
-    auto warp = [&](auto kern) {
-      lg::launch(kern, dim3((unsigned)(((int64_t)rows * parts + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, (const __nv_bfloat16*)y, ld_y, (const __nv_bfloat16*)z, ld_z,
-                 (const float*)gain_f32, (__nv_bfloat16*)out, ld_out, rows, parts, width, eps);
-      return lg::launch_status();
-    };
-    return width <= 256 ? warp(gated_norm_warp_kernel<1>) : width <= 512 ? warp(gated_norm_warp_kernel<2>) : width <= 1024 ? warp(gated_norm_warp_kernel<4>)
-                                                                                                           : warp(gated_norm_warp_kernel<8>);
-  }
-  const dim3 grid((unsigned)rows, (unsigned)parts);
-  auto go = [&](auto kern, auto* t) {
-    using T = std::remove_pointer_t<decltype(t)>;
-    lg::launch(kern, grid, dim3((unsigned)threads), 0, (cudaStream_t)stream, (const T*)y, ld_y, (const T*)z, ld_z, (const float*)gain_f32, (T*)out, ld_out, width, v, vp, eps);
-    return lg::launch_status();
-  };
-  if (is_f32) return vec ? go(gated_group_norm_kernel<float, true>, (float*)nullptr) : go(gated_group_norm_kernel<float, false>, (float*)nullptr);
-  return vec ? go(gated_group_norm_kernel<__nv_bfloat16, true>, (__nv_bfloat16*)nullptr) : go(gated_group_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16*)nullptr);
+  return launch_gated_norm<false>(y, ld_y, z, ld_z, gain_f32, out, ld_out, is_f32, rows, heads, v, vp, parts, eps, stream);
+}
+
+uint32_t logismos_launch_norm_gate(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32, void* out, int32_t ld_out, int32_t is_f32,
+                                   int32_t rows, int32_t heads, int32_t v, int32_t vp, float eps, void* stream) {
+  lg::LaunchScope launch_scope_;
+  return launch_gated_norm<true>(y, ld_y, z, ld_z, gain_f32, out, ld_out, is_f32, rows, heads, v, vp, 1, eps, stream);
 }
 
 }  // extern "C"

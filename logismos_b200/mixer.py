@@ -1,6 +1,6 @@
 """Decoders over a stack of mixers and feed-forwards of several kinds, over the C ABI (``lg_mixer_*``): weights and the
 packed continuous-batching step, and the configuration of the post-norm stack of state-space layers and parallel layers,
-attention beside time mixing (Katadra; ``vugedra`` has the other design's). The contract is that of the other executors:
+attention beside time mixing (Katadra; ``vugedra`` and ``zetalorn`` have the other designs'). The contract is that of the other executors:
 a packed step equals running every sequence alone."""
 from __future__ import annotations
 
@@ -12,9 +12,10 @@ from ._lib import lib
 from .executor import SlotExecutor, bits_pointer
 
 _vp = C.c_void_p
-SSD, PARALLEL, ATTENTION, GLA, LATENT = range(5)
+SSD, PARALLEL, ATTENTION, GLA, LATENT, DIFF, PAIR = range(7)
 RELU2, GATED, MIXTURE = range(3)            # feed-forwards
-POST_LAYER_NORM, TANH_AROUND = range(2)     # norms of the stack
+POST_LAYER_NORM, TANH_AROUND, RMS_GATED = range(3)     # norms of the stack
+SOFTMAX, SIGMOID = range(2)                 # scores of a router
 KINDS = {"mamba2": SSD, "parallel": PARALLEL}
 
 _INT_A = ("kind", "weights_of", "ff", "ssd_heads", "ssd_vdim", "ssd_state", "ssd_groups", "ssd_norm_groups", "ssd_taps", "heads", "kv_heads", "dim", "vdim",
@@ -24,17 +25,24 @@ _INT_B = ("tm_heads", "tm_dim", "tm_rank")
 _FLOAT_B = ("left_scale", "right_scale")
 _INT_C = ("ff_kind", "experts", "identity", "top", "shared_ff", "window", "keep_first", "q_rank", "kv_rank", "rot_dims")
 _DOUBLE_C = ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")
+_INT_D = ("rot_halves", "chunked", "pool")
+_INT_E = ("lin_heads", "lin_dim", "lin_vdim")
+_FLOAT_E = ("glu_alpha", "glu_limit", "glu_shift")
+_INT_F = ("scoring", "route_groups", "keep_groups", "no_correction", "file_layer", "pass")
 
 
 class _LayerCfg(C.Structure):
     _fields_ = [(n, C.c_int32) for n in _INT_A] + [(n, C.c_float) for n in _FLOAT_A] + [(n, C.c_int32) for n in _INT_B] + [(n, C.c_float) for n in _FLOAT_B] + [
-        (n, C.c_int32) for n in _INT_C] + [("tau", C.c_float)] + [(n, C.c_double) for n in _DOUBLE_C]
+        (n, C.c_int32) for n in _INT_C] + [("tau", C.c_float)] + [(n, C.c_double) for n in _DOUBLE_C] + [(n, C.c_int32) for n in _INT_D] + [
+        ("diff", C.c_float)] + [(n, C.c_int32) for n in _INT_E] + [("decay", C.POINTER(C.c_double))] + [(n, C.c_float) for n in _FLOAT_E] + [
+        (n, C.c_int32) for n in _INT_F]
 
 
 class _Cfg(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "n_layers")] + [("norm_eps", C.c_float)] + [
         (n, C.c_int32) for n in ("is_f32", "n_pool_blocks", "max_blocks_per_seq", "max_step_tokens", "max_step_seqs", "n_state_slots", "max_out_rows",
-                                 "keep_layers")] + [("layers", C.POINTER(_LayerCfg)), ("norm", C.c_int32)]
+                                 "keep_layers")] + [("layers", C.POINTER(_LayerCfg)), ("norm", C.c_int32), ("passes", C.c_int32),
+                                                                                  ("logit_scale", C.c_float)]
 
 
 MIXES = "rkvgw"   # order of the token-shift mixes
@@ -45,14 +53,16 @@ _RIGHT = tuple("right_" + n for n in ("r", "k", "v", "g", "w1", "w2", "w0", "u",
 _TANH = tuple(n + s for n in ("norm1", "norm1b", "norm2", "norm2b") for s in ("", "_b", "_alpha") if n + s not in _COMMON)
 _GATED = ("q", "q_b", "q_norm", "k", "k_b", "k_norm", "v", "v_b", "g", "a1", "a2", "a2_b", "dq", "dq_norm", "uq", "dkv", "dkv_norm", "uk", "uv",
           "gate", "router", "correction", "shared_gate", "shared_up", "shared_down")
+_PAIRED = ("rg1", "rg1_b", "rg2", "rg2_b", "lq1", "lk1", "lq2", "lk2", "left_q_norm", "left_k_norm", "left_out", "right_q", "right_out")
 
 
 class _LayerW(C.Structure):
-    _fields_ = [(n, _vp) for n in _COMMON + _SSD + _LEFT] + [("mu", _vp * len(MIXES))] + [(n, _vp) for n in _RIGHT + _TANH + _GATED] + [("experts", C.POINTER(_vp))]
+    _fields_ = [(n, _vp) for n in _COMMON + _SSD + _LEFT] + [("mu", _vp * len(MIXES))] + [(n, _vp) for n in _RIGHT + _TANH + _GATED] + [("experts", C.POINTER(_vp))] + [
+        (n, _vp) for n in _PAIRED]
 
 
 class _Weights(C.Structure):
-    _fields_ = [(n, _vp) for n in ("embed", "final_norm", "final_norm_b", "head")] + [("layers", C.POINTER(_LayerW)), ("final_norm_alpha", _vp)]
+    _fields_ = [(n, _vp) for n in ("embed", "final_norm", "final_norm_b", "head")] + [("layers", C.POINTER(_LayerW)), ("final_norm_alpha", _vp), ("loop_step", _vp)]
 
 
 def _ssd(m: dict) -> dict:
@@ -106,7 +116,7 @@ def parse_config(config: dict) -> dict:
 
 class MixerModel(SlotExecutor):
     """``weights``: dict of bf16 bit patterns (uint16 arrays) embed, final_norm, final_norm_b, head (tanh norms: also
-    final_norm_alpha) and ``layers``: per layer a dict (empty for a layer that uses another's tensors) with the tensors of
+    final_norm_alpha; a gated RMS stack: no final_norm_b, with repeated layers loop_step) and ``layers``: per layer a dict (empty for a layer that uses another's tensors) with the tensors of
     lg_mixer_layer_weights_t that its kind has, by name; ``mu`` is a list of five arrays in the order r, k, v, g, w and
     ``experts`` one of gate, up, down of every expert. ``dtype`` "bfloat16" serves, "float32" computes everything in fp32.
     With ``keep_layers`` ``snapshot(j)`` is the stream before layer j."""
@@ -122,7 +132,9 @@ class MixerModel(SlotExecutor):
         n = cfg["n_layers"]
         lc = (_LayerCfg * max(1, n))()
         for i, y in enumerate(cfg["layers"]):
-            lc[i] = _LayerCfg(**y)
+            lc[i] = _LayerCfg(**{k: v for k, v in y.items() if k != "decay"})
+            if y.get("decay"):
+                lc[i].decay = (C.c_double * len(y["decay"]))(*y["decay"])
             if weights is not None and weights["layers"][i]:
                 w = weights["layers"][i]
                 if y["kind"] == PARALLEL:
@@ -130,7 +142,7 @@ class MixerModel(SlotExecutor):
                 elif y["kind"] == GLA:
                     lc[i].tm_rank = w["a1"].shape[0]
         c = _Cfg(cfg["vocab"], cfg["hidden"], n, cfg["norm_eps"], int(dtype == "float32"), n_pool_blocks, max_blocks_per_seq, max_step_tokens, max_step_seqs,
-                 n_state_slots, max(max_out_rows, max_step_seqs), int(keep_layers), lc, cfg.get("norm", POST_LAYER_NORM))
+                 n_state_slots, max(max_out_rows, max_step_seqs), int(keep_layers), lc, cfg.get("norm", POST_LAYER_NORM), cfg.get("passes", 0), cfg.get("logit_scale", 1.0))
         h = _vp()
         if path is not None:
             rc = lib.lg_mixer_load(device, str(path).encode(), C.byref(c), C.byref(h))
@@ -145,9 +157,10 @@ class MixerModel(SlotExecutor):
                         lw[i].experts = C.cast(keep[-1], C.POINTER(_vp))
                     else:
                         setattr(lw[i], name, bits_pointer(value))
-            w = _Weights(*[bits_pointer(weights[k]) for k in ("embed", "final_norm", "final_norm_b", "head")], lw)
-            if "final_norm_alpha" in weights:
-                w.final_norm_alpha = bits_pointer(weights["final_norm_alpha"])
+            w = _Weights(layers=lw)
+            for k in ("embed", "final_norm", "final_norm_b", "final_norm_alpha", "head", "loop_step"):
+                if k in weights:
+                    setattr(w, k, bits_pointer(weights[k]))
             rc = lib.lg_mixer_create(device, C.byref(c), C.byref(w), C.byref(h))
         self._adopt(rc, h, cfg, max_blocks_per_seq, max_step_tokens, max_step_seqs, device, dtype)
 

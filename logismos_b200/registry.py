@@ -76,6 +76,12 @@ def _vugedra(folder: str, config: dict, limits: Limits, dtype: str, device: int)
                              device=device, dtype=dtype, max_out_rows=limits.max_out_rows)
 
 
+def _zetalorn(folder: str, config: dict, limits: Limits, dtype: str, device: int):
+    from .zetalorn import ZetalornModel
+    return ZetalornModel.load(folder, config, limits.pool_blocks, limits.pool_blocks, limits.step_tokens, limits.max_seqs, limits.max_seqs,
+                              device=device, dtype=dtype, max_out_rows=limits.max_out_rows)
+
+
 def _qwen2(folder: str, config: dict, limits: Limits, dtype: str, device: int):
     from .decoder import DecoderModel
     cfg = dict(vocab=config["vocab_size"], hidden=config["hidden_size"], n_layers=config["num_hidden_layers"],
@@ -97,6 +103,7 @@ REGISTRY: Dict[str, Entry] = {
     "Vofosun": Entry(_vofosun, ("bfloat16", "float32"), True, "latent"),
     "Katadra": Entry(_katadra, ("bfloat16", "float32"), True, "mixer"),
     "Vugedra": Entry(_vugedra, ("bfloat16", "float32"), True, "mixer"),
+    "Zetalorn": Entry(_zetalorn, ("bfloat16", "float32"), True, "mixer"),
     "Qwen2ForCausalLM": Entry(_qwen2, ("bfloat16",), False, None),   # int4 weights, bf16 activations
 }
 

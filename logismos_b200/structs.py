@@ -13,7 +13,8 @@ def _pointers(*names):
 
 
 class Groups(C.Structure):
-    _fields_ = [("n_groups", i32), ("end", i32 * 8), ("n_main", i32), ("tail", vp), ("ld_tail", i32), ("tail_cap", f32), ("tail_parts", vp), ("bias", vp)]
+    _fields_ = [("n_groups", i32), ("end", i32 * 8), ("n_main", i32), ("tail", vp), ("ld_tail", i32), ("tail_cap", f32), ("tail_parts", vp), ("bias", vp),
+                ("silu_begin", i32), ("silu_end", i32)]
 
 
 class TimeMix(C.Structure):
@@ -24,7 +25,7 @@ class TimeMix(C.Structure):
 
 class Ssd(C.Structure):
     _fields_ = [("proj", vp), ("ld", i32), ("dt", vp), ("ld_dt", i32)] + _pointers("conv_w", "conv_b", "conv_state") + _ints("taps") + _pointers(
-               "dt_bias", "log_a", "skip", "state", "state_slots", "fresh", "phase", "cu", "y") + _ints("ld_y", "heads", "groups", "np", "vp") + [("xbc", vp), ("ld_xbc", i32)]
+               "dt_bias", "log_a", "skip", "state", "state_slots", "fresh", "phase", "cu", "y") + _ints("ld_y", "heads", "groups", "np", "vp") + [("xbc", vp), ("ld_xbc", i32), ("log2_decay", vp)]
 
 
 class ScoreBias(C.Structure):
@@ -32,7 +33,7 @@ class ScoreBias(C.Structure):
 
 
 class Window(C.Structure):
-    _fields_ = [("scale", f32)] + _ints("size", "keep_first", "sink") + [("gate", vp), ("ld_gate", i32)]
+    _fields_ = [("scale", f32)] + _ints("size", "keep_first", "sink") + [("gate", vp), ("ld_gate", i32)] + _ints("chunked", "pool") + _pointers("k_mean", "v_mean") + [("out_f32", i32)]
 
 
 class LatentRotary(C.Structure):
@@ -49,4 +50,15 @@ class MixtureOut(C.Structure):
 
 class MoeRoute(C.Structure):
     _fields_ = [("logits", vp)] + _ints("ld", "zero_logits") + [("correction", vp)] + _ints("n_experts", "n_identity", "top", "n_always") + _pointers(
-               "weights", "pair_row", "identity", "offsets", "row_token", "counts", "pair_expert", "tiles", "n_tiles", "h", "w") + [("width", i32), ("arrived", vp)]
+               "weights", "pair_row", "identity", "offsets", "row_token", "counts", "pair_expert", "tiles", "n_tiles", "h", "w") + [("width", i32), ("arrived", vp)] + _ints("scoring", "groups", "keep_groups")
+
+
+class HeadNorm(C.Structure):
+    _fields_ = [("qkv", vp)] + _ints("ld", "rows", "heads", "n_kv", "maps", "hd", "dim") + _pointers("gain_q", "gain_k") + [("eps", f32), ("table", vp), ("rot_dims", i32),
+               ("q_out", vp), ("ld_q", i32)] + _pointers("k_pool", "v_pool", "slots", "positions") + [("n_pool_slots", C.c_int64)] + _ints("pool", "pool_rows") + _pointers(
+               "k_mean", "v_mean", "tables", "seq_ids") + _ints("max_blocks", "n_pool_blocks")
+
+
+class GatedResidual(C.Structure):
+    _fields_ = [("x", vp), ("branch", vp * 2), ("zero_branches", i32), ("branch_gain", vp * 2), ("mixture", C.POINTER(MixtureOut)), ("gate", vp), ("ld_gate", i32)] + _pointers(
+               "kept", "embed", "ids", "step") + [("vocab", i32), ("h", vp), ("gain", f32), ("eps", f32), ("row_idx", vp)] + _ints("n_src_rows", "rows", "n", "ld", "is_f32")

@@ -426,8 +426,8 @@ def test_mixture_of_experts(E, I, top, always, F, H, tokens, form):
             check(lib.logismos_launch_linear_experts_f32(P(mid), P(keep[3]), P(rows), P(off), P(None), G, tokens, H, F, F, H, 3, 0.0, 0.0, 0.0, stream()), "down")
         else:
             expected = -(-tokens * top // E)
-            check(lib.logismos_launch_linear_experts_small_bf16(P(hd), P(keep[2]), P(mid), P(off), P(tok), G, tokens, expected, 2 * F, H, H, F, 2, stream()), "up")
-            check(lib.logismos_launch_linear_experts_small_bf16(P(mid), P(keep[3]), P(rows), P(off), P(None), G, tokens, expected, H, F, F, H, 0, stream()), "down")
+            check(lib.logismos_launch_linear_experts_small_bf16(P(hd), P(keep[2]), P(mid), P(off), P(tok), G, tokens, expected, 2 * F, H, H, F, 2, 0, 0, 0, stream()), "up")
+            check(lib.logismos_launch_linear_experts_small_bf16(P(mid), P(keep[3]), P(rows), P(off), P(None), G, tokens, expected, H, F, F, H, 0, 0, 0, 0, stream()), "down")
         o = off.cpu().numpy()
         assert o[0] == 0 and (np.diff(o) >= 0).all() and (np.diff(o)[E:] == tokens).all()
     else:
@@ -438,8 +438,8 @@ def test_mixture_of_experts(E, I, top, always, F, H, tokens, form):
         check(lib.logismos_launch_moe_place(C.byref(r), P(hd), P(gat), H, tokens, stream()), "place")
         direct = always > 0
         check(lib.logismos_launch_linear_experts_tc_bf16(P(gat), tokens * pairs, P(hd if direct else None), tokens if direct else 0, P(keep[2]), P(mid), P(tiles), P(nt), mt, G, 2 * F,
-                                                         H, H, F, 2, P(st), stream()), "up")
-        check(lib.logismos_launch_linear_experts_tc_bf16(P(mid), tokens * pairs, P(None), 0, P(keep[3]), P(rows), P(tiles), P(nt), mt, G, H, F, F, H, 0, P(st), stream()), "down")
+                                                         H, H, F, 2, 0, 0, 0, P(st), stream()), "up")
+        check(lib.logismos_launch_linear_experts_tc_bf16(P(mid), tokens * pairs, P(None), 0, P(keep[3]), P(rows), P(tiles), P(nt), mt, G, H, F, F, H, 0, 0, 0, 0, P(st), stream()), "down")
         assert nt.item() <= mt
     torch.cuda.synchronize()
     assert st.item() == 0
