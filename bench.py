@@ -10,7 +10,7 @@ every rank holds a full replica and its own batch (request sharding, no collecti
 
   python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference] [--layers L]
   python bench.py --workload ragged_step                    (continuous-batching step of the int4 decoder)
-  python bench.py --workload latent | mixer [--sizes A,B --kernels]   (bf16 decoders beside an int4 one of equal size)
+  python bench.py --workload latent | mixer | vugedra | zetalorn [--sizes A,B --kernels]   (bf16 decoders beside another one of equal size)
   python bench.py --workload serving_sweep [--requests R --max-seqs S --arrival-rate L --tp T]
                                                             (hybrid decoder under the host scheduler)
 
@@ -633,9 +633,9 @@ def main():
     ap.add_argument("--no-cpu", action="store_true")
     ap.add_argument("--no-extra", action="store_true", help="skip the decode workloads of the default line")
     ap.add_argument("--ref-budget", type=float, default=150.0, help="--impl reference: seconds of timed CPU work (each step is a full batch)")
-    ap.add_argument("--workload", default="stella", choices=["stella", "ragged_step", "serving_sweep", "latent", "mixer", "vugedra"])
-    ap.add_argument("--sizes", default="", help="latent, mixer, vugedra: comma-separated sizes of the workload's SIZES (default all)")
-    ap.add_argument("--kernels", action="store_true", help="latent, mixer, vugedra: also every kernel against its roofline, per size")
+    ap.add_argument("--workload", default="stella", choices=["stella", "ragged_step", "serving_sweep", "latent", "mixer", "vugedra", "zetalorn"])
+    ap.add_argument("--sizes", default="", help="latent, mixer, vugedra, zetalorn: comma-separated sizes of the workload's SIZES (default all)")
+    ap.add_argument("--kernels", action="store_true", help="latent, mixer, vugedra, zetalorn: also every kernel against its roofline, per size")
     ap.add_argument("--requests", type=int, default=96, help="serving_sweep: requests per GPU")
     ap.add_argument("--extra-requests", type=int, default=64, help="requests per GPU of the serving sample inside the default line")
     ap.add_argument("--max-seqs", type=int, default=256, help="serving_sweep: concurrent sequences per GPU")
@@ -717,6 +717,22 @@ def main():
                 "clocks": clocks, "sizes": rows}
         if args.kernels:
             line["kernels"] = {n: bench_vugedra.kernel_table(bench_vugedra.SIZES[n], peaks) for n in sizes}
+        print(json.dumps(line))
+    elif args.workload == "zetalorn":
+        import bench_zetalorn
+        if world > 1:
+            raise SystemExit("--workload zetalorn runs on one GPU")
+        peaks, sizes = measured_peaks(), [n for n in args.sizes.split(",") if n] or list(bench_zetalorn.SIZES)
+        sampler = ClockSampler(local)
+        sampler.start()
+        rows = bench_zetalorn.measure(sizes, args.steps, peaks)
+        clocks = sampler.stop()
+        line = {"metric": "zetalorn_decoder_tokens_per_s", "value": rows[0]["zetalorn"]["prefill"]["tokens_per_s"], "unit": "tokens/s (prefill of the first size)", "n_gpus": 1,
+                "steps": args.steps, "warmup": 3, "higher_is_better": True, "vs_baseline": None, "dtype": "bf16 weights and activations",
+                "data": "synthetic", "config": {"workload": "Zetalorn decoder beside the Vugedra decoder at equal width, depth and attention heads", "sizes": sizes},
+                "clocks": clocks, "sizes": rows}
+        if args.kernels:
+            line["kernels"] = {n: bench_zetalorn.kernel_table(bench_zetalorn.SIZES[n], peaks) for n in sizes}
         print(json.dumps(line))
     elif args.workload == "ragged_step":
         line = ragged_step_measure(R, steps=args.steps, warmup=args.warmup, layers=args.layers)

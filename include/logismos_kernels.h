@@ -1042,6 +1042,17 @@ uint32_t logismos_launch_attention_difference(const void* a_f32, int32_t ld_a, v
                                               int32_t rows, int32_t heads, int32_t n_kv, int32_t v, int32_t vp,
                                               float lambda, float scale, float eps, void* stream);
 
+/* Decode rows of differential attention: queries as logismos_launch_head_norm_store leaves them (2 * heads of head_dim), the
+ * window's attention for both maps, and the difference above where their chunks are merged; out bf16 [n_seqs, ld_out], head h
+ * at h * head_dim. Otherwise as logismos_launch_window_attention_decode_bf16, scratch for 2 * heads. */
+uint32_t logismos_launch_differential_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool,
+                                                  const void* block_tables, const void* context_lens,
+                                                  const void* chunk_offsets, void* out, int32_t ld_out, void* scratch,
+                                                  int32_t n_seqs, int32_t total_chunks, int32_t chunk_tokens,
+                                                  int32_t max_blocks, int32_t n_pool_blocks, int32_t heads,
+                                                  int32_t n_kv_heads, int32_t head_dim, const lg_window_t* window, int32_t v,
+                                                  float lambda, float scale, float eps, void* status_i32, void* stream);
+
 /* Residual stream with RMS norms of one gain and gated sublayers, one launch between two sublayers:
  *   y = branch[0] (one branch), half the sum of both, each divided by its root mean square, times its gain, or a mixture
  *   x += y sigmoid(gate);   kept = x;   x += embed[ids] + step;   h = x / rms(x) * gain

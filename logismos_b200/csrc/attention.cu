@@ -324,6 +324,8 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
   const int head0 = kvh * (n_heads / n_kv) + r_base;
   int64_t q_stride = (int64_t)n_heads * HD;
   if constexpr (EXT) q_stride = ext.ld_q;
+  bool partial = false;   // the result is left to a merge whatever the number of chunks
+  if constexpr (MODE == kWindowed) partial = ext.raw == kRawPartial;
   constexpr int D = HD, kRowBytes = HD * 2, DT = HD / 8, CH = HD / 8;
   constexpr int kDecStageBytes = DecCfg<HD, kDecWarps, kDecStages>::kStageBytes;
   const int row_elems = n_kv * D;
@@ -544,7 +546,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
       float acc = 0.0f;
 #pragma unroll
       for (int w = 0; w < kDecWarps; ++w) acc += so[(w * 16 + r) * D + d] * f[w];
-      if (EXT && n_chunks == 1) {
+      if (EXT && n_chunks == 1 && !partial) {
         if constexpr (MODE == kBiased)
           out[(int64_t)seq * ext.ld_out + head * D + d] =
               __float2bfloat16_rn(ext.gated(acc / L, __bfloat162float(ext.gate[(int64_t)seq * ext.ld_gate + head * D + d])));
@@ -553,10 +555,10 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restri
           if (ext.raw) reinterpret_cast<float*>(out)[at] = acc / L * gate;
           else out[at] = __float2bfloat16_rn(acc / L * gate);
         }
-      } else if (n_chunks == 1) out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
+      } else if (n_chunks == 1 && !partial) out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
       else part_o[((int64_t)chunk_id * n_heads + head) * D + d] = acc;
     }
-    if (n_chunks != 1 && tid == 0) {
+    if ((n_chunks != 1 || partial) && tid == 0) {
       part_ml[((int64_t)chunk_id * n_heads + head) * 2] = M;
       part_ml[((int64_t)chunk_id * n_heads + head) * 2 + 1] = L;
     }
@@ -591,6 +593,34 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o, cons
     else out[at] = __float2bfloat16_rn(acc / L * ext.head_gate(seq, head));
   } else
     out[((int64_t)seq * n_heads + head) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
+}
+
+// The same of differential attention, for any number of chunks: the outputs of a head's two maps, which stand rep heads apart
+// in the partial results, and their difference over its root mean square. CTA = (sequence, head), thread = channel.
+__global__ void paged_decode_merge_difference_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const int* __restrict__ chunk_offsets,
+                                                     __nv_bfloat16* __restrict__ out, int ld_out, int n_heads, int rep, int D, int v, float sl2, float lambda, float scale,
+                                                     float eps) {
+  lg::pdl_prologue();
+  __shared__ float red[32];
+  const int seq = blockIdx.x, h = blockIdx.y, d = threadIdx.x, first = h / rep * 2 * rep + h % rep;
+  const int c0 = chunk_offsets[seq], c1 = chunk_offsets[seq + 1];
+  float o[2];
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const int head = first + m * rep;
+    float M = -INFINITY, L = 0.0f, acc = 0.0f;
+    for (int ck = c0; ck < c1; ++ck) M = fmaxf(M, part_ml[((int64_t)ck * n_heads + head) * 2]);
+    for (int ck = c0; ck < c1; ++ck) {
+      const float mw = part_ml[((int64_t)ck * n_heads + head) * 2];
+      const float f = (mw == -INFINITY) ? 0.0f : exp2f((mw - M) * sl2);
+      L += part_ml[((int64_t)ck * n_heads + head) * 2 + 1] * f;
+      acc += part_o[((int64_t)ck * n_heads + head) * D + d] * f;
+    }
+    o[m] = acc / L;
+  }
+  const float x = o[0] - lambda * o[1];
+  const float inv = scale / sqrtf(block_sum(x * x, red) / (float)v + eps);
+  out[(int64_t)seq * ld_out + h * D + d] = __float2bfloat16_rn(x * inv);
 }
 
 // ================================ paged KV store / gather ======================================
@@ -737,6 +767,8 @@ static uint32_t launch_ext_decode(const void* q, int32_t ld_q, const void* k_poo
   uint32_t rc = head_dim == 64 ? launch(paged_decode_kernel<64, 4, 4, MODE>, 4, DecCfg<64, 4, 4>::kSmem)
               : head_dim == 128 ? launch(paged_decode_kernel<128, 4, 2, MODE>, 4, DecCfg<128, 4, 2>::kSmem)
                                 : launch(paged_decode_kernel<256, 3, 2, MODE>, 3, DecCfg<256, 3, 2>::kSmem);
+  if constexpr (MODE == kWindowed)
+    if (ext.raw == kRawPartial) return rc;
   if (rc || total_chunks == n_seqs) return rc;
   lg::launch(paged_decode_merge_kernel<MODE>, dim3((unsigned)n_seqs, (unsigned)n_heads), dim3((unsigned)head_dim), 0, (cudaStream_t)stream, (const float*)part_o,
              (const float*)part_ml, (const int*)chunk_offsets, (__nv_bfloat16*)out, n_heads, head_dim, sl2, ext);
@@ -780,6 +812,25 @@ uint32_t logismos_launch_window_attention_decode_bf16(const void* q, int32_t ld_
   if (!window_ok(window, n_heads)) return lg::kInvalidValue;
   return launch_ext_decode<kWindowed>(q, ld_q, k_pool, v_pool, block_tables, context_lens, chunk_offsets, out, ld_out, scratch, n_seqs, total_chunks, chunk_tokens,
                                       max_blocks, n_pool_blocks, n_heads, n_kv_heads, head_dim, window->scale * kLog2e, window_ext(window, ld_q, ld_out), status, stream);
+}
+
+uint32_t logismos_launch_differential_decode_bf16(const void* q, int32_t ld_q, const void* k_pool, const void* v_pool, const void* block_tables, const void* context_lens,
+                                                  const void* chunk_offsets, void* out, int32_t ld_out, void* scratch, int32_t n_seqs, int32_t total_chunks,
+                                                  int32_t chunk_tokens, int32_t max_blocks, int32_t n_pool_blocks, int32_t heads, int32_t n_kv_heads, int32_t head_dim,
+                                                  const lg_window_t* window, int32_t v, float lambda, float scale, float eps, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (!window_ok(window, 2 * heads) || window->gate || heads <= 0 || n_kv_heads <= 0 || heads % n_kv_heads || v <= 0 || v > head_dim || ld_out < heads * head_dim) return lg::kInvalidValue;
+  WindowExt ext = window_ext(window, ld_q, 2 * heads * head_dim);
+  ext.raw = kRawPartial;
+  const float sl2 = window->scale * kLog2e;
+  if (uint32_t rc = launch_ext_decode<kWindowed>(q, ld_q, k_pool, v_pool, block_tables, context_lens, chunk_offsets, out, 2 * heads * head_dim, scratch, n_seqs, total_chunks,
+                                                 chunk_tokens, max_blocks, n_pool_blocks, 2 * heads, n_kv_heads, head_dim, sl2, ext, status, stream))
+    return rc;
+  const float* part_o = (const float*)scratch;
+  lg::launch(paged_decode_merge_difference_kernel, dim3((unsigned)n_seqs, (unsigned)heads), dim3((unsigned)head_dim), 0, (cudaStream_t)stream, part_o,
+             part_o + (size_t)total_chunks * 2 * heads * head_dim, (const int*)chunk_offsets, (__nv_bfloat16*)out, ld_out, 2 * heads, heads / n_kv_heads, head_dim, v, sl2, lambda, scale,
+             eps);
+  return lg::launch_status();
 }
 
 uint32_t logismos_launch_paged_kv_store_bf16(const void* k, const void* v, int32_t src_row_stride, void* k_pool,

@@ -226,7 +226,8 @@ uint32_t logismos_launch_gated_residual(const lg_gated_residual_t* a, void* stat
   p.gate = a->gate; p.ld_gate = a->ld_gate; p.kept = (float4*)a->kept; p.embed = a->embed; p.ids = (const uint32_t*)a->ids; p.step = (const float4*)a->step; p.vocab = a->vocab;
   p.h = a->h; p.gain = a->gain; p.eps = a->eps; p.row_idx = (const int*)a->row_idx; p.n_src_rows = a->n_src_rows; p.n = a->n; p.nv = a->ld / 4; p.f32 = a->is_f32; p.status = (int*)status;
   int nv = 1;
-  while (p.nv > kMaxThreads * nv) nv *= 2;
+  const int most = a->rows > 512 && p.nv <= 256 * kMaxVec ? 256 : kMaxThreads;   // many rows: smaller CTAs with more in flight per thread
+  while (p.nv > most * nv) nv *= 2;
   const int threads = ((p.nv + nv - 1) / nv + 31) / 32 * 32;
   auto go = [&](auto kern) -> uint32_t {
     lg::launch(kern, dim3((unsigned)a->rows), dim3((unsigned)threads), 0, (cudaStream_t)stream, p);

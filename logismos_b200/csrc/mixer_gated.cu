@@ -127,7 +127,7 @@ void gate_up_rows(Mat& dst, int row0, const void* gate, const void* up, int firs
 
 }  // namespace
 
-uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int ld_q, int heads, int kv, int hd, void* out, int ld_out, cudaStream_t s) {
+uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int ld_q, int heads, int kv, int hd, void* out, int ld_out, cudaStream_t s, bool prompts_only) {
   const lg_mixer_config_t& c = m->cfg;
   StepBatch& B = m->batch;
   const DecodeView& V = m->views[(size_t)L.view];
@@ -139,7 +139,7 @@ uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int
     m->launches += 1;
     return 0;
   }
-  if (B.n_dec > 0) {
+  if (B.n_dec > 0 && !prompts_only) {
     LG_TRY(logismos_launch_window_attention_decode_bf16(q, ld_q, L.kpool.p, L.vpool.p, m->dev(B.tables), m->dev(B.ctx), m->dev(V.chunks), out, ld_out, m->dec_scratch.p,
                                                         B.n_dec, V.total, V.chunk_tokens, MB, c.n_pool_blocks, heads, kv, hd, &w, st, s), "decode attention");
     m->launches += V.total > B.n_dec ? 2 : 1;

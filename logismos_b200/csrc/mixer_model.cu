@@ -176,6 +176,7 @@ uint32_t gated_residual(Mixer* m, int l, bool second, void* y, bool zero_y, cons
   return logismos_launch_gated_residual(&a, m->status.p, s);
 }
 
+constexpr int kStreamRows = 16;   // up to so many rows the output projections of a gated stack stream their weights (us, small / tiles that split k: 1024 x 1024 2.6 / 4.8, 4096 x 4096 8.9 / 10.8)
 constexpr int kFusedNormRows = 16;   // up to so many rows the norms around the residual ride on the output projection
 
 // What follows a sublayer of layer l: the norm of its output y, the residual, and the input of the next sublayer.
@@ -195,7 +196,7 @@ uint32_t finish_sublayer(Mixer* m, int l, bool second, void* y, bool zero_y, con
 
 uint32_t output_projection(Mixer* m, int l, bool second, const void* a, int k, const Buf& w, cudaStream_t s) {
   const int T = m->batch.T, Hp = m->Hp;
-  const bool acc = m->accumulates(T);
+  const bool acc = m->accumulates(T) && !(m->cfg.norm == LG_NORM_RMS_GATED && T <= kStreamRows);
   void* y = acc ? m->y_acc.p : m->y.p;
   if (m->cfg.norm == LG_NORM_TANH_AROUND && !m->cfg.is_f32 && T <= kFusedNormRows) {  // the norms in the product's epilogue
     const TanhNorm *post, *next;
@@ -216,11 +217,20 @@ uint32_t mixer_output(Mixer* m, int l, cudaStream_t s) {
   const MWeights& W = m->weights[(size_t)L.owner];
   if (L.c.kind != LG_MIXER_PAIR) return output_projection(m, l, false, m->act.p, L.Kout, W.w_out, s);
   const int T = m->batch.T, Hp = m->Hp;
-  const bool acc = m->accumulates(T);
+  const bool acc = m->accumulates(T) && T > kStreamRows, both = L.Kout == 2 * L.Kleft;
   float *y = (float*)(acc ? m->y_acc.p : m->y.p), *y2 = y + (acc ? m->acc_bytes / 8 : (size_t)m->cfg.max_step_tokens * Hp);
-  LG_TRY(linear(m, m->act.p, L.Kout, W.w_out, Hp, L.Kleft, y, Hp, acc ? LG_EPI_RESID_F32 : LG_EPI_F32, T, s), "left output projection");
-  const void* right = (const uint8_t*)m->act.p + (size_t)L.Kleft * (m->cfg.is_f32 ? 4 : 2);
-  LG_TRY(linear(m, right, L.Kout, W.w_out2, Hp, L.Kout - L.Kleft, y2, Hp, acc ? LG_EPI_RESID_F32 : LG_EPI_F32, T, s), "right output projection");
+  const int epi = acc ? LG_EPI_RESID_F32 : LG_EPI_F32;
+  if (both && !m->cfg.is_f32 && T <= kStreamRows) {
+    LG_TRY(logismos_launch_linear_small_bf16(m->act.p, W.w_out.p, nullptr, y, T, Hp, L.Kleft, L.Kout, Hp, 2, L.Kleft, (int64_t)Hp * L.Kleft, y2 - y, LG_EPI_F32, 0, 0, 0, s),
+           "output projections");
+    m->launches += 1;
+  } else {
+    LG_TRY(linear(m, m->act.p, L.Kout, W.w_out, Hp, L.Kleft, y, Hp, epi, T, s), "left output projection");
+    const void* right = (const uint8_t*)m->act.p + (size_t)L.Kleft * (m->cfg.is_f32 ? 4 : 2);
+    Buf second = W.w_out2;
+    if (both) second.p = (uint16_t*)W.w_out.p + (size_t)Hp * L.Kleft;
+    LG_TRY(linear(m, right, L.Kout, second, Hp, L.Kout - L.Kleft, y2, Hp, epi, T, s), "right output projection");
+  }
   LG_TRY(finish_sublayer(m, l, false, y, acc, nullptr, s), "output norm");
   return 0;
 }

@@ -52,14 +52,24 @@ uint32_t store_heads(Mixer* m, MLayer& L, const MWeights& W, int maps, cudaStrea
 
 uint32_t differential(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   const lg_mixer_config_t& c = m->cfg;
-  const int heads = 2 * L.c.heads, ld = heads * L.Dh, T = m->batch.T;
+  StepBatch& B = m->batch;
+  const int heads = 2 * L.c.heads, ld = heads * L.Dh, T = B.T;
   LG_TRY(projections(m, L, W, false, s), "input projections");
   if (uint32_t rc = store_heads(m, L, W, 2, s)) return rc;
   lg_window_t w = m->views[(size_t)L.view].shape;
   w.scale = L.c.scale; w.out_f32 = 1;
-  if (uint32_t rc = window_attention(m, L, w, m->qx.p, ld, heads, L.c.kv_heads, L.Dh, m->maps_out.p, ld, s)) return rc;
-  LG_TRY(logismos_launch_attention_difference(m->maps_out.p, ld, m->act.p, L.Kout, c.is_f32, T, L.c.heads, L.c.kv_heads, L.c.vdim, L.Dh, W.lambda, 1.0f - L.c.diff,
-                                              c.norm_eps, s), "difference");
+  const int alone = c.is_f32 ? 0 : B.n_dec;   // decode rows whose merge takes the difference too
+  if (alone > 0) {
+    const DecodeView& V = m->views[(size_t)L.view];
+    LG_TRY(logismos_launch_differential_decode_bf16(m->qx.p, ld, L.kpool.p, L.vpool.p, m->dev(B.tables), m->dev(B.ctx), m->dev(V.chunks), m->act.p, L.Kout, m->dec_scratch.p, alone,
+                                                    V.total, V.chunk_tokens, c.max_blocks_per_seq, c.n_pool_blocks, L.c.heads, L.c.kv_heads, L.Dh, &w, L.c.vdim, W.lambda,
+                                                    1.0f - L.c.diff, c.norm_eps, m->status.p, s), "differential decode");
+    m->launches += 2;
+  }
+  if (T == alone) return 0;
+  if (uint32_t rc = window_attention(m, L, w, m->qx.p, ld, heads, L.c.kv_heads, L.Dh, m->maps_out.p, ld, s, true)) return rc;
+  LG_TRY(logismos_launch_attention_difference((const float*)m->maps_out.p + (size_t)alone * ld, ld, (uint8_t*)m->act.p + (size_t)alone * L.Kout * (c.is_f32 ? 4 : 2), L.Kout, c.is_f32,
+                                              T - alone, L.c.heads, L.c.kv_heads, L.c.vdim, L.Dh, W.lambda, 1.0f - L.c.diff, c.norm_eps, s), "difference");
   m->launches += 1;
   return 0;
 }
@@ -176,7 +186,16 @@ bool upload_paired_kinds(Mixer* m, const MLayer& L, MWeights& W, const lg_mixer_
     head_cols(out2, 0, w.right_o, H, lin, c.lin_vdim, L.Vp);
     std::vector<float> decay((size_t)lin);
     for (int h = 0; h < lin; ++h) decay[(size_t)h] = (float)std::max(std::log2(c.decay[h]), -1e4);  // nothing is left of a step further down
-    ok = ok && out2.up(W.w_out2) && W.log2_decay.upload(decay.data(), decay.size() * 4) && upload_heads(W.gain, w.right_norm, lin, c.lin_vdim, L.Vp) &&
+    if (L.Kout == 2 * L.Kleft) {  // one batch of two products
+      Mat both(2 * Hp, L.Kleft);
+      std::copy(out.v.begin(), out.v.end(), both.v.begin());
+      std::copy(out2.v.begin(), out2.v.end(), both.v.begin() + (std::ptrdiff_t)out.v.size());
+      W.w_out.release();
+      ok = ok && both.up(W.w_out);
+    } else {
+      ok = ok && out2.up(W.w_out2);
+    }
+    ok = ok && W.log2_decay.upload(decay.data(), decay.size() * 4) && upload_heads(W.gain, w.right_norm, lin, c.lin_vdim, L.Vp) &&
          upload_vec(W.branch_gain[0], w.left_out, H, Hp, 0.0f) && upload_vec(W.branch_gain[1], w.right_out, H, Hp, 0.0f);
   }
   std::vector<float> b((size_t)L.N, 0.0f);

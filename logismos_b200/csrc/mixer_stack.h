@@ -178,8 +178,10 @@ bool alloc_gated_kinds(Mixer* m, MLayer& L, Sizes& z);
 bool want_gated_kinds(Wanted& t, const std::string& mix, int64_t width, lg_mixer_layer_config_t& y, lg_mixer_layer_weights_t& L);
 uint32_t run_gated_kinds(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s);
 
-// attention over a window from queries and the layer's cache: `heads` query heads of hd channels, kv key heads
-uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int ld_q, int heads, int kv, int hd, void* out, int ld_out, cudaStream_t s);
+// attention over a window from queries and the layer's cache: `heads` query heads of hd channels, kv key heads (bf16: prompt rows
+// alone, where decode rows have a launch of their own)
+uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int ld_q, int heads, int kv, int hd, void* out, int ld_out, cudaStream_t s,
+                          bool prompts_only = false);
 
 const char* check_paired_kinds(const lg_mixer_layer_config_t& y);
 void layout_paired_kinds(const Mixer* m, MLayer& L);

@@ -31,6 +31,8 @@ struct ScoreExt {
   LG_DEVINL float gated(float o, float g) const { return o * __fdividef(gate_scale, 1.0f + __expf(-g)); }
 };
 
+constexpr int kRawPartial = 2;
+
 // The window form: where a query at position i looks, and what becomes of its output. What stands ahead of the window, kept
 // first keys or pooled blocks, is numbered through with it: `lead` of them, then the window's keys from a place rounded down.
 struct WindowExt {
@@ -38,7 +40,7 @@ struct WindowExt {
   const float* gate;             // [rows, ld_gate], NULL: none
   int ld_gate;
   int ld_q, ld_out;
-  int raw;                       // the output is fp32
+  int raw;                       // the output is fp32 (kRawPartial: decode leaves all partial results to another merge)
   const void *kmean, *vmean;     // pooled keys and values, mean_rows() of them per cache block
   // first key of the window
   __host__ __device__ int first(int i) const { return chunked ? i - i % size : i < size ? 0 : i - size + 1; }
@@ -71,7 +73,7 @@ inline bool window_ok(const lg_window_t* w, int heads) {
          (!w->pool || (w->k_mean && w->v_mean && (((uintptr_t)w->k_mean | (uintptr_t)w->v_mean) & 15) == 0));
 }
 inline WindowExt window_ext(const lg_window_t* w, int ld_q, int ld_out) {
-  return WindowExt{w->size ? w->size : 0x7fffffff, w->keep_first, w->sink, w->chunked, w->pool, (const float*)w->gate, w->ld_gate, ld_q, ld_out, w->out_f32, w->k_mean, w->v_mean};
+  return WindowExt{w->size ? w->size : 0x7fffffff, w->keep_first, w->sink, w->chunked, w->pool, (const float*)w->gate, w->ld_gate, ld_q, ld_out, w->out_f32 ? 1 : 0, w->k_mean, w->v_mean};
 }
 
 inline bool score_ok(const lg_score_bias_t* s, int width) {

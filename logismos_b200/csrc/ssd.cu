@@ -424,7 +424,8 @@ gated_norm_warp_kernel(const __nv_bfloat16* __restrict__ y, int ld_y, const __nv
 
 // The same for any width and format, a CTA per (row, part). VEC: channels are contiguous (no
 // padding between heads) and eight of them are moved at once.
-template <typename T, bool VEC, bool AFTER>
+// KM: pieces of eight channels per thread
+template <typename T, bool VEC, bool AFTER, int KM = 1>
 __global__ void __launch_bounds__(512)
 gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__ z, int ld_z, const float* __restrict__ gain, T* __restrict__ out,
                         int ld_out, int width, int v, int vp, float eps) {
@@ -434,11 +435,10 @@ gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__
   const T *yr = y + (size_t)r * ld_y, *zr = z + (size_t)r * ld_z;
   T* o = out + (size_t)r * ld_out;
   if constexpr (VEC) {
-    constexpr int kMax = 4;  // width <= 4 * 8 * 512
-    float x[kMax][8], after[AFTER ? kMax : 1][8];
+    float x[KM][8], after[AFTER ? KM : 1][8];  // width <= KM * 8 * 512
     float ss = 0.0f;
 #pragma unroll
-    for (int i = 0; i < kMax; ++i) {
+    for (int i = 0; i < KM; ++i) {
       const int c = 8 * (threadIdx.x + i * blockDim.x);
       if (c >= width) break;
       float a[8], g[8];
@@ -457,13 +457,13 @@ gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
         x[i][k] = AFTER ? a[k] : a[k] * (sizeof(T) == 2 ? __fdividef(g[k], 1.0f + __expf(-g[k])) : silu_f(g[k]));
-        if (AFTER) after[AFTER ? i : 0][k] = sigmoid_f(g[k]);
+        if (AFTER) after[AFTER ? i : 0][k] = sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(-g[k])) : sigmoid_f(g[k]);
         ss += x[i][k] * x[i][k];
       }
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
 #pragma unroll
-    for (int i = 0; i < kMax; ++i) {
+    for (int i = 0; i < KM; ++i) {
       const int c = 8 * (threadIdx.x + i * blockDim.x);
       if (c >= width) break;
       const float4 g0 = __ldg(reinterpret_cast<const float4*>(gain + c0 + c)), g1 = __ldg(reinterpret_cast<const float4*>(gain + c0 + c + 4));
@@ -539,8 +539,12 @@ uint32_t launch_gated_norm(const void* y, int32_t ld_y, const void* z, int32_t l
     lg::launch(kern, grid, dim3((unsigned)threads), 0, (cudaStream_t)stream, (const T*)y, ld_y, (const T*)z, ld_z, (const float*)gain_f32, (T*)out, ld_out, width, v, vp, eps);
     return lg::launch_status();
   };
-  if (is_f32) return vec ? go(gated_group_norm_kernel<float, true, AFTER>, (float*)nullptr) : go(gated_group_norm_kernel<float, false, AFTER>, (float*)nullptr);
-  return vec ? go(gated_group_norm_kernel<__nv_bfloat16, true, AFTER>, (__nv_bfloat16*)nullptr) : go(gated_group_norm_kernel<__nv_bfloat16, false, AFTER>, (__nv_bfloat16*)nullptr);
+  auto pick = [&](auto* t) {
+    using T = std::remove_pointer_t<decltype(t)>;
+    if (!vec) return go(gated_group_norm_kernel<T, false, AFTER>, t);
+    return width <= 4096 ? go(gated_group_norm_kernel<T, true, AFTER, 1>, t) : go(gated_group_norm_kernel<T, true, AFTER, 4>, t);
+  };
+  return is_f32 ? pick((float*)nullptr) : pick((__nv_bfloat16*)nullptr);
 }
 
 }  // namespace
