@@ -72,6 +72,25 @@ LG_DEVINL int group_of(const lg_linear_groups_t& g, int c) {
   return i;
 }
 
+// 32 columns from ncol on of a row of the fp32 tail
+LG_DEVINL void store_tail(const lg_linear_groups_t& groups, const uint32_t (&r)[32], int row, int ncol, int N) {
+  const int c0 = ncol - groups.n_main, width = N - groups.n_main;
+  float* dst = reinterpret_cast<float*>(groups.tail) + (size_t)row * groups.ld_tail + c0;
+  __nv_bfloat16* parts = reinterpret_cast<__nv_bfloat16*>(groups.tail_parts) + (size_t)row * 2 * width + c0;
+#pragma unroll
+  for (int j = 0; j < 32; ++j) {
+    if (ncol + j >= N) continue;
+    float v = __uint_as_float(r[j]);
+    if (groups.tail_cap > 0.0f) v = groups.tail_cap * tanhf(v / groups.tail_cap);
+    dst[j] = v;
+    if (groups.tail_parts) {
+      const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+      parts[j] = hi;
+      parts[width + j] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    }
+  }
+}
+
 // One matrix per group of rows (EXPERTS): the row tiles are listed on the device; map_out then describes the activations
 // that some groups read directly.
 struct RowTiles {
@@ -261,51 +280,59 @@ linear_t_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
           }
           slab_release(b, ncol, row0, ncol < N && row0 < M);
         }
-      } else if (EPI == LG_EPI_BF16 || EPI == LG_EPI_RELU2 || EPI == kEpiGroups) {
+      } else if (!EXPERTS && (EPI == LG_EPI_BF16 || EPI == LG_EPI_RELU2 || EPI == kEpiGroups)) {  // 64 columns at a time through the staging slabs
+        const int n_out = EPI == kEpiGroups ? groups.n_main : N;
+        for (int c = 0; c < BN; c += 64) {
+          const int ncol = n_blk * BN + c;
+          if (ncol >= N) break;
+          uint32_t ra[32], rb[32];
+          tc_ld32(t_row + c, ra);
+          tc_ld32(t_row + c + 32, rb);
+          tc_wait_ld();
+          if (EPI == kEpiGroups && ncol >= n_out) {
+            if (row < row_end) {
+              store_tail(groups, ra, row, ncol, N);
+              store_tail(groups, rb, row, ncol + 32, N);
+            }
+            continue;
+          }
+          const int b = slab_acquire();
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            const int col = ncol + 8 * j;
+            float bv[8] = {};
+            if (bias && col < n_out) load_bias8(bias + col, bias_vec, bv);
+            const bool silu = EPI == kEpiGroups && col >= groups.silu_begin && col < groups.silu_end;
+            uint32_t w[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const int e = (8 * j + 2 * i) & 31;
+              float x = __uint_as_float(j < 4 ? ra[e] : rb[e]) + bv[2 * i], y = __uint_as_float(j < 4 ? ra[e + 1] : rb[e + 1]) + bv[2 * i + 1];
+              if (EPI == LG_EPI_RELU2) { x = fmaxf(x, 0.0f); y = fmaxf(y, 0.0f); x *= x; y *= y; }
+              if (silu) { x = lg::silu_fast(x); y = lg::silu_fast(y); }
+              w[i] = pack_bf16x2(x, y);
+            }
+            slab_write(slabs + b * 4096, lane, j, make_uint4(w[0], w[1], w[2], w[3]));
+          }
+          slab_release(b, ncol, row0, row0 < M);
+        }
+      } else if (EPI == LG_EPI_BF16) {  // a group's rows may end inside a tile
         for (int c = 0; c < BN; c += 32) {
           uint32_t r[32];
           tc_ld32(t_row + c, r);
           tc_wait_ld();
           const int ncol = n_blk * BN + c;
-          if (EPI == kEpiGroups && ncol >= groups.n_main) {
-            if (row < row_end) {
-              const int c0 = ncol - groups.n_main, width = N - groups.n_main;
-              float* dst = reinterpret_cast<float*>(groups.tail) + (size_t)row * groups.ld_tail + c0;
-              __nv_bfloat16* parts = reinterpret_cast<__nv_bfloat16*>(groups.tail_parts) + (size_t)row * 2 * width + c0;
+          if (row < row_end) {
+            __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * ldc + ncol;
 #pragma unroll
-              for (int j = 0; j < 32; ++j) {
-                if (ncol + j >= N) continue;
-                float v = __uint_as_float(r[j]);
-                if (groups.tail_cap > 0.0f) v = groups.tail_cap * tanhf(v / groups.tail_cap);
-                dst[j] = v;
-                if (groups.tail_parts) {
-                  const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-                  parts[j] = hi;
-                  parts[width + j] = __float2bfloat16_rn(v - __bfloat162float(hi));
-                }
+            for (int j = 0; j < 4; ++j) {
+              if (ncol + j * 8 < N) {
+                uint32_t w[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) w[i] = pack_bf16x2(__uint_as_float(r[j * 8 + i * 2]), __uint_as_float(r[j * 8 + i * 2 + 1]));
+                *reinterpret_cast<uint4*>(dst + j * 8) = make_uint4(w[0], w[1], w[2], w[3]);
               }
             }
-            continue;
-          }
-          const bool silu = EPI == kEpiGroups && ncol >= groups.silu_begin && ncol < groups.silu_end;
-          if (row < row_end) {
-              __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * ldc + ncol;
-#pragma unroll
-              for (int j = 0; j < 4; ++j) {
-                if (ncol + j * 8 < N) {
-                  uint32_t w[4];
-#pragma unroll
-                  for (int i = 0; i < 4; ++i) {
-                    const int e = j * 8 + i * 2;
-                    float a = __uint_as_float(r[e]), b = __uint_as_float(r[e + 1]);
-                    if (bias) { a += bias[ncol + e]; b += bias[ncol + e + 1]; }
-                    if (EPI == LG_EPI_RELU2) { a = fmaxf(a, 0.0f); b = fmaxf(b, 0.0f); a *= a; b *= b; }
-                    if (silu) { a = lg::silu_fast(a); b = lg::silu_fast(b); }
-                    w[i] = pack_bf16x2(a, b);
-                  }
-                  *reinterpret_cast<uint4*>(dst + j * 8) = make_uint4(w[0], w[1], w[2], w[3]);
-                }
-              }
           }
         }
       } else if (EPI == LG_EPI_F32 && (ldc & 3) == 0) {  // whole 128-byte rows through the staging slabs
@@ -435,6 +462,8 @@ uint32_t launch_cfg(const void* a, const void* w, const float* bias, void* out, 
   if (!make_map(&mw, w, (uint64_t)n, (uint64_t)k, (uint64_t)k, BN)) return lg::kInvalidValue;
   if (EPI == LG_EPI_RESID_F32 || (EPI == LG_EPI_F32 && ldc % 4 == 0)) {  // fp32 [m, n] in 32 x 32 boxes
     if (!make_map(&mo, out, (uint64_t)m, (uint64_t)n, (uint64_t)ldc, 32, true)) return lg::kInvalidValue;
+  } else if (EPI == LG_EPI_BF16 || EPI == LG_EPI_RELU2 || (EPI == kEpiGroups && groups.n_main > 0)) {  // bf16 in 32 x 64 boxes
+    if (!make_map(&mo, out, (uint64_t)m, (uint64_t)(EPI == kEpiGroups ? groups.n_main : n), (uint64_t)ldc, 32)) return lg::kInvalidValue;
   } else {
     mo = ma;  // unused by the direct-store epilogues
   }

@@ -231,16 +231,26 @@ head_norm_store_kernel(HeadArgs p) {
   }
 }
 
+// A thread owns eight channels of all blocks that end in `pool` consecutive rows: one, unless a sequence ends among them
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
 pool_blocks_kernel(HeadArgs p, int octs) {
   lg::pdl_prologue();
   const uint32_t at = blockIdx.x * kThreads + threadIdx.x;
-  const int r = p.pool_rows + (int)(at / (2 * octs)), piece = (int)(at % (2 * octs));
-  if (r >= p.rows || (p.pos[r] + 1) % p.pool) return;
+  const int r0 = p.pool_rows + (int)(at / (2 * octs)) * p.pool, piece = (int)(at % (2 * octs));
   const bool is_v = piece >= octs;
-  pool_piece<T>(p, reinterpret_cast<const T*>(is_v ? p.vpool : p.kpool), reinterpret_cast<T*>(is_v ? p.vmean : p.kmean), p.seq_ids[r], p.pos[r], octs * 8,
-                8 * (is_v ? piece - octs : piece));
+  const int end = min(r0 + p.pool, p.rows);
+  for (int r = r0; r < end;) {
+    const int seq = p.seq_ids[r], pos = p.pos[r], last = r + p.pool - 1 - pos % p.pool;   // where the block of row r ends
+    if (last < end && p.seq_ids[last] == seq) {
+      pool_piece<T>(p, reinterpret_cast<const T*>(is_v ? p.vpool : p.kpool), reinterpret_cast<T*>(is_v ? p.vmean : p.kmean), seq, pos + last - r, octs * 8,
+                    8 * (is_v ? piece - octs : piece));
+      r = last + 1;
+    } else {
+      do ++r;
+      while (r < end && p.seq_ids[r] == seq);
+    }
+  }
 }
 
 bool head_args(const lg_head_norm_t* a, int is_f32, void* status, HeadArgs* p) {
@@ -283,7 +293,7 @@ uint32_t logismos_launch_pool_blocks(const lg_head_norm_t* a, int32_t is_f32, vo
   HeadArgs p;
   if (!head_args(a, is_f32, status, &p) || a->pool <= 0 || a->pool_rows >= a->rows) return lg::kInvalidValue;
   const int octs = a->n_kv * a->maps * a->hd / 8;
-  const int64_t threads = (int64_t)(a->rows - a->pool_rows) * 2 * octs;
+  const int64_t threads = (int64_t)((a->rows - a->pool_rows + a->pool - 1) / a->pool) * 2 * octs;
   if (threads > 0x7fffff00) return lg::kInvalidValue;
   const dim3 grid((unsigned)((threads + kThreads - 1) / kThreads));
   if (is_f32) lg::launch(pool_blocks_kernel<float>, grid, dim3(kThreads), 0, (cudaStream_t)stream, p, octs);
