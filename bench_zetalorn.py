@@ -295,12 +295,13 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         add(ph, "sum of the experts + gated residual + norm", [lambda s, r=r: lib.logismos_launch_gated_residual(Y(r), P(st), s) for r in rs], m * H * 12.0 + 2.0 * n_rows * H, like="sum of the experts + tanh norms")
         add(ph, "= sum of the experts + tanh norms", [lambda s, o=o: lib.logismos_launch_tanh_norm(P(None), 0, Y(o), P(None), m, P(x), Y(norm), P(h), Y(norm), 0, m, H, P(st), s) for o in mo], m * H * 10.0 + 2.0 * n_rows * H)
 
-    decay = torch.log2(1.0 - 2.0 ** (-1.0 - 8.0 * torch.arange(lh, device=dev) / lh)).float()
+    decay = 1.0 - 2.0 ** (-1.0 - 8.0 * torch.arange(lh, device=dev) / lh)
+    decay = torch.stack([torch.log2(decay), decay, torch.zeros_like(decay)], dim=1).float().contiguous()
 
     def linear_args(proj, state, slots, cu, y):
         fresh = u8(slots.numel())
         keep.append(fresh)
-        return Ssd(state=A(state), state_slots=A(slots), fresh=A(fresh), cu=A(cu), y=A(y), ld_y=vw, heads=lh, groups=lh, np=lk, vp=lv, xbc=A(proj), ld_xbc=proj.shape[1], log2_decay=A(decay))
+        return Ssd(state=A(state), state_slots=A(slots), fresh=A(fresh), cu=A(cu), y=A(y), ld_y=vw, heads=lh, groups=lh, np=lk, vp=lv, xbc=A(proj), ld_xbc=proj.shape[1], decay=A(decay))
 
     def gla_args(proj, zz, low, w2, state, slots, cu, out):
         q = [torch.full((kw,), 2.0, device=dev), u8(slots.numel())]

@@ -814,9 +814,10 @@ typedef struct lg_ssd {
   int32_t ld_y, heads, groups, np, vp;
   void* xbc;                    /* activation format [rows, ld_xbc]: the convolved channels x | B | C */
   int32_t ld_xbc;
-  /* given: f32 [heads], log2 of a fixed decay per head. Every step then has size one, S <- decay S + B x^T, y = S^T C (linear
-   * attention: x, B, C its values, keys and queries); only xbc, state and its indices, y and the sizes are used. */
-  const void* log2_decay;
+  /* given: f32 [heads][3], a fixed decay per head as its log2 (at least -1e4), its value and what the value's rounding dropped.
+   * Every step then has size one, S <- decay S + B x^T, y = S^T C (linear attention: x, B, C its values, keys and queries); only
+   * xbc, state and its indices, y and the sizes are used. */
+  const void* decay;
 } lg_ssd_t;
 /* Convolution and silu of rows [row0, rows) from proj into xbc (seq_ids [rows]; cu, slots, fresh and phase indexed by
  * them). single: rows are one token per sequence. */

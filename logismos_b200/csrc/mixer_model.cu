@@ -16,7 +16,7 @@ namespace lgm {
 void MWeights::release() {
   Buf* wb[] = {&norm1, &norm1_b, &norm2, &norm2_b, &w_up, &w_down, &w_in, &w_out, &pre1.w, &pre1.b, &post1.w, &post1.b, &pre2.w, &pre2.b, &post2.w, &post2.b,
                &conv, &conv_b, &dt_bias, &A_log, &D, &gain, &bias, &mu, &w2, &w0, &u, &b_in, &gain_q, &gain_k, &w_uq, &w_uk, &w_ukt, &w_uv, &w_router, &correction,
-               &w_gate2, &b_gate2, &w_out2, &branch_gain[0], &branch_gain[1], &log2_decay};
+               &w_gate2, &b_gate2, &w_out2, &branch_gain[0], &branch_gain[1], &decay};
   for (Buf* b : wb) b->release();
 }
 

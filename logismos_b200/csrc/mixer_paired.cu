@@ -80,7 +80,7 @@ uint32_t linear_attention(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s
   const int f32 = c.is_f32, inner = L.c.lin_heads * L.Vp, P = L.groups.n_main;
   const size_t esz = f32 ? 4 : 2;
   lg_ssd_t a{};
-  a.xbc = (uint8_t*)m->proj.p + (size_t)L.off_right * esz; a.ld_xbc = P; a.log2_decay = W.log2_decay.p;
+  a.xbc = (uint8_t*)m->proj.p + (size_t)L.off_right * esz; a.ld_xbc = P; a.decay = W.decay.p;
   a.state = L.state.p; a.state_slots = m->dev(B.state); a.fresh = m->dev(B.fresh); a.cu = m->dev(B.cu);
   a.y = m->ffb.p; a.ld_y = inner; a.heads = a.groups = L.c.lin_heads; a.np = L.Np; a.vp = L.Vp;
   const bool chunked = !f32 && B.n_pre > 0 && logismos_ssd_has_chunked(L.Np, L.Vp);
@@ -184,8 +184,13 @@ bool upload_paired_kinds(Mixer* m, const MLayer& L, MWeights& W, const lg_mixer_
     head_rows(in, qr + lin * L.Np, w.right_g, lin, c.lin_vdim, L.Vp, H);
     Mat out2(Hp, L.Kout - L.Kleft);
     head_cols(out2, 0, w.right_o, H, lin, c.lin_vdim, L.Vp);
-    std::vector<float> decay((size_t)lin);
-    for (int h = 0; h < lin; ++h) decay[(size_t)h] = (float)std::max(std::log2(c.decay[h]), -1e4);  // nothing is left of a step further down
+    std::vector<float> decay((size_t)lin * 3);
+    for (int h = 0; h < lin; ++h) {
+      float* d = decay.data() + (size_t)h * 3;
+      d[0] = (float)std::max(std::log2(c.decay[h]), -1e4);  // nothing is left of a step further down
+      d[1] = (float)c.decay[h];
+      d[2] = (float)(c.decay[h] - (double)d[1]);
+    }
     if (L.Kout == 2 * L.Kleft) {  // one batch of two products
       Mat both(2 * Hp, L.Kleft);
       std::copy(out.v.begin(), out.v.end(), both.v.begin());
@@ -195,7 +200,7 @@ bool upload_paired_kinds(Mixer* m, const MLayer& L, MWeights& W, const lg_mixer_
     } else {
       ok = ok && out2.up(W.w_out2);
     }
-    ok = ok && W.log2_decay.upload(decay.data(), decay.size() * 4) && upload_heads(W.gain, w.right_norm, lin, c.lin_vdim, L.Vp) &&
+    ok = ok && W.decay.upload(decay.data(), decay.size() * 4) && upload_heads(W.gain, w.right_norm, lin, c.lin_vdim, L.Vp) &&
          upload_vec(W.branch_gain[0], w.left_out, H, Hp, 0.0f) && upload_vec(W.branch_gain[1], w.right_out, H, Hp, 0.0f);
   }
   std::vector<float> b((size_t)L.N, 0.0f);

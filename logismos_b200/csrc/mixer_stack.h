@@ -46,7 +46,7 @@ struct MWeights {   // of a layer that owns tensors
   Buf w_uq, w_uk, w_ukt, w_uv;                            // latent attention
   Buf w_router, correction;                               // mixture: w_up, w_down hold its experts one after the other
   Buf w_gate2, b_gate2;                                   // gated residual: the gate of a feed-forward, then the router's rows
-  Buf w_out2, branch_gain[2], log2_decay;                 // a pair
+  Buf w_out2, branch_gain[2], decay;                 // a pair
   float gain1 = 0.0f, gain2 = 0.0f, lambda = 0.0f;        // norms of one value; differential attention
   float max_bias = 0.0f;
   void release();

@@ -49,7 +49,7 @@ struct SsdArgs {
   int heads, groups, np, vp;
   void* xbc;               // convolved channels [rows, ld_xbc], activation format
   int ld_xbc;
-  const float* log2_decay;
+  const float* decay;
   __host__ __device__ __forceinline__ int channels() const { return heads * vp + 2 * groups * np; }
 };
 
@@ -68,7 +68,7 @@ ssd_step_kernel(SsdArgs p, int in_smem) {
   S.request(t, fresh);
   const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
   const float bias = FIXED ? 0.0f : __ldg(p.dt_bias + head), a = FIXED ? 0.0f : expf(__ldg(p.log_a + head)), skip = FIXED ? 0.0f : __ldg(p.skip + head);
-  const float fixed = FIXED ? exp2f(__ldg(p.log2_decay + head)) : 0.0f;
+  const float fixed = FIXED ? __ldg(p.decay + 3 * head + 1) : 0.0f, dropped = FIXED ? __ldg(p.decay + 3 * head + 2) : 0.0f;
   lg::pdl_wait();
   for (int tok = t0; tok < t1; ++tok) {
     const T* row = reinterpret_cast<const T*>(p.xbc) + (size_t)tok * p.ld_xbc;
@@ -84,7 +84,10 @@ ssd_step_kernel(SsdArgs p, int in_smem) {
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
     S.visit(t, fresh && tok == t0, tok + 1 == t1, [&](int r, float4& s) {
       const float b = bs[r], c = cs[r];
-      s = make_float4(fmaf(decay, s.x, b * x4.x), fmaf(decay, s.y, b * x4.y), fmaf(decay, s.z, b * x4.z), fmaf(decay, s.w, b * x4.w));
+      float4 add = make_float4(b * x4.x, b * x4.y, b * x4.z, b * x4.w);
+      // what the decay's rounding dropped joins the smaller term, where it is not rounded away: no drift over a thousand steps
+      if (FIXED) add = make_float4(fmaf(dropped, s.x, add.x), fmaf(dropped, s.y, add.y), fmaf(dropped, s.z, add.z), fmaf(dropped, s.w, add.w));
+      s = make_float4(fmaf(decay, s.x, add.x), fmaf(decay, s.y, add.y), fmaf(decay, s.z, add.z), fmaf(decay, s.w, add.w));
       o.x = fmaf(c, s.x, o.x); o.y = fmaf(c, s.y, o.y); o.z = fmaf(c, s.z, o.z); o.w = fmaf(c, s.w, o.w);
     });
     reduce_store(t, o, red);
@@ -216,7 +219,7 @@ ssd_chunk_kernel(SsdArgs p) {
   const __nv_bfloat16* xbc = reinterpret_cast<const __nv_bfloat16*>(p.xbc);
   const __nv_bfloat16 *xs = xbc + head * vp, *bs = xbc + inner + group * NP, *cs = bs + p.groups * NP;
   __nv_bfloat16* ys = reinterpret_cast<__nv_bfloat16*>(p.y) + head * vp;
-  const float bias = FIXED ? 0.0f : p.dt_bias[head], a2 = FIXED ? -p.log2_decay[head] : expf(p.log_a[head]) * 1.4426950408889634f, skip = FIXED ? 0.0f : p.skip[head];
+  const float bias = FIXED ? 0.0f : p.dt_bias[head], a2 = FIXED ? -p.decay[3 * head] : expf(p.log_a[head]) * 1.4426950408889634f, skip = FIXED ? 0.0f : p.skip[head];
   float* st = p.state + ((size_t)p.state_slots[seq] * p.heads + head) * NP * vp;
   float S[NT][4];   // state channels 16 m + g, + 8; values v0 + 2 t, + 1
 #pragma unroll
@@ -499,7 +502,7 @@ gated_group_norm_kernel(const T* __restrict__ y, int ld_y, const T* __restrict__
 bool pow2(int v, int lo, int hi) { return v >= lo && v <= hi && (v & (v - 1)) == 0; }
 
 bool args_ok(const lg_ssd_t* a, int n_seqs) {
-  if (a && a->log2_decay)
+  if (a && a->decay)
     return n_seqs > 0 && n_seqs <= 65535 && a->xbc && a->state && a->state_slots && a->fresh && a->cu && a->y && a->heads > 0 && a->groups == a->heads && pow2(a->np, 16, 256) &&
            pow2(a->vp, 16, 256) && a->ld_y >= a->heads * a->vp;
   return a && n_seqs > 0 && n_seqs <= 65535 && a->proj && a->dt && a->conv_w && a->conv_b && a->dt_bias && a->log_a && a->skip && a->state && a->state_slots &&
@@ -511,7 +514,7 @@ bool args_ok(const lg_ssd_t* a, int n_seqs) {
 SsdArgs make_args(const lg_ssd_t* a) {
   return SsdArgs{a->proj, a->ld, (const float*)a->dt, a->ld_dt, (const float*)a->conv_w, (const float*)a->conv_b, (float*)a->conv_state, a->taps,
                  (const float*)a->dt_bias, (const float*)a->log_a, (const float*)a->skip, (float*)a->state, (const int*)a->state_slots,
-                 (const uint8_t*)a->fresh, (const uint8_t*)a->phase, (const int*)a->cu, a->y, a->ld_y, a->heads, a->groups, a->np, a->vp, a->xbc, a->ld_xbc, (const float*)a->log2_decay};
+                 (const uint8_t*)a->fresh, (const uint8_t*)a->phase, (const int*)a->cu, a->y, a->ld_y, a->heads, a->groups, a->np, a->vp, a->xbc, a->ld_xbc, (const float*)a->decay};
 }
 
 template <bool AFTER>
@@ -563,7 +566,7 @@ uint32_t logismos_launch_ssd_step(const lg_ssd_t* a, int32_t n_seqs, int32_t is_
     lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3(kThreads), smem, (cudaStream_t)stream, p, smem > 0 ? 1 : 0);
     return lg::launch_status();
   };
-  if (p.log2_decay) return is_f32 ? go(ssd_step_kernel<float, true>) : go(ssd_step_kernel<__nv_bfloat16, true>);
+  if (p.decay) return is_f32 ? go(ssd_step_kernel<float, true>) : go(ssd_step_kernel<__nv_bfloat16, true>);
   return is_f32 ? go(ssd_step_kernel<float, false>) : go(ssd_step_kernel<__nv_bfloat16, false>);
 }
 
@@ -571,7 +574,7 @@ int32_t logismos_ssd_has_chunked(int32_t np, int32_t vp) { return pow2(np, 32, 1
 
 uint32_t logismos_launch_ssd_conv(const lg_ssd_t* a, const void* seq_ids_i32, int32_t row0, int32_t rows, int32_t single, int32_t is_f32, void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!args_ok(a, 1) || a->log2_decay || !seq_ids_i32 || row0 < 0 || rows <= row0 || !a->xbc || a->ld % 4 || a->ld_xbc % 4 || a->ld_xbc < make_args(a).channels()) return lg::kInvalidValue;
+  if (!args_ok(a, 1) || a->decay || !seq_ids_i32 || row0 < 0 || rows <= row0 || !a->xbc || a->ld % 4 || a->ld_xbc % 4 || a->ld_xbc < make_args(a).channels()) return lg::kInvalidValue;
   const SsdArgs p = make_args(a);
   const int* ids = (const int*)seq_ids_i32;
   cudaStream_t s = (cudaStream_t)stream;
@@ -591,7 +594,7 @@ uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* a, int32_t n_seqs, voi
     lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3((unsigned)(4 * p.vp)), smem, (cudaStream_t)stream, p);
     return lg::launch_status();
   };
-  if (p.log2_decay) return a->np == 32 ? go(ssd_chunk_kernel<32, true>) : a->np == 64 ? go(ssd_chunk_kernel<64, true>) : go(ssd_chunk_kernel<128, true>);
+  if (p.decay) return a->np == 32 ? go(ssd_chunk_kernel<32, true>) : a->np == 64 ? go(ssd_chunk_kernel<64, true>) : go(ssd_chunk_kernel<128, true>);
   return a->np == 32 ? go(ssd_chunk_kernel<32, false>) : a->np == 64 ? go(ssd_chunk_kernel<64, false>) : go(ssd_chunk_kernel<128, false>);
 }
 

@@ -25,7 +25,7 @@ class TimeMix(C.Structure):
 
 class Ssd(C.Structure):
     _fields_ = [("proj", vp), ("ld", i32), ("dt", vp), ("ld_dt", i32)] + _pointers("conv_w", "conv_b", "conv_state") + _ints("taps") + _pointers(
-               "dt_bias", "log_a", "skip", "state", "state_slots", "fresh", "phase", "cu", "y") + _ints("ld_y", "heads", "groups", "np", "vp") + [("xbc", vp), ("ld_xbc", i32), ("log2_decay", vp)]
+               "dt_bias", "log_a", "skip", "state", "state_slots", "fresh", "phase", "cu", "y") + _ints("ld_y", "heads", "groups", "np", "vp") + [("xbc", vp), ("ld_xbc", i32), ("decay", vp)]
 
 
 class ScoreBias(C.Structure):

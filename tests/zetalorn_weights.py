@@ -43,7 +43,7 @@ _B = [attention(4, 1, 64, 128, 70, rotation(64, 5e4), 0.8, moe(12, 1, 40, 4, 1, 
 _C = [parallel(left(20, 1, 8, 8, 5, 1, rotation(2, 50.0)), right(10, 8, (0.7, 1.0, 0.0, 0.95, 0.3)), moe(3, 3, 33, 1, 1)), attention(20, 1, 8, 8, 3, rotation(8, 9.0, 1.5), 0.5),
       parallel(left(1, 1, 16, 9, 33, 40, rotation(10)), right(16, 16, (0.97,)), moe(4, 2, 16, 4, 2))]
 _D = [attention(2, 1, 120, 200, 130, rotation(100, 1e4), 0.6, moe(40, 4, 24, 8, 3)), parallel(left(2, 2, 150, 200, 64, 3, rotation(150, 1e4)), right(136, 20, (0.99, 0.4))),
-      parallel(left(2, 1, 40, 140, 1, 2, rotation(4)), right(40, 140, (0.98,)), moe(36, 2, 16, 4, 3)), attention(4, 2, 130 - 2, 40, 1, rotation(12), 0.9)]
+      parallel(left(2, 1, 40, 140, 1, 2, rotation(4)), right(40, 140, (0.98,))), attention(4, 2, 130 - 2, 40, 1, rotation(12), 0.9)]
 
 CONFIGS = {
     # nothing a multiple of 64, grouped keys, a pool that straddles pages, a run of layers repeated three times
