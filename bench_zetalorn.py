@@ -331,7 +331,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
     slot64 = torch.as_tensor((perm[:, :, None] * 16 + np.arange(16)).reshape(-1).astype(np.int64)).to(dev)
     pools, means = (bf(nb, 16, KD), bf(nb, 16, KD)), (bf(nb, 2, KD), bf(nb, 2, KD))
     qkvs = [bf(T, HD + 2 * KD) for _ in range(copies(2 * T * (HD + 2 * KD)))]
-    att, qx, maps = bf(T, HD), bf(T, 2 * HD), rf(T, 2 * HD)
+    att, qx = bf(T, HD), bf(T, 2 * HD)
     ha = [head_args(q, T, 1, pools, means, tabs, seq_ids, slot64, pos, nb, None) for q in qkvs]
     hb = [head_args(q, T, 2, pools, None, tabs, seq_ids, slot64, pos, nb, qx) for q in qkvs]
     move = T * (4.0 * HD + 8.0 * KD)
@@ -341,7 +341,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
                                                                                                                   1e-6, P(table), ROT, T, 0, P(st), s) for q in qkvs], move)
     add(ph, "means of blocks", [lambda s: lib.logismos_launch_pool_blocks(Y(ha[0]), 0, P(st), s)] * 4, T * 4.0 * KD * (1 + 1 / POOL), like="q, k norm + rotation + store, whole rows")
     gate = rf(T, 2 * heads)
-    wins = {"pooled": Window(scale=DIM ** -0.5, size=WINDOW, pool=POOL, k_mean=A(means[0]), v_mean=A(means[1])), "chunked": Window(scale=MAP ** -0.5, size=CHUNK, chunked=1, out_f32=1),
+    wins = {"pooled": Window(scale=DIM ** -0.5, size=WINDOW, pool=POOL, k_mean=A(means[0]), v_mean=A(means[1])), "chunked": Window(scale=MAP ** -0.5, size=CHUNK, chunked=1),
             "kept": Window(DIM ** -0.5, WINDOW, 4, 1, A(gate), heads)}
     scr = torch.empty(lib.logismos_paged_prefix_attention_scratch_bytes(T * 2, nq, kv, DIM), dtype=torch.uint8, device=dev)
 
@@ -354,10 +354,11 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
     add(ph, "= window attention (with gather)", [lambda s, q=q: prefix(s, q, wins["kept"], att, heads) for q in qkvs], T * 4.0 * HD + kvb, 4.0 * HD * nq * BV.window_pairs(1024))
 
     def differential(s):
-        return prefix(s, qx, wins["chunked"], maps, 2 * heads) or lib.logismos_launch_attention_difference(P(maps), 2 * HD, P(att), HD, 0, T, heads, kv, DIM, DIM, 0.4, 0.7, 1e-6, s)
-    add(ph, "differential attention (with gather and difference)", [differential] * 4, T * 4.0 * HD + kvb, 4.0 * heads * (MAP + DIM) * nq * attention_pairs(1024, False), "window attention (with gather)")
-    add(ph, "  of it the difference", [lambda s: lib.logismos_launch_attention_difference(P(maps), 2 * HD, P(att), HD, 0, T, heads, kv, DIM, DIM, 0.4, 0.7, 1e-6, s)] * 4, T * 10.0 * HD, like="post_norm")
-    del qkvs, qx, maps
+        n = lib.logismos_window_view_keys(Y(wins["chunked"]), 1024, 1024)
+        return lib.logismos_launch_differential_prefix_bf16(P(qx), 2 * HD, P(cu), P(kv_lens), P(pools[0]), P(pools[1]), P(tabs), nblk, nb, P(att), HD, P(scr), T, n * nq, nq, 1024, n, heads, kv, DIM,
+                                                            Y(wins["chunked"]), DIM, 0.4, 0.7, 1e-6, P(st), s)
+    add(ph, "differential attention (with gather)", [differential] * 4, T * 4.0 * HD + kvb, 4.0 * heads * (MAP + DIM) * nq * attention_pairs(1024, False), "window attention (with gather)")
+    del qkvs, qx
     prs, lst, ly = [bf(T, 2 * kw + 2 * vw) for _ in range(copies(4 * T * (kw + vw)))], zf(nq, lh, lk, lv), bf(T, vw)
     la = [linear_args(q, lst, slots, cu, ly) for q in prs]
     rec_b, rec_f = T * (4.0 * kw + 4.0 * vw), T * lh * (4.0 * lk * lv + 64.0 * (lk + lv))
@@ -415,7 +416,7 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
         add(ph, "= q, k norm + rotation + store, whole rows", [lambda s: lib.logismos_launch_qk_norm_rotary_store(P(dq), dq.shape[1], P(pools[0]), P(pools[1]), P(s1), P(ps), m, heads, kv, DIM, DIM, P(ones), P(ones), 1e-6,
                                                                                                                  P(table), ROT, nb * 16, 0, P(st), s)] * 4, move)
         tabw = [torch.roll(tab, 33 * i, 1).contiguous() for i in range(12)]   # shifted tables, so that the keys seen exceed L2 together
-        wins = {"pooled": Window(scale=DIM ** -0.5, size=WINDOW, pool=POOL, k_mean=A(means[0]), v_mean=A(means[1])), "chunked": Window(scale=MAP ** -0.5, size=CHUNK, chunked=1, out_f32=1),
+        wins = {"pooled": Window(scale=DIM ** -0.5, size=WINDOW, pool=POOL, k_mean=A(means[0]), v_mean=A(means[1])), "chunked": Window(scale=MAP ** -0.5, size=CHUNK, chunked=1),
                 "kept": Window(DIM ** -0.5, WINDOW, 4, 1, A(gd), heads)}
 
         def decode(name, w, q, out, nh, seen, like, differential=False):

@@ -1054,6 +1054,17 @@ uint32_t logismos_launch_differential_decode_bf16(const void* q, int32_t ld_q, c
                                                   int32_t n_kv_heads, int32_t head_dim, const lg_window_t* window, int32_t v,
                                                   float lambda, float scale, float eps, void* status_i32, void* stream);
 
+/* The same of prompt rows, both maps in one pass over the keys (head_dim 64 or 128: logismos_differential_has_prompts); a window
+ * or chunks. Otherwise as logismos_launch_window_attention_prefix_bf16. */
+int32_t logismos_differential_has_prompts(int32_t head_dim);
+uint32_t logismos_launch_differential_prefix_bf16(const void* q, int32_t ld_q, const void* cu_seqlens_q, const void* kv_lens,
+                                                  const void* k_pool, const void* v_pool, const void* block_tables,
+                                                  int32_t max_blocks, int32_t n_pool_blocks, void* out, int32_t ld_out,
+                                                  void* scratch, int32_t n_q_tokens, int32_t total_keys, int32_t n_seqs,
+                                                  int32_t max_q_len, int32_t max_keys, int32_t heads, int32_t n_kv_heads,
+                                                  int32_t head_dim, const lg_window_t* window, int32_t v, float lambda,
+                                                  float scale, float eps, void* status_i32, void* stream);
+
 /* Residual stream with RMS norms of one gain and gated sublayers, one launch between two sublayers:
  *   y = branch[0] (one branch), half the sum of both, each divided by its root mean square, times its gain, or a mixture
  *   x += y sigmoid(gate);   kept = x;   x += embed[ids] + step;   h = x / rms(x) * gain

@@ -171,6 +171,7 @@ def _declare(l, partial=False):
         "logismos_launch_pool_blocks": [vp, i32, vp, vp],
         "logismos_launch_attention_difference": [vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp],
         "logismos_launch_gated_residual": [vp, vp, vp],
+        "logismos_launch_differential_prefix_bf16": [vp, i32, vp, vp, vp, vp, vp, i32, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, i32, f32, f32, f32, vp, vp],
         "logismos_launch_differential_decode_bf16": [vp, i32, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, i32, f32, f32, f32, vp, vp],
         "logismos_launch_unit_qk_store": [vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, f32, f32, i64, i32, vp, vp],
         "logismos_launch_bias_attention_decode_bf16": [vp, i32, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp],
@@ -244,6 +245,7 @@ def _declare(l, partial=False):
         "lg_mixer_destroy": ([vp], None),
         "lg_mixer_logits_device": ([vp], vp),
         "logismos_window_context": ([i32, i32, i32], i32),
+        "logismos_differential_has_prompts": ([i32], i32),
         "logismos_window_view_context": ([vp, i32], i32),
         "logismos_window_view_keys": ([vp, i32, i32], i32),
         "logismos_window_keys": ([i32, i32, i32, i32], i32),

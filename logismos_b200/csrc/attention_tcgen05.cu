@@ -720,6 +720,248 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   }
 }
 
+// Differential attention of prompts: both maps of a head over one pass of the keys and values, and their difference.
+// CTA = (128 queries, one head, one sequence), 10 warps: TMA producer, MMA issuer, and four softmax warps per map as above. A key
+// row holds both maps' keys, so a K tile serves both score products and a V^T tile both P V products:
+//   S_m = Q_m K_m^T (64 columns of the key row each; narrower heads: all 64, the other map's half of Q_m being zero), O_m += P_m V
+// K and V have two slots each. Per block the issuer waits for one map's P, queues its P V and the next scores of that map, then
+// the same of the other: one map's softmax runs while the tensor pipe works for the other. At the end each group of softmax
+// threads takes half of the columns of both outputs: o = O_1 / l_1 - lambda O_2 / l_2, over its root mean square, times scale.
+struct DiffOut {
+  float lambda, scale, eps;
+  int v;                        // true channels of a head
+};
+constexpr int kDiffThreads = 320, kDiffBars = 14;   // q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], o_done
+template <int HD> struct DiffAttn {
+  static constexpr int kQBytes = 2 * kTileBytes, kKBytes = (HD / 64) * kTileBytes, kVTile = HD * 128, kVBytes = 2 * kVTile;
+  // queries, two slots of keys and of values, barriers, 1 / l and partial sums of squares of both maps' rows
+  static constexpr size_t kSmem = 1024 + kQBytes + 2 * (kKBytes + kVBytes) + 8 * kDiffBars + 16 + 4 * 128 * 4;
+};
+
+template <int HD>
+__global__ void __launch_bounds__(kDiffThreads, 1)
+diff_attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_vt,
+                         const int* __restrict__ cu, const int* __restrict__ pstart, const int* __restrict__ kv_lens, __nv_bfloat16* __restrict__ out, int out_stride,
+                         int heads, int n_kv, float sl2, const WindowExt ext, const DiffOut diff, int* __restrict__ status) {
+  lg::pdl_prologue();
+  using C = DiffAttn<HD>;
+  constexpr uint32_t kTmemCols = 512, kColO = 256;
+  const int s = blockIdx.z, h = blockIdx.y, q0 = (int)(gridDim.x - 1 - blockIdx.x) * 128;
+  const int t0 = cu[s], len = cu[s + 1] - t0;
+  if (q0 >= len) return;  // before any barrier or TMEM allocation
+  const int kv_total = kv_lens[s], q_off = kv_total - len;
+  if (q_off < 0) {
+    if (threadIdx.x == 0 && status) atomicExch(status, 1);
+    return;
+  }
+  const int rep = heads / n_kv, kvh = h / rep, first_head = kvh * 2 * rep + h % rep, row_k = pstart[s];
+  const int kv_len = min(kv_total, q_off + q0 + 128), gap = ext.gap_keys(kv_total, len);
+  const int skip = max(ext.first(q_off + q0) - gap, 0) >> 7, nb = ((kv_len - gap + 127) >> 7) - skip;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+  extern __shared__ uint8_t smem_raw[];
+  const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* smem_gen = smem_raw + (smem_base - smem_u32(smem_raw));
+  constexpr int kBarOff = C::kQBytes + 2 * (C::kKBytes + C::kVBytes);
+  const uint32_t q_smem = smem_base, k_smem = q_smem + C::kQBytes, v_smem = k_smem + 2 * C::kKBytes, bars = smem_base + kBarOff;
+  auto bar = [&](int i) { return bars + 8u * (uint32_t)i; };
+  const uint32_t q_full = bar(0), k_full = bar(1), k_empty = bar(3), v_full = bar(5), v_empty = bar(7), s_full = bar(9), p_full = bar(11), o_done = bar(13);
+  uint8_t* bars_gen = smem_gen + kBarOff;
+  volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(bars_gen + 8 * kDiffBars);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars_gen + 8 * kDiffBars + 8);
+  float *inv_l = reinterpret_cast<float*>(bars_gen + 8 * kDiffBars + 16), *sums = inv_l + 2 * 128;   // [map][row]
+
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kDiffBars; ++i) mbar_init(bar(i), i == 11 || i == 12 ? 4u : 1u);  // p_full: one arrival per softmax warp
+    *abort_flag = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+    asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+  }
+  if (warp == 1) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_u32((const void*)tmem_slot)), "r"(kTmemCols) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      mbar_expect_tx(q_full, (uint32_t)C::kQBytes);
+#pragma unroll
+      for (int m = 0; m < 2; ++m) tma_load_2d(q_smem + m * kTileBytes, &map_q, q_full, (first_head + m * rep) * HD + (HD == 128 ? m * 64 : 0), t0 + q0);
+      for (int j = 0; j < nb; ++j) {
+        const uint32_t st = (uint32_t)j & 1u, phase = (uint32_t)(j >> 1) & 1u;
+        const int row = row_k + (j + skip) * 128;
+        if (!mbar_wait(k_empty + 8 * st, phase ^ 1u, abort_flag)) break;
+        mbar_expect_tx(k_full + 8 * st, (uint32_t)C::kKBytes);
+#pragma unroll
+        for (int i = 0; i < HD / 64; ++i) tma_load_2d(k_smem + st * C::kKBytes + i * kTileBytes, &map_k, k_full + 8 * st, kvh * HD + i * 64, row);
+        if (!mbar_wait(v_empty + 8 * st, phase ^ 1u, abort_flag)) break;
+        mbar_expect_tx(v_full + 8 * st, (uint32_t)C::kVBytes);
+        tma_load_2d(v_smem + st * C::kVBytes, &map_vt, v_full + 8 * st, row, kvh * HD);
+        tma_load_2d(v_smem + st * C::kVBytes + C::kVTile, &map_vt, v_full + 8 * st, row + 64, kvh * HD);
+      }
+    }
+  } else if (warp == 1) {
+    // The tensor pipe runs these in issue order: the next scores of a map never overwrite the P that its P V still reads, and
+    // "S_m(j) complete" implies "P_m V(j - 1) complete".
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = make_idesc<128>(), idesc_o = make_idesc<HD>();
+      auto scores = [&](int m, int j) {
+        const uint32_t k_tile = k_smem + ((uint32_t)j & 1u) * C::kKBytes + (HD == 128 ? (uint32_t)m * kTileBytes : 0u);
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk)
+          tc_mma_bf16(tmem_base + 128u * m, make_smem_desc(q_smem + m * kTileBytes) + (uint64_t)(2 * kk), make_smem_desc(k_tile) + (uint64_t)(2 * kk), idesc_s, kk ? 1u : 0u);
+        tc_commit(s_full + 8 * m);
+      };
+      bool ok = mbar_wait(q_full, 0u, abort_flag) && mbar_wait(k_full, 0u, abort_flag);
+      if (ok) {
+        tc_fence_after();
+        scores(0, 0);
+        scores(1, 0);
+        tc_commit(k_empty);
+      }
+      for (int j = 0; j < nb && ok; ++j) {
+        const uint32_t st = (uint32_t)j & 1u, next = st ^ 1u;
+        if (!mbar_wait(v_full + 8 * st, (uint32_t)(j >> 1) & 1u, abort_flag)) { ok = false; break; }
+        if (j + 1 < nb && !mbar_wait(k_full + 8 * next, (uint32_t)((j + 1) >> 1) & 1u, abort_flag)) { ok = false; break; }
+        for (int m = 0; m < 2; ++m) {
+          if (!mbar_wait(p_full + 8 * m, (uint32_t)j & 1u, abort_flag)) { ok = false; break; }
+          tc_fence_after();
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk) {
+            const uint64_t db = make_smem_desc(v_smem + st * C::kVBytes + (kk >> 2) * C::kVTile) + (uint64_t)(2 * (kk & 3));
+            tc_mma_bf16_ts(tmem_base + kColO + (uint32_t)(m * HD), tmem_base + 128u * m + 8u * kk, db, idesc_o, (j | kk) ? 1u : 0u);
+          }
+          if (m == 1) tc_commit(v_empty + 8 * st);
+          if (j + 1 < nb) scores(m, j + 1);
+        }
+        if (!ok) break;
+        if (j + 1 < nb) tc_commit(k_empty + 8 * next);
+        else tc_commit(o_done);
+      }
+    }
+  } else {
+    const int m = warp >= 6 ? 1 : 0, q = warp & 3, row = q * 32 + lane, at = q_off + q0 + row;
+    const uint32_t lane_off = (uint32_t)(q * 32) << 16;
+    const uint32_t t_s = tmem_base + lane_off + 128u * m, t_o = tmem_base + lane_off + kColO;
+    const int seen_from = ext.first(at);
+    float mx_run = -1e30f, l = 0.0f;
+    bool ok = true;
+    for (int j = 0; j < nb; ++j) {
+      if (!mbar_wait_warp(s_full + 8 * m, (uint32_t)j & 1u, abort_flag)) { ok = false; break; }
+      tc_fence_after();
+      const int base = (j + skip) * 128 + gap, lim = min(kv_len, at + 1) - base, lo = seen_from - base;  // keys [lo, lim) of the block
+      const bool full = lim >= 128 && lo <= 0;
+      float mx = -1e30f;
+#pragma unroll
+      for (int c2 = 0; c2 < 2; ++c2) {
+        uint32_t ra[32], rb[32];
+        tc_ld32(t_s + c2 * 64, ra);
+        tc_ld32(t_s + c2 * 64 + 32, rb);
+        tc_wait_ld();
+        if (full) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fmaxf(__uint_as_float(ra[i]), __uint_as_float(rb[i])));
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const int ka = c2 * 64 + i, kb = ka + 32;
+            if (ka < lim && ka >= lo) mx = fmaxf(mx, __uint_as_float(ra[i]));
+            if (kb < lim && kb >= lo) mx = fmaxf(mx, __uint_as_float(rb[i]));
+          }
+        }
+      }
+      const float cand = mx * sl2;   // the maximum moves when it would grow by more than 2^8
+      float alpha = 1.0f;
+      if (cand > mx_run + 8.0f) { alpha = fast_exp2(mx_run - cand); mx_run = cand; }
+      float sum = 0.0f;
+#pragma unroll
+      for (int c2 = 0; c2 < 2; ++c2) {
+        uint32_t ra[32], rb[32], v[32];
+        tc_ld32(t_s + c2 * 64, ra);
+        tc_ld32(t_s + c2 * 64 + 32, rb);
+        tc_wait_ld();
+        auto prob = [&](uint32_t raw, int key) {
+          const float e = fast_exp2(fmaf(__uint_as_float(raw), sl2, -mx_run));
+          return full || (key < lim && key >= lo) ? e : 0.0f;
+        };
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+          const int ka = c2 * 64 + i, kb = ka + 32;
+          const float a0 = prob(ra[i], ka), a1 = prob(ra[i + 1], ka + 1), b0 = prob(rb[i], kb), b1 = prob(rb[i + 1], kb + 1);
+          sum += (a0 + a1) + (b0 + b1);
+          v[i >> 1] = pack_bf16x2(a0, a1);
+          v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
+        }
+        tc_st32(t_s + c2 * 32, v);
+      }
+      l = l * alpha + sum;
+      if (j > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
+#pragma unroll
+        for (int c = 0; c < HD / 32; ++c) {
+          uint32_t r[32];
+          tc_ld32(t_o + m * HD + c * 32, r);
+          tc_wait_ld();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
+          tc_st32(t_o + m * HD + c * 32, r);
+        }
+      }
+      tc_wait_st();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_full + 8 * m);
+    }
+    ok = ok && mbar_wait_warp(o_done, 0u, abort_flag);
+    inv_l[m * 128 + row] = 1.0f / l;
+    asm volatile("bar.sync 1, 256;\n" ::: "memory");   // reached by all softmax warps whatever their waits returned
+    constexpr int kHalf = HD / 2;
+    float x[kHalf], ss = 0.0f;
+    if (ok) {
+      tc_fence_after();
+      const float i1 = inv_l[row], i2 = inv_l[128 + row] * diff.lambda;
+#pragma unroll
+      for (int c = 0; c < kHalf / 32; ++c) {
+        uint32_t ra[32], rb[32];
+        tc_ld32(t_o + m * kHalf + c * 32, ra);
+        tc_ld32(t_o + HD + m * kHalf + c * 32, rb);
+        tc_wait_ld();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          x[c * 32 + i] = __uint_as_float(ra[i]) * i1 - __uint_as_float(rb[i]) * i2;
+          ss = fmaf(x[c * 32 + i], x[c * 32 + i], ss);
+        }
+      }
+    }
+    sums[m * 128 + row] = ss;
+    asm volatile("bar.sync 1, 256;\n" ::: "memory");
+    if (ok && q0 + row < len) {
+      const float inv = diff.scale / sqrtf((sums[row] + sums[128 + row]) / (float)diff.v + diff.eps);
+      uint4* dst = reinterpret_cast<uint4*>(out + (size_t)(t0 + q0 + row) * (size_t)out_stride + h * HD + m * kHalf);
+#pragma unroll
+      for (int i = 0; i < kHalf; i += 8)
+        dst[i / 8] = make_uint4(pack_bf16x2(x[i] * inv, x[i + 1] * inv), pack_bf16x2(x[i + 2] * inv, x[i + 3] * inv), pack_bf16x2(x[i + 4] * inv, x[i + 5] * inv),
+                                pack_bf16x2(x[i + 6] * inv, x[i + 7] * inv));
+    }
+  }
+
+  // ---------------- teardown ----------------
+  __syncwarp();
+  if (*abort_flag) {
+    for (int i = 0; i < 2000; ++i) __nanosleep(1000);   // copies that may still be in flight land before the memory is released
+    if (threadIdx.x == 0 && status) atomicExch(status, 2 | (3 << 8));
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem_base), "r"(kTmemCols) : "memory");
+  }
+}
+
 }  // namespace
 
 namespace {
@@ -814,7 +1056,7 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
                                    const void* v_pool, const void* block_tables, int32_t max_blocks, int32_t n_pool_blocks, void* out,
                                    void* scratch, int32_t n_q_tokens, int32_t total_kv_tokens, int32_t n_seqs, int32_t max_q_len,
                                    int32_t max_kv_len, int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, bool turbo3, void* status,
-                                   void* stream, const ScoreExt* ext = nullptr, int score = kPlain, const WindowExt* win = nullptr, float scale = 0.0f) {
+                                   void* stream, const ScoreExt* ext = nullptr, int score = kPlain, const WindowExt* win = nullptr, float scale = 0.0f, const DiffOut* diff = nullptr) {
   const int D = head_dim;
   if (n_q_tokens < 0 || total_kv_tokens < 0 || n_seqs < 0 || max_q_len < 0 || max_kv_len < 0 || max_blocks <= 0 ||
       n_pool_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 || (D != 128 && D != 256 && !(D == 64 && (ext || win))) || (n_heads % n_kv_heads) ||
@@ -853,6 +1095,17 @@ static uint32_t launch_prefix_attn(const void* q, int32_t q_row_stride, const vo
     }
     uint32_t rc = lg::launch_status();
     if (rc) return rc;
+  }
+  if (diff) {  // n_heads counts both maps
+    const dim3 grid((max_q_len + 127) / 128, n_heads / 2, n_seqs);
+    auto go = [&](auto kern, size_t smem) -> uint32_t {
+      cudaError_t rc = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (rc != cudaSuccess) return (uint32_t)rc;
+      lg::launch(kern, grid, dim3(kDiffThreads), smem, s, map_q, map_k, map_vt, (const int*)cu_seqlens_q, (const int*)pstart, (const int*)kv_lens, (__nv_bfloat16*)out, win->ld_out,
+                 n_heads / 2, n_kv_heads, 1.4426950408889634f * scale, *win, *diff, (int*)status);
+      return lg::launch_status();
+    };
+    return D == 64 ? go(diff_attn_tcgen05_kernel<64>, DiffAttn<64>::kSmem) : go(diff_attn_tcgen05_kernel<128>, DiffAttn<128>::kSmem);
   }
   const float sl2 = win ? 1.4426950408889634f * scale : 1.4426950408889634f / sqrtf((float)D);
   const int ld_out = win ? win->ld_out : ext ? ext->ld_out : n_heads * D;
@@ -935,6 +1188,22 @@ uint32_t logismos_launch_window_attention_prefix_bf16(const void* q, int32_t ld_
   const WindowExt win = window_ext(window, ld_q, ld_out);
   return launch_prefix_attn(q, ld_q, cu_seqlens_q, kv_lens, k_pool, v_pool, block_tables, max_blocks, n_pool_blocks, out, scratch, n_q_tokens, total_keys, n_seqs,
                             max_q_len, max_keys, n_heads, n_kv_heads, head_dim, false, status, stream, nullptr, kPlain, &win, window->scale);
+}
+
+int32_t logismos_differential_has_prompts(int32_t head_dim) { return head_dim == 64 || head_dim == 128 ? 1 : 0; }
+
+uint32_t logismos_launch_differential_prefix_bf16(const void* q, int32_t ld_q, const void* cu_seqlens_q, const void* kv_lens, const void* k_pool, const void* v_pool,
+                                                  const void* block_tables, int32_t max_blocks, int32_t n_pool_blocks, void* out, int32_t ld_out, void* scratch,
+                                                  int32_t n_q_tokens, int32_t total_keys, int32_t n_seqs, int32_t max_q_len, int32_t max_keys, int32_t heads, int32_t n_kv_heads,
+                                                  int32_t head_dim, const lg_window_t* window, int32_t v, float lambda, float scale, float eps, void* status, void* stream) {
+  lg::LaunchScope launch_scope_;
+  if (heads <= 0 || n_kv_heads <= 0 || heads % n_kv_heads || !logismos_differential_has_prompts(head_dim) || !window_ok(window, 2 * heads) || window->gate || window->sink ||
+      window->keep_first || window->pool || v <= 0 || v > head_dim || (ld_out % 8) || ld_out < heads * head_dim)
+    return lg::kInvalidValue;
+  const WindowExt win = window_ext(window, ld_q, ld_out);
+  const DiffOut diff{lambda, scale, eps, v};
+  return launch_prefix_attn(q, ld_q, cu_seqlens_q, kv_lens, k_pool, v_pool, block_tables, max_blocks, n_pool_blocks, out, scratch, n_q_tokens, total_keys, n_seqs, max_q_len, max_keys,
+                            2 * heads, n_kv_heads, head_dim, false, status, stream, nullptr, kPlain, &win, window->scale, &diff);
 }
 
 uint32_t logismos_launch_varlen_attention_kv_tc_bf16(const void* q, int32_t q_row_stride, const void* cu_seqlens_q, const void* kv_lens,

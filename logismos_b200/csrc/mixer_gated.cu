@@ -127,6 +127,15 @@ void gate_up_rows(Mat& dst, int row0, const void* gate, const void* up, int firs
 
 }  // namespace
 
+void gathered_keys(const StepBatch& B, const lg_window_t& w, const PrefixRun& r, int* total, int* longest) {
+  *total = *longest = 0;
+  for (int k = r.s0; k < r.s1; ++k) {
+    const int n = logismos_window_view_keys(&w, B.pre_kv[k], B.newl[(size_t)(B.n_dec + k)]);
+    *total += n;
+    *longest = std::max(*longest, n);
+  }
+}
+
 uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int ld_q, int heads, int kv, int hd, void* out, int ld_out, cudaStream_t s, bool prompts_only) {
   const lg_mixer_config_t& c = m->cfg;
   StepBatch& B = m->batch;
@@ -147,12 +156,8 @@ uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int
   const size_t row0 = (size_t)B.n_dec;
   if (w.gate) w.gate = (const float*)w.gate + row0 * w.ld_gate;
   for (const PrefixRun& r : B.runs) {
-    int total = 0, longest = 0;
-    for (int k = r.s0; k < r.s1; ++k) {
-      const int n = logismos_window_view_keys(&w, B.pre_kv[k], B.newl[row0 + (size_t)k]);
-      total += n;
-      longest = std::max(longest, n);
-    }
+    int total, longest;
+    gathered_keys(B, w, r, &total, &longest);
     LG_TRY(logismos_launch_window_attention_prefix_bf16((const uint16_t*)q + row0 * ld_q, ld_q, m->dev(B.cu_pre) + r.s0, m->dev(B.pre_kv) + r.s0, L.kpool.p, L.vpool.p,
                                                         m->dev(B.tables) + (row0 + r.s0) * MB, MB, c.n_pool_blocks, (uint8_t*)out + row0 * ld_out * (w.out_f32 ? 4 : 2),
                                                         ld_out, m->attn_ws.p, T - B.n_dec, total, r.s1 - r.s0, r.max_q, longest, heads, kv, hd, &w, st, s), "attention");

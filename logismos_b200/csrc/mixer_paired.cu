@@ -67,6 +67,19 @@ uint32_t differential(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
     m->launches += 2;
   }
   if (T == alone) return 0;
+  if (!c.is_f32 && logismos_differential_has_prompts(L.Dh)) {
+    const size_t row0 = (size_t)alone;
+    for (const PrefixRun& r : B.runs) {
+      int total, longest;
+      gathered_keys(B, w, r, &total, &longest);
+      LG_TRY(logismos_launch_differential_prefix_bf16((const uint16_t*)m->qx.p + row0 * ld, ld, m->dev(B.cu_pre) + r.s0, m->dev(B.pre_kv) + r.s0, L.kpool.p, L.vpool.p,
+                                                      m->dev(B.tables) + (row0 + r.s0) * c.max_blocks_per_seq, c.max_blocks_per_seq, c.n_pool_blocks,
+                                                      (uint16_t*)m->act.p + row0 * L.Kout, L.Kout, m->attn_ws.p, T - alone, total, r.s1 - r.s0, r.max_q, longest, L.c.heads,
+                                                      L.c.kv_heads, L.Dh, &w, L.c.vdim, W.lambda, 1.0f - L.c.diff, c.norm_eps, m->status.p, s), "differential attention");
+      m->launches += 2;
+    }
+    return 0;
+  }
   if (uint32_t rc = window_attention(m, L, w, m->qx.p, ld, heads, L.c.kv_heads, L.Dh, m->maps_out.p, ld, s, true)) return rc;
   LG_TRY(logismos_launch_attention_difference((const float*)m->maps_out.p + (size_t)alone * ld, ld, (uint8_t*)m->act.p + (size_t)alone * L.Kout * (c.is_f32 ? 4 : 2), L.Kout, c.is_f32,
                                               T - alone, L.c.heads, L.c.kv_heads, L.c.vdim, L.Dh, W.lambda, 1.0f - L.c.diff, c.norm_eps, s), "difference");

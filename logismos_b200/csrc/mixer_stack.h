@@ -182,6 +182,8 @@ uint32_t run_gated_kinds(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s)
 // alone, where decode rows have a launch of their own)
 uint32_t window_attention(Mixer* m, MLayer& L, lg_window_t w, const void* q, int ld_q, int heads, int kv, int hd, void* out, int ld_out, cudaStream_t s,
                           bool prompts_only = false);
+// keys that a launch over a run of prompt sequences gathers: of all, and of the longest
+void gathered_keys(const StepBatch& B, const lg_window_t& w, const PrefixRun& r, int* total, int* longest);
 
 const char* check_paired_kinds(const lg_mixer_layer_config_t& y);
 void layout_paired_kinds(const Mixer* m, MLayer& L);

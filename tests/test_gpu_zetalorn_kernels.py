@@ -209,6 +209,47 @@ def test_differential_decode(H, G, D, d, v, size):
         close(host(out)[:, :H * D].reshape(n, H, D), want, 1e-2)
 
 
+@pytest.mark.parametrize("H,G,D,d,v,size,chunked", [(6, 3, 64, 22, 30, 20, 1), (20, 1, 64, 8, 8, 3, 1), (4, 1, 128, 64, 128, 700, 1), (2, 2, 128, 40, 100, 1, 1), (3, 1, 128, 64, 128, 130, 1),
+                                                      (4, 2, 64, 32, 64, 200, 0), (2, 1, 128, 50, 128, 0, 0)])
+def test_differential_prompts(H, G, D, d, v, size, chunked):
+    """Both maps in one pass; one pair of keys in sight stands out in the first map alone and another in the second."""
+    rng = np.random.default_rng(H + size)
+    lens, new = [2, 130, 300, 700, 523, 411, 1], [2, 130, 2, 300, 129, 17, 1]
+    c, n, half, lam, eps, T = Cache(rng, lens, G, D, D, v, False), len(lens), D // 2, 0.6, 1e-3, sum(new)
+    assert lib.logismos_differential_has_prompts(D) and not lib.logismos_differential_has_prompts(256)
+    q = padded(rng.standard_normal((T, H, 2, d)), half)
+    cu = np.concatenate([[0], np.cumsum(new)]).astype(np.int32)
+    for s in range(n):
+        maps = c.k[s].reshape(lens[s], G, 2, half)
+        for i in range(new[s]):
+            p = lens[s] - new[s] + i
+            first = (p - p % size if chunked else max(0, p - size + 1)) if size else 0
+            for m, j in ((0, first), (1, max(first, p - 1))):
+                q[cu[s] + i, 0, m, :d] += 1.5 * maps[j, 0, m, :d]
+    q = host(act(q, False))
+    wide = np.zeros((T, H, 2, 2, half))
+    wide[:, :, 0, 0], wide[:, :, 1, 1] = q[:, :, 0], q[:, :, 1]
+    qd, scale = act(by_map(wide.reshape(T, H, 2, D), G).reshape(T, -1), False), 1.0 / np.sqrt(d)
+    want = np.zeros((T, H, D))
+    for s in range(n):
+        maps, rows = c.k[s].reshape(lens[s], G, 2, half), np.arange(lens[s] - new[s], lens[s])
+        mask = (R.chunk_mask(lens[s], size) if chunked else R.window_mask(lens[s], size or lens[s]))[rows]
+        a = [R.attend(q[cu[s]:cu[s + 1], :, m], maps[:, :, m], c.v[s], scale, mask) for m in range(2)]
+        want[cu[s]:cu[s + 1], :, :v] = R.difference(a[0][..., :v], a[1][..., :v], lam, 0.2, eps)
+    w, st = c.window(scale, size, chunked), status()
+    keys = [lib.logismos_window_view_keys(C.byref(w), x, y) for x, y in zip(lens, new)]
+    scr = torch.empty(lib.logismos_paged_prefix_attention_scratch_bytes(sum(keys), n, G, D), dtype=torch.uint8, device=DEV)
+    scr.fill_(255)
+    out, keep = act(np.full((T, H * D + 8), 5.0), False), [ints(cu), ints(lens)]
+    check(lib.logismos_launch_differential_prefix_bf16(P(qd), 2 * H * D, P(keep[0]), P(keep[1]), P(c.kp), P(c.vp), P(c.tables), c.mb, c.nb, P(out), H * D + 8, P(scr), T, sum(keys), n, max(new),
+                                                       max(keys), H, G, D, C.byref(w), v, lam, 0.8, eps, P(st), stream()), "prefix")
+    torch.cuda.synchronize()
+    assert st.item() == 0
+    got = host(out)
+    close(got[:, :H * D].reshape(T, H, D), want, 1e-2)
+    assert (got[:, H * D:] == 5.0).all()
+
+
 @FP32
 @pytest.mark.parametrize("rows,H,G,v,vp_", [(1, 1, 1, 9, 64), (37, 6, 2, 30, 64), (300, 4, 4, 128, 128), (9, 20, 1, 200, 256)])
 def test_difference_of_two_attentions(rows, H, G, v, vp_, fp32):
