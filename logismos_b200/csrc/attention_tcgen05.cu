@@ -374,6 +374,49 @@ LG_DEVINL float bounded_block(uint32_t t_s, const ScoreExt& ext, const float* wi
   return sum;
 }
 
+// ---- softmax of a block whose 128 scores per row are held in registers: one read of TMEM, one wait ---------------------------
+LG_DEVINL void load_scores(uint32_t t_s, uint32_t (&r)[4][32]) {
+#pragma unroll
+  for (int w = 0; w < 4; ++w) tc_ld32(t_s + 32 * w, r[w]);
+  tc_wait_ld();
+}
+LG_DEVINL uint32_t bits_below(int n) { return n >= 32 ? 0xffffffffu : n <= 0 ? 0u : (1u << n) - 1u; }
+// scores whose bit is not set become -inf
+LG_DEVINL void hide(uint32_t (&r)[32], uint32_t seen) {
+#pragma unroll
+  for (int i = 0; i < 32; ++i) r[i] = seen & (1u << i) ? r[i] : 0xff800000u;
+}
+// The running maximum m (log2 units) moves when it would grow by more than 2^8, so that what it scales is rescaled by alpha far less
+// often; P, rounded, takes the place of S. Returns the row's sum. Independent chains: a scheduler has one or two warps to issue from.
+LG_DEVINL float softmax_block(uint32_t t_s, const uint32_t (&r)[4][32], float sl2, float& m, float& alpha) {
+  float mx[4];
+#pragma unroll
+  for (int w = 0; w < 4; ++w) mx[w] = __uint_as_float(r[w][0]);
+#pragma unroll
+  for (int i = 1; i < 32; ++i)
+#pragma unroll
+    for (int w = 0; w < 4; ++w) mx[w] = fmaxf(mx[w], __uint_as_float(r[w][i]));
+  const float cand = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * sl2;
+  alpha = 1.0f;
+  if (cand > m + 8.0f) { alpha = fast_exp2(m - cand); m = cand; }
+  float sum[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {  // columns [32 h, 32 h + 32) hold keys [64 h, 64 h + 64)
+    uint32_t v[32];
+#pragma unroll
+    for (int i = 0; i < 32; i += 2)
+#pragma unroll
+      for (int w = 0; w < 2; ++w) {
+        const float a = fast_exp2(fmaf(__uint_as_float(r[2 * h + w][i]), sl2, -m)), b = fast_exp2(fmaf(__uint_as_float(r[2 * h + w][i + 1]), sl2, -m));
+        sum[w] += a;
+        sum[2 + w] += b;
+        v[16 * w + (i >> 1)] = pack_bf16x2(a, b);
+      }
+    tc_st32(t_s + 32 * h, v);
+  }
+  return (sum[0] + sum[1]) + (sum[2] + sum[3]);
+}
+
 template <bool CAUSAL, int HD, int SCORE = kPlain>
 __global__ void __launch_bounds__(192, HD <= 128 ? 2 : 1)
 attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -548,7 +591,6 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         }
         full = lim >= 128 && (lo <= 0 || keep >= 128);
       }
-      auto seen = [&](int key) { return key < lim && (SCORE != kWindowed || key >= lo || key < keep); };
       if constexpr (SCORE == kBounded || SCORE == kPoly) {
         constexpr int S = SCORE == kPoly ? kPoly : kBounded;
         // every lane of a warp takes the same branch: TMEM accesses are warp-wide
@@ -561,43 +603,38 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         if (lane == 0) mbar_arrive(p_full);
         continue;
       }
-      float mx = -1e30f;
+      float alpha = 1.0f, sum = 0.0f;
+      if constexpr (!BIASED) {
+        uint32_t r[4][32];
+        load_scores(t_s, r);
+        if (!__all_sync(0xffffffffu, full)) {
 #pragma unroll
-      for (int c2 = 0; c2 < 2; ++c2) {
-        uint32_t ra[32], rb[32];
-        tc_ld32(t_s + c2 * 64, ra);
-        tc_ld32(t_s + c2 * 64 + 32, rb);
-        tc_wait_ld();
-        if (SCORE == kBiased) {
+          for (int w = 0; w < 4; ++w) hide(r[w], bits_below(lim - 32 * w) & (SCORE == kWindowed ? ~bits_below(lo - 32 * w) | bits_below(keep - 32 * w) : 0xffffffffu));
+        }
+        sum = softmax_block(t_s, r, sl2, m, alpha);
+      } else {
+        float mx = -1e30f;
+#pragma unroll
+        for (int c2 = 0; c2 < 2; ++c2) {
+          uint32_t ra[32], rb[32];
+          tc_ld32(t_s + c2 * 64, ra);
+          tc_ld32(t_s + c2 * 64 + 32, rb);
+          tc_wait_ld();
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             if (c2 * 64 + i < lim) mx = fmaxf(mx, score(ra[i], c2 * 64 + i));
             if (c2 * 64 + 32 + i < lim) mx = fmaxf(mx, score(rb[i], c2 * 64 + 32 + i));
           }
-        } else if (full) {
-#pragma unroll
-          for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fmaxf(__uint_as_float(ra[i]), __uint_as_float(rb[i])));
-        } else {
-#pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            if (seen(c2 * 64 + i)) mx = fmaxf(mx, __uint_as_float(ra[i]));
-            if (seen(c2 * 64 + 32 + i)) mx = fmaxf(mx, __uint_as_float(rb[i]));
-          }
         }
-      }
-      // The maximum only moves when it would grow by more than 2^8: P then stays below 256 (exact
-      // enough in bf16, summed in fp32) and O is rescaled far less often.
-      const float cand = BIASED ? mx : mx * sl2;
-      float alpha = 1.0f;
-      if (cand > m + 8.0f) { alpha = fast_exp2(m - cand); m = cand; }
-      float sum = 0.0f;
+        // The maximum only moves when it would grow by more than 2^8: P then stays below 256 (exact enough in bf16, summed in
+        // fp32) and O is rescaled far less often.
+        if (mx > m + 8.0f) { alpha = fast_exp2(m - mx); m = mx; }
 #pragma unroll
-      for (int c2 = 0; c2 < 2; ++c2) {
-        uint32_t ra[32], rb[32], v[32];
-        tc_ld32(t_s + c2 * 64, ra);
-        tc_ld32(t_s + c2 * 64 + 32, rb);
-        tc_wait_ld();
-        if (BIASED) {
+        for (int c2 = 0; c2 < 2; ++c2) {
+          uint32_t ra[32], rb[32], v[32];
+          tc_ld32(t_s + c2 * 64, ra);
+          tc_ld32(t_s + c2 * 64 + 32, rb);
+          tc_wait_ld();
           auto prob = [&](uint32_t raw, int key) {
             const float e = fast_exp2(score(raw, key) - m);
             return full || key < lim ? e : 0.0f;
@@ -610,31 +647,10 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             v[i >> 1] = pack_bf16x2(a0, a1);
             v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
           }
-        } else if (full) {
-#pragma unroll
-          for (int i = 0; i < 32; i += 2) {
-            const float a0 = fast_exp2(fmaf(__uint_as_float(ra[i]), sl2, -m)), a1 = fast_exp2(fmaf(__uint_as_float(ra[i + 1]), sl2, -m));
-            const float b0 = fast_exp2(fmaf(__uint_as_float(rb[i]), sl2, -m)), b1 = fast_exp2(fmaf(__uint_as_float(rb[i + 1]), sl2, -m));
-            sum += (a0 + a1) + (b0 + b1);
-            v[i >> 1] = pack_bf16x2(a0, a1);
-            v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
-          }
-        } else {
-#pragma unroll
-          for (int i = 0; i < 32; i += 2) {
-            const int ka = c2 * 64 + i, kb = ka + 32;
-            const float a0 = seen(ka) ? fast_exp2(fmaf(__uint_as_float(ra[i]), sl2, -m)) : 0.0f;
-            const float a1 = seen(ka + 1) ? fast_exp2(fmaf(__uint_as_float(ra[i + 1]), sl2, -m)) : 0.0f;
-            const float b0 = seen(kb) ? fast_exp2(fmaf(__uint_as_float(rb[i]), sl2, -m)) : 0.0f;
-            const float b1 = seen(kb + 1) ? fast_exp2(fmaf(__uint_as_float(rb[i + 1]), sl2, -m)) : 0.0f;
-            sum += (a0 + a1) + (b0 + b1);
-            v[i >> 1] = pack_bf16x2(a0, a1);
-            v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
-          }
+          // P takes the place of S: columns [32 c2, 32 c2 + 32) hold keys [64 c2, 64 c2 + 64); the S values
+          // they replace (keys [32 c2, 32 c2 + 32)) were read in this or the previous half
+          tc_st32(t_s + c2 * 32, v);
         }
-        // P takes the place of S: columns [32 c2, 32 c2 + 32) hold keys [64 c2, 64 c2 + 64); the S values
-        // they replace (keys [32 c2, 32 c2 + 32)) were read in this or the previous half
-        tc_st32(t_s + c2 * 32, v);
       }
       l = l * alpha + sum;
       // S(j) complete means PV(j-1) is complete: O may be rescaled in place
@@ -854,50 +870,14 @@ diff_attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       if (!mbar_wait_warp(s_full + 8 * m, (uint32_t)j & 1u, abort_flag)) { ok = false; break; }
       tc_fence_after();
       const int base = (j + skip) * 128 + gap, lim = min(kv_len, at + 1) - base, lo = seen_from - base;  // keys [lo, lim) of the block
-      const bool full = lim >= 128 && lo <= 0;
-      float mx = -1e30f;
+      uint32_t r[4][32];
+      load_scores(t_s, r);
+      if (!__all_sync(0xffffffffu, lim >= 128 && lo <= 0)) {
 #pragma unroll
-      for (int c2 = 0; c2 < 2; ++c2) {
-        uint32_t ra[32], rb[32];
-        tc_ld32(t_s + c2 * 64, ra);
-        tc_ld32(t_s + c2 * 64 + 32, rb);
-        tc_wait_ld();
-        if (full) {
-#pragma unroll
-          for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fmaxf(__uint_as_float(ra[i]), __uint_as_float(rb[i])));
-        } else {
-#pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const int ka = c2 * 64 + i, kb = ka + 32;
-            if (ka < lim && ka >= lo) mx = fmaxf(mx, __uint_as_float(ra[i]));
-            if (kb < lim && kb >= lo) mx = fmaxf(mx, __uint_as_float(rb[i]));
-          }
-        }
+        for (int w = 0; w < 4; ++w) hide(r[w], bits_below(lim - 32 * w) & ~bits_below(lo - 32 * w));
       }
-      const float cand = mx * sl2;   // the maximum moves when it would grow by more than 2^8
-      float alpha = 1.0f;
-      if (cand > mx_run + 8.0f) { alpha = fast_exp2(mx_run - cand); mx_run = cand; }
-      float sum = 0.0f;
-#pragma unroll
-      for (int c2 = 0; c2 < 2; ++c2) {
-        uint32_t ra[32], rb[32], v[32];
-        tc_ld32(t_s + c2 * 64, ra);
-        tc_ld32(t_s + c2 * 64 + 32, rb);
-        tc_wait_ld();
-        auto prob = [&](uint32_t raw, int key) {
-          const float e = fast_exp2(fmaf(__uint_as_float(raw), sl2, -mx_run));
-          return full || (key < lim && key >= lo) ? e : 0.0f;
-        };
-#pragma unroll
-        for (int i = 0; i < 32; i += 2) {
-          const int ka = c2 * 64 + i, kb = ka + 32;
-          const float a0 = prob(ra[i], ka), a1 = prob(ra[i + 1], ka + 1), b0 = prob(rb[i], kb), b1 = prob(rb[i + 1], kb + 1);
-          sum += (a0 + a1) + (b0 + b1);
-          v[i >> 1] = pack_bf16x2(a0, a1);
-          v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
-        }
-        tc_st32(t_s + c2 * 32, v);
-      }
+      float alpha;
+      const float sum = softmax_block(t_s, r, sl2, mx_run, alpha);
       l = l * alpha + sum;
       if (j > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
 #pragma unroll
