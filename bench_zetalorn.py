@@ -362,7 +362,9 @@ def kernel_table(z, peaks, T=4096, ctx=8192, batches=(8, 64)):
     prs, lst, ly = [bf(T, 2 * kw + 2 * vw) for _ in range(copies(4 * T * (kw + vw)))], zf(nq, lh, lk, lv), bf(T, vw)
     la = [linear_args(q, lst, slots, cu, ly) for q in prs]
     rec_b, rec_f = T * (4.0 * kw + 4.0 * vw), T * lh * (4.0 * lk * lv + 64.0 * (lk + lv))
-    add(ph, "linear attention", [lambda s, a=a: lib.logismos_launch_ssd_chunked_bf16(Y(a), nq, s) for a in la], rec_b, rec_f, "gated linear attention")
+    entries = lib.logismos_ssd_segments(T, nq, 1024, lh)
+    seg = torch.empty(max(16, lib.logismos_ssd_scratch_bytes(entries, lh, lk, lv)), dtype=torch.uint8, device=dev)
+    add(ph, "linear attention", [lambda s, a=a: lib.logismos_launch_ssd_segmented_bf16(Y(a), nq, 1024, P(seg), entries, s) for a in la], rec_b, rec_f, "gated linear attention")
     gq, zz, go = [bf(T, 2 * kw + 2 * vw) for _ in range(2)], rf(T, kw) + 2.0, bf(T, vw)
     ga = [gla_args(q, zz, None, None, lst, slots, cu, go) for q in gq]
     add(ph, "= gated linear attention", [lambda s, a=a: lib.logismos_launch_time_mix_chunked_bf16(Y(a), nq, s) for a in ga], T * (8.0 * kw + 6.0 * vw), T * lh * (4.0 * lk * lv + 32.0 * (lk + lv)))

@@ -828,6 +828,13 @@ uint32_t logismos_launch_ssd_step(const lg_ssd_t* args, int32_t n_seqs, int32_t 
 /* Prompts: the recurrence 64 tokens at a time on the tensor cores (np 32 .. 128, vp <= 128). */
 int32_t logismos_ssd_has_chunked(int32_t np, int32_t vp);
 uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* args, int32_t n_seqs, void* stream);
+/* The same with sequences cut in segments that run side by side, for few heads and long prompts: entries = logismos_ssd_segments
+ * of the step's prompt rows (0: not worth it, the launch above), scratch of logismos_ssd_scratch_bytes, longest >= every
+ * sequence. */
+int32_t logismos_ssd_segments(int32_t rows, int32_t n_seqs, int32_t longest, int32_t heads);
+size_t logismos_ssd_scratch_bytes(int32_t entries, int32_t heads, int32_t np, int32_t vp);
+uint32_t logismos_launch_ssd_segmented_bf16(const lg_ssd_t* args, int32_t n_seqs, int32_t longest, void* scratch, int32_t entries,
+                                            void* stream);
 /* out = y silu(z), divided in `parts` equal parts of the heads * v true channels by each part's root mean square,
  * times gain. Rows are laid out [heads][vp]. */
 uint32_t logismos_launch_gated_group_norm(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32,

@@ -166,6 +166,7 @@ def _declare(l, partial=False):
         "logismos_launch_ssd_conv": [vp, vp, i32, i32, i32, i32, vp],
         "logismos_launch_ssd_chunked_bf16": [vp, i32, vp],
         "logismos_launch_gated_group_norm": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp],
+        "logismos_launch_ssd_segmented_bf16": [vp, i32, i32, vp, i32, vp],
         "logismos_launch_norm_gate": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp],
         "logismos_launch_head_norm_store": [vp, i32, vp, vp],
         "logismos_launch_pool_blocks": [vp, i32, vp, vp],
@@ -240,6 +241,8 @@ def _declare(l, partial=False):
         "lg_latent_logits_device": ([vp], vp),
         "logismos_time_mix_has_chunked": ([i32, i32], i32),
         "logismos_ssd_has_chunked": ([i32, i32], i32),
+        "logismos_ssd_segments": ([i32, i32, i32, i32], i32),
+        "logismos_ssd_scratch_bytes": ([i32, i32, i32, i32], sz),
         "lg_mixer_launches_last_step": ([vp], i32),
         "lg_mixer_device_status": ([vp], i32),
         "lg_mixer_destroy": ([vp], None),

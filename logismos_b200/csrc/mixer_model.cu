@@ -581,9 +581,10 @@ uint32_t lg_mixer_create(int32_t device, const lg_mixer_config_t* cfg, const lg_
   m->acc_bytes = branches * acc_rows * Hp * 4;
   m->raw_acc_bytes = c.is_f32 ? 0 : acc_rows * z.raw * 4;
   m->route_acc_bytes = c.is_f32 ? 0 : T * z.route * 4;
+  m->segment_bytes = z.segments;
   m->counts_bytes = z.groups ? (z.groups + 1) * 4 : 0;  // the last one counts the router's finished tokens
   ok = ok && m->x.alloc(T * Hp * 4) && zeroed(m->h, copies * T * Hp * esz) && zeroed(m->proj, T * z.proj * esz) && m->tail.alloc(T * z.tail * 4) &&
-       zeroed(m->act, T * z.act * esz) && zeroed(m->ffb, T * z.ff * esz) && zeroed(m->xbc, T * z.xbc * esz) && m->y.alloc(branches * T * Hp * 4) && zeroed(m->qx, T * z.maps * esz) && m->maps_out.alloc(T * z.maps * 4) && m->y_acc.alloc(m->acc_bytes) && m->raw_acc.alloc(m->raw_acc_bytes) &&
+       zeroed(m->act, T * z.act * esz) && zeroed(m->ffb, T * z.ff * esz) && zeroed(m->xbc, T * z.xbc * esz) && m->y.alloc(branches * T * Hp * 4) && zeroed(m->qx, T * z.maps * esz) && m->maps_out.alloc(T * z.maps * 4) && m->segments.alloc(z.segments) && m->y_acc.alloc(m->acc_bytes) && m->raw_acc.alloc(m->raw_acc_bytes) &&
        m->last.alloc((size_t)c.max_out_rows * Hp * esz) && m->logits.alloc((size_t)c.max_out_rows * c.vocab * 4) && m->tokens.alloc((size_t)c.max_out_rows * 4) &&
        m->status.alloc(4) && (!c.keep_layers || m->hist.alloc((size_t)(c.n_layers + 1) * T * Hp * 4));
   if (!c.is_f32)
@@ -669,7 +670,7 @@ void lg_mixer_destroy(void* model) {
                  &m->act, &m->ffb, &m->y, &m->y_acc, &m->hist, &m->last, &m->logits, &m->tokens, &m->status, &m->attn_ws, &m->dec_scratch, &m->dev_batch, &m->raw_acc,
                  &m->cq, &m->gate, &m->qlat, &m->olat, &m->lat, &m->kbuf, &m->vt, &m->kv_start, &m->route, &m->route_acc, &m->pair_w, &m->pair_row, &m->pair_expert,
                  &m->identity, &m->offsets, &m->row_token, &m->counts, &m->tiles, &m->gathered, &m->expert_rows,
-                 &m->loop_step, &m->qx, &m->maps_out};
+                 &m->loop_step, &m->qx, &m->maps_out, &m->segments};
   for (Buf* b : bufs) b->release();
   for (MWeights& W : m->weights) W.release();
   for (MLayer& L : m->layers) {

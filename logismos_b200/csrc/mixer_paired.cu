@@ -104,8 +104,7 @@ uint32_t linear_attention(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s
   }
   if (chunked) {
     a.state_slots = m->dev(B.state) + B.n_dec; a.fresh = m->dev(B.fresh) + B.n_dec; a.cu = m->dev(B.cu) + B.n_dec;
-    LG_TRY(logismos_launch_ssd_chunked_bf16(&a, B.n_pre, s), "linear attention (prompts)");
-    m->launches += 1;
+    LG_TRY(prompt_recurrence(m, &a, s), "linear attention (prompts)");
   }
   const uint8_t* gate = (const uint8_t*)m->proj.p + (size_t)(L.off_right + L.channels) * esz;
   LG_TRY(logismos_launch_norm_gate(m->ffb.p, inner, gate, P, W.gain.p, (uint8_t*)m->act.p + (size_t)L.Kleft * esz, L.Kout, f32, B.T, L.c.lin_heads, L.c.lin_vdim, L.Vp,
@@ -242,6 +241,7 @@ bool alloc_paired_kinds(Mixer* m, MLayer& L, Sizes& z) {
   }
   if (L.c.kind == LG_MIXER_PAIR) {
     grow(z.ff, (size_t)L.c.lin_heads * L.Vp);
+    size_prompt_recurrence(m, L.c.lin_heads, L.Np, L.Vp, z);
     ok = ok && zeroed(L.state, (size_t)c.n_state_slots * L.c.lin_heads * L.Np * L.Vp * 4);
   }
   return ok;

@@ -30,13 +30,27 @@ uint32_t run_ssd(Mixer* m, MLayer& L, const MWeights& W, cudaStream_t s) {
   }
   if (chunked) {
     a.state_slots = m->dev(B.state) + B.n_dec; a.fresh = m->dev(B.fresh) + B.n_dec; a.phase = m->dev(B.phase) + B.n_dec; a.cu = m->dev(B.cu) + B.n_dec;
-    LG_TRY(logismos_launch_ssd_chunked_bf16(&a, B.n_pre, s), "state-space recurrence (prompts)");
-    m->launches += 1;
+    LG_TRY(prompt_recurrence(m, &a, s), "state-space recurrence (prompts)");
   }
   LG_TRY(logismos_launch_gated_group_norm(m->ffb.p, inner, m->proj.p, L.groups.n_main, W.gain.p, m->act.p, L.Kout, f32, T, L.c.ssd_heads, L.c.ssd_vdim, L.Vp,
                                           L.c.ssd_norm_groups, c.norm_eps, s), "gate and norm");
   m->launches += 1;
   return 0;
+}
+
+uint32_t prompt_recurrence(Mixer* m, lg_ssd_t* a, cudaStream_t s) {
+  const StepBatch& B = m->batch;
+  int entries = logismos_ssd_segments(B.T - B.n_dec, B.n_pre, B.max_pre_len, a->heads);
+  if (logismos_ssd_scratch_bytes(entries, a->heads, a->np, a->vp) > m->segment_bytes) entries = 0;
+  m->launches += entries > 0 ? 3 : 1;
+  return logismos_launch_ssd_segmented_bf16(a, B.n_pre, B.max_pre_len, m->segments.p, entries, s);
+}
+
+// room for a step of one long prompt, and of as many as are still cut
+void size_prompt_recurrence(const Mixer* m, int heads, int np, int vp, Sizes& z) {
+  if (m->cfg.is_f32 || !logismos_ssd_has_chunked(np, vp)) return;
+  const int T = m->cfg.max_step_tokens;
+  for (int n = 1; n <= m->cfg.max_step_seqs; ++n) grow(z.segments, logismos_ssd_scratch_bytes(logismos_ssd_segments(T, n, T, heads), heads, np, vp));
 }
 
 namespace {
@@ -252,6 +266,7 @@ bool alloc_parallel_kinds(Mixer* m, MLayer& L, Sizes& z) {
   if (L.c.kind == LG_MIXER_SSD) {
     grow(z.ff, (size_t)L.c.ssd_heads * L.Vp);
     grow(z.xbc, (size_t)L.channels);
+    size_prompt_recurrence(m, L.c.ssd_heads, L.Np, L.Vp, z);
     return zeroed(L.state, slots * L.c.ssd_heads * L.Np * L.Vp * 4) && zeroed(L.conv_state, slots * 2 * (L.c.ssd_taps - 1) * L.channels * 4);
   }
   const size_t pool = (size_t)c.n_pool_blocks * kKvBlock * L.c.kv_heads * L.Dh * (c.is_f32 ? 4 : 2), cap_tokens = std::max(MB * kKvBlock, T);

@@ -96,6 +96,7 @@ struct Mixer {
   Buf x, h, proj, tail, low2, z, xbc, act, ffb, y, y_acc, hist, last, logits, tokens, status, attn_ws, dec_scratch, dev_batch;
   Buf raw_acc;                          // sums of input projections over slices of k
   Buf cq, gate, qlat, olat, lat, kbuf, vt, kv_start;                                                      // latent attention
+  Buf segments;                         // scalar-decay recurrences of long prompts
   Buf qx, maps_out;                     // differential attention: queries of both maps, outputs of both (fp32)
   Buf route, route_acc, pair_w, pair_row, pair_expert, identity, offsets, row_token, counts, tiles, gathered, expert_rows;  // mixture
   StepBatch batch;
@@ -106,7 +107,7 @@ struct Mixer {
   // `y_acc`, `raw_acc`, `route_acc` and `counts` are all zero between their uses (the kernel that reads them zeroes them); a
   // step that failed part-way may have left sums there, so the next one clears them
   bool acc_dirty = true, ready = false;
-  size_t acc_bytes = 0, raw_acc_bytes = 0, route_acc_bytes = 0, counts_bytes = 0;
+  size_t acc_bytes = 0, raw_acc_bytes = 0, route_acc_bytes = 0, counts_bytes = 0, segment_bytes = 0;
   template <typename T> T* dev(T* host) const { return (T*)((uint8_t*)dev_batch.p + ((uint8_t*)host - batch.pinned)); }
   bool accumulates(int rows) const { return !cfg.is_f32 && rows <= kAccRows && !logismos_get_deterministic(); }
 };
@@ -117,6 +118,7 @@ struct Sizes {
   size_t raw = 0;                                                                                    // of summed input projections
   size_t cq = 0, heads = 0, lat_q = 0, lat = 0, lat_heads = 0;                             // latent attention
   size_t route = 0, pairs = 0, top = 0, groups = 0, expert_ff = 0;                                  // mixture
+  size_t segments = 0;                                                                               // bytes
   size_t maps = 0;                                                                                   // differential attention
 };
 inline void grow(size_t& a, size_t b) { if (b > a) a = b; }
@@ -149,6 +151,9 @@ uint32_t head_linear(Mixer* m, const void* a, int lda, const Buf& w, int heads, 
 uint32_t projections(Mixer* m, const MLayer& L, const MWeights& W, bool tail_parts, cudaStream_t s);
 // one grouped projection of the step's rows of h (n columns in all) to m->proj
 uint32_t grouped_projection(Mixer* m, const Buf& w, int n, const lg_linear_groups_t& g, cudaStream_t s);
+// a scalar-decay recurrence over the step's prompt sequences (args: theirs), cut in segments where that pays
+uint32_t prompt_recurrence(Mixer* m, lg_ssd_t* args, cudaStream_t s);
+void size_prompt_recurrence(const Mixer* m, int heads, int np, int vp, Sizes& z);
 // whether a grouped projection is summed over slices of k at this number of rows
 bool splits_projections(const lg_linear_groups_t& g, int n, int rows);
 bool zeroed(Buf& b, size_t bytes);

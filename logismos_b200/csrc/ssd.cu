@@ -16,6 +16,8 @@
 //   S <- exp(c_last) S + sum_j B_j (dt_j exp(c_last - c_j) x_j)^T
 // The products run on mma.sync with bf16 operands: B, C and x are bf16 already; the state, P and the weighted x go
 // in as a rounded part and a remainder (two products), so that what is fp32 keeps about 16 bits; sums are fp32.
+// Long prompts of few heads are cut in segments that run at once: every segment's own state from zero and its decay, a scan
+// over the segments of a sequence, then the segments' outputs from the states that they start with.
 #include "common.cuh"
 #include "logismos_kernels.h"
 #include "recurrent.cuh"
@@ -202,17 +204,28 @@ constexpr int kPitchP = kChunk * 2 + 16;
 inline size_t ssd_chunk_smem(int np, int vp) {
   return (size_t)kChunk * (2 * (2 * (2 * np + 16) + 2 * vp + 16) + 2 * kPitchP) + 4 * kChunk * 4;
 }
-template <int NP, bool FIXED>
+// PART: whole sequences, or segments' states (all but a sequence's last), or segments' outputs. The segments of a sequence have
+// consecutive entries of the scratch (state they start with, decay of the segment before them).
+enum { kWhole = 0, kStates = 1, kOutputs = 2 };
+constexpr int kSegment = 256;
+struct Segments {
+  float* state;   // [entries][heads][np][vp]
+  float* decay;   // [entries][heads], log2
+};
+LG_DEVINL int first_entry(const int* cu, int seq) { return (cu[seq] - cu[0]) / kSegment + seq; }
+
+template <int NP, bool FIXED, int PART>
 __global__ void __launch_bounds__(512)
-ssd_chunk_kernel(SsdArgs p) {
+ssd_chunk_kernel(SsdArgs p, Segments segs) {
   lg::pdl_prologue();
   constexpr int NT = NP / 16, kPitchN = NP * 2 + 16;
   extern __shared__ __align__(16) uint8_t smem[];
   const int vp = p.vp, pitch_v = vp * 2 + 16;
   const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
   const int g = lane >> 2, t = lane & 3, v0 = 8 * warp;
-  const int t0 = p.cu[seq], t1 = p.cu[seq + 1];
-  if (t1 <= t0) return;
+  const int t0 = p.cu[seq] + (PART == kWhole ? 0 : (int)blockIdx.z * kSegment), end = p.cu[seq + 1], t1 = PART == kWhole ? end : min(end, t0 + kSegment);
+  if (t1 <= t0 || (PART == kStates && t1 == end)) return;
+  const int entry = PART == kWhole ? 0 : first_entry(p.cu, seq) + (int)blockIdx.z;
   const int group = head / (p.heads / p.groups), inner = p.heads * vp;
   uint8_t *Bt = smem, *Ct = Bt + 2 * kChunk * kPitchN, *Xt = Ct + 2 * kChunk * kPitchN, *Ph = Xt + 2 * kChunk * pitch_v, *Pl = Ph + kChunk * kPitchP;
   float *cums = reinterpret_cast<float*>(Pl + kChunk * kPitchP), *dtss = cums + 2 * kChunk;
@@ -225,16 +238,17 @@ ssd_chunk_kernel(SsdArgs p) {
 #pragma unroll
   for (int m = 0; m < NT; ++m) {
     float2 a = make_float2(0.f, 0.f), b = a;
-    if (!p.fresh[seq]) {
-      a = *reinterpret_cast<const float2*>(st + (size_t)(16 * m + g) * vp + v0 + 2 * t);
-      b = *reinterpret_cast<const float2*>(st + (size_t)(16 * m + g + 8) * vp + v0 + 2 * t);
+    const float* from = PART == kOutputs ? segs.state + ((size_t)entry * p.heads + head) * NP * vp : st;
+    if (PART == kOutputs || (PART == kWhole && !p.fresh[seq])) {
+      a = *reinterpret_cast<const float2*>(from + (size_t)(16 * m + g) * vp + v0 + 2 * t);
+      b = *reinterpret_cast<const float2*>(from + (size_t)(16 * m + g + 8) * vp + v0 + 2 * t);
     }
     S[m][0] = a.x; S[m][1] = a.y; S[m][2] = b.x; S[m][3] = b.y;
   }
   auto stage = [&](int tb, int buf) {
     const int n = min(kChunk, t1 - tb);
     stage_tile(Bt + buf * kChunk * kPitchN, kPitchN, bs + (int64_t)tb * p.ld_xbc, p.ld_xbc, n, NP);
-    stage_tile(Ct + buf * kChunk * kPitchN, kPitchN, cs + (int64_t)tb * p.ld_xbc, p.ld_xbc, n, NP);
+    if (PART != kStates) stage_tile(Ct + buf * kChunk * kPitchN, kPitchN, cs + (int64_t)tb * p.ld_xbc, p.ld_xbc, n, NP);
     stage_tile(Xt + buf * kChunk * pitch_v, pitch_v, xs + (int64_t)tb * p.ld_xbc, p.ld_xbc, n, vp);
     cp_async_commit();
   };
@@ -259,6 +273,7 @@ ssd_chunk_kernel(SsdArgs p) {
   };
   stage(t0, 0);
   if (warp == 0) { fetch_dt(t0); sum_decays(t0, 0); }
+  float total = 0.0f;     // log2 of the decay so far
   int buf = 0, turn = 0;  // the warp whose turn it is prepares the next chunk's decays
   for (int tb = t0; tb < t1; tb += kChunk, buf ^= 1, turn = turn + 1 < n_warps ? turn + 1 : 0) {
     const int n = min(kChunk, t1 - tb);
@@ -271,7 +286,7 @@ ssd_chunk_kernel(SsdArgs p) {
     }
     const uint32_t B_a = smem_u32(Bt + buf * kChunk * kPitchN), C_a = smem_u32(Ct + buf * kChunk * kPitchN), X_a = smem_u32(Xt + buf * kChunk * pitch_v);
     // ---- P: sixteen by sixteen blocks on and below the diagonal, dealt to the warps
-    for (int b = warp; b < 10; b += n_warps) {
+    for (int b = warp; b < 10 && PART != kStates; b += n_warps) {
       const int I = b < 4 ? 3 : b < 7 ? 2 : b < 9 ? 1 : 0, J = b - (b < 4 ? 0 : b < 7 ? 4 : b < 9 ? 7 : 9);
       float acc[2][4] = {};
 #pragma unroll
@@ -299,7 +314,7 @@ ssd_chunk_kernel(SsdArgs p) {
     // ---- outputs of this warp's eight values
     float acc[4][4] = {};
 #pragma unroll
-    for (int ks = 0; ks < NT; ++ks) {
+    for (int ks = 0; ks < NT && PART != kStates; ++ks) {
       uint32_t hi[2], lo[2];
       state_operand(S[ks], hi, lo);
 #pragma unroll
@@ -315,7 +330,7 @@ ssd_chunk_kernel(SsdArgs p) {
     frag_bt(xb[1], X_a, pitch_v, 32, v0, lane);
     const uint32_t Ph_a = smem_u32(Ph), Pl_a = smem_u32(Pl);
 #pragma unroll
-    for (int mt = 0; mt < 4; ++mt) {
+    for (int mt = 0; mt < 4 && PART != kStates; ++mt) {
       const float e0 = fast_exp2(cum[16 * mt + g]), e1 = fast_exp2(cum[16 * mt + g + 8]);
       acc[mt][0] *= e0; acc[mt][1] *= e0; acc[mt][2] *= e1; acc[mt][3] *= e1;
 #pragma unroll
@@ -335,6 +350,7 @@ ssd_chunk_kernel(SsdArgs p) {
     }
     // ---- state
     const float c_last = cum[kChunk - 1], e_last = fast_exp2(c_last);
+    total += c_last;
 #pragma unroll
     for (int m = 0; m < NT; ++m)
 #pragma unroll
@@ -359,16 +375,49 @@ ssd_chunk_kernel(SsdArgs p) {
     if (warp == turn && tb + kChunk < t1) sum_decays(tb + kChunk, buf ^ 1);
     __syncthreads();
     const int pieces_v = vp >> 3, lg_v = 31 - __clz(pieces_v);
-    for (int e = tid; e < n * pieces_v; e += blockDim.x) {
+    for (int e = tid; e < n * pieces_v && PART != kStates; e += blockDim.x) {
       const int row = e >> lg_v, piece = e & (pieces_v - 1);
       *reinterpret_cast<uint4*>(ys + (int64_t)(tb + row) * p.ld_y + piece * 8) =
           *reinterpret_cast<const uint4*>(Xt + buf * kChunk * pitch_v + row * pitch_v + piece * 16);
     }
   }
+  if (PART == kOutputs && t1 < end) return;
+  float* to = PART == kStates ? segs.state + ((size_t)(entry + 1) * p.heads + head) * NP * vp : st;
+  if (PART == kStates && tid == 0) segs.decay[(size_t)(entry + 1) * p.heads + head] = total;
 #pragma unroll
   for (int m = 0; m < NT; ++m) {
-    *reinterpret_cast<float2*>(st + (size_t)(16 * m + g) * vp + v0 + 2 * t) = make_float2(S[m][0], S[m][1]);
-    *reinterpret_cast<float2*>(st + (size_t)(16 * m + g + 8) * vp + v0 + 2 * t) = make_float2(S[m][2], S[m][3]);
+    *reinterpret_cast<float2*>(to + (size_t)(16 * m + g) * vp + v0 + 2 * t) = make_float2(S[m][0], S[m][1]);
+    *reinterpret_cast<float2*>(to + (size_t)(16 * m + g + 8) * vp + v0 + 2 * t) = make_float2(S[m][2], S[m][3]);
+  }
+}
+
+// The states that the segments of a sequence start with: a thread owns four values of one head
+__global__ void __launch_bounds__(256)
+ssd_scan_kernel(SsdArgs p, Segments segs) {
+  lg::pdl_prologue();
+  const int seq = blockIdx.y, len = p.cu[seq + 1] - p.cu[seq], n = (len + kSegment - 1) / kSegment, per_head = p.np * p.vp / 4;
+  const int64_t width = (int64_t)p.heads * per_head, at = (int64_t)blockIdx.x * 256 + threadIdx.x;
+  if (at >= width || n == 0) return;
+  const int head = (int)(at / per_head);
+  float4* entry = reinterpret_cast<float4*>(segs.state) + first_entry(p.cu, seq) * width + at;
+  const float* decay = segs.decay + (size_t)first_entry(p.cu, seq) * p.heads + head;
+  float4 S = p.fresh[seq] ? make_float4(0.f, 0.f, 0.f, 0.f) : reinterpret_cast<const float4*>(p.state)[p.state_slots[seq] * width + at];
+  entry[0] = S;
+  constexpr int kBatch = 4;   // segments in flight
+  for (int g0 = 1; g0 < n; g0 += kBatch) {
+    float4 own[kBatch];
+    float e[kBatch];
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const bool in = g0 + i < n;
+      own[i] = in ? entry[(g0 + i) * width] : make_float4(0.f, 0.f, 0.f, 0.f);
+      e[i] = in ? exp2f(decay[(size_t)(g0 + i) * p.heads]) : 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      S = make_float4(fmaf(e[i], S.x, own[i].x), fmaf(e[i], S.y, own[i].y), fmaf(e[i], S.z, own[i].z), fmaf(e[i], S.w, own[i].w));
+      if (g0 + i < n) entry[(g0 + i) * width] = S;
+    }
   }
 }
 
@@ -582,20 +631,43 @@ uint32_t logismos_launch_ssd_conv(const lg_ssd_t* a, const void* seq_ids_i32, in
   return single ? launch_conv<__nv_bfloat16, 1>(p, ids, row0, rows, s) : launch_conv<__nv_bfloat16, 16>(p, ids, row0, rows, s);
 }
 
-uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* a, int32_t n_seqs, void* stream) {
+int32_t logismos_ssd_segments(int32_t rows, int32_t n_seqs, int32_t longest, int32_t heads) {
+  // Measured (us, whole / segments; 64 x 128 states): 4 prompts of 1024, 8 / 16 / 32 heads 71 / 40, 71 / 60, 73 / 107; one of 16384, 8 /
+  // 32 heads 1075 / 126, 1077 / 415. Whole sequences take 4.4 us per 64 tokens of the longest, segments 0.052 us per 64 tokens and head.
+  return longest > 2 * kSegment && (int64_t)rows * heads < (int64_t)72 * longest ? rows / kSegment + n_seqs + 1 : 0;
+}
+
+size_t logismos_ssd_scratch_bytes(int32_t entries, int32_t heads, int32_t np, int32_t vp) {
+  return entries <= 0 ? 0 : (size_t)entries * heads * ((size_t)np * vp + 4) * 4;
+}
+
+uint32_t logismos_launch_ssd_chunked_bf16(const lg_ssd_t* a, int32_t n_seqs, void* stream) { return logismos_launch_ssd_segmented_bf16(a, n_seqs, 0, nullptr, 0, stream); }
+
+uint32_t logismos_launch_ssd_segmented_bf16(const lg_ssd_t* a, int32_t n_seqs, int32_t longest, void* scratch, int32_t entries, void* stream) {
   lg::LaunchScope launch_scope_;
-  if (!args_ok(a, n_seqs) || !logismos_ssd_has_chunked(a->np, a->vp) || !a->xbc || a->ld_xbc % 8 || a->ld_y % 8 || (((uintptr_t)a->xbc | (uintptr_t)a->y) & 15))
+  if (!args_ok(a, n_seqs) || !logismos_ssd_has_chunked(a->np, a->vp) || !a->xbc || a->ld_xbc % 8 || a->ld_y % 8 || (((uintptr_t)a->xbc | (uintptr_t)a->y) & 15) ||
+      (entries > 0 && (!scratch || ((uintptr_t)scratch & 15) || longest <= 0 || longest > 65535 * kSegment)))
     return lg::kInvalidValue;
   const SsdArgs p = make_args(a);
   const size_t smem = ssd_chunk_smem(a->np, a->vp);
-  auto go = [&](auto kern) -> uint32_t {
+  const bool cut = entries > 0;
+  Segments segs{(float*)scratch, (float*)scratch + (size_t)(cut ? entries : 0) * p.heads * p.np * p.vp};
+  const int per_seq = cut ? (longest + kSegment - 1) / kSegment : 1;
+  auto go = [&](auto kern, int n) -> uint32_t {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (uint32_t)e;
-    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs), dim3((unsigned)(4 * p.vp)), smem, (cudaStream_t)stream, p);
+    lg::launch(kern, dim3((unsigned)p.heads, (unsigned)n_seqs, (unsigned)n), dim3((unsigned)(4 * p.vp)), smem, (cudaStream_t)stream, p, segs);
     return lg::launch_status();
   };
-  if (p.decay) return a->np == 32 ? go(ssd_chunk_kernel<32, true>) : a->np == 64 ? go(ssd_chunk_kernel<64, true>) : go(ssd_chunk_kernel<128, true>);
-  return a->np == 32 ? go(ssd_chunk_kernel<32, false>) : a->np == 64 ? go(ssd_chunk_kernel<64, false>) : go(ssd_chunk_kernel<128, false>);
+#define LG_PART(FIXED, PART, N) (a->np == 32 ? go(ssd_chunk_kernel<32, FIXED, PART>, N) : a->np == 64 ? go(ssd_chunk_kernel<64, FIXED, PART>, N) : go(ssd_chunk_kernel<128, FIXED, PART>, N))
+  if (!cut) return p.decay ? LG_PART(true, kWhole, 1) : LG_PART(false, kWhole, 1);
+  if (per_seq > 1)
+    if (uint32_t rc = p.decay ? LG_PART(true, kStates, per_seq - 1) : LG_PART(false, kStates, per_seq - 1)) return rc;
+  const int64_t width = (int64_t)p.heads * p.np * p.vp / 4;
+  lg::launch(ssd_scan_kernel, dim3((unsigned)((width + 255) / 256), (unsigned)n_seqs), dim3(256), 0, (cudaStream_t)stream, p, segs);
+  if (uint32_t rc = lg::launch_status()) return rc;
+  return p.decay ? LG_PART(true, kOutputs, per_seq) : LG_PART(false, kOutputs, per_seq);
+#undef LG_PART
 }
 
 uint32_t logismos_launch_gated_group_norm(const void* y, int32_t ld_y, const void* z, int32_t ld_z, const void* gain_f32, void* out, int32_t ld_out,

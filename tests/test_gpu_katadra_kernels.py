@@ -270,6 +270,10 @@ def run_ssd(form, heads, v, groups, n, taps, lens, seed, fp32=False, a_hi=1.0):
     check(lib.logismos_launch_ssd_conv(C.byref(a), P(seq), 0, T, int(single), int(fp32), stream()), "conv")
     if form == "chunked":
         check(lib.logismos_launch_ssd_chunked_bf16(C.byref(a), k, stream()), "chunked")
+    elif form == "segments":
+        entries = T // 256 + k + 1
+        scr = torch.full((lib.logismos_ssd_scratch_bytes(entries, heads, N, V) // 4,), float("nan"), device=DEV)
+        check(lib.logismos_launch_ssd_segmented_bf16(C.byref(a), k, max(lens), P(scr), entries, stream()), "segments")
     else:
         check(lib.logismos_launch_ssd_step(C.byref(a), k, int(fp32), stream()), "step")
     torch.cuda.synchronize()
@@ -282,6 +286,15 @@ def run_ssd(form, heads, v, groups, n, taps, lens, seed, fp32=False, a_hi=1.0):
             assert np.allclose(cstate[slots[s], 1 - int(phase[s])].cpu().numpy(), chan(ends[s][1]), rtol=0, atol=1e-6), s
         assert np.array_equal(cstate[slots[-1], int(phase[-1])].cpu().numpy(), chan(past).astype(np.float32))
     return got[..., :v], np.concatenate(want), st[:, :, :n, :v], np.stack([e[0] for e in ends])
+
+
+@pytest.mark.parametrize("heads,v,groups,n,taps", [(6, 12, 2, 20, 4), (4, 64, 1, 128, 4), (2, 16, 1, 30, 2)])
+def test_state_space_recurrence_in_segments(heads, v, groups, n, taps):
+    """Decays that depend on the data, over segments that run side by side."""
+    for lens in ([1200], [256, 257, 3, 600]):
+        o, want, st, ends = run_ssd("segments", heads, v, groups, n, taps, lens, 7)
+        close(o, want, 4e-3)
+        close(st, ends, 3e-3)
 
 
 @pytest.mark.parametrize("heads,v,groups,n,taps", [(6, 12, 2, 20, 4), (4, 64, 1, 128, 4), (2, 100, 2, 60, 1), (3, 20, 3, 100, 8), (2, 16, 1, 30, 2), (2, 140, 1, 70, 3), (1, 40, 1, 200, 3)])

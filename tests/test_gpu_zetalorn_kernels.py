@@ -423,6 +423,10 @@ def run_linear(form, heads, dk, dv, lens, seed, fp32=False, decays=None):
                 xbc=A(rows) + 8 * (4 if fp32 else 2), ld_xbc=rows.shape[1], decay=A(parts))
         if form == "chunked":
             check(lib.logismos_launch_ssd_chunked_bf16(C.byref(a), n, stream()), "chunked")
+        elif form == "segments":
+            entries = T // 256 + n + 1
+            scr = torch.full((lib.logismos_ssd_scratch_bytes(entries, heads, dp, wp) // 4,), float("nan"), device=DEV)
+            check(lib.logismos_launch_ssd_segmented_bf16(C.byref(a), n, max(ll), P(scr), entries, stream()), "segments")
         else:
             check(lib.logismos_launch_ssd_step(C.byref(a), n, int(fp32), stream()), "step")
         want = np.zeros((T, heads, dv))
@@ -446,6 +450,17 @@ def test_linear_attention_with_a_fixed_decay(heads, dk, dv, lens):
         o, want, st, S = run_linear(form, heads, dk, dv, lens, 7, fp32)
         close(o, want, tol)
         close(st, S, 1e-4 if form == "chunked" else 1e-5)
+
+
+@pytest.mark.parametrize("heads,dk,dv", [(3, 24, 40), (1, 64, 128), (2, 128, 16)])
+@pytest.mark.parametrize("lens", [[1500], [256, 257, 3, 255, 700], [511, 512, 513]])
+def test_segments_of_long_prompts(heads, dk, dv, lens):
+    for decays in (None, [0.9999] * heads, [0.0] * heads):
+        o, want, st, S = run_linear("segments", heads, dk, dv, lens, 3, decays=decays)
+        close(o, want, 4e-3)
+        close(st, S, 1e-4)
+    assert lib.logismos_ssd_segments(1500, 1, 1500, 8) == 1500 // 256 + 2
+    assert lib.logismos_ssd_segments(1500, 3, 512, 8) == 0 and lib.logismos_ssd_segments(4096, 4, 1024, 32) == 0 and lib.logismos_ssd_segments(16384, 1, 16384, 32) > 0
 
 
 def test_linear_attention_at_the_ends_of_the_decay_and_in_large_heads():

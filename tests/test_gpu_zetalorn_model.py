@@ -253,6 +253,21 @@ def test_far_tokens_of_the_recurrence(dtype):
     h.close()
 
 
+@BOTH
+def test_long_prompts_whose_recurrences_run_in_segments(dtype):
+    """One long prompt beside short ones and decoded tokens, then portions that end inside a segment."""
+    cfg = config(90, 48, [parallel(left(2, 1, 16, 16, 40, 8, rotation(8)), right(24, 20, (0.9, 0.999))), attention(2, 1, 16, 24, 100, rotation(8), 0.3)])
+    h = Harness(cfg, R.random_weights(cfg, 23), dtype, pool_tokens=4096, step_tokens=2600)
+    rng = np.random.default_rng(5)
+    T = lambda n: tokens(rng, cfg, n)
+    h.run([("a", T(1)), ("b", T(40))])
+    h.run([("long", T(1100)), ("a", T(1)), ("b", T(2)), ("c", T(700))])
+    h.run([("c", T(600)), ("long", T(1)), ("a", T(3))])
+    h.run([("long", T(1030)), ("c", T(1))])
+    h.run([("long", T(1)), ("c", T(1)), ("a", T(1)), ("b", T(1))])
+    h.close()
+
+
 def test_passes_keep_their_caches_and_states_apart():
     """A model whose passes are written out as layers with equal tensors, the embedding and the steps added by hand."""
     base = [parallel(left(2, 1, 16, 16, 9, 2, rotation(8)), right(16, 16, (0.9, 0.8)), moe(4, 2, 16, 2, 1)), attention(2, 1, 8, 16, 6, rotation(8), 0.2)]
