@@ -374,47 +374,73 @@ LG_DEVINL float bounded_block(uint32_t t_s, const ScoreExt& ext, const float* wi
   return sum;
 }
 
-// ---- softmax of a block whose 128 scores per row are held in registers: one read of TMEM, one wait ---------------------------
-LG_DEVINL void load_scores(uint32_t t_s, uint32_t (&r)[4][32]) {
-#pragma unroll
-  for (int w = 0; w < 4; ++w) tc_ld32(t_s + 32 * w, r[w]);
-  tc_wait_ld();
-}
+// ---- softmax of a block of 128 keys -----------------------------------------------------------------------------------------
 LG_DEVINL uint32_t bits_below(int n) { return n >= 32 ? 0xffffffffu : n <= 0 ? 0u : (1u << n) - 1u; }
 // scores whose bit is not set become -inf
 LG_DEVINL void hide(uint32_t (&r)[32], uint32_t seen) {
 #pragma unroll
   for (int i = 0; i < 32; ++i) r[i] = seen & (1u << i) ? r[i] : 0xff800000u;
 }
-// The running maximum m (log2 units) moves when it would grow by more than 2^8, so that what it scales is rescaled by alpha far less
-// often; P, rounded, takes the place of S. Returns the row's sum. Independent chains: a scheduler has one or two warps to issue from.
-LG_DEVINL float softmax_block(uint32_t t_s, const uint32_t (&r)[4][32], float sl2, float& m, float& alpha) {
-  float mx[4];
+// The largest score of 64 keys; independent chains: a scheduler has one or two warps to issue from
+LG_DEVINL float max64(const uint32_t (&a)[32], const uint32_t (&b)[32]) {
+  float x = fmaxf(__uint_as_float(a[0]), __uint_as_float(a[1])), y = fmaxf(__uint_as_float(b[0]), __uint_as_float(b[1]));
 #pragma unroll
-  for (int w = 0; w < 4; ++w) mx[w] = __uint_as_float(r[w][0]);
-#pragma unroll
-  for (int i = 1; i < 32; ++i)
-#pragma unroll
-    for (int w = 0; w < 4; ++w) mx[w] = fmaxf(mx[w], __uint_as_float(r[w][i]));
-  const float cand = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * sl2;
+  for (int i = 2; i < 32; i += 2) {
+    x = fmaxf(x, fmaxf(__uint_as_float(a[i]), __uint_as_float(a[i + 1])));
+    y = fmaxf(y, fmaxf(__uint_as_float(b[i]), __uint_as_float(b[i + 1])));
+  }
+  return fmaxf(x, y);
+}
+// The running maximum m (log2 units) moves when it would grow by more than 2^8, so that P stays below 256 (exact enough in bf16,
+// summed in fp32) and what it scales is rescaled by alpha far less often
+LG_DEVINL void move_max(float mx, float sl2, float& m, float& alpha) {
+  const float cand = mx * sl2;
   alpha = 1.0f;
   if (cand > m + 8.0f) { alpha = fast_exp2(m - cand); m = cand; }
+}
+// P of 64 keys, rounded, over S: columns [32 h, 32 h + 32) hold keys [64 h, 64 h + 64). Returns the sum.
+LG_DEVINL float probs64(uint32_t t_p, const uint32_t (&a)[32], const uint32_t (&b)[32], float sl2, float m) {
   float sum[4] = {0.f, 0.f, 0.f, 0.f};
+  uint32_t v[32];
 #pragma unroll
-  for (int h = 0; h < 2; ++h) {  // columns [32 h, 32 h + 32) hold keys [64 h, 64 h + 64)
-    uint32_t v[32];
-#pragma unroll
-    for (int i = 0; i < 32; i += 2)
-#pragma unroll
-      for (int w = 0; w < 2; ++w) {
-        const float a = fast_exp2(fmaf(__uint_as_float(r[2 * h + w][i]), sl2, -m)), b = fast_exp2(fmaf(__uint_as_float(r[2 * h + w][i + 1]), sl2, -m));
-        sum[w] += a;
-        sum[2 + w] += b;
-        v[16 * w + (i >> 1)] = pack_bf16x2(a, b);
-      }
-    tc_st32(t_s + 32 * h, v);
+  for (int i = 0; i < 32; i += 2) {
+    const float a0 = fast_exp2(fmaf(__uint_as_float(a[i]), sl2, -m)), a1 = fast_exp2(fmaf(__uint_as_float(a[i + 1]), sl2, -m));
+    const float b0 = fast_exp2(fmaf(__uint_as_float(b[i]), sl2, -m)), b1 = fast_exp2(fmaf(__uint_as_float(b[i + 1]), sl2, -m));
+    sum[0] += a0; sum[1] += a1; sum[2] += b0; sum[3] += b1;
+    v[i >> 1] = pack_bf16x2(a0, a1);
+    v[16 + (i >> 1)] = pack_bf16x2(b0, b1);
   }
+  tc_st32(t_p, v);
   return (sum[0] + sum[1]) + (sum[2] + sum[3]);
+}
+// The keys [lo, lim) and [0, keep) of a block count (all: every one does). S is read twice, 64 keys at a time, in loops that stay
+// rolled: the CTAs of a short launch start beside those of the launch before it (118 against 168 registers), and the code is small.
+LG_DEVINL float softmax_block(uint32_t t_s, int lim, int lo, int keep, bool all, float sl2, float& m, float& alpha) {
+  auto read = [&](int h, uint32_t (&a)[32], uint32_t (&b)[32]) {
+    tc_ld32(t_s + 64 * h, a);
+    tc_ld32(t_s + 64 * h + 32, b);
+    tc_wait_ld();
+    if (!all) {
+      const int c = 64 * h;
+      hide(a, bits_below(lim - c) & (~bits_below(lo - c) | bits_below(keep - c)));
+      hide(b, bits_below(lim - c - 32) & (~bits_below(lo - c - 32) | bits_below(keep - c - 32)));
+    }
+  };
+  float mx = -1e30f, sum = 0.0f;
+#pragma unroll 1
+  for (int h = 0; h < 2; ++h) {
+    uint32_t a[32], b[32];
+    read(h, a, b);
+    mx = fmaxf(mx, max64(a, b));
+  }
+  move_max(mx, sl2, m, alpha);
+#pragma unroll 1
+  for (int h = 0; h < 2; ++h) {  // P of the first half replaces scores that both passes have read
+    uint32_t a[32], b[32];
+    read(h, a, b);
+    sum += probs64(t_s + 32 * h, a, b, sl2, m);
+  }
+  return sum;
 }
 
 template <bool CAUSAL, int HD, int SCORE = kPlain>
@@ -605,13 +631,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       }
       float alpha = 1.0f, sum = 0.0f;
       if constexpr (!BIASED) {
-        uint32_t r[4][32];
-        load_scores(t_s, r);
-        if (!__all_sync(0xffffffffu, full)) {
-#pragma unroll
-          for (int w = 0; w < 4; ++w) hide(r[w], bits_below(lim - 32 * w) & (SCORE == kWindowed ? ~bits_below(lo - 32 * w) | bits_below(keep - 32 * w) : 0xffffffffu));
-        }
-        sum = softmax_block(t_s, r, sl2, m, alpha);
+        sum = softmax_block(t_s, lim, lo, keep, __all_sync(0xffffffffu, full), sl2, m, alpha);
       } else {
         float mx = -1e30f;
 #pragma unroll
@@ -870,14 +890,8 @@ diff_attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       if (!mbar_wait_warp(s_full + 8 * m, (uint32_t)j & 1u, abort_flag)) { ok = false; break; }
       tc_fence_after();
       const int base = (j + skip) * 128 + gap, lim = min(kv_len, at + 1) - base, lo = seen_from - base;  // keys [lo, lim) of the block
-      uint32_t r[4][32];
-      load_scores(t_s, r);
-      if (!__all_sync(0xffffffffu, lim >= 128 && lo <= 0)) {
-#pragma unroll
-        for (int w = 0; w < 4; ++w) hide(r[w], bits_below(lim - 32 * w) & ~bits_below(lo - 32 * w));
-      }
       float alpha;
-      const float sum = softmax_block(t_s, r, sl2, mx_run, alpha);
+      const float sum = softmax_block(t_s, lim, lo, 0, __all_sync(0xffffffffu, lim >= 128 && lo <= 0), sl2, mx_run, alpha);
       l = l * alpha + sum;
       if (j > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
 #pragma unroll
