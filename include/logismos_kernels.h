@@ -937,7 +937,7 @@ uint32_t logismos_launch_rotary_heads(void* q, int32_t ld, const void* positions
  * f32 [rows, ld_gate]: head h of a row is multiplied by the sigmoid of its column h (NULL: none). Scores are scaled by scale
  * (> 0).
  * pool > 0: a query also sees the blocks of `pool` positions, as a key and a value each (block b: b pool .. b pool + pool - 1)
- * that lies wholly before it. They are rows of k_mean and v_mean [n_pool_blocks][ceil(16 / pool)], as wide as the cache's:
+ * that lie wholly before it. They are rows of k_mean and v_mean [n_pool_blocks][ceil(16 / pool)], as wide as the cache's:
  * block b is kept with the cache block that holds its last token, the blocks ending there one after the other
  * (logismos_launch_pool_blocks). */
 typedef struct lg_window {
